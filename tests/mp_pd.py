@@ -31,7 +31,7 @@ def main():
                      tie_word_embeddings=False, max_position_embeddings=4096)
     model = create_model(args, torch.bfloat16, dev, single())
     model.init_random(seed=7)                      # the same weights in both processes
-    kv_bytes = ModelRunner.kv_bytes_per_block(args, 2, 16, torch.bfloat16) * NUM_BLOCKS
+    kv_bytes = ModelRunner.kv_bytes_per_block(model, args, 16, torch.bfloat16) * NUM_BLOCKS
     link = PDLink(ps.job_group, dev, kv_bytes)
     cfg = EngineConfig(model="t", device=str(dev), dtype="bfloat16", block_size=16, num_blocks=NUM_BLOCKS,
                        max_seqs_per_batch=8, max_tokens_per_batch=256, max_model_len=1024, enable_graph=True,

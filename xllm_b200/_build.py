@@ -44,6 +44,9 @@ NVCC_FLAGS = [
     "--expt-relaxed-constexpr",
     "-I", str(CSRC),
 ]
+# Sources built without --use_fast_math: their exponentials feed recurrences (errors of a decay multiply up over a
+# sequence) or serve the fp32 execution type.
+PRECISE_SOURCES = {"linear_attn", "residual", "rope_norm_kv", "attn_generic"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread",
              "-I", str(CSRC / "runtime"), "-I", str(CSRC / "frontend"), "-I", str(CSRC / "server"),
              "-Wall", "-Wno-sign-compare", "-I", str(CSRC), "-I", "/usr/local/cuda/include"]
@@ -126,7 +129,7 @@ def _build_kernels(force, verbose, ptxas_info) -> Path:
     for s in srcs:
         o = OBJDIR / (s.stem + ".o")
         stamp = OBJDIR / (s.stem + ".sha")
-        want = _sha([s], hdr_hash)
+        want = _sha([s], hdr_hash + ("precise" if s.stem in PRECISE_SOURCES else ""))
         objs.append(o)
         if force or not o.exists() or not stamp.exists() or stamp.read_text() != want:
             todo.append((s, o, stamp, want))
@@ -135,7 +138,8 @@ def _build_kernels(force, verbose, ptxas_info) -> Path:
 
     def one(item):
         s, o, stamp, want = item
-        _run([NVCC, *flags, "-c", s, "-o", o], verbose or ptxas_info)
+        own = [f for f in flags if f != "--use_fast_math"] if s.stem in PRECISE_SOURCES else flags
+        _run([NVCC, *own, "-c", s, "-o", o], verbose or ptxas_info)
         stamp.write_text(want)
 
     if todo:

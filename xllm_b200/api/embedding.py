@@ -10,6 +10,7 @@ from typing import List
 
 import torch
 
+from ..engine.model_runner import ModelRunner
 from ..models.layers import AttentionMetadata
 
 
@@ -20,17 +21,18 @@ def hidden_states(engine, ids: List[int]) -> torch.Tensor:
     bs = engine.cfg.block_size
     T = len(ids)
     n_blocks = (T + bs - 1) // bs
-    nkv, d = model.num_kv_heads_local, model.head_dim
-    kv = [(torch.zeros(n_blocks + 1, nkv, bs, d, dtype=engine.dtype, device=dev),
-           torch.zeros(n_blocks + 1, nkv, bs, d, dtype=engine.dtype, device=dev))
-          for _ in range(engine.args.num_hidden_layers)]
+    kv = [(None, None) if g is None else
+          tuple(torch.zeros(n_blocks + 1, g[1], bs, g[2], dtype=engine.dtype, device=dev) for _ in range(2))
+          for g in ModelRunner.kv_layout(model, engine.args)]
     meta = AttentionMetadata(
         n_decode=0, n_prefill=1, slots=torch.arange(bs, bs + T, dtype=torch.int32, device=dev),
         block_table=torch.arange(1, n_blocks + 1, dtype=torch.int32, device=dev)[None],
         kv_lens=torch.tensor([T], dtype=torch.int32, device=dev),
         cu_q=torch.tensor([0, T], dtype=torch.int32, device=dev), max_q_len=T, max_kv_len=T)
     if getattr(model, "needs_state", False):        # linear-attention layers: a scratch state slot, reset for this pass
-        meta.state_slots = torch.tensor([model.state.n_slots - 1], dtype=torch.long, device=dev)
+        st = model.state
+        meta.state_slots = torch.tensor([getattr(st, "scratch_slot", st.n_slots - 1)], device=dev,
+                                        dtype=torch.int32 if getattr(model, "state_on_device", False) else torch.long)
         meta.state_fresh, meta.seq_bounds = [True], [(0, T)]
     return model.forward(torch.tensor(ids, dtype=torch.int64, device=dev), torch.arange(T, device=dev), meta, kv)
 
@@ -54,23 +56,9 @@ def rerank_scores(engine, query_ids: List[int], doc_ids: List[List[int]]) -> Lis
 
 @torch.no_grad()
 def embed_token_lists(engine, token_lists: List[List[int]], normalize: bool = True) -> List[List[float]]:
-    model, dev = engine.model, engine.device
-    bs = engine.cfg.block_size
     out = []
     for ids in token_lists:
-        T = len(ids)
-        n_blocks = (T + bs - 1) // bs
-        nkv, d = model.num_kv_heads_local, model.head_dim
-        # a private scratch cache: embedding requests never touch the serving KV pool
-        kv = [(torch.zeros(n_blocks + 1, nkv, bs, d, dtype=engine.dtype, device=dev),
-               torch.zeros(n_blocks + 1, nkv, bs, d, dtype=engine.dtype, device=dev))
-              for _ in range(engine.args.num_hidden_layers)]
-        meta = AttentionMetadata(
-            n_decode=0, n_prefill=1, slots=torch.arange(bs, bs + T, dtype=torch.int32, device=dev),
-            block_table=torch.arange(1, n_blocks + 1, dtype=torch.int32, device=dev)[None],
-            kv_lens=torch.tensor([T], dtype=torch.int32, device=dev),
-            cu_q=torch.tensor([0, T], dtype=torch.int32, device=dev), max_q_len=T, max_kv_len=T)
-        h = model.forward(torch.tensor(ids, dtype=torch.int64, device=dev), torch.arange(T, device=dev), meta, kv)
+        h = hidden_states(engine, ids)     # a private scratch cache: embedding requests never touch the serving KV pool
         v = h[-1].float()
         if normalize:
             v = v / v.norm().clamp_min(1e-12)

@@ -422,6 +422,7 @@ PYBIND11_MODULE(_rt, m) {
       .def("held_blocks", &Scheduler::held_blocks)
       .def("release_held", &Scheduler::release_held)
       .def("schedule", &Scheduler::schedule, py::call_guard<py::gil_scoped_release>())
+      .def("schedule_replay", &Scheduler::schedule_replay, py::arg("ids"), py::arg("tokens"), py::arg("want"))
       .def("process_output",
            [](Scheduler& s, int64_t batch_id, py::array_t<int64_t, py::array::c_style | py::array::forcecast> toks,
               py::object logprobs) {

@@ -308,6 +308,7 @@ class Scheduler {
       if (s->finished()) continue;
       remove_from_queues(s.get());
       finish_seq(s.get(), FinishReason::ABORT);
+      preempted_ids_.push_back(s->seq_id);   // its per-sequence state is free (one event speaks for all samples)
     }
     pending_events_.push_back(make_event(r->seqs[0].get(), -1, 0.f, false));
     pending_events_.back().request_finished = true;
@@ -333,6 +334,93 @@ class Scheduler {
       }
     }
     return out;
+  }
+
+  // Replay of recorded requests: the caller, not the queues, decides which tokens a step brings.  Entry i appends
+  // tokens[i] to request ids[i] (admitted at its first entry) and all entries form one batch: a single token behind
+  // an existing context is a decode row, anything else a prompt chunk.  `want[i]` are the places among tokens[i]
+  // whose logits the caller asks for; they become the sample rows of the batch, in batch order (a batch of decode
+  // rows only samples every row).  Blocks come from the same pool as those of scheduled requests; the step ends
+  // with process_output(batch_id, {}, 0) and a request with abort_request().
+  Batch schedule_replay(const std::vector<std::string>& ids, const std::vector<std::vector<int32_t>>& tokens,
+                        const std::vector<std::vector<int32_t>>& want) {
+    if (ids.size() != tokens.size() || ids.size() != want.size()) throw std::invalid_argument("replay: ragged entries");
+    int64_t total = 0;
+    for (size_t i = 0; i < ids.size(); ++i) {
+      if (tokens[i].empty()) throw std::invalid_argument("replay: an entry without tokens");
+      for (size_t j = 0; j < i; ++j)
+        if (ids[j] == ids[i]) throw std::invalid_argument("replay: a request twice in one step");
+      for (int32_t w : want[i])
+        if (w < 0 || w >= (int32_t)tokens[i].size()) throw std::invalid_argument("replay: a wanted place out of range");
+      total += (int64_t)tokens[i].size();
+    }
+    if (total > cfg_.max_tokens_per_batch || (int32_t)ids.size() > cfg_.max_seqs_per_batch)
+      throw std::runtime_error("replay: the step is larger than a batch may be");
+    std::vector<Pick> decodes, prefills;
+    std::vector<const std::vector<int32_t>*> want_of_pick[2];
+    for (size_t i = 0; i < ids.size(); ++i) {
+      Sequence* s = nullptr;
+      auto it = requests_.find(ids[i]);
+      if (it == requests_.end()) {
+        if (cfg_.max_running_seqs > 0 && (int32_t)running_.size() >= cfg_.max_running_seqs)
+          throw std::runtime_error("replay: more live requests than the engine holds");
+        auto req = std::make_unique<Request>();
+        req->request_id = ids[i];
+        req->arrival_time = now_seconds();
+        auto seq = std::make_unique<Sequence>();
+        seq->seq_id = next_seq_id_++;
+        seq->request = req.get();
+        seq->stage = SeqStage::PREFILL;
+        s = seq.get();
+        req->seqs.push_back(std::move(seq));
+        requests_.emplace(ids[i], std::move(req));
+        running_.push_back(s);
+      } else {
+        s = it->second->seqs[0].get();
+      }
+      s->tokens.insert(s->tokens.end(), tokens[i].begin(), tokens[i].end());
+      s->num_prompt_tokens = s->num_tokens();
+      if (!ensure_blocks(s, s->num_tokens())) throw std::runtime_error("replay: the KV pool is too small for the live requests");
+      const bool decode = tokens[i].size() == 1 && s->kv_computed > 0;
+      s->stage = decode ? SeqStage::DECODE : SeqStage::PREFILL;
+      (decode ? decodes : prefills).push_back({s, (int32_t)tokens[i].size(), decode});
+      want_of_pick[decode ? 0 : 1].push_back(&want[i]);
+    }
+    Batch b = build_batch(0, decodes, prefills);
+    for (Sequence* s : b.seqs) s->pending_samples = 0;      // nothing is sampled: the next tokens are given
+    std::vector<const std::vector<int32_t>*> w = want_of_pick[0];
+    w.insert(w.end(), want_of_pick[1].begin(), want_of_pick[1].end());
+    b.sample_rows.clear();
+    b.sample_seq.clear();
+    for (int32_t i = 0; i < b.n_seqs(); ++i) {
+      if (b.n_prefill == 0) {
+        b.sample_rows.push_back(i);
+        b.sample_seq.push_back(i);
+        continue;
+      }
+      for (int32_t at : *w[i]) {
+        b.sample_rows.push_back(b.cu_q[i] + at);
+        b.sample_seq.push_back(i);
+      }
+    }
+    const size_t ns = b.sample_rows.size();
+    b.temperature.assign(ns, 0.f);
+    b.top_p.assign(ns, 1.f);
+    b.top_k.assign(ns, -1);
+    b.freq_pen.assign(ns, 0.f);
+    b.pres_pen.assign(ns, 0.f);
+    b.rep_pen.assign(ns, 1.f);
+    b.seeds.assign(ns, 0);
+    b.sample_offsets.assign(ns, 0);
+    if (!b.empty()) {
+      b.batch_id = next_batch_id_++;
+      InFlight f;
+      f.seqs = b.seqs;
+      f.q_lens = b.q_lens;
+      f.n_decode = b.n_decode;
+      in_flight_batches_.emplace(b.batch_id, std::move(f));
+    }
+    return b;
   }
 
   // next_tokens: one id per sample row of the batch (in order).  logprobs may be null.
@@ -428,8 +516,8 @@ class Scheduler {
     it->second.top_lps.assign(lps, lps + n_rows * n);
   }
 
-  // Sequence ids preempted since the last call (their KV - and any per-sequence state - is gone and
-  // will be rebuilt from position 0).
+  // Sequence ids preempted or aborted since the last call (their KV - and any per-sequence state - is gone; a
+  // preempted sequence rebuilds it from position 0).
   std::vector<int64_t> take_preempted() {
     std::vector<int64_t> out;
     out.swap(preempted_ids_);

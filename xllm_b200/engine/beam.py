@@ -66,6 +66,8 @@ def beam_search(engine, prompt_token_ids, beam_width: int = 4, max_tokens: int =
                 eos_token_id: Optional[int] = None, ignore_eos: bool = False, num_return: Optional[int] = None
                 ) -> List[BeamOutput]:
     runner = engine.runner
+    if getattr(runner.model, "needs_state", False):
+        raise ValueError("beam search forks KV block tables; models with recurrent per-sequence state are not supported")
     model, kv, dev = runner.model, runner.kv_caches, runner.device
     bs = engine.cfg.block_size
     eos = engine.args.eos_token_id if eos_token_id is None else eos_token_id

@@ -57,6 +57,8 @@ class PDCoordinator:
 
     def __init__(self, prefill_engine, decode_engine, transfer=None):
         self.p, self.d = prefill_engine, decode_engine
+        if getattr(self.p.model, "needs_state", False):
+            raise ValueError("a disaggregated pair hands over KV blocks; recurrent per-sequence state does not travel with them")
         assert self.p.cfg.block_size == self.d.cfg.block_size, "P and D must use the same KV block size"
         self.transfer = transfer or copy_kv_blocks
         self.params: Dict[str, dict] = {}

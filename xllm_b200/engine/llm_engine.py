@@ -69,6 +69,7 @@ class EngineConfig:
     fp8_execution: Optional[bool] = None  # block-scaled fp8 checkpoints: None / True = run the fp8 GEMMs, False = dequantise at load
     min_prefill_tokens: int = 0         # mixing policies: hold prompt chunks back until this many prompt tokens are pending
     max_prefill_wait_steps: int = 8     # ... or this many steps have passed
+    max_sample_rows: int = 0            # rows of a step whose logits may be asked for at once (replay); 0: one per sequence
     max_running_seqs: int = 0           # cap on sequences holding KV / state at once; 0: no cap (state models: max_seqs_per_batch + 1)
     scheduler_type: str = "continuous"  # "continuous" | "zero_eviction" (never preempts: admits by simulation) | "fixed_steps" (waves)
     # latency-aware budgets: profile the model at start-up and cap the tokens of a step so that a step
@@ -117,6 +118,9 @@ class LLMEngine:
             self.args = load_model_args(cfg.model)
         else:
             self.args = preset(cfg.model)
+        if self.args.extra.get("unbounded_positions") and cfg.max_model_len > self.args.max_position_embeddings:
+            import dataclasses                          # the rotary table is as long as the longest sequence asked for
+            self.args = dataclasses.replace(self.args, max_position_embeddings=int(cfg.max_model_len))
         if cfg.mla_latent_cache and self.args.kv_lora_rank:
             import dataclasses
             self.args = dataclasses.replace(self.args, mla_latent_cache=True)
@@ -170,10 +174,11 @@ class LLMEngine:
         # ---- KV capacity
         max_len = cfg.max_model_len or min(self.args.max_position_embeddings, 32768)
         self.max_model_len = max_len
-        nkv = self.model.num_kv_heads_local
-        per_block = ModelRunner.kv_bytes_per_block(self.args, nkv, cfg.block_size, self.dtype,
-                                                   head_dim=getattr(self.model, "head_dim", None),
-                                                   planes=int(getattr(self.model, "kv_planes", 2)))
+        per_block = ModelRunner.kv_bytes_per_block(self.model, self.args, cfg.block_size, self.dtype)
+        if getattr(self.model, "needs_state", False):
+            # one state slot per sequence that can hold KV at the same time; the scheduler admits no
+            # more than that (max_running_seqs below), so a slot is always free when one is needed
+            self.state_slots = cfg.max_running_seqs or (cfg.max_seqs_per_batch + 1)
         num_blocks = cfg.num_blocks or self._estimate_blocks(per_block)
         if self.ps.world_size > 1 and self.ps.tp_size > 1:
             # every tensor-parallel rank runs the same scheduler: they must agree on the size of the
@@ -197,16 +202,17 @@ class LLMEngine:
         self.runner = ModelRunner(self.model, cfg.block_size, num_blocks, cfg.max_seqs_per_batch,
                                   cfg.max_tokens_per_batch, max_len, self.device, self.dtype,
                                   enable_graph=cfg.enable_graph and bool(getattr(self.model, "supports_graph", True)),
-                                  graph_buckets=cfg.graph_buckets, kv_allocator=kv_allocator)
+                                  graph_buckets=cfg.graph_buckets, kv_allocator=kv_allocator,
+                                  max_sample_rows=cfg.max_sample_rows)
         self.runner.overlap = cfg.enable_schedule_overlap
         if getattr(self.model, "needs_index_cache", False):
             self.model.alloc_index_cache(num_blocks, cfg.block_size)
         if getattr(self.model, "needs_state", False):
-            # one state slot per sequence that can hold KV at the same time; the scheduler admits no
-            # more than that (max_running_seqs below), so a slot is always free when one is needed
-            self.state_slots = cfg.max_running_seqs or (cfg.max_seqs_per_batch + 1)
             self.model.alloc_state(self.state_slots)
-            self.runner.meta_hook = self._state_hook
+            if getattr(self.model, "state_on_device", False):
+                self.runner.state_slots = self._slots_of
+            else:
+                self.runner.meta_hook = self._state_hook
         # ---- scheduler
         sc = rt.SchedulerConfig()
         sc.max_tokens_per_batch = cfg.max_tokens_per_batch
@@ -244,8 +250,8 @@ class LLMEngine:
         self.mm = {}                 # request id -> MMInput of multimodal requests
         self.host_tier = None
         if cfg.host_kv_blocks <= 0 and cfg.host_blocks_factor > 0:
-            cfg.host_kv_blocks = max(1, int(cfg.host_blocks_factor * self.runner.kv_caches[0][0].shape[0]))
-        if cfg.host_kv_blocks > 0 and cfg.enable_prefix_cache:
+            cfg.host_kv_blocks = max(1, int(cfg.host_blocks_factor * num_blocks))
+        if cfg.host_kv_blocks > 0 and sc.enable_prefix_cache:
             from .host_tier import HostKVTier
             store = None
             if cfg.enable_kvcache_store and cfg.kvcache_store_path:
@@ -340,6 +346,11 @@ class LLMEngine:
         act += cfg.max_seqs_per_batch * a.vocab_size * 4 * 2
         reserve = cfg.activation_reserve_bytes or (act + (2 << 30))
         budget -= reserve
+        state = getattr(self.model, "state_bytes_per_slot", None)
+        if state is not None:
+            budget -= state() * (self.state_slots + 1)
+        if per_block == 0:                # no layer caches keys: blocks only count positions
+            return cfg.max_seqs_per_batch * (-(-self.max_model_len // cfg.block_size)) + 1
         if cfg.max_cache_size > 0:
             budget = min(budget, cfg.max_cache_size)
         n = budget // per_block
@@ -402,6 +413,17 @@ class LLMEngine:
         self.runner.logits_hook = self._grammar_hook
 
     # ------------------------------------------------------------------ linear-attention state slots
+    def _slots_of(self, batch):
+        st = self.model.state
+        return np.asarray([st.slot_of(int(i)) for i in np.asarray(batch.seq_ids)], dtype=np.int32)
+
+    def _release_lost_states(self):
+        """State slots of sequences preempted or aborted since the last call go back to the pool (a preempted
+        sequence rebuilds its state from position 0)."""
+        if getattr(self.model, "needs_state", False):
+            for sid in self.scheduler.take_preempted():
+                self.model.state.release(int(sid))
+
     def _state_hook(self, batch, meta):
         """Gives every sequence of the batch its state slot and marks the ones that start at
         position 0 (new, or recomputed after a preemption) so that their state is reset."""
@@ -503,6 +525,7 @@ class LLMEngine:
             nvls = self.ps.world_size > 1 and self.device.type == "cuda" and os.environ.get("NCCL_NVLS_ENABLE", "1") != "0"
             self.fault.before_step(self.steps, multicast_bound=bool(getattr(comm, "mc_base", 0)) or nvls)
         batches = self.scheduler.schedule()
+        self._release_lost_states()         # before slots are assigned: a sequence may be preempted and re-admitted at once
         batch = batches[0] if batches else None
         if self.ps.dp_size > 1 and self.ps.ep_size > 1:
             self._dp_lockstep(batch)
@@ -533,8 +556,6 @@ class LLMEngine:
             for ev in events:
                 if ev.finished and ev.seq_id >= 0:
                     self.model.state.release(int(ev.seq_id))
-            for sid in self.scheduler.take_preempted():
-                self.model.state.release(int(sid))     # the state is rebuilt from position 0 anyway
         if self.mm:
             for ev in events:
                 if ev.request_finished:
@@ -544,6 +565,34 @@ class LLMEngine:
             if self.record_steps:
                 self.step_log.append((batch.n_decode, batch.n_prefill, batch.n_tokens))
         return events
+
+    # ------------------------------------------------------------------ replay of recorded requests
+    @torch.no_grad()
+    def replay_step(self, entries):
+        """One step whose tokens the caller gives: `entries` = [(request id, tokens, wanted places)], all run as one
+        batch (single tokens behind an existing context as decode rows, the rest as prompt chunks) from the cache and
+        state earlier steps left.  A request is admitted at its first entry and stays until `replay_end`.  Returns the
+        logits at the wanted places, fp32 [wanted, vocab] on the host, in the order of the entries."""
+        ids = [str(e[0]) for e in entries]
+        want = [[int(w) for w in e[2]] for e in entries]
+        batch = self.scheduler.schedule_replay(ids, [[int(t) for t in e[1]] for e in entries], want)
+        out = self.runner.execute(batch, want_host=False, want_logits=True)
+        # rows come in batch order (decode rows first); a batch of decode rows has one row per sequence
+        where, row = {}, 0
+        for i in range(batch.n_seqs):
+            rid = batch.request_id(i)
+            where[rid] = row
+            row += 1 if batch.n_prefill == 0 else len(want[ids.index(rid)])
+        pick = [where[r] + (0 if batch.n_prefill == 0 else j) for r, w in zip(ids, want) for j in range(len(w))]
+        logits = out.float()[torch.tensor(pick, device=out.device)].cpu() if pick else torch.empty(0, self.args.vocab_size)
+        self.scheduler.process_output(batch.batch_id, np.empty(0, dtype=np.int64), None)
+        return logits
+
+    def replay_end(self, request_id):
+        """The request is finished: its blocks and its state slot are free."""
+        self.scheduler.abort_request(str(request_id))
+        self.scheduler.take_pending_events()
+        self._release_lost_states()
 
     def drain(self):
         events = []
@@ -640,7 +689,7 @@ class LLMEngine:
                     torch.cuda.empty_cache()
             self.asleep = level
             return
-        self._kv_shapes = [(k.shape, v.shape, k.dtype, k.device) for k, v in r.kv_caches]
+        self._kv_shapes = [None if k is None else (k.shape, v.shape, k.dtype, k.device) for k, v in r.kv_caches]
         r.graphs.clear()
         r.graph_in.clear()
         r.graph_out.clear()
@@ -678,7 +727,11 @@ class LLMEngine:
             self.asleep = 0
             self.resume()
             return
-        for i, (ks, vs, dt, dev) in enumerate(self._kv_shapes):
+        for i, shapes in enumerate(self._kv_shapes):
+            if shapes is None:
+                r.kv_caches[i] = (None, None)
+                continue
+            ks, vs, dt, dev = shapes
             r.kv_caches[i] = (torch.zeros(ks, dtype=dt, device=dev), torch.zeros(vs, dtype=dt, device=dev))
         if getattr(self.spec, "drafter", None) is not None and hasattr(self.spec.drafter, "kv"):
             k0, v0 = r.kv_caches[0]

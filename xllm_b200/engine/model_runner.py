@@ -78,6 +78,7 @@ class _Staging:
         self.dev = torch.empty(nbytes, dtype=torch.uint8, device=device)
         self.ids_host = None
         self.lp_host = None
+        self.copied = None           # event behind the last H2D copy out of `host`
 
 
 def _view(buf, off, n, dtype):
@@ -90,7 +91,7 @@ class ModelRunner:
                  max_model_len: int, device, dtype, enable_graph: bool = True,
                  graph_buckets: Optional[List[int]] = None, n_staging: int = 2,
                  prefill_graph_tokens: Optional[List[int]] = None, prefill_graph_seqs: int = 4,
-                 kv_allocator=None):
+                 kv_allocator=None, max_sample_rows: int = 0):
         from .. import _rt
         self._rt = _rt
         self.model = model
@@ -109,7 +110,8 @@ class ModelRunner:
         self.kv_caches = self._alloc_kv()
         # a padded mixed step has up to `prefill_graph_seqs` prompt-chunk sequences besides a full decode bucket
         extra = max(1, int(prefill_graph_seqs))
-        cap = self._capacity(self.max_tokens + extra, self.max_seqs + extra, self.max_seqs + extra, self.bt_cols)
+        cap = self._capacity(self.max_tokens + extra, self.max_seqs + extra, max(self.max_seqs + extra, max_sample_rows),
+                             self.bt_cols)
         self.staging = [_Staging(cap, self.device, self.cuda) for _ in range(n_staging)]
         for s in self.staging:
             s.ids_host = torch.empty(self.max_seqs, dtype=torch.int64, pin_memory=self.cuda)
@@ -123,7 +125,10 @@ class ModelRunner:
         self.graph_launches = 0      # kernel launches re-issued by graph replays
         self.logits_hook = None
         self.mm_hook = None          # multimodal requests: (batch) -> None | (embeds, rope_table, rope_rows)
-        self.meta_hook = None        # (batch, meta) -> None: per-sequence state slots of linear-attention models
+        self.meta_hook = None        # (batch, meta) -> None: per-sequence state slots, models that run eagerly
+        # batch -> int32 numpy [n_seqs]: per-sequence state slots as a device input behind the packed buffer, so
+        # that captured steps read them (models with `state_on_device`)
+        self.state_slots = None
         self.keep_hidden = False     # speculative decoding with a draft layer needs the step's hidden states
         self.last_hidden = self.last_meta = self.last_positions = None
         self.graph_launches_per_replay: Dict[tuple, int] = {}
@@ -144,33 +149,46 @@ class ModelRunner:
         self._ws: Dict[int, Optional[torch.Tensor]] = {}
 
     # ------------------------------------------------------------------ memory
+    @staticmethod
+    def kv_layout(model, args):
+        """Per layer (planes, kv heads, head size) of the paged cache, or None for a layer without one.  Models whose
+        layers differ say so (`model.kv_layout()`); the others are uniform."""
+        if hasattr(model, "kv_layout"):
+            return model.kv_layout()
+        return [(int(getattr(model, "kv_planes", 2)), model.num_kv_heads_local, model.head_dim)] * args.num_hidden_layers
+
     def _alloc_kv(self):
-        m = self.model
-        L = self.args.num_hidden_layers
-        planes = int(getattr(m, "kv_planes", 2))
-        shape = (L, planes, self.num_blocks, m.num_kv_heads_local, self.block_size, m.head_dim)
+        layout = self.kv_layout(self.model, self.args)
+        sizes = [0 if g is None else g[0] * self.num_blocks * g[1] * self.block_size * g[2] for g in layout]
+        n = sum(sizes)
         if self.kv_allocator is not None:
-            n = 1
-            for d in shape:
-                n *= d
-            raw = self.kv_allocator(n * torch.empty((), dtype=self.dtype).element_size())
-            kv = raw.view(self.dtype).view(shape)
-            kv.zero_()
+            flat = self.kv_allocator(n * torch.empty((), dtype=self.dtype).element_size()).view(self.dtype)
+            flat.zero_()
         else:
-            kv = torch.zeros(shape, dtype=self.dtype, device=self.device)
-        self.kv_tensor = kv
-        return [(kv[i, 0], kv[i, planes - 1]) for i in range(L)]
+            flat = torch.zeros(n, dtype=self.dtype, device=self.device)
+        shapes = [None if g is None else (g[0], self.num_blocks, g[1], self.block_size, g[2]) for g in layout]
+        uniform = bool(shapes) and all(x is not None and x == shapes[0] for x in shapes)
+        self.kv_tensor = flat.view(len(layout), *shapes[0]) if uniform else flat
+        out, off = [], 0
+        for shape, size in zip(shapes, sizes):
+            if shape is None:
+                out.append((None, None))
+                continue
+            kv = flat[off:off + size].view(shape)
+            off += size
+            out.append((kv[0], kv[shape[0] - 1]))
+        return out
 
     @staticmethod
-    def kv_bytes_per_block(args, nkv_local, block_size, dtype, head_dim=None, planes=2):
+    def kv_bytes_per_block(model, args, block_size, dtype):
         esz = torch.empty((), dtype=dtype).element_size()
-        return args.num_hidden_layers * planes * nkv_local * block_size * (head_dim or args.head_dim) * esz
+        return sum(g[0] * g[1] * block_size * g[2] * esz for g in ModelRunner.kv_layout(model, args) if g is not None)
 
     @staticmethod
     def _capacity(T, S, NS, bt):
         al = lambda x: (x + 15) & ~15
         return (al(T * 8) * 2 + al(NS * 8) * 2 + al(T * 4) + al(S * 4) + al((S + 1) * 4) + al(S * 4)
-                + al(NS * 4) * 4 + al(S * bt * 4) + 256)
+                + al(NS * 4) * 4 + al(S * bt * 4) + al(S * 4) + 256)
 
     # ------------------------------------------------------------------ helpers
     def _decode_splits(self, B):
@@ -193,6 +211,17 @@ class ModelRunner:
             cu_q=_view(buf, off[5], S + 1, torch.int32),
             max_q_len=max_q_len, max_kv_len=max_kv_len, decode_splits=splits,
             decode_workspace=self._workspace(n_decode, splits) if splits > 1 else None, padded=padded)
+
+    def _put_state_slots(self, batch, host, off, n_decode_rows):
+        """Writes the sequences' state slots (-1: padding) behind the packed inputs; returns the bytes in use."""
+        S, nd = off[13], batch.n_decode
+        slots = np.full(S, -1, dtype=np.int32)
+        real = self.state_slots(batch)
+        slots[:nd] = real[:nd]
+        slots[n_decode_rows:n_decode_rows + batch.n_prefill] = real[nd:]
+        at = off[11]
+        host[at:at + 4 * S].numpy().view(np.int32)[:] = slots
+        return at + 4 * S
 
     def _bucket(self, n):
         for b in self.buckets:
@@ -242,6 +271,8 @@ class ModelRunner:
                 or self.keep_hidden:
             return None
         nd, npf = batch.n_decode, batch.n_prefill
+        if npf > 0 and batch.n_samples > nd + npf:      # a replayed step may ask for more rows than sequences
+            return None
         if npf == 0:
             Bp = self._bucket(nd)
             return None if Bp is None else (Bp, 0, 0, mode)
@@ -265,13 +296,16 @@ class ModelRunner:
         T, S = Bp + Tq, Bp + P
         NS = S
         off = list(self._rt.packed_layout(T, S, NS, self.bt_cols))
-        gin = torch.zeros(off[11], dtype=torch.uint8, device=self.device)
+        gin = torch.zeros(off[11] + (4 * S if self.state_slots is not None else 0), dtype=torch.uint8, device=self.device)
         _view(gin, off[3], T, torch.int32).fill_(-1)   # slots: no KV write during warm-up
         cu = _view(gin, off[5], S + 1, torch.int32)
         cu[: Bp + 1].copy_(torch.arange(Bp + 1, dtype=torch.int32))
         cu[Bp + 1:].fill_(Bp)                           # prompt-chunk sequences without rows
         _view(gin, off[9], NS, torch.float32).fill_(1.0)
         meta = self._meta_from(gin, off, Bp, P, Tq if P else 1, 0, self.bt_cols, padded=P > 0)
+        if self.state_slots is not None:
+            meta.state_slots = _view(gin, off[11], S, torch.int32)
+            meta.state_slots.fill_(-1)                  # warm-up passes touch no state
         tokens = _view(gin, off[0], T, torch.int64)
         positions = _view(gin, off[1], T, torch.int64)
         rows = _view(gin, off[2], NS, torch.int64)
@@ -324,12 +358,16 @@ class ModelRunner:
 
     # ------------------------------------------------------------------ one step
     @torch.no_grad()
-    def execute(self, batch, want_host=True) -> StepOutput:
+    def execute(self, batch, want_host=True, want_logits=False):
+        """One scheduled step.  `want_logits`: nothing is sampled, the full-vocabulary logits of the batch's sample rows
+        are returned instead of a StepOutput (None when it has none)."""
         st = self.staging[self._turn % len(self.staging)]
         self._turn += 1
+        if st.copied is not None:
+            st.copied.synchronize()  # a caller that does not wait for every step must not overwrite a copy in flight
         nd, npf = batch.n_decode, batch.n_prefill
         mm = self.mm_hook(batch) if self.mm_hook is not None else None
-        mode = self.sample_mode(batch)
+        mode = "logits" if want_logits else self.sample_mode(batch)
         key = self.graph_key(batch, mode, mm)
         n_real = batch.n_samples
         if key is not None:
@@ -340,8 +378,13 @@ class ModelRunner:
             bt_stride = max(8, (batch.max_blocks + 7) // 8 * 8)
             off = batch.fill_packed(st.host.data_ptr(), st.host.numel(), bt_stride, 0)
         nbytes = off[11]
+        if self.state_slots is not None:
+            nbytes = self._put_state_slots(batch, st.host, off, key[0] if key is not None else nd)
         if self.cuda:
             st.dev[:nbytes].copy_(st.host[:nbytes], non_blocking=True)
+            if st.copied is None:
+                st.copied = torch.cuda.Event()
+            st.copied.record()
             self.h2d_bytes += nbytes
             buf = st.dev
         else:
@@ -369,6 +412,8 @@ class ModelRunner:
             meta = self._meta_from(buf, off, nd, npf, batch.max_q_len, batch.max_kv_len, bt_stride)
             if self.meta_hook is not None:
                 self.meta_hook(batch, meta)
+            if self.state_slots is not None:
+                meta.state_slots = _view(buf, off[11], S, torch.int32)
             if mm is not None:
                 embeds, meta.rope_table, meta.rope_rows = mm
                 hidden = self.model.forward(tokens, positions, meta, self.kv_caches, embeds=embeds)
@@ -376,6 +421,8 @@ class ModelRunner:
                 hidden = self.model.forward(tokens, positions, meta, self.kv_caches)
             if self.keep_hidden:
                 self.last_hidden, self.last_meta, self.last_positions = hidden, meta, positions
+            if NS == 0 and want_logits:
+                return None
             rows = _view(buf, off[2], NS, torch.int64)
             h = hidden if (NS == T and npf == 0) else ops.gather_rows(hidden, rows)
             logits = self.model.logits_local(h)
@@ -383,6 +430,9 @@ class ModelRunner:
             if mode != "logits":
                 ids, lp = self._device_sample(logits, src, off, NS, mode, want_lp=batch.any_logprobs)
 
+        if want_logits:
+            logits = self.model.gather_logits(logits) if self.model.ps.tp_size > 1 else logits
+            return logits[:n_real, :self.model.lm_head.vocab] if n_real else None
         top = None
         if mode == "logits":
             # the host takes part: penalties over the sequences' token histories, grammar masks,

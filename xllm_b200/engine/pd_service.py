@@ -276,6 +276,8 @@ class SocketCopy:
 # ------------------------------------------------------------------------------------------ helpers
 def _topology(engine) -> dict:
     r = engine.runner
+    if getattr(r.model, "needs_state", False):
+        raise ValueError("a disaggregated pair hands over KV blocks; recurrent per-sequence state does not travel with them")
     k0 = r.kv_caches[0][0]
     return {"block_size": int(r.block_size), "n_layers": len(r.kv_caches), "n_kv_heads": int(k0.shape[1]),
             "head_dim": int(k0.shape[3]), "dtype": str(k0.dtype), "tp": int(engine.ps.tp_size),

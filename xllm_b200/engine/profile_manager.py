@@ -117,6 +117,11 @@ class ProfileManager:
                         kv_lens=torch.full((nseq,), ctx + q, dtype=torch.int32, device=dev),
                         cu_q=torch.arange(0, nseq * q + 1, q, dtype=torch.int32, device=dev), max_q_len=q,
                         max_kv_len=ctx + q)
+            if getattr(runner.model, "needs_state", False):
+                on_dev = bool(getattr(runner.model, "state_on_device", False))
+                meta.state_slots = (torch.arange(nseq) % runner.model.state.n_slots).to(
+                    torch.int32 if on_dev else torch.long).to(dev)
+                meta.state_fresh, meta.seq_bounds = [True] * nseq, [(i * q, i * q + q) for i in range(nseq)]
             toks = torch.zeros(nseq * q, dtype=torch.int64, device=dev)
             best = 1e9
             for _ in range(repeats):

@@ -109,7 +109,39 @@ def _eos_list(v):
     return int(v), [int(v)]
 
 
-def model_args_from_dict(cfg: Dict[str, Any]) -> ModelArgs:
+def _femirax_args(cfg: Dict[str, Any], shapes: Dict[str, List[int]]) -> ModelArgs:
+    """Femirax configurations list every layer; the rank of a low-rank decay projection is only in its tensor's shape."""
+    import copy
+    layers = copy.deepcopy(cfg["layers"])
+    for i, layer in enumerate(layers):
+        shape = shapes.get(f"l{i}.mix.right.a1")
+        if shape is not None:
+            layer["mixer"]["right"]["rank"] = int(shape[0])
+    a = ModelArgs(model_type="femirax", architectures=["Femirax"], vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
+                  num_hidden_layers=len(layers), rms_norm_eps=float(cfg["norm"]["eps"]), qk_norm=False, tie_word_embeddings=False)
+    left = [l["mixer"]["left"] for l in layers if l["type"] == "parallel"]
+    a.num_attention_heads = max([l["heads"] for l in left] + [1])
+    a.num_key_value_heads = max([l["kv_heads"] for l in left] + [1])
+    a.head_dim = max([l["dim"] for l in left] + [1])
+    a.intermediate_size = max([l["mlp"]["ff"] for l in layers if l.get("mlp")] + [a.hidden_size])
+    a.max_position_embeddings = int(_g(cfg, "max_position_embeddings", default=32768))
+    a.extra = {"layers": layers, "side_dim": int(cfg["token_side"]["dim"]),
+               # positions are unbounded unless the configuration names a limit: the engine may ask for longer sequences
+               "unbounded_positions": "max_position_embeddings" not in cfg}
+    a.bos_token_id = _g(cfg, "bos_token_id", default=-1)
+    a.eos_token_id, a.stop_token_ids = _eos_list(_g(cfg, "eos_token_id"))
+    return a
+
+
+# `architecture` names whose configurations do not follow the HuggingFace layout: name -> fn(config, tensor shapes)
+_OWN_LAYOUTS = {"femirax": _femirax_args}
+
+
+def model_args_from_dict(cfg: Dict[str, Any], shapes: Optional[Dict[str, List[int]]] = None) -> ModelArgs:
+    """`shapes`: tensor name -> shape of the checkpoint, for layouts that leave a size to a tensor's shape."""
+    own = _OWN_LAYOUTS.get(str(cfg.get("architecture", "")).lower())
+    if own is not None:
+        return own(cfg, shapes or {})
     text = cfg.get("text_config", cfg)  # VLM configs nest the language model
     mt = text.get("model_type", cfg.get("model_type", "qwen3"))
     a = ModelArgs(model_type=cfg.get("model_type", mt))
@@ -220,7 +252,11 @@ def load_model_args(model_dir: str) -> ModelArgs:
     p = Path(model_dir) / "config.json"
     with open(p) as f:
         cfg = json.load(f)
-    args = model_args_from_dict(cfg)
+    shapes = None
+    if str(cfg.get("architecture", "")).lower() in _OWN_LAYOUTS:
+        from ..utils.loader import tensor_shapes
+        shapes = tensor_shapes(model_dir)
+    args = model_args_from_dict(cfg, shapes)
     gen = Path(model_dir) / "generation_config.json"
     if gen.exists():
         with open(gen) as f:

@@ -52,6 +52,9 @@ class AttentionMetadata:
     # prompt pages plus each beam's tail (ops/xattn.py).  Object with tail_of(k_cache) -> (ku, vu), anc,
     # n_tail, max_rows.
     xattn: Optional[object] = None
+    # models with per-sequence recurrent state: the state slot of every sequence row [B] (-1: padding).  int32 on the
+    # device for models with `state_on_device`, whose layers see from kv_lens and cu_q which sequences start afresh
+    state_slots: Optional[torch.Tensor] = None
 
     @property
     def n_seqs(self):

@@ -27,34 +27,17 @@ from .layers import Attention, DenseMLP, Linear, MergedColumnLinear, Module, RMS
 from .qwen import DecoderLayer, DenseCausalLM
 from .qwen_moe import SparseMoeBlock
 from .registry import register_model
+from .state import StateSlots
 from ..parallel.state import single
 
 
-class LinearStateCache:
-    """Convolution tails and recurrent states of every linear-attention layer, one slot per running
-    sequence (keyed by the scheduler's sequence id: parallel samples of one request have their own
-    state).  The scheduler admits at most `slots` sequences at a time and slots return on finish and
-    on preemption, so `slot_of` finds a free slot whenever it needs one."""
+class LinearStateCache(StateSlots):
+    """Convolution tails and recurrent states of every linear-attention layer, one slot per running sequence."""
 
     def __init__(self, n_layers, slots, conv_dim, kernel, nv, dk, dv, device, dtype):
+        super().__init__(slots)
         self.conv = torch.zeros(n_layers, slots, conv_dim, kernel - 1, dtype=dtype, device=device)
         self.rec = torch.zeros(n_layers, slots, nv, dk, dv, dtype=torch.float32, device=device)
-        self.free = list(range(slots - 1, -1, -1))
-        self.owner = {}
-        self.n_slots = slots
-
-    def slot_of(self, request_id):
-        s = self.owner.get(request_id)
-        if s is None:
-            if not self.free:
-                raise RuntimeError("no free linear-state slot: the scheduler admitted more sequences than the pool holds")
-            s = self.owner[request_id] = self.free.pop()
-        return s
-
-    def release(self, request_id):
-        s = self.owner.pop(request_id, None)
-        if s is not None:
-            self.free.append(s)
 
 
 class GatedDeltaNet(Module):

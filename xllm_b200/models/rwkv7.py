@@ -25,6 +25,7 @@ import torch.nn.functional as F
 
 from .layers import LMHead, Linear, Module, VocabEmbedding
 from .registry import register_model
+from .state import StateSlots
 from ..parallel.state import single
 
 
@@ -41,29 +42,14 @@ class _LayerNorm(Module):
     __call__ = forward
 
 
-class Rwkv7State:
+class Rwkv7State(StateSlots):
     """Per running sequence: shift vectors of both mixers and the wkv state of every layer."""
 
     def __init__(self, n_layers, slots, hidden, heads, head_size, device, dtype):
+        super().__init__(slots)
         self.att_shift = torch.zeros(n_layers, slots, hidden, dtype=dtype, device=device)
         self.ffn_shift = torch.zeros(n_layers, slots, hidden, dtype=dtype, device=device)
         self.wkv = torch.zeros(n_layers, slots, heads, head_size, head_size, dtype=torch.float32, device=device)
-        self.free = list(range(slots - 1, -1, -1))
-        self.owner = {}
-        self.n_slots = slots
-
-    def slot_of(self, seq_id):
-        s = self.owner.get(seq_id)
-        if s is None:
-            if not self.free:
-                raise RuntimeError("no free state slot: the scheduler admitted more sequences than the pool holds")
-            s = self.owner[seq_id] = self.free.pop()
-        return s
-
-    def release(self, seq_id):
-        s = self.owner.pop(seq_id, None)
-        if s is not None:
-            self.free.append(s)
 
 
 class TimeMix(Module):

@@ -78,6 +78,14 @@ def rmsnorm(x, w, eps=1e-6, residual=None, out=None, gemma=False):
 def act_and_mul(x, act="silu", out=None):
     if not x.is_cuda:
         return reference.act_and_mul(x, act)
+    if x.dtype == torch.float32 and act == "silu":
+        d = x.shape[-1] // 2
+        x2 = x.reshape(-1, 2 * d)
+        if out is None:
+            out = torch.empty((x2.shape[0], d), dtype=x.dtype, device=x.device)
+        check(_lib_().xllm_silu_mul_f32(ptr(out), ptr(x2), x2.shape[0], d, x2.stride(0), stream()), "silu_mul_f32")
+        _count()
+        return out.reshape(*x.shape[:-1], d)
     _bf16(x, "act_and_mul")
     d = x.shape[-1] // 2
     x2 = x.reshape(-1, 2 * d)
@@ -133,7 +141,63 @@ def rope_kv_write(qkv, nq, nkv, d, positions, cos_sin, rot, slots=None, k_cache=
     return (q_out, k_out, v_out) if return_kv else q_out
 
 
+def rope_norm_kv_write(q, k, v, nq, nkv, d, positions, cos_sin, rot, slots, k_cache, v_cache, eps=1e-6,
+                       interleaved=False, unit_norm=True):
+    """Rotary positions on the first `rot` elements of every q and k head, THEN (`unit_norm`) each head divided by its
+    root mean square; k and v rows are scattered into the paged caches.  q, k, v: column blocks [T, heads * d] of the
+    same projection rows (v may be the key block).  The caches may hold wider heads than d (zero filled); returns q
+    [T, nq, cache head size]."""
+    T, dp = q.shape[0], k_cache.shape[3]
+    if _debug.enabled():
+        _debug.check_range(positions, 0, cos_sin.shape[0], "rope_norm_kv_write positions")
+        _debug.check_range(slots, 0, k_cache.shape[0] * k_cache.shape[2], "rope_norm_kv_write slots", allow_negative_skip=True)
+    if not q.is_cuda:
+        return reference.rope_norm_kv(q, k, v, nq, nkv, d, positions, cos_sin, rot, slots, k_cache, v_cache, eps, interleaved,
+                                      unit_norm)
+    assert q.stride(0) == k.stride(0) == v.stride(0) and q.stride(1) == k.stride(1) == v.stride(1) == 1
+    assert q.dtype == k_cache.dtype and k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.shape[1] == nkv
+    positions = _index(positions, torch.int64, "rope_norm_kv_write positions")
+    slots = _index(slots, torch.int32, "rope_norm_kv_write slots")
+    out = torch.empty((T, nq, dp), dtype=q.dtype, device=q.device)
+    check(_lib_().xllm_rope_norm_kv(ptr(q), ptr(k), ptr(v), q.stride(0), ptr(out), ptr(k_cache), ptr(v_cache), ptr(cos_sin),
+                                    cos_sin.shape[0] if cos_sin is not None else 0, ptr(positions), ptr(slots), T, nq, nkv, d,
+                                    dp, rot, k_cache.shape[2], int(interleaved), int(unit_norm), eps,
+                                    0 if q.dtype == torch.bfloat16 else 1, stream()), "rope_norm_kv")
+    _count()
+    return out
+
+
 # ----------------------------------------------------------------------------- attention
+def attention_head_size(d):
+    """Head size a cache should be laid out with for heads of d: the sizes of the tensor-core kernels (zero filled),
+    d itself beyond them (the generic kernel takes any)."""
+    return next((s for s in (64, 128, 256) if d <= s), d)
+
+
+def paged_attention_generic(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, out=None, row0=0, rows=None, window=0):
+    """Rows [row0, row0 + rows) of q [T, nq, d], decode rows and prompt chunks alike (row ranges by cu_q), fp32 or bf16
+    caches, any head size up to 512: the path of the fp32 execution type."""
+    T, nq, d = q.shape
+    rows = T - row0 if rows is None else rows
+    if not q.is_cuda:
+        y = reference.paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, True, window)
+        if out is not None:
+            out[row0:row0 + rows].copy_(y[row0:row0 + rows])
+            return out
+        return y
+    if out is None:
+        out = torch.empty_like(q)
+    assert q.stride(-1) == 1 and q.stride(1) == d and q.dtype == k_cache.dtype == out.dtype
+    cu_q = _index(cu_q, torch.int32, "paged_attention_generic cu_q")
+    kv_lens = _index(kv_lens, torch.int32, "paged_attention_generic kv_lens")
+    check(_lib_().xllm_paged_attn_generic(ptr(out), out.stride(0), ptr(q), q.stride(0), ptr(k_cache), ptr(v_cache),
+                                          ptr(block_table), block_table.stride(0), ptr(cu_q), ptr(kv_lens), kv_lens.shape[0],
+                                          row0, rows, nq, k_cache.shape[1], d, k_cache.shape[2], scale, int(window or 0),
+                                          0 if q.dtype == torch.bfloat16 else 1, stream()), "paged_attn_generic")
+    _count()
+    return out
+
+
 def decode_splits(batch, nkv, group, max_kv_len=None, n_sm=148):
     """Split-KV factor.  Without a context length: enough CTAs to cover ~2 per SM.  With one: the factor in
     1..16 that minimises (waves of CTAs over 2 resident per SM) x (tokens per split + a fixed cost for the

@@ -105,6 +105,9 @@ def _declare(lib):
         "xllm_block_copy": [P, I, P, I, L, P],
         "xllm_decode_advance": [P, P, P, P, P, I, P, I, I, P],
         "xllm_resolve_placeholders": [P, P, L, L, P],
+        "xllm_rope_norm_kv": [P, P, P, L, P, P, P, P, L, P, P, I, I, I, I, I, I, I, I, I, F, I, P],
+        "xllm_paged_attn_generic": [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, I, F, I, I, P],
+        "xllm_silu_mul_f32": [P, P, L, I, L, P],
     }
     for name, args in sig.items():
         lib.declare(name, args, I)

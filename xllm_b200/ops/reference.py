@@ -131,6 +131,28 @@ def rope_kv(qkv, nq, nkv, d, positions, cos_sin, rot, q_norm_w=None, k_norm_w=No
     return qf.to(qkv.dtype), kf.to(qkv.dtype), v.contiguous()
 
 
+def rope_norm_kv(q, k, v, nq, nkv, d, positions, cos_sin, rot, slots, k_cache, v_cache, eps, interleaved, unit_norm):
+    """Rotation, then a per-head RMS norm without a weight; k and v go to caches whose heads may be wider than d."""
+    T, dp = q.shape[0], k_cache.shape[3]
+    half = rot // 2
+    cs = cos_sin[positions.long()].float() if rot else None
+
+    def prep(x, n):
+        x = x.reshape(T, n, d).float()
+        if rot:
+            c, s = cs[:, None, :half], cs[:, None, half:]
+            xr = x[..., :rot]
+            a, b = (xr[..., 0::2], xr[..., 1::2]) if interleaved else (xr[..., :half], xr[..., half:])
+            y, z = a * c - b * s, b * c + a * s
+            xr = torch.stack([y, z], dim=-1).flatten(-2) if interleaved else torch.cat([y, z], dim=-1)
+            x = torch.cat([xr, x[..., rot:]], dim=-1)
+        return x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) if unit_norm else x
+
+    pad = lambda x: torch.nn.functional.pad(x, (0, dp - d)).to(k_cache.dtype)
+    write_kv_cache(pad(prep(k, nkv)), pad(v.reshape(T, nkv, d).float()), k_cache, v_cache, slots)
+    return pad(prep(q, nq))
+
+
 def write_kv_cache(k, v, k_cache, v_cache, slots):
     """k,v: [T, nkv, d]; caches [n_blocks, nkv, page, d]; slots [T] (negative => skip)."""
     page = k_cache.shape[2]

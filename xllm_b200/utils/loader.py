@@ -60,6 +60,18 @@ def iterate_weights(model_dir: str) -> Iterator[Tuple[str, torch.Tensor]]:
         yield from iterate_file(p)
 
 
+def tensor_shapes(model_dir: str) -> Dict[str, List[int]]:
+    """Name -> shape of every tensor of a checkpoint directory (headers only; {} without safetensors files)."""
+    out = {}
+    for path in shard_files(model_dir):
+        with open(path, "rb") as f:
+            n = int.from_bytes(f.read(8), "little")
+            for name, e in json.loads(f.read(n)).items():
+                if name != "__metadata__":
+                    out[name] = list(e["shape"])
+    return out
+
+
 def save_file(tensors: Dict[str, torch.Tensor], path: str, metadata: Dict[str, str] = None) -> None:
     """Write a safetensors file (used by tests, by `update_weights` round trips and by tools)."""
     header = {}
