@@ -31,13 +31,14 @@ def rotate(x, base, dims, layout, first_position=0):
     """Rotary positions on the first `dims` of every head of x [T, heads, dim]; row t sits at position
     first_position + t.  layout 'half': i with i + dims/2; 'pairs': 2i with 2i + 1."""
     y = x.clone()
-    for t in range(x.shape[0]):
-        for i in range(dims // 2):
-            a = (first_position + t) * base ** (-2.0 * i / dims)
-            j0, j1 = (i, i + dims // 2) if layout == "half" else (2 * i, 2 * i + 1)
-            u, v = x[t, :, j0], x[t, :, j1]
-            y[t, :, j0] = u * math.cos(a) - v * math.sin(a)
-            y[t, :, j1] = v * math.cos(a) + u * math.sin(a)
+    position = first_position + torch.arange(x.shape[0], dtype=torch.float64)
+    for i in range(dims // 2):
+        a = position * base ** (-2.0 * i / dims)
+        cos, sin = a.cos().to(x.dtype)[:, None], a.sin().to(x.dtype)[:, None]
+        j0, j1 = (i, i + dims // 2) if layout == "half" else (2 * i, 2 * i + 1)
+        u, v = x[:, :, j0], x[:, :, j1]
+        y[:, :, j0] = u * cos - v * sin
+        y[:, :, j1] = v * cos + u * sin
     return y
 
 
@@ -46,12 +47,12 @@ def causal_attention(q, k, v, scale):
     T, H, _ = q.shape
     G = k.shape[1]
     out = q.new_zeros(T, H, v.shape[-1])
-    for t in range(T):
-        for h in range(H):
-            g = h // (H // G)
-            s = (k[: t + 1, g] @ q[t, h]) * scale
-            p = torch.exp(s - s.max())
-            out[t, h] = (p / p.sum()) @ v[: t + 1, g]
+    hidden = torch.ones(T, T, dtype=torch.bool).triu(1)             # key j > query i
+    for h in range(H):
+        g = h // (H // G)
+        s = ((q[:, h] @ k[:, g].T) * scale).masked_fill(hidden, -math.inf)
+        p = torch.exp(s - s.max(-1, keepdim=True).values)
+        out[:, h] = (p / p.sum(-1, keepdim=True)) @ v[:, g]
     return out
 
 
