@@ -1,6 +1,5 @@
 """Femirax through the engine (loading, cache, state slots, scheduler, sampling) against a plain implementation of its
 equations: whole prompts, portions, token by token, mixed batches, reused pages and slots, far keys, greedy generation."""
-import io
 import json
 import os
 import subprocess
@@ -97,3 +96,211 @@ def test_mixed_batches_and_reused_pages_and_slots(tmp_path, name, target):
             at = [p for p, _ in rows]
             assert error(torch.stack([x for _, x in rows]), want[r][at]) < LIMIT[target[1]], r
     assert steps > 10 and len(eng.model.state.free) == 4 and eng.scheduler.block_stats(0).num_used == 0
+
+
+# ------------------------------------------------------------------------------------------- far keys
+def _far_model(kind):
+    """One layer in which the query of token 91 points along the key of token 92: that key's score stands out among
+    hundreds (attention), or its share of a slowly decaying state does."""
+    if kind == "attention":
+        cfg = config([parallel(3, 3, 24, 8, 1.6, 1, 8, 8, 1.0, base=1e5)], vocab=96, width=64)
+    elif kind == "channel":
+        cfg = config([parallel(1, 1, 8, 0, 0.1, 3, 24, 20, 16.0)], vocab=96, width=64)
+    else:
+        cfg = config([retention(3, 24, 20, [0.9999, 0.9995, 0.999], 8, base=1e5)], vocab=96, width=64)
+    w = oracle.random_weights(cfg, 4, seed=11)
+    p = {"attention": "l0.mix.left.", "channel": "l0.mix.right.", "retention": "l0.mix."}[kind]
+    w["embed"][:, :2] = 0.0                                           # coordinates 0 and 1 belong to the two tokens
+    w["embed"][92, 0] = w["embed"][91, 1] = 20.0
+    w[p + "k"][:, 0] *= 2.0
+    w[p + "q"][:, 1] = w[p + "k"][:, 0]
+    if kind == "retention":
+        w["l0.mix.o"] *= 8.0
+    if kind == "channel":
+        w[p + "a2.b"].fill_(12.0)                                     # decays within 1e-6 of one
+    # what the other side of the layer says is turned down
+    if kind == "attention":
+        w["l0.mix.right.out"] *= 0.05
+        w["l0.mix.left.out"] *= 4.0
+    if kind == "channel":
+        w["l0.mix.left.out"] *= 0.05
+        w["l0.mix.right.out"] *= 4.0
+    return cfg, w
+
+
+@pytest.mark.parametrize("target", TARGETS)
+@pytest.mark.parametrize("kind", ["attention", "channel", "retention"])
+def test_far_keys(tmp_path, kind, target):
+    """The last token asks for one far back: at the first places, on both sides of page borders and of the sixteen-token
+    chunks of the recurrence, and at a border of the portions.  The far token must show in the answer, whether the
+    query ends a prompt's portion or is decoded alone."""
+    cfg, w = _far_model(kind)
+    eng = make_engine(tmp_path, cfg, w, target)
+    base = random_tokens(300, 90, 4)
+    lim = LIMIT[target[1]]
+    for far in (0, 1, 15, 16, 31, 32, 33, 63, 64, 200, 287, 288):
+        toks = list(base)
+        toks[far] = 92                                               # ids 90.. appear nowhere else
+        toks[-1] = 91
+        want = expect(cfg, w, toks)[-1:]
+        without = list(base)
+        without[-1] = 91
+        seen = error(expect(cfg, w, without)[-1:], want)
+        assert seen > 2 * lim, (kind, far, seen)                     # leaving the far key out would show
+        for cuts in ([300], [64, 33, 2, 200, 1], [297, 3], [299, 1]):
+            at, i = 0, 0
+            while at < 300:
+                n = min(cuts[i], 300 - at)
+                got = eng.replay_step([("f", toks[at:at + n], [n - 1] if at + n == 300 else [])])
+                at, i = at + n, i + 1
+            eng.replay_end("f")
+            assert error(got, want) < lim, (kind, far, cuts)
+
+
+@pytest.mark.parametrize("target", TARGETS)
+def test_long_decoding(tmp_path, target):
+    """A short prompt, then hundreds of tokens one at a time across many page borders."""
+    cfg, w = weights_of("odd", seed=6)
+    toks = random_tokens(260, cfg["vocab"], 9)
+    want = expect(cfg, w, toks)
+    eng = make_engine(tmp_path, cfg, w, target)
+    assert error(feed(eng, "d", toks, [3] + [1] * 300), want) < LIMIT[target[1]]
+
+
+@pytest.mark.parametrize("target", TARGETS)
+def test_a_batch_does_not_change_its_members(tmp_path, target):
+    """The same request alone and beside three others; first tokens of a sequence included."""
+    cfg, w = weights_of("aligned", seed=8)
+    reqs = [random_tokens(n, cfg["vocab"], 30 + n) for n in (1, 2, 37, 48)]
+    eng = make_engine(tmp_path, cfg, w, target)
+    alone = [eng.replay_step([(f"a{i}", t, list(range(len(t))))]) for i, t in enumerate(reqs)]
+    for i in range(4):
+        eng.replay_end(f"a{i}")
+    both = eng.replay_step([(f"b{i}", t, list(range(len(t)))) for i, t in enumerate(reqs)])
+    row = 0
+    for t, a in zip(reqs, alone):
+        assert error(both[row:row + len(t)], a) < LIMIT[target[1]] / 2
+        row += len(t)
+    # all four decode in one batch, in another order, one left out
+    nxt = {f"b{i}": [(7 * i + 3) % cfg["vocab"]] for i in (3, 0, 2)}
+    got = eng.replay_step([(r, t, [0]) for r, t in nxt.items()])
+    for j, (r, t) in enumerate(nxt.items()):
+        want = expect(cfg, w, reqs[int(r[1])] + t)[-1:]
+        assert error(got[j:j + 1], want) < LIMIT[target[1]]
+
+
+# ------------------------------------------------------------------------------------------- scheduler and sampling
+GREEDY_TARGETS = TARGETS[:2]                                          # fp32: no near ties between two implementations
+
+
+def _llm(engine):
+    from xllm_b200 import LLM
+    llm = LLM.__new__(LLM)
+    llm.engine, llm.tokenizer, llm._workers = engine, None, None
+    return llm
+
+
+@pytest.mark.parametrize("target", GREEDY_TARGETS)
+@pytest.mark.parametrize("policy,overlap", [("prefill_first", False), ("decode_first", False), ("decode_first", True)])
+def test_greedy_generation(tmp_path, policy, overlap, target):
+    """LLM.generate through the scheduler: more requests than slots, prompts cut by a small token budget."""
+    from xllm_b200 import SamplingParams
+    cfg, w = weights_of("odd", seed=5)
+    prompts = [random_tokens(n, cfg["vocab"], 50 + n) for n in (5, 40, 17, 1, 66, 23)]
+    eng = make_engine(tmp_path, cfg, w, target, max_tokens_per_batch=24, policy=policy, enable_schedule_overlap=overlap)
+    outs = _llm(eng).generate(prompts, SamplingParams(max_tokens=12, temperature=0.0, ignore_eos=True))
+    w64 = {n: t.double() for n, t in w.items()}
+    for p, o in zip(prompts, outs):
+        assert o.outputs[0].token_ids == oracle.greedy(p, 12, cfg, w64)
+    assert len(eng.model.state.free) == 4 and not eng.model.state.owner
+
+
+@pytest.mark.parametrize("target", GREEDY_TARGETS)
+@pytest.mark.parametrize("policy", ["prefill_first", "decode_first"])
+def test_preemption_rebuilds_the_state(tmp_path, policy, target):
+    """So few pages that sequences are preempted, some re-admitted in the very step that pushed them out."""
+    from xllm_b200 import SamplingParams
+    cfg, w = weights_of("odd", seed=5)
+    prompts = [random_tokens(n, cfg["vocab"], 70 + n) for n in (30, 45, 18, 60, 25)]
+    eng = make_engine(tmp_path, cfg, w, target, num_blocks=11, max_tokens_per_batch=32, policy=policy)
+    outs = _llm(eng).generate(prompts, SamplingParams(max_tokens=16, temperature=0.0, ignore_eos=True))
+    w64 = {n: t.double() for n, t in w.items()}
+    for p, o in zip(prompts, outs):
+        assert o.outputs[0].token_ids == oracle.greedy(p, 16, cfg, w64)
+    assert eng.scheduler.num_preemptions > 0
+    assert len(eng.model.state.free) == 4 and not eng.model.state.owner
+
+
+@pytest.mark.parametrize("target", TARGETS)
+def test_sampling_parallel_samples_and_abort(tmp_path, target):
+    from xllm_b200 import SamplingParams
+    cfg, w = weights_of("retention_only")
+    eng = make_engine(tmp_path, cfg, w, target)
+    llm = _llm(eng)
+    sp = SamplingParams(max_tokens=9, temperature=0.9, top_p=0.95, n=3, seed=4, ignore_eos=True)
+    a, b = (llm.generate([[3, 1, 4, 1, 5]], sp)[0] for _ in range(2))
+    assert [o.token_ids for o in a.outputs] == [o.token_ids for o in b.outputs]
+    assert len({tuple(o.token_ids) for o in a.outputs}) > 1
+    eng.add_request("gone", [5, 6, 7, 8], max_tokens=50, ignore_eos=True, n=2)
+    for _ in range(3):
+        eng.step()
+    eng.abort("gone")
+    while eng.has_unfinished():
+        eng.step()
+    eng.step()
+    assert len(eng.model.state.free) == 4 and not eng.model.state.owner
+    emb = llm.embed([[1, 2, 3], [4, 5, 6, 7]])
+    assert len(emb) == 2
+
+
+def test_replay_program(tmp_path):
+    """bin/trace_run as a process: protocol, output files, answers."""
+    cfg, w = weights_of("odd", seed=12)
+    model = write_checkpoint(tmp_path / "m", cfg, w)
+    os.makedirs(tmp_path / "out")
+    a, b = random_tokens(40, cfg["vocab"], 1), random_tokens(9, cfg["vocab"], 2)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:20], "want": [3, 19]}, {"id": "b", "tokens": b[:8], "want": []}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": a[20:39], "want": []}], "end": []},
+             {"step": 2, "entries": [{"id": "b", "tokens": b[8:], "want": [0]}, {"id": "a", "tokens": a[39:], "want": [0]}], "end": ["b"]}]
+    r = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", model, "--dtype", "float32", "--out",
+                        str(tmp_path / "out"), "--max-tokens", "128", "--device", "cpu"],
+                       input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=300)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert [l for l in r.stdout.splitlines() if l.startswith("done")] == ["done 0", "done 1", "done 2"]
+    assert sorted(os.listdir(tmp_path / "out")) == ["0.f32", "2.f32"]
+    V = cfg["vocab"]
+    read = lambda n: torch.from_numpy(np.fromfile(tmp_path / "out" / n, dtype="<f4").reshape(-1, V))
+    wa, wb = expect(cfg, w, a), expect(cfg, w, b)
+    assert error(read("0.f32"), wa[[3, 19]]) < 2e-4
+    assert error(read("2.f32"), torch.stack([wb[8], wa[39]])) < 2e-4
+
+
+def test_replay_refuses_what_it_cannot_hold(tmp_path):
+    cfg, w = weights_of("retention_only")
+    eng = make_engine(tmp_path, cfg, w, ("cpu", "float32"), num_blocks=4)       # three usable pages
+    eng.replay_step([("a", [1] * 30, [0])])
+    with pytest.raises(RuntimeError):
+        eng.replay_step([("b", [1] * 20, [])])
+    with pytest.raises(ValueError):
+        eng.replay_step([("a", [1, 2], [2])])
+    with pytest.raises(ValueError):
+        eng.replay_step([("c", [], [])])
+
+
+def test_configuration_is_read_from_the_checkpoint(tmp_path):
+    from xllm_b200.models import load_model_args, supported_models
+    cfg, w = weights_of("odd")
+    args = load_model_args(write_checkpoint(tmp_path, cfg, w))
+    assert args.model_type == "femirax" and "femirax" in supported_models()
+    assert args.extra["layers"][0]["mixer"]["right"]["rank"] == 5 and args.rms_norm_eps == cfg["norm"]["eps"]
+    eng = make_engine(tmp_path, cfg, w, ("cpu", "float32"))
+    assert eng.model.kv_layout()[0] == (2, 2, 64) and eng.model.kv_layout()[1] is None
+    # a tensor the model needs is missing: loading says so
+    w2 = dict(w)
+    del w2["l1.mix.g"]
+    with pytest.raises(KeyError):
+        make_engine(tmp_path / "x", cfg, w2, ("cpu", "float32"))
+    bad = json.loads(json.dumps(cfg))
+    bad["layers"][1]["type"] = "convolution"
+    with pytest.raises(ValueError):
+        make_engine(tmp_path / "y", bad, w, ("cpu", "float32"))
