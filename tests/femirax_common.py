@@ -12,7 +12,8 @@ from xllm_b200.utils.loader import save_file
 TARGETS = [pytest.param(("cpu", "float32"), id="cpu-fp32"),
            pytest.param(("cuda:0", "float32"), id="gpu-fp32", marks=pytest.mark.gpu),
            pytest.param(("cuda:0", "bfloat16"), id="gpu-bf16", marks=pytest.mark.gpu)]
-# root mean square of the error over that of the logits
+# root mean square of a row's error over that of the logits; in bfloat16 a row may be off by more where rounding alone
+# (the plain implementation with jittered activations) moves it by more
 LIMIT = {"float32": 2e-4, "bfloat16": 0.06}
 
 
@@ -80,12 +81,35 @@ def random_tokens(n, vocab, seed):
     return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
 
 
-def error(got, want):
-    """Largest row error: rms of the difference (mean taken off) over the rms of all wanted logits."""
+def row_errors(got, want):
+    """rms of every row's difference (mean taken off) over the rms of all wanted logits."""
     d = got.double() - want.double()
     d = d - d.mean(-1, keepdim=True)
     scale = (want - want.mean(-1, keepdim=True)).pow(2).mean().sqrt()
-    return float(d.pow(2).mean(-1).sqrt().max() / scale)
+    return d.pow(2).mean(-1).sqrt() / scale
+
+
+def error(got, want):
+    return float(row_errors(got, want).max())
+
+
+def row_limits(cfg, weights, tokens, want, dtype):
+    """Per place of one sequence: the error a correct implementation may show."""
+    lim = torch.full((len(tokens),), LIMIT[dtype], dtype=torch.float64)
+    if dtype == "bfloat16":
+        for seed in range(24):
+            oracle.NOISE = torch.Generator().manual_seed(seed)
+            try:
+                lim = torch.maximum(lim, 3 * row_errors(expect(cfg, weights, tokens), want))
+            finally:
+                oracle.NOISE = None
+    return lim
+
+
+def close(got, want, limits):
+    """All rows within one and a half times their limit and at most a fiftieth (or one) above it."""
+    r = row_errors(got, want) / limits
+    return bool(r.max() <= 1.5 and int((r > 1).sum()) <= max(1, len(r) // 50)), float(r.max())
 
 
 def feed(engine, rid, tokens, cuts, end=True):

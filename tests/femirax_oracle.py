@@ -9,6 +9,18 @@ import math
 import torch
 
 
+# With a generator here every projection's input and output is multiplied by 1 + 2^-9 randn: what rounding activations
+# to bfloat16 does to an answer (a head whose output nearly vanishes is divided by its tiny root mean square).
+NOISE = None
+
+
+def linear(x, w):
+    if NOISE is None:
+        return x @ w.T
+    jitter = lambda t: t * (1 + 2.0 ** -9 * torch.randn(t.shape, generator=NOISE, dtype=t.dtype))
+    return jitter(jitter(x) @ w.T)
+
+
 # ------------------------------------------------------------------------------------------- mechanisms
 def unit_rms(x, eps):
     """x over its root mean square along the last dimension, eps inside the root."""
@@ -71,36 +83,36 @@ def decayed_state(q, k, v, alpha):
 def retention(h, w, cfg, eps):
     T, H, dk, dv = h.shape[0], cfg["heads"], cfg["dim"], cfg["vdim"]
     rot = cfg["rot"]
-    q = rotate((h @ w["q"].T).view(T, H, dk), rot["base"], rot["dims"], "half")
-    k = rotate((h @ w["k"].T).view(T, H, dk), rot["base"], rot["dims"], "half") * dk ** -0.5
-    v = (h @ w["v"].T).view(T, H, dv)
+    q = rotate(linear(h, w["q"]).view(T, H, dk), rot["base"], rot["dims"], "half")
+    k = rotate(linear(h, w["k"]).view(T, H, dk), rot["base"], rot["dims"], "half") * dk ** -0.5
+    v = linear(h, w["v"]).view(T, H, dv)
     alpha = torch.tensor(cfg["decay"], dtype=h.dtype).view(1, H, 1).expand(T, H, dk)
     o = unit_rms(decayed_state(q, k, v, alpha), eps).reshape(T, H * dv)
-    return (o * silu(h @ w["g"].T)) @ w["o"].T
+    return linear(o * silu(linear(h, w["g"])), w["o"])
 
 
 def key_value_attention(h, w, cfg, eps):
     T, H, G, d = h.shape[0], cfg["heads"], cfg["kv_heads"], cfg["dim"]
     rot = cfg["rot"]
-    raw = (h @ w["k"].T).view(T, G, d)
-    q = unit_rms(rotate((h @ w["q"].T).view(T, H, d), rot["base"], rot["dims"], "pairs"), eps)
+    raw = linear(h, w["k"]).view(T, G, d)
+    q = unit_rms(rotate(linear(h, w["q"]).view(T, H, d), rot["base"], rot["dims"], "pairs"), eps)
     k = unit_rms(rotate(raw, rot["base"], rot["dims"], "pairs"), eps)
-    return causal_attention(q, k, raw, cfg["scale"]).reshape(T, H * d) @ w["o"].T
+    return linear(causal_attention(q, k, raw, cfg["scale"]).reshape(T, H * d), w["o"])
 
 
 def channel_decay(h, a1, a2, b, tau):
-    z = (h @ a1.T) @ a2.T + b
+    z = linear(h, a1) @ a2.T + b
     return (1.0 / (1.0 + torch.exp(-z))) ** (1.0 / tau)
 
 
 def gated_linear(h, w, cfg, eps):
     T, H, dk, dv = h.shape[0], cfg["heads"], cfg["dim"], cfg["vdim"]
-    q = (h @ w["q"].T).view(T, H, dk) * dk ** -0.5
-    k = (h @ w["k"].T).view(T, H, dk)
-    v = (h @ w["v"].T).view(T, H, dv)
+    q = linear(h, w["q"]).view(T, H, dk) * dk ** -0.5
+    k = linear(h, w["k"]).view(T, H, dk)
+    v = linear(h, w["v"]).view(T, H, dv)
     alpha = channel_decay(h, w["a1"], w["a2"], w["a2.b"], cfg["tau"]).view(T, H, dk)
     o = rms_norm(decayed_state(q, k, v, alpha), w["norm"], eps).reshape(T, H * dv)
-    return (o * silu(h @ w["g"].T)) @ w["o"].T
+    return linear(o * silu(linear(h, w["g"])), w["o"])
 
 
 def _sub(w, prefix):
@@ -114,12 +126,12 @@ def parallel(h, w, cfg, eps):
 
 
 def dense_mlp(h, w):
-    return (silu(h @ w["gate"].T) * (h @ w["up"].T)) @ w["down"].T
+    return linear(silu(linear(h, w["gate"])) * linear(h, w["up"]), w["down"])
 
 
 def token_side(x, tokens, table, layer, dim, w, eps):
     e = table[tokens][:, layer * dim:(layer + 1) * dim]
-    y = (gelu_tanh(x @ w["gate"].T) * e) @ w["proj"].T
+    y = linear(gelu_tanh(linear(x, w["gate"])) * e, w["proj"])
     return rms_norm(y, w["norm"], eps)
 
 
@@ -138,7 +150,7 @@ def forward(tokens, config, weights, layers_out=None):
         x = x + token_side(x, tokens, weights["side.embed"], i, sdim, _sub(w, "side."), eps)
         if layers_out is not None:
             layers_out.append(x)
-    return rms_norm(x, weights["final.norm"], eps) @ weights["head"].T
+    return linear(rms_norm(x, weights["final.norm"], eps), weights["head"])
 
 
 def greedy(prompt, n, config, weights):

@@ -158,7 +158,7 @@ __global__ void __launch_bounds__(256) linattn_decode_kernel(LinAttnParams<T> p)
     float a = 0.f;
     for (int w = 0; w < RG; ++w) a += red[w * dvp + i];
     vs[i] = a;                            // v is no longer needed; each thread reads back its own entries
-    ss += a * a;
+    if (i < dv) ss += a * a;
   }
   float inv = 1.f;
   if (p.unit_norm) inv = 1.f / sqrtf(block_sum(ss, red32) / (float)dv + p.eps);
