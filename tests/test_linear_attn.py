@@ -136,6 +136,33 @@ def test_linear_attention(name, target):
     c.check(c.step(p, decode=True), p, tol * 2)
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("length", [16, 48, 128])
+@pytest.mark.parametrize("name", ["r64", "r_odd", "r_wide", "c64", "c_odd", "c_resets"])
+def test_segments_side_by_side(name, length, monkeypatch):
+    """Long prompts run as segments with a scan over their states; borders of segments, several sequences of unequal
+    numbers of segments, continued from a state, and the state they leave."""
+    lens = (150, 16, 1, 97)
+    c = Case(("cuda", torch.bfloat16), lens=lens, seed=2, **SIZES[name])
+
+    def segments(self, T, n_seqs, max_q_len, device):
+        segs = -(-max_q_len // length)
+        m = T // length + n_seqs + 1
+        nan = float("nan")
+        return (torch.full((m, self.heads, self.dk, (self.dv + 3) // 4 * 4), nan, device=device),
+                torch.full((m, self.heads, self.dk), nan, device=device), length, segs)
+
+    monkeypatch.setattr(LinearAttention, "_segments", segments)
+    p = [(s, 0, n) for s, n in enumerate(lens)]
+    c.check(c.step(p, max_q_len=150), p, 4e-3)
+    p = [(0, 0, 100), (3, 0, 31)]
+    c.check(c.step(p, max_q_len=100), p, 4e-3)
+    p = [(3, 31, 96), (0, 100, 149)]
+    c.check(c.step(p, max_q_len=65), p, 6e-3)
+    p = [(0, 149, 150), (3, 96, 97)]
+    c.check(c.step(p, decode=True), p, 8e-3)
+
+
 @pytest.mark.parametrize("target", TARGETS)
 @pytest.mark.parametrize("name", ["r64", "c64", "c_resets"])
 def test_token_by_token_form(name, target):

@@ -249,22 +249,38 @@ __global__ void __launch_bounds__(256) linattn_recurrent_kernel(LinAttnParams<T>
 }
 
 // ------------------------------------------------------------------------------------------------ chunks of 16 tokens
+// A prompt of several segments runs as three launches: the state every segment adds on its own (STATE_ONLY, from zero),
+// a scan over the segments' states, and the outputs of all segments side by side, each from its start state.  A prompt
+// of one segment needs the last launch only.
 constexpr int kLC = 16;                     // tokens per chunk
-constexpr float kLogRange = 60.f;           // |log decay| between a chunk's ends and its reference token
+constexpr float kLogRange = 86.f;           // |log2 decay| between a chunk's ends and its reference token
+
+struct SegParams {
+  float* state;      // [slot][H][dk][dv_pad]: local states, then (after the scan) start states; null: one segment
+  float* decay;      // [slot][H][dk]: decay over a segment
+  int len;           // tokens per segment (multiple of 16)
+  void* fused_out;   // bf16 [T, out_ld], finished rows (dv fits one CTA), or null: raw fp32 to out
+  int64_t out_ld;
+};
+
+// slots of the segments of sequence b: unique because a sequence of n rows has at most n / len + 1 whole segments
+__device__ __forceinline__ int64_t seg_slot(int row0, int b, int s, int len) { return (int64_t)row0 / len + b + s; }
 
 template <int DK, int NW>
 struct ChunkSmem {
   static constexpr int VC = NW * 16;        // value columns per CTA
   static constexpr int VCP = VC < 64 ? 64 : VC;
-  static constexpr int tile = kLC * DK * 2;
-  static constexpr int qhi = 0, qlo = tile, khi = 2 * tile, klo = 3 * tile;
+  static constexpr int tile = kLC * DK * 2, vtile = kLC * VCP * 2;
+  static constexpr int khi = 0, klo = tile, qhi = 2 * tile, qlo = 3 * tile;
   static constexpr int v = 4 * tile;                       // 2 x [16][VCP] swizzled
-  static constexpr int raw = v + 2 * kLC * VCP * 2;        // 2 x (q, k) [16][DK]
-  static constexpr int lw = raw + 4 * tile;                // [16][DK] fp32
-  static constexpr int fs = lw + kLC * DK * 4;             // [DK] scale of the state rows
+  static constexpr int g = v + 2 * vtile;                  // 2 x [16][VCP] plain
+  static constexpr int raw = g + 2 * vtile;                // 2 x (q, k) [16][DK]
+  static constexpr int fs = raw + 4 * tile;                // [DK] scale of the state rows
   static constexpr int et = fs + DK * 4;                   // [DK] decay from the reference token to the chunk's end
-  static constexpr int bias = et + DK * 4;                 // [DK]
-  static constexpr int dyn = bias + DK * 4;                // cos | sin 2 x [16][rot], raw r 2 x [16][RP], a2 [DK][RP + 8]
+  static constexpr int tot = et + DK * 4;                  // [DK] log2 decay over the segment so far
+  static constexpr int ssm = tot + DK * 4;                 // [NW][16] partial sums of squares
+  static constexpr int dyn = ssm + NW * kLC * 4;
+  // dyn: cos | sin 2 x [16][rot] fp32; channel decay: lw [16][DK] fp32, bias [DK], raw r 2 x [16][RP], a2 [DK][RP + 8]
 };
 
 __device__ __forceinline__ void split_pack(float a, float b, uint32_t& hi, uint32_t& lo) {
@@ -274,39 +290,47 @@ __device__ __forceinline__ void split_pack(float a, float b, uint32_t& hi, uint3
   hi = *reinterpret_cast<const uint32_t*>(&h);
   lo = *reinterpret_cast<const uint32_t*>(&l);
 }
+__device__ __forceinline__ float2 unpack2(uint32_t u) { return __bfloat1622float2(*reinterpret_cast<const bf162*>(&u)); }
 
-template <int DK, int NW>
-__global__ void __launch_bounds__(NW * 32) linattn_chunk_kernel(LinAttnParams<bf16> p) {
+template <int DK, int NW, bool STATE_ONLY>
+__global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 512 / (NW * 32)) linattn_chunk_kernel(LinAttnParams<bf16> p, SegParams sp) {
   using L = ChunkSmem<DK, NW>;
   constexpr int CH = DK / 8, VCH = L::VCP / 8, NT = NW * 32;
   extern __shared__ __align__(128) uint8_t smem[];
   const uint32_t sb = smem_u32(smem);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int h = blockIdx.x, b = blockIdx.y, c0 = blockIdx.z * L::VC;
+  const int h = blockIdx.x, b = blockIdx.y;
+  const int slices = (p.dv + L::VC - 1) / L::VC;
+  const int seg = blockIdx.z / slices, c0 = (blockIdx.z - seg * slices) * L::VC;
   const int dk = p.dk, rot = p.cos_sin != nullptr ? p.rot : 0;
   const bool channel = p.log_decay == nullptr;
   const int RP = channel ? (p.rank + 15) & ~15 : 0, A2S = RP + 8;
-  float* lw = reinterpret_cast<float*>(smem + L::lw);
   float* fs = reinterpret_cast<float*>(smem + L::fs);
   float* et = reinterpret_cast<float*>(smem + L::et);
-  float* bias = reinterpret_cast<float*>(smem + L::bias);
+  float* tot = reinterpret_cast<float*>(smem + L::tot);
+  float* ssm = reinterpret_cast<float*>(smem + L::ssm);
   float* csb = reinterpret_cast<float*>(smem + L::dyn);                       // [2][16][rot]
-  bf16* rb = reinterpret_cast<bf16*>(smem + L::dyn + 2 * kLC * rot * 4);      // [2][16][RP]
+  float* lw = csb + 2 * kLC * rot;                                            // [16][DK]
+  float* bias = lw + (channel ? kLC * DK : 0);
+  bf16* rb = reinterpret_cast<bf16*>(bias + (channel ? DK : 0));              // [2][16][RP]
   bf16* a2s = rb + 2 * kLC * RP;                                              // [DK][A2S]
   __shared__ float elog[2 * kLC];
   pdl_wait();
   pdl_launch_dependents();
-  const int row0 = p.cu_q[b], n_all = p.cu_q[b + 1] - row0;
+  const int row_first = p.cu_q[b], n_seq = p.cu_q[b + 1] - row_first;
   const int slot = p.slots[b];
-  if (n_all <= 0 || slot < 0) return;
-  const bool fresh = p.kv_lens[b] == n_all;
-  const float lg = channel ? 0.f : fmaxf(p.log_decay[h], -1e4f);
+  if (n_seq <= 0 || slot < 0 || seg * sp.len >= n_seq) return;
+  const int row0 = row_first + seg * sp.len, n_all = min(sp.len, n_seq - seg * sp.len);
+  const bool one_seg = sp.state == nullptr;
+  const bool fresh = STATE_ONLY || (one_seg && p.kv_lens[b] == n_seq);
+  const float lg = channel ? 0.f : fmaxf(p.log_decay[h], -1e4f) * 1.44269504088896341f;    // log2 of the constant decay
 
   // ---- state columns of this warp: acc[nt] holds S^T rows (value columns) lane/4, +8 and key channels nt*8 + ..
   float acc[DK / 8][4];
   const int vrow = c0 + warp * 16 + (lane >> 2);
   const bool has_cols = c0 + warp * 16 < p.dv;
-  float* S = p.state + (((int64_t)slot * p.H + h) * dk) * p.dv_pad;
+  const int64_t seg_at = one_seg ? 0 : seg_slot(row_first, b, seg, sp.len) * p.H + h;
+  float* S = one_seg ? p.state + (((int64_t)slot * p.H + h) * dk) * p.dv_pad : sp.state + seg_at * dk * p.dv_pad;
 #pragma unroll
   for (int nt = 0; nt < DK / 8; ++nt) {
 #pragma unroll
@@ -317,7 +341,8 @@ __global__ void __launch_bounds__(NW * 32) linattn_chunk_kernel(LinAttnParams<bf
   }
   for (int i = tid; i < DK; i += NT) {
     et[i] = 1.f;
-    bias[i] = (channel && i < dk) ? __bfloat162float(p.a2_b[(int64_t)h * dk + i]) : 0.f;
+    tot[i] = 0.f;
+    if (channel) bias[i] = i < dk ? __bfloat162float(p.a2_b[(int64_t)h * dk + i]) : 0.f;
   }
   if (channel) {
     for (int i = tid; i < DK * RP; i += NT) {
@@ -325,27 +350,28 @@ __global__ void __launch_bounds__(NW * 32) linattn_chunk_kernel(LinAttnParams<bf
       a2s[c * A2S + j] = (c < dk && j < p.rank) ? p.a2[((int64_t)h * dk + c) * p.rank + j] : __float2bfloat16(0.f);
     }
   } else {
-    // powers of the head's constant: elog[16 + i] = decay^i
-    if (tid < 2 * kLC) elog[tid] = expf((float)(tid - kLC) * lg);
+    if (tid < 2 * kLC) elog[tid] = exp2f((float)(tid - kLC) * lg);      // elog[16 + i] = decay^i
   }
 
-  const auto load_raw = [&](int t0, int buf) {              // 16 token rows from t0 (of this sequence)
-    uint8_t* raw = smem + L::raw + buf * 2 * L::tile;
-    const uint32_t raws = sb + L::raw + buf * 2 * L::tile, vsm = sb + L::v + buf * kLC * L::VCP * 2;
+  const auto load_raw = [&](int t0, int buf) {              // 16 token rows from t0 (of this segment)
+    const uint32_t raws = sb + L::raw + buf * 2 * L::tile, vsm = sb + L::v + buf * L::vtile, gsm = sb + L::g + buf * L::vtile;
     const int64_t base = (int64_t)(row0 + t0);
+    const bool gate = !STATE_ONLY && sp.fused_out != nullptr && p.g != nullptr;
     if (p.vec_ok) {
       const int per = dk >> 3;
       for (int i = tid; i < kLC * per; i += NT) {
         const int r = i / per, c = i - r * per;
         const bool ok = t0 + r < n_all;
         const int64_t go = (base + (ok ? r : 0)) * p.ld + (int64_t)h * dk + c * 8;
-        cp_async16(raws + (r * DK + c * 8) * 2, p.q + go, ok);
+        if (!STATE_ONLY) cp_async16(raws + (r * DK + c * 8) * 2, p.q + go, ok);
         cp_async16(raws + L::tile + (r * DK + c * 8) * 2, p.k + go, ok);
       }
       for (int i = tid; i < kLC * (L::VC / 8); i += NT) {
         const int r = i / (L::VC / 8), c = i - r * (L::VC / 8);
         const bool ok = t0 + r < n_all && c0 + c * 8 < p.dv;
-        cp_async16(vsm + swz<VCH>(r, c), ok ? p.v + (base + r) * p.ld + (int64_t)h * p.dv + c0 + c * 8 : p.v, ok);
+        const int64_t go = ok ? (base + r) * p.ld + (int64_t)h * p.dv + c0 + c * 8 : 0;
+        cp_async16(vsm + swz<VCH>(r, c), p.v + go, ok);
+        if (gate) cp_async16(gsm + (r * L::VCP + c * 8) * 2, p.g + go, ok);
       }
       if (channel) {
         const int pr = RP >> 3;
@@ -356,7 +382,7 @@ __global__ void __launch_bounds__(NW * 32) linattn_chunk_kernel(LinAttnParams<bf
         }
       }
     } else {
-      bf16* rq = reinterpret_cast<bf16*>(raw);
+      bf16* rq = reinterpret_cast<bf16*>(smem + L::raw + buf * 2 * L::tile);
       const bf16 zero = __float2bfloat16(0.f);
       for (int i = tid; i < kLC * dk; i += NT) {
         const int r = i / dk, c = i - r * dk;
@@ -368,8 +394,9 @@ __global__ void __launch_bounds__(NW * 32) linattn_chunk_kernel(LinAttnParams<bf
       for (int i = tid; i < kLC * L::VC; i += NT) {
         const int r = i / L::VC, c = i - r * L::VC;
         const bool ok = t0 + r < n_all && c0 + c < p.dv;
-        *reinterpret_cast<bf16*>(smem + L::v + buf * kLC * L::VCP * 2 + swz<VCH>(r, c >> 3) + (c & 7) * 2) =
-            ok ? p.v[(base + r) * p.ld + (int64_t)h * p.dv + c0 + c] : zero;
+        const int64_t go = ok ? (base + r) * p.ld + (int64_t)h * p.dv + c0 + c : 0;
+        *reinterpret_cast<bf16*>(smem + L::v + buf * L::vtile + swz<VCH>(r, c >> 3) + (c & 7) * 2) = ok ? p.v[go] : zero;
+        if (gate) reinterpret_cast<bf16*>(smem + L::g + buf * L::vtile)[r * L::VCP + c] = ok ? p.g[go] : zero;
       }
       for (int i = tid; i < kLC * RP; i += NT) {
         const int r = i / RP, c = i - r * RP;
@@ -395,8 +422,8 @@ __global__ void __launch_bounds__(NW * 32) linattn_chunk_kernel(LinAttnParams<bf
     }
     cp_async_commit();
   };
+  const bool by_four = dk % 4 == 0 && rot % 4 == 0;       // four channels of a token at a time
 
-  float* out = reinterpret_cast<float*>(p.out);
   load_raw(0, 0);
   int buf = 0;
   for (int t0 = 0; t0 < n_all; t0 += kLC, buf ^= 1) {
@@ -407,10 +434,11 @@ __global__ void __launch_bounds__(NW * 32) linattn_chunk_kernel(LinAttnParams<bf
     const bf16* rq = reinterpret_cast<const bf16*>(smem + L::raw + buf * 2 * L::tile);
     const bf16* rk = rq + kLC * DK;
 
-    // ---- cumulative log decays of the chunk (channel decay)
+    // ---- cumulative log2 decays of the chunk (channel decay): z on the tensor cores, the sum over tokens by shuffles
     bool unsafe = false;
     if (channel) {
       const bf16* r = rb + buf * kLC * RP;
+      const int ref = n >> 1;
       for (int nt = warp; nt < DK / 8; nt += NW) {
         float z[4];
         const int c = nt * 8 + (lane & 3) * 2;
@@ -426,22 +454,30 @@ __global__ void __launch_bounds__(NW * 32) linattn_chunk_kernel(LinAttnParams<bf
           const bf16* w = a2s + (nt * 8 + (lane >> 2)) * A2S + k0;
           mma_bf16_16816(z, a, *reinterpret_cast<const uint32_t*>(w), *reinterpret_cast<const uint32_t*>(w + 8));
         }
+        const int ta = lane >> 2;
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int t = (lane >> 2) + (e >> 1) * 8;
-          lw[t * DK + c + (e & 1)] = t < n ? log_sigmoid(z[e]) * p.inv_tau : 0.f;
-        }
-      }
-      __syncthreads();
-      for (int c = tid; c < DK; c += NT) {
-        float s = 0.f;
+        for (int e = 0; e < 4; ++e)
+          z[e] = ta + (e >> 1) * 8 < n ? log_sigmoid(z[e]) * (p.inv_tau * 1.44269504088896341f) : 0.f;
 #pragma unroll
-        for (int t = 0; t < kLC; ++t) {
-          s += lw[t * DK + c];
-          lw[t * DK + c] = s;
+        for (int d = 4; d < 32; d <<= 1) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float up = __shfl_up_sync(0xffffffffu, z[e], d);
+            if (lane >= d) z[e] += up;
+          }
         }
-        const float m = lw[(n >> 1) * DK + c];
-        if (c < dk && (lw[c] - m > kLogRange || m - s > kLogRange)) unsafe = true;
+        z[2] += __shfl_sync(0xffffffffu, z[0], 28 + (lane & 3));
+        z[3] += __shfl_sync(0xffffffffu, z[1], 28 + (lane & 3));
+        *reinterpret_cast<float2*>(lw + ta * DK + c) = make_float2(z[0], z[1]);
+        *reinterpret_cast<float2*>(lw + (ta + 8) * DK + c) = make_float2(z[2], z[3]);
+        const int rl = (ref & 7) * 4 + (lane & 3);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float m0 = __shfl_sync(0xffffffffu, z[e], rl), m1 = __shfl_sync(0xffffffffu, z[e + 2], rl);
+          const float m = ref < 8 ? m0 : m1;
+          // (the first token's lane, the last token's lane) see the extremes: the sums fall monotonically
+          if (c + e < dk && ((lane < 4 && z[e] - m > kLogRange) || (lane >= 28 && m - z[e + 2] > kLogRange))) unsafe = true;
+        }
       }
     } else {
       unsafe = -lg * (float)kLC > kLogRange;
@@ -453,139 +489,302 @@ __global__ void __launch_bounds__(NW * 32) linattn_chunk_kernel(LinAttnParams<bf
       const int s1 = s0 + step, ref = s0 + (step >> 1);
       if (s0 > 0) __syncthreads();
       // ---- operand tiles: q and k rotated, scaled, and multiplied by their decay against token `ref`
-      for (int i = tid; i < kLC * (DK / 2); i += NT) {
-        const int t = i / (DK / 2), c = (i - t * (DK / 2)) * 2;
-        float qv[2] = {0.f, 0.f}, kv[2] = {0.f, 0.f};
-        if (t >= s0 && t < s1 && c < dk) {
-          const float* cs = rot > 0 ? csb + (buf * kLC + t) * rot : nullptr;
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            if (c + e >= dk) break;
-            float eq, ek;
-            if (channel) {
-              const float d = lw[t * DK + c + e] - lw[ref * DK + c + e];
-              eq = expf(d);
-              ek = expf(-d);
-            } else {
-              eq = step == 1 ? 1.f : elog[kLC + t - ref];
-              ek = step == 1 ? 1.f : elog[kLC + ref - t];
+      if (by_four) {
+        const int half = rot >> 1, r4 = rot >> 2;
+        for (int i = tid; i < kLC * (DK / 4); i += NT) {
+          const int t = i / (DK / 4), m = i - t * (DK / 4);
+          const bool turns = m < r4, split = turns && !p.interleaved;
+          const int ca = split ? 2 * m : 4 * m, cb = split ? 2 * m + half : 4 * m + 2;     // two channels each
+          float k4[4] = {0.f, 0.f, 0.f, 0.f}, q4[4] = {0.f, 0.f, 0.f, 0.f};
+          if (t >= s0 && t < s1 && 4 * m < dk) {
+            const float2 ka = unpack2(*reinterpret_cast<const uint32_t*>(rk + t * DK + ca));
+            const float2 kb = unpack2(*reinterpret_cast<const uint32_t*>(rk + t * DK + cb));
+            k4[0] = ka.x; k4[1] = ka.y; k4[2] = kb.x; k4[3] = kb.y;
+            if (!STATE_ONLY) {
+              const float2 qa = unpack2(*reinterpret_cast<const uint32_t*>(rq + t * DK + ca));
+              const float2 qb = unpack2(*reinterpret_cast<const uint32_t*>(rq + t * DK + cb));
+              q4[0] = qa.x; q4[1] = qa.y; q4[2] = qb.x; q4[3] = qb.y;
             }
-            qv[e] = rotated(rq + t * DK, c + e, rot, p.interleaved, cs) * p.q_scale * eq;
-            kv[e] = rotated(rk + t * DK, c + e, rot, p.interleaved, cs) * p.k_scale * ek;
+            if (turns) {
+              const float* cs = csb + (buf * kLC + t) * rot;
+              const float2 co = *reinterpret_cast<const float2*>(cs + 2 * m);
+              const float2 si = *reinterpret_cast<const float2*>(cs + half + 2 * m);
+              const auto turn = [&](float* x) {
+                const float x0 = x[0], x1 = x[1], x2 = x[2], x3 = x[3];
+                if (split) {                 // partners (0, 2) and (1, 3)
+                  x[0] = x0 * co.x - x2 * si.x; x[2] = x2 * co.x + x0 * si.x;
+                  x[1] = x1 * co.y - x3 * si.y; x[3] = x3 * co.y + x1 * si.y;
+                } else {                     // partners (0, 1) and (2, 3)
+                  x[0] = x0 * co.x - x1 * si.x; x[1] = x1 * co.x + x0 * si.x;
+                  x[2] = x2 * co.y - x3 * si.y; x[3] = x3 * co.y + x2 * si.y;
+                }
+              };
+              turn(k4);
+              if (!STATE_ONLY) turn(q4);
+            }
+            if (channel) {
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const int c = (e < 2 ? ca : cb) + (e & 1);
+                const float d = lw[t * DK + c] - lw[ref * DK + c];
+                k4[e] *= p.k_scale * exp2f(-d);
+                if (!STATE_ONLY) q4[e] *= p.q_scale * exp2f(d);
+              }
+            } else {
+              const float fk = p.k_scale * (step == 1 ? 1.f : elog[kLC + ref - t]);
+              const float fq = p.q_scale * (step == 1 ? 1.f : elog[kLC + t - ref]);
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                k4[e] *= fk;
+                q4[e] *= fq;
+              }
+            }
+          }
+          const uint32_t oa = swz<CH>(t, ca >> 3) + (ca & 7) * 2, ob = swz<CH>(t, cb >> 3) + (cb & 7) * 2;
+          uint32_t hi, lo;
+          split_pack(k4[0], k4[1], hi, lo);
+          *reinterpret_cast<uint32_t*>(smem + L::khi + oa) = hi;
+          *reinterpret_cast<uint32_t*>(smem + L::klo + oa) = lo;
+          split_pack(k4[2], k4[3], hi, lo);
+          *reinterpret_cast<uint32_t*>(smem + L::khi + ob) = hi;
+          *reinterpret_cast<uint32_t*>(smem + L::klo + ob) = lo;
+          if (!STATE_ONLY) {
+            split_pack(q4[0], q4[1], hi, lo);
+            *reinterpret_cast<uint32_t*>(smem + L::qhi + oa) = hi;
+            *reinterpret_cast<uint32_t*>(smem + L::qlo + oa) = lo;
+            split_pack(q4[2], q4[3], hi, lo);
+            *reinterpret_cast<uint32_t*>(smem + L::qhi + ob) = hi;
+            *reinterpret_cast<uint32_t*>(smem + L::qlo + ob) = lo;
           }
         }
-        uint32_t qh, ql, kh, kl;
-        split_pack(qv[0], qv[1], qh, ql);
-        split_pack(kv[0], kv[1], kh, kl);
-        const uint32_t o = swz<CH>(t, c >> 3) + (c & 7) * 2;
-        *reinterpret_cast<uint32_t*>(smem + L::qhi + o) = qh;
-        *reinterpret_cast<uint32_t*>(smem + L::qlo + o) = ql;
-        *reinterpret_cast<uint32_t*>(smem + L::khi + o) = kh;
-        *reinterpret_cast<uint32_t*>(smem + L::klo + o) = kl;
+      } else {
+        for (int i = tid; i < kLC * (DK / 2); i += NT) {
+          const int t = i / (DK / 2), c = (i - t * (DK / 2)) * 2;
+          float qv[2] = {0.f, 0.f}, kv[2] = {0.f, 0.f};
+          if (t >= s0 && t < s1 && c < dk) {
+            const float* cs = rot > 0 ? csb + (buf * kLC + t) * rot : nullptr;
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              if (c + e >= dk) break;
+              float eq = 1.f, ek = 1.f;
+              if (channel) {
+                const float d = lw[t * DK + c + e] - lw[ref * DK + c + e];
+                eq = exp2f(d);
+                ek = exp2f(-d);
+              } else if (step > 1) {
+                eq = elog[kLC + t - ref];
+                ek = elog[kLC + ref - t];
+              }
+              qv[e] = rotated(rq + t * DK, c + e, rot, p.interleaved, cs) * p.q_scale * eq;
+              kv[e] = rotated(rk + t * DK, c + e, rot, p.interleaved, cs) * p.k_scale * ek;
+            }
+          }
+          uint32_t qh, ql, kh, kl;
+          split_pack(qv[0], qv[1], qh, ql);
+          split_pack(kv[0], kv[1], kh, kl);
+          const uint32_t o = swz<CH>(t, c >> 3) + (c & 7) * 2;
+          *reinterpret_cast<uint32_t*>(smem + L::khi + o) = kh;
+          *reinterpret_cast<uint32_t*>(smem + L::klo + o) = kl;
+          *reinterpret_cast<uint32_t*>(smem + L::qhi + o) = qh;
+          *reinterpret_cast<uint32_t*>(smem + L::qlo + o) = ql;
+        }
       }
       for (int c = tid; c < DK; c += NT) {
-        float eref, eend;
+        float lref, lend;                     // log2 decay: state -> reference token, reference token -> end
         if (channel) {
           const float m = lw[ref * DK + c];
-          eref = expf(m - (s0 > 0 ? lw[(s0 - 1) * DK + c] : 0.f));
-          eend = expf(lw[(s1 - 1) * DK + c] - m);
+          lref = m - (s0 > 0 ? lw[(s0 - 1) * DK + c] : 0.f);
+          lend = lw[(s1 - 1) * DK + c] - m;
         } else {
-          eref = expf((float)(ref - s0 + 1) * lg);
-          eend = expf((float)(s1 - 1 - ref) * lg);
+          lref = (float)(ref - s0 + 1) * lg;
+          lend = (float)(s1 - 1 - ref) * lg;
         }
-        fs[c] = et[c] * eref;
-        et[c] = eend;
+        fs[c] = et[c] * exp2f(lref);
+        et[c] = exp2f(lend);
+        tot[c] += lref + lend;
       }
       __syncthreads();
-      if (!has_cols) continue;
 
       // ---- O = Q S + mask(Q K^T) V ;  S^T += V^T K
-      float oh[2][4], ol[2][4], ph[2][4], pl[2][4];
+      const int arow = (lane & 7) + (((lane >> 3) & 1) << 3), acb = lane >> 4;
+      float o[2][4];
 #pragma unroll
       for (int j = 0; j < 2; ++j)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) oh[j][e] = ol[j][e] = ph[j][e] = pl[j][e] = 0.f;
-      const int arow = (lane & 7) + (((lane >> 3) & 1) << 3), acb = lane >> 4;
-      const int brow = (lane & 7) + ((lane >> 4) << 3), bcb = (lane >> 3) & 1;
+        for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
+      if (has_cols) {
+        uint32_t v0, v1, v2, v3;
+        ldmatrix_x4_trans(v0, v1, v2, v3, sb + L::v + buf * L::vtile + swz<VCH>(arow, warp * 2 + acb));
+        if (!STATE_ONLY) {
+          float pw[2][4];
 #pragma unroll
-      for (int kk = 0; kk < DK / 16; ++kk) {
-        uint32_t qh[4], ql[4], kh[4], kl[4];
-        const uint32_t ao = swz<CH>(arow, kk * 2 + acb), bo = swz<CH>(brow, kk * 2 + bcb);
-        ldmatrix_x4(qh[0], qh[1], qh[2], qh[3], sb + L::qhi + ao);
-        ldmatrix_x4(ql[0], ql[1], ql[2], ql[3], sb + L::qlo + ao);
-        ldmatrix_x4(kh[0], kh[1], kh[2], kh[3], sb + L::khi + bo);
-        ldmatrix_x4(kl[0], kl[1], kl[2], kl[3], sb + L::klo + bo);
-        const float2 f0 = *reinterpret_cast<const float2*>(fs + kk * 16 + (lane & 3) * 2);
-        const float2 f1 = *reinterpret_cast<const float2*>(fs + kk * 16 + 8 + (lane & 3) * 2);
+          for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) pw[j][e] = 0.f;
+          const int brow = (lane & 7) + ((lane >> 4) << 3), bcb = (lane >> 3) & 1;
+#pragma unroll
+          for (int kk = 0; kk < DK / 16; ++kk) {
+            uint32_t qh[4], ql[4], kh[4], kl[4];
+            const uint32_t ao = swz<CH>(arow, kk * 2 + acb), bo = swz<CH>(brow, kk * 2 + bcb);
+            ldmatrix_x4(qh[0], qh[1], qh[2], qh[3], sb + L::qhi + ao);
+            ldmatrix_x4(ql[0], ql[1], ql[2], ql[3], sb + L::qlo + ao);
+            ldmatrix_x4(kh[0], kh[1], kh[2], kh[3], sb + L::khi + bo);
+            ldmatrix_x4(kl[0], kl[1], kl[2], kl[3], sb + L::klo + bo);
+            const float2 f0 = *reinterpret_cast<const float2*>(fs + kk * 16 + (lane & 3) * 2);
+            const float2 f1 = *reinterpret_cast<const float2*>(fs + kk * 16 + 8 + (lane & 3) * 2);
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+              float* x = acc[2 * kk] + 2 * j;
+              float* y = acc[2 * kk + 1] + 2 * j;
+              x[0] *= f0.x; x[1] *= f0.y;
+              y[0] *= f1.x; y[1] *= f1.y;
+              uint32_t bh0, bl0, bh1, bl1;
+              split_pack(x[0], x[1], bh0, bl0);
+              split_pack(y[0], y[1], bh1, bl1);
+              mma_bf16_16816(o[j], qh, bh0, bh1);
+              mma_bf16_16816(pw[j], qh, kh[2 * j], kh[2 * j + 1]);
+              mma_bf16_16816(o[j], ql, bh0, bh1);
+              mma_bf16_16816(pw[j], ql, kh[2 * j], kh[2 * j + 1]);
+              mma_bf16_16816(o[j], qh, bl0, bl1);
+              mma_bf16_16816(pw[j], qh, kl[2 * j], kl[2 * j + 1]);
+            }
+          }
+#pragma unroll
+          for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const int s = j * 8 + (lane & 3) * 2 + (e & 1), t = (lane >> 2) + (e >> 1) * 8;
+              if (s > t) pw[j][e] = 0.f;
+            }
+          uint32_t pa[4], pb[4];
+          split_pack(pw[0][0], pw[0][1], pa[0], pb[0]);
+          split_pack(pw[0][2], pw[0][3], pa[1], pb[1]);
+          split_pack(pw[1][0], pw[1][1], pa[2], pb[2]);
+          split_pack(pw[1][2], pw[1][3], pa[3], pb[3]);
+          mma_bf16_16816(o[0], pa, v0, v1);
+          mma_bf16_16816(o[1], pa, v2, v3);
+          mma_bf16_16816(o[0], pb, v0, v1);
+          mma_bf16_16816(o[1], pb, v2, v3);
+        } else {
+#pragma unroll
+          for (int nt = 0; nt < DK / 8; ++nt) {
+            const float2 f = *reinterpret_cast<const float2*>(fs + nt * 8 + (lane & 3) * 2);
+            acc[nt][0] *= f.x; acc[nt][1] *= f.y; acc[nt][2] *= f.x; acc[nt][3] *= f.y;
+          }
+        }
+        const uint32_t va[4] = {v0, v2, v1, v3};
+#pragma unroll
+        for (int kk = 0; kk < DK / 16; ++kk) {
+          uint32_t kh[4], kl[4];
+          const uint32_t ko = swz<CH>(arow, kk * 2 + acb);
+          ldmatrix_x4_trans(kh[0], kh[1], kh[2], kh[3], sb + L::khi + ko);
+          ldmatrix_x4_trans(kl[0], kl[1], kl[2], kl[3], sb + L::klo + ko);
+          mma_bf16_16816(acc[2 * kk], va, kh[0], kh[1]);
+          mma_bf16_16816(acc[2 * kk + 1], va, kh[2], kh[3]);
+          mma_bf16_16816(acc[2 * kk], va, kl[0], kl[1]);
+          mma_bf16_16816(acc[2 * kk + 1], va, kl[2], kl[3]);
+        }
+      }
+      if (STATE_ONLY) continue;
+      // ---- rows out: raw, or finished (norm over the head, weight, gate) when this CTA holds all of the head
+      if (sp.fused_out == nullptr) {
+        if (!has_cols) continue;
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int t = (lane >> 2) + (e >> 1) * 8, c = c0 + warp * 16 + j * 8 + (lane & 3) * 2 + (e & 1);
+            if (t >= s0 && t < s1 && c < p.dv)
+              reinterpret_cast<float*>(p.out)[((int64_t)(row0 + t0 + t) * p.H + h) * p.dv + c] = o[j][e];
+          }
+        continue;
+      }
+      if (p.unit_norm) {
+        float sa = o[0][0] * o[0][0] + o[0][1] * o[0][1] + o[1][0] * o[1][0] + o[1][1] * o[1][1];
+        float sc = o[0][2] * o[0][2] + o[0][3] * o[0][3] + o[1][2] * o[1][2] + o[1][3] * o[1][3];
+        sa += __shfl_xor_sync(0xffffffffu, sa, 1);
+        sa += __shfl_xor_sync(0xffffffffu, sa, 2);
+        sc += __shfl_xor_sync(0xffffffffu, sc, 1);
+        sc += __shfl_xor_sync(0xffffffffu, sc, 2);
+        if ((lane & 3) == 0) {
+          ssm[warp * kLC + (lane >> 2)] = sa;
+          ssm[warp * kLC + (lane >> 2) + 8] = sc;
+        }
+        __syncthreads();
+      }
+      const bf16* gs = reinterpret_cast<const bf16*>(smem + L::g + buf * L::vtile);
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const int t = (lane >> 2) + u * 8;
+        float inv = 1.f;
+        if (p.unit_norm) {
+          float ss = 0.f;
+#pragma unroll
+          for (int w = 0; w < NW; ++w) ss += ssm[w * kLC + t];
+          inv = 1.f / sqrtf(ss / (float)p.dv + p.eps);
+        }
+        if (t < s0 || t >= s1) continue;
+        bf16* orow = reinterpret_cast<bf16*>(sp.fused_out) + (int64_t)(row0 + t0 + t) * sp.out_ld + (int64_t)h * p.dv;
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
-          float* x = acc[2 * kk] + 2 * j;
-          float* y = acc[2 * kk + 1] + 2 * j;
-          x[0] *= f0.x; x[1] *= f0.y;
-          y[0] *= f1.x; y[1] *= f1.y;
-          uint32_t bh0, bl0, bh1, bl1;
-          split_pack(x[0], x[1], bh0, bl0);
-          split_pack(y[0], y[1], bh1, bl1);
-          mma_bf16_16816(oh[j], qh, bh0, bh1);
-          mma_bf16_16816(ol[j], ql, bh0, bh1);
-          mma_bf16_16816(ol[j], qh, bl0, bl1);
-          mma_bf16_16816(ph[j], qh, kh[2 * j], kh[2 * j + 1]);
-          mma_bf16_16816(pl[j], ql, kh[2 * j], kh[2 * j + 1]);
-          mma_bf16_16816(pl[j], qh, kl[2 * j], kl[2 * j + 1]);
+          float y[2];
+          const int c = warp * 16 + j * 8 + (lane & 3) * 2;
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            y[e] = 0.f;
+            if (c + e >= p.dv) continue;
+            y[e] = o[j][u * 2 + e] * inv;
+            if (p.norm_w != nullptr) y[e] *= __bfloat162float(p.norm_w[c + e]);
+            if (p.g != nullptr) y[e] *= silu_f32(__bfloat162float(gs[t * L::VCP + c + e]));
+          }
+          if (p.vec_ok && c + 1 < p.dv) {
+            *reinterpret_cast<bf162*>(orow + c) = __floats2bfloat162_rn(y[0], y[1]);
+          } else {
+            if (c < p.dv) orow[c] = __float2bfloat16(y[0]);
+            if (c + 1 < p.dv) orow[c + 1] = __float2bfloat16(y[1]);
+          }
         }
       }
-#pragma unroll
-      for (int j = 0; j < 2; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int s = j * 8 + (lane & 3) * 2 + (e & 1), t = (lane >> 2) + (e >> 1) * 8;
-          ph[j][e] = s <= t ? ph[j][e] + pl[j][e] : 0.f;
-        }
-      uint32_t v0, v1, v2, v3;
-      ldmatrix_x4_trans(v0, v1, v2, v3, sb + L::v + buf * kLC * L::VCP * 2 + swz<VCH>(arow, warp * 2 + acb));
-      {
-        uint32_t pa[4], pb[4];
-        split_pack(ph[0][0], ph[0][1], pa[0], pb[0]);
-        split_pack(ph[0][2], ph[0][3], pa[1], pb[1]);
-        split_pack(ph[1][0], ph[1][1], pa[2], pb[2]);
-        split_pack(ph[1][2], ph[1][3], pa[3], pb[3]);
-        mma_bf16_16816(oh[0], pa, v0, v1);
-        mma_bf16_16816(oh[1], pa, v2, v3);
-        mma_bf16_16816(ol[0], pb, v0, v1);
-        mma_bf16_16816(ol[1], pb, v2, v3);
-      }
-      const uint32_t va[4] = {v0, v2, v1, v3};
-#pragma unroll
-      for (int kk = 0; kk < DK / 16; ++kk) {
-        uint32_t kh[4], kl[4];
-        const uint32_t ko = swz<CH>(arow, kk * 2 + acb);
-        ldmatrix_x4_trans(kh[0], kh[1], kh[2], kh[3], sb + L::khi + ko);
-        ldmatrix_x4_trans(kl[0], kl[1], kl[2], kl[3], sb + L::klo + ko);
-        mma_bf16_16816(acc[2 * kk], va, kh[0], kh[1]);
-        mma_bf16_16816(acc[2 * kk + 1], va, kh[2], kh[3]);
-        mma_bf16_16816(acc[2 * kk], va, kl[0], kl[1]);
-        mma_bf16_16816(acc[2 * kk + 1], va, kl[2], kl[3]);
-      }
-#pragma unroll
-      for (int j = 0; j < 2; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int t = (lane >> 2) + (e >> 1) * 8, c = c0 + warp * 16 + j * 8 + (lane & 3) * 2 + (e & 1);
-          if (t >= s0 && t < s1 && c < p.dv)
-            out[((int64_t)(row0 + t0 + t) * p.H + h) * p.dv + c] = oh[j][e] + ol[j][e];
-        }
     }
   }
+  if (!STATE_ONLY && !one_seg) return;      // the scan has written the state behind the last segment
   __syncthreads();
+  if (STATE_ONLY && c0 == 0)
+    for (int c = tid; c < dk; c += NT) sp.decay[seg_at * dk + c] = exp2f(tot[c]);
   if (has_cols) {
 #pragma unroll
     for (int nt = 0; nt < DK / 8; ++nt)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int c = nt * 8 + (lane & 3) * 2 + (e & 1), v = vrow + (e >> 1) * 8;
-        if (c < dk && v < p.dv) S[(int64_t)c * p.dv_pad + v] = acc[nt][e] * et[c];
+        if (c < dk && v < p.dv_pad) S[(int64_t)c * p.dv_pad + v] = acc[nt][e] * et[c];
       }
   }
+}
+
+// Segment states -> start states: S <- decay * S + local, from the slot's state (or zero) through the segments of a
+// sequence; the state behind the last one goes to the slot.  grid (heads, sequences, parts of the dk x dv_pad matrix).
+__global__ void __launch_bounds__(256) linattn_scan_kernel(LinAttnParams<bf16> p, SegParams sp) {
+  const int h = blockIdx.x, b = blockIdx.y;
+  const int i = (blockIdx.z * 256 + threadIdx.x) * 4;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row0 = p.cu_q[b], n = p.cu_q[b + 1] - row0;
+  const int slot = p.slots[b];
+  if (n <= 0 || slot < 0 || i >= p.dk * p.dv_pad) return;
+  const int c = i / p.dv_pad;
+  float4* S = reinterpret_cast<float4*>(p.state + ((int64_t)slot * p.H + h) * p.dk * p.dv_pad + i);
+  float4 s = p.kv_lens[b] == n ? make_float4(0.f, 0.f, 0.f, 0.f) : *S;
+  const int segs = (n + sp.len - 1) / sp.len;
+  for (int g = 0; g < segs; ++g) {
+    const int64_t at = seg_slot(row0, b, g, sp.len) * p.H + h;
+    float4* L = reinterpret_cast<float4*>(sp.state + at * p.dk * p.dv_pad + i);
+    const float4 l = *L;
+    const float d = sp.decay[at * p.dk + c];
+    *L = s;
+    s.x = d * s.x + l.x; s.y = d * s.y + l.y; s.z = d * s.z + l.z; s.w = d * s.w + l.w;
+  }
+  *S = s;
 }
 
 // out[t, h * dv + i] = o[t, h, i] (/ rms over the head) (* w[i]) (* silu(g[t, h * dv + i]));  one warp per (t, h)
@@ -617,17 +816,36 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(T* __restrict__ out
   }
 }
 
-template <int DK, int NW>
-static int launch_chunk(const LinAttnParams<bf16>& p, cudaStream_t s) {
+template <int DK, int NW, bool STATE_ONLY>
+static int launch_chunk_kernel(const LinAttnParams<bf16>& p, const SegParams& sp, int segs, cudaStream_t s) {
   using L = ChunkSmem<DK, NW>;
   const int rot = p.cos_sin != nullptr ? p.rot : 0;
   const int RP = p.log_decay == nullptr ? (p.rank + 15) & ~15 : 0;
-  const size_t smem = L::dyn + (size_t)2 * kLC * rot * 4 + (size_t)2 * kLC * RP * 2 + (RP ? (size_t)DK * (RP + 8) * 2 : 0);
+  const size_t smem = L::dyn + (size_t)2 * kLC * rot * 4 +
+                      (RP ? (size_t)(kLC + 1) * DK * 4 + (size_t)2 * kLC * RP * 2 + (size_t)DK * (RP + 8) * 2 : 0);
   if (smem > 224 * 1024) return (int)cudaErrorInvalidValue;
-  const cudaError_t e = cudaFuncSetAttribute(linattn_chunk_kernel<DK, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const cudaError_t e = cudaFuncSetAttribute(linattn_chunk_kernel<DK, NW, STATE_ONLY>,
+                                             cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
-  launch_pdl(linattn_chunk_kernel<DK, NW>, dim3(p.H, p.n_seqs, (p.dv + L::VC - 1) / L::VC), dim3(NW * 32), smem, s, p);
+  const int slices = (p.dv + L::VC - 1) / L::VC;
+  launch_pdl(linattn_chunk_kernel<DK, NW, STATE_ONLY>, dim3(p.H, p.n_seqs, slices * segs), dim3(NW * 32), smem, s, p, sp);
   return XLLM_LAUNCH_CHECK();
+}
+
+template <int DK, int NW>
+static int launch_chunk(const LinAttnParams<bf16>& p, SegParams sp, int segs, cudaStream_t s) {
+  if (p.dv > NW * 16) sp.fused_out = nullptr;
+  if (segs > 1) {
+    int rc = launch_chunk_kernel<DK, NW, true>(p, sp, segs, s);
+    if (rc != 0) return rc;
+    const int n = p.dk * p.dv_pad;
+    launch_pdl(linattn_scan_kernel, dim3(p.H, p.n_seqs, (n + 1023) / 1024), dim3(256), 0, s, p, sp);
+    rc = XLLM_LAUNCH_CHECK();
+    if (rc != 0) return rc;
+  } else {
+    sp.state = nullptr;
+  }
+  return launch_chunk_kernel<DK, NW, false>(p, sp, segs, s);
 }
 
 }  // namespace xllm
@@ -641,9 +859,12 @@ XLLM_API int xllm_linattn(void* state, const void* slots, const void* cu_q, cons
                           const void* positions, const void* log_decay, const void* a2, const void* a2_b, const void* norm_w,
                           void* out, int64_t out_ld, int n_seqs, int H, int dk, int dv, int rot, int interleaved, int rank,
                           int unit_norm, float q_scale, float k_scale, float inv_tau, float eps, int dtype, int mode,
-                          void* stream) {
+                          void* seg_state, void* seg_decay, int seg_len, int segs, int finish, void* stream) {
   // mode 0: one token per sequence, sequence s is row s, `out` finished in the activation type (cu_q unused)
-  // mode 1: prompt rows by cu_q, `out` raw fp32 [T, H, dv];  mode 2: the same, token by token
+  // mode 1: prompt rows by cu_q, `out` raw fp32 [T, H, dv], or with `finish` (dv <= 128) finished bf16 rows [T, out_ld].
+  //         Prompts longer than seg_len run as up to `segs` segments side by side: seg_state fp32 [n, H, dk, dv_pad] and
+  //         seg_decay fp32 [n, H, dk] with n = T / seg_len + n_seqs + 1, seg_len a multiple of 16.
+  // mode 2: prompt rows token by token, `out` raw fp32
   using namespace xllm;
   if (n_seqs == 0) return 0;
   if (H <= 0 || dk <= 0 || dv <= 0 || dk > 512 || dv > 1024 || rot < 0 || rot > dk || rot % 2 != 0)
@@ -678,9 +899,19 @@ XLLM_API int xllm_linattn(void* state, const void* slots, const void* cu_q, cons
     }
     if constexpr (sizeof(T) == 2) {
       if (mode == 1) {
-        if (dk <= 64) rc = launch_chunk<64, 4>(p, s);
-        else if (dk <= 128) rc = launch_chunk<128, 4>(p, s);
-        else if (dk <= 256) rc = launch_chunk<256, 4>(p, s);
+        SegParams sp;
+        sp.state = (float*)seg_state; sp.decay = (float*)seg_decay; sp.len = seg_len; sp.out_ld = out_ld;
+        sp.fused_out = finish ? out : nullptr;
+        if (finish) p.vec_ok = p.vec_ok && (g == nullptr || a16(g)) && out_ld % 2 == 0;
+        if (seg_len <= 0 || seg_len % kLC != 0 || segs < 1 || (segs > 1 && (seg_state == nullptr || seg_decay == nullptr)) ||
+            (finish && dv > 128)) {
+          rc = (int)cudaErrorInvalidValue;
+          return;
+        }
+        const bool wide = dv > 64;
+        if (dk <= 64) rc = wide ? launch_chunk<64, 8>(p, sp, segs, s) : launch_chunk<64, 4>(p, sp, segs, s);
+        else if (dk <= 128) rc = wide ? launch_chunk<128, 8>(p, sp, segs, s) : launch_chunk<128, 4>(p, sp, segs, s);
+        else if (dk <= 256) rc = wide ? launch_chunk<256, 8>(p, sp, segs, s) : launch_chunk<256, 4>(p, sp, segs, s);
         else rc = (int)cudaErrorInvalidValue;
         return;
       }

@@ -116,7 +116,7 @@ class LinearAttentionMixer(Module):
                            g=p["g"][:nd], r=r[:nd] if r is not None else None, out=out[:nd])
         if meta.n_prefill > 0:
             self.op.prefill(state, slots[nd:], meta.cu_q[nd:], meta.kv_lens[nd:], positions, p["q"], p["k"], p["v"],
-                            g=p["g"], r=r, out=out, row0=nd, padded=meta.padded)
+                            g=p["g"], r=r, out=out, row0=nd, padded=meta.padded, max_q_len=meta.max_q_len)
         return self.o(out)
 
     __call__ = forward

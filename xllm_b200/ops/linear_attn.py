@@ -13,7 +13,7 @@ import torch
 from . import _lib
 from ._lib import F, I, L, P, check, ptr, stream
 
-_lib.register_signature("xllm_linattn", [P] * 9 + [L, P, L, P, P, P, P, P, P, L] + [I] * 8 + [F] * 4 + [I, I, P])
+_lib.register_signature("xllm_linattn", [P] * 9 + [L, P, L, P, P, P, P, P, P, L] + [I] * 8 + [F] * 4 + [I, I, P, P, I, I, I, P])
 _lib.register_signature("xllm_head_norm_gate", [P, L, P, P, L, P, L, I, I, I, F, I, P])
 
 _DT = {torch.bfloat16: 0, torch.float32: 1}
@@ -41,7 +41,7 @@ class LinearAttention:
     norm_w: Optional[torch.Tensor] = None
     eps: float = 1e-6
 
-    def _launch(self, mode, state, slots, cu_q, kv_lens, positions, q, k, v, g, r, out, out_ld, n_seqs):
+    def _launch(self, mode, state, slots, cu_q, kv_lens, positions, q, k, v, g, r, out, out_ld, n_seqs, seg=(None, None, 16, 1), finish=False):
         ld = q.stride(0)
         for t in (k, v, g, r):
             assert t is None or (t.stride(0) == ld and t.stride(1) == 1 and t.dtype == q.dtype)
@@ -56,7 +56,8 @@ class LinearAttention:
             ptr(self.cos_sin if use_rope else None), self.cos_sin.shape[0] if use_rope else 0, ptr(positions),
             ptr(self.log_decay), ptr(self.a2), ptr(self.a2_bias), ptr(self.norm_w), ptr(out), out_ld, n_seqs, self.heads,
             self.dk, self.dv, self.rot, int(self.interleaved), self.a2.shape[1] if channel else 0, int(self.unit_norm),
-            self.q_scale, self.k_scale, self.inv_tau, self.eps, _DT[q.dtype], mode, stream()), "linattn")
+            self.q_scale, self.k_scale, self.inv_tau, self.eps, _DT[q.dtype], mode, ptr(seg[0]), ptr(seg[1]),
+            seg[2], seg[3], int(finish), stream()), "linattn")
         from . import _count
         _count()
 
@@ -72,22 +73,40 @@ class LinearAttention:
         return out
 
     def prefill(self, state, slots, cu_q, kv_lens, positions, q, k, v, g=None, r=None, out=None, row0=0, padded=False,
-                token_by_token=False):
+                token_by_token=False, max_q_len=None):
         """Prompt rows of several sequences (absolute token rows cu_q, all at or behind row0); fills rows [row0, T) of
         `out` [T, heads * dv].  `padded`: rows outside every sequence exist and must come out finite.
-        `token_by_token`: the fp32 recurrence instead of the chunked form."""
+        `max_q_len`: the most rows any sequence has (default: all rows).  `token_by_token`: the fp32 recurrence instead of the chunked form."""
         n = slots.shape[0]
         if not q.is_cuda:
             return self._cpu(state, slots, cu_q, kv_lens, positions, q, k, v, r, g, out)
         T = q.shape[0]
-        o = (torch.zeros if padded else torch.empty)((T, self.heads, self.dv), dtype=torch.float32, device=q.device)
-        chunked = q.dtype == torch.bfloat16 and self.dk <= 256 and not token_by_token and \
-            (self.a2 is None or self.a2.shape[1] <= 128)
-        self._launch(1 if chunked else 2, state, slots, cu_q, kv_lens, positions, q, k, v, None, r, o, 0, n)
         if out is None:
             out = torch.empty((T, self.heads * self.dv), dtype=q.dtype, device=q.device)
+        chunked = q.dtype == torch.bfloat16 and self.dk <= 256 and not token_by_token and \
+            (self.a2 is None or self.a2.shape[1] <= 64)
+        fused = chunked and self.dv <= 128
+        seg = self._segments(T, n, max_q_len or T, q.device) if chunked else (None, None, 16, 1)
+        if fused:
+            self._launch(1, state, slots, cu_q, kv_lens, positions, q, k, v, g, r, out, out.stride(0), n, seg=seg, finish=True)
+            return out
+        o = (torch.zeros if padded else torch.empty)((T, self.heads, self.dv), dtype=torch.float32, device=q.device)
+        self._launch(1 if chunked else 2, state, slots, cu_q, kv_lens, positions, q, k, v, None, r, o, 0, n, seg=seg)
         self.finish(o[row0:], g[row0:] if g is not None else None, out[row0:])
         return out
+
+    def _segments(self, T, n_seqs, max_q_len, device):
+        """(states, decays, segment length, segments per sequence): long prompts are cut so that the CTAs of one launch
+        (heads x value slices x segments) fill the GPU about twice; short ones stay whole."""
+        ctas = self.heads * -(-self.dv // 128)
+        length = min(1024, max(128, -(-T * ctas // 592)))
+        length = -(-length // 64) * 64
+        segs = -(-max_q_len // length)
+        if segs == 1:
+            return None, None, length, 1
+        m = T // length + n_seqs + 1
+        st = torch.empty((m, self.heads, self.dk, (self.dv + 3) // 4 * 4), dtype=torch.float32, device=device)
+        return st, torch.empty((m, self.heads, self.dk), dtype=torch.float32, device=device), length, segs
 
     def finish(self, o, g, out):
         """Per-head norm, weight and gate of raw fp32 outputs o [T, heads, dv]."""
