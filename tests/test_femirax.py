@@ -311,3 +311,12 @@ def test_configuration_is_read_from_the_checkpoint(tmp_path):
     bad["layers"][1]["type"] = "convolution"
     with pytest.raises(ValueError):
         make_engine(tmp_path / "y", bad, w, ("cpu", "float32"))
+
+
+def test_kernel_sources_of_the_model():
+    from xllm_b200 import _build
+    from xllm_b200.models import ModelArgs
+    from xllm_b200.models.registry import kernel_sources_of
+    names = kernel_sources_of(ModelArgs(model_type="femirax"))
+    assert set(names) <= {s.stem for s in _build.kernel_sources()} and "linear_attn" in names
+    assert kernel_sources_of(ModelArgs(model_type="qwen3")) is None

@@ -112,14 +112,26 @@ def _link_atomic(cmd_prefix, out: Path, objs, tail, verbose):
     os.replace(tmp, out)  # readers never see a half-written library
 
 
-def build_kernels(force: bool = False, verbose: bool = False, ptxas_info: bool = False) -> Path:
-    """Compile every ``csrc/kernels/*.cu`` for sm_100a and link the C-ABI library."""
+def build_kernels(force: bool = False, verbose: bool = False, ptxas_info: bool = False, only=None) -> Path:
+    """Compile every ``csrc/kernels/*.cu`` for sm_100a and link the C-ABI library.  `only`: a set of source names (file
+    stems); just those are compiled, into a library of their own, unless the whole library is there and fresh."""
     with _BuildLock():
-        return _build_kernels(force, verbose, ptxas_info)
+        return _build_kernels(force, verbose, ptxas_info, only)
 
 
-def _build_kernels(force, verbose, ptxas_info) -> Path:
+def _build_kernels(force, verbose, ptxas_info, only=None) -> Path:
     srcs = kernel_sources()
+    lib, link_stamp = KERNEL_LIB, LIBDIR / "libxllm_kernels.sha"
+    if only is not None:
+        whole = _sha(srcs + _headers("kernels"), " ".join(NVCC_FLAGS))
+        if KERNEL_LIB.exists() and link_stamp.exists() and link_stamp.read_text() == whole:
+            return KERNEL_LIB
+        missing = set(only) - {s.stem for s in srcs}
+        if missing:
+            raise ValueError(f"no kernel sources named {sorted(missing)}")
+        srcs = [s for s in srcs if s.stem in only]
+        tag = hashlib.sha256(" ".join(sorted(only)).encode()).hexdigest()[:8]
+        lib, link_stamp = LIBDIR / f"libxllm_kernels_{tag}.so", LIBDIR / f"libxllm_kernels_{tag}.sha"
     hdrs = _headers("kernels")
     flags = list(NVCC_FLAGS) + (["-Xptxas", "-v"] if ptxas_info else [])
     LIBDIR.mkdir(exist_ok=True)
@@ -145,13 +157,11 @@ def _build_kernels(force, verbose, ptxas_info) -> Path:
     if todo:
         with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 4)) as ex:
             list(ex.map(one, todo))
-    link_stamp = LIBDIR / "libxllm_kernels.sha"
     want = _sha(srcs + hdrs, " ".join(flags))
-    if todo or force or not KERNEL_LIB.exists() or not link_stamp.exists() \
-            or link_stamp.read_text() != want:
-        _link_atomic([NVCC, "-shared"], KERNEL_LIB, objs, ["-lcudart"], verbose)
+    if todo or force or not lib.exists() or not link_stamp.exists() or link_stamp.read_text() != want:
+        _link_atomic([NVCC, "-shared"], lib, objs, ["-lcudart"], verbose)
         link_stamp.write_text(want)
-    return KERNEL_LIB
+    return lib
 
 
 def runtime_sources():

@@ -90,6 +90,9 @@ class FemiraxCausalLM(Module):
     state_on_device = True          # state slots are a device input of the step: graphs capture it
     supports_graph = True
     supports_prefill_graph = True
+    # the kernel sources a process that runs nothing but this model needs
+    kernel_sources = ("gemm_tcgen05", "activation", "attn_decode", "attn_prefill", "attn_prefill_tc", "attn_generic",
+                      "linear_attn", "residual", "rope_norm_kv", "misc", "sampling")
     fused_tp = False
 
     def __init__(self, args, dtype=torch.bfloat16, device="cpu", ps=None):
@@ -180,6 +183,6 @@ class FemiraxCausalLM(Module):
     __call__ = forward
 
 
-@register_model("femirax", "Femirax")
+@register_model("femirax", "Femirax", kernel_sources=FemiraxCausalLM.kernel_sources)
 def build_femirax(args, dtype, device, ps):
     return FemiraxCausalLM(args, dtype, device, ps)

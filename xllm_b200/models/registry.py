@@ -10,10 +10,16 @@ from typing import Callable, Dict
 _FACTORIES: Dict[str, Callable] = {}
 
 
-def register_model(*names):
+_KERNEL_SOURCES: Dict[str, tuple] = {}
+
+
+def register_model(*names, kernel_sources=None):
+    """`kernel_sources`: the kernel files a process that runs only this model needs (default: all of them)."""
     def deco(fn):
         for n in names:
             _FACTORIES[n.lower()] = fn
+            if kernel_sources is not None:
+                _KERNEL_SOURCES[n.lower()] = tuple(kernel_sources)
         return fn
     return deco
 
@@ -31,6 +37,13 @@ def _import_all():
         except ModuleNotFoundError as e:
             if e.name != f"{__package__}.{mod}":
                 raise
+
+
+def kernel_sources_of(args):
+    """Kernel sources of the model `args` describes, or None when its family does not say."""
+    _import_all()
+    return next((_KERNEL_SOURCES[k] for k in [args.model_type.lower()] + [a.lower() for a in args.architectures]
+                 if k in _KERNEL_SOURCES), None)
 
 
 def create_model(args, dtype, device, ps=None):

@@ -30,15 +30,26 @@ def have_gpu() -> bool:
     return torch.cuda.is_available()
 
 
+_ONLY = None
+
+
+def select_sources(names):
+    """Before the first `load`: this process needs the kernels of these sources only, so an unbuilt tree compiles no
+    others (a built one is used as it is).  None: all of them."""
+    global _ONLY
+    if _LIB is None:
+        _ONLY = None if names is None else frozenset(names)
+
+
 def load(build_if_missing: bool = True):
     """Return the loaded kernel library (building it in-tree if it is absent or stale)."""
-    global _LIB
+    global _LIB, _LIB_PATH
     if _LIB is not None:
         return _LIB
     if build_if_missing and os.environ.get("XLLM_NO_BUILD", "0") != "1":
         try:
             from .. import _build
-            _build.build_kernels()
+            _LIB_PATH = _build.build_kernels(only=_ONLY)
         except Exception as e:  # a box without nvcc still works from a pre-built library
             if not _LIB_PATH.exists():
                 raise KernelLibraryMissing(f"cannot build {_LIB_PATH}: {e}") from e

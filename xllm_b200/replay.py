@@ -20,6 +20,10 @@ import sys
 
 def build_engine(model: str, dtype: str, max_tokens: int, device: str = "auto", max_live: int = 4, block_size: int = 16):
     from .engine.llm_engine import EngineConfig, LLMEngine
+    from .models import load_model_args
+    from .models.registry import kernel_sources_of
+    from .ops import _lib
+    _lib.select_sources(kernel_sources_of(load_model_args(model)))
     blocks = -(-max_tokens // block_size)
     tokens = blocks * block_size
     return LLMEngine(EngineConfig(
