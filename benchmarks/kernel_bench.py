@@ -277,6 +277,112 @@ def moe_rows(results, hbm, tf, tag):
               f" | GEMM, activation kernel, GEMM: {t_plain*1e3:7.3f} ms")
 
 
+def bench_queued(fn, iters=10, warmup=3):
+    """Like `bench`, but the timed launches are queued while the L2 flush still runs: device time without the host's
+    launch latency, for kernels of a few microseconds."""
+    bench(fn, iters=0, warmup=warmup)
+    ts = []
+    for _ in range(iters):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        for _ in range(4):
+            _flush.zero_()
+        e0.record()
+        fn()
+        e1.record()
+        torch.cuda.synchronize()
+        ts.append(e0.elapsed_time(e1))
+    ts.sort()
+    return ts[len(ts) // 2] * 1e-3
+
+
+def hybrid_rows(results, hbm, tf, tag):
+    """The kernels of the hybrid decoders (Femirax) beside the like kernels of Qwen3-Next: decayed linear attention
+    against the gated delta rule (decode, prompts), the fp32 residual update against add + RMSNorm, rotation + unit norm +
+    cache write against norm + rotation + cache write, the side input's products and activation.  32 heads of 128, width
+    4096."""
+    from xllm_b200.ops import gdn
+    from xllm_b200.ops.linear_attn import LinearAttention
+    from xllm_b200.ops.residual import gelu_mul_rows, residual_update
+    dev, bf, H, d, W = "cuda", torch.bfloat16, 32, 128, 4096
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    rows = lambda t, n: torch.randn(t, n, device=dev, dtype=bf)
+    cs = torch.randn(8192, d, device=dev)
+
+    def report(name, shape, t, nbytes, flops=0.0):
+        ideal = max(nbytes / (hbm * 1e9), flops / (tf * 1e12))
+        results.append(dict(kernel=name, shape=shape, ms=t * 1e3, gbs=nbytes / t / 1e9, tflops=flops / t / 1e12,
+                            frac_of_roofline=ideal / t, peaks=tag))
+        print(f"{name:<34} {shape:<26} {t*1e6:9.1f} us {nbytes/t/1e9:7.0f} GB/s {flops/t/1e12:7.1f} TF/s  {ideal/t:6.3f} of {tag}",
+              flush=True)
+
+    def op_of(kind):
+        op = LinearAttention(H, d, d, k_scale=d ** -0.5)
+        if kind == "retention":
+            op.log_decay, op.cos_sin, op.rot = torch.full((H,), -0.01, device=dev), cs, d
+        else:
+            op.a2, op.a2_bias = rows(H * d, 16) * 0.1, torch.full((H * d,), 4.0, device=dev, dtype=bf)
+            op.inv_tau, op.norm_w = 1 / 16, torch.ones(d, device=dev, dtype=bf)
+        return op
+
+    cut = lambda r: [r[:, i * H * d:(i + 1) * H * d] for i in range(4)] + [r[:, 4 * H * d:4 * H * d + 16]]
+    for B in (16, 64, 256):
+        st = torch.zeros(B + 1, H, d, d, device=dev)
+        c, sl = cut(rows(B, 4 * H * d + 16)), i32(list(range(B)))
+        kl, pos, out = torch.full_like(sl, 100), torch.full((B,), 99, device=dev), torch.empty(B, H * d, device=dev, dtype=bf)
+        nb = 2 * B * H * d * d * 4 + B * H * d * 10
+        for kind in ("retention", "channel decay"):
+            op = op_of(kind)
+            report(f"linattn_decode, {kind}", f"B={B}", bench_queued(
+                lambda: op.decode(st, sl, kl, pos, c[0], c[1], c[2], g=c[3], r=c[4], out=out)), nb)
+        q, k, v = (torch.randn(B, H, d, device=dev) for _ in range(3))
+        g, be, o, s64 = -torch.rand(B, H, device=dev), torch.rand(B, H, device=dev), torch.empty(B, H, d, device=dev), sl.long()
+        report("gdn_decode", f"B={B}", bench_queued(lambda: gdn.decode_step(st, s64, q, k, v, g, be, out=o)),
+               2 * B * H * d * d * 4 + B * H * d * 16)
+        del st
+    for S, L in ((1, 2048), (1, 8192), (4, 2048)):
+        T = S * L
+        st = torch.zeros(S + 1, H, d, d, device=dev)
+        c, sl = cut(rows(T, 4 * H * d + 16)), i32(list(range(S)))
+        cu, kl, pos = i32([i * L for i in range(S + 1)]), i32([L] * S), torch.arange(L, device=dev).repeat(S)
+        out = torch.empty(T, H * d, device=dev, dtype=bf)
+        fl = 4.0 * T * H * d * d
+        for kind in ("retention", "channel decay"):
+            op = op_of(kind)
+            report(f"linattn prompts, {kind}", f"{S} x {L}", bench_queued(
+                lambda: op.prefill(st, sl, cu, kl, pos, c[0], c[1], c[2], g=c[3], r=c[4], out=out, max_q_len=L), iters=5),
+                T * H * d * 10 + S * H * d * d * 8, fl)
+        q, k, v = (torch.randn(L, H, d, device=dev) for _ in range(3))
+        g, be, o = -torch.rand(L, H, device=dev), torch.rand(L, H, device=dev), torch.empty(L, H, d, device=dev)
+        report("gdn_prefill", f"{S} x {L}", bench_queued(
+            lambda: [gdn.prefill(st, s, True, q, k, v, g, be, out=o) for s in range(S)], iters=3), T * H * d * 16, 2 * fl)
+    nq, nkv = 32, 8
+    for T in (64, 8192):
+        x, y, y2, w, res = torch.randn(T, W, device=dev), rows(T, W), rows(T, W), torch.ones(W, device=dev, dtype=bf), rows(T, W)
+        report("residual_update", f"T={T}", bench_queued(lambda: residual_update(x, y, w_out=w)), T * W * 12)
+        report("residual_update, normed branch", f"T={T}", bench_queued(lambda: residual_update(x, y, w=w, w_out=w)), T * W * 12)
+        report("residual_update, two branches", f"T={T}", bench_queued(
+            lambda: residual_update(x, y, w=w, y2=y2, w2=w, coef=0.5, w_out=w)), T * W * 14)
+        report("rmsnorm (bf16 residual)", f"T={T}", bench_queued(lambda: ops.rmsnorm(y, w, 1e-6, residual=res)), T * W * 8)
+        qkv, pos = rows(T, (nq + 2 * nkv) * d), torch.arange(T, device=dev) % 8192
+        kc = torch.zeros(T // 16 + 2, nkv, 16, d, device=dev, dtype=bf)
+        vc, sl, wn = torch.zeros_like(kc), torch.arange(16, 16 + T, dtype=torch.int32, device=dev), torch.ones(d, device=dev, dtype=bf)
+        q, k = qkv[:, :nq * d], qkv[:, nq * d:(nq + nkv) * d]
+        report("rope_norm_kv", f"T={T}", bench_queued(lambda: ops.rope_norm_kv_write(
+            q, k, k, nq, nkv, d, pos, cs, d, sl, kc, vc, interleaved=True)), T * d * 2 * (2 * nq + 3 * nkv))
+        report("rope_kv", f"T={T}", bench_queued(lambda: ops.rope_kv_write(
+            qkv, nq, nkv, d, pos, cs, d, slots=sl, k_cache=kc, v_cache=vc, q_norm_w=wn, k_norm_w=wn)), T * d * 4 * (nq + 2 * nkv))
+        for dim in (16, 64, 256):
+            gate, table, ids = rows(T, dim), rows(32000, dim * 4), torch.randint(0, 32000, (T,), device=dev)
+            xb, wg, wp = rows(T, W), rows(dim, W), rows(W, dim)
+            nb, fl = 2.0 * (T * W + dim * W + T * dim), 2.0 * T * W * dim
+            report("gelu_mul_rows", f"T={T} dim={dim}", bench_queued(lambda: gelu_mul_rows(gate, table, ids, dim, dim)), T * dim * 6)
+            report("side gate GEMM", f"T={T} dim={dim}", bench_queued(lambda: ops.linear(xb, wg)), nb, fl)
+            report("side gate, cuBLAS", f"T={T} dim={dim}", bench_queued(lambda: torch.nn.functional.linear(xb, wg)), nb, fl)
+            report("side proj GEMM", f"T={T} dim={dim}", bench_queued(lambda: ops.linear(gate, wp)), nb, fl)
+            report("side proj, cuBLAS", f"T={T} dim={dim}", bench_queued(lambda: torch.nn.functional.linear(gate, wp)), nb, fl)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--what", default="gemm,decode,prefill,small")
@@ -286,7 +392,7 @@ def main():
     results = []
     for w in a.what.split(","):
         {"gemm": gemm_rows, "decode": decode_rows, "prefill": prefill_rows, "small": small_rows, "gdn": gdn_rows, "mla": mla_rows,
-         "fp8": fp8_rows, "moe": moe_rows}[w](results, hbm, tf, tag)
+         "fp8": fp8_rows, "moe": moe_rows, "hybrid": hybrid_rows}[w](results, hbm, tf, tag)
     if a.json:
         with open(a.json, "w") as f:
             json.dump(results, f, indent=1)

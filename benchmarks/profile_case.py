@@ -20,6 +20,7 @@ hundred MB on the device, a handful of launches).
     python benchmarks/profile_case.py --kernel logsoftmax # log-softmax, 1024 rows x 151936
     python benchmarks/profile_case.py --kernel gemm_act   # gate_up GEMM with the SiLU-mul epilogue, 2304 x 24576 x 4096
     python benchmarks/profile_case.py --kernel xattn      # beam attention: 16 requests x 128 beams over 2048-token prompts
+    python benchmarks/profile_case.py --kernel linattn    # decayed linear attention, 4096-token prompt x 32 heads (linattn_channel: per-channel decay)
     python benchmarks/profile_case.py --kernel gdn_prefill # gated-delta-rule prompt chunk, 4096 tokens x 32 heads
 """
 import argparse
@@ -190,6 +191,22 @@ def main():
         v = torch.randn(n, nv, dv, device=dev)
         g, beta = -torch.rand(n, nv, device=dev), torch.rand(n, nv, device=dev)
         fn = lambda: gdn.prefill(state, 1, True, q, k, v, g, beta)
+    elif a.kernel in ("linattn", "linattn_channel"):
+        from xllm_b200.ops.linear_attn import LinearAttention
+        T, H, d = 4096, 32, 128
+        op = LinearAttention(H, d, d, k_scale=d ** -0.5)
+        if a.kernel == "linattn":
+            op.log_decay, op.cos_sin, op.rot = torch.full((H,), -0.01, device=dev), torch.randn(T, d, device=dev), d
+        else:
+            op.a2 = torch.randn(H * d, 16, device=dev, dtype=torch.bfloat16) * 0.1
+            op.a2_bias, op.inv_tau = torch.full((H * d,), 4.0, device=dev, dtype=torch.bfloat16), 1 / 16
+        st = torch.zeros(2, H, d, d, device=dev)
+        r = torch.randn(T, 4 * H * d + 16, device=dev, dtype=torch.bfloat16)
+        c = [r[:, i * H * d:(i + 1) * H * d] for i in range(4)] + [r[:, 4 * H * d:]]
+        i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+        sl, cu, kl, pos = i32([0]), i32([0, T]), i32([T]), torch.arange(T, device=dev)
+        out = torch.empty(T, H * d, device=dev, dtype=torch.bfloat16)
+        fn = lambda: op.prefill(st, sl, cu, kl, pos, c[0], c[1], c[2], g=c[3], r=c[4], out=out, max_q_len=T)
     else:
         raise SystemExit(f"unknown kernel {a.kernel}")
     for _ in range(a.iters):

@@ -48,6 +48,9 @@ CONFIGS = {
     # large heads, no feed-forward anywhere, no parallel layer first
     "wide": (config([retention(2, 200, 72, [0.97, 0.9995], 40),
                      parallel(2, 2, 144, 8, 0.09, 1, 192, 80, 2.0)], vocab=64, width=96, side=8), 16),
+    # a width and a vocabulary that no tensor-core product takes
+    "ragged": (config([parallel(3, 3, 22, 8, 0.2, 2, 34, 26, 3.0, ff=30), retention(2, 10, 70, [0.96, 0.8], 6)],
+                      vocab=101, width=100, side=5), 7),
     "retention_only": (config([retention(2, 16, 16, [0.9, 0.99], 8, ff=24), retention(1, 40, 24, [0.95], 40)], side=3), 4),
 }
 

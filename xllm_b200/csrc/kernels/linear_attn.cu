@@ -50,6 +50,8 @@ struct LinAttnParams {
 
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float silu_f32(float z) { return z / (1.f + expf(-z)); }
+// for rows that leave as bf16: hardware exponential and division (2^-21 relative)
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 
 // element i of a head after the rotation of its first `rot` elements; `cs` is the position's cos | sin row
 template <typename T>
@@ -278,7 +280,7 @@ struct ChunkSmem {
   static constexpr int fs = raw + 4 * tile;                // [DK] scale of the state rows
   static constexpr int et = fs + DK * 4;                   // [DK] decay from the reference token to the chunk's end
   static constexpr int tot = et + DK * 4;                  // [DK] log2 decay over the segment so far
-  static constexpr int ssm = tot + DK * 4;                 // [NW][16] partial sums of squares
+  static constexpr int ssm = tot + DK * 4;                 // [16][NW] partial sums of squares
   static constexpr int dyn = ssm + NW * kLC * 4;
   // dyn: cos | sin 2 x [16][rot] fp32; channel decay: lw [16][DK] fp32, bias [DK], raw r 2 x [16][RP], a2 [DK][RP + 8]
 };
@@ -353,23 +355,28 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 512 / (NW * 32)) linat
     if (tid < 2 * kLC) elog[tid] = exp2f((float)(tid - kLC) * lg);      // elog[16 + i] = decay^i
   }
 
+  const int64_t last_pos = p.max_pos - 1;
+  const int64_t pos0 = rot > 0 ? max((int64_t)0, min(p.positions[row0], last_pos)) : 0;
   const auto load_raw = [&](int t0, int buf) {              // 16 token rows from t0 (of this segment)
     const uint32_t raws = sb + L::raw + buf * 2 * L::tile, vsm = sb + L::v + buf * L::vtile, gsm = sb + L::g + buf * L::vtile;
     const int64_t base = (int64_t)(row0 + t0);
     const bool gate = !STATE_ONLY && sp.fused_out != nullptr && p.g != nullptr;
     if (p.vec_ok) {
-      const int per = dk >> 3;
-      for (int i = tid; i < kLC * per; i += NT) {
-        const int r = i / per, c = i - r * per;
+      const int64_t row = base * p.ld;
+#pragma unroll
+      for (int i = tid; i < kLC * CH; i += NT) {
+        const int r = i / CH, c = i % CH;                    // powers of two
+        if (c * 8 >= dk) continue;
         const bool ok = t0 + r < n_all;
-        const int64_t go = (base + (ok ? r : 0)) * p.ld + (int64_t)h * dk + c * 8;
+        const int64_t go = row + (ok ? r : 0) * p.ld + h * dk + c * 8;
         if (!STATE_ONLY) cp_async16(raws + (r * DK + c * 8) * 2, p.q + go, ok);
         cp_async16(raws + L::tile + (r * DK + c * 8) * 2, p.k + go, ok);
       }
+#pragma unroll
       for (int i = tid; i < kLC * (L::VC / 8); i += NT) {
-        const int r = i / (L::VC / 8), c = i - r * (L::VC / 8);
+        const int r = i / (L::VC / 8), c = i % (L::VC / 8);
         const bool ok = t0 + r < n_all && c0 + c * 8 < p.dv;
-        const int64_t go = ok ? (base + r) * p.ld + (int64_t)h * p.dv + c0 + c * 8 : 0;
+        const int64_t go = ok ? row + r * p.ld + h * p.dv + c0 + c * 8 : 0;
         cp_async16(vsm + swz<VCH>(r, c), p.v + go, ok);
         if (gate) cp_async16(gsm + (r * L::VCP + c * 8) * 2, p.g + go, ok);
       }
@@ -378,7 +385,7 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 512 / (NW * 32)) linat
         for (int i = tid; i < kLC * pr; i += NT) {
           const int r = i / pr, c = i - r * pr;
           const bool ok = t0 + r < n_all && c * 8 < p.rank;
-          cp_async16(smem_u32(rb + (buf * kLC + r) * RP + c * 8), ok ? p.r + (base + r) * p.ld + c * 8 : p.r, ok);
+          cp_async16(smem_u32(rb + (buf * kLC + r) * RP + c * 8), ok ? p.r + row + r * p.ld + c * 8 : p.r, ok);
         }
       }
     } else {
@@ -406,12 +413,12 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 512 / (NW * 32)) linat
     }
     if (rot > 0) {
       if (rot % 4 == 0) {
-        const int per = rot >> 2;
-        for (int i = tid; i < kLC * per; i += NT) {
-          const int r = i / per, c = i - r * per;
-          const bool ok = t0 + r < n_all;
-          const float* cs = rope_row(p, base + (ok ? r : 0));
-          cp_async16(smem_u32(csb + (buf * kLC + r) * rot + c * 4), cs + c * 4, ok);
+#pragma unroll
+        for (int i = tid; i < kLC * (DK / 4); i += NT) {
+          const int r = i / (DK / 4), c = i % (DK / 4);
+          if (c * 4 >= rot) continue;
+          const int64_t pos = min(pos0 + t0 + r, last_pos);   // the rows of a sequence are consecutive positions
+          cp_async16(smem_u32(csb + (buf * kLC + r) * rot + c * 4), p.cos_sin + pos * rot + c * 4, t0 + r < n_all);
         }
       } else {
         for (int i = tid; i < kLC * rot; i += NT) {
@@ -422,6 +429,7 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 512 / (NW * 32)) linat
     }
     cp_async_commit();
   };
+  const float inv_dv = 1.f / (float)p.dv;
   const bool by_four = dk % 4 == 0 && rot % 4 == 0;       // four channels of a token at a time
 
   load_raw(0, 0);
@@ -707,8 +715,8 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 512 / (NW * 32)) linat
         sc += __shfl_xor_sync(0xffffffffu, sc, 1);
         sc += __shfl_xor_sync(0xffffffffu, sc, 2);
         if ((lane & 3) == 0) {
-          ssm[warp * kLC + (lane >> 2)] = sa;
-          ssm[warp * kLC + (lane >> 2) + 8] = sc;
+          ssm[(lane >> 2) * NW + warp] = sa;
+          ssm[((lane >> 2) + 8) * NW + warp] = sc;
         }
         __syncthreads();
       }
@@ -720,22 +728,28 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 512 / (NW * 32)) linat
         if (p.unit_norm) {
           float ss = 0.f;
 #pragma unroll
-          for (int w = 0; w < NW; ++w) ss += ssm[w * kLC + t];
-          inv = 1.f / sqrtf(ss / (float)p.dv + p.eps);
+          for (int w = 0; w < NW; w += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(ssm + t * NW + w);
+            ss += (x.x + x.y) + (x.z + x.w);
+          }
+          inv = rsqrtf(ss * inv_dv + p.eps);
         }
         if (t < s0 || t >= s1) continue;
+        const bf16* gr = gs + t * L::VCP;
         bf16* orow = reinterpret_cast<bf16*>(sp.fused_out) + (int64_t)(row0 + t0 + t) * sp.out_ld + (int64_t)h * p.dv;
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
-          float y[2];
           const int c = warp * 16 + j * 8 + (lane & 3) * 2;
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            y[e] = 0.f;
-            if (c + e >= p.dv) continue;
-            y[e] = o[j][u * 2 + e] * inv;
-            if (p.norm_w != nullptr) y[e] *= __bfloat162float(p.norm_w[c + e]);
-            if (p.g != nullptr) y[e] *= silu_f32(__bfloat162float(gs[t * L::VCP + c + e]));
+          if (c >= p.dv) continue;
+          float y[2] = {o[j][u * 2] * inv, o[j][u * 2 + 1] * inv};
+          if (p.norm_w != nullptr) {
+            y[0] *= __bfloat162float(p.norm_w[c]);
+            if (c + 1 < p.dv) y[1] *= __bfloat162float(p.norm_w[c + 1]);
+          }
+          if (p.g != nullptr) {
+            const float2 gg = unpack2(*reinterpret_cast<const uint32_t*>(gr + c));
+            y[0] *= silu_fast(gg.x);
+            y[1] *= silu_fast(gg.y);
           }
           if (p.vec_ok && c + 1 < p.dv) {
             *reinterpret_cast<bf162*>(orow + c) = __floats2bfloat162_rn(y[0], y[1]);

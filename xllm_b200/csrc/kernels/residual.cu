@@ -169,28 +169,34 @@ static int launch_residual(const ResidualParams& p, cudaStream_t s) {
   return XLLM_LAUNCH_CHECK();
 }
 
-// out[t, i] = gelu_tanh(gate[t, i]) * table[ids[t], col0 + i] for i < dim, 0 for dim <= i < dim_pad.
-template <typename T>
+// out[t, i] = gelu_tanh(gate[t, i]) * table[ids[t], col0 + i] for i < dim, 0 for dim <= i < dim_pad; V columns a thread.
+template <typename T, int V>
 __global__ void __launch_bounds__(256) gelu_mul_rows_kernel(T* __restrict__ out, const T* __restrict__ gate, int64_t gate_ld,
                                                             const T* __restrict__ table, int64_t table_ld, int64_t n_rows,
                                                             const int64_t* __restrict__ ids, int64_t col0, int tokens, int dim,
                                                             int dim_pad) {
   pdl_wait();
   pdl_launch_dependents();
-  const int64_t total = (int64_t)tokens * dim_pad;
+  const int per = dim_pad / V;
+  const int64_t total = (int64_t)tokens * per;
   for (int64_t n = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; n < total; n += (int64_t)gridDim.x * blockDim.x) {
-    const int64_t t = n / dim_pad;
-    const int i = (int)(n - t * dim_pad);
-    float r = 0.f;
-    if (i < dim) {
+    const int64_t t = n / per;
+    const int i = (int)(n - t * per) * V;
+    float r[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) r[j] = 0.f;
+    if (i < dim) {                                   // V divides dim, or V = 1
       int64_t id = ids[t];
       id = id < 0 ? 0 : (id >= n_rows ? n_rows - 1 : id);
-      const float z = to_f32(gate[t * gate_ld + i]);
-      const float e = to_f32(table[id * table_ld + col0 + i]);
-      const float k = 0.79788456080286535588f;   // sqrt(2 / pi)
-      r = 0.5f * z * (1.f + tanhf(k * (z + 0.044715f * z * z * z))) * e;
+      float z[V], e[V];
+      load_f32<V>(gate + t * gate_ld + i, z);
+      load_f32<V>(table + id * table_ld + col0 + i, e);
+      const float k = 0.79788456080286535588f;       // sqrt(2 / pi)
+#pragma unroll
+      for (int j = 0; j < V; ++j)
+        r[j] = 0.5f * z[j] * (1.f + tanhf(k * (z[j] + 0.044715f * z[j] * z[j] * z[j]))) * e[j];
     }
-    out[n] = from_f32<T>(r);
+    store_f32<V>(out + t * dim_pad + i, r);
   }
 }
 
@@ -239,16 +245,24 @@ XLLM_API int xllm_gelu_mul_rows(void* out, const void* gate, int64_t gate_ld, co
   using namespace xllm;
   if (tokens == 0) return 0;
   if (dim <= 0 || dim_pad < dim || col0 < 0 || col0 + dim > table_ld) return (int)cudaErrorInvalidValue;
-  const int64_t total = (int64_t)tokens * dim_pad;
-  const int64_t want = (total + 255) / 256;
+  const auto a16 = [](const void* q) { return (((uintptr_t)q) & 15) == 0; };
+  const bool v8 = dim % 8 == 0 && dim_pad % 8 == 0 && gate_ld % 8 == 0 && table_ld % 8 == 0 && col0 % 8 == 0 && a16(out) &&
+                  a16(gate) && a16(table);
+  const int64_t want = ((int64_t)tokens * (v8 ? dim_pad / 8 : dim_pad) + 255) / 256;
   const dim3 grid((unsigned)(want < 148 * 8 ? want : 148 * 8));
   cudaStream_t s = (cudaStream_t)stream;
-  if (dtype == 0)
-    launch_pdl(gelu_mul_rows_kernel<bf16>, grid, dim3(256), 0, s, (bf16*)out, (const bf16*)gate, gate_ld, (const bf16*)table,
-               table_ld, n_rows, (const int64_t*)ids, col0, tokens, dim, dim_pad);
-  else
-    launch_pdl(gelu_mul_rows_kernel<float>, grid, dim3(256), 0, s, (float*)out, (const float*)gate, gate_ld,
-               (const float*)table, table_ld, n_rows, (const int64_t*)ids, col0, tokens, dim, dim_pad);
+  const auto run = [&](auto tag, auto kernel) {
+    using T = decltype(tag);
+    launch_pdl(kernel, grid, dim3(256), 0, s, (T*)out, (const T*)gate, gate_ld, (const T*)table, table_ld, n_rows,
+               (const int64_t*)ids, col0, tokens, dim, dim_pad);
+  };
+  if (dtype == 0) {
+    if (v8) run(bf16(), gelu_mul_rows_kernel<bf16, 8>);
+    else run(bf16(), gelu_mul_rows_kernel<bf16, 1>);
+  } else {
+    if (v8) run(float(), gelu_mul_rows_kernel<float, 8>);
+    else run(float(), gelu_mul_rows_kernel<float, 1>);
+  }
   return XLLM_LAUNCH_CHECK();
 }
 
