@@ -15,7 +15,7 @@
 //               of the previous step is added with the usual rescaling O = (O + O_tile) * alpha.
 // The reference reaches the same op through FlashInfer's fa2 kernels
 // (xllm/core/kernels/cuda/flashinfer_attention.cpp:239-301); the mma.sync kernel of attn_prefill.cu
-// stays as the path for other head sizes, sliding windows and small pages.
+// stays as the path for other head sizes and small pages.
 //
 // Every mbarrier wait is bounded; on expiry all roles leave, TMEM is released and an error word
 // is set (xllm_fmha_error_status).
@@ -140,6 +140,7 @@ struct Params {
   const int32_t* kv_lens;
   int64_t o_stride;
   int bt_stride, nq, nkv, page, causal;
+  int window;                  // > 0: a query sees its last `window` positions only
   float scale_log2;
   int* err;
   float* lse;                  // optional [total_q, nq]: log2-domain log-sum-exp of every row's scaled scores
@@ -178,7 +179,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
   const int kv_len = p.kv_lens[b];
   const int ctx_off = kv_len - q_len;                 // absolute position of this chunk's first query
   const int kv_hi = p.causal ? min(kv_len, ctx_off + m0 + kBM) : kv_len;
-  const int n_tiles = (kv_hi + kBN - 1) / kBN;
+  const int first = p.window > 0 ? max(0, ctx_off + m0 - p.window + 1) / kBN : 0;   // tiles before every row's window
+  const int n_tiles = (kv_hi + kBN - 1) / kBN - first;
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -219,7 +221,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
       const int st = j & 1;
-      const int pg = j * pages + lane;
+      const int pg = (first + j) * pages + lane;
       const int myblk = (lane < pages && pg < n_blk) ? bt[pg] : 0;   // pages past the sequence read block 0 (masked)
       const int y = (myblk * p.nkv + hk) * p.page;
       const uint32_t off = (uint32_t)(lane * p.page * 128);
@@ -305,6 +307,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
     const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
     const int q_pos = ctx_off + m0 + row;             // absolute position of this query token
     const int limit = p.causal ? min(kv_len - 1, q_pos) : kv_len - 1;   // last kv index this row may see
+    const int low = p.window > 0 ? q_pos - p.window + 1 : 0;            // the first one
     float* smax = reinterpret_cast<float*>(smem + XCH_OFF);             // [2 tile parities][2 halves][128 rows]
     float* lsum = smax + 2 * 2 * kBM;                                   // [2 halves][128 rows]
     // O stays in TMEM and the MMAs accumulate into it over all kv tiles.  The exponent uses a row
@@ -322,8 +325,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       ok = ok && mbar_wait(s_full(sb), (j >> 1) & 1, abort_flag);
       tc_fence_after();
       const uint32_t saddr = TS0 + sb * 128 + half * 64 + lane_addr;
-      const int kv0 = j * kBN + half * 64;
-      const bool full_tile = kv0 + 63 <= limit;
+      const int kv0 = (first + j) * kBN + half * 64;
+      const bool full_tile = kv0 + 63 <= limit && kv0 >= low;
       uint32_t sv[64];
       tmem_ld32(saddr, sv);
       tmem_ld32(saddr + 32, sv + 32);
@@ -334,7 +337,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       float mx = -INFINITY;
 #pragma unroll
       for (int i = 0; i < 64; ++i)
-        if (full_tile || kv0 + i <= limit) mx = fmaxf(mx, __uint_as_float(sv[i]));
+        if (full_tile || (kv0 + i <= limit && kv0 + i >= low)) mx = fmaxf(mx, __uint_as_float(sv[i]));
       smax[(sb * 2 + half) * kBM + row] = mx;
       asm volatile("bar.sync 1, 256;" ::: "memory");
       mx = fmaxf(mx, smax[(sb * 2 + (half ^ 1)) * kBM + row]);
@@ -372,8 +375,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
           float p0 = exp2f(__uint_as_float(sv[i]) * p.scale_log2 - m_use);
           float p1 = exp2f(__uint_as_float(sv[i + 1]) * p.scale_log2 - m_use);
           if (!full_tile) {
-            if (kv0 + i > limit) p0 = 0.f;
-            if (kv0 + i + 1 > limit) p1 = 0.f;
+            if (kv0 + i > limit || kv0 + i < low) p0 = 0.f;
+            if (kv0 + i + 1 > limit || kv0 + i + 1 < low) p1 = 0.f;
           }
           rs += p0 + p1;
           const __nv_bfloat162 pb = __floats2bfloat162_rn(p0, p1);
@@ -474,7 +477,7 @@ static int* g_err[64] = {};
 }  // namespace fmha
 }  // namespace xllm
 
-// Same contract as xllm_paged_prefill_attn for head_dim 128, no sliding window, page_size in
+// Same contract as xllm_paged_prefill_attn for head_dim 128, page_size in
 // {16, 32, 64, 128}: q [total_q, nq, 128] (row stride q_stride elements), caches
 // [n_blocks, nkv, page, 128], cu_q absolute row offsets [batch + 1], kv_lens [batch].
 // `lse` (optional, fp32 [total_q, nq]) receives every row's log-sum-exp in the log2 domain, so that the
@@ -483,7 +486,7 @@ XLLM_API int xllm_paged_prefill_attn_tc_lse(void* out, int64_t o_stride, const v
                                             const void* k_cache, const void* v_cache, int64_t n_blocks,
                                             const void* block_table, int bt_stride, const void* cu_q,
                                             const void* kv_lens, int batch, int max_q_len, int nq, int nkv,
-                                            int page_size, float scale, int causal, void* lse, void* stream) {
+                                            int page_size, float scale, int causal, int window, void* lse, void* stream) {
   using namespace xllm;
   using namespace xllm::fmha;
   if (batch == 0 || max_q_len == 0) return 0;
@@ -510,7 +513,7 @@ XLLM_API int xllm_paged_prefill_attn_tc_lse(void* out, int64_t o_stride, const v
   Params p;
   p.out = (bf16*)out; p.block_table = (const int32_t*)block_table; p.cu_q = (const int32_t*)cu_q;
   p.kv_lens = (const int32_t*)kv_lens; p.o_stride = o_stride; p.bt_stride = bt_stride; p.nq = nq; p.nkv = nkv;
-  p.page = page_size; p.causal = causal; p.scale_log2 = scale * 1.4426950408889634f; p.err = g_err[dev & 63];
+  p.page = page_size; p.causal = causal; p.window = window; p.scale_log2 = scale * 1.4426950408889634f; p.err = g_err[dev & 63];
   p.lse = (float*)lse;
   dim3 grid((max_q_len + kBM - 1) / kBM, nq, batch);
   prefill_tc_kernel<<<grid, 320, SMEM_TOTAL, (cudaStream_t)stream>>>(tq, tk, tv, p);
@@ -521,10 +524,10 @@ XLLM_API int xllm_paged_prefill_attn_tc(void* out, int64_t o_stride, const void*
                                         const void* k_cache, const void* v_cache, int64_t n_blocks,
                                         const void* block_table, int bt_stride, const void* cu_q, const void* kv_lens,
                                         int batch, int max_q_len, int nq, int nkv, int page_size, float scale,
-                                        int causal, void* stream) {
+                                        int causal, int window, void* stream) {
   return xllm_paged_prefill_attn_tc_lse(out, o_stride, q, q_stride, total_q, k_cache, v_cache, n_blocks, block_table,
                                         bt_stride, cu_q, kv_lens, batch, max_q_len, nq, nkv, page_size, scale, causal,
-                                        nullptr, stream);
+                                        window, nullptr, stream);
 }
 
 // 0 = no bounded wait expired in the prefill kernel on this device since the last call.

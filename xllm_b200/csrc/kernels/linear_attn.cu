@@ -16,7 +16,7 @@
 //                             products as a sum of two bf16 terms, so the recurrence keeps about 16 bits of
 //                             significand per operand and accumulates in fp32.
 //   linattn_recurrent_kernel  prompt chunks of any dtype and size, token by token in fp32
-//   head_norm_gate_kernel     finishes the fp32 outputs of the two prompt kernels
+// (head_norm.cu finishes the fp32 outputs of the two prompt kernels)
 //
 // A sequence whose rows in the batch are its first tokens (kv_len == number of rows) starts from S = 0 whatever its
 // slot holds; slot < 0 marks padding rows.  The reference has no such layer; its nearest relative is the Triton
@@ -801,35 +801,6 @@ __global__ void __launch_bounds__(256) linattn_scan_kernel(LinAttnParams<bf16> p
   *S = s;
 }
 
-// out[t, h * dv + i] = o[t, h, i] (/ rms over the head) (* w[i]) (* silu(g[t, h * dv + i]));  one warp per (t, h)
-template <typename T>
-__global__ void __launch_bounds__(256) head_norm_gate_kernel(T* __restrict__ out, int64_t out_ld, const float* __restrict__ o,
-                                                             const T* __restrict__ g, int64_t g_ld, const T* __restrict__ w,
-                                                             int64_t items, int H, int dv, int unit_norm, float eps) {
-  const int lane = threadIdx.x & 31;
-  const int64_t it = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
-  pdl_wait();
-  pdl_launch_dependents();
-  if (it >= items) return;
-  const int64_t t = it / H;
-  const int h = (int)(it - t * H);
-  const float* src = o + it * dv;
-  float inv = 1.f;
-  if (unit_norm) {
-    float ss = 0.f;
-    for (int i = lane; i < dv; i += 32) ss += src[i] * src[i];
-    inv = 1.f / sqrtf(warp_sum(ss) / (float)dv + eps);
-  }
-  T* dst = out + t * out_ld + (int64_t)h * dv;
-  const T* gr = g != nullptr ? g + t * g_ld + (int64_t)h * dv : nullptr;
-  for (int i = lane; i < dv; i += 32) {
-    float a = src[i] * inv;
-    if (w != nullptr) a *= to_f32(w[i]);
-    if (gr != nullptr) a *= silu_f32(to_f32(gr[i]));
-    dst[i] = from_f32<T>(a);
-  }
-}
-
 template <int DK, int NW, bool STATE_ONLY>
 static int launch_chunk_kernel(const LinAttnParams<bf16>& p, const SegParams& sp, int segs, cudaStream_t s) {
   using L = ChunkSmem<DK, NW>;
@@ -941,21 +912,4 @@ XLLM_API int xllm_linattn(void* state, const void* slots, const void* cu_q, cons
   if (dtype == 0) run(bf16());
   else run(float());
   return rc;
-}
-
-XLLM_API int xllm_head_norm_gate(void* out, int64_t out_ld, const void* o, const void* g, int64_t g_ld, const void* w,
-                                 int64_t tokens, int H, int dv, int unit_norm, float eps, int dtype, void* stream) {
-  using namespace xllm;
-  if (tokens == 0) return 0;
-  if (H <= 0 || dv <= 0) return (int)cudaErrorInvalidValue;
-  const int64_t items = tokens * H;
-  const dim3 grid((unsigned)((items + 7) / 8)), block(256);
-  cudaStream_t s = (cudaStream_t)stream;
-  if (dtype == 0)
-    launch_pdl(head_norm_gate_kernel<bf16>, grid, block, 0, s, (bf16*)out, out_ld, (const float*)o, (const bf16*)g, g_ld,
-               (const bf16*)w, items, H, dv, unit_norm, eps);
-  else
-    launch_pdl(head_norm_gate_kernel<float>, grid, block, 0, s, (float*)out, out_ld, (const float*)o, (const float*)g, g_ld,
-               (const float*)w, items, H, dv, unit_norm, eps);
-  return XLLM_LAUNCH_CHECK();
 }

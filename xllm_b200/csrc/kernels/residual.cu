@@ -1,7 +1,7 @@
 // An fp32 residual stream: branch outputs join it and the next sublayer's input leaves it in one pass.
 //
 //   x[t] = (init ? 0 : x[t]) + coef * sum_i n_i(y_i[t])        n_i: identity, or RMS norm with a weight
-//   out[t] = rmsnorm(x[t]) * w   or   cast(x[t])
+//   out[t] = rmsnorm(x[t]) * (w + offset)   or   cast(x[t])       offset: 1 for weights stored around zero
 //
 // One launch covers: the embedding (init, y_0 gathered by token id) + first norm; a plain branch + the
 // next norm; a branch that is normalised before it joins (post-norm) + the next norm; two branches that
@@ -26,7 +26,7 @@ struct ResidualParams {
   int64_t y_ld[2];
   int64_t n_rows;         // rows of the gathered table
   int tokens, hidden, init;
-  float coef, eps;
+  float coef, eps, w_out_offset;   // the output's norm weight is w_out + w_out_offset
 };
 
 constexpr int kResVec = 4;   // vectors per thread
@@ -135,7 +135,7 @@ __global__ void __launch_bounds__(TPR > 256 ? TPR : 256) residual_kernel(Residua
       float w[V];
       load_f32<V>(reinterpret_cast<const T*>(p.w_out) + v * V, w);
 #pragma unroll
-      for (int j = 0; j < V; ++j) o[j] = acc[i][j] * inv * w[j];
+      for (int j = 0; j < V; ++j) o[j] = acc[i][j] * inv * (w[j] + p.w_out_offset);
     } else {
 #pragma unroll
       for (int j = 0; j < V; ++j) o[j] = acc[i][j];
@@ -219,14 +219,15 @@ __global__ void __launch_bounds__(256) silu_mul_f32_kernel(float* __restrict__ o
 // dtype: 0 bf16, 1 fp32 (branches, weights, out).  y1 / w0 / w1 / rows / w_out / out may be null.
 XLLM_API int xllm_residual_update(void* x, const void* y0, int64_t y0_ld, const void* w0, const void* y1, int64_t y1_ld,
                                   const void* w1, const void* rows, int64_t n_rows, const void* w_out, void* out, int tokens,
-                                  int hidden, int init, float coef, float eps, int dtype, void* stream) {
+                                  int hidden, int init, float coef, float eps, float w_out_offset, int dtype,
+                                  void* stream) {
   using namespace xllm;
   if (tokens == 0) return 0;
   if (hidden <= 0 || y0 == nullptr || x == nullptr) return (int)cudaErrorInvalidValue;
   ResidualParams p;
   p.x = (float*)x; p.y[0] = y0; p.y[1] = y1; p.w[0] = w0; p.w[1] = w1; p.rows = (const int64_t*)rows;
   p.w_out = w_out; p.out = out; p.y_ld[0] = y0_ld; p.y_ld[1] = y1_ld; p.n_rows = n_rows; p.tokens = tokens;
-  p.hidden = hidden; p.init = init; p.coef = coef; p.eps = eps;
+  p.hidden = hidden; p.init = init; p.coef = coef; p.eps = eps; p.w_out_offset = w_out_offset;
   const auto a16 = [](const void* q) { return (((uintptr_t)q) & 15) == 0; };
   const bool al = a16(x) && a16(y0) && a16(w0) && a16(y1) && a16(w1) && a16(w_out) && a16(out);
   cudaStream_t s = (cudaStream_t)stream;

@@ -19,7 +19,7 @@ struct RopeNormParams {
   const float* cos_sin;     // [max_pos, rot]: cos | sin, or null
   const int64_t* positions;
   const int32_t* slots;     // < 0: nothing is cached
-  int tokens, nq, nkv, d, d_pad, rot, page, interleaved, unit_norm;
+  int tokens, nq, nkv, d, dv, d_pad, rot, page, interleaved, unit_norm;
   int64_t max_pos;
   float eps;
 };
@@ -89,9 +89,9 @@ __global__ void __launch_bounds__(256) rope_norm_kv_kernel(RopeNormParams<T> p) 
   }
   for (int i = p.d + lane; i < p.d_pad; i += 32) dst[i] = from_f32<T>(0.f);
   if (!is_q) {
-    const T* vs = p.v + t * p.ld + (int64_t)g * p.d;
+    const T* vs = p.v + t * p.ld + (int64_t)g * p.dv;
     T* vd = p.v_cache + crow;
-    for (int i = lane; i < p.d_pad; i += 32) vd[i] = i < p.d ? vs[i] : from_f32<T>(0.f);
+    for (int i = lane; i < p.d_pad; i += 32) vd[i] = i < p.dv ? vs[i] : from_f32<T>(0.f);
   }
 }
 
@@ -190,14 +190,14 @@ __global__ void __launch_bounds__(256) rope_norm_kv_vec_kernel(RopeNormParams<bf
 
 }  // namespace xllm
 
-// dtype: 0 bf16, 1 fp32.  rot <= d, rot even.
+// dtype: 0 bf16, 1 fp32.  rot <= d, rot even.  dv: size of a value head (d where v is the key block).
 XLLM_API int xllm_rope_norm_kv(const void* q, const void* k, const void* v, int64_t ld, void* q_out, void* k_cache,
                                void* v_cache, const void* cos_sin, int64_t max_pos, const void* positions, const void* slots,
-                               int tokens, int nq, int nkv, int d, int d_pad, int rot, int page, int interleaved, int unit_norm,
+                               int tokens, int nq, int nkv, int d, int dv, int d_pad, int rot, int page, int interleaved, int unit_norm,
                                float eps, int dtype, void* stream) {
   using namespace xllm;
   if (tokens == 0) return 0;
-  if (d <= 0 || d > 64 * kPairs || d_pad < d || rot < 0 || rot > d || rot % 2 != 0 || page <= 0 || nq <= 0 || nkv <= 0)
+  if (d <= 0 || d > 64 * kPairs || d_pad < d || dv <= 0 || d_pad < dv || rot < 0 || rot > d || rot % 2 != 0 || page <= 0 || nq <= 0 || nkv <= 0)
     return (int)cudaErrorInvalidValue;
   const int64_t items = (int64_t)tokens * (nq + nkv);
   const dim3 grid((unsigned)((items + 7) / 8)), block(256);
@@ -207,12 +207,12 @@ XLLM_API int xllm_rope_norm_kv(const void* q, const void* k, const void* v, int6
     RopeNormParams<T> p;
     p.q = (const T*)q; p.k = (const T*)k; p.v = (const T*)v; p.ld = ld; p.q_out = (T*)q_out; p.k_cache = (T*)k_cache;
     p.v_cache = (T*)v_cache; p.cos_sin = rot > 0 ? (const float*)cos_sin : nullptr; p.positions = (const int64_t*)positions;
-    p.slots = (const int32_t*)slots; p.tokens = tokens; p.nq = nq; p.nkv = nkv; p.d = d; p.d_pad = d_pad; p.rot = rot;
+    p.slots = (const int32_t*)slots; p.tokens = tokens; p.nq = nq; p.nkv = nkv; p.d = d; p.dv = dv; p.d_pad = d_pad; p.rot = rot;
     p.page = page; p.interleaved = interleaved; p.unit_norm = unit_norm; p.max_pos = max_pos; p.eps = eps;
     if constexpr (sizeof(T) == 2) {
       const auto a16 = [](const void* x) { return (((uintptr_t)x) & 15) == 0; };
       const int tph = d >> 3, hl = rot >> 4;
-      if (d % 8 == 0 && d <= 256 && (tph & (tph - 1)) == 0 && d_pad % 8 == 0 && ld % 8 == 0 && a16(q) && a16(k) && a16(v) &&
+      if (d % 8 == 0 && d == dv && d <= 256 && (tph & (tph - 1)) == 0 && d_pad % 8 == 0 && ld % 8 == 0 && a16(q) && a16(k) && a16(v) &&
           a16(q_out) && a16(k_cache) && a16(v_cache) && (rot == 0 || (rot % 8 == 0 && a16(cos_sin))) &&
           (interleaved || rot == 0 || (rot % 16 == 0 && (hl & (hl - 1)) == 0))) {
         launch_pdl(rope_norm_kv_vec_kernel, dim3(tokens), dim3(256), 0, s, p);

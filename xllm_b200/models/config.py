@@ -53,6 +53,7 @@ class ModelArgs:
     topk_group: int = 1
     routed_scaling_factor: float = 1.0
     router_bias: bool = False  # e_score_correction_bias
+    moe_group_score: str = "auto"  # expert groups rank by the sum of their two best biased scores, or by the best ("max")
     # MLA
     q_lora_rank: int = 0
     kv_lora_rank: int = 0
@@ -133,8 +134,40 @@ def _femirax_args(cfg: Dict[str, Any], shapes: Dict[str, List[int]]) -> ModelArg
     return a
 
 
+def _sodedra_args(cfg: Dict[str, Any], shapes: Dict[str, List[int]]) -> ModelArgs:
+    """Sodedra configurations list every layer; the ranks of low-rank projections are only in their tensors' shapes."""
+    import copy
+    layers = copy.deepcopy(cfg["layers"])
+    for i, layer in enumerate(layers):
+        for name in ("a1", "g1"):
+            shape = shapes.get(f"l{i}.mix.{name}")
+            if shape is not None:
+                layer["mixer"][name] = int(shape[0])
+    a = ModelArgs(model_type="sodedra", architectures=["Sodedra"], vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
+                  num_hidden_layers=len(layers), rms_norm_eps=float(cfg["norm"]["eps"]), qk_norm=False, tie_word_embeddings=True)
+    att = [l["mixer"] for l in layers if l["type"] == "attention"]
+    a.num_attention_heads = max([m["heads"] for m in att] + [1])
+    a.num_key_value_heads = max([m["kv_heads"] for m in att] + [1])
+    a.head_dim = max([max(m["dim"], m["vdim"]) for m in att] + [1])
+    # every attention layer has a window: what lies before the widest one can be given back
+    a.sliding_window = max([int(m["mask"]["size"]) for m in att] + [0])
+    mlps = [l["mlp"] for l in layers if l.get("mlp")]
+    moe = [m for m in mlps if m["kind"] == "moe"]
+    a.intermediate_size = max([m["ff"] for m in mlps if m["kind"] == "dense"] + [a.hidden_size])
+    a.num_experts = max([m["router"]["experts"] for m in moe] + [0])
+    a.num_experts_per_tok = max([m["router"]["top"] for m in moe] + [0])
+    a.moe_intermediate_size = max([m["expert"]["ff"] for m in moe] + [0])
+    a.max_position_embeddings = int(_g(cfg, "max_position_embeddings", default=32768))
+    a.extra = {"layers": layers, "embedding_scale": float(cfg["embedding"]["scale"]),
+               # positions are unbounded unless the configuration names a limit: the engine may ask for longer sequences
+               "unbounded_positions": "max_position_embeddings" not in cfg}
+    a.bos_token_id = _g(cfg, "bos_token_id", default=-1)
+    a.eos_token_id, a.stop_token_ids = _eos_list(_g(cfg, "eos_token_id"))
+    return a
+
+
 # `architecture` names whose configurations do not follow the HuggingFace layout: name -> fn(config, tensor shapes)
-_OWN_LAYOUTS = {"femirax": _femirax_args}
+_OWN_LAYOUTS = {"femirax": _femirax_args, "sodedra": _sodedra_args}
 
 
 def model_args_from_dict(cfg: Dict[str, Any], shapes: Optional[Dict[str, List[int]]] = None) -> ModelArgs:

@@ -92,7 +92,7 @@ class FemiraxCausalLM(Module):
     supports_prefill_graph = True
     # the kernel sources a process that runs nothing but this model needs
     kernel_sources = ("gemm_tcgen05", "activation", "attn_decode", "attn_prefill", "attn_prefill_tc", "attn_generic",
-                      "linear_attn", "residual", "rope_norm_kv", "misc", "sampling")
+                      "linear_attn", "head_norm", "residual", "rope_norm_kv", "misc", "sampling")
     fused_tp = False
 
     def __init__(self, args, dtype=torch.bfloat16, device="cpu", ps=None):

@@ -23,7 +23,9 @@ from ..parallel.state import single
 
 
 class SparseMoeBlock(Module):
-    def __init__(self, args, dtype, device, ps=None):
+    """`own_router=False`: the router logits come from the caller (forward's `logits`)."""
+
+    def __init__(self, args, dtype, device, ps=None, own_router=True):
         super().__init__()
         self.ps = ps or single()
         self.args = args
@@ -39,7 +41,7 @@ class SparseMoeBlock(Module):
             self.e_local, self.e_begin = E, 0
             self.i_local, i_rank, i_parts = I // tp, self.ps.tp_rank, tp
         self.top_k = args.num_experts_per_tok
-        self.gate = self.add_module("gate", Linear(H, E, False, dtype, device, self.ps))  # replicated router
+        self.gate = self.add_module("gate", Linear(H, E, False, dtype, device, self.ps)) if own_router else None  # replicated router
         il = self.i_local
         # block-scaled fp8 experts: e4m3 weights + 128 x 128 scales, grouped block-scaled GEMMs
         self.fp8 = bool(getattr(args, "fp8_execution", False)) and il % 128 == 0 and H % 128 == 0
@@ -79,13 +81,15 @@ class SparseMoeBlock(Module):
                 L_[f"experts.{ge}.down_proj.weight_scale_inv"] = lambda sc, e=e: put_s(self.s_down, e, 0, sc, 1)
         else:
             self.w_gate_up = torch.empty(self.e_local, 2 * self.i_local, H, dtype=dtype, device=device)
-            self.w_down = torch.empty(self.e_local, H, self.i_local, dtype=dtype, device=device)
+            # the grouped product writes widths in steps of 64: rows of zeros behind the hidden size
+            Y = H if ep > 1 or dtype != torch.bfloat16 or torch.device(device).type != "cuda" else (H + 63) // 64 * 64
+            self.w_down = (torch.empty if Y == H else torch.zeros)(self.e_local, Y, self.i_local, dtype=dtype, device=device)
             self._params["experts.gate_up"] = self.w_gate_up
             self._params["experts.down"] = self.w_down
         # On the device, without expert parallelism, every expert's gate|up rows are stored in groups of
         # 128 = [64 gate | 64 up of the same features]: the grouped GEMM's epilogue then applies SiLU(gate) * up
         # itself (ops/moe.py).  Expert-parallel layers keep the plain layout (their weights move between ranks).
-        self.interleaved = (not self.fp8 and ep == 1 and il % 64 == 0 and dtype == torch.bfloat16
+        self.interleaved = (not self.fp8 and ep == 1 and il % 64 == 0 and H % 8 == 0 and dtype == torch.bfloat16
                             and torch.device(device).type == "cuda" and os.environ.get("XLLM_FUSED_ACT", "1") != "0")
         if self.interleaved:
             self.w_gate_up._xllm_interleaved = True
@@ -105,7 +109,7 @@ class SparseMoeBlock(Module):
                 half(e, 1).copy_(w.narrow(0, i_rank * il, il).to(dtype).view(half(e, 1).shape))
 
             def ld(w, e=e):
-                self.w_down[e].copy_(w.narrow(1, i_rank * il, il).to(dtype))
+                self.w_down[e, :H].copy_(w.narrow(1, i_rank * il, il).to(dtype))
 
             self._loaders[f"experts.{ge}.gate_proj.weight"] = lg
             self._loaders[f"experts.{ge}.up_proj.weight"] = lu
@@ -123,12 +127,13 @@ class SparseMoeBlock(Module):
         self.shared_gate = None
         if self.shared is not None and args.extra.get("shared_expert_gate"):
             self.shared_gate = self.add_module("shared_gate", Linear(H, 1, False, dtype, device, self.ps))
-        self._ws = None
+        self._ws = {}           # every workspace a captured graph may hold
 
-    def forward(self, x):
+    def forward(self, x, logits=None):
         a = self.args
         T = x.shape[0]
-        logits = self.gate(x)
+        if logits is None:
+            logits = self.gate(x)
         shared_out = None
         if self.shared is not None:
             # the shared expert is TP-sharded like a dense MLP: its partial joins the routed partial.
@@ -150,14 +155,16 @@ class SparseMoeBlock(Module):
         out = comm.partial_buffer(T) if (comm is not None and x.is_cuda) else None
         if self._use_a2a(x, comm):
             return self._forward_a2a(x, logits, shared_out, comm, out)
-        if x.is_cuda and (self._ws is None or self._ws.max_tokens < T):
-            self._ws = moe_ops.MoeWorkspace(max(T, 256), self.top_k, a.num_experts, self.e_local, a.hidden_size,
-                                            self.i_local, x.device, x.dtype)
+        ws = None
+        if x.is_cuda:
+            ws = moe_ops.shared_workspace(T, self.top_k, a.num_experts, self.e_local, a.hidden_size, self.i_local, x.device,
+                                          x.dtype, self.w_down.shape[1])
+            self._ws[ws.max_tokens] = ws
         y = moe_ops.fused_moe(x, logits, self.w_gate_up, self.w_down, self.top_k, a.scoring_func, self.bias,
                               a.n_group, a.topk_group, a.norm_topk_prob, a.routed_scaling_factor, self.e_begin,
-                              a.num_experts, shared_out, self._ws, out,
+                              a.num_experts, shared_out, ws, out,
                               w_scales=(self.s_gate_up, self.s_down) if self.fp8 else None,
-                              interleaved=self.interleaved)
+                              interleaved=self.interleaved, group_score=a.moe_group_score)
         if out is None and self.ps.tp_size > 1:
             y = self.ps.all_reduce(y)
         return y

@@ -5,7 +5,8 @@ The scheduler admits at most `n_slots` sequences at a time and slots return on f
 xllm/core/framework/block/)."""
 from __future__ import annotations
 
-from typing import Dict, Tuple
+import math
+from typing import Dict, Tuple, Union
 
 import torch
 
@@ -34,16 +35,31 @@ class StateSlots:
 
 
 class RecurrentStatePool(StateSlots):
-    """fp32 matrix states of any set of layers: `shapes[layer] = (heads, key size, value size)`; the value size is
-    stored rounded up to four.  One more slot than `n_slots` exists: `scratch_slot`, for passes outside the scheduler.
+    """States of any set of layers, by layer: (heads, key size, value size) is one fp32 matrix state per head, the value
+    size stored rounded up to four; a dict {name: (shape, dtype)} is a state of several named parts, of which a part with
+    dtype None is such a matrix state.  One more slot than `n_slots` exists: `scratch_slot`, for passes outside the scheduler.
     Slots are not cleared: a layer ignores what a slot holds when a sequence starts at position 0."""
 
-    def __init__(self, shapes: Dict[int, Tuple[int, int, int]], n_slots: int, device):
+    def __init__(self, shapes: Dict[int, Union[Tuple[int, int, int], dict]], n_slots: int, device):
         super().__init__(n_slots)
         self.scratch_slot = n_slots
-        self.layers = {i: torch.zeros(n_slots + 1, h, dk, (dv + 3) // 4 * 4, dtype=torch.float32, device=device)
-                       for i, (h, dk, dv) in shapes.items()}
+
+        def make(part):
+            shape, dtype = self._stored(part)
+            return torch.zeros(n_slots + 1, *shape, dtype=dtype, device=device)
+
+        self.layers = {i: {n: make(p) for n, p in s.items()} if isinstance(s, dict) else make((s, None))
+                       for i, s in shapes.items()}
+
+    @staticmethod
+    def _stored(part):
+        shape, dtype = part
+        if dtype is not None:
+            return tuple(shape), dtype
+        h, dk, dv = shape
+        return (h, dk, (dv + 3) // 4 * 4), torch.float32
 
     @staticmethod
     def bytes_per_slot(shapes) -> int:
-        return sum(h * dk * ((dv + 3) // 4 * 4) * 4 for h, dk, dv in shapes.values())
+        parts = [p for s in shapes.values() for p in (s.values() if isinstance(s, dict) else [(s, None)])]
+        return sum(math.prod(shape) * dtype.itemsize for shape, dtype in map(RecurrentStatePool._stored, parts))

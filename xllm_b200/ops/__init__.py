@@ -145,9 +145,10 @@ def rope_norm_kv_write(q, k, v, nq, nkv, d, positions, cos_sin, rot, slots, k_ca
                        interleaved=False, unit_norm=True):
     """Rotary positions on the first `rot` elements of every q and k head, THEN (`unit_norm`) each head divided by its
     root mean square; k and v rows are scattered into the paged caches.  q, k, v: column blocks [T, heads * d] of the
-    same projection rows (v may be the key block).  The caches may hold wider heads than d (zero filled); returns q
-    [T, nq, cache head size]."""
+    same projection rows (v may be the key block, or have heads of a size of its own).  The caches may hold wider heads
+    than that (zero filled); returns q [T, nq, cache head size]."""
     T, dp = q.shape[0], k_cache.shape[3]
+    dv = v.shape[1] // nkv
     if _debug.enabled():
         _debug.check_range(positions, 0, cos_sin.shape[0], "rope_norm_kv_write positions")
         _debug.check_range(slots, 0, k_cache.shape[0] * k_cache.shape[2], "rope_norm_kv_write slots", allow_negative_skip=True)
@@ -161,7 +162,7 @@ def rope_norm_kv_write(q, k, v, nq, nkv, d, positions, cos_sin, rot, slots, k_ca
     out = torch.empty((T, nq, dp), dtype=q.dtype, device=q.device)
     check(_lib_().xllm_rope_norm_kv(ptr(q), ptr(k), ptr(v), q.stride(0), ptr(out), ptr(k_cache), ptr(v_cache), ptr(cos_sin),
                                     cos_sin.shape[0] if cos_sin is not None else 0, ptr(positions), ptr(slots), T, nq, nkv, d,
-                                    dp, rot, k_cache.shape[2], int(interleaved), int(unit_norm), eps,
+                                    dv, dp, rot, k_cache.shape[2], int(interleaved), int(unit_norm), eps,
                                     0 if q.dtype == torch.bfloat16 else 1, stream()), "rope_norm_kv")
     _count()
     return out
@@ -290,13 +291,13 @@ def paged_prefill_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, max
         out = torch.empty((T, nq, d), dtype=q.dtype, device=q.device)
     assert q.stride(-1) == 1 and q.stride(1) == d
     B = kv_lens.shape[0]
-    if (d == 128 and window == 0 and page in (16, 32, 64, 128) and k_cache.is_contiguous() and v_cache.is_contiguous()
+    if (d == 128 and page in (16, 32, 64, 128) and k_cache.is_contiguous() and v_cache.is_contiguous()
             and os.environ.get("XLLM_PREFILL_ATTN", "tcgen05") != "legacy"):
         # tcgen05 / TMEM kernel (csrc/kernels/attn_prefill_tc.cu)
         check(_lib_().xllm_paged_prefill_attn_tc(ptr(out), out.stride(0), ptr(q), q.stride(0), T, ptr(k_cache),
                                                  ptr(v_cache), k_cache.shape[0], ptr(block_table),
                                                  block_table.stride(0), ptr(cu_q), ptr(kv_lens), B, int(max_q_len),
-                                                 nq, nkv, page, scale, int(causal), stream()),
+                                                 nq, nkv, page, scale, int(causal), int(window), stream()),
               "paged_prefill_attn_tc")
         _count()
         return out
@@ -458,4 +459,4 @@ def resolve_placeholders(tokens, prev):
     return tokens
 
 
-from .gemm import linear  # noqa: E402,F401
+from .gemm import linear, linear_f32  # noqa: E402,F401

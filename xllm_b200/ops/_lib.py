@@ -104,7 +104,7 @@ def _declare(lib):
         "xllm_paged_decode_attn_window": [P, P, L, P, P, P, I, P, I, I, I, I, I, F, I, P, I, P],
         "xllm_attn_merge": [P, P, P, L, I, I, P],
         "xllm_paged_prefill_attn": [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, F, I, I, P],
-        "xllm_paged_prefill_attn_tc": [P, L, P, L, L, P, P, L, P, I, P, P, I, I, I, I, I, F, I, P],
+        "xllm_paged_prefill_attn_tc": [P, L, P, L, L, P, P, L, P, I, P, P, I, I, I, I, I, F, I, I, P],
         "xllm_fmha_error_status": [],
         "xllm_sample": [P, L, I, I, I, P, P, P, P, P, U64, U64, P],
         "xllm_sample_rows": [P, L, I, I, I, P, P, P, P, P, P, P, P],
@@ -116,7 +116,8 @@ def _declare(lib):
         "xllm_block_copy": [P, I, P, I, L, P],
         "xllm_decode_advance": [P, P, P, P, P, I, P, I, I, P],
         "xllm_resolve_placeholders": [P, P, L, L, P],
-        "xllm_rope_norm_kv": [P, P, P, L, P, P, P, P, L, P, P, I, I, I, I, I, I, I, I, I, F, I, P],
+        "xllm_rope_norm_kv": [P, P, P, L, P, P, P, P, L, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P],
+        "xllm_proj_f32": [P, L, P, L, P, P, I, I, I, P],
         "xllm_paged_attn_generic": [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, I, F, I, I, P],
         "xllm_silu_mul_f32": [P, P, L, I, L, P],
     }

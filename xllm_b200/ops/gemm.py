@@ -60,3 +60,20 @@ def linear(x, w, bias=None, out=None):
         out.copy_(y)
         return out
     return y
+
+
+def linear_f32(x, w, bias=None):
+    """x @ W^T (+ bias) as fp32, for results that must not be rounded to the activations' type (router logits, gates of a
+    recurrence).  Meant for few outputs (csrc/kernels/proj_f32.cu)."""
+    if x.is_cuda and x.dtype == torch.bfloat16:
+        T, K = x.shape
+        if K % 8 == 0 and x.stride(1) == 1 and x.stride(0) % 8 == 0 and not (x.data_ptr() | w.data_ptr()) & 15 and w.is_contiguous():
+            from . import _count, _lib
+            from ._lib import check, ptr, stream
+            out = torch.empty((T, w.shape[0]), dtype=torch.float32, device=x.device)
+            check(_lib.load().xllm_proj_f32(ptr(out), out.stride(0), ptr(x), x.stride(0), ptr(w), ptr(bias), T, w.shape[0], K,
+                                            stream()), "proj_f32")
+            _count()
+            return out
+        _note_fallback("fp32 result, shape or alignment", x, w)
+    return F.linear(x.float(), w.float(), None if bias is None else bias.float())

@@ -12,9 +12,9 @@ import torch
 
 from . import _lib
 from ._lib import F, I, L, P, check, ptr, stream
+from .head_norm import head_norm_gate
 
 _lib.register_signature("xllm_linattn", [P] * 9 + [L, P, L, P, P, P, P, P, P, L] + [I] * 8 + [F] * 4 + [I, I, P, P, I, I, I, P])
-_lib.register_signature("xllm_head_norm_gate", [P, L, P, P, L, P, L, I, I, I, F, I, P])
 
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 
@@ -110,12 +110,7 @@ class LinearAttention:
 
     def finish(self, o, g, out):
         """Per-head norm, weight and gate of raw fp32 outputs o [T, heads, dv]."""
-        check(_lib.load().xllm_head_norm_gate(ptr(out), out.stride(0), ptr(o), ptr(g), g.stride(0) if g is not None else 0,
-                                              ptr(self.norm_w), o.shape[0], self.heads, self.dv, int(self.unit_norm),
-                                              self.eps, _DT[out.dtype], stream()), "head_norm_gate")
-        from . import _count
-        _count()
-        return out
+        return head_norm_gate(o, out, g=g, w=self.norm_w, unit_norm=self.unit_norm, eps=self.eps)
 
     # ------------------------------------------------------------------ tensor-op form
     def _rope(self, x, positions):

@@ -7,28 +7,34 @@ tcgen05 GEMM); the reference calls FlashInfer's CUTLASS MoE runner for the same 
 """
 from __future__ import annotations
 
+import weakref
+
 import torch
 
 from . import _lib
 from ._lib import F, I, L, P, check, ptr, stream
 
 _lib.register_signature("xllm_moe_route", [P, I, P, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P])
+_lib.register_signature("xllm_moe_route_ld", [P, L, I, P, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P])
 _lib.register_signature("xllm_moe_offsets", [P, P, P, P, I, I, I, P])
-_lib.register_signature("xllm_moe_permute", [P, P, P, P, P, P, I, I, I, P])
-_lib.register_signature("xllm_moe_finalize", [P, P, P, P, P, I, I, I, P])
+_lib.register_signature("xllm_moe_permute", [P, P, P, P, P, P, I, I, I, I, P])
+_lib.register_signature("xllm_moe_finalize", [P, P, L, P, P, P, I, I, I, I, P])
+_lib.register_signature("xllm_moe_grouped_simt", [P, P, P, P, I, I, I, L, L, I, P])
 _lib.register_signature("xllm_gemm_bf16_grouped", [P, P, P, P, I, I, I, I, L, L, P])
 _lib.register_signature("xllm_gemm_bf16_grouped_act_mul", [P, P, P, P, I, I, I, I, L, L, I, P])
 
 
-def route_reference(logits, top_k, scoring="softmax", bias=None, n_group=1, topk_group=1, renorm=True, scale=1.0):
-    """Returns (ids [T,K] int64, weights [T,K] fp32)."""
+def route_reference(logits, top_k, scoring="softmax", bias=None, n_group=1, topk_group=1, renorm=True, scale=1.0,
+                    group_score="auto"):
+    """Returns (ids [T,K] int64, weights [T,K] fp32).  group_score: a group counts by its best selection score ("max"), or
+    ("auto") by the sum of its two best when there is a bias."""
     x = logits.float()
     scores = torch.softmax(x, -1) if scoring == "softmax" else torch.sigmoid(x)
     sel = scores + bias.float() if bias is not None else scores
     if n_group > 1 and topk_group < n_group:
         T, E = sel.shape
         g = sel.view(T, n_group, E // n_group)
-        gs = g.topk(2, dim=-1).values.sum(-1) if bias is not None else g.max(-1).values
+        gs = g.topk(2, dim=-1).values.sum(-1) if bias is not None and group_score == "auto" else g.max(-1).values
         keep = torch.zeros_like(gs, dtype=torch.bool).scatter_(1, gs.topk(topk_group, dim=-1).indices, True)
         sel = sel.masked_fill(~keep[:, :, None].expand_as(g).reshape(T, E), float("-inf"))
     ids = sel.topk(top_k, dim=-1).indices
@@ -39,8 +45,8 @@ def route_reference(logits, top_k, scoring="softmax", bias=None, n_group=1, topk
 
 
 def fused_moe_reference(x, logits, w_gate_up, w_down, top_k, scoring="softmax", bias=None, n_group=1, topk_group=1,
-                        renorm=True, scale=1.0, expert_begin=0, shared_out=None, act="silu"):
-    ids, w = route_reference(logits, top_k, scoring, bias, n_group, topk_group, renorm, scale)
+                        renorm=True, scale=1.0, expert_begin=0, shared_out=None, act="silu", group_score="auto"):
+    ids, w = route_reference(logits, top_k, scoring, bias, n_group, topk_group, renorm, scale, group_score)
     out = torch.zeros_like(x, dtype=torch.float32)
     if shared_out is not None:
         out += shared_out.float()
@@ -61,7 +67,7 @@ def fused_moe_reference(x, logits, w_gate_up, w_down, top_k, scoring="softmax", 
 class MoeWorkspace:
     """Static-size buffers of one MoE layer shape (sized for max_tokens; reusable across layers)."""
 
-    def __init__(self, max_tokens, top_k, n_experts, n_local, hidden, inter, device, dtype=torch.bfloat16):
+    def __init__(self, max_tokens, top_k, n_experts, n_local, hidden, inter, device, dtype=torch.bfloat16, y_width=None):
         self.rows = (max_tokens * top_k + n_local * 127 + 127) // 128 * 128
         self.max_tiles = self.rows // 128
         i32 = dict(dtype=torch.int32, device=device)
@@ -76,14 +82,30 @@ class MoeWorkspace:
         self.xp = torch.zeros(self.rows, hidden, dtype=dtype, device=device)
         self.h = torch.zeros(self.rows, 2 * inter, dtype=dtype, device=device)
         self.a = torch.zeros(self.rows, inter, dtype=dtype, device=device)
-        self.y = torch.zeros(self.rows, hidden, dtype=dtype, device=device)
+        self.y = torch.zeros(self.rows, y_width or hidden, dtype=dtype, device=device)
         self.max_tokens = max_tokens
+
+
+_WORKSPACES = weakref.WeakValueDictionary()
+
+
+def shared_workspace(T, *key):
+    """The workspace of at least T tokens for one layer shape (`key`: the rest of MoeWorkspace's arguments), common to the
+    layers of that shape, which run one after another.  The caller keeps what it gets: captured graphs hold its address,
+    so a larger batch takes another workspace beside it."""
+    cap = max(256, 1 << (T - 1).bit_length())
+    k = (cap, *(str(x) for x in key))
+    ws = _WORKSPACES.get(k)
+    if ws is None:
+        ws = _WORKSPACES[k] = MoeWorkspace(cap, *key)
+    return ws
 
 
 def fused_moe(x, logits, w_gate_up, w_down, top_k, scoring="softmax", bias=None, n_group=1, topk_group=1,
               renorm=True, scale=1.0, expert_begin=0, n_experts=None, shared_out=None, ws: MoeWorkspace = None,
-              out=None, w_scales=None, interleaved=False):
-    """x [T,H], logits [T,E]; w_gate_up [E_local, 2I, H], w_down [E_local, H, I] -> [T,H].
+              out=None, w_scales=None, interleaved=False, group_score="auto"):
+    """x [T,H], logits [T,E]; w_gate_up [E_local, 2I, H], w_down [E_local, H, I] -> [T,H].  w_down may have more rows than H (zeros
+    that make the product's width one the tensor-core kernel takes).
     `interleaved`: every expert's gate|up rows are stored in groups of 128 = [64 gate | the 64 up rows of the
     same features] (`ops.gemm_tcgen05.interleave_gate_up`); the first grouped GEMM then applies SiLU(gate) * up
     in its epilogue and the [rows, 2I] intermediate is never written.
@@ -98,27 +120,30 @@ def fused_moe(x, logits, w_gate_up, w_down, top_k, scoring="softmax", bias=None,
             from . import fp8
             w_gate_up = torch.stack([fp8.dequant_block128_ref(w_gate_up[e], w_scales[0][e], x.dtype) for e in range(w_gate_up.shape[0])])
             w_down = torch.stack([fp8.dequant_block128_ref(w_down[e], w_scales[1][e], x.dtype) for e in range(w_down.shape[0])])
-        return fused_moe_reference(x, logits, w_gate_up, w_down, top_k, scoring, bias, n_group, topk_group, renorm,
-                                   scale, expert_begin, shared_out)
+        return fused_moe_reference(x, logits, w_gate_up, w_down[:, :x.shape[1]], top_k, scoring, bias, n_group, topk_group, renorm,
+                                   scale, expert_begin, shared_out, group_score=group_score)
     from . import _count, act_and_mul
     lib = _lib.load()
     T, H = x.shape
     E = logits.shape[1]
     E_local, I2, _ = w_gate_up.shape
-    inter = I2 // 2
+    inter, Y, dt = I2 // 2, w_down.shape[1], 0 if x.dtype == torch.bfloat16 else 1
+    x = x.contiguous()
     if ws is None or ws.max_tokens < T:
-        ws = MoeWorkspace(T, top_k, E, E_local, H, inter, x.device, x.dtype)
+        ws = MoeWorkspace(T, top_k, E, E_local, H, inter, x.device, x.dtype, Y)
     s = stream()
+    if logits.stride(1) != 1:
+        logits = logits.contiguous()
     lf = logits.dtype == torch.float32
     if not lf and logits.dtype != torch.bfloat16:
         logits, lf = logits.float(), True
-    check(lib.xllm_moe_route(ptr(logits), int(lf), ptr(bias), ptr(ws.topk_ids), ptr(ws.topk_w), ptr(ws.counts),
-                             ptr(ws.slot), T, E, top_k, n_group, topk_group, 0 if scoring == "softmax" else 1,
-                             int(renorm), float(scale), expert_begin, expert_begin + E_local, s), "moe_route")
+    check(lib.xllm_moe_route_ld(ptr(logits), logits.stride(0), int(lf), ptr(bias), ptr(ws.topk_ids), ptr(ws.topk_w), ptr(ws.counts),
+                             ptr(ws.slot), T, E, top_k, n_group, topk_group,
+                             (0 if scoring == "softmax" else 1) + (2 if group_score == "max" else 0), int(renorm), float(scale), expert_begin, expert_begin + E_local, s), "moe_route")
     check(lib.xllm_moe_offsets(ptr(ws.counts), ptr(ws.offsets), ptr(ws.tile_expert), ptr(ws.meta), E, ws.max_tiles,
                                expert_begin, s), "moe_offsets")
     check(lib.xllm_moe_permute(ptr(ws.xp), ptr(ws.rows_of), ptr(x), ptr(ws.topk_ids), ptr(ws.slot), ptr(ws.offsets),
-                               T, top_k, H, s), "moe_permute")
+                               T, top_k, H, dt, s), "moe_permute")
     if w_scales is not None:
         from . import fp8
         xq, xs = fp8.quant_group128(ws.xp)
@@ -126,6 +151,15 @@ def fused_moe(x, logits, w_gate_up, w_down, top_k, scoring="softmax", bias=None,
         act_and_mul(ws.h, "silu", out=ws.a)
         aq, as_ = fp8.quant_group128(ws.a)
         fp8.block_scaled_mm_grouped(aq, as_, w_down, w_scales[1], ws.tile_expert, ws.y)
+    elif dt == 1 or H % 8 or I2 % 64 or inter % 8 or Y % 64:
+        # fp32, or sizes the tensor-core kernel does not take
+        simt = lambda a, w, c: check(lib.xllm_moe_grouped_simt(ptr(a), ptr(w), ptr(c), ptr(ws.tile_expert), ws.rows, c.shape[1],
+                                                               a.shape[1], a.stride(0), c.stride(0), dt, s), "moe_gemm_simt")
+        if interleaved:
+            raise ValueError("interleaved expert rows need the tensor-core product")
+        simt(ws.xp, w_gate_up, ws.h)
+        act_and_mul(ws.h, "silu", out=ws.a)
+        simt(ws.a, w_down, ws.y)
     else:
         if interleaved:
             check(lib.xllm_gemm_bf16_grouped_act_mul(ptr(ws.xp), ptr(w_gate_up), ptr(ws.a), ptr(ws.tile_expert), ws.rows,
@@ -134,11 +168,11 @@ def fused_moe(x, logits, w_gate_up, w_down, top_k, scoring="softmax", bias=None,
             check(lib.xllm_gemm_bf16_grouped(ptr(ws.xp), ptr(w_gate_up), ptr(ws.h), ptr(ws.tile_expert), ws.rows, I2, H,
                                              E_local, H, I2, s), "moe_gemm1")
             act_and_mul(ws.h, "silu", out=ws.a)
-        check(lib.xllm_gemm_bf16_grouped(ptr(ws.a), ptr(w_down), ptr(ws.y), ptr(ws.tile_expert), ws.rows, H, inter,
-                                         E_local, inter, H, s), "moe_gemm2")
+        check(lib.xllm_gemm_bf16_grouped(ptr(ws.a), ptr(w_down), ptr(ws.y), ptr(ws.tile_expert), ws.rows, Y, inter,
+                                         E_local, inter, Y, s), "moe_gemm2")
     if out is None:
         out = torch.empty_like(x)
-    check(lib.xllm_moe_finalize(ptr(out), ptr(ws.y), ptr(ws.rows_of), ptr(ws.topk_w), ptr(shared_out), T, top_k, H, s),
+    check(lib.xllm_moe_finalize(ptr(out), ptr(ws.y), Y, ptr(ws.rows_of), ptr(ws.topk_w), ptr(shared_out), T, top_k, H, dt, s),
           "moe_finalize")
     _count(6)
     return out

@@ -148,8 +148,8 @@ def rope_norm_kv(q, k, v, nq, nkv, d, positions, cos_sin, rot, slots, k_cache, v
             x = torch.cat([xr, x[..., rot:]], dim=-1)
         return x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) if unit_norm else x
 
-    pad = lambda x: torch.nn.functional.pad(x, (0, dp - d)).to(k_cache.dtype)
-    write_kv_cache(pad(prep(k, nkv)), pad(v.reshape(T, nkv, d).float()), k_cache, v_cache, slots)
+    pad = lambda x: torch.nn.functional.pad(x, (0, dp - x.shape[-1])).to(k_cache.dtype)
+    write_kv_cache(pad(prep(k, nkv)), pad(v.reshape(T, nkv, -1).float()), k_cache, v_cache, slots)
     return pad(prep(q, nq))
 
 

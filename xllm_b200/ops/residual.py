@@ -7,15 +7,16 @@ import torch
 from . import _lib
 from ._lib import F, I, L, P, check, ptr, stream
 
-_lib.register_signature("xllm_residual_update", [P, P, L, P, P, L, P, P, L, P, P, I, I, I, F, F, I, P])
+_lib.register_signature("xllm_residual_update", [P, P, L, P, P, L, P, P, L, P, P, I, I, I, F, F, F, I, P])
 _lib.register_signature("xllm_gelu_mul_rows", [P, P, L, P, L, L, P, L, I, I, I, I, P])
 
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 
 
-def residual_update(x, y, w=None, y2=None, w2=None, coef=1.0, rows=None, w_out=None, eps=1e-6, want_out=True):
+def residual_update(x, y, w=None, y2=None, w2=None, coef=1.0, rows=None, w_out=None, eps=1e-6, want_out=True,
+                    w_out_offset=0.0):
     """x <- x + coef * (n(y) + n(y2)), n = RMS norm with the branch's weight (w, w2) or the identity without one;
-    returns (x, out) with out = rmsnorm(x) * w_out, or x cast to the branch type when w_out is None (None when
+    returns (x, out) with out = rmsnorm(x) * (w_out + w_out_offset), or x cast to the branch type when w_out is None (None when
     `want_out` is false).  x is fp32 [T, H] and updated in place; x None starts the stream: x = coef * n(y).
     `rows`: y is a table and row t joins as y[rows[t]] (token embedding)."""
     T = rows.shape[0] if rows is not None else y.shape[0]
@@ -34,7 +35,7 @@ def residual_update(x, y, w=None, y2=None, w2=None, coef=1.0, rows=None, w_out=N
             x += add * coef
         out = None
         if want_out:
-            out = (x if w_out is None else x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w_out.float()).to(y.dtype)
+            out = (x if w_out is None else x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * (w_out.float() + w_out_offset)).to(y.dtype)
             if out is x:
                 out = x.clone()
         return x, out
@@ -46,7 +47,7 @@ def residual_update(x, y, w=None, y2=None, w2=None, coef=1.0, rows=None, w_out=N
     out = torch.empty((T, H), dtype=y.dtype, device=y.device) if want_out else None
     check(_lib.load().xllm_residual_update(
         ptr(x), ptr(y), y.stride(0), ptr(w), ptr(y2), y2.stride(0) if y2 is not None else 0, ptr(w2), ptr(rows), y.shape[0],
-        ptr(w_out), ptr(out), T, H, int(init), float(coef), float(eps), _DT[y.dtype], stream()), "residual_update")
+        ptr(w_out), ptr(out), T, H, int(init), float(coef), float(eps), float(w_out_offset), _DT[y.dtype], stream()), "residual_update")
     from . import _count
     _count()
     return x, out

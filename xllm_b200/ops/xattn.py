@@ -28,7 +28,7 @@ from ._lib import I, L, P, F, check, ptr, stream
 TAIL_MAX = 8
 
 _lib.register_signature("xllm_paged_prefill_attn_tc_lse",
-                        [P, L, P, L, L, P, P, L, P, I, P, P, I, I, I, I, I, F, I, P, P])
+                        [P, L, P, L, L, P, P, L, P, I, P, P, I, I, I, I, I, F, I, I, P, P])
 _lib.register_signature("xllm_xattn_tail_merge", [P, L, P, P, L, P, P, P, I, I, I, I, I, I, I, F, P])
 
 
@@ -95,7 +95,7 @@ def xattention(q, k_cache, v_cache, block_table, cu_q, kv_lens, max_rows, ku, vu
     B = kv_lens.shape[0]
     check(lib.xllm_paged_prefill_attn_tc_lse(ptr(out), out.stride(0), ptr(q), q.stride(0), T, ptr(k_cache), ptr(v_cache),
                                              k_cache.shape[0], ptr(block_table), block_table.stride(0), ptr(cu_q),
-                                             ptr(kv_lens), B, int(max_rows), nq, nkv, page, scale, 0, ptr(lse), stream()),
+                                             ptr(kv_lens), B, int(max_rows), nq, nkv, page, scale, 0, 0, ptr(lse), stream()),
           "xattention shared stage")
     anc = (anc if anc.dtype == torch.int32 else anc.to(torch.int32))
     if anc.stride(-1) != 1:
