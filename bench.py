@@ -6,7 +6,7 @@ BASELINE.json on N GPUs of one node.
     python bench.py --gpus 1 --steps 20 --warmup 5  # config 2, K steps of the steady state
     python bench.py --gpus 8 --config 3 --steps 20  # Qwen3-32B shape, chunked 2048-token prefill
     python bench.py --gpus 8 --config 4 --steps 20  # Qwen3-30B-A3B shape, EP + DP attention
-    python bench.py --design femirax                # Femirax at a few sizes beside Qwen3-Next (benchmarks/femirax_bench.py)
+    python bench.py --design femirax                # a model design at a few sizes beside Qwen3-Next (benchmarks/design_bench.py; also sodedra)
 
 Workload (config 2): Qwen3-8B-shaped bf16 decoder, random-init weights, 1024 requests of uniform
 random token ids, input 1024 / output 512 with ignore_eos, at most 256 requests in flight (a closed
@@ -497,8 +497,8 @@ def main():
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="xllm_b200", choices=["xllm_b200", "ours", "reference", "library"])
     ap.add_argument("--library-attention", default="", help="library arm: attention backend name handed to vLLM")
-    ap.add_argument("--design", default="", choices=["", "femirax"],
-                    help="throughput of one model design at a few sizes, beside the closest model (benchmarks/femirax_bench.py)")
+    ap.add_argument("--design", default="", choices=["", "femirax", "sodedra"],
+                    help="throughput of one model design at a few sizes, beside the closest model (benchmarks/design_bench.py)")
     ap.add_argument("--config", default="2", choices=sorted(CONFIGS), help="BASELINE.json config number")
     ap.add_argument("--model", default="")
     ap.add_argument("--requests", type=int, default=0)
@@ -524,10 +524,10 @@ def main():
         return 0
     if args.impl == "library":
         return run_library(args)
-    if args.design == "femirax":
+    if args.design:
         sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "benchmarks"))
-        import femirax_bench
-        femirax_bench.run(args.steps or 40, args.warmup, ClockSampler(0))
+        import design_bench
+        design_bench.run(args.design, args.steps or 40, args.warmup, ClockSampler(0))
         return 0
     world = int(os.environ.get("WORLD_SIZE", "1"))
     if args.gpus > 1 and world == 1:

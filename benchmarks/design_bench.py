@@ -1,8 +1,9 @@
 #!/usr/bin/env python
-"""Prefill and decode throughput of Femirax beside the framework's closest model (Qwen3-Next: three gated-delta-net
-layers per attention layer) at equal size, random weights, one GPU.
+"""Prefill and decode throughput of one model design beside the framework's closest model (Qwen3-Next: three
+gated-delta-net layers per attention layer) at equal size, random weights, one GPU.
 
     python bench.py --design femirax [--steps K] [--warmup W]      # prints one JSON line
+    python bench.py --design sodedra
 
 Prefill: four prompts of 2048 tokens in one step.  Decode: 64 sequences of 512 prompt tokens, one token each per step.
 Both go through the engine (scheduler, state slots, cache, sampling) and are timed with CUDA events around K steps
@@ -18,6 +19,7 @@ sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 
 SIZES = {"1024": 1024, "2048": 2048, "4096": 4096}
 LAYERS, VOCAB, SIDE = 8, 32768, 64
+EXPERTS, TOP = 32, 4
 
 
 def femirax_args(W):
@@ -35,6 +37,23 @@ def femirax_args(W):
                                  "token_side": {"dim": SIDE}, "layers": [par if i % 4 == 3 else ret for i in range(LAYERS)]})
 
 
+def sodedra_args(W):
+    """Two delta-rule layers and one matrix-memory layer per attention layer; every other layer with experts."""
+    from xllm_b200.models import model_args_from_dict
+    H = W // 128
+    dense = {"ff": 3 * W, "kind": "dense"}
+    moe = {"kind": "moe", "expert": {"ff": W // 2},
+           "router": {"experts": EXPERTS, "top": TOP, "scale": 1.0, "groups": {"count": 8, "keep": 4}}}
+    delta = ("channel_delta", {"heads": H, "kv_heads": H, "dim": 128, "vdim": 128, "conv": 4, "a1": 128, "g1": 128})
+    mlstm = ("mlstm", {"heads": H, "dim": 128, "vdim": 128, "gate_cap": 15.0})
+    att = ("attention", {"heads": H, "kv_heads": max(1, H // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                         "mask": {"size": 1024}, "rot": {"base": 1e6, "dims": 128}})
+    kinds = [delta, mlstm, delta, att]
+    layers = [{"type": kinds[i % 4][0], "mixer": dict(kinds[i % 4][1]), "mlp": moe if i % 2 else dense} for i in range(LAYERS)]
+    return model_args_from_dict({"architecture": "Sodedra", "vocab": VOCAB, "width": W, "norm": {"eps": 1e-6},
+                                 "embedding": {"scale": 1.0}, "layers": layers})
+
+
 def qwen3_next_args(W):
     from xllm_b200.models import ModelArgs
     H = W // 128
@@ -43,6 +62,15 @@ def qwen3_next_args(W):
                      max_position_embeddings=32768, tie_word_embeddings=False,
                      extra=dict(linear_num_value_heads=H, linear_num_key_heads=H, linear_key_head_dim=128,
                                 linear_value_head_dim=128, linear_conv_kernel_dim=4, full_attention_interval=4))
+
+
+def qwen3_next_moe_args(W):
+    import dataclasses
+    return dataclasses.replace(qwen3_next_args(W), num_experts=EXPERTS, num_experts_per_tok=TOP, moe_intermediate_size=W // 2,
+                               moe_layer_freq=2)
+
+
+DESIGNS = {"femirax": ("Femirax", femirax_args, qwen3_next_args), "sodedra": ("Sodedra", sodedra_args, qwen3_next_moe_args)}
 
 
 def engine_of(args):
@@ -102,30 +130,31 @@ def measure(args, steps, warmup):
     return out
 
 
-def run(steps=40, warmup=8, sampler=None):
+def run(design, steps=40, warmup=8, sampler=None):
+    title, make_args, make_closest = DESIGNS[design]
     rows = []
     launches = 0
     if sampler is not None:
         sampler.start()
     for name, W in SIZES.items():
         row = {"width": W}
-        for model, make in (("femirax", femirax_args), ("qwen3_next", qwen3_next_args)):
+        for model, make in ((design, make_args), ("qwen3_next", make_closest)):
             row[model] = measure(make(W), steps, max(3, warmup))
-        launches += row["femirax"]["launches"]
-        row["prefill_ratio"] = round(row["femirax"]["prefill_tok_s"] / row["qwen3_next"]["prefill_tok_s"], 2)
-        row["decode_ratio"] = round(row["femirax"]["decode_tok_s"] / row["qwen3_next"]["decode_tok_s"], 2)
+        launches += row[design]["launches"]
+        row["prefill_ratio"] = round(row[design]["prefill_tok_s"] / row["qwen3_next"]["prefill_tok_s"], 2)
+        row["decode_ratio"] = round(row[design]["decode_tok_s"] / row["qwen3_next"]["decode_tok_s"], 2)
         rows.append(row)
     clocks = sampler.stop() if sampler is not None else None
-    big = rows[-1]["femirax"]
+    big = rows[-1][design]
     print(json.dumps({
-        "metric": "Femirax decode tok/s", "value": big["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": steps,
+        "metric": f"{title} decode tok/s", "value": big["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": steps,
         "warmup": warmup, "ms_per_step": big["decode_ms"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None,
         "dtype": "bf16", "data": "synthetic tokens, random weights", "impl": "xllm_b200",
-        "config": {"model": f"Femirax, {LAYERS} layers, widths {list(SIZES.values())}, beside Qwen3-Next of equal size",
+        "config": {"model": f"{title}, {LAYERS} layers, widths {list(SIZES.values())}, beside Qwen3-Next of equal size",
                    "prefill": "4 x 2048 tokens in one step", "decode": "64 sequences behind 512 prompt tokens",
                    "l2": "weights and states larger than L2"},
         "sizes": rows, "gpu_launches": launches, "clocks": clocks}), flush=True)
 
 
 if __name__ == "__main__":
-    run()
+    run(sys.argv[1])

@@ -383,6 +383,125 @@ def hybrid_rows(results, hbm, tf, tag):
             report("side proj, cuBLAS", f"T={T} dim={dim}", bench_queued(lambda: torch.nn.functional.linear(gate, wp)), nb, fl)
 
 
+def recurrent_rows(results, hbm, tf, tag):
+    """The kernels of Sodedra beside their likes: gated delta rule with channel decays and matrix memory against the gated
+    delta rule of Qwen3-Next and the decayed linear attention of Femirax (decode, prompts), windowed attention against the
+    same kernels without a window, head norms and gates, fp32 projections, expert layers.  32 heads of 128, width 4096."""
+    from xllm_b200.ops import gdn, moe
+    from xllm_b200.ops.delta_rule import ChannelDelta
+    from xllm_b200.ops.head_norm import head_gate, head_norm_gate
+    from xllm_b200.ops.linear_attn import LinearAttention
+    from xllm_b200.ops.mlstm import MatrixMemory
+    from xllm_b200.ops.residual import residual_update
+    dev, bf, H, d, W, R = "cuda", torch.bfloat16, 32, 128, 4096, 128
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    rows = lambda t, n: torch.randn(t, n, device=dev, dtype=bf)
+
+    def report(name, shape, t, nbytes, flops=0.0):
+        ideal = max(nbytes / (hbm * 1e9), flops / (tf * 1e12))
+        results.append(dict(kernel=name, shape=shape, ms=t * 1e3, gbs=nbytes / t / 1e9, tflops=flops / t / 1e12,
+                            frac_of_roofline=ideal / t, peaks=tag))
+        print(f"{name:<34} {shape:<26} {t*1e6:9.1f} us {nbytes/t/1e9:7.0f} GB/s {flops/t/1e12:7.1f} TF/s  {ideal/t:6.3f} of {tag}",
+              flush=True)
+
+    delta = ChannelDelta(H, H, d, d, 4, q_scale=d ** -0.5, conv_w=rows(3 * H * d, 4) * 0.5, a2=rows(H * d, R) * 0.05,
+                         dt_bias=torch.full((H * d,), -4.0, device=dev, dtype=bf), a_log=torch.zeros(H, device=dev, dtype=bf),
+                         norm_w=torch.ones(d, device=dev, dtype=bf))
+    mem = MatrixMemory(H, d, d, 15.0, q_scale=d ** -0.5, norm_w=torch.ones(H * d, device=dev, dtype=bf))
+    lin = LinearAttention(H, d, d, k_scale=d ** -0.5)
+    lin.log_decay = torch.full((H,), -0.01, device=dev)
+    cut = lambda r: [r[:, i * H * d:(i + 1) * H * d] for i in range(4)] + [r[:, 4 * H * d:4 * H * d + R]]
+    state = lambda n: torch.zeros(n, H, d, d, device=dev)
+    for B in (16, 64, 256):
+        st, ring = state(B + 1), torch.zeros(B + 1, 4, 3 * H * d, device=dev, dtype=bf)
+        mst = {"S": st, "n": torch.zeros(B + 1, H, d, device=dev), "m": torch.zeros(B + 1, H, device=dev)}
+        c, sl, z = cut(rows(B, 4 * H * d + R)), i32(list(range(B))), torch.randn(B, 2 * H, device=dev)
+        kl, out, cu = torch.full_like(sl, 100), torch.empty(B, H * d, device=dev, dtype=bf), i32(list(range(B + 1)))
+        pos = torch.full((B,), 99, device=dev)
+        nb = 2 * B * H * d * d * 4 + B * H * d * 10
+        report("delta_decode", f"B={B}", bench_queued(lambda: delta.decode(st, ring, sl, cu, kl, *c[:3], c[4], z, c[3], out)),
+               nb + B * 3 * H * d * 2 * 4)
+        report("mlstm_decode", f"B={B}", bench_queued(lambda: mem.decode(mst, sl, cu, kl, *c[:3], z[:, :H], z[:, H:], c[3], out)), nb)
+        report("linattn_decode", f"B={B}", bench_queued(lambda: lin.decode(st, sl, kl, pos, *c[:3], g=c[3], out=out)), nb)
+        q, k, v = (torch.randn(B, H, d, device=dev) for _ in range(3))
+        g, be, o, s64 = -torch.rand(B, H, device=dev), torch.rand(B, H, device=dev), torch.empty(B, H, d, device=dev), sl.long()
+        report("gdn_decode", f"B={B}", bench_queued(lambda: gdn.decode_step(st, s64, q, k, v, g, be, out=o)),
+               2 * B * H * d * d * 4 + B * H * d * 16)
+        del st, mst
+    for S, L in ((1, 2048), (1, 8192), (4, 2048)):
+        T = S * L
+        st, ring = state(S + 1), torch.zeros(S + 1, 4, 3 * H * d, device=dev, dtype=bf)
+        mst = {"S": st, "n": torch.zeros(S + 1, H, d, device=dev), "m": torch.zeros(S + 1, H, device=dev)}
+        c, sl, z = cut(rows(T, 4 * H * d + R)), i32(list(range(S))), torch.randn(T, 2 * H, device=dev)
+        cu, kl, pos = i32([i * L for i in range(S + 1)]), i32([L] * S), torch.arange(L, device=dev).repeat(S)
+        out = torch.empty(T, H * d, device=dev, dtype=bf)
+        fl, nb = 4.0 * T * H * d * d, T * H * d * 10 + S * H * d * d * 8
+        report("delta rule prompts", f"{S} x {L}", bench_queued(
+            lambda: delta.prefill(st, ring, sl, cu, kl, *c[:3], c[4], z, c[3], out), iters=5), nb, 2 * fl)
+        report("mlstm prompts", f"{S} x {L}", bench_queued(
+            lambda: mem.prefill(mst, sl, cu, kl, *c[:3], z[:, :H], z[:, H:], c[3], out), iters=5), nb, fl)
+        report("linattn prompts", f"{S} x {L}", bench_queued(
+            lambda: lin.prefill(st, sl, cu, kl, pos, *c[:3], g=c[3], out=out, max_q_len=L), iters=5), nb, fl)
+        q, k, v = (torch.randn(L, H, d, device=dev) for _ in range(3))
+        g, be, o = -torch.rand(L, H, device=dev), torch.rand(L, H, device=dev), torch.empty(L, H, d, device=dev)
+        report("gdn_prefill", f"{S} x {L}", bench_queued(
+            lambda: [gdn.prefill(st, s, True, q, k, v, g, be, out=o) for s in range(S)], iters=3), T * H * d * 16, 2 * fl)
+    nq, nkv = 32, 8
+    for S, L, win in ((4, 2048, 0), (4, 2048, 1024), (1, 8192, 0), (1, 8192, 1024)):
+        T = S * L
+        kc = rows(T // 16 * nkv * 16, d).view(T // 16, nkv, 16, d)
+        bt = torch.arange(T // 16, device=dev, dtype=torch.int32).view(S, L // 16)
+        cu, kl, q = i32([i * L for i in range(S + 1)]), i32([L] * S), rows(T, nq * d).view(T, nq, d)
+        pairs = sum(min(i + 1, win or L) for i in range(L)) * S
+        report("attention prompts", f"{S} x {L} window {win}", bench_queued(lambda: ops.paged_prefill_attention(
+            q, kc, kc, bt, cu, kl, L, d ** -0.5, window=win), iters=5), T * d * 2 * (2 * nq + 2 * nkv), 4.0 * pairs * nq * d)
+    for B, ctx, win in ((64, 4096, 0), (64, 4096, 1024), (256, 1024, 0), (256, 4096, 1024)):
+        kc = rows(B * ctx // 16 * nkv * 16, d).view(B * ctx // 16, nkv, 16, d)
+        bt = torch.arange(B * ctx // 16, device=dev, dtype=torch.int32).view(B, ctx // 16)
+        kl, q = i32([ctx] * B), rows(B, nq * d).view(B, nq, d)
+        splits = min(ops.decode_splits(B, nkv, nq // nkv), max(1, win // 256)) if win else None
+        report("attention decode", f"B={B} ctx {ctx} window {win}", bench_queued(lambda: ops.paged_decode_attention(
+            q, kc, kc, bt, kl, d ** -0.5, window=win, splits=splits)), 4.0 * B * min(ctx, win or ctx) * nkv * d)
+        del kc
+    for T in (64, 8192):
+        x, y, y2, w = torch.randn(T, W, device=dev), rows(T, W), rows(T, W), torch.ones(W, device=dev, dtype=bf)
+        report("residual_update, two branches", f"T={T}", bench_queued(
+            lambda: residual_update(x, y, y2=y2, w_out=w, w_out_offset=1.0)), T * W * 14)
+        res = rows(T, W)
+        report("rmsnorm (bf16 residual)", f"T={T}", bench_queued(lambda: ops.rmsnorm(y, w, 1e-6, residual=res)), T * W * 8)
+        o, out, g, div = torch.randn(T, H, d, device=dev), torch.empty(T, H * d, device=dev, dtype=bf), rows(T, H * d), torch.ones(T, H, device=dev)
+        wn = torch.ones(d, device=dev, dtype=bf)
+        report("head_norm_gate", f"T={T}", bench_queued(lambda: head_norm_gate(o, out, div=div, g=g, w=wn, act="sigmoid")), T * H * d * 8)
+        a = rows(T, H * d).view(T, H, d)
+        report("head_gate", f"T={T}", bench_queued(lambda: head_gate(a, g, d)), T * H * d * 6)
+        report("gate by tensor ops (Qwen3-Next)", f"T={T}", bench_queued(
+            lambda: a.view(T, H * d) * torch.sigmoid(g.float()).to(bf)), T * H * d * 6)
+        for N in (32, 64, 128):
+            xb, wr = rows(T, W), rows(N, W)
+            nb, fl = 2.0 * (T * W + N * W) + 4 * T * N, 2.0 * T * W * N
+            report("fp32 projection", f"T={T} N={N}", bench_queued(lambda: ops.linear_f32(xb, wr)), nb, fl)
+            report("router GEMM (bf16 result)", f"T={T} N={N}", bench_queued(lambda: ops.linear(xb, wr)), nb, fl)
+        qkv, pos = rows(T, (nq + 2 * nkv) * d), torch.arange(T, device=dev) % 8192
+        cs = torch.randn(8192, d, device=dev)
+        kc = torch.zeros(T // 16 + 2, nkv, 16, d, device=dev, dtype=bf)
+        vc, sl = torch.zeros_like(kc), torch.arange(16, 16 + T, dtype=torch.int32, device=dev)
+        q, k, v = qkv[:, :nq * d], qkv[:, nq * d:(nq + nkv) * d], qkv[:, (nq + nkv) * d:]
+        nb = T * d * 4 * (nq + 2 * nkv)
+        report("rotation + cache write", f"T={T}", bench_queued(lambda: ops.rope_norm_kv_write(
+            q, k, v, nq, nkv, d, pos, cs, d, sl, kc, vc, unit_norm=False)), nb)
+        report("rope_kv", f"T={T}", bench_queued(lambda: ops.rope_kv_write(
+            qkv, nq, nkv, d, pos, cs, d, slots=sl, k_cache=kc, v_cache=vc, q_norm_w=wn, k_norm_w=wn)), nb)
+        E, K, I = 32, 4, W // 2
+        w1, w2, xb = rows(E * 2 * I, W).view(E, 2 * I, W), rows(E * W, I).view(E, W, I), rows(T, W)
+        lg, bias = torch.randn(T, E, device=dev), torch.randn(E, device=dev) * 0.1
+        ws = moe.shared_workspace(T, K, E, E, W, I, torch.device(dev), bf, W)
+        nb = 2.0 * (min(E, T * K) * 3 * I * W + 2 * T * W)
+        report("experts (groups by best score)", f"T={T} E={E} top{K}", bench_queued(lambda: moe.fused_moe(
+            xb, lg, w1, w2, K, bias=bias, n_group=8, topk_group=4, ws=ws, interleaved=True, group_score="max")), nb, 6.0 * T * K * W * I)
+        report("experts (plain softmax)", f"T={T} E={E} top{K}", bench_queued(lambda: moe.fused_moe(
+            xb, lg, w1, w2, K, ws=ws, interleaved=True)), nb, 6.0 * T * K * W * I)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--what", default="gemm,decode,prefill,small")
@@ -392,7 +511,7 @@ def main():
     results = []
     for w in a.what.split(","):
         {"gemm": gemm_rows, "decode": decode_rows, "prefill": prefill_rows, "small": small_rows, "gdn": gdn_rows, "mla": mla_rows,
-         "fp8": fp8_rows, "moe": moe_rows, "hybrid": hybrid_rows}[w](results, hbm, tf, tag)
+         "fp8": fp8_rows, "moe": moe_rows, "hybrid": hybrid_rows, "recurrent": recurrent_rows}[w](results, hbm, tf, tag)
     if a.json:
         with open(a.json, "w") as f:
             json.dump(results, f, indent=1)

@@ -46,7 +46,7 @@ NVCC_FLAGS = [
 ]
 # Sources built without --use_fast_math: their exponentials feed recurrences (errors of a decay multiply up over a
 # sequence) or serve the fp32 execution type.
-PRECISE_SOURCES = {"linear_attn", "residual", "rope_norm_kv", "attn_generic", "delta_rule", "mlstm", "head_norm", "proj_f32"}
+PRECISE_SOURCES = {"linear_attn", "residual", "rope_norm_kv", "attn_generic", "delta_rule", "mlstm", "head_norm", "proj_f32", "moe"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread",
              "-I", str(CSRC / "runtime"), "-I", str(CSRC / "frontend"), "-I", str(CSRC / "server"),
              "-Wall", "-Wno-sign-compare", "-I", str(CSRC), "-I", "/usr/local/cuda/include"]

@@ -8,11 +8,11 @@
 // weighted, and multiplied by the sigmoid of a gate.  The sibling of gdn.cu, whose decay is one number per head and
 // whose inputs are prepared by tensor operations.
 //
-//   delta_decode_kernel        one token per sequence, everything above from the projection rows to the finished row;
-//                              the state crosses HBM once in each direction
+//   delta_decode_kernel        one token per sequence, from the projection rows and the decays to the finished row; the
+//                              state crosses HBM once in each direction
 //   conv_heads_kernel          prompts: convolution, silu, unit norm of q and k -> fp32
 //   conv_ring_kernel           prompts: the last inputs of every sequence -> its ring
-//   channel_decay_kernel       prompts: the decays, W_2 r on the tensor cores
+//   channel_decay_kernel       the decays, W_2 r on the tensor cores
 //   delta_prefill_kernel       prompts: the recurrence, token by token with the state in registers (recurrence.cuh)
 // (head_norm.cu finishes the prompts' rows.)
 //
@@ -65,8 +65,7 @@ __global__ void __launch_bounds__(256) delta_decode_kernel(DeltaParams<T> p) {
   float* ks = qs + dkp;
   float* gs = ks + dkp;
   float* vs = gs + dkp;                    // [dvp]
-  float* rs = vs + dvp;                    // [rank rounded up to 4]
-  float* red = rs + ((p.rank + 3) & ~3);   // [RG][dvp]
+  float* red = vs + dvp;                   // [RG][dvp]
   __shared__ float red32[2][32];
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int CG = dvp >> 2, RG = 256 / CG;
@@ -109,7 +108,7 @@ __global__ void __launch_bounds__(256) delta_decode_kernel(DeltaParams<T> p) {
     if (taps > 1 && (keeps_qk || i >= 2 * dk)) ring_now[c] = *x;
   }
   for (int i = dv + tid; i < dvp; i += 256) vs[i] = 0.f;
-  for (int i = tid; i < p.rank; i += 256) rs[i] = to_f32(p.r[b * p.ld + i]);
+  for (int i = tid; i < dk; i += 256) gs[i] = p.gn[((int64_t)b * p.H + h) * dkp + i];
   sq = warp_sum(sq);
   sk = warp_sum(sk);
   if (lane == 0) { red32[0][warp] = sq; red32[1][warp] = sk; }
@@ -118,24 +117,9 @@ __global__ void __launch_bounds__(256) delta_decode_kernel(DeltaParams<T> p) {
 #pragma unroll
   for (int w = 0; w < 8; ++w) { sq += red32[0][w]; sk += red32[1][w]; }
   const float iq = p.q_scale / sqrtf(sq + kUnitEps), ik = 1.f / sqrtf(sk + kUnitEps);
-  const float A = expf(to_f32(p.a_log[h]));
   for (int i = tid; i < dk; i += 256) {
     qs[i] *= iq;
     ks[i] *= ik;
-    const int64_t c = (int64_t)h * dk + i;
-    float z = to_f32(p.dt_bias[c]);
-    const T* w = p.a2 + c * p.rank;
-    if (p.rank % 8 == 0) {
-      for (int j = 0; j < p.rank; j += 8) {
-        float x[8];
-        load_f32<8>(w + j, x);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) z += rs[j + e] * x[e];
-      }
-    } else {
-      for (int j = 0; j < p.rank; ++j) z += rs[j] * to_f32(w[j]);
-    }
-    gs[i] = expf(-A * softplus_exact(z));
   }
   const float beta = sigmoid_exact(p.zb[b * p.zb_ld + h]);
   __syncthreads();
@@ -259,16 +243,26 @@ __global__ void __launch_bounds__(128) channel_decay_tile_kernel(DeltaParams<bf1
   const int r0 = p.row0 + blockIdx.x * 64, c0 = blockIdx.y * 64, tid = threadIdx.x, nc = p.H * p.dk;
   const int warp = tid >> 5, lane = tid & 31;
   const bf16 zero = __float2bfloat16(0.f);
-  for (int i = tid; i < 64 * RP; i += 128) {
-    const int y = i / RP, x = i - y * RP;
-    ws[y * st + x] = (c0 + y < nc && x < p.rank) ? p.a2[(int64_t)(c0 + y) * p.rank + x] : zero;
-  }
+  const bool v8 = p.rank % 8 == 0 && p.ld % 8 == 0 && (((uintptr_t)p.a2 | (uintptr_t)p.r) & 15) == 0;
+  const uint4 zero8 = make_uint4(0, 0, 0, 0);
+  const auto copy = [&](bf16* dst, const bf16* src, int64_t ld, int n) {     // n rows of `rank` elements, zeros behind
+    if (v8) {
+      const int per = RP >> 3;
+      for (int i = tid; i < 64 * per; i += 128) {
+        const int y = i / per, x = (i - y * per) * 8;
+        *reinterpret_cast<uint4*>(dst + y * st + x) = (y < n && x < p.rank) ? *reinterpret_cast<const uint4*>(src + y * ld + x) : zero8;
+      }
+    } else {
+      for (int i = tid; i < 64 * RP; i += 128) {
+        const int y = i / RP, x = i - y * RP;
+        dst[y * st + x] = (y < n && x < p.rank) ? src[y * ld + x] : zero;
+      }
+    }
+  };
+  copy(ws, p.a2 + (int64_t)c0 * p.rank, p.rank, nc - c0);
   pdl_wait();
   pdl_launch_dependents();
-  for (int i = tid; i < 64 * RP; i += 128) {
-    const int y = i / RP, x = i - y * RP;
-    rs[y * st + x] = (r0 + y < p.rows && x < p.rank) ? p.r[(int64_t)(r0 + y) * p.ld + x] : zero;
-  }
+  copy(rs, p.r + (int64_t)r0 * p.ld, p.ld, p.rows - r0);
   __syncthreads();
   float z[8][4];
 #pragma unroll
@@ -425,6 +419,23 @@ __global__ void __launch_bounds__(256) delta_prefill_kernel(DeltaScan p) {
   if (col < p.dvp) st.store(S, p.dk, p.dvp, rgrp);
 }
 
+template <typename T>
+static int launch_channel_decay(const DeltaParams<T>& p, cudaStream_t s) {
+  const int n = p.rows - p.row0;
+  if constexpr (sizeof(T) == 2) {
+    if (p.rank <= 256) {
+      const size_t smem = (size_t)2 * 64 * (((p.rank + 15) & ~15) + 8) * 2;
+      const cudaError_t e = cudaFuncSetAttribute(channel_decay_tile_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) return (int)e;
+      launch_pdl(channel_decay_tile_kernel, dim3((n + 63) / 64, (p.H * p.dk + 63) / 64), dim3(128), smem, s, p);
+      return XLLM_LAUNCH_CHECK();
+    }
+  }
+  const int64_t blocks = ((int64_t)n * p.H * p.dk + 255) / 256;
+  launch_pdl(channel_decay_kernel<T>, dim3((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16)), dim3(256), 0, s, p);
+  return XLLM_LAUNCH_CHECK();
+}
+
 template <int J>
 static int launch_delta_prefill(const DeltaScan& p, int n_seqs, cudaStream_t s) {
   const int warps = min(8, (p.dvp + kRecCols - 1) / kRecCols), cols = warps * kRecCols;
@@ -440,9 +451,9 @@ static int launch_delta_prefill(const DeltaScan& p, int n_seqs, cudaStream_t s) 
 // dtype: 0 bf16, 1 fp32 (projection rows, weights, ring, finished rows).
 //   state [slots, H, dk, dvp] fp32, dvp = dv rounded up to 4;  ring [slots, taps, 2 G dk + H dv]
 //   q, k, v, r: column blocks of rows with stride ld;  zb fp32 [rows, zb_ld]
+// gn [rows, H, dkp] fp32 is scratch (dkp = dk rounded up to 4, zeros behind dk).
 // mode 0: one token per sequence (sequence s is row s): gate, norm_w, out are used; dk <= 256, dv <= 128
-// mode 1: rows [row0, rows) by cu_q: qn, kn [rows, G, dkp], vn [rows, H, dvp], gn [rows, H, dkp] (dkp = dk rounded up to
-//         4) are scratch, the raw fp32 outputs go to o [rows, H, dv];  dk <= 512
+// mode 1: rows [row0, rows) by cu_q: qn, kn [rows, G, dkp], vn [rows, H, dvp] are scratch, the raw fp32 outputs go to o [rows, H, dv];  dk <= 512
 XLLM_API int xllm_delta_rule(void* state, void* ring, const void* slots, const void* cu_q, const void* kv_lens, const void* q,
                              const void* k, const void* v, const void* r, int64_t ld, const void* zb, int64_t zb_ld,
                              const void* conv_w, const void* a2, const void* dt_bias, const void* a_log, const void* gate,
@@ -466,9 +477,10 @@ XLLM_API int xllm_delta_rule(void* state, void* ring, const void* slots, const v
     p.out_ld = out_ld; p.qn = (float*)qn; p.kn = (float*)kn; p.vn = (float*)vn; p.gn = (float*)gn; p.o = (float*)o;
     p.n_seqs = n_seqs; p.rows = rows; p.row0 = row0; p.H = H; p.G = G; p.dk = dk; p.dv = dv; p.dkp = (dk + 3) & ~3;
     p.dvp = (dv + 3) & ~3; p.taps = taps; p.rank = rank; p.q_scale = q_scale; p.eps = eps;
+    if ((rc = launch_channel_decay(p, s)) != 0) return;
     if (mode == 0) {
       const int RG = 256 / (p.dvp >> 2), nr = (dk + RG - 1) / RG;
-      const size_t smem = (size_t)(3 * p.dkp + p.dvp + ((rank + 3) & ~3) + RG * p.dvp) * 4;
+      const size_t smem = (size_t)(3 * p.dkp + p.dvp + RG * p.dvp) * 4;
       const dim3 grid(H, n_seqs), block(256);
       if (nr <= 4) launch_pdl(delta_decode_kernel<T, 4>, grid, block, smem, s, p);
       else if (nr <= 8) launch_pdl(delta_decode_kernel<T, 8>, grid, block, smem, s, p);
@@ -489,20 +501,6 @@ XLLM_API int xllm_delta_rule(void* state, void* ring, const void* slots, const v
       launch_pdl(conv_ring_kernel<T>, dim3((unsigned)((p.channels() + 255) / 256), n_seqs), dim3(256), 0, s, p);
       if ((rc = XLLM_LAUNCH_CHECK()) != 0) return;
     }
-    bool tiled = false;
-    if constexpr (sizeof(T) == 2) {
-      if (rank <= 256) {
-        const size_t smem = (size_t)2 * 64 * (((rank + 15) & ~15) + 8) * 2;
-        cudaFuncSetAttribute(channel_decay_tile_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        launch_pdl(channel_decay_tile_kernel, dim3((rows - row0 + 63) / 64, (H * dk + 63) / 64), dim3(128), smem, s, p);
-        tiled = true;
-      }
-    }
-    if (!tiled) {
-      const int64_t blocks = ((int64_t)(rows - row0) * H * dk + 255) / 256;
-      launch_pdl(channel_decay_kernel<T>, dim3((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16)), dim3(256), 0, s, p);
-    }
-    if ((rc = XLLM_LAUNCH_CHECK()) != 0) return;
     DeltaScan d{p.state, p.slots, p.cu_q, p.kv_lens, p.qn, p.kn, p.vn, p.gn, p.zb, zb_ld, p.o, H, G, dk, dv, p.dkp, p.dvp};
     if (dk <= 32) rc = launch_delta_prefill<1>(d, n_seqs, s);
     else if (dk <= 64) rc = launch_delta_prefill<2>(d, n_seqs, s);

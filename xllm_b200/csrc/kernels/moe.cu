@@ -61,7 +61,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(RouteParams p) {
     float sum = 0.f;
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
-      score[i] = (i < per && lane + i * 32 < p.E) ? __expf(score[i] - mx) : 0.f;
+      score[i] = (i < per && lane + i * 32 < p.E) ? expf(score[i] - mx) : 0.f;
       sum += score[i];
     }
     sum = warp_sum(sum);
@@ -70,7 +70,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(RouteParams p) {
     for (int i = 0; i < PER; ++i) score[i] *= inv;
   } else {  // sigmoid
 #pragma unroll
-    for (int i = 0; i < PER; ++i) score[i] = (i < per && lane + i * 32 < p.E) ? 1.f / (1.f + __expf(-score[i])) : 0.f;
+    for (int i = 0; i < PER; ++i) score[i] = (i < per && lane + i * 32 < p.E) ? 1.f / (1.f + expf(-score[i])) : 0.f;
   }
 #pragma unroll
   for (int i = 0; i < PER; ++i) {

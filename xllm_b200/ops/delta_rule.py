@@ -51,14 +51,18 @@ class ChannelDelta:
         assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (H, dk, round4(dv))
         assert ring.dtype == q.dtype and ring.is_contiguous() and ring.shape[1:] == (self.taps, self.channels)
         assert slots.dtype == torch.int32 and kv_lens.dtype == torch.int32 and zb.dtype == torch.float32 and zb.stride(1) == 1
-        qn, kn, vn, gn, o = scratch or (None,) * 5
+        qn, kn, vn, gn, o = scratch
         check(_lib.load().xllm_delta_rule(
             ptr(state), ptr(ring), ptr(slots), ptr(cu_q), ptr(kv_lens), ptr(q), ptr(k), ptr(v), ptr(r), ld, ptr(zb), zb.stride(0),
             ptr(self.conv_w), ptr(self.a2), ptr(self.dt_bias), ptr(self.a_log), ptr(gate), gate.stride(0), ptr(self.norm_w),
             ptr(out), out.stride(0), ptr(qn), ptr(kn), ptr(vn), ptr(gn), ptr(o), slots.shape[0], rows, row0, H, self.kv_heads,
             dk, dv, self.taps, self.a2.shape[1], self.q_scale, self.eps, _DT[q.dtype], mode, stream()), "delta_rule")
         from . import _count
-        _count(1 if mode == 0 else (4 if self.taps > 1 else 3))
+        _count(2 if mode == 0 else (4 if self.taps > 1 else 3))
+
+    def _decays(self, rows, device):
+        dkp = round4(self.dk)
+        return (torch.zeros if dkp != self.dk else torch.empty)((rows, self.heads, dkp), dtype=torch.float32, device=device)
 
     def decode(self, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out):
         """One token per sequence (sequence s is row s; cu_q [B + 1] counts up by one); `out` [B, heads * dv] is filled with
@@ -68,7 +72,8 @@ class ChannelDelta:
             return self.prefill(state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out, padded=True)
         if not q.is_cuda:
             return self._cpu(state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out)
-        self._launch(0, state, ring, slots, None, kv_lens, q, k, v, r, zb, gate, out, None, B, 0)
+        scratch = (None, None, None, self._decays(B, q.device), None)
+        self._launch(0, state, ring, slots, None, kv_lens, q, k, v, r, zb, gate, out, scratch, B, 0)
         return out
 
     def prefill(self, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out, row0=0, padded=False):
@@ -80,7 +85,7 @@ class ChannelDelta:
         f32 = dict(dtype=torch.float32, device=q.device)
         dkp, dvp = round4(self.dk), round4(self.dv)
         scratch = (torch.empty((T, G, dkp), **f32), torch.empty((T, G, dkp), **f32), torch.empty((T, H, dvp), **f32),
-                   (torch.zeros if dkp != self.dk else torch.empty)((T, H, dkp), **f32),
+                   self._decays(T, q.device),
                    (torch.zeros if padded else torch.empty)((T, H, self.dv), **f32))
         self._launch(1, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out, scratch, T, row0)
         head_norm_gate(scratch[4][row0:], out[row0:], g=gate[row0:], w=self.norm_w, act="sigmoid", eps=self.eps)
