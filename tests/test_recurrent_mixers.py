@@ -95,11 +95,11 @@ class DeltaCase(Case):
         self.state = torch.full((len(lens) + 2, H, dk, (dv + 3) // 4 * 4), 1e9, device=self.dev)
         self.ring = torch.full((len(lens) + 2, taps, C), 1e9, dtype=self.dt, device=self.dev)
 
-    def step(self, parts, decode=False):
+    def step(self, parts, decode=False, **kw):
         idx, (q, k, v, r, gate), slots, cu, lens = self.batch(parts)
         out = torch.empty(len(idx), self.op.heads * self.op.dv, dtype=self.dt, device=self.dev)
         run = self.op.decode if decode else self.op.prefill
-        return run(self.state, self.ring, slots, cu, lens, q, k, v, r, self.zb[idx], gate, out)
+        return run(self.state, self.ring, slots, cu, lens, q, k, v, r, self.zb[idx], gate, out, **kw)
 
 
 class MemoryCase(Case):
@@ -122,13 +122,13 @@ class MemoryCase(Case):
         full = lambda *s: torch.full((len(lens) + 2, *s), 1e9, device=self.dev)
         self.state = {"S": full(H, dk, (dv + 3) // 4 * 4), "n": full(H, dk), "m": full(H)}
 
-    def step(self, parts, decode=False):
+    def step(self, parts, decode=False, **kw):
         idx, (q, k, v, gate), slots, cu, lens = self.batch(parts)
         H = self.op.heads
         out = torch.empty(len(idx), H * self.op.dv, dtype=self.dt, device=self.dev)
         z = self.z[idx]
         run = self.op.decode if decode else self.op.prefill
-        return run(self.state, slots, cu, lens, q, k, v, z[:, :H], z[:, H:], gate, out)
+        return run(self.state, slots, cu, lens, q, k, v, z[:, :H], z[:, H:], gate, out, **kw)
 
 
 LENS = (49, 16, 1, 34)
@@ -197,6 +197,20 @@ def test_long_prompt(name, target):
     c.check(c.step(p), p, tol)
     p = [(0, 65, 330), (2, 100, 205)]
     c.check(c.step(p), p, tol)
+
+
+@pytest.mark.parametrize("target", TARGETS)
+@pytest.mark.parametrize("name", sorted(CASES))
+def test_token_by_token_form(name, target):
+    """The fp32 recurrence of every type, before and behind the form in chunks."""
+    c = CASES[name](target)
+    tol = (2e-5 if target[1] == torch.float32 else 4e-3) * (6 if name == "memory_forgets" else 1)
+    p = [(0, 0, 23), (1, 0, 16), (3, 0, 2)]
+    c.check(c.step(p, token_by_token=True), p, tol)
+    p = [(0, 23, 40), (3, 2, 20)]
+    c.check(c.step(p), p, tol * 2)
+    p = [(0, 40, 49), (3, 20, 34)]
+    c.check(c.step(p, token_by_token=True), p, tol * 2)
 
 
 @pytest.mark.parametrize("target", TARGETS)

@@ -41,6 +41,16 @@ __device__ __forceinline__ uint32_t pack_bf162(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// Two fp32 values as two bf16 pairs whose sum keeps about 16 bits of their significands.
+__device__ __forceinline__ void split_pack(float a, float b, uint32_t& hi, uint32_t& lo) {
+  const bf162 h = __floats2bfloat162_rn(a, b);
+  const float2 f = __bfloat1622float2(h);
+  const bf162 l = __floats2bfloat162_rn(a - f.x, b - f.y);
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+__device__ __forceinline__ float2 unpack2(uint32_t u) { return __bfloat1622float2(*reinterpret_cast<const bf162*>(&u)); }
+
 // Byte offset of 16-byte chunk `c` of row `r` in a tile whose rows hold CH chunks; the XOR
 // swizzle makes 8 consecutive rows of one chunk column hit 8 different bank groups.
 template <int CH>

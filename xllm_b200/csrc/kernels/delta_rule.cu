@@ -13,7 +13,10 @@
 //   conv_heads_kernel          prompts: convolution, silu, unit norm of q and k -> fp32
 //   conv_ring_kernel           prompts: the last inputs of every sequence -> its ring
 //   channel_decay_kernel       the decays, W_2 r on the tensor cores
-//   delta_prefill_kernel       prompts: the recurrence, token by token with the state in registers (recurrence.cuh)
+//   delta_chunk_prep_kernel,   prompts, bf16: sixteen tokens at a time on the tensor cores (below)
+//   delta_chunk_kernel
+//   delta_prefill_kernel       prompts of any type and size: token by token in fp32 with the state in registers
+//                              (recurrence.cuh)
 // (head_norm.cu finishes the prompts' rows.)
 //
 // A sequence whose rows in the batch are its first tokens (kv_len == number of rows) starts from S = 0 whatever its
@@ -48,6 +51,7 @@ struct DeltaParams {
   float* o;                  // [rows, H, dv]
   int n_seqs, rows, row0, H, G, dk, dv, dkp, dvp, taps, rank;
   float q_scale, eps;
+  int log_decay;             // gn receives log2 of the decays (chunked prompts)
   __host__ __device__ int64_t channels() const { return (int64_t)2 * G * dk + (int64_t)H * dv; }
 };
 
@@ -293,7 +297,10 @@ __global__ void __launch_bounds__(128) channel_decay_tile_kernel(DeltaParams<bf1
 #pragma unroll
       for (int u = 0; u < 2; ++u) {
         const int row = r0 + ra + 8 * u;
-        if (row < p.rows) p.gn[((int64_t)row * p.H + h) * p.dkp + ch] = expf(-A * softplus_exact(z[n][2 * u + e] + bias));
+        if (row < p.rows) {
+          const float g = -A * softplus_exact(z[n][2 * u + e] + bias);
+          p.gn[((int64_t)row * p.H + h) * p.dkp + ch] = p.log_decay ? g * 1.44269504088896341f : expf(g);
+        }
       }
     }
   }
@@ -312,7 +319,8 @@ __global__ void __launch_bounds__(256) channel_decay_kernel(DeltaParams<T> p) {
     const T* r = p.r + (int64_t)row * p.ld;
     const T* w = p.a2 + (int64_t)c * p.rank;
     for (int j = 0; j < p.rank; ++j) z += to_f32(r[j]) * to_f32(w[j]);
-    p.gn[((int64_t)row * p.H + h) * p.dkp + c - h * p.dk] = expf(-expf(to_f32(p.a_log[h])) * softplus_exact(z));
+    const float g = -expf(to_f32(p.a_log[h])) * softplus_exact(z);
+    p.gn[((int64_t)row * p.H + h) * p.dkp + c - h * p.dk] = p.log_decay ? g * 1.44269504088896341f : expf(g);
   }
 }
 
@@ -419,6 +427,394 @@ __global__ void __launch_bounds__(256) delta_prefill_kernel(DeltaScan p) {
   if (col < p.dvp) st.store(S, p.dk, p.dvp, rgrp);
 }
 
+// ------------------------------------------------------------------------------------------------ prompts, chunks of 16
+// With L_t the log2 decay from a chunk's start through token t (per key channel), S_0 the state before the chunk and
+//
+//   A_ts = sum_c k_t k_s 2^(L_t - L_s)  (s < t),     P_ts = sum_c q_t k_s 2^(L_t - L_s)  (s <= t),
+//   M = (I + diag(beta) A)^-1 diag(beta)
+//
+// the chunk is   U = M (V - (k 2^L) S_0),   O = (q 2^L) S_0 + P U,   S <- 2^(L_end) S_0 + (k 2^(L_end - L))^T U.
+//
+// Everything but S_0 and V is made by delta_chunk_prep_kernel, all chunks side by side, and stored as the operands the
+// tensor cores read: k 2^L, q 2^L, k 2^(L_end - L), M and P, each fp32 value as two bf16 terms.  All their decays are at
+// most 1.  A and P factor their decays against the chunk's middle token; channels whose decays span more than fp32 holds
+// take their share pair by pair instead.  delta_chunk_kernel walks the chunks of a sequence: a warp owns 16 state columns
+// for all of dk as fp32 accumulators of S^T, which are the A operand of S^T (k 2^L)^T and S^T (q 2^L)^T without leaving
+// the registers, as U^T is of the products after it.
+constexpr int kDC = 16;
+constexpr int kDWarps = 4;                   // warps of 16 columns
+constexpr int kDStages = 3;
+constexpr float kDLogRange = 86.f;
+
+template <int DK>
+struct ChunkBlob {                           // bytes of one (chunk, head), in this order
+  static constexpr int tile = kDC * DK * 2;  // [16][DK] bf16, 16-byte pieces swizzled
+  static constexpr int kt = 0, qt = 2 * tile, kc = 4 * tile;      // first and second term behind one another
+  static constexpr int m = 6 * tile, p = m + 2 * kDC * kDC * 2;   // [16][16] bf16, two terms
+  static constexpr int end = p + 2 * kDC * kDC * 2;               // [DK] fp32: 2^(L_end)
+  static constexpr int bytes = end + DK * 4;
+};
+
+// chunk i of sequence b: unique because a sequence of n rows has at most n / 16 + 1 chunks
+__device__ __forceinline__ int64_t chunk_slot(int row0, int b, int i) { return (int64_t)row0 / kDC + b + i; }
+
+struct DeltaChunk {
+  DeltaScan s;
+  uint8_t* blobs;                            // [chunk slots, H, ChunkBlob]
+};
+
+// grid (chunks of a sequence, heads, sequences), 256 threads; a warp owns every eighth group of 16 channels.
+template <int DK>
+__global__ void __launch_bounds__(256) delta_chunk_prep_kernel(DeltaChunk d) {
+  using B = ChunkBlob<DK>;
+  constexpr int CH = DK / 8;
+  const DeltaScan& p = d.s;
+  __shared__ float part[8][2][kDC][kDC + 1];
+  __shared__ float am[kDC][kDC + 1];
+  __shared__ float betas[kDC];
+  const int h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row_first = p.cu_q[b], n_seq = p.cu_q[b + 1] - row_first;
+  const int i0 = blockIdx.x * kDC;
+  if (i0 >= n_seq || p.slots[b] < 0) return;
+  const int n = min(kDC, n_seq - i0), row0 = row_first + i0;
+  uint8_t* blob = d.blobs + (chunk_slot(row_first, b, blockIdx.x) * p.H + h) * B::bytes;
+  if (tid < kDC) betas[tid] = tid < n ? sigmoid_exact(p.zb[(int64_t)(row0 + tid) * p.zb_ld + h]) : 0.f;
+  const int g = h / (p.H / p.G), ta = lane >> 2, kc = (lane & 3) * 2;
+  float ca[2][4], cp[2][4];                  // A and P: rows ta (+ 8), columns 8 j + kc (+ 1)
+#pragma unroll
+  for (int j = 0; j < 2; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) ca[j][e] = cp[j][e] = 0.f;
+  for (int c0 = warp * 16; c0 < DK; c0 += 128) {
+    // elements [u][v]: token ta + 8 u, channels c0 + 8 v + kc, + 1
+    float2 q[2][2], k[2][2], L[2][2];
+#pragma unroll
+    for (int u = 0; u < 2; ++u)
+#pragma unroll
+      for (int v = 0; v < 2; ++v) {
+        const int c = c0 + 8 * v + kc;
+        const int64_t row = row0 + ta + 8 * u;
+        q[u][v] = k[u][v] = L[u][v] = make_float2(0.f, 0.f);
+        if (ta + 8 * u < n && c < p.dkp) {   // dkp is a multiple of 4, zeros behind dk
+          const int64_t at = (row * p.G + g) * p.dkp + c;
+          q[u][v] = *reinterpret_cast<const float2*>(p.qn + at);
+          k[u][v] = *reinterpret_cast<const float2*>(p.kn + at);
+          L[u][v] = *reinterpret_cast<const float2*>(p.gn + (row * p.H + h) * p.dkp + c);
+        }
+      }
+    float2 ref[2], end[2];
+    bool unsafe = false;
+#pragma unroll
+    for (int v = 0; v < 2; ++v) {
+#pragma unroll
+      for (int s = 4; s < 32; s <<= 1) {
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          const float x = __shfl_up_sync(0xffffffffu, L[u][v].x, s), y = __shfl_up_sync(0xffffffffu, L[u][v].y, s);
+          if (lane >= s) { L[u][v].x += x; L[u][v].y += y; }
+        }
+      }
+      ref[v].x = __shfl_sync(0xffffffffu, L[0][v].x, 28 + (lane & 3));     // token 7
+      ref[v].y = __shfl_sync(0xffffffffu, L[0][v].y, 28 + (lane & 3));
+      L[1][v].x += ref[v].x;
+      L[1][v].y += ref[v].y;
+      end[v].x = __shfl_sync(0xffffffffu, L[1][v].x, 28 + (lane & 3));     // rows behind the last one add nothing
+      end[v].y = __shfl_sync(0xffffffffu, L[1][v].y, 28 + (lane & 3));
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+        unsafe |= fabsf(L[u][v].x - ref[v].x) > kDLogRange || fabsf(L[u][v].y - ref[v].y) > kDLogRange;
+    }
+    if (lane < 4) {
+#pragma unroll
+      for (int v = 0; v < 2; ++v)
+        *reinterpret_cast<float2*>(blob + B::end + (c0 + 8 * v + kc) * 4) = make_float2(exp2f(end[v].x), exp2f(end[v].y));
+    }
+    uint32_t hi, lo;
+#pragma unroll
+    for (int u = 0; u < 2; ++u)
+#pragma unroll
+      for (int v = 0; v < 2; ++v) {
+        const uint32_t at = swz<CH>(ta + 8 * u, (c0 >> 3) + v) + kc * 2;
+        const auto put = [&](int where, float x, float y) {
+          split_pack(x, y, hi, lo);
+          *reinterpret_cast<uint32_t*>(blob + where + at) = hi;
+          *reinterpret_cast<uint32_t*>(blob + where + B::tile + at) = lo;
+        };
+        const float ex = exp2f(L[u][v].x), ey = exp2f(L[u][v].y);
+        put(B::kt, k[u][v].x * ex, k[u][v].y * ey);
+        put(B::qt, q[u][v].x * ex, q[u][v].y * ey);
+        put(B::kc, k[u][v].x * exp2f(end[v].x - L[u][v].x), k[u][v].y * exp2f(end[v].y - L[u][v].y));
+      }
+    if (!__any_sync(0xffffffffu, unsafe)) {
+      uint32_t kh[4], kl[4], qh[4], ql[4], sh[4], sl[4];     // [2 v + u]: A fragments; s: B fragments [2 v + token half]
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int v = 0; v < 2; ++v) {
+          const float dx = L[u][v].x - ref[v].x, dy = L[u][v].y - ref[v].y;
+          const float ex = exp2f(dx), ey = exp2f(dy);
+          split_pack(k[u][v].x * ex, k[u][v].y * ey, kh[2 * v + u], kl[2 * v + u]);
+          split_pack(q[u][v].x * ex, q[u][v].y * ey, qh[2 * v + u], ql[2 * v + u]);
+          split_pack(k[u][v].x * exp2f(-dx), k[u][v].y * exp2f(-dy), sh[2 * v + u], sl[2 * v + u]);
+        }
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        mma_bf16_16816(ca[j], kh, sh[j], sh[2 + j]);
+        mma_bf16_16816(cp[j], qh, sh[j], sh[2 + j]);
+        mma_bf16_16816(ca[j], kl, sh[j], sh[2 + j]);
+        mma_bf16_16816(cp[j], ql, sh[j], sh[2 + j]);
+        mma_bf16_16816(ca[j], kh, sl[j], sl[2 + j]);
+        mma_bf16_16816(cp[j], qh, sl[j], sl[2 + j]);
+      }
+    } else {
+      // token pairs one by one: this lane's entries (ta + 8 u, 8 j + kc + e), channels walked through shuffles
+#pragma unroll 1
+      for (int c = 0; c < 16; ++c) {
+        const int v = c >> 3, src = (c & 7) >> 1, odd = c & 1;             // channel c lives in lanes 4 t + src
+        float kt[2], qt[2], lt[2];
+        const auto pick = [&](const float2& x) { return odd ? x.y : x.x; };
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          kt[u] = v ? pick(k[u][1]) : pick(k[u][0]);
+          qt[u] = v ? pick(q[u][1]) : pick(q[u][0]);
+          lt[u] = v ? pick(L[u][1]) : pick(L[u][0]);
+        }
+        float rk[2], rq[2], rl[2];           // of this lane's rows
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          rk[u] = __shfl_sync(0xffffffffu, kt[u], (lane & ~3) + src);
+          rq[u] = __shfl_sync(0xffffffffu, qt[u], (lane & ~3) + src);
+          rl[u] = __shfl_sync(0xffffffffu, lt[u], (lane & ~3) + src);
+        }
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const float sk = __shfl_sync(0xffffffffu, kt[j], 4 * (kc + e) + src);
+            const float sl = __shfl_sync(0xffffffffu, lt[j], 4 * (kc + e) + src);
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+              const float x = sk * exp2f(fminf(rl[u] - sl, 0.f));          // pairs with s > t are dropped later
+              ca[j][2 * u + e] += rk[u] * x;
+              cp[j][2 * u + e] += rq[u] * x;
+            }
+          }
+      }
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < 2; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      part[warp][0][ta + (e >> 1) * 8][8 * j + kc + (e & 1)] = ca[j][e];
+      part[warp][1][ta + (e >> 1) * 8][8 * j + kc + (e & 1)] = cp[j][e];
+    }
+  __syncthreads();
+  {
+    const int t = tid >> 4, s = tid & 15;
+    float a = 0.f, q = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) {
+      a += part[w][0][t][s];
+      q += part[w][1][t][s];
+    }
+    am[t][s] = s < t ? a * betas[t] : 0.f;
+    if (s > t) q = 0.f;
+    const bf16 hi = __float2bfloat16(q);
+    bf16* pm = reinterpret_cast<bf16*>(blob + B::p);
+    pm[tid] = hi;
+    pm[kDC * kDC + tid] = __float2bfloat16(q - __bfloat162float(hi));
+  }
+  __syncthreads();
+  if (tid < kDC) {                           // column tid of the inverse by forward substitution
+    float x[kDC];
+    bf16* mm = reinterpret_cast<bf16*>(blob + B::m);
+    const float bt = betas[tid];
+#pragma unroll
+    for (int t = 0; t < kDC; ++t) {
+      float y = t == tid ? 1.f : 0.f;
+#pragma unroll
+      for (int s = 0; s < t; ++s) y -= am[t][s] * x[s];
+      x[t] = y;
+      const bf16 hi = __float2bfloat16(y * bt);
+      mm[t * kDC + tid] = hi;
+      mm[kDC * kDC + t * kDC + tid] = __float2bfloat16(y * bt - __bfloat162float(hi));
+    }
+  }
+}
+
+// grid (slices of 64 columns, heads, sequences)
+template <int DK>
+__global__ void __launch_bounds__(32 * kDWarps, DK > 128 ? 1 : 2) delta_chunk_kernel(DeltaChunk d) {
+  using B = ChunkBlob<DK>;
+  constexpr int CH = DK / 8, COLS = kDWarps * 16, VLD = COLS + 4, NT = 32 * kDWarps;
+  constexpr int STAGE = (B::bytes + kDC * VLD * 4 + 127) / 128 * 128;
+  const DeltaScan& p = d.s;
+  extern __shared__ __align__(128) uint8_t smem[];
+  const uint32_t sb = smem_u32(smem);
+  const int h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int c0 = blockIdx.x * COLS, dk = p.dk;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row0 = p.cu_q[b], n_all = p.cu_q[b + 1] - row0, slot = p.slots[b];
+  if (n_all <= 0 || slot < 0) return;
+  const bool fresh = p.kv_lens[b] == n_all, works = c0 + warp * 16 < p.dv;
+  float* S = p.state + (((int64_t)slot * p.H + h) * dk) * p.dvp;
+  const int vloc = warp * 16 + (lane >> 2), vrow = c0 + vloc, kc = (lane & 3) * 2;
+  float acc[DK / 8][4];                      // S^T: rows (value columns) lane / 4, + 8; key channels 8 nt + kc, + 1
+#pragma unroll
+  for (int nt = 0; nt < DK / 8; ++nt)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int c = nt * 8 + kc + (e & 1), v = vrow + (e >> 1) * 8;
+      acc[nt][e] = (!fresh && c < dk && v < p.dv) ? S[(int64_t)c * p.dvp + v] : 0.f;
+    }
+  const int chunks = (n_all + kDC - 1) / kDC;
+  const uint8_t* blobs = d.blobs + (chunk_slot(row0, b, 0) * p.H + h) * B::bytes;
+  const auto load = [&](int j) {
+    if (j < chunks) {
+      const uint32_t st = sb + (j % kDStages) * STAGE;
+      const uint8_t* src = blobs + (int64_t)j * p.H * B::bytes;
+      for (int i = tid; i < B::bytes / 16; i += NT) cp_async16(st + i * 16, src + i * 16, true);
+      for (int i = tid; i < kDC * (COLS / 4); i += NT) {
+        const int r = i / (COLS / 4), c = (i % (COLS / 4)) * 4;
+        const bool ok = j * kDC + r < n_all && c0 + c < p.dvp;
+        cp_async16(st + B::bytes + (r * VLD + c) * 4,
+                   p.vn + (ok ? ((int64_t)(row0 + j * kDC + r) * p.H + h) * p.dvp + c0 + c : 0), ok);
+      }
+    }
+    cp_async_commit();
+  };
+#pragma unroll
+  for (int s = 0; s < kDStages - 1; ++s) load(s);
+  const int arow = (lane & 7) + (((lane >> 3) & 1) << 3), acb = lane >> 4;
+  const int brow = (lane & 7) + ((lane >> 4) << 3), bcb = (lane >> 3) & 1;
+  for (int j = 0; j < chunks; ++j) {
+    const int n = min(kDC, n_all - j * kDC);
+    cp_async_wait<kDStages - 2>();
+    __syncthreads();                         // chunk j is here, and everybody is done with the stage that is filled next
+    load(j + kDStages - 1);
+    if (!works) continue;
+    const uint32_t st = sb + (j % kDStages) * STAGE;
+    const uint8_t* stp = smem + (j % kDStages) * STAGE;
+    float w[2][4], wl[2][4], o[2][4], ol[2][4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) w[i][e] = wl[i][e] = o[i][e] = ol[i][e] = 0.f;
+    // ---- W^T = S^T (k 2^L)^T, O^T = S^T (q 2^L)^T
+#pragma unroll
+    for (int kk = 0; kk < DK / 16; ++kk) {
+      uint32_t kh[4], kl[4], qh[4], ql[4], hi[4], lo[4];
+      const uint32_t at = st + swz<CH>(brow, kk * 2 + bcb);
+      ldmatrix_x4(kh[0], kh[1], kh[2], kh[3], at + B::kt);
+      ldmatrix_x4(kl[0], kl[1], kl[2], kl[3], at + B::kt + B::tile);
+      ldmatrix_x4(qh[0], qh[1], qh[2], qh[3], at + B::qt);
+      ldmatrix_x4(ql[0], ql[1], ql[2], ql[3], at + B::qt + B::tile);
+      split_pack(acc[2 * kk][0], acc[2 * kk][1], hi[0], lo[0]);
+      split_pack(acc[2 * kk][2], acc[2 * kk][3], hi[1], lo[1]);
+      split_pack(acc[2 * kk + 1][0], acc[2 * kk + 1][1], hi[2], lo[2]);
+      split_pack(acc[2 * kk + 1][2], acc[2 * kk + 1][3], hi[3], lo[3]);
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        mma_bf16_16816(w[i], hi, kh[2 * i], kh[2 * i + 1]);
+        mma_bf16_16816(o[i], hi, qh[2 * i], qh[2 * i + 1]);
+        mma_bf16_16816(wl[i], lo, kh[2 * i], kh[2 * i + 1]);
+        mma_bf16_16816(ol[i], lo, qh[2 * i], qh[2 * i + 1]);
+        mma_bf16_16816(wl[i], hi, kl[2 * i], kl[2 * i + 1]);
+        mma_bf16_16816(ol[i], hi, ql[2 * i], ql[2 * i + 1]);
+      }
+    }
+    // ---- U^T = (V - W)^T M^T
+    const float* vs = reinterpret_cast<const float*>(stp + B::bytes);
+    uint32_t rh[4], rl[4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const float* v = vs + (8 * i + kc) * VLD + vloc + 8 * u;
+        split_pack(v[0] - (w[i][2 * u] + wl[i][2 * u]), v[VLD] - (w[i][2 * u + 1] + wl[i][2 * u + 1]), rh[2 * i + u], rl[2 * i + u]);
+      }
+    float uu[2][4];
+    uint32_t mh[4], ml[4], uh[4], ul[4];
+    const uint32_t small = (uint32_t)(brow * kDC * 2 + bcb * 16);
+    ldmatrix_x4(mh[0], mh[1], mh[2], mh[3], st + B::m + small);
+    ldmatrix_x4(ml[0], ml[1], ml[2], ml[3], st + B::m + kDC * kDC * 2 + small);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) uu[i][e] = 0.f;
+      mma_bf16_16816(uu[i], rh, mh[2 * i], mh[2 * i + 1]);
+      mma_bf16_16816(uu[i], rl, mh[2 * i], mh[2 * i + 1]);
+      mma_bf16_16816(uu[i], rh, ml[2 * i], ml[2 * i + 1]);
+      split_pack(uu[i][0], uu[i][1], uh[2 * i], ul[2 * i]);
+      split_pack(uu[i][2], uu[i][3], uh[2 * i + 1], ul[2 * i + 1]);
+    }
+    // ---- O^T += U^T P^T
+    ldmatrix_x4(mh[0], mh[1], mh[2], mh[3], st + B::p + small);
+    ldmatrix_x4(ml[0], ml[1], ml[2], ml[3], st + B::p + kDC * kDC * 2 + small);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      mma_bf16_16816(o[i], uh, mh[2 * i], mh[2 * i + 1]);
+      mma_bf16_16816(ol[i], ul, mh[2 * i], mh[2 * i + 1]);
+      mma_bf16_16816(ol[i], uh, ml[2 * i], ml[2 * i + 1]);
+    }
+    // ---- S^T <- 2^(L_end) S^T + U^T (k 2^(L_end - L))
+    const float* ge = reinterpret_cast<const float*>(stp + B::end);
+#pragma unroll
+    for (int nt = 0; nt < DK / 8; ++nt) {
+      const float2 f = *reinterpret_cast<const float2*>(ge + nt * 8 + kc);
+      acc[nt][0] *= f.x; acc[nt][1] *= f.y; acc[nt][2] *= f.x; acc[nt][3] *= f.y;
+    }
+#pragma unroll
+    for (int kk = 0; kk < DK / 16; ++kk) {
+      uint32_t kh[4], kl[4];
+      const uint32_t at = st + B::kc + swz<CH>(arow, kk * 2 + acb);
+      ldmatrix_x4_trans(kh[0], kh[1], kh[2], kh[3], at);
+      ldmatrix_x4_trans(kl[0], kl[1], kl[2], kl[3], at + B::tile);
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        mma_bf16_16816(acc[2 * kk + i], uh, kh[2 * i], kh[2 * i + 1]);
+        mma_bf16_16816(acc[2 * kk + i], ul, kh[2 * i], kh[2 * i + 1]);
+        mma_bf16_16816(acc[2 * kk + i], uh, kl[2 * i], kl[2 * i + 1]);
+      }
+    }
+    const int64_t row = row0 + j * kDC;
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int t = 8 * i + kc + (e & 1), v = vrow + (e >> 1) * 8;
+        if (t < n && v < p.dv) p.o[((row + t) * p.H + h) * p.dv + v] = o[i][e] + ol[i][e];
+      }
+  }
+  cp_async_wait<0>();
+  if (!works) return;
+#pragma unroll
+  for (int nt = 0; nt < DK / 8; ++nt)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int c = nt * 8 + kc + (e & 1), v = vrow + (e >> 1) * 8;
+      if (c < dk && v < p.dvp) S[(int64_t)c * p.dvp + v] = acc[nt][e];
+    }
+}
+
+template <int DK>
+static int launch_delta_chunk(const DeltaChunk& d, int n_seqs, int max_q_len, cudaStream_t s) {
+  using B = ChunkBlob<DK>;
+  constexpr int COLS = kDWarps * 16;
+  launch_pdl(delta_chunk_prep_kernel<DK>, dim3((max_q_len + kDC - 1) / kDC, d.s.H, n_seqs), dim3(256), 0, s, d);
+  const int rc = XLLM_LAUNCH_CHECK();
+  if (rc != 0) return rc;
+  const size_t smem = (size_t)kDStages * ((B::bytes + kDC * (COLS + 4) * 4 + 127) / 128 * 128);
+  const cudaError_t e = cudaFuncSetAttribute(delta_chunk_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (e != cudaSuccess) return (int)e;
+  launch_pdl(delta_chunk_kernel<DK>, dim3((d.s.dv + COLS - 1) / COLS, d.s.H, n_seqs), dim3(32 * kDWarps), smem, s, d);
+  return XLLM_LAUNCH_CHECK();
+}
+
 template <typename T>
 static int launch_channel_decay(const DeltaParams<T>& p, cudaStream_t s) {
   const int n = p.rows - p.row0;
@@ -448,23 +844,32 @@ static int launch_delta_prefill(const DeltaScan& p, int n_seqs, cudaStream_t s) 
 
 }  // namespace xllm
 
+XLLM_API int64_t xllm_delta_chunk_bytes(int rows, int n_seqs, int H, int dk) {
+  using namespace xllm;
+  const int64_t one = dk <= 64 ? ChunkBlob<64>::bytes : (dk <= 128 ? ChunkBlob<128>::bytes : ChunkBlob<256>::bytes);
+  return ((int64_t)rows / kDC + n_seqs + 1) * H * one;
+}
+
 // dtype: 0 bf16, 1 fp32 (projection rows, weights, ring, finished rows).
 //   state [slots, H, dk, dvp] fp32, dvp = dv rounded up to 4;  ring [slots, taps, 2 G dk + H dv]
 //   q, k, v, r: column blocks of rows with stride ld;  zb fp32 [rows, zb_ld]
 // gn [rows, H, dkp] fp32 is scratch (dkp = dk rounded up to 4, zeros behind dk).
 // mode 0: one token per sequence (sequence s is row s): gate, norm_w, out are used; dk <= 256, dv <= 128
 // mode 1: rows [row0, rows) by cu_q: qn, kn [rows, G, dkp], vn [rows, H, dvp] are scratch, the raw fp32 outputs go to o [rows, H, dv];  dk <= 512
+// mode 2: the same in chunks of 16 tokens, no sequence longer than max_q_len rows; dk <= 256;
+//         blobs: scratch of xllm_delta_chunk_bytes(rows, n_seqs, H, dk) bytes
 XLLM_API int xllm_delta_rule(void* state, void* ring, const void* slots, const void* cu_q, const void* kv_lens, const void* q,
                              const void* k, const void* v, const void* r, int64_t ld, const void* zb, int64_t zb_ld,
                              const void* conv_w, const void* a2, const void* dt_bias, const void* a_log, const void* gate,
                              int64_t gate_ld, const void* norm_w, void* out, int64_t out_ld, void* qn, void* kn, void* vn,
                              void* gn, void* o, int n_seqs, int rows, int row0, int H, int G, int dk, int dv, int taps,
-                             int rank, float q_scale, float eps, int dtype, int mode, void* stream) {
+                             int rank, float q_scale, float eps, int dtype, int mode, void* blobs, int max_q_len, void* stream) {
   using namespace xllm;
   if (n_seqs == 0 || rows - row0 <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G != 0 || dk <= 0 || dk > 512 || dv <= 0 || taps <= 0 || rank <= 0)
     return (int)cudaErrorInvalidValue;
   if (mode == 0 && (dk > 256 || dv > 128)) return (int)cudaErrorInvalidValue;
+  if (mode == 2 && (dk > 256 || blobs == nullptr || max_q_len <= 0)) return (int)cudaErrorInvalidValue;
   cudaStream_t s = (cudaStream_t)stream;
   int rc = 0;
   const auto run = [&](auto tag) {
@@ -477,6 +882,7 @@ XLLM_API int xllm_delta_rule(void* state, void* ring, const void* slots, const v
     p.out_ld = out_ld; p.qn = (float*)qn; p.kn = (float*)kn; p.vn = (float*)vn; p.gn = (float*)gn; p.o = (float*)o;
     p.n_seqs = n_seqs; p.rows = rows; p.row0 = row0; p.H = H; p.G = G; p.dk = dk; p.dv = dv; p.dkp = (dk + 3) & ~3;
     p.dvp = (dv + 3) & ~3; p.taps = taps; p.rank = rank; p.q_scale = q_scale; p.eps = eps;
+    p.log_decay = mode == 2;
     if ((rc = launch_channel_decay(p, s)) != 0) return;
     if (mode == 0) {
       const int RG = 256 / (p.dvp >> 2), nr = (dk + RG - 1) / RG;
@@ -502,6 +908,13 @@ XLLM_API int xllm_delta_rule(void* state, void* ring, const void* slots, const v
       if ((rc = XLLM_LAUNCH_CHECK()) != 0) return;
     }
     DeltaScan d{p.state, p.slots, p.cu_q, p.kv_lens, p.qn, p.kn, p.vn, p.gn, p.zb, zb_ld, p.o, H, G, dk, dv, p.dkp, p.dvp};
+    if (mode == 2) {
+      const DeltaChunk c{d, (uint8_t*)blobs};
+      if (dk <= 64) rc = launch_delta_chunk<64>(c, n_seqs, max_q_len, s);
+      else if (dk <= 128) rc = launch_delta_chunk<128>(c, n_seqs, max_q_len, s);
+      else rc = launch_delta_chunk<256>(c, n_seqs, max_q_len, s);
+      return;
+    }
     if (dk <= 32) rc = launch_delta_prefill<1>(d, n_seqs, s);
     else if (dk <= 64) rc = launch_delta_prefill<2>(d, n_seqs, s);
     else if (dk <= 96) rc = launch_delta_prefill<3>(d, n_seqs, s);

@@ -285,15 +285,6 @@ struct ChunkSmem {
   // dyn: cos | sin 2 x [16][rot] fp32; channel decay: lw [16][DK] fp32, bias [DK], raw r 2 x [16][RP], a2 [DK][RP + 8]
 };
 
-__device__ __forceinline__ void split_pack(float a, float b, uint32_t& hi, uint32_t& lo) {
-  const bf162 h = __floats2bfloat162_rn(a, b);
-  const float2 f = __bfloat1622float2(h);
-  const bf162 l = __floats2bfloat162_rn(a - f.x, b - f.y);
-  hi = *reinterpret_cast<const uint32_t*>(&h);
-  lo = *reinterpret_cast<const uint32_t*>(&l);
-}
-__device__ __forceinline__ float2 unpack2(uint32_t u) { return __bfloat1622float2(*reinterpret_cast<const bf162*>(&u)); }
-
 template <int DK, int NW, bool STATE_ONLY>
 __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 512 / (NW * 32)) linattn_chunk_kernel(LinAttnParams<bf16> p, SegParams sp) {
   using L = ChunkSmem<DK, NW>;

@@ -9,12 +9,20 @@
 //
 //   mlstm_decode_kernel     one token per sequence, from the projection rows to the finished row; the state crosses HBM
 //                           once in each direction
-//   mlstm_prefill_kernel    prompts: token by token with the state in registers (recurrence.cuh); the gates of a tile of
-//                           tokens come from a scan over (sum of f, maximum); one more warp keeps n.  Raw sums and
-//                           denominators go to head_norm.cu
+//   mlstm_gates_kernel,     prompts, bf16: sixteen tokens at a time on the tensor cores.  A scan over (sum of f, maximum)
+//   mlstm_chunk_kernel      gives every token's m; with F the sum of f since the chunk's start, token t sees token s of its
+//                           chunk with weight exp(F_t - F_s + i_s - m_t) and the state before the chunk with
+//                           exp(F_t + m_before - m_t), all of them at most 1.  A warp owns 16 state columns for all of dk
+//                           as fp32 accumulators of S^T, which are the A operand of O^T = S^T Q^T without leaving the
+//                           registers; so are the token-token weights (B operand of V^T P^T).  q, k and v are bf16 as
+//                           projected; S, the weights and the weighted v enter the products as a sum of two bf16 terms
+//   mlstm_prefill_kernel    prompts of any type and size: token by token in fp32 with the state in registers
+//                           (recurrence.cuh)
+// One more warp keeps n, as the state column of a value that is always 1.  Raw sums and denominators go to head_norm.cu.
 //
 // A sequence whose rows in the batch are its first tokens (kv_len == number of rows) starts from zero whatever its slot
 // holds; slot < 0 marks padding rows.  Built without fast-math: errors of the gates multiply up over a sequence.
+#include "attn_common.cuh"
 #include "recurrence.cuh"
 #include "short_conv.cuh"
 
@@ -358,6 +366,285 @@ __global__ void __launch_bounds__(256) mlstm_top_kernel(MlstmParams<T> p) {
   if (threadIdx.x == 0) *top = m;
 }
 
+// ------------------------------------------------------------------------------------------------ prompts, chunks of 16
+constexpr int kMC = 16;              // tokens per chunk
+constexpr int kMStages = 4;
+constexpr int kMWarps = 4;           // warps of 16 columns; one more for n
+
+struct MlstmGates {
+  float *a, *b, *em;                 // [H, rows]: i - F, F - m, exp(-m)
+  float* before;                     // [H, chunks]: m before the chunk; chunk j of sequence s at cu_q[s] / 16 + s + j
+  int rows, chunks;
+};
+
+// grid (heads, sequences), 256 threads; also leaves the running maximum behind the prompt in `top`
+__global__ void __launch_bounds__(256) mlstm_gates_kernel(MlstmParams<bf16> p, MlstmGates g) {
+  const int h = blockIdx.x, b = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  __shared__ float wa[8], wc[8], wm[8];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row0 = p.cu_q[b], n = p.cu_q[b + 1] - row0, slot = p.slots[b];
+  if (n <= 0 || slot < 0) return;
+  float* top = p.top + (int64_t)slot * p.H + h;
+  float m_in = p.kv_lens[b] == n ? 0.f : *top;
+  const int64_t at = (int64_t)h * g.rows + row0;
+  for (int t0 = 0; t0 < n; t0 += 256) {
+    const int t = t0 + threadIdx.x;
+    float f = 0.f, i = -INFINITY;
+    if (t < n) {
+      i = p.cap * tanhf(p.zi[(int64_t)(row0 + t) * p.z_ld + h] / p.cap);
+      f = log_sigmoid_exact(p.cap * tanhf(p.zf[(int64_t)(row0 + t) * p.z_ld + h] / p.cap));
+    }
+    float F = f;                                     // within the chunk
+#pragma unroll
+    for (int d = 1; d < kMC; d <<= 1) {
+      const float up = __shfl_up_sync(0xffffffffu, F, d, kMC);
+      if ((lane & (kMC - 1)) >= d) F += up;
+    }
+    float a = f, c = i;                              // token maps m to max(a + m, c)
+#pragma unroll
+    for (int d = 1; d < 32; d <<= 1) {
+      const float pa = __shfl_up_sync(0xffffffffu, a, d), pc = __shfl_up_sync(0xffffffffu, c, d);
+      if (lane >= d) {
+        c = fmaxf(a + pc, c);
+        a += pa;
+      }
+    }
+    if (lane == 31) { wa[warp] = a; wc[warp] = c; }
+    __syncthreads();
+    float m_warp = m_in;                             // before this warp's tokens
+    for (int w = 0; w < warp; ++w) m_warp = fmaxf(wa[w] + m_warp, wc[w]);
+    const float m = fmaxf(a + m_warp, c);
+    float prev = __shfl_up_sync(0xffffffffu, m, 1);
+    if (lane == 0) prev = m_warp;
+    if (t < n) {
+      g.a[at + t] = i - F;
+      g.b[at + t] = F - m;
+      g.em[at + t] = expf(-m);
+      if (t % kMC == 0) g.before[(int64_t)h * g.chunks + row0 / kMC + b + t / kMC] = prev;
+    }
+    for (int w = warp; w < 8; ++w) m_warp = fmaxf(wa[w] + m_warp, wc[w]);
+    m_in = m_warp;
+    __syncthreads();
+  }
+  if (threadIdx.x == 0) *top = m_in;
+}
+
+// grid (slices of 64 columns, heads, sequences)
+template <int DK>
+__global__ void __launch_bounds__(32 * (kMWarps + 1), DK > 128 ? 1 : 2) mlstm_chunk_kernel(MlstmParams<bf16> p, MlstmGates g) {
+  constexpr int CH = DK / 8, COLS = kMWarps * 16, VCH = COLS / 8, NT = 32 * (kMWarps + 1);
+  constexpr int TILE = kMC * DK * 2, STAGE = 2 * TILE + kMC * COLS * 2 + 3 * kMC * 4 + 64;
+  extern __shared__ __align__(128) uint8_t smem[];
+  const uint32_t sb = smem_u32(smem);
+  const int h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const bool keeper = warp == kMWarps;
+  const int c0 = blockIdx.x * COLS, dk = p.dk;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row0 = p.cu_q[b], n_all = p.cu_q[b + 1] - row0, slot = p.slots[b];
+  if (n_all <= 0 || slot < 0) return;
+  const bool fresh = p.kv_lens[b] == n_all;
+  const bool works = keeper ? blockIdx.x == 0 : c0 + warp * 16 < p.dv;
+  const int64_t sh = (int64_t)slot * p.H + h;
+  float* S = p.state + sh * dk * p.dvp;
+  float* N = p.norm + sh * dk;
+  const int vrow = c0 + warp * 16 + (lane >> 2), kc = (lane & 3) * 2;
+  float acc[DK / 8][4];              // S^T: rows (value columns) lane / 4, + 8; key channels 8 nt + kc, + 1
+#pragma unroll
+  for (int nt = 0; nt < DK / 8; ++nt)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int c = nt * 8 + kc + (e & 1), v = vrow + (e >> 1) * 8;
+      float x = 0.f;
+      if (works && !fresh && c < dk) {
+        if (keeper) x = (lane < 4 && e < 2) ? N[c] : 0.f;
+        else if (v < p.dv) x = S[(int64_t)c * p.dvp + v];
+      }
+      acc[nt][e] = x;
+    }
+  const int chunks = (n_all + kMC - 1) / kMC;
+  const float* before = g.before + (int64_t)h * g.chunks + row0 / kMC + b;
+  const int64_t gate_at = (int64_t)h * g.rows + row0;
+  const auto load = [&](int j) {
+    if (j < chunks) {
+      const uint32_t st = sb + (j % kMStages) * STAGE;
+      const int t0 = j * kMC;
+      const int64_t row = (int64_t)(row0 + t0) * p.ld;
+      for (int i = tid; i < kMC * CH; i += NT) {
+        const int r = i / CH, c = i % CH;
+        const bool ok = t0 + r < n_all && c * 8 < dk;
+        const int64_t go = ok ? row + r * p.ld + (int64_t)h * dk + c * 8 : 0;
+        cp_async16(st + swz<CH>(r, c), p.q + go, ok);
+        cp_async16(st + TILE + swz<CH>(r, c), p.k + go, ok);
+      }
+      for (int i = tid; i < kMC * VCH; i += NT) {
+        const int r = i / VCH, c = i % VCH;
+        const bool ok = t0 + r < n_all && c0 + c * 8 < p.dv;
+        cp_async16(st + 2 * TILE + swz<VCH>(r, c), p.v + (ok ? row + r * p.ld + (int64_t)h * p.dv + c0 + c * 8 : 0), ok);
+      }
+      float* gs = reinterpret_cast<float*>(smem + (j % kMStages) * STAGE + 2 * TILE + kMC * COLS * 2);
+      if (tid < 3 * kMC) {
+        const int which = tid / kMC, t = tid % kMC;
+        const float* src = which == 0 ? g.a : (which == 1 ? g.b : g.em);
+        gs[tid] = t0 + t < n_all ? src[gate_at + t0 + t] : 0.f;
+      } else if (tid == 3 * kMC) {
+        gs[tid] = before[j];
+      }
+    }
+    cp_async_commit();
+  };
+#pragma unroll
+  for (int s = 0; s < kMStages - 1; ++s) load(s);
+  const int arow = (lane & 7) + (((lane >> 3) & 1) << 3), acb = lane >> 4;
+  const int brow = (lane & 7) + ((lane >> 4) << 3), bcb = (lane >> 3) & 1;
+  const float qs = p.q_scale;
+  for (int j = 0; j < chunks; ++j) {
+    const int n = min(kMC, n_all - j * kMC);
+    cp_async_wait<kMStages - 2>();
+    __syncthreads();                 // chunk j is here, and everybody is done with chunk j - 1, whose stage is filled next
+    load(j + kMStages - 1);
+    if (!works) continue;
+    const uint32_t sq = sb + (j % kMStages) * STAGE, sk = sq + TILE, sv = sk + TILE;
+    const float* gs = reinterpret_cast<const float*>(smem + (j % kMStages) * STAGE + 2 * TILE + kMC * COLS * 2);
+    const float m_before = gs[3 * kMC], b_last = gs[kMC + n - 1];
+    float o[2][4], ol[2][4], pw[2][4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[i][e] = ol[i][e] = pw[i][e] = 0.f;
+    // ---- O^T = S^T Q^T and P = Q K^T
+#pragma unroll
+    for (int kk = 0; kk < DK / 16; ++kk) {
+      uint32_t qb[4], kb[4], hi[4], lo[4];
+      ldmatrix_x4(qb[0], qb[1], qb[2], qb[3], sq + swz<CH>(brow, kk * 2 + bcb));
+      ldmatrix_x4(kb[0], kb[1], kb[2], kb[3], sk + swz<CH>(brow, kk * 2 + bcb));
+      split_pack(acc[2 * kk][0], acc[2 * kk][1], hi[0], lo[0]);
+      split_pack(acc[2 * kk][2], acc[2 * kk][3], hi[1], lo[1]);
+      split_pack(acc[2 * kk + 1][0], acc[2 * kk + 1][1], hi[2], lo[2]);
+      split_pack(acc[2 * kk + 1][2], acc[2 * kk + 1][3], hi[3], lo[3]);
+      const uint32_t qa[4] = {qb[0], qb[2], qb[1], qb[3]};
+      mma_bf16_16816(o[0], hi, qb[0], qb[1]);
+      mma_bf16_16816(o[1], hi, qb[2], qb[3]);
+      mma_bf16_16816(pw[0], qa, kb[0], kb[1]);
+      mma_bf16_16816(pw[1], qa, kb[2], kb[3]);
+      mma_bf16_16816(ol[0], lo, qb[0], qb[1]);
+      mma_bf16_16816(ol[1], lo, qb[2], qb[3]);
+    }
+    // ---- weights: tokens 8 i + kc (+ 1) of this lane as columns, lane / 4 (+ 8) as rows
+    float av[2][2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int t = 8 * i + kc + e;
+        av[i][e] = gs[t];
+        const float f = qs * expf(gs[kMC + t] + m_before);
+        o[i][e] = (o[i][e] + ol[i][e]) * f;
+        o[i][e + 2] = (o[i][e + 2] + ol[i][e + 2]) * f;
+      }
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int t = (lane >> 2) + 8 * u;
+      const float bt = gs[kMC + t];
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+          pw[i][2 * u + e] = 8 * i + kc + e <= t ? pw[i][2 * u + e] * (qs * expf(bt + av[i][e])) : 0.f;
+    }
+    // ---- O^T += V^T P^T
+    uint32_t va[4];
+    if (keeper) {
+      va[0] = va[2] = lane < 4 ? 0x3F803F80u : 0u;
+      va[1] = va[3] = 0u;
+    } else {
+      ldmatrix_x4_trans(va[0], va[2], va[1], va[3], sv + swz<VCH>(arow, warp * 2 + acb));
+    }
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      uint32_t h0, h1, l0, l1;
+      split_pack(pw[0][2 * u], pw[0][2 * u + 1], h0, l0);
+      split_pack(pw[1][2 * u], pw[1][2 * u + 1], h1, l1);
+      mma_bf16_16816(o[u], va, h0, h1);
+      mma_bf16_16816(o[u], va, l0, l1);
+    }
+    // ---- S^T <- keep S^T + (w V)^T K
+    uint32_t wh[4], wl[4];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int t = 8 * i + kc;
+      const float w0 = t < n ? expf(b_last + av[i][0]) : 0.f, w1 = t + 1 < n ? expf(b_last + av[i][1]) : 0.f;
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const float2 x = unpack2(va[2 * i + u]);
+        split_pack(x.x * w0, x.y * w1, wh[2 * i + u], wl[2 * i + u]);
+      }
+    }
+    const float keep = expf(b_last + m_before);
+#pragma unroll
+    for (int nt = 0; nt < DK / 8; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[nt][e] *= keep;
+#pragma unroll
+    for (int kk = 0; kk < DK / 16; ++kk) {
+      uint32_t kt[4];
+      ldmatrix_x4_trans(kt[0], kt[1], kt[2], kt[3], sk + swz<CH>(arow, kk * 2 + acb));
+      mma_bf16_16816(acc[2 * kk], wh, kt[0], kt[1]);
+      mma_bf16_16816(acc[2 * kk + 1], wh, kt[2], kt[3]);
+      mma_bf16_16816(acc[2 * kk], wl, kt[0], kt[1]);
+      mma_bf16_16816(acc[2 * kk + 1], wl, kt[2], kt[3]);
+    }
+    const int64_t row = row0 + j * kMC;
+    if (keeper) {
+      if (lane < 4) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int t = 8 * i + kc + e;
+            if (t < n) p.div[(row + t) * p.H + h] = fmaxf(fabsf(o[i][e]), gs[2 * kMC + t]) + kDivEps;
+          }
+      }
+      continue;
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int t = 8 * i + kc + (e & 1), v = vrow + (e >> 1) * 8;
+        if (t < n && v < p.dv) p.o[((row + t) * p.H + h) * p.dv + v] = o[i][e];
+      }
+  }
+  cp_async_wait<0>();
+  if (!works) return;
+#pragma unroll
+  for (int nt = 0; nt < DK / 8; ++nt)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int c = nt * 8 + kc + (e & 1), v = vrow + (e >> 1) * 8;
+      if (c >= dk) continue;
+      if (keeper) {
+        if (lane < 4 && e < 2) N[c] = acc[nt][e];
+      } else if (v < p.dvp) {
+        S[(int64_t)c * p.dvp + v] = acc[nt][e];
+      }
+    }
+}
+
+template <int DK>
+static int launch_mlstm_chunk(const MlstmParams<bf16>& p, const MlstmGates& g, int n_seqs, cudaStream_t s) {
+  constexpr int COLS = kMWarps * 16;
+  const size_t smem = (size_t)kMStages * (2 * kMC * DK * 2 + kMC * COLS * 2 + 3 * kMC * 4 + 64);
+  const cudaError_t e = cudaFuncSetAttribute(mlstm_chunk_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (e != cudaSuccess) return (int)e;
+  launch_pdl(mlstm_gates_kernel, dim3(p.H, n_seqs), dim3(256), 0, s, p, g);
+  const int rc = XLLM_LAUNCH_CHECK();
+  if (rc != 0) return rc;
+  launch_pdl(mlstm_chunk_kernel<DK>, dim3((p.dv + COLS - 1) / COLS, p.H, n_seqs), dim3(32 * (kMWarps + 1)), smem, s, p, g);
+  return XLLM_LAUNCH_CHECK();
+}
+
 template <typename T, int V, int J>
 static int launch_mlstm_prefill(const MlstmParams<T>& p, int n_seqs, cudaStream_t s) {
   constexpr int COLS = kMlstmWarps * kRecCols;
@@ -387,10 +674,12 @@ static int run_mlstm_prefill(const MlstmParams<T>& p, int n_seqs, cudaStream_t s
 //   q, k, v: column blocks of rows with stride ld;  zi, zf fp32 with row stride z_ld
 // mode 0: one token per sequence (sequence s is row s): gate, norm_w, out are used; dk <= 256, dv <= 128
 // mode 1: prompt rows by cu_q: sums to o fp32 [rows, H, dv], denominators to div fp32 [rows, H];  dk <= 512
+// mode 2: the same in chunks of 16 tokens (bf16, dk and dv multiples of 8, dk <= 256, aligned rows; otherwise mode 1);
+//         gates: fp32 scratch of 3 H rows + H (rows / 16 + n_seqs + 1)
 XLLM_API int xllm_mlstm(void* state, void* norm, void* top, const void* slots, const void* cu_q, const void* kv_lens,
                         const void* q, const void* k, const void* v, int64_t ld, const void* zi, const void* zf, int64_t z_ld,
                         const void* gate, int64_t gate_ld, const void* norm_w, void* out, int64_t out_ld, void* o, void* div,
-                        int n_seqs, int H, int dk, int dv, float q_scale, float cap, float eps, int dtype, int mode,
+                        void* gates, int rows, int n_seqs, int H, int dk, int dv, float q_scale, float cap, float eps, int dtype, int mode,
                         void* stream) {
   using namespace xllm;
   if (n_seqs == 0) return 0;
@@ -416,6 +705,18 @@ XLLM_API int xllm_mlstm(void* state, void* norm, void* top, const void* slots, c
       else launch_pdl(mlstm_decode_kernel<T, 32>, grid, block, smem, s, p);
       rc = XLLM_LAUNCH_CHECK();
       return;
+    }
+    if constexpr (sizeof(T) == 2) {
+      const auto a16 = [](const void* x) { return (((uintptr_t)x) & 15) == 0; };
+      if (mode == 2 && gates != nullptr && dk % 8 == 0 && dv % 8 == 0 && dk <= 256 && ld % 8 == 0 && a16(q) && a16(k) && a16(v)) {
+        MlstmGates g;
+        g.rows = rows; g.chunks = rows / kMC + n_seqs + 1;
+        g.a = (float*)gates; g.b = g.a + (int64_t)H * rows; g.em = g.b + (int64_t)H * rows; g.before = g.em + (int64_t)H * rows;
+        if (dk <= 64) rc = launch_mlstm_chunk<64>(p, g, n_seqs, s);
+        else if (dk <= 128) rc = launch_mlstm_chunk<128>(p, g, n_seqs, s);
+        else rc = launch_mlstm_chunk<256>(p, g, n_seqs, s);
+        return;
+      }
     }
     const auto al = [](const void* x) { return (((uintptr_t)x) & (4 * sizeof(T) - 1)) == 0; };
     if (dk % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && al(q) && al(k) && al(v)) rc = run_mlstm_prefill<T, 4>(p, n_seqs, s);

@@ -282,7 +282,7 @@ class DeltaRuleMixer(Module):
                            r[:nd], zb[:nd], gate[:nd], out[:nd])
         if meta.n_prefill > 0:
             self.op.prefill(state["S"], state["conv"], slots[nd:], meta.cu_q[nd:], meta.kv_lens[nd:], q, k, v, r, zb, gate, out,
-                            row0=nd, padded=meta.padded)
+                            row0=nd, padded=meta.padded, max_q_len=meta.max_q_len)
         return self.o(out)
 
     __call__ = forward

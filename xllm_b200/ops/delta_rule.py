@@ -15,7 +15,8 @@ from . import _lib
 from ._lib import F, I, L, P, check, ptr, stream
 from .head_norm import head_norm_gate
 
-_lib.register_signature("xllm_delta_rule", [P] * 9 + [L, P, L] + [P] * 5 + [L, P, P, L] + [P] * 5 + [I] * 9 + [F, F, I, I, P])
+_lib.register_signature("xllm_delta_rule", [P] * 9 + [L, P, L] + [P] * 5 + [L, P, P, L] + [P] * 5 + [I] * 9 + [F, F, I, I, P, I, P])
+_lib.register_signature("xllm_delta_chunk_bytes", [I, I, I, I], L)
 
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 
@@ -43,7 +44,8 @@ class ChannelDelta:
     def channels(self):
         return 2 * self.kv_heads * self.dk + self.heads * self.dv
 
-    def _launch(self, mode, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out, scratch, rows, row0):
+    def _launch(self, mode, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out, scratch, rows, row0, blobs=None,
+                max_q_len=0):
         ld = q.stride(0)
         for t in (q, k, v, r):
             assert t.stride(0) == ld and t.stride(1) == 1 and t.dtype == q.dtype
@@ -56,9 +58,10 @@ class ChannelDelta:
             ptr(state), ptr(ring), ptr(slots), ptr(cu_q), ptr(kv_lens), ptr(q), ptr(k), ptr(v), ptr(r), ld, ptr(zb), zb.stride(0),
             ptr(self.conv_w), ptr(self.a2), ptr(self.dt_bias), ptr(self.a_log), ptr(gate), gate.stride(0), ptr(self.norm_w),
             ptr(out), out.stride(0), ptr(qn), ptr(kn), ptr(vn), ptr(gn), ptr(o), slots.shape[0], rows, row0, H, self.kv_heads,
-            dk, dv, self.taps, self.a2.shape[1], self.q_scale, self.eps, _DT[q.dtype], mode, stream()), "delta_rule")
+            dk, dv, self.taps, self.a2.shape[1], self.q_scale, self.eps, _DT[q.dtype], mode, ptr(blobs), max_q_len, stream()),
+            "delta_rule")
         from . import _count
-        _count(2 if mode == 0 else (4 if self.taps > 1 else 3))
+        _count(2 if mode == 0 else 2 + mode + int(self.taps > 1))
 
     def _decays(self, rows, device):
         dkp = round4(self.dk)
@@ -76,9 +79,11 @@ class ChannelDelta:
         self._launch(0, state, ring, slots, None, kv_lens, q, k, v, r, zb, gate, out, scratch, B, 0)
         return out
 
-    def prefill(self, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out, row0=0, padded=False):
+    def prefill(self, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out, row0=0, padded=False,
+                max_q_len=None, token_by_token=False):
         """Prompt rows of several sequences (absolute token rows cu_q, all at or behind row0); fills rows [row0, T) of `out`.
-        `padded`: rows outside every sequence exist and must come out finite."""
+        `padded`: rows outside every sequence exist and must come out finite.  `max_q_len`: the most rows any sequence has
+        (default: all rows).  `token_by_token`: the fp32 recurrence instead of the chunked form."""
         if not q.is_cuda:
             return self._cpu(state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out)
         T, H, G = q.shape[0], self.heads, self.kv_heads
@@ -87,7 +92,11 @@ class ChannelDelta:
         scratch = (torch.empty((T, G, dkp), **f32), torch.empty((T, G, dkp), **f32), torch.empty((T, H, dvp), **f32),
                    self._decays(T, q.device),
                    (torch.zeros if padded else torch.empty)((T, H, self.dv), **f32))
-        self._launch(1, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out, scratch, T, row0)
+        blobs, n = None, slots.shape[0]
+        if q.dtype == torch.bfloat16 and self.dk <= 256 and not token_by_token:
+            blobs = torch.empty(_lib.load().xllm_delta_chunk_bytes(T, n, H, self.dk), dtype=torch.uint8, device=q.device)
+        self._launch(1 if blobs is None else 2, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out, scratch, T, row0,
+                     blobs, int(max_q_len or T))
         head_norm_gate(scratch[4][row0:], out[row0:], g=gate[row0:], w=self.norm_w, act="sigmoid", eps=self.eps)
         return out
 

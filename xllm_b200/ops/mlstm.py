@@ -17,7 +17,7 @@ from ._lib import F, I, L, P, check, ptr, stream
 from .delta_rule import round4
 from .head_norm import head_norm_gate
 
-_lib.register_signature("xllm_mlstm", [P] * 9 + [L, P, P, L, P, L, P, P, L, P, P] + [I] * 4 + [F] * 3 + [I, I, P])
+_lib.register_signature("xllm_mlstm", [P] * 9 + [L, P, P, L, P, L, P, P, L, P, P, P] + [I] * 5 + [F] * 3 + [I, I, P])
 
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 
@@ -32,7 +32,7 @@ class MatrixMemory:
     eps: float = 1e-6
     norm_w: Optional[torch.Tensor] = None        # [heads * dv]
 
-    def _launch(self, mode, st, slots, cu_q, kv_lens, q, k, v, zi, zf, gate, out, o, div):
+    def _launch(self, mode, st, slots, cu_q, kv_lens, q, k, v, zi, zf, gate, out, o, div, gates=None):
         ld = q.stride(0)
         for t in (q, k, v):
             assert t.stride(0) == ld and t.stride(1) == 1 and t.dtype == q.dtype
@@ -45,7 +45,7 @@ class MatrixMemory:
         check(_lib.load().xllm_mlstm(
             ptr(S), ptr(n), ptr(m), ptr(slots), ptr(cu_q), ptr(kv_lens), ptr(q), ptr(k), ptr(v), ld, ptr(zi), ptr(zf),
             zi.stride(0), ptr(gate), gate.stride(0), ptr(self.norm_w), ptr(out), out.stride(0), ptr(o), ptr(div),
-            slots.shape[0], H, dk, dv, self.q_scale, self.cap, self.eps, _DT[q.dtype], mode, stream()), "mlstm")
+            ptr(gates), q.shape[0], slots.shape[0], H, dk, dv, self.q_scale, self.cap, self.eps, _DT[q.dtype], mode, stream()), "mlstm")
         from . import _count
         _count(1 if mode == 0 else 2)
 
@@ -59,15 +59,21 @@ class MatrixMemory:
         self._launch(0, st, slots, None, kv_lens, q, k, v, zi, zf, gate, out, None, None)
         return out
 
-    def prefill(self, st, slots, cu_q, kv_lens, q, k, v, zi, zf, gate, out, row0=0, padded=False):
+    def prefill(self, st, slots, cu_q, kv_lens, q, k, v, zi, zf, gate, out, row0=0, padded=False,
+                token_by_token=False):
         """Prompt rows of several sequences (absolute token rows cu_q, all at or behind row0); fills rows [row0, T) of `out`.
-        `padded`: rows outside every sequence exist and must come out finite."""
+        `padded`: rows outside every sequence exist and must come out finite.  `token_by_token`: the fp32 recurrence instead of
+        the chunked form."""
         if not q.is_cuda:
             return self._cpu(st, slots, cu_q, kv_lens, q, k, v, zi, zf, gate, out)
         make = torch.zeros if padded else torch.empty
         o = make((q.shape[0], self.heads, self.dv), dtype=torch.float32, device=q.device)
         div = make((q.shape[0], self.heads), dtype=torch.float32, device=q.device)
-        self._launch(1, st, slots, cu_q, kv_lens, q, k, v, zi, zf, gate, out, o, div)
+        gates = None
+        if q.dtype == torch.bfloat16 and not token_by_token:
+            T, n = q.shape[0], slots.shape[0]
+            gates = torch.empty(self.heads * (3 * T + T // 16 + n + 1), dtype=torch.float32, device=q.device)
+        self._launch(1 if gates is None else 2, st, slots, cu_q, kv_lens, q, k, v, zi, zf, gate, out, o, div, gates)
         head_norm_gate(o[row0:], out[row0:], div=div[row0:], g=gate[row0:], w=self.norm_w, act="sigmoid", eps=self.eps)
         return out
 
