@@ -404,7 +404,7 @@ def recurrent_rows(results, hbm, tf, tag):
         print(f"{name:<34} {shape:<26} {t*1e6:9.1f} us {nbytes/t/1e9:7.0f} GB/s {flops/t/1e12:7.1f} TF/s  {ideal/t:6.3f} of {tag}",
               flush=True)
 
-    delta = ChannelDelta(H, H, d, d, 4, q_scale=d ** -0.5, conv_w=rows(3 * H * d, 4) * 0.5, a2=rows(H * d, R) * 0.05,
+    delta = ChannelDelta(H, H, d, d, 4, q_scale=d ** -0.5, conv_w=rows(4, 3 * H * d) * 0.5, a2=rows(H * d, R) * 0.05,
                          dt_bias=torch.full((H * d,), -4.0, device=dev, dtype=bf), a_log=torch.zeros(H, device=dev, dtype=bf),
                          norm_w=torch.ones(d, device=dev, dtype=bf))
     mem = MatrixMemory(H, d, d, 15.0, q_scale=d ** -0.5, norm_w=torch.ones(H * d, device=dev, dtype=bf))

@@ -21,6 +21,7 @@ hundred MB on the device, a handful of launches).
     python benchmarks/profile_case.py --kernel gemm_act   # gate_up GEMM with the SiLU-mul epilogue, 2304 x 24576 x 4096
     python benchmarks/profile_case.py --kernel xattn      # beam attention: 16 requests x 128 beams over 2048-token prompts
     python benchmarks/profile_case.py --kernel linattn    # decayed linear attention, 4096-token prompt x 32 heads (linattn_channel: per-channel decay)
+    python benchmarks/profile_case.py --kernel delta      # delta rule prompts, 4 x 1024 tokens x 32 heads (mlstm: matrix memory; *_decode: 64 sequences)
     python benchmarks/profile_case.py --kernel gdn_prefill # gated-delta-rule prompt chunk, 4096 tokens x 32 heads
 """
 import argparse
@@ -207,6 +208,29 @@ def main():
         sl, cu, kl, pos = i32([0]), i32([0, T]), i32([T]), torch.arange(T, device=dev)
         out = torch.empty(T, H * d, device=dev, dtype=torch.bfloat16)
         fn = lambda: op.prefill(st, sl, cu, kl, pos, c[0], c[1], c[2], g=c[3], r=c[4], out=out, max_q_len=T)
+    elif a.kernel in ("delta", "delta_decode", "mlstm", "mlstm_decode"):
+        from xllm_b200.ops.delta_rule import ChannelDelta
+        from xllm_b200.ops.mlstm import MatrixMemory
+        S, L, H, d, R, bf = (64, 1, 32, 128, 128, torch.bfloat16) if a.kernel.endswith("decode") else (4, 1024, 32, 128, 128, torch.bfloat16)
+        T = S * L
+        rnd = lambda *s: torch.randn(*s, device=dev, dtype=bf)
+        i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+        r, z, out = rnd(T, 4 * H * d + R), torch.randn(T, 2 * H, device=dev), torch.empty(T, H * d, device=dev, dtype=bf)
+        c = [r[:, i * H * d:(i + 1) * H * d] for i in range(4)] + [r[:, 4 * H * d:]]
+        sl, cu, kl = i32(list(range(S))), i32([i * L for i in range(S + 1)]), i32([L if L > 1 else 100] * S)
+        st = torch.zeros(S + 1, H, d, d, device=dev)
+        if a.kernel.startswith("delta"):
+            op = ChannelDelta(H, H, d, d, 4, q_scale=d ** -0.5, conv_w=rnd(4, 3 * H * d) * 0.5, a2=rnd(H * d, R) * 0.05,
+                              dt_bias=torch.full((H * d,), -4.0, device=dev, dtype=bf), a_log=torch.zeros(H, device=dev, dtype=bf),
+                              norm_w=torch.ones(d, device=dev, dtype=bf))
+            ring = torch.zeros(S + 1, 4, 3 * H * d, device=dev, dtype=bf)
+            run = op.decode if L == 1 else op.prefill
+            fn = lambda: run(st, ring, sl, cu, kl, *c[:3], c[4], z, c[3], out)
+        else:
+            op = MatrixMemory(H, d, d, 15.0, q_scale=d ** -0.5, norm_w=torch.ones(H * d, device=dev, dtype=bf))
+            mst = {"S": st, "n": torch.zeros(S + 1, H, d, device=dev), "m": torch.zeros(S + 1, H, device=dev)}
+            run = op.decode if L == 1 else op.prefill
+            fn = lambda: run(mst, sl, cu, kl, *c[:3], z[:, :H], z[:, H:], c[3], out)
     else:
         raise SystemExit(f"unknown kernel {a.kernel}")
     for _ in range(a.iters):

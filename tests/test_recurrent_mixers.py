@@ -75,11 +75,11 @@ class DeltaCase(Case):
         self.zb = (2 * mk(self.T, H)).to(self.dev)
         put = lambda t: t.to(self.dt).to(self.dev)
         C = 2 * G * dk + H * dv
-        self.op = op = ChannelDelta(H, G, dk, dv, taps, q_scale=dk ** -0.5, eps=1e-5, conv_w=put(mk(C, taps) * 0.6),
+        self.op = op = ChannelDelta(H, G, dk, dv, taps, q_scale=dk ** -0.5, eps=1e-5, conv_w=put(mk(C, taps).T.contiguous() * 0.6),
                                     a2=put(mk(H * dk, rank) * rank ** -0.5), dt_bias=put(bias + mk(H * dk)),
                                     a_log=put(a_log + 0.5 * mk(H)), norm_w=put(1 + 0.3 * mk(dv)))
         d = lambda t: t.double().cpu()
-        cw, share = d(op.conv_w), torch.arange(H) // (H // G)
+        cw, share = d(op.conv_w).T, torch.arange(H) // (H // G)
         unit = lambda x: x / torch.sqrt((x * x).sum(-1, keepdim=True) + 1e-6)
         self.want = []
         for a, b in self.bounds:

@@ -36,7 +36,7 @@ struct DeltaParams {
   int64_t ld;
   const float* zb;           // [rows, zb_ld] fp32: pre-sigmoid beta of head h in column h
   int64_t zb_ld;
-  const T* conv_w;           // [C, taps]
+  const T* conv_w;           // [taps, C], the last row is the current token's
   const T* a2;               // [H dk, rank]
   const T* dt_bias;          // [H dk]
   const T* a_log;            // [H]
@@ -56,13 +56,25 @@ struct DeltaParams {
 };
 
 __device__ __forceinline__ float softplus_exact(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+// log(1 + e) = 2 artanh(s), s = e / (2 + e) <= 1/3 for e <= 1: six terms of the series leave a relative error of 2e-7
+__device__ __forceinline__ float softplus_series(float z) {
+  const float e = __expf(-fabsf(z)), s = __fdividef(e, 2.f + e), q = s * s;
+  const float y = 1.f + q * (1.f / 3 + q * (1.f / 5 + q * (1.f / 7 + q * (1.f / 9 + q * (1.f / 11)))));
+  return fmaxf(z, 0.f) + 2.f * s * y;
+}
+// 2^x, flushing denormal results
+__device__ __forceinline__ float exp2_flush(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 
 constexpr float kUnitEps = 1e-6f;
 
 // ------------------------------------------------------------------------------------------------ decode
 // grid (heads, sequences), 256 threads: dvp / 4 column groups x row groups, NR rows of four columns per thread.
 template <typename T, int NR>
-__global__ void __launch_bounds__(256) delta_decode_kernel(DeltaParams<T> p) {
+__global__ void __launch_bounds__(256, NR <= 8 ? 3 : (NR <= 16 ? 2 : 1)) delta_decode_kernel(DeltaParams<T> p) {
   extern __shared__ __align__(16) float sm[];
   const int dk = p.dk, dv = p.dv, dvp = p.dvp, dkp = p.dkp;
   float* qs = sm;
@@ -83,6 +95,37 @@ __global__ void __launch_bounds__(256) delta_decode_kernel(DeltaParams<T> p) {
     return;
   }
   const bool active = rg < RG, fresh = len == 1;
+  const int pos = len - 1, g = h / (p.H / p.G), G = p.G, taps = p.taps;
+  const int64_t C = p.channels();
+  T* ring = p.ring + (int64_t)slot * taps * C;
+  T* ring_now = ring + (int64_t)(pos % taps) * C;
+  const bool keeps_qk = h % (p.H / G) == 0;
+  // channels of this head in the order q | k | v; the loads of up to four taps go out before those of the state
+  constexpr int NE = 3;                    // 2 dk + dv <= 640
+  const auto channel = [&](int i, const T*& x) {
+    if (i < dk) { x = p.q + b * p.ld + (int64_t)g * dk + i; return (int64_t)g * dk + i; }
+    if (i < 2 * dk) { x = p.k + b * p.ld + (int64_t)g * dk + i - dk; return (int64_t)(G + g) * dk + i - dk; }
+    x = p.v + b * p.ld + (int64_t)h * dv + i - 2 * dk;
+    return (int64_t)2 * G * dk + (int64_t)h * dv + i - 2 * dk;
+  };
+  T xin[NE][4], win[NE][4];
+  if (taps <= 4) {
+#pragma unroll
+    for (int e = 0; e < NE; ++e) {
+      const int i = tid + 256 * e;
+#pragma unroll
+      for (int t = 0; t < 4; ++t) xin[e][t] = win[e][t] = from_f32<T>(0.f);
+      if (i >= 2 * dk + dv) continue;
+      const T* x;
+      const int64_t c = channel(i, x);
+      xin[e][0] = *x;
+#pragma unroll
+      for (int t = 0; t < 4; ++t) {
+        if (t < taps) win[e][t] = p.conv_w[(taps - 1 - t) * C + c];
+        if (t > 0 && t < taps && t <= pos) xin[e][t] = ring[(int64_t)((pos - t) % taps) * C + c];
+      }
+    }
+  }
   float* S = p.state + (((int64_t)slot * p.H + h) * dk) * dvp + cg * 4;
   float4 s[NR];
 #pragma unroll
@@ -91,25 +134,25 @@ __global__ void __launch_bounds__(256) delta_decode_kernel(DeltaParams<T> p) {
     s[u] = (active && !fresh && r < dk) ? *reinterpret_cast<const float4*>(S + (int64_t)r * dvp)
                                         : make_float4(0.f, 0.f, 0.f, 0.f);
   }
-  const int pos = len - 1, g = h / (p.H / p.G), G = p.G, taps = p.taps;
-  const int64_t C = p.channels();
-  T* ring = p.ring + (int64_t)slot * taps * C;
-  T* ring_now = ring + (int64_t)(pos % taps) * C;
-  const bool keeps_qk = h % (p.H / G) == 0;
-  // channels of this head in the order q | k | v; the token's own inputs go to its ring row
   float sq = 0.f, sk = 0.f;
-  for (int i = tid; i < 2 * dk + dv; i += 256) {
+#pragma unroll
+  for (int e = 0; e < NE; ++e) {
+    const int i = tid + 256 * e;
+    if (i >= 2 * dk + dv) continue;
     const T* x;
-    int64_t c;
-    if (i < dk) { x = p.q + b * p.ld + (int64_t)g * dk + i; c = (int64_t)g * dk + i; }
-    else if (i < 2 * dk) { x = p.k + b * p.ld + (int64_t)g * dk + i - dk; c = (int64_t)(G + g) * dk + i - dk; }
-    else { x = p.v + b * p.ld + (int64_t)h * dv + i - 2 * dk; c = (int64_t)2 * G * dk + (int64_t)h * dv + i - 2 * dk; }
-    float y;
-    conv_silu<T, 1>(x, p.ld, 0, pos, ring + c, C, p.conv_w + c * taps, taps, &y);
+    const int64_t c = channel(i, x);
+    float y = 0.f;
+    if (taps <= 4) {
+#pragma unroll
+      for (int t = 0; t < 4; ++t) y += to_f32(xin[e][t]) * to_f32(win[e][t]);
+      y = silu_as<T>(y);
+    } else {
+      conv_silu<T, 1>(x, p.ld, 0, pos, ring + c, C, p.conv_w + c, taps, &y);
+    }
     if (i < dk) { qs[i] = y; sq += y * y; }
     else if (i < 2 * dk) { ks[i - dk] = y; sk += y * y; }
     else vs[i - 2 * dk] = y;
-    if (taps > 1 && (keeps_qk || i >= 2 * dk)) ring_now[c] = *x;
+    if (taps > 1 && (keeps_qk || i >= 2 * dk)) ring_now[c] = *x;      // the token's own inputs go to its ring row
   }
   for (int i = dv + tid; i < dvp; i += 256) vs[i] = 0.f;
   for (int i = tid; i < dk; i += 256) gs[i] = p.gn[((int64_t)b * p.H + h) * dkp + i];
@@ -196,7 +239,7 @@ __global__ void __launch_bounds__(256) conv_heads_kernel(DeltaParams<T> p) {
   const T* x = (part == 0 ? p.q : (part == 1 ? p.k : p.v)) + row * p.ld + (int64_t)h * d;
   const int64_t C = p.channels();
   const T* ring = p.ring + (int64_t)p.slots[b] * p.taps * C + c0;
-  const T* w = p.conv_w + c0 * p.taps;
+  const T* w = p.conv_w + c0;
   float* dst = (part == 0 ? p.qn : (part == 1 ? p.kn : p.vn)) + ((int64_t)row * (part == 2 ? p.H : p.G) + h) * dp;
   float y[NI][V];
   float ss = 0.f;
@@ -206,7 +249,7 @@ __global__ void __launch_bounds__(256) conv_heads_kernel(DeltaParams<T> p) {
 #pragma unroll
     for (int j = 0; j < V; ++j) y[i][j] = 0.f;
     if (c >= d) continue;
-    conv_silu<T, V>(x + c, p.ld, back, pos, ring + c, C, w + (int64_t)c * p.taps, p.taps, y[i]);
+    conv_silu<T, V>(x + c, p.ld, back, pos, ring + c, C, w + c, p.taps, y[i]);
 #pragma unroll
     for (int j = 0; j < V; ++j) ss += y[i][j] * y[i][j];
   }
@@ -219,6 +262,87 @@ __global__ void __launch_bounds__(256) conv_heads_kernel(DeltaParams<T> p) {
 #pragma unroll
     for (int j = 0; j < V; ++j) y[i][j] *= f;
     store_f32<V>(dst + c, y[i]);
+  }
+}
+
+// The same for up to four taps and heads of up to 128 channels: one warp per (run of rows, head), which reads every input
+// once and keeps the last ones in registers; a lane owns four neighbouring channels.
+constexpr int kConvRun = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(256) conv_heads_run_kernel(DeltaParams<T> p) {
+  const int lane = threadIdx.x & 31, items = 2 * p.G + p.H;
+  const unsigned it = blockIdx.x * 8 + (threadIdx.x >> 5), run = it / items;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int first = p.row0 + (int)run * kConvRun;
+  if (first >= p.rows) return;
+  int h = (int)(it - run * items);
+  const int part = h < p.G ? 0 : (h < 2 * p.G ? 1 : 2);
+  h -= part == 0 ? 0 : (part == 1 ? p.G : 2 * p.G);
+  const int d = part == 2 ? p.dv : p.dk, c = lane * 4;
+  const int64_t c0 = (part == 2 ? (int64_t)2 * p.G * p.dk : (int64_t)part * p.G * p.dk) + (int64_t)h * d + c, C = p.channels();
+  const T* x = (part == 0 ? p.q : (part == 1 ? p.k : p.v)) + (int64_t)h * d + c;
+  float* dst = (part == 0 ? p.qn : (part == 1 ? p.kn : p.vn)) + (int64_t)h * d + c;
+  const int64_t dst_ld = (int64_t)(part == 2 ? p.H : p.G) * d;      // d is a multiple of 4: no padding
+  const bool on = c < d;
+  float v[kConvRun + 3][4], w[4][4];                                // w[taps back][channel]
+#pragma unroll
+  for (int r = 0; r < kConvRun + 3; ++r) {
+    const int row = first + r - 3;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v[r][j] = 0.f;
+    if (on && row >= 0 && row < p.rows) load_f32<4>(x + row * p.ld, v[r]);
+  }
+#pragma unroll
+  for (int b = 0; b < 4; ++b)
+  {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) w[b][j] = 0.f;
+    if (on && b < p.taps) load_f32<4>(p.conv_w + (p.taps - 1 - b) * C + c0, w[b]);
+  }
+  int b = -1, begin = 0, end = 0;
+#pragma unroll
+  for (int r = 0; r < kConvRun; ++r) {
+    const int row = first + r;
+    if (row >= p.rows) break;
+    if (row >= end) {                                               // the row starts another sequence, or is the first
+      b = seq_of_row(p.cu_q, p.n_seqs, row);
+      begin = b < 0 ? row : p.cu_q[b];
+      end = b < 0 ? row + 1 : p.cu_q[b + 1];
+    }
+    const int slot = b < 0 ? -1 : p.slots[b];
+    if (slot < 0) continue;
+    const int back = row - begin;
+    float y[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      y[j] = v[r + 3][j] * w[0][j];
+      if (back >= 1) y[j] += v[r + 2][j] * w[1][j];
+      if (back >= 2) y[j] += v[r + 1][j] * w[2][j];
+      if (back >= 3) y[j] += v[r][j] * w[3][j];
+    }
+    if (back < p.taps - 1) {                                        // inputs of earlier steps
+      const int pos = p.kv_lens[b] - (end - row);
+      for (int t = back + 1; t < p.taps && t <= pos && on; ++t) {
+        float z[4];
+        load_f32<4>(p.ring + ((int64_t)slot * p.taps + (pos - t) % p.taps) * C + c0, z);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[j] += z[j] * (t == 1 ? w[1][j] : (t == 2 ? w[2][j] : w[3][j]));
+      }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      y[j] = silu_as<T>(y[j]);
+      ss += y[j] * y[j];
+    }
+    if (part < 2) {
+      const float f = (part == 0 ? p.q_scale : 1.f) / sqrtf(warp_sum(ss) + kUnitEps);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) y[j] *= f;
+    }
+    if (on) store_f32<4>(dst + row * dst_ld, y);
   }
 }
 
@@ -244,17 +368,19 @@ __global__ void __launch_bounds__(128) channel_decay_tile_kernel(DeltaParams<bf1
   const int RP = (p.rank + 15) & ~15, st = RP + 8;
   bf16* rs = reinterpret_cast<bf16*>(raw);          // [64][st]
   bf16* ws = rs + 64 * st;                          // [64][st]
+  __shared__ float rate[64], bias[64];              // -exp(A_log), dt_bias
+  __shared__ int64_t at[64];                        // column of the output row
   const int r0 = p.row0 + blockIdx.x * 64, c0 = blockIdx.y * 64, tid = threadIdx.x, nc = p.H * p.dk;
   const int warp = tid >> 5, lane = tid & 31;
   const bf16 zero = __float2bfloat16(0.f);
   const bool v8 = p.rank % 8 == 0 && p.ld % 8 == 0 && (((uintptr_t)p.a2 | (uintptr_t)p.r) & 15) == 0;
-  const uint4 zero8 = make_uint4(0, 0, 0, 0);
   const auto copy = [&](bf16* dst, const bf16* src, int64_t ld, int n) {     // n rows of `rank` elements, zeros behind
     if (v8) {
       const int per = RP >> 3;
       for (int i = tid; i < 64 * per; i += 128) {
         const int y = i / per, x = (i - y * per) * 8;
-        *reinterpret_cast<uint4*>(dst + y * st + x) = (y < n && x < p.rank) ? *reinterpret_cast<const uint4*>(src + y * ld + x) : zero8;
+        const bool ok = y < n && x < p.rank;
+        cp_async16(smem_u32(dst + y * st + x), ok ? src + y * ld + x : src, ok);
       }
     } else {
       for (int i = tid; i < 64 * RP; i += 128) {
@@ -264,9 +390,17 @@ __global__ void __launch_bounds__(128) channel_decay_tile_kernel(DeltaParams<bf1
     }
   };
   copy(ws, p.a2 + (int64_t)c0 * p.rank, p.rank, nc - c0);
+  if (tid < 64 && c0 + tid < nc) {
+    const int h = (c0 + tid) / p.dk;
+    rate[tid] = -expf(__bfloat162float(p.a_log[h])) * (p.log_decay ? 1.44269504088896341f : 1.f);
+    bias[tid] = __bfloat162float(p.dt_bias[c0 + tid]);
+    at[tid] = (int64_t)h * p.dkp + c0 + tid - h * p.dk;
+  }
   pdl_wait();
   pdl_launch_dependents();
   copy(rs, p.r + (int64_t)r0 * p.ld, p.ld, p.rows - r0);
+  cp_async_commit();
+  cp_async_wait<0>();
   __syncthreads();
   float z[8][4];
 #pragma unroll
@@ -286,21 +420,26 @@ __global__ void __launch_bounds__(128) channel_decay_tile_kernel(DeltaParams<bf1
       mma_bf16_16816(z[n], a, *reinterpret_cast<const uint32_t*>(w), *reinterpret_cast<const uint32_t*>(w + 8));
     }
   }
+  const int64_t ld = (int64_t)p.H * p.dkp;
+  const bool pairs = p.dkp == p.dk && p.dk % 2 == 0;         // a pair of channels is one 8-byte store
 #pragma unroll
   for (int n = 0; n < 8; ++n) {
-    const int c = c0 + n * 8 + kc;
+    const int c = n * 8 + kc;
+    if (c0 + c >= nc) break;
+    const bool two = c0 + c + 1 < nc;
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      if (c + e >= nc) break;
-      const int h = (c + e) / p.dk, ch = c + e - h * p.dk;
-      const float A = expf(__bfloat162float(p.a_log[h])), bias = __bfloat162float(p.dt_bias[c + e]);
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        const int row = r0 + ra + 8 * u;
-        if (row < p.rows) {
-          const float g = -A * softplus_exact(z[n][2 * u + e] + bias);
-          p.gn[((int64_t)row * p.H + h) * p.dkp + ch] = p.log_decay ? g * 1.44269504088896341f : expf(g);
-        }
+    for (int u = 0; u < 2; ++u) {
+      const int row = r0 + ra + 8 * u;
+      if (row >= p.rows) continue;
+      float g0 = rate[c] * softplus_series(z[n][2 * u] + bias[c]);
+      float g1 = two ? rate[c + 1] * softplus_series(z[n][2 * u + 1] + bias[c + 1]) : 0.f;
+      if (!p.log_decay) { g0 = expf(g0); g1 = expf(g1); }
+      float* dst = p.gn + row * ld;
+      if (pairs) {
+        *reinterpret_cast<float2*>(dst + at[c]) = make_float2(g0, g1);
+      } else {
+        dst[at[c]] = g0;
+        if (two) dst[at[c + 1]] = g1;
       }
     }
   }
@@ -529,7 +668,7 @@ __global__ void __launch_bounds__(256) delta_chunk_prep_kernel(DeltaChunk d) {
     if (lane < 4) {
 #pragma unroll
       for (int v = 0; v < 2; ++v)
-        *reinterpret_cast<float2*>(blob + B::end + (c0 + 8 * v + kc) * 4) = make_float2(exp2f(end[v].x), exp2f(end[v].y));
+        *reinterpret_cast<float2*>(blob + B::end + (c0 + 8 * v + kc) * 4) = make_float2(exp2_flush(end[v].x), exp2_flush(end[v].y));
     }
     uint32_t hi, lo;
 #pragma unroll
@@ -542,10 +681,10 @@ __global__ void __launch_bounds__(256) delta_chunk_prep_kernel(DeltaChunk d) {
           *reinterpret_cast<uint32_t*>(blob + where + at) = hi;
           *reinterpret_cast<uint32_t*>(blob + where + B::tile + at) = lo;
         };
-        const float ex = exp2f(L[u][v].x), ey = exp2f(L[u][v].y);
+        const float ex = exp2_flush(L[u][v].x), ey = exp2_flush(L[u][v].y);
         put(B::kt, k[u][v].x * ex, k[u][v].y * ey);
         put(B::qt, q[u][v].x * ex, q[u][v].y * ey);
-        put(B::kc, k[u][v].x * exp2f(end[v].x - L[u][v].x), k[u][v].y * exp2f(end[v].y - L[u][v].y));
+        put(B::kc, k[u][v].x * exp2_flush(end[v].x - L[u][v].x), k[u][v].y * exp2_flush(end[v].y - L[u][v].y));
       }
     if (!__any_sync(0xffffffffu, unsafe)) {
       uint32_t kh[4], kl[4], qh[4], ql[4], sh[4], sl[4];     // [2 v + u]: A fragments; s: B fragments [2 v + token half]
@@ -554,10 +693,10 @@ __global__ void __launch_bounds__(256) delta_chunk_prep_kernel(DeltaChunk d) {
 #pragma unroll
         for (int v = 0; v < 2; ++v) {
           const float dx = L[u][v].x - ref[v].x, dy = L[u][v].y - ref[v].y;
-          const float ex = exp2f(dx), ey = exp2f(dy);
+          const float ex = exp2_flush(dx), ey = exp2_flush(dy);
           split_pack(k[u][v].x * ex, k[u][v].y * ey, kh[2 * v + u], kl[2 * v + u]);
           split_pack(q[u][v].x * ex, q[u][v].y * ey, qh[2 * v + u], ql[2 * v + u]);
-          split_pack(k[u][v].x * exp2f(-dx), k[u][v].y * exp2f(-dy), sh[2 * v + u], sl[2 * v + u]);
+          split_pack(k[u][v].x * exp2_flush(-dx), k[u][v].y * exp2_flush(-dy), sh[2 * v + u], sl[2 * v + u]);
         }
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
@@ -596,7 +735,7 @@ __global__ void __launch_bounds__(256) delta_chunk_prep_kernel(DeltaChunk d) {
             const float sl = __shfl_sync(0xffffffffu, lt[j], 4 * (kc + e) + src);
 #pragma unroll
             for (int u = 0; u < 2; ++u) {
-              const float x = sk * exp2f(fminf(rl[u] - sl, 0.f));          // pairs with s > t are dropped later
+              const float x = sk * exp2_flush(fminf(rl[u] - sl, 0.f));          // pairs with s > t are dropped later
               ca[j][2 * u + e] += rk[u] * x;
               cp[j][2 * u + e] += rq[u] * x;
             }
@@ -897,10 +1036,14 @@ XLLM_API int xllm_delta_rule(void* state, void* ring, const void* slots, const v
     }
     const auto al = [](const void* x, size_t a) { return (((uintptr_t)x) & (a - 1)) == 0; };
     const size_t va = 4 * sizeof(T);
-    const bool v4 = dk % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && al(q, va) && al(k, va) && al(v, va) && al(ring, va);
+    const bool v4 = dk % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && al(q, va) && al(k, va) && al(v, va) && al(ring, va) &&
+                    al(conv_w, va);
     const int64_t warps = (int64_t)(rows - row0) * (2 * G + H);
     const dim3 grid((unsigned)((warps + 7) / 8));
-    if (v4) launch_pdl(conv_heads_kernel<T, 4>, grid, dim3(256), 0, s, p);
+    if (v4 && taps <= 4 && dk <= 128 && dv <= 128) {
+      const int64_t runs = (int64_t)((rows - row0 + kConvRun - 1) / kConvRun) * (2 * G + H);
+      launch_pdl(conv_heads_run_kernel<T>, dim3((unsigned)((runs + 7) / 8)), dim3(256), 0, s, p);
+    } else if (v4) launch_pdl(conv_heads_kernel<T, 4>, grid, dim3(256), 0, s, p);
     else launch_pdl(conv_heads_kernel<T, 1>, grid, dim3(256), 0, s, p);
     if ((rc = XLLM_LAUNCH_CHECK()) != 0) return;
     if (taps > 1) {

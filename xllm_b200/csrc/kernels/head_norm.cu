@@ -4,7 +4,7 @@
 //   out[t, h dv + i] = a[t, h, i] * sigmoid(g[t, h dv + i])                                        head_gate
 //
 // every factor optional in the first (w: one weight per element shared by the heads, or one per head and element; act:
-// silu or sigmoid).  The heads of `a` may be stored wider than dv.  One warp per (token, head).
+// silu or sigmoid).  The heads of `a` may be stored wider than dv.  A warp owns whole heads.
 #include "vec_io.cuh"
 
 namespace xllm {
@@ -21,9 +21,62 @@ struct HeadNormParams {
   float eps;
 };
 
+template <typename T>
 __device__ __forceinline__ float gate_act(float z, int act) {
-  const float s = 1.f / (1.f + expf(-z));
+  const float s = sigmoid_as<T>(z);
   return act == 0 ? z * s : s;
+}
+
+// heads of up to 128 elements, four at a time: a warp owns U neighbouring items whose loads are all in flight together
+template <typename T, int U>
+__global__ void __launch_bounds__(256) head_norm_gate_small_kernel(HeadNormParams<T> p) {
+  const int lane = threadIdx.x & 31, c = lane * 4;
+  const int64_t first = ((int64_t)blockIdx.x * 8 + (threadIdx.x >> 5)) * U;
+  const bool on = c < p.dv;
+  pdl_wait();
+  pdl_launch_dependents();
+  float x[U][4], z[U][4], f[U];
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int64_t it = first + u;
+    f[u] = 1.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) x[u][j] = z[u][j] = 0.f;
+    if (it >= p.items) continue;
+    const unsigned t = (unsigned)it / (unsigned)p.H;         // fewer than 2^32 items
+    const int h = (int)((unsigned)it - t * p.H);
+    if (on) load_f32<4>(p.o + it * p.dv + c, x[u]);
+    if (on && p.g != nullptr) load_f32<4>(p.g + t * p.g_ld + (int64_t)h * p.dv + c, z[u]);
+    if (p.div != nullptr) f[u] = p.div[it];
+  }
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int64_t it = first + u;
+    if (it >= p.items) break;
+    const unsigned t = (unsigned)it / (unsigned)p.H;
+    const int h = (int)((unsigned)it - t * p.H);
+    const float s = f[u] > 0.f ? 1.f / f[u] : 0.f;               // rows of no sequence have no denominator
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      x[u][j] *= s;
+      ss += x[u][j] * x[u][j];
+    }
+    const float inv = p.unit_norm ? 1.f / sqrtf(warp_sum(ss) / (float)p.dv + p.eps) : 1.f;
+    if (!on) continue;
+    float w[4];
+    if (p.w != nullptr) {
+      load_f32<4>(p.w + (int64_t)h * p.w_head + c, w);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) x[u][j] *= w[j];
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      x[u][j] *= inv;
+      if (p.g != nullptr) x[u][j] *= gate_act<T>(z[u][j], p.act);
+    }
+    store_f32<4>(p.out + t * p.out_ld + (int64_t)h * p.dv + c, x[u]);
+  }
 }
 
 // V elements per lane and step; with V = 4 a head of up to 512 elements stays in registers
@@ -84,7 +137,7 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(HeadNormParams<T> p
       if (gr != nullptr) {
         load_f32<V>(gr + c, u);
 #pragma unroll
-        for (int j = 0; j < V; ++j) y[j] *= gate_act(u[j], p.act);
+        for (int j = 0; j < V; ++j) y[j] *= gate_act<T>(u[j], p.act);
       }
       store_f32<V>(dst + c, y);
     }
@@ -96,16 +149,15 @@ __global__ void __launch_bounds__(256) head_gate_kernel(T* __restrict__ out, con
                                                         int64_t g_ld, int64_t tokens, int H, int dv, int d_pad) {
   pdl_wait();
   pdl_launch_dependents();
-  const int per = dv / V;
-  const int64_t row = (int64_t)H * per, total = tokens * row;
-  for (int64_t n = blockIdx.x * (int64_t)256 + threadIdx.x; n < total; n += (int64_t)gridDim.x * 256) {
-    const int64_t t = n / row;
+  const int per = dv / V, row = H * per;
+  for (int64_t n = blockIdx.x * (int64_t)256 + threadIdx.x; n < tokens * row; n += (int64_t)gridDim.x * 256) {
+    const int64_t t = n < (1LL << 32) ? (unsigned)n / (unsigned)row : n / row;
     const int r = (int)(n - t * row), h = r / per, i = (r - h * per) * V;
     float x[V], z[V];
     load_f32<V>(a + (t * H + h) * d_pad + i, x);
     load_f32<V>(g + t * g_ld + (int64_t)h * dv + i, z);
 #pragma unroll
-    for (int j = 0; j < V; ++j) x[j] *= gate_act(z[j], 1);
+    for (int j = 0; j < V; ++j) x[j] *= gate_act<T>(z[j], 1);
     store_f32<V>(out + (t * H + h) * (int64_t)dv + i, x);
   }
 }
@@ -127,7 +179,10 @@ XLLM_API int xllm_head_norm_gate(void* out, int64_t out_ld, const void* o, const
     const size_t v = 4 * sizeof(T);
     const dim3 grid((unsigned)((p.items + 7) / 8)), block(256);
     if (dv % 4 == 0 && out_ld % 4 == 0 && (g == nullptr || g_ld % 4 == 0) && w_head % 4 == 0 && al(out, v) && al(o, 16) &&
-        al(g, v) && al(w, v))
+        al(g, v) && al(w, v) && dv <= 128 && p.items < (1LL << 32))
+      launch_pdl(head_norm_gate_small_kernel<T, 4>, dim3((unsigned)((p.items + 31) / 32)), block, 0, (cudaStream_t)stream, p);
+    else if (dv % 4 == 0 && out_ld % 4 == 0 && (g == nullptr || g_ld % 4 == 0) && w_head % 4 == 0 && al(out, v) && al(o, 16) &&
+             al(g, v) && al(w, v))
       launch_pdl(head_norm_gate_kernel<T, 4>, grid, block, 0, (cudaStream_t)stream, p);
     else
       launch_pdl(head_norm_gate_kernel<T, 1>, grid, block, 0, (cudaStream_t)stream, p);

@@ -53,7 +53,7 @@ constexpr float kDivEps = 1e-6f;
 // ------------------------------------------------------------------------------------------------ decode
 // grid (heads, sequences), 256 threads: dvp / 4 column groups x row groups, NR rows of four columns per thread.
 template <typename T, int NR>
-__global__ void __launch_bounds__(256) mlstm_decode_kernel(MlstmParams<T> p) {
+__global__ void __launch_bounds__(256, NR <= 8 ? 3 : (NR <= 16 ? 2 : 1)) mlstm_decode_kernel(MlstmParams<T> p) {
   extern __shared__ __align__(16) float sm[];
   const int dk = p.dk, dv = p.dv, dvp = p.dvp, dkp = (dk + 3) & ~3;
   float* qs = sm;

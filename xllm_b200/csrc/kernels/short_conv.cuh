@@ -8,26 +8,26 @@
 
 namespace xllm {
 
-__device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
 __device__ __forceinline__ float sigmoid_exact(float z) { return 1.f / (1.f + expf(-z)); }
 
 // V neighbouring channels of one token.  x: the channels' place in the token's projection row (row stride ld); `back`:
-// how many rows before it belong to the same sequence in this batch; ring: the channels' place in the slot's ring row 0
-// (row stride C); w: [channels, taps] at the first channel.
+// how many rows before it belong to the same sequence in this batch; ring, w: the channels' place in row 0 of the slot's
+// ring and of the weights [taps, C] (the last row belongs to the current token).
 template <typename T, int V>
 __device__ __forceinline__ void conv_silu(const T* x, int64_t ld, int back, int pos, const T* ring, int64_t C, const T* w,
                                           int taps, float* y) {
 #pragma unroll
   for (int j = 0; j < V; ++j) y[j] = 0.f;
   for (int d = 0; d < taps && d <= pos; ++d) {
-    float v[V];
+    float v[V], f[V];
     if (d <= back) load_f32<V>(x - d * ld, v);
     else load_f32<V>(ring + (int64_t)((pos - d) % taps) * C, v);
+    load_f32<V>(w + (int64_t)(taps - 1 - d) * C, f);
 #pragma unroll
-    for (int j = 0; j < V; ++j) y[j] += v[j] * to_f32(w[j * taps + taps - 1 - d]);
+    for (int j = 0; j < V; ++j) y[j] += v[j] * f[j];
   }
 #pragma unroll
-  for (int j = 0; j < V; ++j) y[j] = silu_exact(y[j]);
+  for (int j = 0; j < V; ++j) y[j] = silu_as<T>(y[j]);
 }
 
 // the sequence b with cu_q[b] <= row < cu_q[b + 1], or -1

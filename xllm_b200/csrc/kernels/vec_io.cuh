@@ -58,6 +58,16 @@ __device__ __forceinline__ void store_f32(float* p, const float* f) {
   }
 }
 
+// Sigmoid and silu of values whose results leave as T: hardware exponential and division (2^-21 relative) in front of a
+// rounding to bf16, the accurate ones for fp32.
+template <typename T>
+__device__ __forceinline__ float sigmoid_as(float z) {
+  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-z));
+  else return 1.f / (1.f + expf(-z));
+}
+template <typename T>
+__device__ __forceinline__ float silu_as(float z) { return z * sigmoid_as<T>(z); }
+
 __device__ __forceinline__ float to_f32(bf16 x) { return __bfloat162float(x); }
 __device__ __forceinline__ float to_f32(float x) { return x; }
 template <typename T>

@@ -244,10 +244,10 @@ class DeltaRuleMixer(Module):
             raise ValueError("the value heads must be a multiple of the query/key heads")
         op = self.op = ChannelDelta(heads, kv_heads, dk, dv, taps, q_scale=dk ** -0.5, eps=eps)
         self.parts = [("q", kv_heads * dk), ("k", kv_heads * dk), ("v", heads * dv), ("a1", decay_rank), ("g1", gate_rank)]
-        op.conv_w = self._params["conv"] = torch.zeros(op.channels, taps, dtype=dtype, device=device)
+        op.conv_w = self._params["conv"] = torch.zeros(taps, op.channels, dtype=dtype, device=device)
         at = 0
         for n, c in self.parts[:3]:
-            self._loaders[n + ".conv"] = lambda w, o=at, c=c: op.conv_w[o:o + c].copy_(w.reshape(c, taps).to(dtype))
+            self._loaders[n + ".conv"] = lambda w, o=at, c=c: op.conv_w[:, o:o + c].copy_(w.reshape(c, taps).T.to(dtype))
             at += c
         op.a2 = self.add_param("a2", torch.zeros(heads * dk, decay_rank, dtype=dtype, device=device))
         op.dt_bias = self.add_param("dt_bias", torch.zeros(heads * dk, dtype=dtype, device=device))

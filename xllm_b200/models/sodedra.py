@@ -168,7 +168,7 @@ class SodedraCausalLM(Module):
             if name.endswith("mix.norm"):
                 t.fill_(1.0)
             elif name.endswith(".conv"):
-                t[:, -1] += 1.0
+                t[-1] += 1.0
             elif name.endswith("dt_bias"):
                 t.fill_(-4.0)                               # decays near one
             elif name.endswith("small.bias"):

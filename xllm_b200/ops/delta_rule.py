@@ -34,7 +34,7 @@ class ChannelDelta:
     taps: int
     q_scale: float = 1.0
     eps: float = 1e-6
-    conv_w: Optional[torch.Tensor] = None        # [2 kv_heads dk + heads dv, taps]: q | k | v channels
+    conv_w: Optional[torch.Tensor] = None        # [taps, 2 kv_heads dk + heads dv], q | k | v channels; last row: this token's
     a2: Optional[torch.Tensor] = None            # [heads dk, rank]
     dt_bias: Optional[torch.Tensor] = None       # [heads dk]
     a_log: Optional[torch.Tensor] = None         # [heads]
@@ -104,7 +104,7 @@ class ChannelDelta:
     def _cpu(self, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out):
         H, G, dk, dv, taps = self.heads, self.kv_heads, self.dk, self.dv, self.taps
         x = torch.cat([q, k, v], dim=1)
-        w = self.conv_w.float()
+        w = self.conv_w.float().T.contiguous()
         share = torch.arange(H) // (H // G)
         for i in range(slots.shape[0]):
             b, e, slot = int(cu_q[i]), int(cu_q[i + 1]), int(slots[i])
