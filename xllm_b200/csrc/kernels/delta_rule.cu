@@ -8,9 +8,9 @@
 // weighted, and multiplied by the sigmoid of a gate.  The sibling of gdn.cu, whose decay is one number per head and
 // whose inputs are prepared by tensor operations.
 //
-//   delta_decode_kernel        one token per sequence, from the projection rows and the decays to the finished row; the
-//                              state crosses HBM once in each direction
-//   conv_heads_kernel          prompts: convolution, silu, unit norm of q and k -> fp32
+//   conv_heads_kernel          convolution, silu, unit norm of q and k -> fp32
+//   delta_decode_kernel        one token per sequence, from there to the finished row; the state crosses HBM once in each
+//                              direction
 //   conv_ring_kernel           prompts: the last inputs of every sequence -> its ring
 //   channel_decay_kernel       the decays, W_2 r on the tensor cores
 //   delta_chunk_prep_kernel,   prompts, bf16: sixteen tokens at a time on the tensor cores (below)
@@ -51,6 +51,7 @@ struct DeltaParams {
   float* o;                  // [rows, H, dv]
   int n_seqs, rows, row0, H, G, dk, dv, dkp, dvp, taps, rank;
   float q_scale, eps;
+  int write_ring;            // one row per sequence: its inputs go to the ring as they pass
   int log_decay;             // gn receives log2 of the decays (chunked prompts)
   __host__ __device__ int64_t channels() const { return (int64_t)2 * G * dk + (int64_t)H * dv; }
 };
@@ -82,8 +83,8 @@ __global__ void __launch_bounds__(256, NR <= 8 ? 3 : (NR <= 16 ? 2 : 1)) delta_d
   float* gs = ks + dkp;
   float* vs = gs + dkp;                    // [dvp]
   float* red = vs + dvp;                   // [RG][dvp]
-  __shared__ float red32[2][32];
-  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  __shared__ float red32[32];
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
   const int CG = dvp >> 2, RG = 256 / CG;
   const int cg = tid % CG, rg = tid / CG;
   pdl_wait();
@@ -95,80 +96,23 @@ __global__ void __launch_bounds__(256, NR <= 8 ? 3 : (NR <= 16 ? 2 : 1)) delta_d
     return;
   }
   const bool active = rg < RG, fresh = len == 1;
-  const int pos = len - 1, g = h / (p.H / p.G), G = p.G, taps = p.taps;
-  const int64_t C = p.channels();
-  T* ring = p.ring + (int64_t)slot * taps * C;
-  T* ring_now = ring + (int64_t)(pos % taps) * C;
-  const bool keeps_qk = h % (p.H / G) == 0;
-  // channels of this head in the order q | k | v; the loads of up to four taps go out before those of the state
-  constexpr int NE = 3;                    // 2 dk + dv <= 640
-  const auto channel = [&](int i, const T*& x) {
-    if (i < dk) { x = p.q + b * p.ld + (int64_t)g * dk + i; return (int64_t)g * dk + i; }
-    if (i < 2 * dk) { x = p.k + b * p.ld + (int64_t)g * dk + i - dk; return (int64_t)(G + g) * dk + i - dk; }
-    x = p.v + b * p.ld + (int64_t)h * dv + i - 2 * dk;
-    return (int64_t)2 * G * dk + (int64_t)h * dv + i - 2 * dk;
-  };
-  T xin[NE][4], win[NE][4];
-  if (taps <= 4) {
-#pragma unroll
-    for (int e = 0; e < NE; ++e) {
-      const int i = tid + 256 * e;
-#pragma unroll
-      for (int t = 0; t < 4; ++t) xin[e][t] = win[e][t] = from_f32<T>(0.f);
-      if (i >= 2 * dk + dv) continue;
-      const T* x;
-      const int64_t c = channel(i, x);
-      xin[e][0] = *x;
-#pragma unroll
-      for (int t = 0; t < 4; ++t) {
-        if (t < taps) win[e][t] = p.conv_w[(taps - 1 - t) * C + c];
-        if (t > 0 && t < taps && t <= pos) xin[e][t] = ring[(int64_t)((pos - t) % taps) * C + c];
-      }
-    }
-  }
   float* S = p.state + (((int64_t)slot * p.H + h) * dk) * dvp + cg * 4;
   float4 s[NR];
 #pragma unroll
   for (int u = 0; u < NR; ++u) {
     const int r = rg + u * RG;
-    s[u] = (active && !fresh && r < dk) ? *reinterpret_cast<const float4*>(S + (int64_t)r * dvp)
-                                        : make_float4(0.f, 0.f, 0.f, 0.f);
+    s[u] = (active && !fresh && r < dk) ? *reinterpret_cast<const float4*>(S + r * dvp) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
-  float sq = 0.f, sk = 0.f;
-#pragma unroll
-  for (int e = 0; e < NE; ++e) {
-    const int i = tid + 256 * e;
-    if (i >= 2 * dk + dv) continue;
-    const T* x;
-    const int64_t c = channel(i, x);
-    float y = 0.f;
-    if (taps <= 4) {
-#pragma unroll
-      for (int t = 0; t < 4; ++t) y += to_f32(xin[e][t]) * to_f32(win[e][t]);
-      y = silu_as<T>(y);
-    } else {
-      conv_silu<T, 1>(x, p.ld, 0, pos, ring + c, C, p.conv_w + c, taps, &y);
-    }
-    if (i < dk) { qs[i] = y; sq += y * y; }
-    else if (i < 2 * dk) { ks[i - dk] = y; sk += y * y; }
-    else vs[i - 2 * dk] = y;
-    if (taps > 1 && (keeps_qk || i >= 2 * dk)) ring_now[c] = *x;      // the token's own inputs go to its ring row
-  }
-  for (int i = dv + tid; i < dvp; i += 256) vs[i] = 0.f;
-  for (int i = tid; i < dk; i += 256) gs[i] = p.gn[((int64_t)b * p.H + h) * dkp + i];
-  sq = warp_sum(sq);
-  sk = warp_sum(sk);
-  if (lane == 0) { red32[0][warp] = sq; red32[1][warp] = sk; }
-  __syncthreads();
-  sq = sk = 0.f;
-#pragma unroll
-  for (int w = 0; w < 8; ++w) { sq += red32[0][w]; sk += red32[1][w]; }
-  const float iq = p.q_scale / sqrtf(sq + kUnitEps), ik = 1.f / sqrtf(sk + kUnitEps);
+  const int64_t qk = ((int64_t)b * p.G + h / (p.H / p.G)) * dkp, row = (int64_t)b * p.H + h;
   for (int i = tid; i < dk; i += 256) {
-    qs[i] *= iq;
-    ks[i] *= ik;
+    qs[i] = p.qn[qk + i];
+    ks[i] = p.kn[qk + i];
+    gs[i] = p.gn[row * dkp + i];
   }
+  for (int i = tid; i < dvp; i += 256) vs[i] = p.vn[row * dvp + i];
   const float beta = sigmoid_exact(p.zb[b * p.zb_ld + h]);
+  const float g_out = tid < dv ? to_f32(p.gate[b * p.gate_ld + (int64_t)h * dv + tid]) : 0.f;
+  const float w_out = tid < dv ? to_f32(p.norm_w[tid]) : 0.f;
   __syncthreads();
   float4 d = make_float4(0.f, 0.f, 0.f, 0.f);
   if (active) {
@@ -199,7 +143,7 @@ __global__ void __launch_bounds__(256, NR <= 8 ? 3 : (NR <= 16 ? 2 : 1)) delta_d
       const float kk = ks[r], qq = qs[r];
       float4 x = s[u];
       x.x += kk * w.x; x.y += kk * w.y; x.z += kk * w.z; x.w += kk * w.w;
-      *reinterpret_cast<float4*>(S + (int64_t)r * dvp) = x;
+      *reinterpret_cast<float4*>(S + r * dvp) = x;
       o.x += qq * x.x; o.y += qq * x.y; o.z += qq * x.z; o.w += qq * x.w;
     }
   }
@@ -211,10 +155,8 @@ __global__ void __launch_bounds__(256, NR <= 8 ? 3 : (NR <= 16 ? 2 : 1)) delta_d
     for (int w = 0; w < RG; ++w) mine += red[w * dvp + tid];
     ss = mine * mine;
   }
-  const float inv = 1.f / sqrtf(block_sum(ss, red32[0]) / (float)dv + p.eps);
-  if (tid < dv)
-    orow[tid] = from_f32<T>(mine * inv * to_f32(p.norm_w[tid]) *
-                            sigmoid_exact(to_f32(p.gate[b * p.gate_ld + (int64_t)h * dv + tid])));
+  const float inv = 1.f / sqrtf(block_sum(ss, red32) / (float)dv + p.eps);
+  if (tid < dv) orow[tid] = from_f32<T>(mine * inv * w_out * sigmoid_as<T>(g_out));
 }
 
 // ------------------------------------------------------------------------------------------------ prompts: inputs
@@ -250,6 +192,11 @@ __global__ void __launch_bounds__(256) conv_heads_kernel(DeltaParams<T> p) {
     for (int j = 0; j < V; ++j) y[i][j] = 0.f;
     if (c >= d) continue;
     conv_silu<T, V>(x + c, p.ld, back, pos, ring + c, C, w + c, p.taps, y[i]);
+    if (p.write_ring) {
+      T* now = p.ring + ((int64_t)p.slots[b] * p.taps + pos % p.taps) * C + c0 + c;
+#pragma unroll
+      for (int j = 0; j < V; ++j) now[j] = x[c + j];
+    }
 #pragma unroll
     for (int j = 0; j < V; ++j) ss += y[i][j] * y[i][j];
   }
@@ -267,15 +214,13 @@ __global__ void __launch_bounds__(256) conv_heads_kernel(DeltaParams<T> p) {
 
 // The same for up to four taps and heads of up to 128 channels: one warp per (run of rows, head), which reads every input
 // once and keeps the last ones in registers; a lane owns four neighbouring channels.
-constexpr int kConvRun = 8;
-
-template <typename T>
-__global__ void __launch_bounds__(256) conv_heads_run_kernel(DeltaParams<T> p) {
+template <typename T, int RUN>
+__global__ void __launch_bounds__(256, 4) conv_heads_run_kernel(DeltaParams<T> p) {
   const int lane = threadIdx.x & 31, items = 2 * p.G + p.H;
   const unsigned it = blockIdx.x * 8 + (threadIdx.x >> 5), run = it / items;
   pdl_wait();
   pdl_launch_dependents();
-  const int first = p.row0 + (int)run * kConvRun;
+  const int first = p.row0 + (int)run * RUN;
   if (first >= p.rows) return;
   int h = (int)(it - run * items);
   const int part = h < p.G ? 0 : (h < 2 * p.G ? 1 : 2);
@@ -286,9 +231,9 @@ __global__ void __launch_bounds__(256) conv_heads_run_kernel(DeltaParams<T> p) {
   float* dst = (part == 0 ? p.qn : (part == 1 ? p.kn : p.vn)) + (int64_t)h * d + c;
   const int64_t dst_ld = (int64_t)(part == 2 ? p.H : p.G) * d;      // d is a multiple of 4: no padding
   const bool on = c < d;
-  float v[kConvRun + 3][4], w[4][4];                                // w[taps back][channel]
+  float v[RUN + 3][4], w[4][4];                                // w[taps back][channel]
 #pragma unroll
-  for (int r = 0; r < kConvRun + 3; ++r) {
+  for (int r = 0; r < RUN + 3; ++r) {
     const int row = first + r - 3;
 #pragma unroll
     for (int j = 0; j < 4; ++j) v[r][j] = 0.f;
@@ -303,7 +248,7 @@ __global__ void __launch_bounds__(256) conv_heads_run_kernel(DeltaParams<T> p) {
   }
   int b = -1, begin = 0, end = 0;
 #pragma unroll
-  for (int r = 0; r < kConvRun; ++r) {
+  for (int r = 0; r < RUN; ++r) {
     const int row = first + r;
     if (row >= p.rows) break;
     if (row >= end) {                                               // the row starts another sequence, or is the first
@@ -323,14 +268,16 @@ __global__ void __launch_bounds__(256) conv_heads_run_kernel(DeltaParams<T> p) {
       if (back >= 3) y[j] += v[r][j] * w[3][j];
     }
     if (back < p.taps - 1) {                                        // inputs of earlier steps
-      const int pos = p.kv_lens[b] - (end - row);
+      const int pos = p.kv_lens[b] - (end - row), now = pos % p.taps;
       for (int t = back + 1; t < p.taps && t <= pos && on; ++t) {
         float z[4];
-        load_f32<4>(p.ring + ((int64_t)slot * p.taps + (pos - t) % p.taps) * C + c0, z);
+        load_f32<4>(p.ring + ((int64_t)slot * p.taps + now - t + (t > now ? p.taps : 0)) * C + c0, z);
 #pragma unroll
         for (int j = 0; j < 4; ++j) y[j] += z[j] * (t == 1 ? w[1][j] : (t == 2 ? w[2][j] : w[3][j]));
       }
     }
+    if (p.write_ring && on)
+      store_f32<4>(p.ring + ((int64_t)slot * p.taps + (p.kv_lens[b] - 1) % p.taps) * C + c0, v[r + 3]);
     float ss = 0.f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
@@ -338,7 +285,7 @@ __global__ void __launch_bounds__(256) conv_heads_run_kernel(DeltaParams<T> p) {
       ss += y[j] * y[j];
     }
     if (part < 2) {
-      const float f = (part == 0 ? p.q_scale : 1.f) / sqrtf(warp_sum(ss) + kUnitEps);
+      const float f = (part == 0 ? p.q_scale : 1.f) * rsqrtf(warp_sum(ss) + kUnitEps);
 #pragma unroll
       for (int j = 0; j < 4; ++j) y[j] *= f;
     }
@@ -992,9 +939,10 @@ XLLM_API int64_t xllm_delta_chunk_bytes(int rows, int n_seqs, int H, int dk) {
 // dtype: 0 bf16, 1 fp32 (projection rows, weights, ring, finished rows).
 //   state [slots, H, dk, dvp] fp32, dvp = dv rounded up to 4;  ring [slots, taps, 2 G dk + H dv]
 //   q, k, v, r: column blocks of rows with stride ld;  zb fp32 [rows, zb_ld]
-// gn [rows, H, dkp] fp32 is scratch (dkp = dk rounded up to 4, zeros behind dk).
-// mode 0: one token per sequence (sequence s is row s): gate, norm_w, out are used; dk <= 256, dv <= 128
-// mode 1: rows [row0, rows) by cu_q: qn, kn [rows, G, dkp], vn [rows, H, dvp] are scratch, the raw fp32 outputs go to o [rows, H, dv];  dk <= 512
+// qn, kn [rows, G, dkp], vn [rows, H, dvp], gn [rows, H, dkp] are fp32 scratch (dkp = dk rounded up to 4; gn comes with
+// zeros behind dk).
+// mode 0: one token per sequence (sequence s is row s, cu_q counts up by one): gate, norm_w, out are used; dk <= 256, dv <= 128
+// mode 1: rows [row0, rows) by cu_q, the raw fp32 outputs go to o [rows, H, dv];  dk <= 512
 // mode 2: the same in chunks of 16 tokens, no sequence longer than max_q_len rows; dk <= 256;
 //         blobs: scratch of xllm_delta_chunk_bytes(rows, n_seqs, H, dk) bytes
 XLLM_API int xllm_delta_rule(void* state, void* ring, const void* slots, const void* cu_q, const void* kv_lens, const void* q,
@@ -1022,7 +970,20 @@ XLLM_API int xllm_delta_rule(void* state, void* ring, const void* slots, const v
     p.n_seqs = n_seqs; p.rows = rows; p.row0 = row0; p.H = H; p.G = G; p.dk = dk; p.dv = dv; p.dkp = (dk + 3) & ~3;
     p.dvp = (dv + 3) & ~3; p.taps = taps; p.rank = rank; p.q_scale = q_scale; p.eps = eps;
     p.log_decay = mode == 2;
+    p.write_ring = mode == 0 && taps > 1;
     if ((rc = launch_channel_decay(p, s)) != 0) return;
+    const auto al = [](const void* x, size_t a) { return (((uintptr_t)x) & (a - 1)) == 0; };
+    const size_t va = 4 * sizeof(T);
+    const bool v4 = dk % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && al(q, va) && al(k, va) && al(v, va) && al(ring, va) &&
+                    al(conv_w, va);
+    const int run = v4 && taps <= 4 && dk <= 128 && dv <= 128 ? (mode == 0 ? 1 : 4) : 0;
+    const int64_t warps = (int64_t)(run > 0 ? (rows - row0 + run - 1) / run : rows - row0) * (2 * G + H);
+    const dim3 grid((unsigned)((warps + 7) / 8));
+    if (run == 1) launch_pdl(conv_heads_run_kernel<T, 1>, grid, dim3(256), 0, s, p);
+    else if (run > 1) launch_pdl(conv_heads_run_kernel<T, 4>, grid, dim3(256), 0, s, p);
+    else if (v4) launch_pdl(conv_heads_kernel<T, 4>, grid, dim3(256), 0, s, p);
+    else launch_pdl(conv_heads_kernel<T, 1>, grid, dim3(256), 0, s, p);
+    if ((rc = XLLM_LAUNCH_CHECK()) != 0) return;
     if (mode == 0) {
       const int RG = 256 / (p.dvp >> 2), nr = (dk + RG - 1) / RG;
       const size_t smem = (size_t)(3 * p.dkp + p.dvp + RG * p.dvp) * 4;
@@ -1034,18 +995,6 @@ XLLM_API int xllm_delta_rule(void* state, void* ring, const void* slots, const v
       rc = XLLM_LAUNCH_CHECK();
       return;
     }
-    const auto al = [](const void* x, size_t a) { return (((uintptr_t)x) & (a - 1)) == 0; };
-    const size_t va = 4 * sizeof(T);
-    const bool v4 = dk % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && al(q, va) && al(k, va) && al(v, va) && al(ring, va) &&
-                    al(conv_w, va);
-    const int64_t warps = (int64_t)(rows - row0) * (2 * G + H);
-    const dim3 grid((unsigned)((warps + 7) / 8));
-    if (v4 && taps <= 4 && dk <= 128 && dv <= 128) {
-      const int64_t runs = (int64_t)((rows - row0 + kConvRun - 1) / kConvRun) * (2 * G + H);
-      launch_pdl(conv_heads_run_kernel<T>, dim3((unsigned)((runs + 7) / 8)), dim3(256), 0, s, p);
-    } else if (v4) launch_pdl(conv_heads_kernel<T, 4>, grid, dim3(256), 0, s, p);
-    else launch_pdl(conv_heads_kernel<T, 1>, grid, dim3(256), 0, s, p);
-    if ((rc = XLLM_LAUNCH_CHECK()) != 0) return;
     if (taps > 1) {
       launch_pdl(conv_ring_kernel<T>, dim3((unsigned)((p.channels() + 255) / 256), n_seqs), dim3(256), 0, s, p);
       if ((rc = XLLM_LAUNCH_CHECK()) != 0) return;

@@ -127,7 +127,7 @@ __global__ void __launch_bounds__(256, NR <= 8 ? 3 : (NR <= 16 ? 2 : 1)) mlstm_d
   const float inv = 1.f / sqrtf(block_sum(ss, red32) / (float)dv + p.eps);
   if (tid < dv)
     orow[tid] = from_f32<T>(mine * inv * to_f32(p.norm_w[(int64_t)h * dv + tid]) *
-                            sigmoid_exact(to_f32(p.gate[b * p.gate_ld + (int64_t)h * dv + tid])));
+                            sigmoid_as<T>(to_f32(p.gate[b * p.gate_ld + (int64_t)h * dv + tid])));
 }
 
 // ------------------------------------------------------------------------------------------------ prompts

@@ -53,7 +53,7 @@ class ChannelDelta:
         assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (H, dk, round4(dv))
         assert ring.dtype == q.dtype and ring.is_contiguous() and ring.shape[1:] == (self.taps, self.channels)
         assert slots.dtype == torch.int32 and kv_lens.dtype == torch.int32 and zb.dtype == torch.float32 and zb.stride(1) == 1
-        qn, kn, vn, gn, o = scratch
+        qn, kn, vn, gn, o = (*scratch, None)[:5]
         check(_lib.load().xllm_delta_rule(
             ptr(state), ptr(ring), ptr(slots), ptr(cu_q), ptr(kv_lens), ptr(q), ptr(k), ptr(v), ptr(r), ld, ptr(zb), zb.stride(0),
             ptr(self.conv_w), ptr(self.a2), ptr(self.dt_bias), ptr(self.a_log), ptr(gate), gate.stride(0), ptr(self.norm_w),
@@ -61,11 +61,13 @@ class ChannelDelta:
             dk, dv, self.taps, self.a2.shape[1], self.q_scale, self.eps, _DT[q.dtype], mode, ptr(blobs), max_q_len, stream()),
             "delta_rule")
         from . import _count
-        _count(2 if mode == 0 else 2 + mode + int(self.taps > 1))
+        _count(3 if mode == 0 else 2 + mode + int(self.taps > 1))
 
-    def _decays(self, rows, device):
-        dkp = round4(self.dk)
-        return (torch.zeros if dkp != self.dk else torch.empty)((rows, self.heads, dkp), dtype=torch.float32, device=device)
+    def _scratch(self, rows, device):
+        """q, k, v behind the convolutions and the decays."""
+        H, G, dkp, f32 = self.heads, self.kv_heads, round4(self.dk), dict(dtype=torch.float32, device=device)
+        return (torch.empty((rows, G, dkp), **f32), torch.empty((rows, G, dkp), **f32), torch.empty((rows, H, round4(self.dv)), **f32),
+                (torch.zeros if dkp != self.dk else torch.empty)((rows, H, dkp), **f32))
 
     def decode(self, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out):
         """One token per sequence (sequence s is row s; cu_q [B + 1] counts up by one); `out` [B, heads * dv] is filled with
@@ -75,8 +77,7 @@ class ChannelDelta:
             return self.prefill(state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out, padded=True)
         if not q.is_cuda:
             return self._cpu(state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out)
-        scratch = (None, None, None, self._decays(B, q.device), None)
-        self._launch(0, state, ring, slots, None, kv_lens, q, k, v, r, zb, gate, out, scratch, B, 0)
+        self._launch(0, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out, self._scratch(B, q.device), B, 0)
         return out
 
     def prefill(self, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out, row0=0, padded=False,
@@ -86,15 +87,12 @@ class ChannelDelta:
         (default: all rows).  `token_by_token`: the fp32 recurrence instead of the chunked form."""
         if not q.is_cuda:
             return self._cpu(state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out)
-        T, H, G = q.shape[0], self.heads, self.kv_heads
-        f32 = dict(dtype=torch.float32, device=q.device)
-        dkp, dvp = round4(self.dk), round4(self.dv)
-        scratch = (torch.empty((T, G, dkp), **f32), torch.empty((T, G, dkp), **f32), torch.empty((T, H, dvp), **f32),
-                   self._decays(T, q.device),
-                   (torch.zeros if padded else torch.empty)((T, H, self.dv), **f32))
+        T = q.shape[0]
+        scratch = (*self._scratch(T, q.device), (torch.zeros if padded else torch.empty)((T, self.heads, self.dv),
+                                                                                         dtype=torch.float32, device=q.device))
         blobs, n = None, slots.shape[0]
         if q.dtype == torch.bfloat16 and self.dk <= 256 and not token_by_token:
-            blobs = torch.empty(_lib.load().xllm_delta_chunk_bytes(T, n, H, self.dk), dtype=torch.uint8, device=q.device)
+            blobs = torch.empty(_lib.load().xllm_delta_chunk_bytes(T, n, self.heads, self.dk), dtype=torch.uint8, device=q.device)
         self._launch(1 if blobs is None else 2, state, ring, slots, cu_q, kv_lens, q, k, v, r, zb, gate, out, scratch, T, row0,
                      blobs, int(max_q_len or T))
         head_norm_gate(scratch[4][row0:], out[row0:], g=gate[row0:], w=self.norm_w, act="sigmoid", eps=self.eps)
