@@ -449,20 +449,20 @@ def recurrent_rows(results, hbm, tf, tag):
     nq, nkv = 32, 8
     for S, L, win in ((4, 2048, 0), (4, 2048, 1024), (1, 8192, 0), (1, 8192, 1024)):
         T = S * L
-        kc = rows(T // 16 * nkv * 16, d).view(T // 16, nkv, 16, d)
+        kc, vc = (rows(T // 16 * nkv * 16, d).view(T // 16, nkv, 16, d) for _ in range(2))
         bt = torch.arange(T // 16, device=dev, dtype=torch.int32).view(S, L // 16)
         cu, kl, q = i32([i * L for i in range(S + 1)]), i32([L] * S), rows(T, nq * d).view(T, nq, d)
         pairs = sum(min(i + 1, win or L) for i in range(L)) * S
         report("attention prompts", f"{S} x {L} window {win}", bench_queued(lambda: ops.paged_prefill_attention(
-            q, kc, kc, bt, cu, kl, L, d ** -0.5, window=win), iters=5), T * d * 2 * (2 * nq + 2 * nkv), 4.0 * pairs * nq * d)
+            q, kc, vc, bt, cu, kl, L, d ** -0.5, window=win), iters=5), T * d * 2 * (2 * nq + 2 * nkv), 4.0 * pairs * nq * d)
     for B, ctx, win in ((64, 4096, 0), (64, 4096, 1024), (256, 1024, 0), (256, 4096, 1024)):
-        kc = rows(B * ctx // 16 * nkv * 16, d).view(B * ctx // 16, nkv, 16, d)
+        kc, vc = (rows(B * ctx // 16 * nkv * 16, d).view(B * ctx // 16, nkv, 16, d) for _ in range(2))
         bt = torch.arange(B * ctx // 16, device=dev, dtype=torch.int32).view(B, ctx // 16)
         kl, q = i32([ctx] * B), rows(B, nq * d).view(B, nq, d)
         splits = min(ops.decode_splits(B, nkv, nq // nkv), max(1, win // 256)) if win else None
         report("attention decode", f"B={B} ctx {ctx} window {win}", bench_queued(lambda: ops.paged_decode_attention(
-            q, kc, kc, bt, kl, d ** -0.5, window=win, splits=splits)), 4.0 * B * min(ctx, win or ctx) * nkv * d)
-        del kc
+            q, kc, vc, bt, kl, d ** -0.5, window=win, splits=splits)), 4.0 * B * min(ctx, win or ctx) * nkv * d)
+        del kc, vc
     for T in (64, 8192):
         x, y, y2, w = torch.randn(T, W, device=dev), rows(T, W), rows(T, W), torch.ones(W, device=dev, dtype=bf)
         report("residual_update, two branches", f"T={T}", bench_queued(
