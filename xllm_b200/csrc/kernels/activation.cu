@@ -1,4 +1,4 @@
-// Gated activations: out[t, :d] = act(x[t, :d]) * x[t, d:2d]   (bf16, fp32 math)
+// Gated activations: out[t, :d] = act(x[t, :d]) * x[t, d:2d], or clamped_glu of the two   (bf16, fp32 math)
 //
 // Parity: act_and_mul_kernel (silu/gelu/gelu_tanh) of the reference
 // (xllm/core/kernels/cuda/activation.cu:45-159).  Flat grid over 16-byte
@@ -17,7 +17,7 @@ __device__ __forceinline__ float act_gelu_tanh(float x) {
 template <int ACT>
 __global__ void __launch_bounds__(256)
 act_and_mul_kernel(bf16* __restrict__ out, const bf16* __restrict__ x, int64_t tokens, int d,
-                   int64_t x_stride, const int32_t* __restrict__ n_rows_dev) {
+                   int64_t x_stride, const int32_t* __restrict__ n_rows_dev, float limit, float alpha) {
   const int vec_per_row = d >> 3;
   pdl_wait();
   pdl_launch_dependents();  // dependents may be scheduled now; they block in their own pdl_wait()
@@ -35,8 +35,12 @@ act_and_mul_kernel(bf16* __restrict__ out, const bf16* __restrict__ x, int64_t t
     unpack8(row[v + vec_per_row], b);
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
-      float g = ACT == 0 ? act_silu(a[j]) : (ACT == 1 ? act_gelu(a[j]) : act_gelu_tanh(a[j]));
-      o[j] = g * b[j];
+      if constexpr (ACT == 3) {
+        o[j] = clamped_glu(a[j], b[j], limit, alpha);
+      } else {
+        float g = ACT == 0 ? act_silu(a[j]) : (ACT == 1 ? act_gelu(a[j]) : act_gelu_tanh(a[j]));
+        o[j] = g * b[j];
+      }
     }
     reinterpret_cast<bf16x8*>(out + t * (int64_t)d)[v] = pack8(o);
   }
@@ -47,7 +51,8 @@ act_and_mul_kernel(bf16* __restrict__ out, const bf16* __restrict__ x, int64_t t
 // activation in its epilogue, see xllm_gemm_bf16_act_mul).
 template <int ACT>
 __global__ void __launch_bounds__(256)
-act_and_mul_il_kernel(bf16* __restrict__ out, const bf16* __restrict__ x, int64_t tokens, int d, int64_t x_stride) {
+act_and_mul_il_kernel(bf16* __restrict__ out, const bf16* __restrict__ x, int64_t tokens, int d, int64_t x_stride, float limit,
+                      float alpha) {
   const int vec_per_row = d >> 3;
   pdl_wait();
   pdl_launch_dependents();
@@ -63,8 +68,12 @@ act_and_mul_il_kernel(bf16* __restrict__ out, const bf16* __restrict__ x, int64_
     unpack8(row[vin + 8], b);
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
-      float g = ACT == 0 ? act_silu(a[j]) : (ACT == 1 ? act_gelu(a[j]) : act_gelu_tanh(a[j]));
-      o[j] = g * b[j];
+      if constexpr (ACT == 3) {
+        o[j] = clamped_glu(a[j], b[j], limit, alpha);
+      } else {
+        float g = ACT == 0 ? act_silu(a[j]) : (ACT == 1 ? act_gelu(a[j]) : act_gelu_tanh(a[j]));
+        o[j] = g * b[j];
+      }
     }
     reinterpret_cast<bf16x8*>(out + t * (int64_t)d)[v] = pack8(o);
   }
@@ -72,9 +81,9 @@ act_and_mul_il_kernel(bf16* __restrict__ out, const bf16* __restrict__ x, int64_
 
 }  // namespace xllm
 
-// Interleaved layout (groups of 128 columns = 64 gate | 64 up); d % 64 == 0.
+// Interleaved layout (groups of 128 columns = 64 gate | 64 up); d % 64 == 0.  act: see xllm_act_and_mul.
 XLLM_API int xllm_act_and_mul_interleaved(void* out, const void* x, int64_t tokens, int d, int64_t x_stride, int act,
-                                          void* stream) {
+                                          float limit, float alpha, void* stream) {
   using namespace xllm;
   if (tokens == 0) return 0;
   if (d % 64 != 0) return (int)cudaErrorInvalidValue;
@@ -82,15 +91,20 @@ XLLM_API int xllm_act_and_mul_interleaved(void* out, const void* x, int64_t toke
   int grid = (int)((total + 255) / 256);
   if (grid > 148 * 16) grid = 148 * 16;
   cudaStream_t s = (cudaStream_t)stream;
-  if (act == 0) launch_pdl(act_and_mul_il_kernel<0>, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, tokens, d, x_stride);
-  else if (act == 1) launch_pdl(act_and_mul_il_kernel<1>, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, tokens, d, x_stride);
-  else launch_pdl(act_and_mul_il_kernel<2>, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, tokens, d, x_stride);
+  const auto run = [&](auto kernel) {
+    launch_pdl(kernel, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, tokens, d, x_stride, limit, alpha);
+  };
+  if (act == 0) run(act_and_mul_il_kernel<0>);
+  else if (act == 1) run(act_and_mul_il_kernel<1>);
+  else if (act == 2) run(act_and_mul_il_kernel<2>);
+  else run(act_and_mul_il_kernel<3>);
   return XLLM_LAUNCH_CHECK();
 }
 
-// act: 0 silu, 1 gelu(erf), 2 gelu(tanh).  x:[tokens, 2d] with row stride x_stride, out:[tokens, d].
+// act: 0 silu, 1 gelu(erf), 2 gelu(tanh), 3 clamped_glu with `limit` and `alpha`.  x:[tokens, 2d] with row stride x_stride,
+// out:[tokens, d].
 XLLM_API int xllm_act_and_mul(void* out, const void* x, int64_t tokens, int d, int64_t x_stride,
-                              int act, void* stream) {
+                              int act, float limit, float alpha, void* stream) {
   using namespace xllm;
   if (tokens == 0) return 0;
   if (d % 8 != 0) return (int)cudaErrorInvalidValue;
@@ -99,9 +113,13 @@ XLLM_API int xllm_act_and_mul(void* out, const void* x, int64_t tokens, int d, i
   if (grid > 148 * 16) grid = 148 * 16;
   cudaStream_t s = (cudaStream_t)stream;
   const int32_t* none = nullptr;
-  if (act == 0) launch_pdl(act_and_mul_kernel<0>, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, tokens, d, x_stride, none);
-  else if (act == 1) launch_pdl(act_and_mul_kernel<1>, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, tokens, d, x_stride, none);
-  else launch_pdl(act_and_mul_kernel<2>, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, tokens, d, x_stride, none);
+  const auto run = [&](auto kernel) {
+    launch_pdl(kernel, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, tokens, d, x_stride, none, limit, alpha);
+  };
+  if (act == 0) run(act_and_mul_kernel<0>);
+  else if (act == 1) run(act_and_mul_kernel<1>);
+  else if (act == 2) run(act_and_mul_kernel<2>);
+  else run(act_and_mul_kernel<3>);
   return XLLM_LAUNCH_CHECK();
 }
 
@@ -115,8 +133,8 @@ XLLM_API int xllm_act_and_mul_rows(void* out, const void* x, int64_t max_tokens,
   const int grid = 148 * 8;
   cudaStream_t s = (cudaStream_t)stream;
   const int32_t* nr = (const int32_t*)n_rows;
-  if (act == 0) launch_pdl(act_and_mul_kernel<0>, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, max_tokens, d, x_stride, nr);
-  else if (act == 1) launch_pdl(act_and_mul_kernel<1>, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, max_tokens, d, x_stride, nr);
-  else launch_pdl(act_and_mul_kernel<2>, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, max_tokens, d, x_stride, nr);
+  if (act == 0) launch_pdl(act_and_mul_kernel<0>, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, max_tokens, d, x_stride, nr, 0.f, 0.f);
+  else if (act == 1) launch_pdl(act_and_mul_kernel<1>, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, max_tokens, d, x_stride, nr, 0.f, 0.f);
+  else launch_pdl(act_and_mul_kernel<2>, dim3(grid), dim3(256), 0, s, (bf16*)out, (const bf16*)x, max_tokens, d, x_stride, nr, 0.f, 0.f);
   return XLLM_LAUNCH_CHECK();
 }

@@ -51,6 +51,19 @@ __device__ __forceinline__ void split_pack(float a, float b, uint32_t& hi, uint3
 }
 __device__ __forceinline__ float2 unpack2(uint32_t u) { return __bfloat1622float2(*reinterpret_cast<const bf162*>(&u)); }
 
+// Scores bounded by a soft cap, in the log2 domain: cap * log2(e) * tanh(s * scale / cap) = out - 2 out / (1 + 2^(s * in))
+// with in = 2 log2(e) scale / cap and out = cap log2(e).  The quotient leaves an error of a few 1e-7 of the cap.
+struct SoftCap {
+  float in, out;             // out 0: no cap
+};
+inline SoftCap make_soft_cap(float scale, float cap) {
+  const float log2e = 1.4426950408889634f;
+  return cap > 0.f ? SoftCap{2.f * log2e * scale / cap, cap * log2e} : SoftCap{0.f, 0.f};
+}
+__device__ __forceinline__ float soft_cap(float s, const SoftCap& c) {
+  return c.out - __fdividef(2.f * c.out, 1.f + exp2f(s * c.in));
+}
+
 // Byte offset of 16-byte chunk `c` of row `r` in a tile whose rows hold CH chunks; the XOR
 // swizzle makes 8 consecutive rows of one chunk column hit 8 different bank groups.
 template <int CH>

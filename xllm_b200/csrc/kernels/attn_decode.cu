@@ -33,6 +33,8 @@ struct DecodeParams {
   int64_t q_stride;            // elements between sequences in q
   int bt_stride, nq, nkv, group, page_size, splits;
   int window;                  // 0 = attend to the whole sequence
+  int keep;                    // with a window: the first `keep` positions stay visible
+  SoftCap cap;
   float scale_log2;
 };
 
@@ -55,10 +57,17 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(DecodeParams p) {
   // touched (their cache blocks may have been given back already)
   const int win_start = p.window > 0 ? max(0, seq_len - p.window) : 0;
   const int tile_first = win_start >> 4;
-  const int tiles_total = (seq_len + 15) >> 4;
-  const int tps = (tiles_total - tile_first + p.splits - 1) / p.splits;
-  const int t_begin = tile_first + split * tps;
+  const int kept = min((p.keep + 15) >> 4, tile_first);        // tiles of kept positions ahead of the window's
+  const int skip = tile_first - kept;                          // the walk goes over tiles 0 .. kept - 1, tile_first ..
+  const int tiles_total = ((seq_len + 15) >> 4) - skip;
+  const int tps = (tiles_total + p.splits - 1) / p.splits;
+  const int t_begin = split * tps;
   const int t_end = min(t_begin + tps, tiles_total);
+  const auto token_of = [&](int i) {                           // first token of this warp's i-th tile
+    const int t = t_begin + warp + 4 * i;
+    return (t < kept ? t : t + skip) << 4;
+  };
+  const auto hidden = [&](int tok) { return tok >= seq_len || (tok < win_start && tok >= p.keep); };
   const int my_n = (t_end - t_begin - warp + 3) >> 2;  // tiles of this warp (may be <= 0)
   const int rows_valid = min(16, p.group - qt * 16);
   const int head0 = kvh * p.group + qt * 16;
@@ -83,7 +92,7 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(DecodeParams p) {
 
   auto load_tile = [&](int i) {  // i-th tile of this warp -> stage i % STAGES
     if (i < my_n) {
-      const int tok0 = (t_begin + warp + 4 * i) << 4;
+      const int tok0 = token_of(i);
       const int page = tok0 / p.page_size;
       const int off = tok0 - page * p.page_size;
       const int64_t blk = bt[page];
@@ -96,7 +105,7 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(DecodeParams p) {
       for (int j = 0; j < (16 * CH) / 32; ++j) {
         const int id = lane + j * 32;
         const int r = id / CH, c = id - r * CH;
-        const bool valid = tok0 + r < seq_len && tok0 + r >= win_start;
+        const bool valid = !hidden(tok0 + r);
         const int64_t go = valid ? (int64_t)r * D + c * 8 : 0;
         cp_async16(ks + swz<CH>(r, c), kb + go, valid);
         cp_async16(vs + swz<CH>(r, c), vb + go, valid);
@@ -120,7 +129,7 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(DecodeParams p) {
     load_tile(i + STAGES - 1);
     const uint32_t ks_addr = ring + (i % STAGES) * STAGE_BYTES;
     const uint32_t vs_addr = ks_addr + TILE_BYTES;
-    const int tok0 = (t_begin + warp + 4 * i) << 4;
+    const int tok0 = token_of(i);
 
     float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
     {
@@ -140,8 +149,8 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(DecodeParams p) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int tok = tok0 + nt * 8 + (lane & 3) * 2 + (j & 1);
-        float v = s[nt][j] * p.scale_log2;
-        if (tok >= seq_len || tok < win_start) v = -INFINITY;
+        float v = p.cap.out > 0.f ? soft_cap(s[nt][j], p.cap) : s[nt][j] * p.scale_log2;
+        if (hidden(tok)) v = -INFINITY;
         s[nt][j] = v;
         if (j < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
       }
@@ -288,16 +297,17 @@ static int decode_attn_impl(void* out, const void* q, int64_t q_stride, const vo
                             const void* v_cache, const void* block_table, int bt_stride,
                             const void* seq_lens, int batch, int nq, int nkv, int d,
                             int page_size, float scale, int splits, void* workspace, int window,
-                            void* stream) {
+                            void* stream, int keep = 0, float softcap = 0.f) {
   using namespace xllm;
   if (batch == 0) return 0;
-  if (nq % nkv != 0 || page_size % 16 != 0 || splits < 1 || window < 0) return (int)cudaErrorInvalidValue;
+  if (nq % nkv != 0 || page_size % 16 != 0 || splits < 1 || window < 0 || keep < 0) return (int)cudaErrorInvalidValue;
   if (splits > 1 && workspace == nullptr) return (int)cudaErrorInvalidValue;
   DecodeParams p;
   p.q = (const bf16*)q; p.k_cache = (const bf16*)k_cache; p.v_cache = (const bf16*)v_cache;
   p.block_table = (const int32_t*)block_table; p.seq_lens = (const int32_t*)seq_lens;
   p.out = (bf16*)out; p.q_stride = q_stride; p.bt_stride = bt_stride; p.nq = nq; p.nkv = nkv;
   p.group = nq / nkv; p.page_size = page_size; p.splits = splits; p.window = window;
+  p.keep = window > 0 ? keep : 0; p.cap = make_soft_cap(scale, softcap);
   p.scale_log2 = scale * 1.4426950408889634f;
   p.o_part = (float*)workspace;
   p.lse_part = p.o_part ? p.o_part + (int64_t)batch * nq * splits * d : nullptr;
@@ -330,6 +340,16 @@ XLLM_API int xllm_paged_decode_attn_window(void* out, const void* q, int64_t q_s
                                            int window, void* stream) {
   return decode_attn_impl(out, q, q_stride, k_cache, v_cache, block_table, bt_stride, seq_lens, batch, nq, nkv, d,
                           page_size, scale, splits, workspace, window, stream);
+}
+
+// The same, with the first `keep` positions of every sequence visible beside the window (window > 0), and scores bounded
+// by softcap * tanh(score / softcap) (0: none).
+XLLM_API int xllm_paged_decode_attn_kept(void* out, const void* q, int64_t q_stride, const void* k_cache, const void* v_cache,
+                                         const void* block_table, int bt_stride, const void* seq_lens, int batch, int nq, int nkv,
+                                         int d, int page_size, float scale, int splits, void* workspace, int window, int keep,
+                                         float softcap, void* stream) {
+  return decode_attn_impl(out, q, q_stride, k_cache, v_cache, block_table, bt_stride, seq_lens, batch, nq, nkv, d,
+                          page_size, scale, splits, workspace, window, stream, keep, softcap);
 }
 
 // Standalone merge of `splits` normalised partials (also used by context-parallel decode).
@@ -407,7 +427,7 @@ XLLM_API int xllm_paged_decode_attn_noalloc(void* out, const void* q, int64_t q_
   p.q = (const bf16*)q; p.k_cache = (const bf16*)k_cache; p.v_cache = (const bf16*)v_cache;
   p.block_table = (const int32_t*)block_table; p.seq_lens = (const int32_t*)seq_lens;
   p.out = (bf16*)out; p.q_stride = q_stride; p.bt_stride = bt_stride; p.nq = nq; p.nkv = nkv;
-  p.group = nq / nkv; p.page_size = page_size; p.splits = splits; p.window = 0;
+  p.group = nq / nkv; p.page_size = page_size; p.splits = splits; p.window = 0; p.keep = 0; p.cap = make_soft_cap(scale, 0.f);
   p.scale_log2 = scale * 1.4426950408889634f;
   p.o_part = splits > 1 ? scratch : nullptr;
   p.lse_part = p.o_part ? p.o_part + (int64_t)batch * nq * splits * d : nullptr;

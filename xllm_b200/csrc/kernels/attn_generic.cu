@@ -1,5 +1,5 @@
 // Paged causal GQA attention for the cases the tensor-core kernels do not take: fp32 caches and head sizes
-// beyond 256.  Decode rows and prompt chunks alike: row r of sequence b sees the cache positions
+// beyond 256 (with a window the first `keep` positions may stay visible; scores may be bounded by a soft cap).  Decode rows and prompt chunks alike: row r of sequence b sees the cache positions
 // [0, kv_len_b - (rows of b after r)).  One CTA per (query row, head); each of its four warps walks every
 // fourth key with its lanes over the head dimension, keeps a running softmax, and the four are merged at the end.
 #include "vec_io.cuh"
@@ -16,8 +16,8 @@ struct GenericAttnParams {
   const int32_t* cu_q;     // [n_seqs + 1]
   const int32_t* kv_lens;
   int64_t q_ld, o_ld;
-  int bt_stride, n_seqs, nq, nkv, d, page, row0, window;
-  float scale;
+  int bt_stride, n_seqs, nq, nkv, d, page, row0, window, keep;
+  float scale, softcap;
 };
 
 template <typename T, int NPL>
@@ -37,6 +37,7 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(GenericAttnParams<T> 
   const int b = lo;
   const int len = p.kv_lens[b] - (p.cu_q[b + 1] - 1 - row);
   const int first = p.window > 0 ? max(0, len - p.window) : 0;
+  const int kept = min(p.keep, first), keys = kept + len - first;       // the walk: 0 .. kept - 1, then first .. len - 1
   const int g = h / (p.nq / p.nkv);
   const T* qr = p.q + (int64_t)row * p.q_ld + (int64_t)h * p.d;
   const int32_t* bt = p.block_table + (int64_t)b * p.bt_stride;
@@ -48,7 +49,8 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(GenericAttnParams<T> 
     o[i] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  for (int j = first + warp; j < len; j += 4) {
+  for (int n = warp; n < keys; n += 4) {
+    const int j = n < kept ? n : n - kept + first;
     const int pg = j / p.page;
     const int64_t base = (((int64_t)bt[pg] * p.nkv + g) * p.page + (j - pg * p.page)) * p.d;
     float s = 0.f;
@@ -58,6 +60,7 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(GenericAttnParams<T> 
       if (c < p.d) s += q[i] * to_f32(p.k_cache[base + c]);
     }
     s = warp_sum(s);
+    if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
     const float mn = fmaxf(m, s);
     const float keep = expf(m - mn), w = expf(s - mn);
     m = mn;
@@ -89,14 +92,14 @@ __global__ void __launch_bounds__(128) attn_generic_kernel(GenericAttnParams<T> 
 
 }  // namespace xllm
 
-// Rows [row0, row0 + rows) of q / out; dtype: 0 bf16, 1 fp32; d <= 512.
+// Rows [row0, row0 + rows) of q / out; dtype: 0 bf16, 1 fp32; d <= 1024.
 XLLM_API int xllm_paged_attn_generic(void* out, int64_t o_ld, const void* q, int64_t q_ld, const void* k_cache,
                                      const void* v_cache, const void* block_table, int bt_stride, const void* cu_q,
                                      const void* kv_lens, int n_seqs, int row0, int rows, int nq, int nkv, int d, int page,
-                                     float scale, int window, int dtype, void* stream) {
+                                     float scale, int window, int keep, float softcap, int dtype, void* stream) {
   using namespace xllm;
   if (rows == 0 || n_seqs == 0) return 0;
-  if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || d <= 0 || d > 512 || page <= 0) return (int)cudaErrorInvalidValue;
+  if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || d <= 0 || d > 1024 || page <= 0 || keep < 0) return (int)cudaErrorInvalidValue;
   cudaStream_t s = (cudaStream_t)stream;
   const auto run = [&](auto tag) {
     using T = decltype(tag);
@@ -105,11 +108,13 @@ XLLM_API int xllm_paged_attn_generic(void* out, int64_t o_ld, const void* q, int
     p.block_table = (const int32_t*)block_table; p.cu_q = (const int32_t*)cu_q; p.kv_lens = (const int32_t*)kv_lens;
     p.q_ld = q_ld; p.o_ld = o_ld; p.bt_stride = bt_stride; p.n_seqs = n_seqs; p.nq = nq; p.nkv = nkv; p.d = d;
     p.page = page; p.row0 = row0; p.window = window; p.scale = scale;
+    p.keep = window > 0 ? keep : 0; p.softcap = softcap;
     const dim3 grid(rows, nq);
     if (d <= 64) launch_pdl(attn_generic_kernel<T, 2>, grid, dim3(128), 0, s, p);
     else if (d <= 128) launch_pdl(attn_generic_kernel<T, 4>, grid, dim3(128), 0, s, p);
     else if (d <= 256) launch_pdl(attn_generic_kernel<T, 8>, grid, dim3(128), 0, s, p);
-    else launch_pdl(attn_generic_kernel<T, 16>, grid, dim3(128), 0, s, p);
+    else if (d <= 512) launch_pdl(attn_generic_kernel<T, 16>, grid, dim3(128), 0, s, p);
+    else launch_pdl(attn_generic_kernel<T, 32>, grid, dim3(128), 0, s, p);
   };
   if (dtype == 0) run(bf16());
   else run(float());

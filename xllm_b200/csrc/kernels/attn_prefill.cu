@@ -23,6 +23,8 @@ struct PrefillParams {
   int64_t q_stride;            // elements between tokens in q
   int64_t o_stride;
   int bt_stride, nq, nkv, page_size, causal, window;
+  int keep;                    // with a window: the first `keep` positions stay visible
+  SoftCap cap;
   float scale_log2;
 };
 
@@ -53,7 +55,9 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(PrefillParams p) {
   int kv_end = p.causal ? min(kv_len, shift + m0 + BM) : kv_len;
   int kv_begin = 0;
   if (p.window > 0) kv_begin = max(0, shift + m0 - p.window + 1) & ~(BN - 1);
-  const int n_tiles = (kv_end - kv_begin + BN - 1) / BN;
+  const int kept = min((p.keep + BN - 1) / BN, kv_begin / BN);   // tiles of kept positions ahead of the window's
+  const int n_tiles = kept + (kv_end - kv_begin + BN - 1) / BN;
+  const auto token_of = [&](int it) { return it < kept ? it * BN : kv_begin + (it - kept) * BN; };
   const int32_t* bt = p.block_table + (int64_t)b * p.bt_stride;
 
   // Q tile -> smem
@@ -68,7 +72,7 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(PrefillParams p) {
     }
   }
   auto load_kv = [&](int it) {
-    const int n0 = kv_begin + it * BN;
+    const int n0 = token_of(it);
     const uint32_t ks = sk + (it & 1) * KV_TILE, vs = sv + (it & 1) * KV_TILE;
 #pragma unroll
     for (int j = 0; j < (BN * CH) / 128; ++j) {
@@ -113,7 +117,7 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(PrefillParams p) {
         ldmatrix_x4(qa[ks][0], qa[ks][1], qa[ks][2], qa[ks][3], sq + swz<CH>(row, ks * 2 + cb));
     }
     const uint32_t ks_addr = sk + (it & 1) * KV_TILE, vs_addr = sv + (it & 1) * KV_TILE;
-    const int n0 = kv_begin + it * BN;
+    const int n0 = token_of(it);
 
     float s[BN / 8][4];
 #pragma unroll
@@ -139,10 +143,10 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(PrefillParams p) {
       for (int j = 0; j < 4; ++j) {
         const int tok = n0 + nt * 8 + (lane & 3) * 2 + (j & 1);
         const int qpos = j < 2 ? qpos0 : qpos1;
-        float v = s[nt][j] * p.scale_log2;
+        float v = p.cap.out > 0.f ? soft_cap(s[nt][j], p.cap) : s[nt][j] * p.scale_log2;
         bool masked = tok >= kv_len;
         if (p.causal) masked |= tok > qpos;
-        if (p.window > 0) masked |= tok <= qpos - p.window;
+        if (p.window > 0) masked |= tok <= qpos - p.window && tok >= p.keep;
         if (masked) v = -INFINITY;
         s[nt][j] = v;
         if (j < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
@@ -232,24 +236,35 @@ static int launch_prefill(const PrefillParams& p, int batch, int max_q_len, cuda
 // q/out: [T, nq, D] with q_stride / o_stride elements between tokens.  cu_q:[B+1], kv_lens:[B].
 // causal: query i of a sequence sees cache positions <= kv_len - q_len + i.  window > 0 adds a
 // sliding window of that many positions (including the current one).
-XLLM_API int xllm_paged_prefill_attn(void* out, int64_t o_stride, const void* q, int64_t q_stride,
-                                     const void* k_cache, const void* v_cache,
-                                     const void* block_table, int bt_stride, const void* cu_q,
-                                     const void* kv_lens, int batch, int max_q_len, int nq, int nkv,
-                                     int d, int page_size, float scale, int causal, int window,
-                                     void* stream) {
+// keep (with a window): the first positions of a sequence that stay visible; softcap (> 0) bounds the scores.
+XLLM_API int xllm_paged_prefill_attn_kept(void* out, int64_t o_stride, const void* q, int64_t q_stride,
+                                          const void* k_cache, const void* v_cache, const void* block_table, int bt_stride,
+                                          const void* cu_q, const void* kv_lens, int batch, int max_q_len, int nq, int nkv,
+                                          int d, int page_size, float scale, int causal, int window, int keep, float softcap,
+                                          void* stream) {
   using namespace xllm;
   if (batch == 0 || max_q_len == 0) return 0;
-  if (nq % nkv != 0) return (int)cudaErrorInvalidValue;
+  if (nq % nkv != 0 || keep < 0) return (int)cudaErrorInvalidValue;
   PrefillParams p;
   p.q = (const bf16*)q; p.out = (bf16*)out; p.k_cache = (const bf16*)k_cache;
   p.v_cache = (const bf16*)v_cache; p.block_table = (const int32_t*)block_table;
   p.cu_q = (const int32_t*)cu_q; p.kv_lens = (const int32_t*)kv_lens; p.q_stride = q_stride;
   p.o_stride = o_stride; p.bt_stride = bt_stride; p.nq = nq; p.nkv = nkv; p.page_size = page_size;
   p.causal = causal; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
+  p.keep = window > 0 ? keep : 0; p.cap = make_soft_cap(scale, softcap);
   cudaStream_t s = (cudaStream_t)stream;
   if (d == 128) return launch_prefill<128>(p, batch, max_q_len, s);
   if (d == 64) return launch_prefill<64>(p, batch, max_q_len, s);
   if (d == 256) return launch_prefill<256>(p, batch, max_q_len, s);
   return (int)cudaErrorInvalidValue;
+}
+
+XLLM_API int xllm_paged_prefill_attn(void* out, int64_t o_stride, const void* q, int64_t q_stride,
+                                     const void* k_cache, const void* v_cache,
+                                     const void* block_table, int bt_stride, const void* cu_q,
+                                     const void* kv_lens, int batch, int max_q_len, int nq, int nkv,
+                                     int d, int page_size, float scale, int causal, int window,
+                                     void* stream) {
+  return xllm_paged_prefill_attn_kept(out, o_stride, q, q_stride, k_cache, v_cache, block_table, bt_stride, cu_q, kv_lens,
+                                      batch, max_q_len, nq, nkv, d, page_size, scale, causal, window, 0, 0.f, stream);
 }

@@ -19,7 +19,7 @@
 //
 // Every mbarrier wait is bounded; on expiry all roles leave, TMEM is released and an error word
 // is set (xllm_fmha_error_status).
-#include "common.cuh"
+#include "attn_common.cuh"
 #include <cuda.h>
 
 namespace xllm {
@@ -141,11 +141,15 @@ struct Params {
   int64_t o_stride;
   int bt_stride, nq, nkv, page, causal;
   int window;                  // > 0: a query sees its last `window` positions only
+  int keep;                    // ... and the first `keep`
+  int rows_kv;                 // K and V are rows of all heads (page n: rows n * page ..), not one tile per page and head
+  SoftCap cap;
   float scale_log2;
   int* err;
   float* lse;                  // optional [total_q, nq]: log2-domain log-sum-exp of every row's scaled scores
 };
 
+template <bool CAP>
 __global__ void __launch_bounds__(320, 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                   const __grid_constant__ CUtensorMap tma_v, const Params p) {
@@ -180,7 +184,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
   const int ctx_off = kv_len - q_len;                 // absolute position of this chunk's first query
   const int kv_hi = p.causal ? min(kv_len, ctx_off + m0 + kBM) : kv_len;
   const int first = p.window > 0 ? max(0, ctx_off + m0 - p.window + 1) / kBN : 0;   // tiles before every row's window
-  const int n_tiles = (kv_hi + kBN - 1) / kBN - first;
+  const int kept = min((p.keep + kBN - 1) / kBN, first);                             // tiles of kept positions ahead of it
+  const int n_tiles = kept + (kv_hi + kBN - 1) / kBN - first;
+  const auto tile_of = [&](int j) { return j < kept ? j : j - kept + first; };
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -221,9 +227,10 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
       const int st = j & 1;
-      const int pg = (first + j) * pages + lane;
+      const int pg = tile_of(j) * pages + lane;
       const int myblk = (lane < pages && pg < n_blk) ? bt[pg] : 0;   // pages past the sequence read block 0 (masked)
-      const int y = (myblk * p.nkv + hk) * p.page;
+      const int y = p.rows_kv ? myblk * p.page : (myblk * p.nkv + hk) * p.page;
+      const int x = p.rows_kv ? hk * kD : 0;
       const uint32_t off = (uint32_t)(lane * p.page * 128);
       const uint32_t kdst = sbase + KV_OFF + st * 2 * kTile, vdst = kdst + kTile;
       // every lane gathers its own page: the copies of all pages issue together
@@ -231,15 +238,15 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       if (lane == 0) mbar_expect_tx(k_full(st), kTile);
       __syncwarp();
       if (lane < pages) {
-        tma_load_2d(kdst + off, &tma_k, 0, y, k_full(st));
-        tma_load_2d(kdst + kHalf + off, &tma_k, 64, y, k_full(st));
+        tma_load_2d(kdst + off, &tma_k, x, y, k_full(st));
+        tma_load_2d(kdst + kHalf + off, &tma_k, x + 64, y, k_full(st));
       }
       if (!mbar_wait_warp(v_empty(st), ((j >> 1) & 1) ^ 1, abort_flag)) { ok = false; break; }
       if (lane == 0) mbar_expect_tx(v_full(st), kTile);
       __syncwarp();
       if (lane < pages) {
-        tma_load_2d(vdst + off, &tma_v, 0, y, v_full(st));
-        tma_load_2d(vdst + kHalf + off, &tma_v, 64, y, v_full(st));
+        tma_load_2d(vdst + off, &tma_v, x, y, v_full(st));
+        tma_load_2d(vdst + kHalf + off, &tma_v, x + 64, y, v_full(st));
       }
       __syncwarp();
     }
@@ -315,6 +322,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
     // maximum has grown by more than 2^kLag, so after the first tiles the rescale is rare and the
     // common tile costs no pass over O at all.  P stays below 2^kLag, well inside bf16 and fp32 range.
     constexpr float kLag = 8.f;
+    const float sc = CAP ? 1.f : p.scale_log2;        // capped scores are in the log2 domain already
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     const uint32_t oaddr = TO0 + half * 64 + lane_addr;
@@ -325,8 +333,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       ok = ok && mbar_wait(s_full(sb), (j >> 1) & 1, abort_flag);
       tc_fence_after();
       const uint32_t saddr = TS0 + sb * 128 + half * 64 + lane_addr;
-      const int kv0 = (first + j) * kBN + half * 64;
-      const bool full_tile = kv0 + 63 <= limit && kv0 >= low;
+      const int kv0 = tile_of(j) * kBN + half * 64;
+      const bool full_tile = kv0 + 63 <= limit && (kv0 >= low || kv0 + 63 < p.keep);
+      const auto shown = [&](int t) { return t <= limit && (t >= low || t < p.keep); };
       uint32_t sv[64];
       tmem_ld32(saddr, sv);
       tmem_ld32(saddr + 32, sv + 32);
@@ -334,14 +343,18 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(s_free(sb));         // S has been read out: the next QK may overwrite it
+      if constexpr (CAP) {
+#pragma unroll
+        for (int i = 0; i < 64; ++i) sv[i] = __float_as_uint(soft_cap(__uint_as_float(sv[i]), p.cap));
+      }
       float mx = -INFINITY;
 #pragma unroll
       for (int i = 0; i < 64; ++i)
-        if (full_tile || (kv0 + i <= limit && kv0 + i >= low)) mx = fmaxf(mx, __uint_as_float(sv[i]));
+        if (full_tile || shown(kv0 + i)) mx = fmaxf(mx, __uint_as_float(sv[i]));
       smax[(sb * 2 + half) * kBM + row] = mx;
       asm volatile("bar.sync 1, 256;" ::: "memory");
       mx = fmaxf(mx, smax[(sb * 2 + (half ^ 1)) * kBM + row]);
-      const float m_true = fmaxf(m, mx * p.scale_log2);
+      const float m_true = fmaxf(m, mx * sc);
       float factor = 1.f;
       if (m_true - m > kLag) {                        // also the first tile that shows this row a key (m = -inf)
         factor = exp2f(m - m_true);                   // 0 when m was -inf: nothing accumulated yet
@@ -372,11 +385,11 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
 #pragma unroll
         for (int e = 0; e < 8; e += 2) {
           const int i = u * 8 + e;
-          float p0 = exp2f(__uint_as_float(sv[i]) * p.scale_log2 - m_use);
-          float p1 = exp2f(__uint_as_float(sv[i + 1]) * p.scale_log2 - m_use);
+          float p0 = exp2f(__uint_as_float(sv[i]) * sc - m_use);
+          float p1 = exp2f(__uint_as_float(sv[i + 1]) * sc - m_use);
           if (!full_tile) {
-            if (kv0 + i > limit || kv0 + i < low) p0 = 0.f;
-            if (kv0 + i + 1 > limit || kv0 + i + 1 < low) p1 = 0.f;
+            if (!shown(kv0 + i)) p0 = 0.f;
+            if (!shown(kv0 + i + 1)) p1 = 0.f;
           }
           rs += p0 + p1;
           const __nv_bfloat162 pb = __floats2bfloat162_rn(p0, p1);
@@ -482,22 +495,23 @@ static int* g_err[64] = {};
 // [n_blocks, nkv, page, 128], cu_q absolute row offsets [batch + 1], kv_lens [batch].
 // `lse` (optional, fp32 [total_q, nq]) receives every row's log-sum-exp in the log2 domain, so that the
 // result can be merged with attention over other keys (xllm_attn_merge, the beam-tail kernel).
-XLLM_API int xllm_paged_prefill_attn_tc_lse(void* out, int64_t o_stride, const void* q, int64_t q_stride, int64_t total_q,
-                                            const void* k_cache, const void* v_cache, int64_t n_blocks,
-                                            const void* block_table, int bt_stride, const void* cu_q,
-                                            const void* kv_lens, int batch, int max_q_len, int nq, int nkv,
-                                            int page_size, float scale, int causal, int window, void* lse, void* stream) {
+static int prefill_tc(void* out, int64_t o_stride, const void* q, int64_t q_stride, int64_t total_q, const void* k_cache,
+                      const void* v_cache, int64_t n_blocks, int64_t kv_ld, const void* block_table, int bt_stride,
+                      const void* cu_q, const void* kv_lens, int batch, int max_q_len, int nq, int nkv, int page_size,
+                      float scale, int causal, int window, int keep, float softcap, void* lse, void* stream) {
   using namespace xllm;
   using namespace xllm::fmha;
   if (batch == 0 || max_q_len == 0) return 0;
   if (nq % nkv != 0 || (page_size != 16 && page_size != 32 && page_size != 64 && page_size != 128) || q_stride % 8 ||
-      o_stride % 8 || (((uintptr_t)q | (uintptr_t)out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15))
+      o_stride % 8 || keep < 0 || kv_ld % 8 || (((uintptr_t)q | (uintptr_t)out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15))
     return (int)cudaErrorInvalidValue;
   int dev = 0;
   cudaGetDevice(&dev);
   static bool attr_done[64] = {};
   if (!attr_done[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
+    cudaError_t e = cudaFuncSetAttribute(prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
+    if (e == cudaSuccess)
+      e = cudaFuncSetAttribute(prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
     if (e != cudaSuccess) return (int)e;
     attr_done[dev & 63] = true;
   }
@@ -506,18 +520,40 @@ XLLM_API int xllm_paged_prefill_attn_tc_lse(void* out, int64_t o_stride, const v
     cudaMemset(g_err[dev & 63], 0, sizeof(int));
   }
   CUtensorMap tq, tk, tv;
-  const int64_t cache_rows = n_blocks * nkv * page_size;
-  if (!make_map(&tq, q, total_q, (int64_t)nq * kD, q_stride, kBM) || !make_map(&tk, k_cache, cache_rows, kD, kD, page_size) ||
-      !make_map(&tv, v_cache, cache_rows, kD, kD, page_size))
+  const int64_t cache_rows = kv_ld > 0 ? n_blocks * page_size : n_blocks * nkv * page_size;
+  const int64_t cols = kv_ld > 0 ? (int64_t)nkv * kD : kD, ld = kv_ld > 0 ? kv_ld : kD;
+  if (!make_map(&tq, q, total_q, (int64_t)nq * kD, q_stride, kBM) || !make_map(&tk, k_cache, cache_rows, cols, ld, page_size) ||
+      !make_map(&tv, v_cache, cache_rows, cols, ld, page_size))
     return (int)cudaErrorInvalidValue;
   Params p;
   p.out = (bf16*)out; p.block_table = (const int32_t*)block_table; p.cu_q = (const int32_t*)cu_q;
   p.kv_lens = (const int32_t*)kv_lens; p.o_stride = o_stride; p.bt_stride = bt_stride; p.nq = nq; p.nkv = nkv;
   p.page = page_size; p.causal = causal; p.window = window; p.scale_log2 = scale * 1.4426950408889634f; p.err = g_err[dev & 63];
-  p.lse = (float*)lse;
+  p.lse = (float*)lse; p.keep = window > 0 ? keep : 0; p.rows_kv = kv_ld > 0; p.cap = make_soft_cap(scale, softcap);
   dim3 grid((max_q_len + kBM - 1) / kBM, nq, batch);
-  prefill_tc_kernel<<<grid, 320, SMEM_TOTAL, (cudaStream_t)stream>>>(tq, tk, tv, p);
+  if (softcap > 0.f) prefill_tc_kernel<true><<<grid, 320, SMEM_TOTAL, (cudaStream_t)stream>>>(tq, tk, tv, p);
+  else prefill_tc_kernel<false><<<grid, 320, SMEM_TOTAL, (cudaStream_t)stream>>>(tq, tk, tv, p);
   return XLLM_LAUNCH_CHECK();
+}
+
+XLLM_API int xllm_paged_prefill_attn_tc_lse(void* out, int64_t o_stride, const void* q, int64_t q_stride, int64_t total_q,
+                                            const void* k_cache, const void* v_cache, int64_t n_blocks,
+                                            const void* block_table, int bt_stride, const void* cu_q,
+                                            const void* kv_lens, int batch, int max_q_len, int nq, int nkv,
+                                            int page_size, float scale, int causal, int window, void* lse, void* stream) {
+  return prefill_tc(out, o_stride, q, q_stride, total_q, k_cache, v_cache, n_blocks, 0, block_table, bt_stride, cu_q, kv_lens,
+                    batch, max_q_len, nq, nkv, page_size, scale, causal, window, 0, 0.f, lse, stream);
+}
+
+// The same with kept first positions beside the window and soft-capped scores (see xllm_paged_prefill_attn_kept).
+// kv_ld > 0: K and V are matrices [n_blocks * page_size, nkv * 128] of that row stride, a page being page_size rows.
+XLLM_API int xllm_paged_prefill_attn_tc_kept(void* out, int64_t o_stride, const void* q, int64_t q_stride, int64_t total_q,
+                                             const void* k_cache, const void* v_cache, int64_t n_blocks, int64_t kv_ld,
+                                             const void* block_table, int bt_stride, const void* cu_q, const void* kv_lens,
+                                             int batch, int max_q_len, int nq, int nkv, int page_size, float scale, int causal,
+                                             int window, int keep, float softcap, void* stream) {
+  return prefill_tc(out, o_stride, q, q_stride, total_q, k_cache, v_cache, n_blocks, kv_ld, block_table, bt_stride, cu_q,
+                    kv_lens, batch, max_q_len, nq, nkv, page_size, scale, causal, window, keep, softcap, nullptr, stream);
 }
 
 XLLM_API int xllm_paged_prefill_attn_tc(void* out, int64_t o_stride, const void* q, int64_t q_stride, int64_t total_q,

@@ -76,6 +76,12 @@ __device__ __forceinline__ bf16x8 pack8(const float* f) {
   return p;
 }
 
+// Gated activation with both factors clamped: g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = up within +-limit.
+__device__ __forceinline__ float clamped_glu(float gate, float up, float limit, float alpha) {
+  const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+  return g / (1.f + __expf(-alpha * g)) * (u + 1.f);
+}
+
 __device__ __forceinline__ uint32_t smem_u32(const void* p) {
   return (uint32_t)__cvta_generic_to_shared(p);
 }

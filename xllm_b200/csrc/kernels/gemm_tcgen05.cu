@@ -143,8 +143,9 @@ struct GemmMode {
   int push_S, push_rank, push_world;
   // Gated-activation epilogue: the weight rows are interleaved in groups of 128 output columns =
   // [gate of 64 features | up of the same 64 features]; the epilogue writes act(gate) * up, 64 columns per
-  // group, into an output of N / 2 columns.  0 = off, 1 = SiLU, 2 = GELU(erf), 3 = GELU(tanh).
+  // group, into an output of N / 2 columns.  0 = off, 1 = SiLU, 2 = GELU(erf), 3 = GELU(tanh), 4 = clamped_glu.
   int act_mul;
+  float act_limit, act_alpha;
 };
 __device__ __forceinline__ void umma_commit(uint32_t bar) {
   asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar)
@@ -241,11 +242,16 @@ __device__ __forceinline__ void epilogue_slice(uint32_t taddr, const CUtensorMap
             // gate and up are rounded to bf16 first, as the two-launch form stores them: a request's tokens
             // must not depend on which of the two forms its batch size selects
             const float x = __bfloat162float(__float2bfloat16(__uint_as_float(g[j * 8 + e])));
+            const float y = __bfloat162float(__float2bfloat16(__uint_as_float(u[j * 8 + e])));
+            if (mode.act_mul == 4) {
+              f[e] = clamped_glu(x, y, mode.act_limit, mode.act_alpha);
+              continue;
+            }
             float a;
             if (mode.act_mul == 1) a = x / (1.f + __expf(-x));
             else if (mode.act_mul == 2) a = 0.5f * x * (1.f + erff(x * 0.70710678f));
             else a = 0.5f * x * (1.f + tanhf(0.7978845608f * (x + 0.044715f * x * x * x)));
-            f[e] = a * __bfloat162float(__float2bfloat16(__uint_as_float(u[j * 8 + e])));
+            f[e] = a * y;
           }
           const bf16x8 v = pack8(f);
           const uint4 w4 = *reinterpret_cast<const uint4*>(&v);
@@ -980,7 +986,7 @@ gemm_bf16_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap tma_a, const _
       }
       if (ks == 1) {
         GemmMode pm{nullptr, nullptr, 0, 0, 0, 1, nullptr, nullptr, nullptr, 0, nullptr, nullptr, 0, 0, 0, 0, 0};
-        pm.act_mul = mode.act_mul;
+        pm.act_mul = mode.act_mul; pm.act_limit = mode.act_limit; pm.act_alpha = mode.act_alpha;
         epilogue_slice<BN>(taddr, &tma_c, sbase + S::EPI_OFF + q * 2 * kEpiBufBytes, m0 + q * 32, n0, bias, N, lane, ebuf,
                            pm, 0, taddr2);
       } else {
@@ -1150,7 +1156,7 @@ static int launch_gemm(const void* a, const void* w, void* c, const void* bias, 
 template <int BN, int STAGES, int KS = 1, bool DUAL = false>
 static int launch_gemm_pair(const void* a, const void* w, void* c, const void* bias, int M, int N, int K, int64_t lda,
                             int64_t ldw, int64_t ldc, int max_ctas, int w_packed, cudaStream_t s, int split_k = 1,
-                            int act_mul = 0) {
+                            int act_mul = 0, float act_limit = 0.f, float act_alpha = 0.f) {
   using S = GemmSmem2<BN, STAGES, KS>;
   int dev = 0;
   cudaGetDevice(&dev);
@@ -1172,7 +1178,7 @@ static int launch_gemm_pair(const void* a, const void* w, void* c, const void* b
     return (int)cudaErrorInvalidValue;
   const int tiles = ((M + 2 * kBM - 1) / (2 * kBM)) * ((N + BN - 1) / BN);
   GemmMode mode{nullptr, nullptr, 0, 0, 0, 1, nullptr, nullptr, nullptr, 0, nullptr, nullptr, 0, 0, 0, 0, 0};
-  mode.act_mul = act_mul;
+  mode.act_mul = act_mul; mode.act_limit = act_limit; mode.act_alpha = act_alpha;
   if (act_mul) split_k = 1;
   if (split_k > 1) {
     mode.ks = usable_split(split_k, M, N, K, KS, 2 * tiles, dev, s);
@@ -1193,14 +1199,15 @@ static int launch_gemm_pair(const void* a, const void* w, void* c, const void* b
 // C[M, N / 2] = act(A W_gate^T) * (A W_up^T) in one launch.  W [N, K] holds the fused gate|up projection with its
 // rows interleaved in groups of 128 = [64 gate rows | the 64 up rows of the same features] (N % 256 == 0); the
 // 256-wide tiles of the CTA-pair kernel then hold both halves of 128 features and the epilogue applies the gated
-// activation on the fp32 accumulators before anything is written.  act: 1 SiLU, 2 GELU(erf), 3 GELU(tanh).
+// activation on the fp32 accumulators before anything is written.  act: 1 SiLU, 2 GELU(erf), 3 GELU(tanh),
+// 4 clamped_glu with `limit` and `alpha`.
 XLLM_API int xllm_gemm_bf16_act_mul(const void* a, const void* w, void* c, int M, int N, int K, int64_t lda, int64_t ldw,
-                                    int64_t ldc, int act, void* stream) {
+                                    int64_t ldc, int act, float limit, float alpha, void* stream) {
   using namespace xllm;
   if (M == 0 || N == 0) return 0;
-  if (K % 8 || N % 256 || lda % 8 || ldw % 8 || ldc % 8 || act < 1 || act > 3) return (int)cudaErrorInvalidValue;
+  if (K % 8 || N % 256 || lda % 8 || ldw % 8 || ldc % 8 || act < 1 || act > 4) return (int)cudaErrorInvalidValue;
   if (((uintptr_t)a | (uintptr_t)w | (uintptr_t)c) & 15) return (int)cudaErrorInvalidValue;
-  return launch_gemm_pair<256, 6>(a, w, c, nullptr, M, N, K, lda, ldw, ldc, 148, 0, (cudaStream_t)stream, 1, act);
+  return launch_gemm_pair<256, 6>(a, w, c, nullptr, M, N, K, lda, ldw, ldc, 148, 0, (cudaStream_t)stream, 1, act, limit, alpha);
 }
 
 // ===================================================================================== block-scaled fp8
@@ -1651,15 +1658,17 @@ XLLM_API int xllm_gemm_bf16_grouped(const void* a, const void* w, void* c, const
 // xllm_gemm_bf16_act_mul; C is [M, N / 2] = act(gate) * up, and the [M, N] intermediate is never written.
 XLLM_API int xllm_gemm_bf16_grouped_act_mul(const void* a, const void* w, void* c, const void* tile_expert, int M,
                                             int N, int K, int n_experts, int64_t lda, int64_t ldc, int act,
-                                            void* stream) {
+                                            float limit, float alpha, void* stream) {
   using namespace xllm;
   if (M == 0 || N == 0) return 0;
-  if (K % 8 || N % 128 || lda % 8 || ldc % 8 || M % kBM || act < 1 || act > 3) return (int)cudaErrorInvalidValue;
+  if (K % 8 || N % 128 || lda % 8 || ldc % 8 || M % kBM || act < 1 || act > 4) return (int)cudaErrorInvalidValue;
   cudaStream_t s = (cudaStream_t)stream;
   const int32_t* te = (const int32_t*)tile_expert;
   GemmMode mode{};
   mode.ks = 1;
   mode.act_mul = act;
+  mode.act_limit = limit;
+  mode.act_alpha = alpha;
   if (N % 256 == 0) return launch_gemm<256, 4>(a, w, c, nullptr, M, N, K, lda, K, ldc, 148, 0, s, te, n_experts, mode);
   return launch_gemm<128, 6>(a, w, c, nullptr, M, N, K, lda, K, ldc, 148, 0, s, te, n_experts, mode);
 }

@@ -3,7 +3,7 @@
 //   out[t, h dv + i] = o[t, h, i] / div[t, h] / rms over the head * w * act(g[t, h dv + i])       head_norm_gate
 //   out[t, h dv + i] = a[t, h, i] * sigmoid(g[t, h dv + i])                                        head_gate
 //
-// every factor optional in the first (w: one weight per element shared by the heads, or one per head and element; act:
+// every factor optional in the first (a head may be a whole row; w: one weight per element shared by the heads, or one per head and element; act:
 // silu or sigmoid).  The heads of `a` may be stored wider than dv.  A warp owns whole heads.
 #include "vec_io.cuh"
 
@@ -144,6 +144,69 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(HeadNormParams<T> p
   }
 }
 
+// one item per CTA: heads (whole rows, where all heads are normed together) too large for a warp
+template <typename T, int V>
+__global__ void __launch_bounds__(256) row_norm_gate_kernel(HeadNormParams<T> p) {
+  constexpr int NI = 4;
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t it = blockIdx.x, t = it / p.H;
+  const int h = (int)(it - t * p.H);
+  const float* src = p.o + it * p.dv;
+  float f = 1.f;
+  if (p.div != nullptr) {
+    const float d = p.div[it];
+    f = d > 0.f ? 1.f / d : 0.f;
+  }
+  float x[NI][V];
+  float ss = 0.f;
+  for (int c0 = 0; c0 < p.dv; c0 += 256 * V * NI) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int c = c0 + (threadIdx.x + 256 * i) * V;
+      if (c >= p.dv) continue;
+      load_f32<V>(src + c, x[i]);
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        x[i][j] *= f;
+        ss += x[i][j] * x[i][j];
+      }
+    }
+  }
+  float inv = 1.f;
+  if (p.unit_norm) inv = 1.f / sqrtf(block_sum(ss, red) / (float)p.dv + p.eps);
+  T* dst = p.out + t * p.out_ld + (int64_t)h * p.dv;
+  const T* gr = p.g != nullptr ? p.g + t * p.g_ld + (int64_t)h * p.dv : nullptr;
+  const T* w = p.w != nullptr ? p.w + (int64_t)h * p.w_head : nullptr;
+  for (int c0 = 0; c0 < p.dv; c0 += 256 * V * NI) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int c = c0 + (threadIdx.x + 256 * i) * V;
+      if (c >= p.dv) continue;
+      if (p.dv > 256 * V * NI) {             // does not fit the registers: read again
+        load_f32<V>(src + c, x[i]);
+#pragma unroll
+        for (int j = 0; j < V; ++j) x[i][j] *= f;
+      }
+      float y[V], u[V];
+#pragma unroll
+      for (int j = 0; j < V; ++j) y[j] = x[i][j] * inv;
+      if (w != nullptr) {
+        load_f32<V>(w + c, u);
+#pragma unroll
+        for (int j = 0; j < V; ++j) y[j] *= u[j];
+      }
+      if (gr != nullptr) {
+        load_f32<V>(gr + c, u);
+#pragma unroll
+        for (int j = 0; j < V; ++j) y[j] *= gate_act<T>(u[j], p.act);
+      }
+      store_f32<V>(dst + c, y);
+    }
+  }
+}
+
 template <typename T, int V>
 __global__ void __launch_bounds__(256) head_gate_kernel(T* __restrict__ out, const T* __restrict__ a, const T* __restrict__ g,
                                                         int64_t g_ld, int64_t tokens, int H, int dv, int d_pad) {
@@ -181,7 +244,14 @@ XLLM_API int xllm_head_norm_gate(void* out, int64_t out_ld, const void* o, const
     if (dv % 4 == 0 && out_ld % 4 == 0 && (g == nullptr || g_ld % 4 == 0) && w_head % 4 == 0 && al(out, v) && al(o, 16) &&
         al(g, v) && al(w, v) && dv <= 128 && p.items < (1LL << 32))
       launch_pdl(head_norm_gate_small_kernel<T, 4>, dim3((unsigned)((p.items + 31) / 32)), block, 0, (cudaStream_t)stream, p);
-    else if (dv % 4 == 0 && out_ld % 4 == 0 && (g == nullptr || g_ld % 4 == 0) && w_head % 4 == 0 && al(out, v) && al(o, 16) &&
+    else if (dv > 512 && p.items < (1LL << 31)) {
+      const dim3 rows((unsigned)p.items);
+      if (dv % 4 == 0 && out_ld % 4 == 0 && (g == nullptr || g_ld % 4 == 0) && w_head % 4 == 0 && al(out, v) && al(o, 16) &&
+          al(g, v) && al(w, v))
+        launch_pdl(row_norm_gate_kernel<T, 4>, rows, block, 0, (cudaStream_t)stream, p);
+      else
+        launch_pdl(row_norm_gate_kernel<T, 1>, rows, block, 0, (cudaStream_t)stream, p);
+    } else if (dv % 4 == 0 && out_ld % 4 == 0 && (g == nullptr || g_ld % 4 == 0) && w_head % 4 == 0 && al(out, v) && al(o, 16) &&
              al(g, v) && al(w, v))
       launch_pdl(head_norm_gate_kernel<T, 4>, grid, block, 0, (cudaStream_t)stream, p);
     else

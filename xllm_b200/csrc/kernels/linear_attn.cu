@@ -5,8 +5,8 @@
 // The decay a_t is either one constant per head (retention) or a value per token and key channel,
 // a = sigmoid(W_2 r + b)^(1 / tau) with r the low-rank column block of the projection row (gated linear attention).
 // q and k may be rotated (rotate-half or interleaved pairs) and scaled; the output of a head may be divided by its
-// root mean square, weighted, and multiplied by silu(g).  All of that happens here, in fp32, from the projection
-// rows as the GEMM left them.
+// root mean square, weighted, and multiplied by silu(g); q, k and v may pass through silu first.  All of that happens
+// here, in fp32, from the projection rows as the GEMM left them.
 //
 //   linattn_decode_kernel     one token per sequence: state read once and written once, output finished (norm, gate)
 //   linattn_chunk_kernel      prompt chunks, bf16, dk <= 256: 16 tokens at a time on the tensor cores.  A warp owns 16
@@ -19,7 +19,8 @@
 // (head_norm.cu finishes the fp32 outputs of the two prompt kernels)
 //
 // A sequence whose rows in the batch are its first tokens (kv_len == number of rows) starts from S = 0 whatever its
-// slot holds; slot < 0 marks padding rows.  The reference has no such layer; its nearest relative is the Triton
+// slot holds; slot < 0 marks padding rows.  Token by token a state is decayed as S + (a - 1) S with a - 1 = expm1(log a): a
+// itself, rounded to fp32, would be off by 2^-25, which a slow decay multiplies by the 1 / (1 - a) tokens it sums over.  The reference has no such layer; its nearest relative is the Triton
 // gated delta rule (xllm/python/kernels_cuda/triton/gdn_prefill.py).  Built without fast-math: errors of the decay
 // accumulate over a sequence.
 #include "attn_common.cuh"
@@ -42,9 +43,10 @@ struct LinAttnParams {
   const T* a2;               // [H * dk, rank]
   const T* a2_b;             // [H * dk]
   const T* norm_w;           // [dv] or null
-  void* out;                 // decode: T [rows, out_ld]; prompt: float [T, H, dv]
+  void* out;                 // decode: T [rows, out_ld], or with raw_out float [rows, H, dv]; prompt: float [T, H, dv]
   int64_t out_ld;
   int n_seqs, H, dk, dv, dv_pad, rot, interleaved, rank, unit_norm, vec_ok;
+  int in_silu, raw_out;      // q, k and v pass through silu; decode leaves raw fp32 outputs
   float q_scale, k_scale, inv_tau, eps;
 };
 
@@ -53,16 +55,23 @@ __device__ __forceinline__ float silu_f32(float z) { return z / (1.f + expf(-z))
 // for rows that leave as bf16: hardware exponential and division (2^-21 relative)
 __device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 
+// a projected value as it enters the recurrence
+template <typename T>
+__device__ __forceinline__ float entering(T x, int in_silu) {
+  const float u = to_f32(x);
+  return in_silu ? silu_as<T>(u) : u;
+}
+
 // element i of a head after the rotation of its first `rot` elements; `cs` is the position's cos | sin row
 template <typename T>
-__device__ __forceinline__ float rotated(const T* x, int i, int rot, int interleaved, const float* cs) {
-  const float u = to_f32(x[i]);
+__device__ __forceinline__ float rotated(const T* x, int i, int rot, int interleaved, const float* cs, int in_silu) {
+  const float u = entering(x[i], in_silu);
   if (cs == nullptr || i >= rot) return u;
   const int half = rot >> 1;
   const bool first = interleaved ? (i & 1) == 0 : i < half;
   const int n = interleaved ? i >> 1 : (first ? i : i - half);
   const int j = interleaved ? i ^ 1 : (first ? i + half : i - half);
-  const float v = to_f32(x[j]);
+  const float v = entering(x[j], in_silu);
   const float c = cs[n], s = cs[half + n];
   return first ? u * c - v * s : u * c + v * s;
 }
@@ -104,10 +113,14 @@ __global__ void __launch_bounds__(256) linattn_decode_kernel(LinAttnParams<T> p)
   pdl_wait();
   pdl_launch_dependents();
   T* orow = reinterpret_cast<T*>(p.out) + b * p.out_ld + (int64_t)h * dv;
+  float* raw = reinterpret_cast<float*>(p.out) + ((int64_t)b * p.H + h) * dv;
   const int slot = p.slots[b];
   const int len = p.kv_lens[b];
   if (slot < 0 || len <= 0) {
-    for (int i = tid; i < dv; i += 256) orow[i] = from_f32<T>(0.f);
+    for (int i = tid; i < dv; i += 256) {
+      if (p.raw_out) raw[i] = 0.f;
+      else orow[i] = from_f32<T>(0.f);
+    }
     return;
   }
   const bool active = rg < RG, fresh = len == 1;
@@ -128,12 +141,12 @@ __global__ void __launch_bounds__(256) linattn_decode_kernel(LinAttnParams<T> p)
     const T* vr = p.v + b * p.ld + (int64_t)h * dv;
     const float* cs = rope_row(p, b);
     for (int i = tid; i < dk; i += 256) {
-      qs[i] = rotated(qr, i, p.rot, p.interleaved, cs) * p.q_scale;
-      ks[i] = rotated(kr, i, p.rot, p.interleaved, cs) * p.k_scale;
-      as[i] = expf(p.log_decay != nullptr ? p.log_decay[h]
+      qs[i] = rotated(qr, i, p.rot, p.interleaved, cs, p.in_silu) * p.q_scale;
+      ks[i] = rotated(kr, i, p.rot, p.interleaved, cs, p.in_silu) * p.k_scale;
+      as[i] = expm1f(p.log_decay != nullptr ? p.log_decay[h]
                                           : channel_log_decay(p, p.r + b * p.ld, (int64_t)h * dk + i));
     }
-    for (int i = tid; i < dvp; i += 256) vs[i] = i < dv ? to_f32(vr[i]) : 0.f;
+    for (int i = tid; i < dvp; i += 256) vs[i] = i < dv ? entering(vr[i], p.in_silu) : 0.f;
   }
   __syncthreads();
   float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -147,7 +160,8 @@ __global__ void __launch_bounds__(256) linattn_decode_kernel(LinAttnParams<T> p)
         if (r >= dk) break;
         const float a = as[r], kk = ks[r], qq = qs[r];
         float4 x = s[u];
-        x.x = a * x.x + kk * v4.x; x.y = a * x.y + kk * v4.y; x.z = a * x.z + kk * v4.z; x.w = a * x.w + kk * v4.w;
+        x.x = fmaf(a, x.x, x.x) + kk * v4.x; x.y = fmaf(a, x.y, x.y) + kk * v4.y;
+        x.z = fmaf(a, x.z, x.z) + kk * v4.z; x.w = fmaf(a, x.w, x.w) + kk * v4.w;
         *reinterpret_cast<float4*>(S + (int64_t)r * dvp) = x;
         o.x += qq * x.x; o.y += qq * x.y; o.z += qq * x.z; o.w += qq * x.w;
       }
@@ -159,9 +173,11 @@ __global__ void __launch_bounds__(256) linattn_decode_kernel(LinAttnParams<T> p)
   for (int i = tid; i < dvp; i += 256) {
     float a = 0.f;
     for (int w = 0; w < RG; ++w) a += red[w * dvp + i];
+    if (p.raw_out && i < dv) raw[i] = a;
     vs[i] = a;                            // v is no longer needed; each thread reads back its own entries
     if (i < dv) ss += a * a;
   }
+  if (p.raw_out) return;
   float inv = 1.f;
   if (p.unit_norm) inv = 1.f / sqrtf(block_sum(ss, red32) / (float)dv + p.eps);
   for (int i = tid; i < dv; i += 256) {
@@ -207,12 +223,12 @@ __global__ void __launch_bounds__(256) linattn_recurrent_kernel(LinAttnParams<T>
     const T* kr = p.k + row * p.ld + (int64_t)h * dk;
     const float* cs = rope_row(p, row);
     for (int i = tid; i < dk; i += 256) {
-      qs[i] = rotated(qr, i, p.rot, p.interleaved, cs) * p.q_scale;
-      ks[i] = rotated(kr, i, p.rot, p.interleaved, cs) * p.k_scale;
-      as[i] = expf(p.log_decay != nullptr ? p.log_decay[h]
+      qs[i] = rotated(qr, i, p.rot, p.interleaved, cs, p.in_silu) * p.q_scale;
+      ks[i] = rotated(kr, i, p.rot, p.interleaved, cs, p.in_silu) * p.k_scale;
+      as[i] = expm1f(p.log_decay != nullptr ? p.log_decay[h]
                                           : channel_log_decay(p, p.r + row * p.ld, (int64_t)h * dk + i));
     }
-    if (tid < 32) vs[t & 1][tid] = c0 + tid < p.dv ? to_f32(p.v[row * p.ld + (int64_t)h * p.dv + c0 + tid]) : 0.f;
+    if (tid < 32) vs[t & 1][tid] = c0 + tid < p.dv ? entering(p.v[row * p.ld + (int64_t)h * p.dv + c0 + tid], p.in_silu) : 0.f;
     __syncthreads();
     const float4 v4 = *reinterpret_cast<const float4*>(&vs[t & 1][cg * 4]);
     float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -222,7 +238,8 @@ __global__ void __launch_bounds__(256) linattn_recurrent_kernel(LinAttnParams<T>
       if (r >= dk) break;
       const float a = as[r], kk = ks[r], qq = qs[r];
       float4& x = s[u];
-      x.x = a * x.x + kk * v4.x; x.y = a * x.y + kk * v4.y; x.z = a * x.z + kk * v4.z; x.w = a * x.w + kk * v4.w;
+      x.x = fmaf(a, x.x, x.x) + kk * v4.x; x.y = fmaf(a, x.y, x.y) + kk * v4.y;
+      x.z = fmaf(a, x.z, x.z) + kk * v4.z; x.w = fmaf(a, x.w, x.w) + kk * v4.w;
       o.x += qq * x.x; o.y += qq * x.y; o.z += qq * x.z; o.w += qq * x.w;
     }
 #pragma unroll
@@ -504,6 +521,13 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 512 / (NW * 32)) linat
               const float2 qb = unpack2(*reinterpret_cast<const uint32_t*>(rq + t * DK + cb));
               q4[0] = qa.x; q4[1] = qa.y; q4[2] = qb.x; q4[3] = qb.y;
             }
+            if (p.in_silu) {
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                k4[e] = silu_fast(k4[e]);
+                if (!STATE_ONLY) q4[e] = silu_fast(q4[e]);
+              }
+            }
             if (turns) {
               const float* cs = csb + (buf * kLC + t) * rot;
               const float2 co = *reinterpret_cast<const float2*>(cs + 2 * m);
@@ -574,8 +598,8 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 512 / (NW * 32)) linat
                 eq = elog[kLC + t - ref];
                 ek = elog[kLC + ref - t];
               }
-              qv[e] = rotated(rq + t * DK, c + e, rot, p.interleaved, cs) * p.q_scale * eq;
-              kv[e] = rotated(rk + t * DK, c + e, rot, p.interleaved, cs) * p.k_scale * ek;
+              qv[e] = rotated(rq + t * DK, c + e, rot, p.interleaved, cs, p.in_silu) * p.q_scale * eq;
+              kv[e] = rotated(rk + t * DK, c + e, rot, p.interleaved, cs, p.in_silu) * p.k_scale * ek;
             }
           }
           uint32_t qh, ql, kh, kl;
@@ -614,6 +638,13 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 512 / (NW * 32)) linat
       if (has_cols) {
         uint32_t v0, v1, v2, v3;
         ldmatrix_x4_trans(v0, v1, v2, v3, sb + L::v + buf * L::vtile + swz<VCH>(arow, warp * 2 + acb));
+        if (p.in_silu) {                    // a value belongs to one warp only
+          const auto act = [](uint32_t& u) {
+            const float2 f = unpack2(u);
+            u = pack_bf162(silu_fast(f.x), silu_fast(f.y));
+          };
+          act(v0); act(v1); act(v2); act(v3);
+        }
         if (!STATE_ONLY) {
           float pw[2][4];
 #pragma unroll
@@ -691,10 +722,16 @@ __global__ void __launch_bounds__(NW * 32, DK > 128 ? 1 : 512 / (NW * 32)) linat
 #pragma unroll
         for (int j = 0; j < 2; ++j)
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int t = (lane >> 2) + (e >> 1) * 8, c = c0 + warp * 16 + j * 8 + (lane & 3) * 2 + (e & 1);
-            if (t >= s0 && t < s1 && c < p.dv)
-              reinterpret_cast<float*>(p.out)[((int64_t)(row0 + t0 + t) * p.H + h) * p.dv + c] = o[j][e];
+          for (int e = 0; e < 4; e += 2) {
+            const int t = (lane >> 2) + (e >> 1) * 8, c = c0 + warp * 16 + j * 8 + (lane & 3) * 2;
+            if (t < s0 || t >= s1 || c >= p.dv) continue;
+            float* dst = reinterpret_cast<float*>(p.out) + ((int64_t)(row0 + t0 + t) * p.H + h) * p.dv + c;
+            if (p.dv % 2 == 0) {
+              *reinterpret_cast<float2*>(dst) = make_float2(o[j][e], o[j][e + 1]);
+            } else {
+              dst[0] = o[j][e];
+              if (c + 1 < p.dv) dst[1] = o[j][e + 1];
+            }
           }
         continue;
       }
@@ -835,8 +872,10 @@ XLLM_API int xllm_linattn(void* state, const void* slots, const void* cu_q, cons
                           const void* positions, const void* log_decay, const void* a2, const void* a2_b, const void* norm_w,
                           void* out, int64_t out_ld, int n_seqs, int H, int dk, int dv, int rot, int interleaved, int rank,
                           int unit_norm, float q_scale, float k_scale, float inv_tau, float eps, int dtype, int mode,
-                          void* seg_state, void* seg_decay, int seg_len, int segs, int finish, void* stream) {
-  // mode 0: one token per sequence, sequence s is row s, `out` finished in the activation type (cu_q unused)
+                          void* seg_state, void* seg_decay, int seg_len, int segs, int finish, int in_silu, void* stream) {
+  // in_silu: q, k and v pass through silu before anything else
+  // mode 0: one token per sequence, sequence s is row s, `out` finished in the activation type, or without `finish` raw
+  //         fp32 [rows, H, dv] (cu_q unused)
   // mode 1: prompt rows by cu_q, `out` raw fp32 [T, H, dv], or with `finish` (dv <= 128) finished bf16 rows [T, out_ld].
   //         Prompts longer than seg_len run as up to `segs` segments side by side: seg_state fp32 [n, H, dk, dv_pad] and
   //         seg_decay fp32 [n, H, dk] with n = T / seg_len + n_seqs + 1, seg_len a multiple of 16.
@@ -859,6 +898,7 @@ XLLM_API int xllm_linattn(void* state, const void* slots, const void* cu_q, cons
     p.out = out; p.out_ld = out_ld; p.n_seqs = n_seqs; p.H = H; p.dk = dk; p.dv = dv; p.dv_pad = (dv + 3) & ~3; p.rot = rot;
     p.interleaved = interleaved; p.rank = log_decay ? 0 : rank; p.unit_norm = unit_norm; p.q_scale = q_scale;
     p.k_scale = k_scale; p.inv_tau = inv_tau; p.eps = eps;
+    p.in_silu = in_silu; p.raw_out = mode == 0 && !finish;
     const auto a16 = [](const void* x) { return (((uintptr_t)x) & 15) == 0; };
     p.vec_ok = dk % 8 == 0 && dv % 8 == 0 && ld % 8 == 0 && a16(q) && a16(k) && a16(v) &&
                (log_decay != nullptr || (rank % 8 == 0 && a16(r)));

@@ -12,6 +12,10 @@
 //
 //   xllm_mla_cache_write : RMSNorm(c_kv) * w | RoPE(k_pe) -> cache row of the token's slot, and RoPE
 //                          of the rotary part of every query head, in one pass over the token
+//   xllm_latent_norm     : the two norms of a layer whose queries go through a latent too: normed query latents out, normed
+//                          latents to the cache rows, no rotary part
+//   xllm_latent_decode   : the decode kernel over caches of latents alone (rows of 128, 256 or 512 values)
+//   xllm_latent_gather   : the cached latents of a few sequences as dense rows (prompts expand them to keys and values)
 //   xllm_mla_decode      : split-KV attention of N query rows (nh heads each) against the cache.
 //                          A query row names its own visible length and block-table row, so decode
 //                          tokens (one per sequence) and the tokens of prompt chunks (each sees the
@@ -27,6 +31,7 @@
 // are merged through shared memory at the end; splits > 1 write normalised partials for
 // xllm_attn_merge.
 #include "attn_common.cuh"
+#include "vec_io.cuh"
 #include <atomic>
 
 namespace xllm {
@@ -34,15 +39,18 @@ namespace mla {
 
 constexpr int kDQK = 576;         // latent + rope width of a cache row
 constexpr int kDV = 512;          // latent width (the part that is V)
-constexpr int kCH = kDQK / 8;     // 16-byte chunks per row
-constexpr int kTileBytes = 16 * kDQK * 2;
-constexpr int kStages = 2;
 constexpr int kPairs = 4;
 constexpr int kThreads = kPairs * 64;
-constexpr int kQBytes = kTileBytes;                               // 16 heads x 576
-constexpr int kRingBytes = kPairs * kStages * kTileBytes;         // 147456
 constexpr int kXchgBytes = kPairs * 2 * 256 * 4;                  // partial scores of the two halves
-constexpr int kSmem = kQBytes + kRingBytes + kXchgBytes;
+
+template <int DQK, int DV, int STAGES>
+struct DecodeSmem {
+  static constexpr int tile = 16 * DQK * 2;
+  static constexpr int q = tile;                                  // 16 heads
+  static constexpr int ring = kPairs * STAGES * tile;
+  static constexpr int total = q + ring + kXchgBytes;
+  static_assert(ring + kXchgBytes >= (128 + kPairs * 16 * DV) * 4, "the merge reuses the ring");
+};
 
 struct DecodeParams {
   const bf16* q;               // [N, nh, 576]
@@ -63,7 +71,10 @@ __device__ __forceinline__ void pair_sync(int pair) {
   asm volatile("bar.sync %0, 64;" ::"r"(pair + 1) : "memory");
 }
 
+template <int DQK, int DV, int STAGES>
 __global__ void __launch_bounds__(kThreads) mla_decode_kernel(DecodeParams p) {
+  using M = DecodeSmem<DQK, DV, STAGES>;
+  constexpr int CH = DQK / 8;       // 16-byte chunks per row
   extern __shared__ __align__(128) uint8_t smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int pair = warp >> 1, half = warp & 1;
@@ -82,61 +93,62 @@ __global__ void __launch_bounds__(kThreads) mla_decode_kernel(DecodeParams p) {
   // ---- the 16 query rows go to shared memory once (rows beyond nh are zero)
   const uint32_t q_smem = smem_u32(smem);
   {
-    const bf16* qb = p.q + (int64_t)n * p.q_stride + (int64_t)head0 * kDQK;
-    for (int id = threadIdx.x; id < 16 * kCH; id += kThreads) {
-      const int r = id / kCH, c = id - r * kCH;
-      cp_async16(q_smem + swz<kCH>(r, c), qb + (int64_t)(r < rows_valid ? r : 0) * kDQK + c * 8, r < rows_valid);
+    const bf16* qb = p.q + (int64_t)n * p.q_stride + (int64_t)head0 * DQK;
+    for (int id = threadIdx.x; id < 16 * CH; id += kThreads) {
+      const int r = id / CH, c = id - r * CH;
+      cp_async16(q_smem + swz<CH>(r, c), qb + (int64_t)(r < rows_valid ? r : 0) * DQK + c * 8, r < rows_valid);
     }
     cp_async_commit();
   }
-  const uint32_t ring = q_smem + kQBytes + pair * (kStages * kTileBytes);
-  float* xchg = reinterpret_cast<float*>(smem + kQBytes + kRingBytes) + pair * 512;
+  const uint32_t ring = q_smem + M::q + pair * (STAGES * M::tile);
+  float* xchg = reinterpret_cast<float*>(smem + M::q + M::ring) + pair * 512;
   const int32_t* bt = p.block_table + (int64_t)(p.bt_rows ? p.bt_rows[n] : n) * p.bt_stride;
 
-  auto load_tile = [&](int i) {  // i-th tile of this pair -> stage i % kStages; both warps copy half of it
+  auto load_tile = [&](int i) {  // i-th tile of this pair -> stage i % STAGES; both warps copy half of it
     if (i < my_n) {
       const int tok0 = (t_begin + pair + kPairs * i) << 4;
       const int page = tok0 / p.page_size;
       const int off = tok0 - page * p.page_size;
-      const bf16* kb = p.cache + ((int64_t)bt[page] * p.page_size + off) * kDQK;
-      const uint32_t dst = ring + (i % kStages) * kTileBytes;
+      const bf16* kb = p.cache + ((int64_t)bt[page] * p.page_size + off) * DQK;
+      const uint32_t dst = ring + (i % STAGES) * M::tile;
 #pragma unroll
-      for (int j = 0; j < (16 * kCH) / 64; ++j) {
+      for (int j = 0; j < (16 * CH) / 64; ++j) {
         const int id = (half * 32 + lane) + j * 64;
-        const int r = id / kCH, c = id - r * kCH;
+        const int r = id / CH, c = id - r * CH;
         const bool valid = tok0 + r < seq_len;
-        cp_async16(dst + swz<kCH>(r, c), kb + (valid ? (int64_t)r * kDQK + c * 8 : 0), valid);
+        cp_async16(dst + swz<CH>(r, c), kb + (valid ? (int64_t)r * DQK + c * 8 : 0), valid);
       }
     }
     cp_async_commit();
   };
 
-  float o[kDV / 16][4];   // this warp's 256 output columns: 32 n8 tiles
+  float o[DV / 16][4];   // this warp's half of the output columns, in n8 tiles
 #pragma unroll
-  for (int i = 0; i < kDV / 16; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  for (int i = 0; i < DV / 16; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
 
-  load_tile(0);
-  cp_async_wait<1>();   // the query rows (the first group); tile 0 may still be in flight
+#pragma unroll
+  for (int i = 0; i < STAGES - 1; ++i) load_tile(i);
+  cp_async_wait<STAGES - 1>();   // the query rows (the first group); the tiles may still be in flight
   __syncthreads();      // they were copied by all warps of the CTA
   for (int i = 0; i < my_n; ++i) {
-    cp_async_wait<0>();
+    cp_async_wait<STAGES - 2>();
     pair_sync(pair);               // tile i is complete; both warps are done with tile i - 1
-    load_tile(i + 1);
-    const uint32_t k_addr = ring + (i % kStages) * kTileBytes;
+    load_tile(i + STAGES - 1);
+    const uint32_t k_addr = ring + (i % STAGES) * M::tile;
     const int tok0 = (t_begin + pair + kPairs * i) << 4;
 
-    // ---- partial scores over this warp's half of the 576 columns (18 k-steps of 16)
+    // ---- partial scores over this warp's half of the columns (k-steps of 16)
     float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
     {
       const int brow = (lane & 7) + ((lane >> 4) << 3);
       const int bcb = (lane >> 3) & 1;
       const int arow = lane & 15, acb = lane >> 4;
 #pragma unroll 6
-      for (int ks = half * 18; ks < half * 18 + 18; ++ks) {
+      for (int ks = half * (DQK / 32); ks < (half + 1) * (DQK / 32); ++ks) {
         uint32_t a[4], b0, b1, b2, b3;
-        ldmatrix_x4(a[0], a[1], a[2], a[3], q_smem + swz<kCH>(arow, ks * 2 + acb));
-        ldmatrix_x4(b0, b1, b2, b3, k_addr + swz<kCH>(brow, ks * 2 + bcb));
+        ldmatrix_x4(a[0], a[1], a[2], a[3], q_smem + swz<CH>(arow, ks * 2 + acb));
+        ldmatrix_x4(b0, b1, b2, b3, k_addr + swz<CH>(brow, ks * 2 + bcb));
         mma_bf16_16816(s[0], a, b0, b1);
         mma_bf16_16816(s[1], a, b2, b3);
       }
@@ -185,7 +197,7 @@ __global__ void __launch_bounds__(kThreads) mla_decode_kernel(DecodeParams p) {
     l0 = l0 * a0 + rs0;
     l1 = l1 * a1 + rs1;
 #pragma unroll
-    for (int i2 = 0; i2 < kDV / 16; ++i2) {
+    for (int i2 = 0; i2 < DV / 16; ++i2) {
       o[i2][0] *= a0; o[i2][1] *= a0; o[i2][2] *= a1; o[i2][3] *= a1;
     }
     uint32_t pa[4];
@@ -194,13 +206,13 @@ __global__ void __launch_bounds__(kThreads) mla_decode_kernel(DecodeParams p) {
     pa[2] = pack_bf162(s[1][0], s[1][1]);
     pa[3] = pack_bf162(s[1][2], s[1][3]);
     {
-      // V = the first 512 columns of the same tile; this warp takes columns [256 half, 256 half + 256)
+      // V = the first DV columns of the same tile; this warp takes one half of them
       const int row = (lane & 7) + (((lane >> 3) & 1) << 3);
       const int cb = lane >> 4;
 #pragma unroll
-      for (int jn = 0; jn < kDV / 32; ++jn) {
+      for (int jn = 0; jn < DV / 32; ++jn) {
         uint32_t v0, v1, v2, v3;
-        ldmatrix_x4_trans(v0, v1, v2, v3, k_addr + swz<kCH>(row, (half * (kDV / 32) + jn) * 2 + cb));
+        ldmatrix_x4_trans(v0, v1, v2, v3, k_addr + swz<CH>(row, (half * (DV / 32) + jn) * 2 + cb));
         mma_bf16_16816(o[jn * 2], pa, v0, v1);
         mma_bf16_16816(o[jn * 2 + 1], pa, v2, v3);
       }
@@ -213,9 +225,9 @@ __global__ void __launch_bounds__(kThreads) mla_decode_kernel(DecodeParams p) {
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
   __syncthreads();  // every pair is done with its ring; reuse it for the merge
 
-  float* sm_m = reinterpret_cast<float*>(smem + kQBytes);  // [4][16]
+  float* sm_m = reinterpret_cast<float*>(smem + M::q);     // [4][16]
   float* sm_l = sm_m + 64;                                 // [4][16]
-  float* sm_o = sm_l + 64;                                 // [4][16][512]
+  float* sm_o = sm_l + 64;                                 // [4][16][DV]
   {
     const int r0 = lane >> 2, r1 = r0 + 8;
     if (half == 0 && (lane & 3) == 0) {
@@ -223,15 +235,15 @@ __global__ void __launch_bounds__(kThreads) mla_decode_kernel(DecodeParams p) {
       sm_l[pair * 16 + r0] = l0; sm_l[pair * 16 + r1] = l1;
     }
 #pragma unroll
-    for (int nt = 0; nt < kDV / 16; ++nt) {
-      const int col = half * (kDV / 2) + nt * 8 + (lane & 3) * 2;
-      *reinterpret_cast<float2*>(sm_o + (pair * 16 + r0) * kDV + col) = make_float2(o[nt][0], o[nt][1]);
-      *reinterpret_cast<float2*>(sm_o + (pair * 16 + r1) * kDV + col) = make_float2(o[nt][2], o[nt][3]);
+    for (int nt = 0; nt < DV / 16; ++nt) {
+      const int col = half * (DV / 2) + nt * 8 + (lane & 3) * 2;
+      *reinterpret_cast<float2*>(sm_o + (pair * 16 + r0) * DV + col) = make_float2(o[nt][0], o[nt][1]);
+      *reinterpret_cast<float2*>(sm_o + (pair * 16 + r1) * DV + col) = make_float2(o[nt][2], o[nt][3]);
     }
   }
   __syncthreads();
-  for (int idx = threadIdx.x; idx < rows_valid * kDV; idx += kThreads) {
-    const int r = idx / kDV, d = idx - r * kDV;
+  for (int idx = threadIdx.x; idx < rows_valid * DV; idx += kThreads) {
+    const int r = idx / DV, d = idx - r * DV;
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kPairs; ++w) M = fmaxf(M, sm_m[w * 16 + r]);
@@ -240,16 +252,16 @@ __global__ void __launch_bounds__(kThreads) mla_decode_kernel(DecodeParams p) {
 #pragma unroll
       for (int w = 0; w < kPairs; ++w) {
         const float wgt = exp2f(sm_m[w * 16 + r] - M);
-        acc += sm_o[(w * 16 + r) * kDV + d] * wgt;
+        acc += sm_o[(w * 16 + r) * DV + d] * wgt;
         L += sm_l[w * 16 + r] * wgt;
       }
     }
     const float val = L > 0.f ? acc / L : 0.f;
     const int64_t head = (int64_t)n * p.nh + head0 + r;
     if (p.splits == 1) {
-      p.out[head * kDV + d] = __float2bfloat16(val);
+      p.out[head * DV + d] = __float2bfloat16(val);
     } else {
-      p.o_part[(head * p.splits + split) * kDV + d] = val;
+      p.o_part[(head * p.splits + split) * DV + d] = val;
       if (d == 0) p.lse_part[head * p.splits + split] = L > 0.f ? M + log2f(L) : -INFINITY;
     }
   }
@@ -325,6 +337,80 @@ __global__ void __launch_bounds__(128) mla_cache_write_kernel(WriteParams p) {
   }
 }
 
+// grid (tokens, 1 or 2): normed query latents, and normed latents into the cache row of the token's slot
+template <typename T>
+struct LatentNormParams {
+  const T *q, *c;            // [T, q_rank], [T, rank] with row stride ld; c null: query latents only
+  const T *q_w, *c_w;
+  T* q_out;                  // [T, q_pad], zero filled
+  T* cache;                  // rows of `width`, zero filled
+  const int32_t* slots;
+  int64_t ld;
+  int q_rank, q_pad, rank, width;
+  float eps;
+};
+
+template <typename T, int V>
+__global__ void __launch_bounds__(128) latent_norm_kernel(LatentNormParams<T> p) {
+  __shared__ float red[32];
+  constexpr int NI = 4;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int64_t t = blockIdx.x;
+  const bool is_c = blockIdx.y == 1;
+  const int slot = is_c ? p.slots[t] : 0;
+  if (is_c && slot < 0) return;
+  const T* x = (is_c ? p.c : p.q) + t * p.ld;
+  const T* w = is_c ? p.c_w : p.q_w;
+  T* dst = is_c ? p.cache + (int64_t)slot * p.width : p.q_out + t * p.q_pad;
+  const int n = is_c ? p.rank : p.q_rank, pad = is_c ? p.width : p.q_pad;
+  float f[NI][V];
+  float ss = 0.f;
+  for (int c0 = 0; c0 < n; c0 += 128 * V * NI) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int c = c0 + (threadIdx.x + 128 * i) * V;
+      if (c >= n) continue;
+      load_f32<V>(x + c, f[i]);
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += f[i][j] * f[i][j];
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)n + p.eps);
+  for (int c0 = 0; c0 < pad; c0 += 128 * V * NI) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int c = c0 + (threadIdx.x + 128 * i) * V;
+      if (c >= pad) continue;
+      float y[V], g[V];
+#pragma unroll
+      for (int j = 0; j < V; ++j) y[j] = 0.f;
+      if (c < n) {
+        if (n > 128 * V * NI) load_f32<V>(x + c, f[i]);        // does not fit the registers: read again
+        load_f32<V>(w + c, g);
+#pragma unroll
+        for (int j = 0; j < V; ++j) y[j] = f[i][j] * inv * g[j];
+      }
+      store_f32<V>(dst + c, y);
+    }
+  }
+}
+
+// rows i of sequence s -> out[s * rows_per + i], zero behind the sequence; grid (rows_per / 8, sequences), a warp per row
+__global__ void __launch_bounds__(256) latent_gather_kernel(uint4* __restrict__ out, const uint4* __restrict__ cache,
+                                                            const int32_t* __restrict__ block_table, int bt_stride,
+                                                            const int32_t* __restrict__ kv_lens, int rows_per, int page, int nvec) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int s = blockIdx.y, i = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (i >= rows_per) return;
+  uint4* dst = out + ((int64_t)s * rows_per + i) * nvec;
+  const bool in = i < kv_lens[s];
+  const uint4* src = cache;
+  if (in) src += ((int64_t)block_table[(int64_t)s * bt_stride + i / page] * page + i % page) * nvec;
+  for (int v = lane; v < nvec; v += 32) dst[v] = in ? src[v] : make_uint4(0, 0, 0, 0);
+}
+
 }  // namespace mla
 }  // namespace xllm
 
@@ -341,12 +427,14 @@ XLLM_API int64_t xllm_mla_decode_workspace(int64_t n_rows, int nh, int splits) {
 // row; when null, positions [N] int64 gives it as position + 1 (rows of a prompt chunk).  bt_rows [N]
 // int32: block-table row of each query row (null: row n uses table row n).  page_size % 16 == 0.
 // workspace: xllm_mla_decode_workspace() floats when splits > 1.
-XLLM_API int xllm_mla_decode(void* out, const void* q, int64_t q_stride, const void* cache, const void* block_table,
-                             int bt_stride, const void* seq_lens, const void* positions, const void* bt_rows,
-                             int n_rows, int nh, int page_size, float scale, int splits, void* workspace,
-                             void* stream) {
+template <int DQK, int DV, int STAGES>
+static int mla_decode_impl(void* out, const void* q, int64_t q_stride, const void* cache, const void* block_table,
+                           int bt_stride, const void* seq_lens, const void* positions, const void* bt_rows,
+                           int n_rows, int nh, int page_size, float scale, int splits, void* workspace,
+                           void* stream) {
   using namespace xllm;
   using namespace xllm::mla;
+  constexpr int kSmem = DecodeSmem<DQK, DV, STAGES>::total;
   if (n_rows == 0) return 0;
   if (nh <= 0 || page_size <= 0 || page_size % 16 != 0 || splits < 1 || (seq_lens == nullptr && positions == nullptr) ||
       (splits > 1 && workspace == nullptr) || q_stride % 8 || (((uintptr_t)q | (uintptr_t)cache) & 15))
@@ -355,7 +443,7 @@ XLLM_API int xllm_mla_decode(void* out, const void* q, int64_t q_stride, const v
   int dev = 0;
   cudaGetDevice(&dev);
   if (!attr_done[dev & 63].load(std::memory_order_acquire)) {
-    cudaError_t e = cudaFuncSetAttribute(mla_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
+    cudaError_t e = cudaFuncSetAttribute(mla_decode_kernel<DQK, DV, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
     if (e != cudaSuccess) return (int)e;
     attr_done[dev & 63].store(true, std::memory_order_release);
   }
@@ -365,12 +453,74 @@ XLLM_API int xllm_mla_decode(void* out, const void* q, int64_t q_stride, const v
   p.out = (bf16*)out; p.q_stride = q_stride; p.bt_stride = bt_stride; p.nh = nh; p.page_size = page_size;
   p.splits = splits; p.scale_log2 = scale * 1.4426950408889634f;
   p.o_part = splits > 1 ? (float*)workspace : nullptr;
-  p.lse_part = p.o_part ? p.o_part + (int64_t)n_rows * nh * splits * kDV : nullptr;
+  p.lse_part = p.o_part ? p.o_part + (int64_t)n_rows * nh * splits * DV : nullptr;
   cudaStream_t s = (cudaStream_t)stream;
-  launch_pdl(mla_decode_kernel, dim3((nh + 15) / 16, n_rows, splits), dim3(kThreads), (size_t)kSmem, s, p);
+  launch_pdl(mla_decode_kernel<DQK, DV, STAGES>, dim3((nh + 15) / 16, n_rows, splits), dim3(kThreads), (size_t)kSmem, s, p);
   int rc = XLLM_LAUNCH_CHECK();
   if (rc != 0 || splits == 1) return rc;
-  return xllm_attn_merge(out, p.o_part, p.lse_part, (int64_t)n_rows * nh, splits, kDV, stream);
+  return xllm_attn_merge(out, p.o_part, p.lse_part, (int64_t)n_rows * nh, splits, DV, stream);
+}
+
+XLLM_API int xllm_mla_decode(void* out, const void* q, int64_t q_stride, const void* cache, const void* block_table,
+                             int bt_stride, const void* seq_lens, const void* positions, const void* bt_rows,
+                             int n_rows, int nh, int page_size, float scale, int splits, void* workspace,
+                             void* stream) {
+  return mla_decode_impl<xllm::mla::kDQK, xllm::mla::kDV, 2>(out, q, q_stride, cache, block_table, bt_stride, seq_lens, positions,
+                                                             bt_rows, n_rows, nh, page_size, scale, splits, workspace, stream);
+}
+
+// The same over caches without a rotary part: q [N, nh, width], cache [n_blocks, page, width], out [N, nh, width], width 128,
+// 256 or 512; workspace of n_rows * nh * splits * (width + 1) floats when splits > 1.
+XLLM_API int xllm_latent_decode(void* out, const void* q, int64_t q_stride, const void* cache, int width, const void* block_table,
+                                int bt_stride, const void* seq_lens, const void* positions, const void* bt_rows, int n_rows,
+                                int nh, int page_size, float scale, int splits, void* workspace, void* stream) {
+  const auto run = [&](auto impl) {
+    return impl(out, q, q_stride, cache, block_table, bt_stride, seq_lens, positions, bt_rows, n_rows, nh, page_size, scale,
+                splits, workspace, stream);
+  };
+  if (width == 128) return run(mla_decode_impl<128, 128, 3>);
+  if (width == 256) return run(mla_decode_impl<256, 256, 2>);
+  if (width == 512) return run(mla_decode_impl<512, 512, 2>);
+  return (int)cudaErrorInvalidValue;
+}
+
+// q_out [T, q_pad] = rmsnorm(q) * q_w and, with c, the cache row of every token's slot (-1: none) = rmsnorm(c) * c_w; q and c
+// are column blocks of rows with stride ld.  dtype: 0 bf16, 1 fp32.
+XLLM_API int xllm_latent_norm(const void* q, const void* q_w, void* q_out, int q_rank, int q_pad, const void* c, const void* c_w,
+                              void* cache, int rank, int width, const void* slots, int64_t ld, int tokens, float eps, int dtype,
+                              void* stream) {
+  using namespace xllm;
+  using namespace xllm::mla;
+  if (tokens == 0) return 0;
+  if (q_rank <= 0 || q_pad < q_rank || (c != nullptr && (rank <= 0 || width < rank || cache == nullptr || slots == nullptr)))
+    return (int)cudaErrorInvalidValue;
+  const auto run = [&](auto tag) {
+    using T = decltype(tag);
+    LatentNormParams<T> p{(const T*)q, (const T*)c, (const T*)q_w, (const T*)c_w, (T*)q_out, (T*)cache, (const int32_t*)slots, ld,
+                          q_rank, q_pad, rank, width, eps};
+    const auto al = [](const void* x) { return (((uintptr_t)x) & 15) == 0; };
+    const dim3 grid(tokens, c != nullptr ? 2 : 1);
+    if (q_rank % 8 == 0 && q_pad % 8 == 0 && ld % 8 == 0 && al(q) && al(q_w) && al(q_out) &&
+        (c == nullptr || (rank % 8 == 0 && width % 8 == 0 && al(c) && al(c_w) && al(cache))))
+      launch_pdl(latent_norm_kernel<T, 8>, grid, dim3(128), 0, (cudaStream_t)stream, p);
+    else
+      launch_pdl(latent_norm_kernel<T, 1>, grid, dim3(128), 0, (cudaStream_t)stream, p);
+  };
+  if (dtype == 0) run(bf16());
+  else run(float());
+  return XLLM_LAUNCH_CHECK();
+}
+
+// out [n_seqs * rows_per, width] bf16: the first kv_lens[s] rows of sequence s from the cache, then zeros.
+XLLM_API int xllm_latent_gather(void* out, const void* cache, const void* block_table, int bt_stride, const void* kv_lens,
+                                int n_seqs, int rows_per, int page, int width, void* stream) {
+  using namespace xllm;
+  using namespace xllm::mla;
+  if (n_seqs == 0 || rows_per == 0) return 0;
+  if (width % 8 || page <= 0 || (((uintptr_t)out | (uintptr_t)cache) & 15)) return (int)cudaErrorInvalidValue;
+  launch_pdl(latent_gather_kernel, dim3((rows_per + 7) / 8, n_seqs), dim3(256), 0, (cudaStream_t)stream, (uint4*)out,
+             (const uint4*)cache, (const int32_t*)block_table, bt_stride, (const int32_t*)kv_lens, rows_per, page, width / 8);
+  return XLLM_LAUNCH_CHECK();
 }
 
 // Latent-cache write fused with the rotary embeddings of a step's tokens (see the kernel's comment).

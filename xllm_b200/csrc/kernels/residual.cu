@@ -1,6 +1,6 @@
 // An fp32 residual stream: branch outputs join it and the next sublayer's input leaves it in one pass.
 //
-//   x[t] = (init ? 0 : x[t]) + coef * sum_i n_i(y_i[t])        n_i: identity, or RMS norm with a weight
+//   x[t] = (init ? 0 : x[t]) + n(coef * sum_i n_i(y_i[t]))     n_i: identity, or RMS norm with a weight; n likewise
 //   out[t] = rmsnorm(x[t]) * (w + offset)   or   cast(x[t])       offset: 1 for weights stored around zero
 //
 // One launch covers: the embedding (init, y_0 gathered by token id) + first norm; a plain branch + the
@@ -20,6 +20,7 @@ struct ResidualParams {
   float* x;               // [T, hidden] fp32, dense
   const void* y[2];       // branches, row stride y_ld[i] elements
   const void* w[2];       // norm weight of branch i, or null
+  const void* w_sum;      // norm weight of the branches' sum, or null
   const int64_t* rows;    // y[0] row of token t is rows[t] (embedding), or null
   const void* w_out;      // norm weight of the output, or null: cast
   void* out;              // [T, hidden] dense, or null
@@ -48,7 +49,7 @@ __device__ __forceinline__ float row_sum(float v, float* red) {
   return v;
 }
 
-template <typename T, int V, int TPR, int NB>
+template <typename T, int V, int TPR, int NB, bool NORM_SUM>
 __global__ void __launch_bounds__(TPR > 256 ? TPR : 256) residual_kernel(ResidualParams p) {
   __shared__ float red[32];
   const int t = threadIdx.x % TPR;
@@ -108,7 +109,29 @@ __global__ void __launch_bounds__(TPR > 256 ? TPR : 256) residual_kernel(Residua
         for (int j = 0; j < V; ++j) w[j] = 1.f;
       }
 #pragma unroll
-      for (int j = 0; j < V; ++j) acc[i][j] += br[b][i][j] * inv * w[j];
+      for (int j = 0; j < V; ++j) {
+        const float z = br[b][i][j] * inv * w[j];
+        if (!NORM_SUM) acc[i][j] += z;
+        else if (b == 0) br[0][i][j] = z;
+        else br[0][i][j] += z;
+      }
+    }
+  }
+  if constexpr (NORM_SUM) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kResVec; ++i)
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += br[0][i][j] * br[0][i][j];
+    const float inv = 1.f / sqrtf(row_sum<TPR>(ss, red) / (float)p.hidden + p.eps);
+#pragma unroll
+    for (int i = 0; i < kResVec; ++i) {
+      const int v = t + i * TPR;
+      if (!(live && v < nvec)) continue;
+      float w[V];
+      load_f32<V>(reinterpret_cast<const T*>(p.w_sum) + v * V, w);
+#pragma unroll
+      for (int j = 0; j < V; ++j) acc[i][j] += br[0][i][j] * inv * w[j];
     }
   }
   float ss = 0.f;
@@ -144,7 +167,7 @@ __global__ void __launch_bounds__(TPR > 256 ? TPR : 256) residual_kernel(Residua
   }
 }
 
-template <typename T, int V, int NB>
+template <typename T, int V, int NB, bool NORM_SUM = false>
 static int launch_residual(const ResidualParams& p, cudaStream_t s) {
   const int nvec = p.hidden / V;
   int tpr = 32;
@@ -155,7 +178,7 @@ static int launch_residual(const ResidualParams& p, cudaStream_t s) {
   const dim3 grid((unsigned)((p.tokens + rows - 1) / rows));
 #define XLLM_RES_CASE(N)                                                              \
   case N:                                                                             \
-    launch_pdl(residual_kernel<T, V, N, NB>, grid, dim3(block), 0, s, p);             \
+    launch_pdl(residual_kernel<T, V, N, NB, NORM_SUM>, grid, dim3(block), 0, s, p);             \
     break;
   switch (tpr) {
     XLLM_RES_CASE(32)
@@ -200,38 +223,51 @@ __global__ void __launch_bounds__(256) gelu_mul_rows_kernel(T* __restrict__ out,
   }
 }
 
-// out[t, i] = silu(x[t, i]) * x[t, d + i], fp32
+// out[t, i] = silu(x[t, i]) * x[t, d + i], fp32; limit > 0: the clamped form of clamped_glu
 __global__ void __launch_bounds__(256) silu_mul_f32_kernel(float* __restrict__ out, const float* __restrict__ x, int64_t tokens,
-                                                           int d, int64_t x_ld) {
+                                                           int d, int64_t x_ld, float limit, float alpha) {
   pdl_wait();
   pdl_launch_dependents();
   const int64_t total = tokens * d;
   for (int64_t n = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; n < total; n += (int64_t)gridDim.x * blockDim.x) {
     const int64_t t = n / d;
     const int i = (int)(n - t * d);
-    const float z = x[t * x_ld + i];
-    out[n] = z / (1.f + expf(-z)) * x[t * x_ld + d + i];
+    float z = x[t * x_ld + i], u = x[t * x_ld + d + i];
+    if (limit > 0.f) {
+      z = fminf(z, limit);
+      out[n] = z / (1.f + expf(-alpha * z)) * (fminf(fmaxf(u, -limit), limit) + 1.f);
+    } else {
+      out[n] = z / (1.f + expf(-z)) * u;
+    }
   }
 }
 
 }  // namespace xllm
 
-// dtype: 0 bf16, 1 fp32 (branches, weights, out).  y1 / w0 / w1 / rows / w_out / out may be null.
+// dtype: 0 bf16, 1 fp32 (branches, weights, out).  y1 / w0 / w1 / w_sum / rows / w_out / out may be null.
 XLLM_API int xllm_residual_update(void* x, const void* y0, int64_t y0_ld, const void* w0, const void* y1, int64_t y1_ld,
-                                  const void* w1, const void* rows, int64_t n_rows, const void* w_out, void* out, int tokens,
+                                  const void* w1, const void* w_sum, const void* rows, int64_t n_rows, const void* w_out, void* out, int tokens,
                                   int hidden, int init, float coef, float eps, float w_out_offset, int dtype,
                                   void* stream) {
   using namespace xllm;
   if (tokens == 0) return 0;
   if (hidden <= 0 || y0 == nullptr || x == nullptr) return (int)cudaErrorInvalidValue;
   ResidualParams p;
-  p.x = (float*)x; p.y[0] = y0; p.y[1] = y1; p.w[0] = w0; p.w[1] = w1; p.rows = (const int64_t*)rows;
+  p.x = (float*)x; p.y[0] = y0; p.y[1] = y1; p.w[0] = w0; p.w[1] = w1; p.w_sum = w_sum; p.rows = (const int64_t*)rows;
   p.w_out = w_out; p.out = out; p.y_ld[0] = y0_ld; p.y_ld[1] = y1_ld; p.n_rows = n_rows; p.tokens = tokens;
   p.hidden = hidden; p.init = init; p.coef = coef; p.eps = eps; p.w_out_offset = w_out_offset;
   const auto a16 = [](const void* q) { return (((uintptr_t)q) & 15) == 0; };
-  const bool al = a16(x) && a16(y0) && a16(w0) && a16(y1) && a16(w1) && a16(w_out) && a16(out);
+  const bool al = a16(x) && a16(y0) && a16(w0) && a16(y1) && a16(w1) && a16(w_sum) && a16(w_out) && a16(out);
   cudaStream_t s = (cudaStream_t)stream;
   const bool v8 = al && hidden % 8 == 0 && y0_ld % 8 == 0 && y1_ld % 8 == 0;
+  if (w_sum != nullptr) {
+    if (dtype == 0) {
+      if (v8) return y1 ? launch_residual<bf16, 8, 2, true>(p, s) : launch_residual<bf16, 8, 1, true>(p, s);
+      return y1 ? launch_residual<bf16, 1, 2, true>(p, s) : launch_residual<bf16, 1, 1, true>(p, s);
+    }
+    if (v8) return y1 ? launch_residual<float, 8, 2, true>(p, s) : launch_residual<float, 8, 1, true>(p, s);
+    return y1 ? launch_residual<float, 1, 2, true>(p, s) : launch_residual<float, 1, 1, true>(p, s);
+  }
   if (dtype == 0) {
     if (v8) return y1 ? launch_residual<bf16, 8, 2>(p, s) : launch_residual<bf16, 8, 1>(p, s);
     return y1 ? launch_residual<bf16, 1, 2>(p, s) : launch_residual<bf16, 1, 1>(p, s);
@@ -267,11 +303,12 @@ XLLM_API int xllm_gelu_mul_rows(void* out, const void* gate, int64_t gate_ld, co
   return XLLM_LAUNCH_CHECK();
 }
 
-XLLM_API int xllm_silu_mul_f32(void* out, const void* x, int64_t tokens, int d, int64_t x_ld, void* stream) {
+XLLM_API int xllm_silu_mul_f32(void* out, const void* x, int64_t tokens, int d, int64_t x_ld, float limit, float alpha,
+                               void* stream) {
   using namespace xllm;
   if (tokens == 0) return 0;
   const int64_t want = (tokens * d + 255) / 256;
   launch_pdl(silu_mul_f32_kernel, dim3((unsigned)(want < 148 * 8 ? want : 148 * 8)), dim3(256), 0, (cudaStream_t)stream,
-             (float*)out, (const float*)x, tokens, d, x_ld);
+             (float*)out, (const float*)x, tokens, d, x_ld, limit, alpha);
   return XLLM_LAUNCH_CHECK();
 }

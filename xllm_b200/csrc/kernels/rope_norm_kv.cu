@@ -1,11 +1,17 @@
-// Rotary positions, then a per-head RMS norm without a weight, on q and k of packed projection rows; k goes to
-// the paged K cache and the values (any column block of the row: their own projection, or the keys as projected)
-// to the V cache.  One pass, any head size up to 512, bf16 or fp32.
+// What lies between a fused projection and paged attention, in one pass over q, k and v, any head size up to 512, bf16 or
+// fp32, every step optional:
+//   a short causal convolution over time per channel of q, k and v,
+//   a per-head RMS norm of q and k with a weight shared by the heads,
+//   rotary positions on the first `rot` elements of q and k,
+//   a per-head RMS norm of q and k without a weight.
+// k goes to the paged K cache and the values (any column block of the row: their own projection, or the keys as projected)
+// to the V cache.
 //
-// The sibling of rope_kv.cu (norm with a weight BEFORE the rotation, power-of-two head sizes).  Heads may be
-// stored wider than they are (d_pad >= d, zero filled): the attention kernels take head sizes 64, 128 and 256.
-// One warp per (token, head); a lane owns element pairs.
-#include "vec_io.cuh"
+// The sibling of rope_kv.cu (weighted norm and rotation, power-of-two head sizes).  Heads may be stored wider than they are
+// (d_pad >= d, zero filled): the attention kernels take head sizes 64, 128 and 256.  The generic kernel has one warp per
+// (token, head), a lane owns element pairs.  The convolution keeps a sequence's last inputs in a ring (short_conv.cuh); a
+// sequence with one row in the batch stores it here, longer portions in a launch behind this one.
+#include "short_conv.cuh"
 
 namespace xllm {
 
@@ -22,7 +28,42 @@ struct RopeNormParams {
   int tokens, nq, nkv, d, dv, d_pad, rot, page, interleaved, unit_norm;
   int64_t max_pos;
   float eps;
+  const T *q_w, *k_w;        // [d] weights of the norm ahead of the rotation, or null
+  // short convolution (taps 0: none); channels are q | k | v
+  const T* conv_w;           // [taps, channels], the last row belongs to the current token
+  T* ring;                   // [state slots, taps, channels]
+  const int32_t *state_slots, *cu_q, *kv_lens;      // [n_seqs], [n_seqs + 1], [n_seqs]
+  int n_seqs, taps;
+  __host__ __device__ int64_t channels() const { return (int64_t)(nq + nkv) * d + (int64_t)nkv * dv; }
 };
+
+// where a token row stands in its sequence
+struct ConvPlace {
+  int slot, back, pos, alone;          // state slot (-1: no sequence), rows of the sequence ahead of it in the batch, position
+};
+template <typename T>
+__device__ __forceinline__ ConvPlace conv_place(const RopeNormParams<T>& p, int row) {
+  ConvPlace c{-1, 0, 0, 0};
+  const int b = seq_of_row(p.cu_q, p.n_seqs, row);
+  if (b < 0 || p.kv_lens[b] <= 0) return c;
+  c.slot = p.state_slots[b];
+  c.back = row - p.cu_q[b];
+  c.pos = p.kv_lens[b] - (p.cu_q[b + 1] - row);
+  c.alone = p.cu_q[b + 1] - p.cu_q[b] == 1;
+  return c;
+}
+// one channel of one row behind the convolution; x: its place in the row, ch: its number among the channels
+template <typename T>
+__device__ __forceinline__ float conv_one(const RopeNormParams<T>& p, const ConvPlace& c, const T* x, int64_t ch) {
+  if (c.slot < 0) return 0.f;
+  const int64_t C = p.channels();
+  T* ring = p.ring + (int64_t)c.slot * p.taps * C + ch;
+  float y = 0.f;
+  for (int b = 0; b < p.taps && b <= c.pos; ++b)
+    y += to_f32(b <= c.back ? x[-b * p.ld] : ring[(c.pos - b) % p.taps * C]) * to_f32(p.conv_w[(p.taps - 1 - b) * C + ch]);
+  if (c.alone) ring[c.pos % p.taps * C] = x[0];
+  return y;
+}
 
 constexpr int kPairs = 8;   // pairs per lane: d <= 512
 
@@ -39,6 +80,12 @@ __global__ void __launch_bounds__(256) rope_norm_kv_kernel(RopeNormParams<T> p) 
   const bool is_q = h < p.nq;
   const int g = is_q ? h : h - p.nq;
   const T* src = (is_q ? p.q : p.k) + t * p.ld + (int64_t)g * p.d;
+  const bool conv = p.taps > 0;
+  const int64_t ch = (int64_t)h * p.d;
+  ConvPlace place{};
+  if (conv) place = conv_place(p, (int)t);
+  const auto in = [&](int i) { return conv ? conv_one(p, place, src + i, ch + i) : to_f32(src[i]); };
+  const T* w = is_q ? p.q_w : p.k_w;
   const int half = p.rot >> 1;
   const float* cs = nullptr;
   if (p.cos_sin != nullptr) {
@@ -58,40 +105,63 @@ __global__ void __launch_bounds__(256) rope_norm_kv_kernel(RopeNormParams<T> p) 
     int i0, i1;
     if (n < half && !p.interleaved) { i0 = n; i1 = n + half; }
     else { i0 = 2 * n; i1 = 2 * n + 1; }
-    float u = to_f32(src[i0]), v = i1 < p.d ? to_f32(src[i1]) : 0.f;
+    a[i] = in(i0);
+    b[i] = i1 < p.d ? in(i1) : 0.f;
+    ss += a[i] * a[i] + b[i] * b[i];
+  }
+  if (w != nullptr) {
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)p.d + p.eps);
+#pragma unroll
+    for (int i = 0; i < kPairs; ++i) {
+      const int n = lane + 32 * i;
+      if (n >= n_pairs) continue;
+      const bool split = n < half && !p.interleaved;
+      const int i0 = split ? n : 2 * n, i1 = split ? n + half : 2 * n + 1;
+      a[i] *= inv * to_f32(w[i0]);
+      if (i1 < p.d) b[i] *= inv * to_f32(w[i1]);
+    }
+  }
+  ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < kPairs; ++i) {
+    const int n = lane + 32 * i;
     if (n < half && cs != nullptr) {
       const float c = cs[n], s = cs[half + n];
-      const float u2 = u * c - v * s;
-      v = v * c + u * s;
-      u = u2;
+      const float u = a[i], v = b[i];
+      a[i] = u * c - v * s;
+      b[i] = v * c + u * s;
     }
-    a[i] = u;
-    b[i] = v;
-    ss += u * u + v * v;
+    ss += a[i] * a[i] + b[i] * b[i];
   }
   float inv = 1.f;
   if (p.unit_norm) inv = 1.f / sqrtf(warp_sum(ss) / (float)p.d + p.eps);
   const int slot = is_q ? 0 : p.slots[t];
-  if (!is_q && slot < 0) return;
-  const int64_t blk = slot / p.page;
+  if (!is_q && slot < 0 && !conv) return;
+  const bool cached = is_q || slot >= 0;
+  const int64_t blk = slot < 0 ? 0 : slot / p.page;
   const int off = slot - (int)blk * p.page;
   const int64_t crow = ((blk * p.nkv + g) * p.page + off) * (int64_t)p.d_pad;
   T* dst = is_q ? p.q_out + (t * p.nq + g) * p.d_pad : p.k_cache + crow;
 #pragma unroll
   for (int i = 0; i < kPairs; ++i) {
     const int n = lane + 32 * i;
-    if (n >= n_pairs) continue;
+    if (n >= n_pairs || !cached) continue;
     int i0, i1;
     if (n < half && !p.interleaved) { i0 = n; i1 = n + half; }
     else { i0 = 2 * n; i1 = 2 * n + 1; }
     dst[i0] = from_f32<T>(a[i] * inv);
     if (i1 < p.d) dst[i1] = from_f32<T>(b[i] * inv);
   }
-  for (int i = p.d + lane; i < p.d_pad; i += 32) dst[i] = from_f32<T>(0.f);
+  for (int i = p.d + lane; i < p.d_pad && cached; i += 32) dst[i] = from_f32<T>(0.f);
   if (!is_q) {
     const T* vs = p.v + t * p.ld + (int64_t)g * p.dv;
+    const int64_t vch = (int64_t)(p.nq + p.nkv) * p.d + (int64_t)g * p.dv;
     T* vd = p.v_cache + crow;
-    for (int i = lane; i < p.d_pad; i += 32) vd[i] = i < p.dv ? vs[i] : from_f32<T>(0.f);
+    for (int i = lane; i < p.d_pad; i += 32) {
+      T v = from_f32<T>(0.f);
+      if (i < p.dv) v = conv ? from_f32<T>(conv_one(p, place, vs + i, vch + i)) : vs[i];
+      if (cached) vd[i] = v;
+    }
   }
 }
 
@@ -132,7 +202,7 @@ __global__ void __launch_bounds__(256) rope_norm_kv_vec_kernel(RopeNormParams<bf
       if (h >= heads) continue;
       const bool is_q = h < p.nq;
       raw[u] = *reinterpret_cast<const bf16x8*>((is_q ? p.q : p.k) + t * p.ld + (int64_t)(is_q ? h : h - p.nq) * p.d + e0);
-      if (!is_q && p.v != p.k)
+      if (!is_q && p.v != p.k && p.dv == p.d)
         val[u] = *reinterpret_cast<const bf16x8*>(p.v + t * p.ld + (int64_t)(h - p.nq) * p.d + e0);
     }
 #pragma unroll
@@ -143,6 +213,17 @@ __global__ void __launch_bounds__(256) rope_norm_kv_vec_kernel(RopeNormParams<bf
 #pragma unroll
       for (int j = 0; j < 8; ++j) x[j] = 0.f;
       if (active) unpack8(raw[u], x);
+      if (p.q_w != nullptr) {
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ss += x[j] * x[j];
+        for (int o = tph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float inv = 1.f / sqrtf(ss / (float)p.d + p.eps);
+        float w[8];
+        load_f32<8>((h < p.nq ? p.q_w : p.k_w) + e0, w);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[j] *= inv * w[j];
+      }
       if (p.cos_sin != nullptr) {
         if (p.interleaved) {
           if (turns) {
@@ -179,25 +260,164 @@ __global__ void __launch_bounds__(256) rope_norm_kv_vec_kernel(RopeNormParams<bf
       const int64_t crow = ((blk * p.nkv + kvh) * p.page + off) * (int64_t)p.d_pad;
       bf16* dst = is_q ? p.q_out + (t * p.nq + h) * p.d_pad : p.k_cache + crow;
       *reinterpret_cast<bf16x8*>(dst + e0) = pack8(x);
-      if (!is_q) *reinterpret_cast<bf16x8*>(p.v_cache + crow + e0) = p.v != p.k ? val[u] : raw[u];
+      if (!is_q && p.dv == p.d) *reinterpret_cast<bf16x8*>(p.v_cache + crow + e0) = p.v != p.k ? val[u] : raw[u];
       for (int z = p.d + e0; z < p.d_pad; z += p.d) {
         *reinterpret_cast<uint4*>(dst + z) = make_uint4(0, 0, 0, 0);
-        if (!is_q) *reinterpret_cast<uint4*>(p.v_cache + crow + z) = make_uint4(0, 0, 0, 0);
+        if (!is_q && p.dv == p.d) *reinterpret_cast<uint4*>(p.v_cache + crow + z) = make_uint4(0, 0, 0, 0);
       }
     }
   }
+  if (p.dv == p.d || slot < 0) return;
+  const int vph = p.d_pad >> 3;                        // vectors of a stored value head
+  for (int n = threadIdx.x; n < p.nkv * vph; n += 256) {
+    const int h = n / vph, e = (n - h * vph) * 8;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (e < p.dv) v = *reinterpret_cast<const uint4*>(p.v + t * p.ld + (int64_t)h * p.dv + e);
+    *reinterpret_cast<uint4*>(p.v_cache + ((blk * p.nkv + h) * p.page + off) * (int64_t)p.d_pad + e) = v;
+  }
+}
+
+// The same sizes behind a convolution of up to four taps (rotate-half layout, no weightless norm): a CTA takes RUN token
+// rows and 256 vectors of eight channels, a thread reads every input of its vector once and keeps the last ones in
+// registers.  grid (runs, parts): the first `qk_parts` parts are q and k, the others v.
+constexpr int kMaxTaps = 4;
+
+template <int RUN>
+__global__ void __launch_bounds__(256) conv_rope_kv_kernel(RopeNormParams<bf16> p, int qk_parts) {
+  __shared__ ConvPlace place[RUN];
+  __shared__ int cache_slot[RUN];
+  __shared__ int64_t angle_row[RUN];
+  const int first = blockIdx.x * RUN;
+  pdl_wait();
+  pdl_launch_dependents();
+  if (threadIdx.x < RUN) {
+    const int row = first + threadIdx.x;
+    ConvPlace c{-1, 0, 0, 0};
+    int cs = -1;
+    int64_t pos = 0;
+    if (row < p.tokens) {
+      c = conv_place(p, row);
+      cs = p.slots[row];
+      if (p.cos_sin != nullptr) pos = p.positions[row];
+    }
+    place[threadIdx.x] = c;
+    cache_slot[threadIdx.x] = cs;
+    angle_row[threadIdx.x] = (pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos)) * p.rot;
+  }
+  const bool is_v = (int)blockIdx.y >= qk_parts;
+  const int size = is_v ? p.dv : p.d, per = size >> 3;               // vectors of a head
+  const int n = ((int)blockIdx.y - (is_v ? qk_parts : 0)) * 256 + threadIdx.x;
+  const int heads = is_v ? p.nkv : p.nq + p.nkv;
+  const bool on = n < heads * per;                                   // whole heads are on or not together
+  const int h = on ? n / per : 0, e0 = on ? (n - h * per) * 8 : 0;
+  const bool is_q = !is_v && h < p.nq;
+  const int kvh = is_v ? h : h - p.nq;
+  const int64_t C = p.channels(), ch = (is_v ? (int64_t)(p.nq + p.nkv) * p.d : 0) + (int64_t)h * size + e0;
+  const bf16* x = (is_v ? p.v + (int64_t)h * size : (is_q ? p.q + (int64_t)h * size : p.k + (int64_t)kvh * size)) + e0;
+  bf16x8 in[RUN + kMaxTaps - 1], w[kMaxTaps];
+#pragma unroll
+  for (int r = 0; r < RUN + kMaxTaps - 1; ++r) {
+    const int row = first + r - (kMaxTaps - 1);
+    const bool need = on && row >= 0 && row < p.tokens && r + p.taps >= kMaxTaps;
+    in[r] = need ? *reinterpret_cast<const bf16x8*>(x + row * p.ld) : bf16x8{};
+  }
+#pragma unroll
+  for (int b = 0; b < kMaxTaps; ++b)
+    w[b] = on && b < p.taps ? *reinterpret_cast<const bf16x8*>(p.conv_w + (p.taps - 1 - b) * C + ch) : bf16x8{};
+  const bf16* nw = is_v ? nullptr : (is_q ? p.q_w : p.k_w);
+  const int half = p.rot >> 1;
+  const bool turns = !is_v && p.cos_sin != nullptr && e0 < p.rot;
+  __syncthreads();
+#pragma unroll
+  for (int r = 0; r < RUN; ++r) {
+    const int row = first + r;
+    if (row >= p.tokens) break;
+    const ConvPlace c = place[r];
+    float y[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) y[j] = 0.f;
+    if (on && c.slot >= 0) {
+      bf16* ring = p.ring + (int64_t)c.slot * p.taps * C + ch;
+#pragma unroll
+      for (int b = 0; b < kMaxTaps; ++b) {
+        if (b >= p.taps || b > c.pos) break;
+        float u[8], f[8];
+        if (b <= c.back) unpack8(in[r + kMaxTaps - 1 - b], u);
+        else load_f32<8>(ring + (c.pos - b) % p.taps * C, u);
+        unpack8(w[b], f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) y[j] += u[j] * f[j];
+      }
+      if (c.alone) *reinterpret_cast<bf16x8*>(ring + c.pos % p.taps * C) = in[r + kMaxTaps - 1];
+    }
+    const int cs = cache_slot[r];
+    const int64_t blk = cs < 0 ? 0 : cs / p.page;
+    const int64_t crow = ((blk * p.nkv + kvh) * p.page + (cs - (int)blk * p.page)) * (int64_t)p.d_pad;
+    if (!is_v) {
+      if (p.q_w != nullptr) {
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ss += y[j] * y[j];
+        for (int o = per >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float inv = 1.f / sqrtf(ss / (float)p.d + p.eps);
+        float f[8];
+        load_f32<8>(nw + e0, f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) y[j] *= inv * f[j];
+      }
+      if (p.cos_sin != nullptr) {
+        float other[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) other[j] = __shfl_xor_sync(0xffffffffu, y[j], half >> 3);
+        if (turns) {
+          float co[8], si[8];
+          const float* a = p.cos_sin + angle_row[r] + (e0 < half ? e0 : e0 - half);
+          load_f32<8>(a, co);
+          load_f32<8>(a + half, si);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) y[j] = e0 < half ? y[j] * co[j] - other[j] * si[j] : y[j] * co[j] + other[j] * si[j];
+        }
+      }
+    }
+    if (!on || (!is_q && cs < 0)) continue;
+    bf16* dst = is_v ? p.v_cache + crow : (is_q ? p.q_out + ((int64_t)row * p.nq + h) * p.d_pad : p.k_cache + crow);
+    *reinterpret_cast<bf16x8*>(dst + e0) = pack8(y);
+    for (int z = size + e0; z < p.d_pad; z += size) *reinterpret_cast<uint4*>(dst + z) = make_uint4(0, 0, 0, 0);
+  }
+}
+
+// the last inputs of every sequence with more than one row in the batch
+template <typename T>
+__global__ void __launch_bounds__(256) conv_keep_kernel(RopeNormParams<T> p) {
+  const int b = blockIdx.y;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int first = p.cu_q[b], n = p.cu_q[b + 1] - first, slot = p.state_slots[b];
+  const int64_t c = (int64_t)blockIdx.x * 256 + threadIdx.x, C = p.channels();
+  if (n <= 1 || slot < 0 || c >= C) return;
+  const int64_t q_end = (int64_t)p.nq * p.d, k_end = q_end + (int64_t)p.nkv * p.d;
+  const T* x = c < q_end ? p.q + c : (c < k_end ? p.k + c - q_end : p.v + c - k_end);
+  for (int i = max(0, n - (p.taps - 1)); i < n; ++i)
+    p.ring[((int64_t)slot * p.taps + (p.kv_lens[b] - n + i) % p.taps) * C + c] = x[(int64_t)(first + i) * p.ld];
 }
 
 }  // namespace xllm
 
 // dtype: 0 bf16, 1 fp32.  rot <= d, rot even.  dv: size of a value head (d where v is the key block).
+// q_w, k_w: both or neither.  taps > 0: the convolution; conv_w .. kv_lens as in RopeNormParams, over all rows of the batch;
+// long_portions: some sequence may have more than one row.
 XLLM_API int xllm_rope_norm_kv(const void* q, const void* k, const void* v, int64_t ld, void* q_out, void* k_cache,
                                void* v_cache, const void* cos_sin, int64_t max_pos, const void* positions, const void* slots,
                                int tokens, int nq, int nkv, int d, int dv, int d_pad, int rot, int page, int interleaved, int unit_norm,
-                               float eps, int dtype, void* stream) {
+                               float eps, const void* q_w, const void* k_w, const void* conv_w, void* ring, const void* state_slots,
+                               const void* cu_q, const void* kv_lens, int n_seqs, int taps, int long_portions, int dtype,
+                               void* stream) {
   using namespace xllm;
   if (tokens == 0) return 0;
-  if (d <= 0 || d > 64 * kPairs || d_pad < d || dv <= 0 || d_pad < dv || rot < 0 || rot > d || rot % 2 != 0 || page <= 0 || nq <= 0 || nkv <= 0)
+  if (d <= 0 || d > 64 * kPairs || d_pad < d || dv <= 0 || d_pad < dv || rot < 0 || rot > d || rot % 2 != 0 || page <= 0 || nq <= 0 || nkv <= 0 || (q_w == nullptr) != (k_w == nullptr))
+    return (int)cudaErrorInvalidValue;
+  if (taps < 0 || (taps > 0 && (conv_w == nullptr || ring == nullptr || state_slots == nullptr || cu_q == nullptr ||
+                                kv_lens == nullptr || n_seqs <= 0)))
     return (int)cudaErrorInvalidValue;
   const int64_t items = (int64_t)tokens * (nq + nkv);
   const dim3 grid((unsigned)((items + 7) / 8)), block(256);
@@ -209,17 +429,34 @@ XLLM_API int xllm_rope_norm_kv(const void* q, const void* k, const void* v, int6
     p.v_cache = (T*)v_cache; p.cos_sin = rot > 0 ? (const float*)cos_sin : nullptr; p.positions = (const int64_t*)positions;
     p.slots = (const int32_t*)slots; p.tokens = tokens; p.nq = nq; p.nkv = nkv; p.d = d; p.dv = dv; p.d_pad = d_pad; p.rot = rot;
     p.page = page; p.interleaved = interleaved; p.unit_norm = unit_norm; p.max_pos = max_pos; p.eps = eps;
+    p.q_w = (const T*)q_w; p.k_w = (const T*)k_w; p.conv_w = (const T*)conv_w; p.ring = (T*)ring;
+    p.state_slots = (const int32_t*)state_slots; p.cu_q = (const int32_t*)cu_q; p.kv_lens = (const int32_t*)kv_lens;
+    p.n_seqs = n_seqs; p.taps = taps;
+    const auto keep = [&] {
+      if (taps > 1 && long_portions)
+        launch_pdl(conv_keep_kernel<T>, dim3((unsigned)((p.channels() + 255) / 256), n_seqs), dim3(256), 0, s, p);
+    };
     if constexpr (sizeof(T) == 2) {
       const auto a16 = [](const void* x) { return (((uintptr_t)x) & 15) == 0; };
       const int tph = d >> 3, hl = rot >> 4;
-      if (d % 8 == 0 && d == dv && d <= 256 && (tph & (tph - 1)) == 0 && d_pad % 8 == 0 && ld % 8 == 0 && a16(q) && a16(k) && a16(v) &&
-          a16(q_out) && a16(k_cache) && a16(v_cache) && (rot == 0 || (rot % 8 == 0 && a16(cos_sin))) &&
+      if (d % 8 == 0 && dv % 8 == 0 && d <= 256 && (tph & (tph - 1)) == 0 && d_pad % 8 == 0 && ld % 8 == 0 && a16(q) && a16(k) && a16(v) &&
+          a16(q_out) && a16(k_cache) && a16(v_cache) && (rot == 0 || (rot % 8 == 0 && a16(cos_sin))) && a16(q_w) && a16(k_w) &&
           (interleaved || rot == 0 || (rot % 16 == 0 && (hl & (hl - 1)) == 0))) {
-        launch_pdl(rope_norm_kv_vec_kernel, dim3(tokens), dim3(256), 0, s, p);
-        return;
+        if (taps == 0) {
+          launch_pdl(rope_norm_kv_vec_kernel, dim3(tokens), dim3(256), 0, s, p);
+          return;
+        }
+        if (taps <= kMaxTaps && !unit_norm && !(interleaved && rot > 0) && a16(conv_w) && a16(ring)) {
+          const int qk = ((nq + nkv) * tph + 255) / 256, parts = qk + (nkv * (dv >> 3) + 255) / 256;
+          if (long_portions) launch_pdl(conv_rope_kv_kernel<4>, dim3((tokens + 3) / 4, parts), dim3(256), 0, s, p, qk);
+          else launch_pdl(conv_rope_kv_kernel<1>, dim3(tokens, parts), dim3(256), 0, s, p, qk);
+          keep();
+          return;
+        }
       }
     }
     launch_pdl(rope_norm_kv_kernel<T>, grid, block, 0, s, p);
+    keep();
   };
   if (dtype == 0) run(bf16());
   else run(float());

@@ -189,7 +189,8 @@ PYBIND11_MODULE(_rt, m) {
       .def_readwrite("max_prefill_wait_steps", &SchedulerConfig::max_prefill_wait_steps)
       .def_readwrite("hold_finished_blocks", &SchedulerConfig::hold_finished_blocks)
       .def_readwrite("admission", &SchedulerConfig::admission)
-      .def_readwrite("sliding_window", &SchedulerConfig::sliding_window);
+      .def_readwrite("sliding_window", &SchedulerConfig::sliding_window)
+      .def_readwrite("sliding_window_keep", &SchedulerConfig::sliding_window_keep);
 
   py::enum_<PauseMode>(m, "PauseMode")
       .value("KEEP", PauseMode::KEEP)

@@ -55,6 +55,8 @@ struct SchedulerConfig {
   // Sliding-window attention in every layer: KV blocks that lie entirely before the window of the
   // next query are given back while the sequence runs (0 = full attention)
   int32_t sliding_window = 0;
+  // ... but for the blocks of the first `sliding_window_keep` positions, which every query sees.
+  int32_t sliding_window_keep = 0;
   std::string priority_strategy = "fcfs";
   double prefill_scheduling_memory_usage_threshold = 0.95;
   bool enable_schedule_overlap = false;
@@ -653,8 +655,9 @@ class Scheduler {
     if (cfg_.sliding_window <= 0 || s->in_flight > 0) return;
     const int32_t dead = (s->kv_computed - cfg_.sliding_window + 1) / cfg_.block_size;
     if (dead <= s->window_released) return;
+    const int32_t kept = (cfg_.sliding_window_keep + cfg_.block_size - 1) / cfg_.block_size;
     std::vector<int32_t> give;
-    for (int32_t i = s->window_released; i < dead && i < (int32_t)s->blocks.size(); ++i) {
+    for (int32_t i = std::max(s->window_released, kept); i < dead && i < (int32_t)s->blocks.size(); ++i) {
       if (s->blocks[i] > 0) give.push_back(s->blocks[i]);
       s->blocks[i] = 0;
     }

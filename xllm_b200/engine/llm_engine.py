@@ -232,6 +232,7 @@ class LLMEngine:
         # sliding-window models (the window in every layer) give dead blocks back while they run
         if int(getattr(self.args, "sliding_window", 0) or 0) > 0 and not getattr(self.model, "mixed_window_layers", False):
             sc.sliding_window = int(self.args.sliding_window)
+            sc.sliding_window_keep = int(self.args.extra.get("sliding_window_keep", 0))     # first tokens that stay visible
         sc.priority_strategy = cfg.priority_strategy
         sc.enable_schedule_overlap = cfg.enable_schedule_overlap
         sc.dp_size = 1  # one scheduler instance per DP replica

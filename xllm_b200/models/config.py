@@ -166,8 +166,35 @@ def _sodedra_args(cfg: Dict[str, Any], shapes: Dict[str, List[int]]) -> ModelArg
     return a
 
 
+def _lukinex_args(cfg: Dict[str, Any], shapes: Dict[str, List[int]]) -> ModelArgs:
+    """Lukinex configurations list every layer; nothing is left to a tensor's shape."""
+    import copy
+    layers = copy.deepcopy(cfg["layers"])
+    a = ModelArgs(model_type="lukinex", architectures=["Lukinex"], vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
+                  num_hidden_layers=len(layers), rms_norm_eps=float(cfg["norm"]["eps"]), qk_norm=False, tie_word_embeddings=False)
+    att = [l["mixer"]["left"] if l["type"] == "parallel" else l["mixer"] for l in layers if l["type"] in ("parallel", "attention")]
+    latent = [l["mixer"] for l in layers if l["type"] == "latent_attention"]
+    a.num_attention_heads = max([m["heads"] for m in att + latent] + [1])
+    a.num_key_value_heads = max([m["kv_heads"] for m in att] + [1])
+    a.head_dim = max([max(m["dim"], m["vdim"]) for m in att] + [1])
+    moe = [l["mlp"] for l in layers if l.get("mlp")]
+    a.num_experts = max([m["router"]["experts"] for m in moe] + [0])
+    a.num_experts_per_tok = max([m["router"]["top"] for m in moe] + [0])
+    a.moe_intermediate_size = max([m["expert"]["ff"] for m in moe] + [0])
+    a.intermediate_size = max([m["shared"]["ff"] for m in moe] + [a.hidden_size])
+    a.max_position_embeddings = int(_g(cfg, "max_position_embeddings", default=32768))
+    a.extra = {"layers": layers, "unbounded_positions": "max_position_embeddings" not in cfg}
+    if not latent:
+        # every layer with a cache has a window: what lies between the kept first tokens and the widest one can be given back
+        a.sliding_window = max([int(m["mask"]["size"]) for m in att] + [0])
+        a.extra["sliding_window_keep"] = max([int(m["mask"].get("keep_first", 0)) for m in att] + [0])
+    a.bos_token_id = _g(cfg, "bos_token_id", default=-1)
+    a.eos_token_id, a.stop_token_ids = _eos_list(_g(cfg, "eos_token_id"))
+    return a
+
+
 # `architecture` names whose configurations do not follow the HuggingFace layout: name -> fn(config, tensor shapes)
-_OWN_LAYOUTS = {"femirax": _femirax_args, "sodedra": _sodedra_args}
+_OWN_LAYOUTS = {"femirax": _femirax_args, "sodedra": _sodedra_args, "lukinex": _lukinex_args}
 
 
 def model_args_from_dict(cfg: Dict[str, Any], shapes: Optional[Dict[str, List[int]]] = None) -> ModelArgs:

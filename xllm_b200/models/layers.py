@@ -17,7 +17,7 @@ from typing import Callable, Dict, Iterable, List, Optional, Tuple
 import torch
 
 from .. import ops
-from ..ops import reference
+from ..ops import glu, reference
 from ..parallel.state import ParallelState, single
 
 
@@ -561,7 +561,7 @@ class Attention(Module):
 
 
 class DenseMLP(Module):
-    """SwiGLU MLP: fused gate|up column-parallel GEMM -> silu·mul -> row-parallel down GEMM."""
+    """Gated MLP: fused gate|up column-parallel GEMM -> act(gate) · up -> row-parallel down GEMM (`act`: ops/glu.py)."""
 
     def __init__(self, hidden, inter, act, dtype, device, ps: ParallelState = None, reduce=True, fuse_reduce=True,
                  quant=None):
@@ -571,7 +571,7 @@ class DenseMLP(Module):
         # on a CUDA device the gate and up rows are stored interleaved, so that prompt-size batches run the
         # GEMM whose epilogue applies the gated activation (XLLM_FUSED_ACT=0 keeps the plain layout)
         il = (torch.device(device).type == "cuda" and dtype == torch.bfloat16 and quant is None
-              and act in ("silu", "gelu", "gelu_tanh", "gelu_pytorch_tanh") and os.environ.get("XLLM_FUSED_ACT", "1") != "0")
+              and glu.known(act) and os.environ.get("XLLM_FUSED_ACT", "1") != "0")
         self.gate_up = self.add_module("gate_up_proj", MergedColumnLinear(
             hidden, [inter, inter], ["gate_proj", "up_proj"], False, dtype, device, self.ps, quant=quant, interleave=il))
         self.down = self.add_module("down_proj", Linear(inter, hidden, False, dtype, device, self.ps,

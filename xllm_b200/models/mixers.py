@@ -1,6 +1,7 @@
 """Sublayers of hybrid decoders over an fp32 residual stream, with their constants as parameters: decayed linear
 attention (per-head or per-channel decay), the gated delta rule with channel decays, exponentially gated matrix memory,
-attention whose values are its keys, windowed attention with an output gate, a gated per-token side input.
+attention whose values are its keys, windowed attention with an output gate, windowed attention with kept first tokens,
+attention over cached latents, a gated per-token side input.
 
 Each mixer names its tensors as a checkpoint does (loader names relative to the mixer) and exposes
   width_parts()   the projections it needs of its input, which the owner fuses into one GEMM,
@@ -14,6 +15,7 @@ from typing import Dict, List, Tuple
 import torch
 
 from .. import ops
+from ..ops import mla
 from ..ops.delta_rule import ChannelDelta
 from ..ops.head_norm import head_gate
 from ..ops.linear_attn import LinearAttention
@@ -68,10 +70,13 @@ class FusedProjection(Module):
 
 
 class OutProjection(Module):
-    """y = x W^T where x may be wider than the checkpoint's W: heads stored zero-padded (`head`, `head_pad`)."""
+    """y = x W^T (+ b) where x may be wider than the checkpoint's W: heads stored zero-padded (`head`, `head_pad`)."""
 
-    def __init__(self, heads, head, head_pad, out_f, dtype, device):
+    def __init__(self, heads, head, head_pad, out_f, dtype, device, bias=False):
         super().__init__()
+        self.bias = None
+        if bias:
+            self.bias = self.add_param("b", torch.zeros(out_f, dtype=dtype, device=device))
         self.weight = torch.zeros(out_f, heads * head_pad, dtype=dtype, device=device)
 
         def load(w):
@@ -81,26 +86,28 @@ class OutProjection(Module):
         self._loaders["weight"] = load
 
     def forward(self, x):
-        return ops.linear(x, self.weight)
+        return ops.linear(x, self.weight, self.bias)
 
     __call__ = forward
 
 
 class LinearAttentionMixer(Module):
     """Multi-head linear attention with a decaying state and gated output: retention (`decay`: one constant per head,
-    rotated q and k) or per-channel decay (`rank` > 0: low-rank projection a1, a2 and bias a2.b, temperature tau)."""
+    rotated q and k) or per-channel decay (`rank` > 0: low-rank projection a1, a2 and bias a2.b, temperature tau).
+    `in_silu`: q, k and v pass through silu; `row_norm`: the heads are normed together with a weight per element and gated with
+    a sigmoid instead of one by one with silu."""
 
     def __init__(self, hidden, heads, dk, dv, eps, dtype, device, decay=None, rank=0, tau=1.0, q_scale=1.0, k_scale=1.0,
-                 rope: RotaryEmbedding = None, norm_weight=False, prefix=""):
+                 rope: RotaryEmbedding = None, norm_weight=False, prefix="", in_silu=False, row_norm=False):
         super().__init__()
         self.prefix, self.state_shape = prefix, (heads, dk, dv)
         self.heads, self.dv = heads, dv
         self.parts = [("q", heads * dk), ("k", heads * dk), ("v", heads * dv), ("g", heads * dv)]
-        op = LinearAttention(heads, dk, dv, q_scale=q_scale, k_scale=k_scale, eps=eps)
+        op = LinearAttention(heads, dk, dv, q_scale=q_scale, k_scale=k_scale, eps=eps, in_silu=in_silu, rows=row_norm)
         if decay is not None:
             d = torch.tensor([float(x) for x in decay], dtype=torch.float64)
             if d.numel() != heads or bool((d < 0).any()) or bool((d > 1).any()):
-                raise ValueError(f"retention needs {heads} decays in [0, 1]")
+                raise ValueError(f"linear attention needs {heads} decays in [0, 1]")
             op.log_decay = torch.log(d.clamp_min(1e-300)).to(torch.float32).to(device)
         else:
             self.parts.append(("a1", rank))
@@ -110,7 +117,7 @@ class LinearAttentionMixer(Module):
         if rope is not None:
             op.cos_sin, op.rot, op.interleaved = rope.cos_sin, rope.rot_dim, rope.interleaved
         if norm_weight:
-            op.norm_w = self.add_param("norm", torch.ones(dv, dtype=dtype, device=device))
+            op.norm_w = self.add_param("norm", torch.ones(heads * dv if row_norm else dv, dtype=dtype, device=device))
         self.op = op
         self.o = self.add_module("o", Linear(heads * dv, hidden, False, dtype, device))
 
@@ -230,6 +237,172 @@ class WindowAttention(Module):
         if self.gate:
             return self.o(head_gate(out, fused.part(rows, "g"), self.dv))
         return self.o(out[..., : self.dv].reshape(out.shape[0], self.heads * self.dv))
+
+    __call__ = forward
+
+
+class KeptWindowAttention(Module):
+    """GQA over a sliding window whose first `keep` tokens stay visible (window 0: everything before a token).  Optional: a
+    short causal convolution (`taps` > 0) on q, k and v, RMS norms of the q and k heads with weights (`qk_norm`), rotary
+    positions, a soft cap on the scores, biases on q, k, v and the output."""
+
+    def __init__(self, hidden, heads, kv_heads, d, dv, scale, window, keep, eps, dtype, device, rope: RotaryEmbedding = None,
+                 softcap=0.0, taps=0, qk_norm=False, bias=False, prefix=""):
+        super().__init__()
+        if heads % kv_heads:
+            raise ValueError("the query heads must be a multiple of the key/value heads")
+        if int(window) < 0 or int(keep) < 0 or float(softcap) < 0:
+            raise ValueError("window, kept tokens and soft cap must not be negative")
+        self.prefix, self.heads, self.kv_heads, self.d, self.dv, self.eps = prefix, heads, kv_heads, d, dv, eps
+        self.scale, self.window, self.keep, self.softcap = float(scale), int(window), int(keep), float(softcap)
+        self.rope, self.taps = rope, int(taps)
+        self.d_pad = ops.attention_head_size(max(d, dv))
+        self.o = self.add_module("o_pad", OutProjection(heads, dv, self.d_pad, hidden, dtype, device, bias))
+        self.biased = tuple(prefix + n for n in "qkv") if bias else ()
+        self.q_norm = self.k_norm = self.conv = None
+        if qk_norm:
+            self.q_norm = self.add_param("q.norm", torch.ones(d, dtype=dtype, device=device))
+            self.k_norm = self.add_param("k.norm", torch.ones(d, dtype=dtype, device=device))
+        if self.taps:
+            self.conv = self._params["conv"] = torch.zeros(self.taps, sum(w for _, w in self.width_parts()), dtype=dtype,
+                                                           device=device)
+            at = 0
+            for n, (_, c) in zip("qkv", self.width_parts()):
+                self._loaders[n + ".conv"] = lambda w, o=at, c=c: self.conv[:, o:o + c].copy_(w.reshape(c, self.taps).T.to(dtype))
+                at += c
+
+    def named_loaders(self, prefix=""):
+        for n, f in super().named_loaders(prefix):
+            yield n.replace("o_pad.", "o."), f
+
+    def width_parts(self):
+        return [(self.prefix + "q", self.heads * self.d), (self.prefix + "k", self.kv_heads * self.d),
+                (self.prefix + "v", self.kv_heads * self.dv)]
+
+    def kv_geometry(self):
+        return (2, self.kv_heads, self.d_pad)
+
+    def state_parts(self):
+        return {"conv": (tuple(self.conv.shape), self.conv.dtype)} if self.conv is not None else {}
+
+    def forward(self, fused: FusedProjection, rows, positions, meta: AttentionMetadata, kv, state):
+        q, k, v = (fused.part(rows, self.prefix + n) for n in "qkv")
+        rope, (k_cache, v_cache) = self.rope, kv
+        conv = None
+        if self.conv is not None:
+            conv = (self.conv, state["conv"], meta.state_slots, meta.cu_q, meta.kv_lens)
+        q = ops.rope_norm_kv_write(q, k, v, self.heads, self.kv_heads, self.d, positions, rope.cos_sin if rope else None,
+                                   rope.rot_dim if rope else 0, meta.slots, k_cache, v_cache, eps=self.eps, unit_norm=False,
+                                   q_w=self.q_norm, k_w=self.k_norm, conv=conv, long_portions=meta.n_prefill > 0)
+        T, nd = q.shape[0], meta.n_decode
+        seen = dict(window=self.window, keep=self.keep, softcap=self.softcap)
+        out = (torch.zeros if meta.padded else torch.empty)(q.shape, dtype=q.dtype, device=q.device)
+        if q.is_cuda and (q.dtype != torch.bfloat16 or self.d_pad not in (64, 128, 256)):
+            ops.paged_attention_generic(q, k_cache, v_cache, meta.block_table, meta.cu_q, meta.kv_lens, self.scale, out=out, **seen)
+        else:
+            if nd > 0:
+                splits = ops.decode_splits(nd, self.kv_heads, self.heads // self.kv_heads)
+                if self.window:
+                    splits = min(splits, max(1, (self.window + self.keep) // 256))
+                ops.paged_decode_attention(q[:nd], k_cache, v_cache, meta.block_table[:nd], meta.kv_lens[:nd], self.scale,
+                                           out=out[:nd], splits=splits, **seen)
+            if meta.n_prefill > 0:
+                ops.paged_prefill_attention(q, k_cache, v_cache, meta.block_table[nd:], meta.cu_q[nd:], meta.kv_lens[nd:],
+                                            meta.max_q_len, self.scale, causal=True, out=out, **seen)
+        return self.o(out.view(T, self.heads * self.d_pad))
+
+    __call__ = forward
+
+
+class LatentAttention(Module):
+    """Causal attention without positions over cached latents: queries behind a latent of their own (dq, its norm, uq), one
+    normed latent c per token (dkv, its norm) that all heads share, keys W_uk c and values W_uv c.  Only c is cached.
+    `own_latents` False: the cache is another layer's, which has written this step's rows already.
+
+    Two forms of one sum.  Absorbed: the query of a head is taken into the latent space (q W_uk), attends to the cached rows
+    themselves, and W_uv is applied to what comes back; decoding reads one row per token for all heads.  Expanded, for prompts
+    of many tokens: the context's latents become keys and values once per step."""
+
+    def __init__(self, hidden, heads, d, dv, q_rank, rank, scale, eps, dtype, device, own_latents=True):
+        super().__init__()
+        self.heads, self.d, self.dv, self.q_rank, self.rank = heads, d, dv, q_rank, rank
+        self.scale, self.eps, self.own = float(scale), eps, own_latents
+        self.width, self.q_pad = mla.latent_width(rank, dtype, device), round_up(q_rank, 8)
+        self.q_norm = self.add_param("dq.norm", torch.ones(q_rank, dtype=dtype, device=device))
+        self.c_norm = self.add_param("dkv.norm", torch.ones(rank, dtype=dtype, device=device)) if own_latents else None
+        self.uq = self._params["uq"] = torch.zeros(heads * d, self.q_pad, dtype=dtype, device=device)
+        self._loaders["uq"] = lambda w: self.uq[:, :q_rank].copy_(w.to(dtype))
+        # W_uk and W_uv behind one another, their columns padded as the cache's rows are
+        self.ukv = self._params["ukv"] = torch.zeros(heads * (d + dv), self.width, dtype=dtype, device=device)
+        self.uk, self.uv = self.ukv[:heads * d].view(heads, d, self.width), self.ukv[heads * d:].view(heads, dv, self.width)
+        self._loaders["uk"] = lambda w: self.ukv[:heads * d, :rank].copy_(w.to(dtype))
+        self._loaders["uv"] = lambda w: self.ukv[heads * d:, :rank].copy_(w.to(dtype))
+        self.o = self.add_module("o", Linear(heads * dv, hidden, False, dtype, device))
+        self.biased = ()
+        # prompt rows from which expanding pays: absorbed, a pair costs 2 width products a head, expanded d + dv
+        self.expand_from = 256 if dtype == torch.bfloat16 and d == dv == 128 and self.width in mla.LATENT_WIDTHS else None
+        self.expand_bytes = 2 << 30
+
+    def width_parts(self):
+        return [("dq", self.q_rank)] + ([("dkv", self.rank)] if self.own else [])
+
+    def kv_geometry(self):
+        return (1, 1, self.width) if self.own else None
+
+    def state_parts(self):
+        return {}
+
+    def _expandable(self, rows, cache, meta: AttentionMetadata):
+        """Rows a sequence's context takes when the prompts of this step run expanded, or 0."""
+        if self.expand_from is None or not rows.is_cuda or meta.padded or meta.max_kv_len <= 0:
+            return 0
+        page = cache.shape[-2]
+        per = round_up(meta.max_kv_len, page)
+        small = rows.shape[0] - meta.n_decode < self.expand_from
+        big = meta.n_prefill * per * self.ukv.shape[0] * 2 > self.expand_bytes
+        return 0 if small or big or page not in (16, 32, 64, 128) else per
+
+    def _absorbed(self, q, cache, positions, meta: AttentionMetadata, prompts, out):
+        """out [T, heads, dv] from q [T, heads, d]: of the decode rows alone, or (`prompts`) of all rows."""
+        nd = meta.n_decode
+        T = q.shape[0] if prompts else nd
+        q, out, alloc = q[:T], out[:T], torch.zeros if meta.padded else torch.empty
+        qa = torch.empty((T, self.heads, self.width), dtype=q.dtype, device=q.device)
+        torch.bmm(q.transpose(0, 1), self.uk, out=qa.transpose(0, 1))
+        oa = alloc(qa.shape, dtype=q.dtype, device=q.device)
+        n = meta.n_seqs if prompts else nd
+        bt, lens, cu = meta.block_table[:n], meta.kv_lens[:n], meta.cu_q[:n + 1]
+        if not q.is_cuda or q.dtype != torch.bfloat16 or self.width not in mla.LATENT_WIDTHS:
+            ops.paged_attention_generic(qa, cache, cache, bt, cu, lens, self.scale, out=oa)
+        else:
+            if nd > 0:
+                mla.latent_decode(qa[:nd], cache, bt, self.scale, seq_lens=lens[:nd], out=oa[:nd])
+            if T > nd and self.width <= 256:
+                # the latents as keys and values of one head that all query heads share
+                ops.paged_prefill_attention(qa, cache, cache, bt[nd:], cu[nd:], lens[nd:], meta.max_q_len, self.scale, out=oa)
+            elif T > nd:
+                row = torch.arange(nd, T, device=q.device, dtype=torch.int32)
+                seq = torch.bucketize(row, cu[nd + 1:].contiguous(), right=True).clamp_(max=meta.n_prefill - 1)
+                mla.latent_decode(qa[nd:], cache, bt, self.scale, positions=positions[nd:], bt_rows=(seq + nd).to(torch.int32),
+                                  out=oa[nd:])
+        torch.bmm(oa.transpose(0, 1), self.uv.transpose(1, 2), out=out.transpose(0, 1))
+
+    def forward(self, fused: FusedProjection, rows, positions, meta: AttentionMetadata, kv, state):
+        cache, nd, T = kv[0], meta.n_decode, rows.shape[0]
+        c = dict(c=fused.part(rows, "dkv"), c_w=self.c_norm, slots=meta.slots, cache=cache) if self.own else {}
+        cq = mla.latent_norm(fused.part(rows, "dq"), self.q_norm, self.q_pad, self.eps, **c)
+        q = ops.linear(cq, self.uq).view(T, self.heads, self.d)
+        out = torch.empty((T, self.heads, self.dv), dtype=rows.dtype, device=rows.device)
+        per = self._expandable(rows, cache, meta) if meta.n_prefill > 0 else 0
+        if per:
+            n, page = meta.n_prefill, cache.shape[-2]
+            kv_rows = ops.linear(mla.latent_gather(cache, meta.block_table[nd:], meta.kv_lens[nd:], per), self.ukv)
+            pages = torch.arange(n * per // page, dtype=torch.int32, device=rows.device).view(n, per // page)
+            ops.ragged_prefill_attention(q, kv_rows[:, :self.heads * self.d], kv_rows[:, self.heads * self.d:], pages, page,
+                                         meta.cu_q[nd:], meta.kv_lens[nd:], meta.max_q_len, self.scale, out)
+        if nd > 0 or not per:
+            self._absorbed(q, cache, positions, meta, not per, out)
+        return self.o(out.view(T, self.heads * self.dv))
 
     __call__ = forward
 

@@ -23,12 +23,13 @@ from ..parallel.state import single
 
 
 class SparseMoeBlock(Module):
-    """`own_router=False`: the router logits come from the caller (forward's `logits`)."""
+    """`own_router=False`: the router logits come from the caller (forward's `logits`).  `act`: the experts' gated activation
+    (ops/glu.py); the shared expert has its own in `shared_act` (default: args.hidden_act)."""
 
-    def __init__(self, args, dtype, device, ps=None, own_router=True):
+    def __init__(self, args, dtype, device, ps=None, own_router=True, act="silu", shared_act=None):
         super().__init__()
         self.ps = ps or single()
-        self.args = args
+        self.args, self.act = args, act
         E, H, I = args.num_experts, args.hidden_size, args.moe_intermediate_size
         ep = self.ps.ep_size if self.ps.ep_size > 1 else 1
         tp = self.ps.tp_size
@@ -122,7 +123,7 @@ class SparseMoeBlock(Module):
         if args.n_shared_experts > 0:
             si = args.shared_expert_intermediate_size or args.moe_intermediate_size * args.n_shared_experts
             self.shared = self.add_module("shared_experts", DenseMLP(
-                H, si, args.hidden_act, dtype, device, self.ps, reduce=False,
+                H, si, shared_act or args.hidden_act, dtype, device, self.ps, reduce=False,
                 quant="fp8_block" if getattr(args, "fp8_execution", False) else None))
         self.shared_gate = None
         if self.shared is not None and args.extra.get("shared_expert_gate"):
@@ -164,7 +165,7 @@ class SparseMoeBlock(Module):
                               a.n_group, a.topk_group, a.norm_topk_prob, a.routed_scaling_factor, self.e_begin,
                               a.num_experts, shared_out, ws, out,
                               w_scales=(self.s_gate_up, self.s_down) if self.fp8 else None,
-                              interleaved=self.interleaved, group_score=a.moe_group_score)
+                              interleaved=self.interleaved, group_score=a.moe_group_score, act=self.act)
         if out is None and self.ps.tp_size > 1:
             y = self.ps.all_reduce(y)
         return y

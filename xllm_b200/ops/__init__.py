@@ -10,7 +10,7 @@ import os
 
 import torch
 
-from . import _lib, reference
+from . import _lib, glu, reference
 from ._lib import check, ptr, stream
 
 from . import _debug  # noqa: E402
@@ -78,12 +78,14 @@ def rmsnorm(x, w, eps=1e-6, residual=None, out=None, gemma=False):
 def act_and_mul(x, act="silu", out=None):
     if not x.is_cuda:
         return reference.act_and_mul(x, act)
-    if x.dtype == torch.float32 and act == "silu":
+    code, limit, alpha = glu.code(act)
+    if x.dtype == torch.float32 and code in (0, 3):
         d = x.shape[-1] // 2
         x2 = x.reshape(-1, 2 * d)
         if out is None:
             out = torch.empty((x2.shape[0], d), dtype=x.dtype, device=x.device)
-        check(_lib_().xllm_silu_mul_f32(ptr(out), ptr(x2), x2.shape[0], d, x2.stride(0), stream()), "silu_mul_f32")
+        check(_lib_().xllm_silu_mul_f32(ptr(out), ptr(x2), x2.shape[0], d, x2.stride(0), limit, alpha, stream()),
+              "silu_mul_f32")
         _count()
         return out.reshape(*x.shape[:-1], d)
     _bf16(x, "act_and_mul")
@@ -93,8 +95,7 @@ def act_and_mul(x, act="silu", out=None):
         x2 = x2.contiguous()
     if out is None:
         out = torch.empty((x2.shape[0], d), dtype=x.dtype, device=x.device)
-    code = {"silu": 0, "gelu": 1, "gelu_tanh": 2, "gelu_pytorch_tanh": 2}[act]
-    check(_lib_().xllm_act_and_mul(ptr(out), ptr(x2), x2.shape[0], d, x2.stride(0), code, stream()),
+    check(_lib_().xllm_act_and_mul(ptr(out), ptr(x2), x2.shape[0], d, x2.stride(0), code, limit, alpha, stream()),
           "act_and_mul")
     _count()
     return out.reshape(*x.shape[:-1], d)
@@ -142,11 +143,14 @@ def rope_kv_write(qkv, nq, nkv, d, positions, cos_sin, rot, slots=None, k_cache=
 
 
 def rope_norm_kv_write(q, k, v, nq, nkv, d, positions, cos_sin, rot, slots, k_cache, v_cache, eps=1e-6,
-                       interleaved=False, unit_norm=True):
-    """Rotary positions on the first `rot` elements of every q and k head, THEN (`unit_norm`) each head divided by its
-    root mean square; k and v rows are scattered into the paged caches.  q, k, v: column blocks [T, heads * d] of the
+                       interleaved=False, unit_norm=True, q_w=None, k_w=None, conv=None, long_portions=True):
+    """(`conv`) a short causal convolution per channel, (q_w, k_w) a per-head RMS norm of q and k with weights [d], rotary
+    positions on the first `rot` elements of every q and k head, THEN (`unit_norm`) each
+    head divided by its root mean square; k and v rows are scattered into the paged caches.  q, k, v: column blocks [T, heads * d] of the
     same projection rows (v may be the key block, or have heads of a size of its own).  The caches may hold wider heads
-    than that (zero filled); returns q [T, nq, cache head size]."""
+    than that (zero filled); returns q [T, nq, cache head size].
+    conv = (weights [taps, channels of q | k | v], ring [state slots, taps, channels], state slots [n_seqs], cu_q, kv_lens)
+    over all rows of the batch; `long_portions`: some sequence may have more than one row."""
     T, dp = q.shape[0], k_cache.shape[3]
     dv = v.shape[1] // nkv
     if _debug.enabled():
@@ -154,16 +158,24 @@ def rope_norm_kv_write(q, k, v, nq, nkv, d, positions, cos_sin, rot, slots, k_ca
         _debug.check_range(slots, 0, k_cache.shape[0] * k_cache.shape[2], "rope_norm_kv_write slots", allow_negative_skip=True)
     if not q.is_cuda:
         return reference.rope_norm_kv(q, k, v, nq, nkv, d, positions, cos_sin, rot, slots, k_cache, v_cache, eps, interleaved,
-                                      unit_norm)
+                                      unit_norm, q_w, k_w, conv)
     assert q.stride(0) == k.stride(0) == v.stride(0) and q.stride(1) == k.stride(1) == v.stride(1) == 1
     assert q.dtype == k_cache.dtype and k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.shape[1] == nkv
     positions = _index(positions, torch.int64, "rope_norm_kv_write positions")
     slots = _index(slots, torch.int32, "rope_norm_kv_write slots")
     out = torch.empty((T, nq, dp), dtype=q.dtype, device=q.device)
+    cw = ring = st = cu = kl = None
+    if conv is not None:
+        cw, ring, st, cu, kl = conv
+        assert cw.dtype == ring.dtype == q.dtype and cw.is_contiguous() and ring.is_contiguous()
+        assert ring.shape[1:] == cw.shape and cw.shape[1] == q.shape[1] + k.shape[1] + v.shape[1]
+        assert st.dtype == cu.dtype == kl.dtype == torch.int32 and cu.shape[0] > st.shape[0] and kl.shape[0] >= st.shape[0]
     check(_lib_().xllm_rope_norm_kv(ptr(q), ptr(k), ptr(v), q.stride(0), ptr(out), ptr(k_cache), ptr(v_cache), ptr(cos_sin),
                                     cos_sin.shape[0] if cos_sin is not None else 0, ptr(positions), ptr(slots), T, nq, nkv, d,
                                     dv, dp, rot, k_cache.shape[2], int(interleaved), int(unit_norm), eps,
-                                    0 if q.dtype == torch.bfloat16 else 1, stream()), "rope_norm_kv")
+                                    ptr(q_w), ptr(k_w), ptr(cw), ptr(ring), ptr(st), ptr(cu), ptr(kl),
+                                    st.shape[0] if conv is not None else 0, cw.shape[0] if conv is not None else 0,
+                                    int(long_portions), 0 if q.dtype == torch.bfloat16 else 1, stream()), "rope_norm_kv")
     _count()
     return out
 
@@ -175,13 +187,15 @@ def attention_head_size(d):
     return next((s for s in (64, 128, 256) if d <= s), d)
 
 
-def paged_attention_generic(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, out=None, row0=0, rows=None, window=0):
+def paged_attention_generic(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, out=None, row0=0, rows=None, window=0,
+                            keep=0, softcap=0.0):
     """Rows [row0, row0 + rows) of q [T, nq, d], decode rows and prompt chunks alike (row ranges by cu_q), fp32 or bf16
-    caches, any head size up to 512: the path of the fp32 execution type."""
+    caches, any head size up to 1024: the path of the fp32 execution type.  With a window the first `keep` positions of a
+    sequence stay visible; softcap > 0: scores become softcap * tanh(score / softcap)."""
     T, nq, d = q.shape
     rows = T - row0 if rows is None else rows
     if not q.is_cuda:
-        y = reference.paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, True, window)
+        y = reference.paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, True, window, keep, softcap)
         if out is not None:
             out[row0:row0 + rows].copy_(y[row0:row0 + rows])
             return out
@@ -194,7 +208,7 @@ def paged_attention_generic(q, k_cache, v_cache, block_table, cu_q, kv_lens, sca
     check(_lib_().xllm_paged_attn_generic(ptr(out), out.stride(0), ptr(q), q.stride(0), ptr(k_cache), ptr(v_cache),
                                           ptr(block_table), block_table.stride(0), ptr(cu_q), ptr(kv_lens), kv_lens.shape[0],
                                           row0, rows, nq, k_cache.shape[1], d, k_cache.shape[2], scale, int(window or 0),
-                                          0 if q.dtype == torch.bfloat16 else 1, stream()), "paged_attn_generic")
+                                          int(keep), float(softcap or 0.0), 0 if q.dtype == torch.bfloat16 else 1, stream()), "paged_attn_generic")
     _count()
     return out
 
@@ -230,13 +244,14 @@ def decode_workspace(batch, nq, d, splits, device):
 
 
 def paged_decode_attention(q, k_cache, v_cache, block_table, seq_lens, scale, splits=None,
-                           workspace=None, out=None, window=0):
+                           workspace=None, out=None, window=0, keep=0, softcap=0.0):
     """q: [B, nq, d] (one query token per sequence) -> [B, nq, d].  `window` > 0: every query sees
-    its last `window` positions only (pages before them are not read)."""
+    its last `window` positions only (pages before them are not read) and the first `keep`; softcap > 0: scores become
+    softcap * tanh(score / softcap)."""
     window = int(window or 0)
     _debug.check_block_table(block_table, seq_lens, k_cache.shape[0], k_cache.shape[2], "paged_decode_attention")
     if not q.is_cuda:
-        y = reference.paged_decode_attention(q, k_cache, v_cache, block_table, seq_lens, scale, window)
+        y = reference.paged_decode_attention(q, k_cache, v_cache, block_table, seq_lens, scale, window, keep, softcap)
         if out is not None:
             out.copy_(y)
             return out
@@ -253,7 +268,12 @@ def paged_decode_attention(q, k_cache, v_cache, block_table, seq_lens, scale, sp
     if out is None:
         out = torch.empty((B, nq, d), dtype=q.dtype, device=q.device)
     assert q.stride(-1) == 1 and q.stride(1) == d
-    if window > 0:
+    if keep or softcap:
+        check(_lib_().xllm_paged_decode_attn_kept(ptr(out), ptr(q), q.stride(0), ptr(k_cache), ptr(v_cache),
+                                                  ptr(block_table), block_table.stride(0), ptr(seq_lens), B, nq, nkv, d, page,
+                                                  scale, splits, ptr(workspace), window, int(keep), float(softcap or 0.0),
+                                                  stream()), "paged_decode_attn_kept")
+    elif window > 0:
         check(_lib_().xllm_paged_decode_attn_window(ptr(out), ptr(q), q.stride(0), ptr(k_cache), ptr(v_cache),
                                                     ptr(block_table), block_table.stride(0), ptr(seq_lens), B,
                                                     nq, nkv, d, page, scale, splits, ptr(workspace), window, stream()),
@@ -268,14 +288,15 @@ def paged_decode_attention(q, k_cache, v_cache, block_table, seq_lens, scale, sp
 
 
 def paged_prefill_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, max_q_len, scale,
-                            causal=True, window=0, out=None):
-    """q: [T, nq, d] ragged by cu_q -> [T, nq, d]; attends to cache positions [0, kv_len)."""
+                            causal=True, window=0, out=None, keep=0, softcap=0.0):
+    """q: [T, nq, d] ragged by cu_q -> [T, nq, d]; attends to cache positions [0, kv_len); window, keep, softcap as in
+    paged_decode_attention."""
     if _debug.enabled():
         _debug.check_block_table(block_table, kv_lens, k_cache.shape[0], k_cache.shape[2], "paged_prefill_attention")
         _debug.check_range(cu_q, 0, q.shape[0] + 1, "paged_prefill_attention cu_q")
     if not q.is_cuda:
         y = reference.paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale,
-                                      causal, window)
+                                      causal, window, keep, softcap)
         if out is not None:
             r0 = int(cu_q[0])
             out[r0:].copy_(y[r0:])
@@ -294,18 +315,36 @@ def paged_prefill_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, max
     if (d == 128 and page in (16, 32, 64, 128) and k_cache.is_contiguous() and v_cache.is_contiguous()
             and os.environ.get("XLLM_PREFILL_ATTN", "tcgen05") != "legacy"):
         # tcgen05 / TMEM kernel (csrc/kernels/attn_prefill_tc.cu)
-        check(_lib_().xllm_paged_prefill_attn_tc(ptr(out), out.stride(0), ptr(q), q.stride(0), T, ptr(k_cache),
-                                                 ptr(v_cache), k_cache.shape[0], ptr(block_table),
-                                                 block_table.stride(0), ptr(cu_q), ptr(kv_lens), B, int(max_q_len),
-                                                 nq, nkv, page, scale, int(causal), int(window), stream()),
-              "paged_prefill_attn_tc")
+        check(_lib_().xllm_paged_prefill_attn_tc_kept(ptr(out), out.stride(0), ptr(q), q.stride(0), T, ptr(k_cache),
+                                                      ptr(v_cache), k_cache.shape[0], 0, ptr(block_table),
+                                                      block_table.stride(0), ptr(cu_q), ptr(kv_lens), B, int(max_q_len),
+                                                      nq, nkv, page, scale, int(causal), int(window), int(keep),
+                                                      float(softcap or 0.0), stream()), "paged_prefill_attn_tc")
         _count()
         return out
-    check(_lib_().xllm_paged_prefill_attn(ptr(out), out.stride(0), ptr(q), q.stride(0), ptr(k_cache),
-                                          ptr(v_cache), ptr(block_table), block_table.stride(0),
-                                          ptr(cu_q), ptr(kv_lens), B, int(max_q_len), nq, nkv, d,
-                                          page, scale, int(causal), int(window), stream()),
-          "paged_prefill_attn")
+    check(_lib_().xllm_paged_prefill_attn_kept(ptr(out), out.stride(0), ptr(q), q.stride(0), ptr(k_cache),
+                                               ptr(v_cache), ptr(block_table), block_table.stride(0),
+                                               ptr(cu_q), ptr(kv_lens), B, int(max_q_len), nq, nkv, d,
+                                               page, scale, int(causal), int(window), int(keep), float(softcap or 0.0),
+                                               stream()), "paged_prefill_attn")
+    _count()
+    return out
+
+
+def ragged_prefill_attention(q, k, v, block_table, page, cu_q, kv_lens, max_q_len, scale, out):
+    """Causal attention of q [T, nq, 128] over keys and values that are rows of all heads: k, v [pages * page, nkv * 128]
+    column blocks of one matrix, a sequence's pages named by its block-table row.  CUDA, bf16."""
+    T, nq, d = q.shape
+    R, width = k.shape
+    assert d == 128 and width % 128 == 0 and R % page == 0 and k.stride() == v.stride() and k.stride(1) == 1
+    _bf16(q, "ragged_prefill_attention")
+    assert q.stride(-1) == 1 and q.stride(1) == d and out.stride(1) == d and k.dtype == v.dtype == out.dtype == q.dtype
+    cu_q = _index(cu_q, torch.int32, "ragged_prefill_attention cu_q")
+    kv_lens = _index(kv_lens, torch.int32, "ragged_prefill_attention kv_lens")
+    check(_lib_().xllm_paged_prefill_attn_tc_kept(ptr(out), out.stride(0), ptr(q), q.stride(0), T, ptr(k), ptr(v), R // page,
+                                                  k.stride(0), ptr(block_table), block_table.stride(0), ptr(cu_q),
+                                                  ptr(kv_lens), kv_lens.shape[0], int(max_q_len), nq, width // 128, page, scale,
+                                                  1, 0, 0, 0.0, stream()), "ragged_prefill_attn_tc")
     _count()
     return out
 

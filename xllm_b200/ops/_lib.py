@@ -98,10 +98,13 @@ def _declare(lib):
     sig = {
         "xllm_rmsnorm": [P, P, P, P, I, I, F, L, L, I, P],
         "xllm_rmsnorm_static_fp8": [P, P, P, P, P, I, I, F, P],
-        "xllm_act_and_mul": [P, P, L, I, L, I, P],
+        "xllm_act_and_mul": [P, P, L, I, L, I, F, F, P],
         "xllm_rope_kv": [P, L, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, P],
         "xllm_paged_decode_attn": [P, P, L, P, P, P, I, P, I, I, I, I, I, F, I, P, P],
         "xllm_paged_decode_attn_window": [P, P, L, P, P, P, I, P, I, I, I, I, I, F, I, P, I, P],
+        "xllm_paged_decode_attn_kept": [P, P, L, P, P, P, I, P, I, I, I, I, I, F, I, P, I, I, F, P],
+        "xllm_paged_prefill_attn_kept": [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, F, I, I, I, F, P],
+        "xllm_paged_prefill_attn_tc_kept": [P, L, P, L, L, P, P, L, L, P, I, P, P, I, I, I, I, I, F, I, I, I, F, P],
         "xllm_attn_merge": [P, P, P, L, I, I, P],
         "xllm_paged_prefill_attn": [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, F, I, I, P],
         "xllm_paged_prefill_attn_tc": [P, L, P, L, L, P, P, L, P, I, P, P, I, I, I, I, I, F, I, I, P],
@@ -116,10 +119,10 @@ def _declare(lib):
         "xllm_block_copy": [P, I, P, I, L, P],
         "xllm_decode_advance": [P, P, P, P, P, I, P, I, I, P],
         "xllm_resolve_placeholders": [P, P, L, L, P],
-        "xllm_rope_norm_kv": [P, P, P, L, P, P, P, P, L, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P],
+        "xllm_rope_norm_kv": [P, P, P, L, P, P, P, P, L, P, P, I, I, I, I, I, I, I, I, I, I, F] + [P] * 7 + [I] * 4 + [P],
         "xllm_proj_f32": [P, L, P, L, P, P, I, I, I, P],
-        "xllm_paged_attn_generic": [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, I, F, I, I, P],
-        "xllm_silu_mul_f32": [P, P, L, I, L, P],
+        "xllm_paged_attn_generic": [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, I, F, I, I, F, I, P],
+        "xllm_silu_mul_f32": [P, P, L, I, L, F, F, P],
     }
     for name, args in sig.items():
         lib.declare(name, args, I)

@@ -14,7 +14,7 @@ from . import _lib
 from ._lib import F, I, L, P, check, ptr, stream
 from .head_norm import head_norm_gate
 
-_lib.register_signature("xllm_linattn", [P] * 9 + [L, P, L, P, P, P, P, P, P, L] + [I] * 8 + [F] * 4 + [I, I, P, P, I, I, I, P])
+_lib.register_signature("xllm_linattn", [P] * 9 + [L, P, L, P, P, P, P, P, P, L] + [I] * 8 + [F] * 4 + [I, I, P, P, I, I, I, I, P])
 
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 
@@ -36,7 +36,11 @@ class LinearAttention:
     cos_sin: Optional[torch.Tensor] = None
     rot: int = 0
     interleaved: bool = False
-    # output of a head: divided by its root mean square, times the weight [dv] when there is one
+    in_silu: bool = False            # q, k and v pass through silu first
+    # `rows`: the heads of a token are normed together over all their elements and gated with the sigmoid of g; otherwise
+    # every head is finished alone and gated with silu(g)
+    rows: bool = False
+    # output of a head: divided by its root mean square, times the weight [dv] when there is one (`rows`: [heads dv])
     unit_norm: bool = True
     norm_w: Optional[torch.Tensor] = None
     eps: float = 1e-6
@@ -57,7 +61,7 @@ class LinearAttention:
             ptr(self.log_decay), ptr(self.a2), ptr(self.a2_bias), ptr(self.norm_w), ptr(out), out_ld, n_seqs, self.heads,
             self.dk, self.dv, self.rot, int(self.interleaved), self.a2.shape[1] if channel else 0, int(self.unit_norm),
             self.q_scale, self.k_scale, self.inv_tau, self.eps, _DT[q.dtype], mode, ptr(seg[0]), ptr(seg[1]),
-            seg[2], seg[3], int(finish), stream()), "linattn")
+            seg[2], seg[3], int(finish), int(self.in_silu), stream()), "linattn")
         from . import _count
         _count()
 
@@ -69,7 +73,11 @@ class LinearAttention:
             return self._cpu(state, slots, torch.arange(B + 1), kv_lens, positions, q, k, v, r, g, out)
         if out is None:
             out = torch.empty((B, self.heads * self.dv), dtype=q.dtype, device=q.device)
-        self._launch(0, state, slots, None, kv_lens, positions, q, k, v, g, r, out, out.stride(0), B)
+        if self.rows:
+            o = torch.empty((B, self.heads, self.dv), dtype=torch.float32, device=q.device)
+            self._launch(0, state, slots, None, kv_lens, positions, q, k, v, None, r, o, 0, B)
+            return self.finish(o, g, out)
+        self._launch(0, state, slots, None, kv_lens, positions, q, k, v, g, r, out, out.stride(0), B, finish=True)
         return out
 
     def prefill(self, state, slots, cu_q, kv_lens, positions, q, k, v, g=None, r=None, out=None, row0=0, padded=False,
@@ -85,7 +93,7 @@ class LinearAttention:
             out = torch.empty((T, self.heads * self.dv), dtype=q.dtype, device=q.device)
         chunked = q.dtype == torch.bfloat16 and self.dk <= 256 and not token_by_token and \
             (self.a2 is None or self.a2.shape[1] <= 64)
-        fused = chunked and self.dv <= 128
+        fused = chunked and self.dv <= 128 and not self.rows
         seg = self._segments(T, n, max_q_len or T, q.device) if chunked else (None, None, 16, 1)
         if fused:
             self._launch(1, state, slots, cu_q, kv_lens, positions, q, k, v, g, r, out, out.stride(0), n, seg=seg, finish=True)
@@ -109,7 +117,10 @@ class LinearAttention:
         return st, torch.empty((m, self.heads, self.dk), dtype=torch.float32, device=device), length, segs
 
     def finish(self, o, g, out):
-        """Per-head norm, weight and gate of raw fp32 outputs o [T, heads, dv]."""
+        """Norm, weight and gate of raw fp32 outputs o [T, heads, dv]."""
+        if self.rows:
+            return head_norm_gate(o.view(o.shape[0], 1, -1), out, g=g, w=self.norm_w, unit_norm=self.unit_norm, act="sigmoid",
+                                  eps=self.eps)
         return head_norm_gate(o, out, g=g, w=self.norm_w, unit_norm=self.unit_norm, eps=self.eps)
 
     # ------------------------------------------------------------------ tensor-op form
@@ -131,14 +142,15 @@ class LinearAttention:
         H, dk, dv = self.heads, self.dk, self.dv
         T = q.shape[0]
         res = out if out is not None else torch.zeros(T, H * dv, dtype=q.dtype)
-        qf = self._rope(q.float().reshape(T, H, dk), positions) * self.q_scale
-        kf = self._rope(k.float().reshape(T, H, dk), positions) * self.k_scale
-        vf = v.float().reshape(T, H, dv)
+        enter = (lambda t: torch.nn.functional.silu(t.float())) if self.in_silu else (lambda t: t.float())
+        qf = self._rope(enter(q).reshape(T, H, dk), positions) * self.q_scale
+        kf = self._rope(enter(k).reshape(T, H, dk), positions) * self.k_scale
+        vf = enter(v).reshape(T, H, dv)
         if self.log_decay is None:
             z = r.float() @ self.a2.float().T + self.a2_bias.float()
-            a = torch.exp(torch.nn.functional.logsigmoid(z) * self.inv_tau).view(T, H, dk)
+            less = torch.expm1(torch.nn.functional.logsigmoid(z) * self.inv_tau).view(T, H, dk)     # a - 1
         else:
-            a = torch.exp(self.log_decay).view(1, H, 1).expand(T, H, dk)
+            less = torch.expm1(self.log_decay).view(1, H, 1).expand(T, H, dk)
         for i in range(slots.shape[0]):
             b, e, slot = int(cu_q[i]), int(cu_q[i + 1]), int(slots[i])
             if slot < 0 or e <= b:
@@ -146,9 +158,12 @@ class LinearAttention:
             S = state[slot, :, :, :dv].clone() if int(kv_lens[i]) != e - b else torch.zeros(H, dk, dv)
             o = torch.empty(e - b, H, dv)
             for t in range(b, e):
-                S = a[t][:, :, None] * S + kf[t][:, :, None] * vf[t][:, None, :]
+                S = S + less[t][:, :, None] * S + kf[t][:, :, None] * vf[t][:, None, :]
                 o[t - b] = torch.einsum("hkv,hk->hv", S, qf[t])
             state[slot, :, :, :dv] = S
+            if self.rows:
+                self.finish(o, g[b:e] if g is not None else None, res[b:e])
+                continue
             if self.unit_norm:
                 o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + self.eps)
             if self.norm_w is not None:

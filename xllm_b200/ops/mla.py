@@ -110,3 +110,83 @@ def decode(q_cat, cache, block_table, scale, seq_lens=None, positions=None, bt_r
     from . import _count
     _count(2 if splits > 1 else 1)
     return out
+
+
+# ----------------------------------------------------------------------------- caches of latents alone
+_lib.register_signature("xllm_latent_decode", [P, P, L, P, I, P, I, P, P, P, I, I, I, F, I, P, P])
+_lib.register_signature("xllm_latent_norm", [P, P, P, I, I, P, P, P, I, I, P, L, I, F, I, P])
+_lib.register_signature("xllm_latent_gather", [P, P, P, I, P, I, I, I, I, P])
+
+LATENT_WIDTHS = (128, 256, 512)
+
+
+def latent_width(rank, dtype, device):
+    """Row size a cache of latents of `rank` values should have: the widths of the tensor-core kernels in bf16 on the device
+    (zero filled), the rank itself otherwise."""
+    if dtype == torch.bfloat16 and torch.device(device).type == "cuda":
+        return next((w for w in LATENT_WIDTHS if rank <= w), (rank + 7) // 8 * 8)
+    return rank
+
+
+def latent_norm(q, q_w, q_pad, eps, c=None, c_w=None, slots=None, cache=None):
+    """Normed query latents [T, q_pad] (zero filled) and, with c, normed latents into the cache rows of the tokens' slots.
+    q [T, q rank], c [T, rank]: column blocks of the same rows; cache [n_blocks, 1, page, width]."""
+    T, q_rank = q.shape
+    out = torch.empty((T, q_pad), dtype=q.dtype, device=q.device)
+    if not q.is_cuda:
+        def norm(x, w, to):
+            x = x.float()
+            x = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+            return torch.nn.functional.pad(x, (0, to - x.shape[1])).to(q.dtype)
+        out.copy_(norm(q, q_w, q_pad))
+        if c is not None:
+            ok = slots >= 0
+            cache.view(-1, cache.shape[-1])[slots[ok].long()] = norm(c, c_w, cache.shape[-1])[ok]
+        return out
+    assert q.stride(1) == 1 and q.dtype in (torch.bfloat16, torch.float32)
+    if c is not None:
+        assert c.stride() == q.stride() and c.dtype == q.dtype == cache.dtype and cache.is_contiguous() and cache.shape[1] == 1
+        assert slots.dtype == torch.int32 and slots.is_contiguous()
+    check(_lib.load().xllm_latent_norm(ptr(q), ptr(q_w), ptr(out), q_rank, q_pad, ptr(c), ptr(c_w), ptr(cache),
+                                       c.shape[1] if c is not None else 0, cache.shape[-1] if c is not None else 0, ptr(slots),
+                                       q.stride(0), T, float(eps), 0 if q.dtype == torch.bfloat16 else 1, stream()),
+          "latent_norm")
+    from . import _count
+    _count()
+    return out
+
+
+def latent_decode(q, cache, block_table, scale, seq_lens=None, positions=None, bt_rows=None, splits=None, out=None):
+    """`decode` over a cache [n_blocks, 1, page, width] of latents alone: q, out [N, nh, width].  CUDA, bf16, width in
+    LATENT_WIDTHS."""
+    N, nh, width = q.shape
+    assert q.dtype == cache.dtype == torch.bfloat16 and q.is_contiguous() and cache.is_contiguous() and cache.shape[-1] == width
+    assert block_table.dtype == torch.int32 and block_table.stride(1) == 1
+    if out is None:
+        out = torch.empty_like(q)
+    assert out.is_contiguous()
+    if N == 0:
+        return out
+    if splits is None:
+        from . import decode_splits
+        splits = decode_splits(N, 1, nh)
+    ws = torch.empty(N * nh * splits * (width + 1), dtype=torch.float32, device=q.device) if splits > 1 else None
+    check(_lib.load().xllm_latent_decode(ptr(out), ptr(q), q.stride(0), ptr(cache), width, ptr(block_table),
+                                         block_table.stride(0), ptr(seq_lens), ptr(positions), ptr(bt_rows), N, nh,
+                                         cache.shape[-2], float(scale), int(splits), ptr(ws), stream()), "latent_decode")
+    from . import _count
+    _count(2 if splits > 1 else 1)
+    return out
+
+
+def latent_gather(cache, block_table, kv_lens, rows_per):
+    """The cached latents of a few sequences as dense rows [n_seqs * rows_per, width], zeros behind each sequence."""
+    n, width = kv_lens.shape[0], cache.shape[-1]
+    assert cache.dtype == torch.bfloat16 and cache.is_contiguous() and cache.shape[1] == 1
+    assert block_table.dtype == kv_lens.dtype == torch.int32 and block_table.stride(1) == 1
+    out = torch.empty((n * rows_per, width), dtype=cache.dtype, device=cache.device)
+    check(_lib.load().xllm_latent_gather(ptr(out), ptr(cache), ptr(block_table), block_table.stride(0), ptr(kv_lens), n,
+                                         rows_per, cache.shape[-2], width, stream()), "latent_gather")
+    from . import _count
+    _count()
+    return out

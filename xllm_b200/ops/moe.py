@@ -11,7 +11,7 @@ import weakref
 
 import torch
 
-from . import _lib
+from . import _lib, glu
 from ._lib import F, I, L, P, check, ptr, stream
 
 _lib.register_signature("xllm_moe_route", [P, I, P, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P])
@@ -21,7 +21,7 @@ _lib.register_signature("xllm_moe_permute", [P, P, P, P, P, P, I, I, I, I, P])
 _lib.register_signature("xllm_moe_finalize", [P, P, L, P, P, P, I, I, I, I, P])
 _lib.register_signature("xllm_moe_grouped_simt", [P, P, P, P, I, I, I, L, L, I, P])
 _lib.register_signature("xllm_gemm_bf16_grouped", [P, P, P, P, I, I, I, I, L, L, P])
-_lib.register_signature("xllm_gemm_bf16_grouped_act_mul", [P, P, P, P, I, I, I, I, L, L, I, P])
+_lib.register_signature("xllm_gemm_bf16_grouped_act_mul", [P, P, P, P, I, I, I, I, L, L, I, F, F, P])
 
 
 def route_reference(logits, top_k, scoring="softmax", bias=None, n_group=1, topk_group=1, renorm=True, scale=1.0,
@@ -58,7 +58,7 @@ def fused_moe_reference(x, logits, w_gate_up, w_down, top_k, scoring="softmax", 
             continue
         h = (x[tok].float() @ w_gate_up[e].float().T).to(x.dtype).float()
         d = h.shape[-1] // 2
-        a = (torch.nn.functional.silu(h[:, :d]) * h[:, d:]).to(x.dtype).float()
+        a = glu.apply(h[:, :d], h[:, d:], act).to(x.dtype).float()
         y = (a @ w_down[e].float().T).to(x.dtype).float()
         out.index_add_(0, tok, y * w[tok, kk, None])
     return out.to(x.dtype)
@@ -103,12 +103,13 @@ def shared_workspace(T, *key):
 
 def fused_moe(x, logits, w_gate_up, w_down, top_k, scoring="softmax", bias=None, n_group=1, topk_group=1,
               renorm=True, scale=1.0, expert_begin=0, n_experts=None, shared_out=None, ws: MoeWorkspace = None,
-              out=None, w_scales=None, interleaved=False, group_score="auto"):
+              out=None, w_scales=None, interleaved=False, group_score="auto", act="silu"):
     """x [T,H], logits [T,E]; w_gate_up [E_local, 2I, H], w_down [E_local, H, I] -> [T,H].  w_down may have more rows than H (zeros
     that make the product's width one the tensor-core kernel takes).
+    `act`: the gated activation (ops/glu.py).
     `interleaved`: every expert's gate|up rows are stored in groups of 128 = [64 gate | the 64 up rows of the
-    same features] (`ops.gemm_tcgen05.interleave_gate_up`); the first grouped GEMM then applies SiLU(gate) * up
-    in its epilogue and the [rows, 2I] intermediate is never written.
+    same features] (`ops.gemm_tcgen05.interleave_gate_up`); the first grouped GEMM then applies the
+    activation in its epilogue and the [rows, 2I] intermediate is never written.
     `w_scales` = (s_gate_up [E_local, 2I/128, H/128], s_down [E_local, H/128, I/128]): the weights are e4m3
     with 128 x 128 block scales and both grouped GEMMs run block-scaled in fp8 (the rows are quantised
     per token in groups of 128 before each of them)."""
@@ -121,7 +122,7 @@ def fused_moe(x, logits, w_gate_up, w_down, top_k, scoring="softmax", bias=None,
             w_gate_up = torch.stack([fp8.dequant_block128_ref(w_gate_up[e], w_scales[0][e], x.dtype) for e in range(w_gate_up.shape[0])])
             w_down = torch.stack([fp8.dequant_block128_ref(w_down[e], w_scales[1][e], x.dtype) for e in range(w_down.shape[0])])
         return fused_moe_reference(x, logits, w_gate_up, w_down[:, :x.shape[1]], top_k, scoring, bias, n_group, topk_group, renorm,
-                                   scale, expert_begin, shared_out, group_score=group_score)
+                                   scale, expert_begin, shared_out, act, group_score)
     from . import _count, act_and_mul
     lib = _lib.load()
     T, H = x.shape
@@ -148,7 +149,7 @@ def fused_moe(x, logits, w_gate_up, w_down, top_k, scoring="softmax", bias=None,
         from . import fp8
         xq, xs = fp8.quant_group128(ws.xp)
         fp8.block_scaled_mm_grouped(xq, xs, w_gate_up, w_scales[0], ws.tile_expert, ws.h)
-        act_and_mul(ws.h, "silu", out=ws.a)
+        act_and_mul(ws.h, act, out=ws.a)
         aq, as_ = fp8.quant_group128(ws.a)
         fp8.block_scaled_mm_grouped(aq, as_, w_down, w_scales[1], ws.tile_expert, ws.y)
     elif dt == 1 or H % 8 or I2 % 64 or inter % 8 or Y % 64:
@@ -158,16 +159,17 @@ def fused_moe(x, logits, w_gate_up, w_down, top_k, scoring="softmax", bias=None,
         if interleaved:
             raise ValueError("interleaved expert rows need the tensor-core product")
         simt(ws.xp, w_gate_up, ws.h)
-        act_and_mul(ws.h, "silu", out=ws.a)
+        act_and_mul(ws.h, act, out=ws.a)
         simt(ws.a, w_down, ws.y)
     else:
         if interleaved:
+            code, limit, alpha = glu.code(act)
             check(lib.xllm_gemm_bf16_grouped_act_mul(ptr(ws.xp), ptr(w_gate_up), ptr(ws.a), ptr(ws.tile_expert), ws.rows,
-                                                     I2, H, E_local, H, inter, 1, s), "moe_gemm1_act")
+                                                     I2, H, E_local, H, inter, code + 1, limit, alpha, s), "moe_gemm1_act")
         else:
             check(lib.xllm_gemm_bf16_grouped(ptr(ws.xp), ptr(w_gate_up), ptr(ws.h), ptr(ws.tile_expert), ws.rows, I2, H,
                                              E_local, H, I2, s), "moe_gemm1")
-            act_and_mul(ws.h, "silu", out=ws.a)
+            act_and_mul(ws.h, act, out=ws.a)
         check(lib.xllm_gemm_bf16_grouped(ptr(ws.a), ptr(w_down), ptr(ws.y), ptr(ws.tile_expert), ws.rows, Y, inter,
                                          E_local, inter, Y, s), "moe_gemm2")
     if out is None:

@@ -9,6 +9,8 @@ import math
 
 import torch
 
+from . import glu
+
 
 def rmsnorm(x, w, eps, residual=None, gemma=False):
     """Returns (normed, new_residual). new_residual = x + residual (rounded to x.dtype)."""
@@ -28,14 +30,7 @@ def rmsnorm(x, w, eps, residual=None, gemma=False):
 
 def act_and_mul(x, act="silu"):
     d = x.shape[-1] // 2
-    a, b = x[..., :d].float(), x[..., d:].float()
-    if act == "silu":
-        g = torch.nn.functional.silu(a)
-    elif act == "gelu":
-        g = torch.nn.functional.gelu(a)
-    else:
-        g = torch.nn.functional.gelu(a, approximate="tanh")
-    return (g * b).to(x.dtype)
+    return glu.apply(x[..., :d].float(), x[..., d:].float(), act).to(x.dtype)
 
 
 def build_cos_sin_cache(rot_dim, max_pos, theta, scaling=None, device="cpu"):
@@ -131,14 +126,40 @@ def rope_kv(qkv, nq, nkv, d, positions, cos_sin, rot, q_norm_w=None, k_norm_w=No
     return qf.to(qkv.dtype), kf.to(qkv.dtype), v.contiguous()
 
 
-def rope_norm_kv(q, k, v, nq, nkv, d, positions, cos_sin, rot, slots, k_cache, v_cache, eps, interleaved, unit_norm):
-    """Rotation, then a per-head RMS norm without a weight; k and v go to caches whose heads may be wider than d."""
+def conv_portions(x, w, ring, state_slots, cu_q, kv_lens):
+    """Causal convolution over time per channel of the rows of several sequences: x [T, C], w [taps, C] (the last row belongs
+    to the current token), ring [state slots, taps, C] the last inputs of every sequence, row (position mod taps)."""
+    taps = w.shape[0]
+    y = torch.zeros(x.shape, dtype=torch.float32)
+    for i in range(state_slots.shape[0]):
+        b, e, slot = int(cu_q[i]), int(cu_q[i + 1]), int(state_slots[i])
+        if slot < 0 or e <= b:
+            continue
+        n, first = e - b, int(kv_lens[i]) - (e - b)
+        old = [ring[slot, p % taps] if p >= 0 else torch.zeros_like(ring[slot, 0]) for p in range(first - taps + 1, first)]
+        full = torch.cat([torch.stack(old), x[b:e]]) if taps > 1 else x[b:e]
+        for j in range(taps):
+            y[b:e] += full[j:j + n].float() * w[j].float()
+        for j in range(max(0, n - taps), n):
+            ring[slot, (first + j) % taps] = x[b + j]
+    return y
+
+
+def rope_norm_kv(q, k, v, nq, nkv, d, positions, cos_sin, rot, slots, k_cache, v_cache, eps, interleaved, unit_norm,
+                 q_w=None, k_w=None, conv=None):
+    """Convolution, weighted per-head RMS norm, rotation, per-head RMS norm without a weight (each optional but for the
+    rotation's place); k and v go to caches whose heads may be wider than d."""
     T, dp = q.shape[0], k_cache.shape[3]
+    if conv is not None:
+        y = conv_portions(torch.cat([q, k, v], dim=1), *conv)
+        q, k, v = y.split([q.shape[1], k.shape[1], v.shape[1]], dim=1)
     half = rot // 2
     cs = cos_sin[positions.long()].float() if rot else None
 
-    def prep(x, n):
+    def prep(x, n, w):
         x = x.reshape(T, n, d).float()
+        if w is not None:
+            x = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w.float()
         if rot:
             c, s = cs[:, None, :half], cs[:, None, half:]
             xr = x[..., :rot]
@@ -149,8 +170,8 @@ def rope_norm_kv(q, k, v, nq, nkv, d, positions, cos_sin, rot, slots, k_cache, v
         return x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) if unit_norm else x
 
     pad = lambda x: torch.nn.functional.pad(x, (0, dp - x.shape[-1])).to(k_cache.dtype)
-    write_kv_cache(pad(prep(k, nkv)), pad(v.reshape(T, nkv, -1).float()), k_cache, v_cache, slots)
-    return pad(prep(q, nq))
+    write_kv_cache(pad(prep(k, nkv, k_w)), pad(v.reshape(T, nkv, -1).float()), k_cache, v_cache, slots)
+    return pad(prep(q, nq, q_w))
 
 
 def write_kv_cache(k, v, k_cache, v_cache, slots):
@@ -172,8 +193,9 @@ def _gather_kv(cache, block_table_row, kv_len):
     return x[:, :kv_len]  # [nkv, kv_len, d]
 
 
-def paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, causal=True, window=0):
-    """q: [T, nq, d]; returns [T, nq, d]. Sequence b owns q rows cu_q[b]:cu_q[b+1]."""
+def paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, causal=True, window=0, keep=0, softcap=0.0):
+    """q: [T, nq, d]; returns [T, nq, d]. Sequence b owns q rows cu_q[b]:cu_q[b+1].  With a window the first `keep`
+    positions stay visible; softcap > 0 bounds the scores."""
     out = torch.zeros_like(q)
     nq, nkv = q.shape[1], k_cache.shape[1]
     group = nq // nkv
@@ -187,13 +209,15 @@ def paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, caus
         v = _gather_kv(v_cache, block_table[b], kl).float().repeat_interleave(group, dim=0)
         qq = q[qs:qe].float().transpose(0, 1)  # [nq, ql, d]
         s = torch.einsum("hqd,hkd->hqk", qq, k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
         qpos = torch.arange(ql, device=q.device)[:, None] + (kl - ql)
         kpos = torch.arange(kl, device=q.device)[None, :]
         mask = torch.zeros(ql, kl, dtype=torch.bool, device=q.device)
         if causal:
             mask |= kpos > qpos
         if window and window > 0:
-            mask |= kpos <= qpos - window
+            mask |= (kpos <= qpos - window) & (kpos >= keep)
         s = s.masked_fill(mask[None], float("-inf"))
         p = torch.softmax(s, dim=-1)
         p = torch.nan_to_num(p, nan=0.0)
@@ -202,11 +226,12 @@ def paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, caus
     return out
 
 
-def paged_decode_attention(q, k_cache, v_cache, block_table, seq_lens, scale, window=0):
+def paged_decode_attention(q, k_cache, v_cache, block_table, seq_lens, scale, window=0, keep=0, softcap=0.0):
     """q: [B, nq, d] one token per sequence."""
     B = q.shape[0]
     cu = torch.arange(B + 1, dtype=torch.int32, device=q.device)
-    return paged_attention(q, k_cache, v_cache, block_table, cu, seq_lens, scale, causal=True, window=window)
+    return paged_attention(q, k_cache, v_cache, block_table, cu, seq_lens, scale, causal=True, window=window, keep=keep,
+                           softcap=softcap)
 
 
 def apply_penalties(logits, ids, counts, freq, presence, repetition):

@@ -7,15 +7,16 @@ import torch
 from . import _lib
 from ._lib import F, I, L, P, check, ptr, stream
 
-_lib.register_signature("xllm_residual_update", [P, P, L, P, P, L, P, P, L, P, P, I, I, I, F, F, F, I, P])
+_lib.register_signature("xllm_residual_update", [P, P, L, P, P, L, P, P, P, L, P, P, I, I, I, F, F, F, I, P])
 _lib.register_signature("xllm_gelu_mul_rows", [P, P, L, P, L, L, P, L, I, I, I, I, P])
 
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 
 
 def residual_update(x, y, w=None, y2=None, w2=None, coef=1.0, rows=None, w_out=None, eps=1e-6, want_out=True,
-                    w_out_offset=0.0):
-    """x <- x + coef * (n(y) + n(y2)), n = RMS norm with the branch's weight (w, w2) or the identity without one;
+                    w_out_offset=0.0, w_sum=None):
+    """x <- x + m(coef * (n(y) + n(y2))), n = RMS norm with the branch's weight (w, w2) or the identity without one, m the
+    same with w_sum;
     returns (x, out) with out = rmsnorm(x) * (w_out + w_out_offset), or x cast to the branch type when w_out is None (None when
     `want_out` is false).  x is fp32 [T, H] and updated in place; x None starts the stream: x = coef * n(y).
     `rows`: y is a table and row t joins as y[rows[t]] (token embedding)."""
@@ -29,10 +30,11 @@ def residual_update(x, y, w=None, y2=None, w2=None, coef=1.0, rows=None, w_out=N
         add = n(y[rows] if rows is not None else y, w)
         if y2 is not None:
             add = add + n(y2, w2)
+        add = n(add * coef, w_sum)
         if init:
-            x = add * coef
+            x = add
         else:
-            x += add * coef
+            x += add
         out = None
         if want_out:
             out = (x if w_out is None else x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * (w_out.float() + w_out_offset)).to(y.dtype)
@@ -46,7 +48,7 @@ def residual_update(x, y, w=None, y2=None, w2=None, coef=1.0, rows=None, w_out=N
     assert rows is None or (rows.dtype == torch.int64 and rows.is_contiguous())
     out = torch.empty((T, H), dtype=y.dtype, device=y.device) if want_out else None
     check(_lib.load().xllm_residual_update(
-        ptr(x), ptr(y), y.stride(0), ptr(w), ptr(y2), y2.stride(0) if y2 is not None else 0, ptr(w2), ptr(rows), y.shape[0],
+        ptr(x), ptr(y), y.stride(0), ptr(w), ptr(y2), y2.stride(0) if y2 is not None else 0, ptr(w2), ptr(w_sum), ptr(rows), y.shape[0],
         ptr(w_out), ptr(out), T, H, int(init), float(coef), float(eps), float(w_out_offset), _DT[y.dtype], stream()), "residual_update")
     from . import _count
     _count()
