@@ -1,9 +1,11 @@
 #!/usr/bin/env python
-"""Prefill and decode throughput of one model design beside the framework's closest model (Qwen3-Next: three
-gated-delta-net layers per attention layer) at equal size, random weights, one GPU.
+"""Prefill and decode throughput of one model design beside the framework's closest models (Qwen3-Next: three
+gated-delta-net layers per attention layer; others where a design has more in common with them) at equal size, random
+weights, one GPU.
 
     python bench.py --design femirax [--steps K] [--warmup W]      # prints one JSON line
     python bench.py --design sodedra
+    python bench.py --design lukinex
 
 Prefill: four prompts of 2048 tokens in one step.  Decode: 64 sequences of 512 prompt tokens, one token each per step.
 Both go through the engine (scheduler, state slots, cache, sampling) and are timed with CUDA events around K steps
@@ -54,6 +56,26 @@ def sodedra_args(W):
                                  "embedding": {"scale": 1.0}, "layers": layers})
 
 
+def lukinex_args(W):
+    """Two parallel layers, one normed attention layer and one latent attention layer in turn, of which the second latent layer
+    reads the first one's latents; every layer with experts and a shared one."""
+    from xllm_b200.models import model_args_from_dict
+    H = W // 128
+    heads = {"heads": H, "kv_heads": max(1, H // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+             "mask": {"size": 1024, "keep_first": 16}, "rot": {"base": 1e6, "dims": 128}}
+    par = ("parallel", {"left": {**heads, "conv": 4, "softcap": 30.0},
+                        "right": {"heads": H, "dim": 128, "vdim": 128,
+                                  "decay": [1.0 - 2.0 ** (-5 - 5 * h / max(H - 1, 1)) for h in range(H)]}})
+    att = ("attention", {**heads, "rot": {"base": 1e6, "dims": 64, "scaling": {"factor": 4.0}}})
+    lat = ("latent_attention", {"heads": H, "dim": 128, "vdim": 128, "q_rank": W // 2, "kv_rank": 512, "scale": 128 ** -0.5})
+    kinds = [par, lat, par, att]
+    moe = {"kind": "moe", "expert": {"ff": W // 2, "limit": 7.0}, "router": {"experts": EXPERTS, "top": TOP},
+           "shared": {"ff": W // 2, "limit": 7.0}}
+    layers = [{"type": kinds[i % 4][0], "mixer": dict(kinds[i % 4][1]), "mlp": moe} for i in range(LAYERS)]
+    layers[5]["mixer"]["kv_from"] = 1
+    return model_args_from_dict({"architecture": "Lukinex", "vocab": VOCAB, "width": W, "norm": {"eps": 1e-6}, "layers": layers})
+
+
 def qwen3_next_args(W):
     from xllm_b200.models import ModelArgs
     H = W // 128
@@ -70,7 +92,25 @@ def qwen3_next_moe_args(W):
                                moe_layer_freq=2)
 
 
-DESIGNS = {"femirax": ("Femirax", femirax_args, qwen3_next_args), "sodedra": ("Sodedra", sodedra_args, qwen3_next_moe_args)}
+def sodedra_moe_args(W):
+    """Every layer with experts (Sodedra has no shared one: one more of them is used)."""
+    a = sodedra_args(W)
+    moe = next(l["mlp"] for l in a.extra["layers"] if l["mlp"]["kind"] == "moe")
+    for l in a.extra["layers"]:
+        l["mlp"] = {**moe, "router": {**moe["router"], "top": TOP + 1, "groups": {"count": 8, "keep": 5}}}
+    return a
+
+
+def qwen3_next_shared_args(W):
+    """Every layer with the same experts and a shared one."""
+    import dataclasses
+    return dataclasses.replace(qwen3_next_moe_args(W), moe_layer_freq=1, n_shared_experts=1, shared_expert_intermediate_size=W // 2)
+
+
+# name -> (title, arguments of the design, {model beside it: its arguments})
+DESIGNS = {"femirax": ("Femirax", femirax_args, {"qwen3_next": qwen3_next_args}),
+           "sodedra": ("Sodedra", sodedra_args, {"qwen3_next": qwen3_next_moe_args}),
+           "lukinex": ("Lukinex", lukinex_args, {"qwen3_next": qwen3_next_shared_args, "sodedra": sodedra_moe_args})}
 
 
 def engine_of(args):
@@ -131,18 +171,20 @@ def measure(args, steps, warmup):
 
 
 def run(design, steps=40, warmup=8, sampler=None):
-    title, make_args, make_closest = DESIGNS[design]
+    title, make_args, beside = DESIGNS[design]
     rows = []
     launches = 0
     if sampler is not None:
         sampler.start()
     for name, W in SIZES.items():
         row = {"width": W}
-        for model, make in ((design, make_args), ("qwen3_next", make_closest)):
+        for model, make in ((design, make_args), *beside.items()):
             row[model] = measure(make(W), steps, max(3, warmup))
         launches += row[design]["launches"]
-        row["prefill_ratio"] = round(row[design]["prefill_tok_s"] / row["qwen3_next"]["prefill_tok_s"], 2)
-        row["decode_ratio"] = round(row[design]["decode_tok_s"] / row["qwen3_next"]["decode_tok_s"], 2)
+        for model in beside:
+            for what in ("prefill", "decode"):
+                row[f"{what}_ratio" + ("" if model == "qwen3_next" else f"_{model}")] = \
+                    round(row[design][f"{what}_tok_s"] / row[model][f"{what}_tok_s"], 2)
         rows.append(row)
     clocks = sampler.stop() if sampler is not None else None
     big = rows[-1][design]
@@ -150,7 +192,7 @@ def run(design, steps=40, warmup=8, sampler=None):
         "metric": f"{title} decode tok/s", "value": big["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": steps,
         "warmup": warmup, "ms_per_step": big["decode_ms"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None,
         "dtype": "bf16", "data": "synthetic tokens, random weights", "impl": "xllm_b200",
-        "config": {"model": f"{title}, {LAYERS} layers, widths {list(SIZES.values())}, beside Qwen3-Next of equal size",
+        "config": {"model": f"{title}, {LAYERS} layers, widths {list(SIZES.values())}, beside {', '.join(beside)} of equal size",
                    "prefill": "4 x 2048 tokens in one step", "decode": "64 sequences behind 512 prompt tokens",
                    "l2": "weights and states larger than L2"},
         "sizes": rows, "gpu_launches": launches, "clocks": clocks}), flush=True)

@@ -502,6 +502,137 @@ def recurrent_rows(results, hbm, tf, tag):
             xb, lg, w1, w2, K, ws=ws, interleaved=True)), nb, 6.0 * T * K * W * I)
 
 
+def latent_rows(results, hbm, tf, tag):
+    """The kernels of Lukinex beside their likes: windows with kept tokens and soft caps against plain windows, convolution and
+    norm ahead of rotation and cache write against the write alone, lightning attention against retention, latent attention
+    against MLA with a rotary part, clamped experts against SiLU, residual updates.  32 heads of 128, width 4096."""
+    from xllm_b200.ops import mla, moe
+    from xllm_b200.ops.glu import ClampedGLU
+    from xllm_b200.ops.linear_attn import LinearAttention
+    from xllm_b200.ops.residual import residual_update
+    dev, bf, H, d, W = "cuda", torch.bfloat16, 32, 128, 4096
+    nq, nkv, R = 32, 8, 512
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    rows = lambda t, n: torch.randn(t, n, device=dev, dtype=bf)
+
+    def report(name, shape, t, nbytes, flops=0.0):
+        ideal = max(nbytes / (hbm * 1e9), flops / (tf * 1e12))
+        results.append(dict(kernel=name, shape=shape, ms=t * 1e3, gbs=nbytes / t / 1e9, tflops=flops / t / 1e12,
+                            frac_of_roofline=ideal / t, peaks=tag))
+        print(f"{name:<38} {shape:<26} {t*1e6:9.1f} us {nbytes/t/1e9:7.0f} GB/s {flops/t/1e12:7.1f} TF/s  {ideal/t:6.3f} of {tag}",
+              flush=True)
+
+    kinds = (("plain", {}), ("kept", dict(keep=16)), ("capped", dict(softcap=30.0)), ("kept, capped", dict(keep=16, softcap=30.0)))
+    for S, L, win in ((4, 2048, 1024), (1, 8192, 1024)):
+        T = S * L
+        kc, vc = (rows(T // 16 * nkv * 16, d).view(T // 16, nkv, 16, d) for _ in range(2))
+        bt = torch.arange(T // 16, device=dev, dtype=torch.int32).view(S, L // 16)
+        cu, kl, q = i32([i * L for i in range(S + 1)]), i32([L] * S), rows(T, nq * d).view(T, nq, d)
+        for name, kw in kinds:
+            keep = kw.get("keep", 0)
+            pairs = sum(min(i + 1, win) + min(keep, max(0, i + 1 - win)) for i in range(L)) * S
+            report(f"window prompts, {name}", f"{S} x {L} window {win}", bench_queued(lambda: ops.paged_prefill_attention(
+                q, kc, vc, bt, cu, kl, L, d ** -0.5, window=win, **kw), iters=5), T * d * 2 * (2 * nq + 2 * nkv), 4.0 * pairs * nq * d)
+    for B, ctx, win in ((64, 4096, 1024), (256, 4096, 1024)):
+        kc, vc = (rows(B * ctx // 16 * nkv * 16, d).view(B * ctx // 16, nkv, 16, d) for _ in range(2))
+        bt = torch.arange(B * ctx // 16, device=dev, dtype=torch.int32).view(B, ctx // 16)
+        kl, q = i32([ctx] * B), rows(B, nq * d).view(B, nq, d)
+        splits = min(ops.decode_splits(B, nkv, nq // nkv), max(1, win // 256))
+        for name, kw in kinds:
+            report(f"window decode, {name}", f"B={B} window {win}", bench_queued(lambda: ops.paged_decode_attention(
+                q, kc, vc, bt, kl, d ** -0.5, window=win, splits=splits, **kw)), 4.0 * B * (win + kw.get("keep", 0)) * nkv * d)
+        del kc, vc
+    for B, ctx in ((16, 8192), (64, 4096), (256, 2048)):
+        bt = (torch.randperm(B * (ctx // 16), device=dev) + 1).view(B, -1).to(torch.int32)
+        sl, pos = i32([ctx] * B), torch.full((B,), ctx - 1, device=dev)
+        for width, name in ((R, "latent decode"), (R + 64, "mla decode (rotary part)")):
+            cache = rows((B * (ctx // 16) + 1) * 16, width).view(-1, 1, 16, width)
+            q, out = rows(B, H * width).view(B, H, width) * 0.3, torch.empty(B, H, R, device=dev, dtype=bf)
+            fn = (lambda: mla.latent_decode(q, cache, bt, 0.09, seq_lens=sl, out=out)) if width == R else \
+                (lambda: mla.decode(q, cache, bt, 0.09, seq_lens=sl, out=out))
+            report(name, f"B={B} ctx {ctx}", bench_queued(fn), 2.0 * B * ctx * width, 2.0 * B * H * ctx * (width + R))
+            del cache
+        uk, q = rows(H * d, R).view(H, d, R), rows(B, H * d).view(B, H, d)
+        qa = torch.empty(B, H, R, device=dev, dtype=bf)
+        report("query into latents (cuBLAS)", f"B={B}", bench_queued(lambda: torch.bmm(q.transpose(0, 1), uk, out=qa.transpose(0, 1))),
+               2.0 * (H * d * R + B * H * (d + R)), 2.0 * B * H * d * R)
+    for S, L in ((4, 512), (4, 2048), (1, 8192)):
+        T, bt = S * L, torch.arange(1, S * L // 16 + 1, device=dev, dtype=torch.int32).view(S, L // 16)
+        cu, kl, pos = i32([i * L for i in range(S + 1)]), i32([L] * S), torch.arange(L, device=dev).repeat(S)
+        seq = torch.arange(S, device=dev, dtype=torch.int32).repeat_interleave(L)
+        pairs = S * L * (L + 1) / 2
+        cache, ukv, q = rows((T // 16 + 1) * 16, R).view(-1, 1, 16, R), rows(2 * H * d, R), rows(T, H * d).view(T, H, d)
+        out, pages = torch.empty(T, H, d, device=dev, dtype=bf), torch.arange(T // 16, device=dev, dtype=torch.int32).view(S, -1)
+
+        def expanded():
+            kv = ops.linear(mla.latent_gather(cache, bt, kl, L), ukv)
+            ops.ragged_prefill_attention(q, kv[:, :H * d], kv[:, H * d:], pages, 16, cu, kl, L, 0.09, out)
+
+        fl = 4.0 * pairs * H * d
+        report("latent prompts, expanded", f"{S} x {L}", bench_queued(expanded, iters=5), 0.0, fl + 4.0 * T * R * H * d)
+        if T <= 2048:
+            qa, oa = rows(T, H * R).view(T, H, R), torch.empty(T, H, R, device=dev, dtype=bf)
+            report("latent prompts, row by row", f"{S} x {L}", bench_queued(lambda: mla.latent_decode(
+                qa, cache, bt, 0.09, positions=pos, bt_rows=seq, out=oa), iters=5), 0.0, 4.0 * pairs * H * R)
+            c2, q2 = rows((T // 16 + 1) * 16, R + 64).view(-1, 1, 16, R + 64), rows(T, H * (R + 64)).view(T, H, R + 64)
+            report("mla prompts, row by row", f"{S} x {L}", bench_queued(lambda: mla.decode(
+                q2, c2, bt, 0.09, positions=pos, bt_rows=seq, out=oa), iters=5), 0.0, 2.0 * pairs * H * (2 * R + 64))
+        del cache
+    decay = torch.linspace(0.9, 0.9995, H, device=dev).log()
+    light = LinearAttention(H, d, d, in_silu=True, rows=True, log_decay=decay, norm_w=torch.ones(H * d, device=dev, dtype=bf))
+    ret = LinearAttention(H, d, d, k_scale=d ** -0.5, log_decay=decay)
+    cut = lambda r: [r[:, i * H * d:(i + 1) * H * d] for i in range(4)]
+    for B in (64, 256):
+        st, c, sl = torch.zeros(B + 1, H, d, d, device=dev), cut(rows(B, 4 * H * d)), i32(list(range(B)))
+        kl, pos, out = i32([100] * B), torch.full((B,), 99, device=dev), torch.empty(B, H * d, device=dev, dtype=bf)
+        for name, op in (("lightning decode", light), ("retention decode", ret)):
+            report(name, f"B={B}", bench_queued(lambda: op.decode(st, sl, kl, pos, *c[:3], g=c[3], out=out)),
+                   2 * B * H * d * d * 4 + B * H * d * 10)
+        del st
+    for S, L in ((4, 2048), (1, 8192)):
+        T, st = S * L, torch.zeros(S + 1, H, d, d, device=dev)
+        c, sl, cu, kl = cut(rows(T, 4 * H * d)), i32(list(range(S))), i32([i * L for i in range(S + 1)]), i32([L] * S)
+        pos, out = torch.arange(L, device=dev).repeat(S), torch.empty(T, H * d, device=dev, dtype=bf)
+        for name, op in (("lightning prompts", light), ("retention prompts", ret)):
+            report(name, f"{S} x {L}", bench_queued(lambda: op.prefill(st, sl, cu, kl, pos, *c[:3], g=c[3], out=out, max_q_len=L), iters=5),
+                   T * H * d * 10 + S * H * d * d * 8, 4.0 * T * H * d * d)
+    C = (nq + 2 * nkv) * d
+    for T in (64, 8192):
+        qkv, cs, wn = rows(T, C), torch.randn(8192, d, device=dev), torch.ones(d, device=dev, dtype=bf)
+        kc = torch.zeros(T // 16 + 2, nkv, 16, d, device=dev, dtype=bf)
+        vc, sl = torch.zeros_like(kc), torch.arange(16, 16 + T, dtype=torch.int32, device=dev)
+        q, k, v = qkv[:, :nq * d], qkv[:, nq * d:(nq + nkv) * d], qkv[:, (nq + nkv) * d:]
+        n = T if T == 64 else 4                                       # decode rows, or four prompts
+        ring, cw, L = torch.zeros(n + 1, 4, C, device=dev, dtype=bf), rows(4, C), T // n
+        conv = (cw, ring, i32(list(range(n))), i32([i * L for i in range(n + 1)]), i32([L if n == 4 else 100] * n))
+        pos, nb = torch.arange(T, device=dev) % 2048, T * d * 4 * (nq + 2 * nkv)
+        write = lambda **kw: ops.rope_norm_kv_write(q, k, v, nq, nkv, d, pos, cs, d, sl, kc, vc, unit_norm=False, **kw)
+        report("rotation + cache write", f"T={T}", bench_queued(lambda: write()), nb)
+        report("norm + rotation + cache write", f"T={T}", bench_queued(lambda: write(q_w=wn, k_w=wn)), nb)
+        report("convolution + rotation + cache write", f"T={T}", bench_queued(lambda: write(conv=conv, long_portions=n == 4)),
+               nb + (T * C * 8 if T == 64 else 0))
+        report("rope_kv (norm)", f"T={T}", bench_queued(lambda: ops.rope_kv_write(
+            qkv, nq, nkv, d, pos, cs, d, slots=sl, k_cache=kc, v_cache=vc, q_norm_w=wn, k_norm_w=wn)), nb)
+        x, y, y2, w = torch.randn(T, W, device=dev), rows(T, W), rows(T, W), torch.ones(W, device=dev, dtype=bf)
+        report("residual, two normed, sum normed", f"T={T}", bench_queued(
+            lambda: residual_update(x, y, w=w, y2=y2, w2=w, coef=0.5, w_sum=w, w_out=w)), T * W * 14)
+        report("residual, two normed", f"T={T}", bench_queued(
+            lambda: residual_update(x, y, w=w, y2=y2, w2=w, coef=0.5, w_out=w)), T * W * 14)
+        cw2, qr = torch.ones(R, device=dev, dtype=bf), 2048
+        lat, cache = rows(T, qr + R), torch.zeros(T // 16 + 2, 1, 16, R, device=dev, dtype=bf)
+        qw = torch.ones(qr, device=dev, dtype=bf)
+        report("latent norms + cache write", f"T={T}", bench_queued(lambda: mla.latent_norm(
+            lat[:, :qr], qw, qr, 1e-6, c=lat[:, qr:], c_w=cw2, slots=sl, cache=cache)), T * (qr + R) * 4)
+        report("rmsnorm", f"T={T}", bench_queued(lambda: ops.rmsnorm(lat[:, :qr], qw, 1e-6)), T * qr * 4)
+        E, K, I = 32, 4, W // 2
+        w1, w2, xb, lg = rows(E * 2 * I, W).view(E, 2 * I, W), rows(E * W, I).view(E, W, I), rows(T, W), torch.randn(T, E, device=dev)
+        ws = moe.shared_workspace(T, K, E, E, W, I, torch.device(dev), bf, W)
+        nb = 2.0 * (min(E, T * K) * 3 * I * W + 2 * T * W)
+        for name, act in (("clamped", ClampedGLU(7.0)), ("SiLU", "silu")):
+            report(f"experts, {name}", f"T={T} E={E} top{K}", bench_queued(lambda: moe.fused_moe(
+                xb, lg, w1, w2, K, ws=ws, interleaved=True, act=act)), nb, 6.0 * T * K * W * I)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--what", default="gemm,decode,prefill,small")
@@ -511,7 +642,8 @@ def main():
     results = []
     for w in a.what.split(","):
         {"gemm": gemm_rows, "decode": decode_rows, "prefill": prefill_rows, "small": small_rows, "gdn": gdn_rows, "mla": mla_rows,
-         "fp8": fp8_rows, "moe": moe_rows, "hybrid": hybrid_rows, "recurrent": recurrent_rows}[w](results, hbm, tf, tag)
+         "fp8": fp8_rows, "moe": moe_rows, "hybrid": hybrid_rows, "recurrent": recurrent_rows,
+         "latent": latent_rows}[w](results, hbm, tf, tag)
     if a.json:
         with open(a.json, "w") as f:
             json.dump(results, f, indent=1)

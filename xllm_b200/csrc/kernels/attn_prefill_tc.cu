@@ -335,7 +335,6 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       const uint32_t saddr = TS0 + sb * 128 + half * 64 + lane_addr;
       const int kv0 = tile_of(j) * kBN + half * 64;
       const bool full_tile = kv0 + 63 <= limit && (kv0 >= low || kv0 + 63 < p.keep);
-      const auto shown = [&](int t) { return t <= limit && (t >= low || t < p.keep); };
       uint32_t sv[64];
       tmem_ld32(saddr, sv);
       tmem_ld32(saddr + 32, sv + 32);
@@ -347,10 +346,20 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
 #pragma unroll
         for (int i = 0; i < 64; ++i) sv[i] = __float_as_uint(soft_cap(__uint_as_float(sv[i]), p.cap));
       }
+      if (!full_tile) {                               // bit i: column i is seen
+        const auto below = [&](int t) {               // columns of positions before t
+          const int n = min(max(t - kv0, 0), 64);
+          return n == 64 ? ~0ull : (1ull << n) - 1;
+        };
+        const unsigned long long seen = below(limit + 1) & (~below(low) | below(p.keep));
+        const uint32_t s0 = (uint32_t)seen, s1 = (uint32_t)(seen >> 32);
+#pragma unroll
+        for (int i = 0; i < 64; ++i)
+          if (!((i < 32 ? s0 : s1) & (1u << (i & 31)))) sv[i] = 0xff800000u;      // -inf
+      }
       float mx = -INFINITY;
 #pragma unroll
-      for (int i = 0; i < 64; ++i)
-        if (full_tile || shown(kv0 + i)) mx = fmaxf(mx, __uint_as_float(sv[i]));
+      for (int i = 0; i < 64; ++i) mx = fmaxf(mx, __uint_as_float(sv[i]));
       smax[(sb * 2 + half) * kBM + row] = mx;
       asm volatile("bar.sync 1, 256;" ::: "memory");
       mx = fmaxf(mx, smax[(sb * 2 + (half ^ 1)) * kBM + row]);
@@ -385,12 +394,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
 #pragma unroll
         for (int e = 0; e < 8; e += 2) {
           const int i = u * 8 + e;
-          float p0 = exp2f(__uint_as_float(sv[i]) * sc - m_use);
-          float p1 = exp2f(__uint_as_float(sv[i + 1]) * sc - m_use);
-          if (!full_tile) {
-            if (!shown(kv0 + i)) p0 = 0.f;
-            if (!shown(kv0 + i + 1)) p1 = 0.f;
-          }
+          const float p0 = exp2f(__uint_as_float(sv[i]) * sc - m_use);
+          const float p1 = exp2f(__uint_as_float(sv[i + 1]) * sc - m_use);
           rs += p0 + p1;
           const __nv_bfloat162 pb = __floats2bfloat162_rn(p0, p1);
           packed[e >> 1] = *reinterpret_cast<const uint32_t*>(&pb);

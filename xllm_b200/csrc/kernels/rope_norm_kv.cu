@@ -169,6 +169,8 @@ __global__ void __launch_bounds__(256) rope_norm_kv_kernel(RopeNormParams<T> p) 
 // of up to four heads, whose 16-byte loads are all issued first (the layout of rope_kv.cu).
 constexpr int kVecHeads = 4;
 
+// NORM: the weighted norm; SAME: value heads of d elements.
+template <bool NORM, bool SAME>
 __global__ void __launch_bounds__(256) rope_norm_kv_vec_kernel(RopeNormParams<bf16> p) {
   const int tph = p.d >> 3, per_pass = 256 / tph;
   const int local = threadIdx.x / tph, g = threadIdx.x - local * tph, e0 = g * 8;
@@ -202,7 +204,7 @@ __global__ void __launch_bounds__(256) rope_norm_kv_vec_kernel(RopeNormParams<bf
       if (h >= heads) continue;
       const bool is_q = h < p.nq;
       raw[u] = *reinterpret_cast<const bf16x8*>((is_q ? p.q : p.k) + t * p.ld + (int64_t)(is_q ? h : h - p.nq) * p.d + e0);
-      if (!is_q && p.v != p.k && p.dv == p.d)
+      if (SAME && !is_q && p.v != p.k)
         val[u] = *reinterpret_cast<const bf16x8*>(p.v + t * p.ld + (int64_t)(h - p.nq) * p.d + e0);
     }
 #pragma unroll
@@ -213,7 +215,7 @@ __global__ void __launch_bounds__(256) rope_norm_kv_vec_kernel(RopeNormParams<bf
 #pragma unroll
       for (int j = 0; j < 8; ++j) x[j] = 0.f;
       if (active) unpack8(raw[u], x);
-      if (p.q_w != nullptr) {
+      if constexpr (NORM) {
         float ss = 0.f;
 #pragma unroll
         for (int j = 0; j < 8; ++j) ss += x[j] * x[j];
@@ -260,14 +262,14 @@ __global__ void __launch_bounds__(256) rope_norm_kv_vec_kernel(RopeNormParams<bf
       const int64_t crow = ((blk * p.nkv + kvh) * p.page + off) * (int64_t)p.d_pad;
       bf16* dst = is_q ? p.q_out + (t * p.nq + h) * p.d_pad : p.k_cache + crow;
       *reinterpret_cast<bf16x8*>(dst + e0) = pack8(x);
-      if (!is_q && p.dv == p.d) *reinterpret_cast<bf16x8*>(p.v_cache + crow + e0) = p.v != p.k ? val[u] : raw[u];
+      if (SAME && !is_q) *reinterpret_cast<bf16x8*>(p.v_cache + crow + e0) = p.v != p.k ? val[u] : raw[u];
       for (int z = p.d + e0; z < p.d_pad; z += p.d) {
         *reinterpret_cast<uint4*>(dst + z) = make_uint4(0, 0, 0, 0);
-        if (!is_q && p.dv == p.d) *reinterpret_cast<uint4*>(p.v_cache + crow + z) = make_uint4(0, 0, 0, 0);
+        if (SAME && !is_q) *reinterpret_cast<uint4*>(p.v_cache + crow + z) = make_uint4(0, 0, 0, 0);
       }
     }
   }
-  if (p.dv == p.d || slot < 0) return;
+  if (SAME || slot < 0) return;
   const int vph = p.d_pad >> 3;                        // vectors of a stored value head
   for (int n = threadIdx.x; n < p.nkv * vph; n += 256) {
     const int h = n / vph, e = (n - h * vph) * 8;
@@ -278,111 +280,139 @@ __global__ void __launch_bounds__(256) rope_norm_kv_vec_kernel(RopeNormParams<bf
 }
 
 // The same sizes behind a convolution of up to four taps (rotate-half layout, no weightless norm): a CTA takes RUN token
-// rows and 256 vectors of eight channels, a thread reads every input of its vector once and keeps the last ones in
-// registers.  grid (runs, parts): the first `qk_parts` parts are q and k, the others v.
+// rows and 256 vectors of V channels; a thread reads every input of its vector once, some rows ahead, and keeps the last
+// ones in registers.  grid (runs, parts): the first `qk_parts` parts are q and k, the others v.
 constexpr int kMaxTaps = 4;
+constexpr int kConvRun = 4;
 
-template <int RUN>
-__global__ void __launch_bounds__(256) conv_rope_kv_kernel(RopeNormParams<bf16> p, int qk_parts) {
+template <int RUN, int V>
+__global__ void __launch_bounds__(256, V == 4 ? 4 : 1) conv_rope_kv_kernel(RopeNormParams<bf16> p, int qk_parts) {
+  constexpr int AHEAD = RUN < 4 ? RUN : 4;
+  struct __align__(V * 2) Vec { bf16 v[V]; };
   __shared__ ConvPlace place[RUN];
-  __shared__ int cache_slot[RUN];
+  __shared__ int64_t cache_row[RUN];                                 // of kv head 0; negative: nothing is cached
   __shared__ int64_t angle_row[RUN];
   const int first = blockIdx.x * RUN;
   pdl_wait();
   pdl_launch_dependents();
-  if (threadIdx.x < RUN) {
-    const int row = first + threadIdx.x;
-    ConvPlace c{-1, 0, 0, 0};
-    int cs = -1;
-    int64_t pos = 0;
-    if (row < p.tokens) {
-      c = conv_place(p, row);
-      cs = p.slots[row];
-      if (p.cos_sin != nullptr) pos = p.positions[row];
-    }
-    place[threadIdx.x] = c;
-    cache_slot[threadIdx.x] = cs;
-    angle_row[threadIdx.x] = (pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos)) * p.rot;
-  }
   const bool is_v = (int)blockIdx.y >= qk_parts;
-  const int size = is_v ? p.dv : p.d, per = size >> 3;               // vectors of a head
+  const int size = is_v ? p.dv : p.d, per = size / V;                // vectors of a head
   const int n = ((int)blockIdx.y - (is_v ? qk_parts : 0)) * 256 + threadIdx.x;
   const int heads = is_v ? p.nkv : p.nq + p.nkv;
   const bool on = n < heads * per;                                   // whole heads are on or not together
-  const int h = on ? n / per : 0, e0 = on ? (n - h * per) * 8 : 0;
+  const int h = on ? n / per : 0, e0 = on ? (n - h * per) * V : 0;
   const bool is_q = !is_v && h < p.nq;
   const int kvh = is_v ? h : h - p.nq;
   const int64_t C = p.channels(), ch = (is_v ? (int64_t)(p.nq + p.nkv) * p.d : 0) + (int64_t)h * size + e0;
   const bf16* x = (is_v ? p.v + (int64_t)h * size : (is_q ? p.q + (int64_t)h * size : p.k + (int64_t)kvh * size)) + e0;
-  bf16x8 in[RUN + kMaxTaps - 1], w[kMaxTaps];
+  const auto fetch = [&](int row) {
+    Vec f{};
+    if (on && row >= 0 && row < p.tokens) f = *reinterpret_cast<const Vec*>(x + row * p.ld);
+    return f;
+  };
+  Vec raw[AHEAD], old[kMaxTaps - 1];
 #pragma unroll
-  for (int r = 0; r < RUN + kMaxTaps - 1; ++r) {
-    const int row = first + r - (kMaxTaps - 1);
-    const bool need = on && row >= 0 && row < p.tokens && r + p.taps >= kMaxTaps;
-    in[r] = need ? *reinterpret_cast<const bf16x8*>(x + row * p.ld) : bf16x8{};
+  for (int r = 0; r < AHEAD; ++r) raw[r] = fetch(first + r);
+#pragma unroll
+  for (int b = 1; b < kMaxTaps; ++b) old[b - 1] = RUN > 1 && b < p.taps ? fetch(first - b) : Vec{};
+  if (threadIdx.x < RUN) {
+    const int row = first + threadIdx.x;
+    ConvPlace c{-1, 0, 0, 0};
+    int64_t pos = 0, at = -1;
+    if (row < p.tokens) {
+      c = conv_place(p, row);
+      const int cs = p.slots[row];
+      if (cs >= 0) at = (int64_t)(cs / p.page) * p.nkv * p.page + cs % p.page;
+      if (p.cos_sin != nullptr) pos = p.positions[row];
+    }
+    place[threadIdx.x] = c;
+    cache_row[threadIdx.x] = at;
+    angle_row[threadIdx.x] = (pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos)) * p.rot;
   }
+  float w[kMaxTaps][V], win[kMaxTaps][V];                            // win[b]: the input b tokens back
 #pragma unroll
-  for (int b = 0; b < kMaxTaps; ++b)
-    w[b] = on && b < p.taps ? *reinterpret_cast<const bf16x8*>(p.conv_w + (p.taps - 1 - b) * C + ch) : bf16x8{};
-  const bf16* nw = is_v ? nullptr : (is_q ? p.q_w : p.k_w);
+  for (int b = 0; b < kMaxTaps; ++b) {
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      w[b][j] = 0.f;
+      win[b][j] = b > 0 ? __bfloat162float(old[b - 1].v[j]) : 0.f;
+    }
+    if (on && b < p.taps) load_f32<V>(p.conv_w + (p.taps - 1 - b) * C + ch, w[b]);
+  }
   const int half = p.rot >> 1;
   const bool turns = !is_v && p.cos_sin != nullptr && e0 < p.rot;
+  const int angle = e0 < half ? e0 : e0 - half;
+  const float sign = e0 < half ? -1.f : 1.f;
   __syncthreads();
 #pragma unroll
   for (int r = 0; r < RUN; ++r) {
     const int row = first + r;
     if (row >= p.tokens) break;
+#pragma unroll
+    for (int j = 0; j < V; ++j) win[0][j] = __bfloat162float(raw[r % AHEAD].v[j]);
+    if (r + AHEAD < RUN) raw[r % AHEAD] = fetch(row + AHEAD);
     const ConvPlace c = place[r];
-    float y[8];
+    const int64_t at = cache_row[r];
+    float y[V];
+    if (c.slot >= 0) {
+      if (c.back < kMaxTaps - 1) {                                   // inputs of earlier steps, or of none
+        const bf16* ring = p.ring + (int64_t)c.slot * p.taps * C + ch;
 #pragma unroll
-    for (int j = 0; j < 8; ++j) y[j] = 0.f;
-    if (on && c.slot >= 0) {
-      bf16* ring = p.ring + (int64_t)c.slot * p.taps * C + ch;
+        for (int b = 1; b < kMaxTaps; ++b) {
+          if (b <= c.back) continue;
+          if (on && b < p.taps && b <= c.pos) load_f32<V>(ring + (c.pos - b) % p.taps * C, win[b]);
+          else {
 #pragma unroll
-      for (int b = 0; b < kMaxTaps; ++b) {
-        if (b >= p.taps || b > c.pos) break;
-        float u[8], f[8];
-        if (b <= c.back) unpack8(in[r + kMaxTaps - 1 - b], u);
-        else load_f32<8>(ring + (c.pos - b) % p.taps * C, u);
-        unpack8(w[b], f);
-#pragma unroll
-        for (int j = 0; j < 8; ++j) y[j] += u[j] * f[j];
+            for (int j = 0; j < V; ++j) win[b][j] = 0.f;
+          }
+        }
+        if (c.alone && on) store_f32<V>(p.ring + ((int64_t)c.slot * p.taps + c.pos % p.taps) * C + ch, win[0]);
       }
-      if (c.alone) *reinterpret_cast<bf16x8*>(ring + c.pos % p.taps * C) = in[r + kMaxTaps - 1];
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        y[j] = win[0][j] * w[0][j];
+#pragma unroll
+        for (int b = 1; b < kMaxTaps; ++b) y[j] = fmaf(win[b][j], w[b][j], y[j]);
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < V; ++j) y[j] = 0.f;
     }
-    const int cs = cache_slot[r];
-    const int64_t blk = cs < 0 ? 0 : cs / p.page;
-    const int64_t crow = ((blk * p.nkv + kvh) * p.page + (cs - (int)blk * p.page)) * (int64_t)p.d_pad;
+#pragma unroll
+    for (int b = kMaxTaps - 1; b > 0; --b)
+#pragma unroll
+      for (int j = 0; j < V; ++j) win[b][j] = win[b - 1][j];
     if (!is_v) {
       if (p.q_w != nullptr) {
         float ss = 0.f;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) ss += y[j] * y[j];
+        for (int j = 0; j < V; ++j) ss += y[j] * y[j];
         for (int o = per >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
         const float inv = 1.f / sqrtf(ss / (float)p.d + p.eps);
-        float f[8];
-        load_f32<8>(nw + e0, f);
+        float f[V];
+        load_f32<V>((is_q ? p.q_w : p.k_w) + e0, f);
 #pragma unroll
-        for (int j = 0; j < 8; ++j) y[j] *= inv * f[j];
+        for (int j = 0; j < V; ++j) y[j] *= inv * f[j];
       }
       if (p.cos_sin != nullptr) {
-        float other[8];
+        float other[V];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) other[j] = __shfl_xor_sync(0xffffffffu, y[j], half >> 3);
+        for (int j = 0; j < V; ++j) other[j] = __shfl_xor_sync(0xffffffffu, y[j], half / V);
         if (turns) {
-          float co[8], si[8];
-          const float* a = p.cos_sin + angle_row[r] + (e0 < half ? e0 : e0 - half);
-          load_f32<8>(a, co);
-          load_f32<8>(a + half, si);
+          float co[V], si[V];
+          const float* a = p.cos_sin + angle_row[r] + angle;
+          load_f32<V>(a, co);
+          load_f32<V>(a + half, si);
 #pragma unroll
-          for (int j = 0; j < 8; ++j) y[j] = e0 < half ? y[j] * co[j] - other[j] * si[j] : y[j] * co[j] + other[j] * si[j];
+          for (int j = 0; j < V; ++j) y[j] = fmaf(y[j], co[j], sign * si[j] * other[j]);
         }
       }
     }
-    if (!on || (!is_q && cs < 0)) continue;
+    if (!on || (!is_q && at < 0)) continue;
+    const int64_t crow = (at + kvh * p.page) * p.d_pad;
     bf16* dst = is_v ? p.v_cache + crow : (is_q ? p.q_out + ((int64_t)row * p.nq + h) * p.d_pad : p.k_cache + crow);
-    *reinterpret_cast<bf16x8*>(dst + e0) = pack8(y);
-    for (int z = size + e0; z < p.d_pad; z += size) *reinterpret_cast<uint4*>(dst + z) = make_uint4(0, 0, 0, 0);
+    store_f32<V>(dst + e0, y);
+    for (int z = size + e0; z < p.d_pad; z += size) *reinterpret_cast<Vec*>(dst + z) = Vec{};
   }
 }
 
@@ -443,13 +473,19 @@ XLLM_API int xllm_rope_norm_kv(const void* q, const void* k, const void* v, int6
           a16(q_out) && a16(k_cache) && a16(v_cache) && (rot == 0 || (rot % 8 == 0 && a16(cos_sin))) && a16(q_w) && a16(k_w) &&
           (interleaved || rot == 0 || (rot % 16 == 0 && (hl & (hl - 1)) == 0))) {
         if (taps == 0) {
-          launch_pdl(rope_norm_kv_vec_kernel, dim3(tokens), dim3(256), 0, s, p);
+          if (q_w == nullptr && d == dv) launch_pdl(rope_norm_kv_vec_kernel<false, true>, dim3(tokens), block, 0, s, p);
+          else if (q_w == nullptr) launch_pdl(rope_norm_kv_vec_kernel<false, false>, dim3(tokens), block, 0, s, p);
+          else if (d == dv) launch_pdl(rope_norm_kv_vec_kernel<true, true>, dim3(tokens), block, 0, s, p);
+          else launch_pdl(rope_norm_kv_vec_kernel<true, false>, dim3(tokens), block, 0, s, p);
           return;
         }
         if (taps <= kMaxTaps && !unit_norm && !(interleaved && rot > 0) && a16(conv_w) && a16(ring)) {
-          const int qk = ((nq + nkv) * tph + 255) / 256, parts = qk + (nkv * (dv >> 3) + 255) / 256;
-          if (long_portions) launch_pdl(conv_rope_kv_kernel<4>, dim3((tokens + 3) / 4, parts), dim3(256), 0, s, p, qk);
-          else launch_pdl(conv_rope_kv_kernel<1>, dim3(tokens, parts), dim3(256), 0, s, p, qk);
+          const int V = d <= 128 ? 4 : 8, qk = ((nq + nkv) * (d / V) + 255) / 256, parts = qk + (nkv * (dv / V) + 255) / 256;
+          const dim3 grid((tokens + kConvRun - 1) / kConvRun, parts), rows(tokens, parts);
+          if (V == 4 && long_portions) launch_pdl(conv_rope_kv_kernel<kConvRun, 4>, grid, block, 0, s, p, qk);
+          else if (V == 4) launch_pdl(conv_rope_kv_kernel<1, 4>, rows, block, 0, s, p, qk);
+          else if (long_portions) launch_pdl(conv_rope_kv_kernel<kConvRun, 8>, grid, block, 0, s, p, qk);
+          else launch_pdl(conv_rope_kv_kernel<1, 8>, rows, block, 0, s, p, qk);
           keep();
           return;
         }
