@@ -38,7 +38,8 @@ struct DecodeParams {
   float scale_log2;
 };
 
-template <int D, int STAGES>
+// EXT: kept first positions and the soft cap
+template <int D, int STAGES, bool EXT>
 __global__ void __launch_bounds__(128) paged_decode_kernel(DecodeParams p) {
   constexpr int CH = D / 8;               // 16-byte chunks per row
   constexpr int TILE_BYTES = 16 * D * 2;  // one 16-token K (or V) tile
@@ -57,17 +58,22 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(DecodeParams p) {
   // touched (their cache blocks may have been given back already)
   const int win_start = p.window > 0 ? max(0, seq_len - p.window) : 0;
   const int tile_first = win_start >> 4;
-  const int kept = min((p.keep + 15) >> 4, tile_first);        // tiles of kept positions ahead of the window's
-  const int skip = tile_first - kept;                          // the walk goes over tiles 0 .. kept - 1, tile_first ..
+  const int kept = EXT ? min((p.keep + 15) >> 4, tile_first) : 0;       // tiles of kept positions ahead of the window's
+  const int skip = EXT ? tile_first - kept : 0;                // the walk goes over tiles 0 .. kept - 1, tile_first ..
+  const int walk0 = EXT ? 0 : tile_first;
   const int tiles_total = ((seq_len + 15) >> 4) - skip;
-  const int tps = (tiles_total + p.splits - 1) / p.splits;
-  const int t_begin = split * tps;
+  const int tps = (tiles_total - walk0 + p.splits - 1) / p.splits;
+  const int t_begin = walk0 + split * tps;
   const int t_end = min(t_begin + tps, tiles_total);
   const auto token_of = [&](int i) {                           // first token of this warp's i-th tile
     const int t = t_begin + warp + 4 * i;
-    return (t < kept ? t : t + skip) << 4;
+    if constexpr (EXT) return (t >= kept ? t + skip : t) << 4;
+    return t << 4;
   };
-  const auto hidden = [&](int tok) { return tok >= seq_len || (tok < win_start && tok >= p.keep); };
+  const auto hidden = [&](int tok) { return tok >= seq_len || (tok < win_start && (!EXT || tok >= p.keep)); };
+  const auto whole = [&](int tok0) {                           // every token of the tile is seen
+    return tok0 + 16 <= seq_len && (tok0 >= win_start || (EXT && tok0 + 16 <= p.keep));
+  };
   const int my_n = (t_end - t_begin - warp + 3) >> 2;  // tiles of this warp (may be <= 0)
   const int rows_valid = min(16, p.group - qt * 16);
   const int head0 = kvh * p.group + qt * 16;
@@ -101,11 +107,12 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(DecodeParams p) {
       const bf16* vb = p.v_cache + base;
       const uint32_t ks = ring + (i % STAGES) * STAGE_BYTES;
       const uint32_t vs = ks + TILE_BYTES;
+      const bool all = EXT && whole(tok0);
 #pragma unroll
       for (int j = 0; j < (16 * CH) / 32; ++j) {
         const int id = lane + j * 32;
         const int r = id / CH, c = id - r * CH;
-        const bool valid = !hidden(tok0 + r);
+        const bool valid = EXT ? all || !hidden(tok0 + r) : tok0 + r < seq_len && tok0 + r >= win_start;
         const int64_t go = valid ? (int64_t)r * D + c * 8 : 0;
         cp_async16(ks + swz<CH>(r, c), kb + go, valid);
         cp_async16(vs + swz<CH>(r, c), vb + go, valid);
@@ -144,13 +151,14 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(DecodeParams p) {
       }
     }
     float mx0 = -INFINITY, mx1 = -INFINITY;
+    const bool all = EXT && whole(tok0);
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int tok = tok0 + nt * 8 + (lane & 3) * 2 + (j & 1);
-        float v = p.cap.out > 0.f ? soft_cap(s[nt][j], p.cap) : s[nt][j] * p.scale_log2;
-        if (hidden(tok)) v = -INFINITY;
+        float v = EXT && p.cap.out > 0.f ? soft_cap(s[nt][j], p.cap) : s[nt][j] * p.scale_log2;
+        if (!all && hidden(tok)) v = -INFINITY;
         s[nt][j] = v;
         if (j < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
       }
@@ -265,22 +273,26 @@ __global__ void attn_merge_kernel(bf16* __restrict__ out, const float* __restric
   }
 }
 
-template <int D, int STAGES>
-static int launch_decode(const DecodeParams& p, int batch, cudaStream_t s) {
+template <int D, int STAGES, bool EXT>
+static int launch_decode_as(const DecodeParams& p, int batch, cudaStream_t s) {
   constexpr int SMEM = 4 * STAGES * 2 * 16 * D * 2;
   static std::atomic<bool> attr_done[64] = {};   // first calls from several host threads may coincide
   int dev = 0;
   cudaGetDevice(&dev);
   if (!attr_done[dev & 63].load(std::memory_order_acquire)) {
-    cudaError_t e = cudaFuncSetAttribute(paged_decode_kernel<D, STAGES>,
+    cudaError_t e = cudaFuncSetAttribute(paged_decode_kernel<D, STAGES, EXT>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
     if (e != cudaSuccess) return (int)e;
     attr_done[dev & 63].store(true, std::memory_order_release);
   }
   const int qtiles = (p.group + 15) / 16;
   dim3 grid(p.nkv * qtiles, batch, p.splits);
-  launch_pdl(paged_decode_kernel<D, STAGES>, dim3(grid), dim3(128), SMEM, s, p);
+  launch_pdl(paged_decode_kernel<D, STAGES, EXT>, dim3(grid), dim3(128), SMEM, s, p);
   return XLLM_LAUNCH_CHECK();
+}
+template <int D, int STAGES>
+static int launch_decode(const DecodeParams& p, int batch, cudaStream_t s) {
+  return p.keep > 0 || p.cap.out > 0.f ? launch_decode_as<D, STAGES, true>(p, batch, s) : launch_decode_as<D, STAGES, false>(p, batch, s);
 }
 
 }  // namespace xllm

@@ -28,7 +28,8 @@ struct PrefillParams {
   float scale_log2;
 };
 
-template <int D>
+// EXT: kept first positions and the soft cap
+template <int D, bool EXT>
 __global__ void __launch_bounds__(128) paged_prefill_kernel(PrefillParams p) {
   constexpr int CH = D / 8;
   constexpr int BM = 64, BN = 64;
@@ -55,9 +56,9 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(PrefillParams p) {
   int kv_end = p.causal ? min(kv_len, shift + m0 + BM) : kv_len;
   int kv_begin = 0;
   if (p.window > 0) kv_begin = max(0, shift + m0 - p.window + 1) & ~(BN - 1);
-  const int kept = min((p.keep + BN - 1) / BN, kv_begin / BN);   // tiles of kept positions ahead of the window's
+  const int kept = EXT ? min((p.keep + BN - 1) / BN, kv_begin / BN) : 0;   // tiles of kept positions ahead of the window's
   const int n_tiles = kept + (kv_end - kv_begin + BN - 1) / BN;
-  const auto token_of = [&](int it) { return it < kept ? it * BN : kv_begin + (it - kept) * BN; };
+  const auto token_of = [&](int it) { return EXT && it < kept ? it * BN : kv_begin + (it - kept) * BN; };
   const int32_t* bt = p.block_table + (int64_t)b * p.bt_stride;
 
   // Q tile -> smem
@@ -137,16 +138,39 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(PrefillParams p) {
       }
     }
     float mx0 = -INFINITY, mx1 = -INFINITY;
+    if constexpr (EXT) {
+      if (p.cap.out > 0.f) {
+#pragma unroll
+        for (int nt = 0; nt < BN / 8; ++nt)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) s[nt][j] = soft_cap(s[nt][j], p.cap);
+      }
+    }
+    const float sc = EXT && p.cap.out > 0.f ? 1.f : p.scale_log2;       // capped scores are in the log2 domain already
+    // the tile lies before the first query of this warp and inside the window of its last one, or among the kept tokens
+    const int qlo = shift + m0 + warp * 16;
+    const bool all = n0 + BN <= kv_len && (!p.causal || n0 + BN - 1 <= qlo) &&
+                     (p.window == 0 || n0 > qlo + 15 - p.window || (EXT && n0 + BN <= p.keep));
+    if (all) {
+#pragma unroll
+      for (int nt = 0; nt < BN / 8; ++nt) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float v = s[nt][j] *= sc;
+          if (j < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
+        }
+      }
+    } else
 #pragma unroll
     for (int nt = 0; nt < BN / 8; ++nt) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int tok = n0 + nt * 8 + (lane & 3) * 2 + (j & 1);
         const int qpos = j < 2 ? qpos0 : qpos1;
-        float v = p.cap.out > 0.f ? soft_cap(s[nt][j], p.cap) : s[nt][j] * p.scale_log2;
+        float v = s[nt][j] * sc;
         bool masked = tok >= kv_len;
         if (p.causal) masked |= tok > qpos;
-        if (p.window > 0) masked |= tok <= qpos - p.window && tok >= p.keep;
+        if (p.window > 0) masked |= tok <= qpos - p.window && (!EXT || tok >= p.keep);
         if (masked) v = -INFINITY;
         s[nt][j] = v;
         if (j < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
@@ -214,21 +238,26 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(PrefillParams p) {
   }
 }
 
-template <int D>
-static int launch_prefill(const PrefillParams& p, int batch, int max_q_len, cudaStream_t s) {
+template <int D, bool EXT>
+static int launch_prefill_as(const PrefillParams& p, int batch, int max_q_len, cudaStream_t s) {
   constexpr int SMEM = 64 * D * 2 + 4 * 64 * D * 2;
   static bool attr_done[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (!attr_done[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(paged_prefill_kernel<D>,
+    cudaError_t e = cudaFuncSetAttribute(paged_prefill_kernel<D, EXT>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
     if (e != cudaSuccess) return (int)e;
     attr_done[dev & 63] = true;
   }
   dim3 grid((max_q_len + 63) / 64, p.nq, batch);
-  paged_prefill_kernel<D><<<grid, 128, SMEM, s>>>(p);
+  paged_prefill_kernel<D, EXT><<<grid, 128, SMEM, s>>>(p);
   return XLLM_LAUNCH_CHECK();
+}
+template <int D>
+static int launch_prefill(const PrefillParams& p, int batch, int max_q_len, cudaStream_t s) {
+  return p.keep > 0 || p.cap.out > 0.f ? launch_prefill_as<D, true>(p, batch, max_q_len, s)
+                                       : launch_prefill_as<D, false>(p, batch, max_q_len, s);
 }
 
 }  // namespace xllm
