@@ -508,6 +508,7 @@ def latent_rows(results, hbm, tf, tag):
     against MLA with a rotary part, clamped experts against SiLU, residual updates.  32 heads of 128, width 4096."""
     from xllm_b200.ops import mla, moe
     from xllm_b200.ops.glu import ClampedGLU
+    from xllm_b200.ops.head_norm import head_norm_gate
     from xllm_b200.ops.linear_attn import LinearAttention
     from xllm_b200.ops.residual import residual_update
     dev, bf, H, d, W = "cuda", torch.bfloat16, 32, 128, 4096
@@ -618,6 +619,9 @@ def latent_rows(results, hbm, tf, tag):
             lambda: residual_update(x, y, w=w, y2=y2, w2=w, coef=0.5, w_sum=w, w_out=w)), T * W * 14)
         report("residual, two normed", f"T={T}", bench_queued(
             lambda: residual_update(x, y, w=w, y2=y2, w2=w, coef=0.5, w_out=w)), T * W * 14)
+        o, g, out, wr = torch.randn(T, 1, W, device=dev), rows(T, W), rows(T, W), torch.ones(W, device=dev, dtype=bf)
+        report("row norm + gate", f"T={T}", bench_queued(lambda: head_norm_gate(o, out, g=g, w=wr, act="sigmoid")), T * W * 8)
+        report("head norm + gate", f"T={T}", bench_queued(lambda: head_norm_gate(o.view(T, H, d), out, g=g, w=wn, act="sigmoid")), T * W * 8)
         cw2, qr = torch.ones(R, device=dev, dtype=bf), 2048
         lat, cache = rows(T, qr + R), torch.zeros(T // 16 + 2, 1, 16, R, device=dev, dtype=bf)
         qw = torch.ones(qr, device=dev, dtype=bf)

@@ -133,6 +133,25 @@ def test_long_prompts_expand_their_latents(tmp_path):
     assert close(both[1:301], want[:300], lim[:300])[0] and close(both[301:], want[:9], lim[:9])[0]
 
 
+@pytest.mark.gpu
+def test_captured_portions_and_expanded_prompts_agree(tmp_path):
+    """Many heads over wide latents: small portions replay captured steps in the absorbed form, large ones run expanded."""
+    cfg = config([latent(16, 128, 128, 32, 300, 0.09), latent(2, 128, 128, 16, 300, 0.09, source=0)], vocab=96, width=64)
+    w = oracle.random_weights(cfg, 3)
+    toks = random_tokens(330, cfg["vocab"], 2)
+    want = expect(cfg, w, toks)
+    lim = row_limits(cfg, w, toks, want, "bfloat16")
+    eng = make_engine(tmp_path, cfg, w, ("cuda:0", "bfloat16"), enable_prefix_cache=False)
+    assert eng.model.max_prefill_graph_tokens == 256 and max(eng.runner.prefill_buckets) == 256
+    for cuts in ([330], [200, 130], [37, 293], [290, 1, 39]):
+        ok, worst = close(feed(eng, "p", toks, cuts), want, lim)
+        assert ok, (cuts, worst)
+    got = [eng.replay_step([("g", toks[a:b], [b - a - 1])]) for a, b in ((0, 200), (200, 330))]
+    assert eng.runner.graph_replays > 0
+    ok, worst = close(torch.cat(got), want[[199, 329]], lim[[199, 329]])
+    assert ok, worst
+
+
 # ------------------------------------------------------------------------------------------- far keys and window edges
 def _one_layer(layer, seed=11):
     """The query of token 91 points along the key of token 92: that key's score stands out among hundreds (attention), or

@@ -135,7 +135,9 @@ class ModelRunner:
         # CUDA graphs: key = (decode rows, prompt-chunk sequences, prompt-chunk token rows, sample mode)
         self.buckets = graph_buckets or default_buckets(max_seqs)
         if prefill_graph_tokens is None:
-            prefill_graph_tokens = [t for t in (128, 256, 512, 1024, 2048) if t <= self.max_tokens]
+            # a model may prefer to run larger prompt chunks eagerly, where it sees their lengths
+            most = min(self.max_tokens, getattr(self.model, "max_prefill_graph_tokens", None) or self.max_tokens)
+            prefill_graph_tokens = [t for t in (128, 256, 512, 1024, 2048) if t <= most]
         self.prefill_buckets = sorted(prefill_graph_tokens) if self.enable_graph else []
         self.prefill_graph_seqs = max(1, int(prefill_graph_seqs))
         self.graphs: Dict[tuple, torch.cuda.CUDAGraph] = {}

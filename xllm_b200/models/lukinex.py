@@ -159,6 +159,13 @@ class LukinexCausalLM(Module):
     def head_dim(self):
         return max([g[2] for g in self.kv_layout() if g] + [64])
 
+    @property
+    def max_prefill_graph_tokens(self):
+        """Latent layers with many heads expand the context of longer prompt portions, whose lengths a captured step hides."""
+        wide = [l.mixer for l in self.layers if isinstance(l.mixer, LatentAttention) and l.mixer.expand_from is not None and
+                l.mixer.heads * l.mixer.width >= 8192]
+        return min([m.expand_from for m in wide]) if wide else None
+
     def _state_shapes(self):
         return {l.idx: l.state_parts() for l in self.layers if l.state_parts()}
 
