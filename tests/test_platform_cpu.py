@@ -57,3 +57,23 @@ def test_capture_lock_excludes_other_threads():
             order.append("capture")
     t.join(timeout=5)
     assert order == ["capture", "other"] and not plat.capturing()
+
+
+def test_no_garbage_collection_during_a_capture():
+    """Freeing a dead engine's graphs in the middle of another one's capture would invalidate it."""
+    import gc
+    from xllm_b200.utils import platform as plat
+    assert gc.isenabled()
+    with plat.graph_capture():
+        assert not gc.isenabled()
+        with plat.graph_capture():
+            assert not gc.isenabled()
+        assert not gc.isenabled()
+    assert gc.isenabled()
+    gc.disable()
+    try:
+        with plat.graph_capture():
+            pass
+        assert not gc.isenabled()
+    finally:
+        gc.enable()

@@ -12,6 +12,7 @@ is a no-op that reports so.
 """
 from __future__ import annotations
 
+import gc
 import os
 import threading
 from contextlib import contextmanager
@@ -128,14 +129,19 @@ def graph_capture():
     """Held by the model runner around warm-up + capture of a CUDA graph.  Anything another thread of the
     process wants to launch meanwhile (a second engine served by the same process, an image pipeline, the
     KV push of a PD pair) takes `device_work()` first and so waits: a launch from another thread on a
-    capturing device would either fail the capture or be recorded into it."""
+    capturing device would either fail the capture or be recorded into it.  The cyclic garbage collector rests
+    meanwhile: it may find an engine that is gone, and freeing that one's graphs would invalidate the capture."""
     with _CAPTURE:
         depth = getattr(_capturing, "depth", 0)
         _capturing.depth = depth + 1
+        collects = gc.isenabled()
+        gc.disable()
         try:
             yield
         finally:
             _capturing.depth = depth
+            if collects:
+                gc.enable()
 
 
 @contextmanager
