@@ -67,6 +67,9 @@ CONFIGS = {
     # a width and a vocabulary that no tensor-core product takes, one expert of four, no rotation, convolution of one tap
     "ragged": config([parallel(3, 3, 22, 22, (11, 2), rotation(0), 0.2, 1, 3.0, 2, 6, 70, [0.9, 0.96], mlp=moe(4, 1, 10, 0.8, 30, 1.5)),
                       latent(2, 10, 34, 9, 15, 0.3), attention(3, 1, 14, 14, (13, 4), rotation(14), 0.3)], vocab=101, width=100),
+    # latents beyond the rows of the tensor-core kernels, heads beyond theirs, a decay of nothing
+    "beyond": config([latent(3, 40, 24, 30, 600, 0.2), attention(2, 1, 320, 264, (19, 3), rotation(64), 0.06),
+                      parallel(2, 2, 16, 16, (12, 12), rotation(16), 0.25, 3, 4.0, 2, 264, 136, [0.0, 0.99])]),
     # only windows: pages between the kept tokens and the window return
     "windows": config([attention(4, 2, 16, 16, (30, 18), rotation(16), 0.25, mlp=moe(4, 2, 16, 1.0, 16, 1.0)),
                        parallel(2, 2, 16, 24, (34, 5), rotation(8), 0.25, 3, 6.0, 2, 16, 24, [0.9, 0.99])]),
