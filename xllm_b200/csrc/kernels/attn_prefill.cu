@@ -26,9 +26,10 @@ struct PrefillParams {
   int keep;                    // with a window: the first `keep` positions stay visible
   SoftCap cap;
   float scale_log2;
+  const float* sink;           // [nq] a score per head that joins the denominator, or null
 };
 
-// EXT: kept first positions and the soft cap
+// EXT: kept first positions, the soft cap and sinks
 template <int D, bool EXT>
 __global__ void __launch_bounds__(128) paged_prefill_kernel(PrefillParams p) {
   constexpr int CH = D / 8;
@@ -98,6 +99,12 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(PrefillParams p) {
 #pragma unroll
   for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float mr0 = -INFINITY, mr1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+  if constexpr (EXT) {
+    if (p.sink != nullptr) {                        // a key with this score and no value
+      mr0 = mr1 = p.sink[h] * 1.4426950408889634f;
+      if ((lane & 3) == 0) l0 = l1 = 1.f;           // the four lanes of a row add their sums
+    }
+  }
   uint32_t qa[KS][4];
   const int qrow0 = m0 + warp * 16 + (lane >> 2);  // query index (within the sequence chunk) of row r0
   const int qpos0 = shift + qrow0, qpos1 = qpos0 + 8;
@@ -256,7 +263,7 @@ static int launch_prefill_as(const PrefillParams& p, int batch, int max_q_len, c
 }
 template <int D>
 static int launch_prefill(const PrefillParams& p, int batch, int max_q_len, cudaStream_t s) {
-  return p.keep > 0 || p.cap.out > 0.f ? launch_prefill_as<D, true>(p, batch, max_q_len, s)
+  return p.keep > 0 || p.cap.out > 0.f || p.sink != nullptr ? launch_prefill_as<D, true>(p, batch, max_q_len, s)
                                        : launch_prefill_as<D, false>(p, batch, max_q_len, s);
 }
 
@@ -266,11 +273,12 @@ static int launch_prefill(const PrefillParams& p, int batch, int max_q_len, cuda
 // causal: query i of a sequence sees cache positions <= kv_len - q_len + i.  window > 0 adds a
 // sliding window of that many positions (including the current one).
 // keep (with a window): the first positions of a sequence that stay visible; softcap (> 0) bounds the scores.
+// sink [nq] fp32 (or null): a score per head whose exponential joins the denominator.
 XLLM_API int xllm_paged_prefill_attn_kept(void* out, int64_t o_stride, const void* q, int64_t q_stride,
                                           const void* k_cache, const void* v_cache, const void* block_table, int bt_stride,
                                           const void* cu_q, const void* kv_lens, int batch, int max_q_len, int nq, int nkv,
                                           int d, int page_size, float scale, int causal, int window, int keep, float softcap,
-                                          void* stream) {
+                                          const void* sink, void* stream) {
   using namespace xllm;
   if (batch == 0 || max_q_len == 0) return 0;
   if (nq % nkv != 0 || keep < 0) return (int)cudaErrorInvalidValue;
@@ -280,7 +288,7 @@ XLLM_API int xllm_paged_prefill_attn_kept(void* out, int64_t o_stride, const voi
   p.cu_q = (const int32_t*)cu_q; p.kv_lens = (const int32_t*)kv_lens; p.q_stride = q_stride;
   p.o_stride = o_stride; p.bt_stride = bt_stride; p.nq = nq; p.nkv = nkv; p.page_size = page_size;
   p.causal = causal; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
-  p.keep = window > 0 ? keep : 0; p.cap = make_soft_cap(scale, softcap);
+  p.keep = window > 0 ? keep : 0; p.cap = make_soft_cap(scale, softcap); p.sink = (const float*)sink;
   cudaStream_t s = (cudaStream_t)stream;
   if (d == 128) return launch_prefill<128>(p, batch, max_q_len, s);
   if (d == 64) return launch_prefill<64>(p, batch, max_q_len, s);
@@ -295,5 +303,5 @@ XLLM_API int xllm_paged_prefill_attn(void* out, int64_t o_stride, const void* q,
                                      int d, int page_size, float scale, int causal, int window,
                                      void* stream) {
   return xllm_paged_prefill_attn_kept(out, o_stride, q, q_stride, k_cache, v_cache, block_table, bt_stride, cu_q, kv_lens,
-                                      batch, max_q_len, nq, nkv, d, page_size, scale, causal, window, 0, 0.f, stream);
+                                      batch, max_q_len, nq, nkv, d, page_size, scale, causal, window, 0, 0.f, nullptr, stream);
 }

@@ -146,6 +146,7 @@ struct Params {
   SoftCap cap;
   float scale_log2;
   int* err;
+  const float* sink;           // [nq] a score per head that joins the denominator, or null
   float* lse;                  // optional [total_q, nq]: log2-domain log-sum-exp of every row's scaled scores
 };
 
@@ -324,6 +325,10 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
     constexpr float kLag = 8.f;
     const float sc = CAP ? 1.f : p.scale_log2;        // capped scores are in the log2 domain already
     float m = -INFINITY, l = 0.f;
+    if (p.sink != nullptr) {                          // a key with this score and no value
+      m = p.sink[h] * 1.4426950408889634f;
+      if (half == 0) l = 1.f;                         // the two halves of a row add their sums
+    }
     bool ok = true;
     const uint32_t oaddr = TO0 + half * 64 + lane_addr;
     // Every thread runs every iteration and every named barrier even after a wait has given up (the
@@ -503,7 +508,7 @@ static int* g_err[64] = {};
 static int prefill_tc(void* out, int64_t o_stride, const void* q, int64_t q_stride, int64_t total_q, const void* k_cache,
                       const void* v_cache, int64_t n_blocks, int64_t kv_ld, const void* block_table, int bt_stride,
                       const void* cu_q, const void* kv_lens, int batch, int max_q_len, int nq, int nkv, int page_size,
-                      float scale, int causal, int window, int keep, float softcap, void* lse, void* stream) {
+                      float scale, int causal, int window, int keep, float softcap, const void* sink, void* lse, void* stream) {
   using namespace xllm;
   using namespace xllm::fmha;
   if (batch == 0 || max_q_len == 0) return 0;
@@ -534,7 +539,7 @@ static int prefill_tc(void* out, int64_t o_stride, const void* q, int64_t q_stri
   p.out = (bf16*)out; p.block_table = (const int32_t*)block_table; p.cu_q = (const int32_t*)cu_q;
   p.kv_lens = (const int32_t*)kv_lens; p.o_stride = o_stride; p.bt_stride = bt_stride; p.nq = nq; p.nkv = nkv;
   p.page = page_size; p.causal = causal; p.window = window; p.scale_log2 = scale * 1.4426950408889634f; p.err = g_err[dev & 63];
-  p.lse = (float*)lse; p.keep = window > 0 ? keep : 0; p.rows_kv = kv_ld > 0; p.cap = make_soft_cap(scale, softcap);
+  p.lse = (float*)lse; p.sink = (const float*)sink; p.keep = window > 0 ? keep : 0; p.rows_kv = kv_ld > 0; p.cap = make_soft_cap(scale, softcap);
   dim3 grid((max_q_len + kBM - 1) / kBM, nq, batch);
   if (softcap > 0.f) prefill_tc_kernel<true><<<grid, 320, SMEM_TOTAL, (cudaStream_t)stream>>>(tq, tk, tv, p);
   else prefill_tc_kernel<false><<<grid, 320, SMEM_TOTAL, (cudaStream_t)stream>>>(tq, tk, tv, p);
@@ -547,18 +552,18 @@ XLLM_API int xllm_paged_prefill_attn_tc_lse(void* out, int64_t o_stride, const v
                                             const void* kv_lens, int batch, int max_q_len, int nq, int nkv,
                                             int page_size, float scale, int causal, int window, void* lse, void* stream) {
   return prefill_tc(out, o_stride, q, q_stride, total_q, k_cache, v_cache, n_blocks, 0, block_table, bt_stride, cu_q, kv_lens,
-                    batch, max_q_len, nq, nkv, page_size, scale, causal, window, 0, 0.f, lse, stream);
+                    batch, max_q_len, nq, nkv, page_size, scale, causal, window, 0, 0.f, nullptr, lse, stream);
 }
 
-// The same with kept first positions beside the window and soft-capped scores (see xllm_paged_prefill_attn_kept).
+// The same with kept first positions beside the window, soft-capped scores and sinks (see xllm_paged_prefill_attn_kept).
 // kv_ld > 0: K and V are matrices [n_blocks * page_size, nkv * 128] of that row stride, a page being page_size rows.
 XLLM_API int xllm_paged_prefill_attn_tc_kept(void* out, int64_t o_stride, const void* q, int64_t q_stride, int64_t total_q,
                                              const void* k_cache, const void* v_cache, int64_t n_blocks, int64_t kv_ld,
                                              const void* block_table, int bt_stride, const void* cu_q, const void* kv_lens,
                                              int batch, int max_q_len, int nq, int nkv, int page_size, float scale, int causal,
-                                             int window, int keep, float softcap, void* stream) {
+                                             int window, int keep, float softcap, const void* sink, void* stream) {
   return prefill_tc(out, o_stride, q, q_stride, total_q, k_cache, v_cache, n_blocks, kv_ld, block_table, bt_stride, cu_q,
-                    kv_lens, batch, max_q_len, nq, nkv, page_size, scale, causal, window, keep, softcap, nullptr, stream);
+                    kv_lens, batch, max_q_len, nq, nkv, page_size, scale, causal, window, keep, softcap, sink, nullptr, stream);
 }
 
 XLLM_API int xllm_paged_prefill_attn_tc(void* out, int64_t o_stride, const void* q, int64_t q_stride, int64_t total_q,

@@ -1,7 +1,7 @@
 // Finishes the raw fp32 head outputs of a recurrence, and gates attention outputs:
 //
 //   out[t, h dv + i] = o[t, h, i] / div[t, h] / rms over the head * w * act(g[t, h dv + i])       head_norm_gate
-//   out[t, h dv + i] = a[t, h, i] * sigmoid(g[t, h dv + i])                                        head_gate
+//   out[t, h dv + i] = a[t, h, i] * sigmoid(g[t, h dv + i])   or sigmoid(g[t, h])                    head_gate
 //
 // every factor optional in the first (a head may be a whole row; w: one weight per element shared by the heads, or one per head and element; act:
 // silu or sigmoid).  The heads of `a` may be stored wider than dv.  A warp owns whole heads.
@@ -209,7 +209,8 @@ __global__ void __launch_bounds__(256) row_norm_gate_kernel(HeadNormParams<T> p)
 
 template <typename T, int V>
 __global__ void __launch_bounds__(256) head_gate_kernel(T* __restrict__ out, const T* __restrict__ a, const T* __restrict__ g,
-                                                        int64_t g_ld, int64_t tokens, int H, int dv, int d_pad) {
+                                                        int64_t g_ld, int64_t tokens, int H, int dv, int d_pad,
+                                                        int per_head) {
   pdl_wait();
   pdl_launch_dependents();
   const int per = dv / V, row = H * per;
@@ -218,6 +219,13 @@ __global__ void __launch_bounds__(256) head_gate_kernel(T* __restrict__ out, con
     const int r = (int)(n - t * row), h = r / per, i = (r - h * per) * V;
     float x[V], z[V];
     load_f32<V>(a + (t * H + h) * d_pad + i, x);
+    if (per_head) {
+      const float f = gate_act<T>(to_f32(g[t * g_ld + h]), 1);
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[j] *= f;
+      store_f32<V>(out + (t * H + h) * (int64_t)dv + i, x);
+      continue;
+    }
     load_f32<V>(g + t * g_ld + (int64_t)h * dv + i, z);
 #pragma unroll
     for (int j = 0; j < V; ++j) x[j] *= gate_act<T>(z[j], 1);
@@ -262,24 +270,24 @@ XLLM_API int xllm_head_norm_gate(void* out, int64_t out_ld, const void* o, const
   return XLLM_LAUNCH_CHECK();
 }
 
-// a [tokens, H, d_pad] -> out [tokens, H * dv] times the sigmoid of g [tokens, H * dv] (row stride g_ld)
+// a [tokens, H, d_pad] -> out [tokens, H * dv] times the sigmoid of g [tokens, H * dv] or (per_head) [tokens, H], row stride g_ld
 XLLM_API int xllm_head_gate(void* out, const void* a, const void* g, int64_t g_ld, int64_t tokens, int H, int dv, int d_pad,
-                            int dtype, void* stream) {
+                            int per_head, int dtype, void* stream) {
   using namespace xllm;
   if (tokens == 0) return 0;
   if (H <= 0 || dv <= 0 || d_pad < dv) return (int)cudaErrorInvalidValue;
   const auto al = [](const void* x) { return (((uintptr_t)x) & 15) == 0; };
-  const bool v8 = dv % 8 == 0 && d_pad % 8 == 0 && g_ld % 8 == 0 && al(out) && al(a) && al(g);
+  const bool v8 = dv % 8 == 0 && d_pad % 8 == 0 && al(out) && al(a) && (per_head || (g_ld % 8 == 0 && al(g)));
   const int64_t want = (tokens * H * (v8 ? dv / 8 : dv) + 255) / 256;
   const dim3 grid((unsigned)(want < 148 * 16 ? want : 148 * 16));
   const auto run = [&](auto tag) {
     using T = decltype(tag);
     if (v8)
       launch_pdl(head_gate_kernel<T, 8>, grid, dim3(256), 0, (cudaStream_t)stream, (T*)out, (const T*)a, (const T*)g, g_ld,
-                 tokens, H, dv, d_pad);
+                 tokens, H, dv, d_pad, per_head);
     else
       launch_pdl(head_gate_kernel<T, 1>, grid, dim3(256), 0, (cudaStream_t)stream, (T*)out, (const T*)a, (const T*)g, g_ld,
-                 tokens, H, dv, d_pad);
+                 tokens, H, dv, d_pad, per_head);
   };
   if (dtype == 0) run(bf16());
   else run(float());

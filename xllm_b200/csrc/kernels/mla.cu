@@ -14,7 +14,8 @@
 //                          of the rotary part of every query head, in one pass over the token
 //   xllm_latent_norm     : the two norms of a layer whose queries go through a latent too: normed query latents out, normed
 //                          latents to the cache rows, no rotary part
-//   xllm_latent_decode   : the decode kernel over caches of latents alone (rows of 128, 256 or 512 values)
+//   xllm_latent_rope_write: the same with a rotated key part beside the latents, and the rotation of the queries, any sizes
+//   xllm_latent_decode   : the decode kernel over rows of 128, 256, 512 or 576 values, with a window and sinks
 //   xllm_latent_gather   : the cached latents of a few sequences as dense rows (prompts expand them to keys and values)
 //   xllm_mla_decode      : split-KV attention of N query rows (nh heads each) against the cache.
 //                          A query row names its own visible length and block-table row, so decode
@@ -64,6 +65,8 @@ struct DecodeParams {
   float* lse_part;             // [N, nh, splits] (log2 domain)
   int64_t q_stride;            // elements between query rows
   int bt_stride, nh, page_size, splits;
+  int window;                  // > 0: a row sees its last `window` tokens only
+  const float* sink;           // [nh] a score per head that joins the denominator, or null
   float scale_log2;
 };
 
@@ -82,9 +85,11 @@ __global__ void __launch_bounds__(kThreads) mla_decode_kernel(DecodeParams p) {
   pdl_wait();
   pdl_launch_dependents();
   const int seq_len = p.seq_lens ? p.seq_lens[n] : (int)p.positions[n] + 1;
+  const int first = p.window > 0 ? max(0, seq_len - p.window) : 0;  // tokens before it are not seen
+  const int tile0 = first >> 4;
   const int tiles_total = (seq_len + 15) >> 4;
-  const int tps = (tiles_total + p.splits - 1) / p.splits;
-  const int t_begin = split * tps;
+  const int tps = (tiles_total - tile0 + p.splits - 1) / p.splits;
+  const int t_begin = tile0 + split * tps;
   const int t_end = min(t_begin + tps, tiles_total);
   const int my_n = (t_end - t_begin - pair + kPairs - 1) / kPairs;  // tiles of this pair (may be <= 0)
   const int rows_valid = min(16, p.nh - qt * 16);
@@ -115,7 +120,7 @@ __global__ void __launch_bounds__(kThreads) mla_decode_kernel(DecodeParams p) {
       for (int j = 0; j < (16 * CH) / 64; ++j) {
         const int id = (half * 32 + lane) + j * 64;
         const int r = id / CH, c = id - r * CH;
-        const bool valid = tok0 + r < seq_len;
+        const bool valid = tok0 + r < seq_len && tok0 + r >= first;
         cp_async16(dst + swz<CH>(r, c), kb + (valid ? (int64_t)r * DQK + c * 8 : 0), valid);
       }
     }
@@ -126,6 +131,12 @@ __global__ void __launch_bounds__(kThreads) mla_decode_kernel(DecodeParams p) {
 #pragma unroll
   for (int i = 0; i < DV / 16; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+  if (p.sink != nullptr && split == 0 && pair == 0) {  // a key with this score and no value, once per row and head
+    const int r = lane >> 2;
+    m0 = r < rows_valid ? p.sink[head0 + r] * 1.4426950408889634f : 0.f;
+    m1 = r + 8 < rows_valid ? p.sink[head0 + r + 8] * 1.4426950408889634f : 0.f;
+    if ((lane & 3) == 0) l0 = l1 = 1.f;               // the four lanes of a row add their sums
+  }
 
 #pragma unroll
   for (int i = 0; i < STAGES - 1; ++i) load_tile(i);
@@ -174,7 +185,7 @@ __global__ void __launch_bounds__(kThreads) mla_decode_kernel(DecodeParams p) {
       for (int j = 0; j < 4; ++j) {
         const int tok = tok0 + nt * 8 + (lane & 3) * 2 + (j & 1);
         float v = s[nt][j] * p.scale_log2;
-        if (tok >= seq_len) v = -INFINITY;
+        if (tok >= seq_len || tok < first) v = -INFINITY;
         s[nt][j] = v;
         if (j < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
       }
@@ -396,16 +407,109 @@ __global__ void __launch_bounds__(128) latent_norm_kernel(LatentNormParams<T> p)
   }
 }
 
-// rows i of sequence s -> out[s * rows_per + i], zero behind the sequence; grid (rows_per / 8, sequences), a warp per row
-__global__ void __launch_bounds__(256) latent_gather_kernel(uint4* __restrict__ out, const uint4* __restrict__ cache,
-                                                            const int32_t* __restrict__ block_table, int bt_stride,
-                                                            const int32_t* __restrict__ kv_lens, int rows_per, int page, int nvec) {
+// One CTA per token.  The cache row of its slot = [rmsnorm(c) * w | zeros | rotated key part at rot_at | zeros]; the rotated part
+// of every query head turns in place and, for the first qa_rows tokens, lands beside absorbed queries as the cache row has it.
+template <typename T>
+struct LatentRopeParams {
+  T* q;                      // [T, heads] with strides ld, q_hs: rotated part at [d, d + rot)
+  const T* c;                // [T, rank + rot], row stride ld
+  const T* c_w;
+  const float* cos_sin;      // [max_pos, rot]: cos | sin
+  const int64_t* positions;
+  const int32_t* slots;      // < 0: nothing is cached
+  T* cache;                  // rows of `width`
+  T* qa;                     // [qa_rows, heads, width]: columns from `rank` on are written, or null
+  int64_t ld, max_pos;
+  int heads, q_hs, d, rank, rot, rot_at, width, qa_rows;
+  float eps;
+};
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256) latent_rope_kernel(LatentRopeParams<T> p) {
+  __shared__ float red[32];
   pdl_wait();
   pdl_launch_dependents();
-  const int s = blockIdx.y, i = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (i >= rows_per) return;
-  uint4* dst = out + ((int64_t)s * rows_per + i) * nvec;
-  const bool in = i < kv_lens[s];
+  const int64_t t = blockIdx.x;
+  int64_t pos = p.positions[t];
+  pos = pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos);
+  const int half = p.rot >> 1;
+  const float *cs = p.cos_sin + pos * p.rot, *sn = cs + half;
+  const int slot = p.slots[t];
+  const T* c = p.c + t * p.ld;
+  float ss = 0.f, first[V];
+  for (int i = threadIdx.x * V; i < p.rank; i += 256 * V) {
+    float f[V];
+    load_f32<V>(c + i, f);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      ss += f[j] * f[j];
+      if (i == (int)threadIdx.x * V) first[j] = f[j];
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)p.rank + p.eps);
+  if (slot >= 0) {
+    T* row = p.cache + (int64_t)slot * p.width;
+    for (int i = threadIdx.x * V; i < p.rank; i += 256 * V) {
+      float f[V], w[V];
+      if (i == (int)threadIdx.x * V) {
+#pragma unroll
+        for (int j = 0; j < V; ++j) f[j] = first[j];
+      } else {
+        load_f32<V>(c + i, f);
+      }
+      load_f32<V>(p.c_w + i, w);
+#pragma unroll
+      for (int j = 0; j < V; ++j) f[j] *= inv * w[j];
+      store_f32<V>(row + i, f);
+    }
+    for (int i = p.rank + threadIdx.x; i < p.width; i += 256)
+      if (i < p.rot_at || i >= p.rot_at + p.rot) row[i] = from_f32<T>(0.f);
+    for (int i = threadIdx.x; i < half; i += 256) {
+      const float a = to_f32(c[p.rank + 2 * i]), b = to_f32(c[p.rank + 2 * i + 1]);
+      row[p.rot_at + 2 * i] = from_f32<T>(a * cs[i] - b * sn[i]);
+      row[p.rot_at + 2 * i + 1] = from_f32<T>(b * cs[i] + a * sn[i]);
+    }
+  }
+  const bool beside = p.qa != nullptr && t < p.qa_rows;
+  for (int n = threadIdx.x; n < p.heads * half; n += 256) {
+    const int h = n / half, i = n - h * half;
+    T* x = p.q + t * p.ld + (int64_t)h * p.q_hs + p.d + 2 * i;
+    const float a = to_f32(x[0]), b = to_f32(x[1]);
+    const T u = from_f32<T>(a * cs[i] - b * sn[i]), v = from_f32<T>(b * cs[i] + a * sn[i]);
+    x[0] = u;
+    x[1] = v;
+    if (beside) {
+      T* y = p.qa + (t * p.heads + h) * p.width + p.rot_at + 2 * i;
+      y[0] = u;
+      y[1] = v;
+    }
+  }
+  if (beside) {
+    const int gap = p.width - p.rank - p.rot;
+    for (int n = threadIdx.x; n < p.heads * gap; n += 256) {
+      const int h = n / gap, i = p.rank + n - h * gap;
+      p.qa[(t * p.heads + h) * p.width + (i < p.rot_at ? i : i + p.rot)] = from_f32<T>(0.f);
+    }
+  }
+}
+
+// Rows start_s + i of sequence s -> out[s * rows_per + i], zero behind the sequence; grid (rows_per / 8, sequences), a warp per
+// row.  start_s: what the window of the sequence's first row in the batch begins with (window 0: the first token); the rows that
+// are left of a sequence go to `lens`.
+__global__ void __launch_bounds__(256) latent_gather_kernel(uint4* __restrict__ out, const uint4* __restrict__ cache,
+                                                            const int32_t* __restrict__ block_table, int bt_stride,
+                                                            const int32_t* __restrict__ kv_lens, const int32_t* __restrict__ cu_q,
+                                                            int32_t* __restrict__ lens, int window, int rows_per, int page,
+                                                            int nvec) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int s = blockIdx.y, n = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (n >= rows_per) return;
+  uint4* dst = out + ((int64_t)s * rows_per + n) * nvec;
+  const int len = kv_lens[s];
+  const int start = window > 0 ? max(0, len - (cu_q[s + 1] - cu_q[s]) - window + 1) : 0, i = start + n;
+  if (lens != nullptr && n == 0 && lane == 0) lens[s] = min(max(len - start, 0), rows_per);
+  const bool in = i < len;
   const uint4* src = cache;
   if (in) src += ((int64_t)block_table[(int64_t)s * bt_stride + i / page] * page + i % page) * nvec;
   for (int v = lane; v < nvec; v += 32) dst[v] = in ? src[v] : make_uint4(0, 0, 0, 0);
@@ -431,7 +535,7 @@ template <int DQK, int DV, int STAGES>
 static int mla_decode_impl(void* out, const void* q, int64_t q_stride, const void* cache, const void* block_table,
                            int bt_stride, const void* seq_lens, const void* positions, const void* bt_rows,
                            int n_rows, int nh, int page_size, float scale, int splits, void* workspace,
-                           void* stream) {
+                           int window, const void* sink, void* stream) {
   using namespace xllm;
   using namespace xllm::mla;
   constexpr int kSmem = DecodeSmem<DQK, DV, STAGES>::total;
@@ -451,7 +555,7 @@ static int mla_decode_impl(void* out, const void* q, int64_t q_stride, const voi
   p.q = (const bf16*)q; p.cache = (const bf16*)cache; p.block_table = (const int32_t*)block_table;
   p.seq_lens = (const int32_t*)seq_lens; p.positions = (const int64_t*)positions; p.bt_rows = (const int32_t*)bt_rows;
   p.out = (bf16*)out; p.q_stride = q_stride; p.bt_stride = bt_stride; p.nh = nh; p.page_size = page_size;
-  p.splits = splits; p.scale_log2 = scale * 1.4426950408889634f;
+  p.splits = splits; p.window = window; p.sink = (const float*)sink; p.scale_log2 = scale * 1.4426950408889634f;
   p.o_part = splits > 1 ? (float*)workspace : nullptr;
   p.lse_part = p.o_part ? p.o_part + (int64_t)n_rows * nh * splits * DV : nullptr;
   cudaStream_t s = (cudaStream_t)stream;
@@ -466,21 +570,26 @@ XLLM_API int xllm_mla_decode(void* out, const void* q, int64_t q_stride, const v
                              int n_rows, int nh, int page_size, float scale, int splits, void* workspace,
                              void* stream) {
   return mla_decode_impl<xllm::mla::kDQK, xllm::mla::kDV, 2>(out, q, q_stride, cache, block_table, bt_stride, seq_lens, positions,
-                                                             bt_rows, n_rows, nh, page_size, scale, splits, workspace, stream);
+                                                             bt_rows, n_rows, nh, page_size, scale, splits, workspace, 0, nullptr,
+                                                             stream);
 }
 
-// The same over caches without a rotary part: q [N, nh, width], cache [n_blocks, page, width], out [N, nh, width], width 128,
-// 256 or 512; workspace of n_rows * nh * splits * (width + 1) floats when splits > 1.
+// The same over other rows: q [N, nh, width], cache [n_blocks, page, width], width 128, 256 or 512 with out [N, nh, width], or
+// width 576 with out [N, nh, 512]; workspace of n_rows * nh * splits * (out width + 1) floats when splits > 1.  window > 0: a row
+// sees its last `window` tokens; sink [nh] fp32 (or null): a score per head whose exponential joins the denominator.
 XLLM_API int xllm_latent_decode(void* out, const void* q, int64_t q_stride, const void* cache, int width, const void* block_table,
                                 int bt_stride, const void* seq_lens, const void* positions, const void* bt_rows, int n_rows,
-                                int nh, int page_size, float scale, int splits, void* workspace, void* stream) {
+                                int nh, int page_size, float scale, int splits, void* workspace, int window, const void* sink,
+                                void* stream) {
+  if (window < 0) return (int)cudaErrorInvalidValue;
   const auto run = [&](auto impl) {
     return impl(out, q, q_stride, cache, block_table, bt_stride, seq_lens, positions, bt_rows, n_rows, nh, page_size, scale,
-                splits, workspace, stream);
+                splits, workspace, window, sink, stream);
   };
   if (width == 128) return run(mla_decode_impl<128, 128, 3>);
   if (width == 256) return run(mla_decode_impl<256, 256, 2>);
   if (width == 512) return run(mla_decode_impl<512, 512, 2>);
+  if (width == xllm::mla::kDQK) return run(mla_decode_impl<xllm::mla::kDQK, xllm::mla::kDV, 2>);
   return (int)cudaErrorInvalidValue;
 }
 
@@ -511,15 +620,44 @@ XLLM_API int xllm_latent_norm(const void* q, const void* q_w, void* q_out, int q
   return XLLM_LAUNCH_CHECK();
 }
 
-// out [n_seqs * rows_per, width] bf16: the first kv_lens[s] rows of sequence s from the cache, then zeros.
+// Normed latents and the rotated key part into the cache rows of the tokens' slots, rotated queries: see LatentRopeParams.
+// q and c are column blocks of rows with stride ld; dtype: 0 bf16, 1 fp32.
+XLLM_API int xllm_latent_rope_write(void* q, int heads, int q_hs, int d, const void* c, const void* c_w, int rank, int rot, int rot_at,
+                                    int64_t ld, const void* cos_sin, int64_t max_pos, const void* positions, const void* slots,
+                                    void* cache, int width, void* qa, int qa_rows, int tokens, float eps, int dtype, void* stream) {
+  using namespace xllm;
+  using namespace xllm::mla;
+  if (tokens == 0) return 0;
+  if (heads <= 0 || rank <= 0 || rot < 0 || rot % 2 || rot_at < rank || width < rot_at + rot || q_hs < d + rot || max_pos <= 0)
+    return (int)cudaErrorInvalidValue;
+  const auto run = [&](auto tag) {
+    using T = decltype(tag);
+    LatentRopeParams<T> p{(T*)q, (const T*)c, (const T*)c_w, (const float*)cos_sin, (const int64_t*)positions,
+                          (const int32_t*)slots, (T*)cache, (T*)qa, ld, max_pos, heads, q_hs, d, rank, rot, rot_at, width,
+                          qa != nullptr ? qa_rows : 0, eps};
+    const auto al = [](const void* x) { return (((uintptr_t)x) & 15) == 0; };
+    if (rank % 8 == 0 && ld % 8 == 0 && width % 8 == 0 && al(c) && al(c_w) && al(cache))
+      launch_pdl(latent_rope_kernel<T, 8>, dim3(tokens), dim3(256), 0, (cudaStream_t)stream, p);
+    else
+      launch_pdl(latent_rope_kernel<T, 1>, dim3(tokens), dim3(256), 0, (cudaStream_t)stream, p);
+  };
+  if (dtype == 0) run(bf16());
+  else run(float());
+  return XLLM_LAUNCH_CHECK();
+}
+
+// out [n_seqs * rows_per, width] bf16: rows of the sequences from the cache, then zeros.  Without a window all kv_lens[s] rows of
+// sequence s; with one only those that the rows of the batch (cu_q [n_seqs + 1]) see, and lens [n_seqs] receives their number.
 XLLM_API int xllm_latent_gather(void* out, const void* cache, const void* block_table, int bt_stride, const void* kv_lens,
-                                int n_seqs, int rows_per, int page, int width, void* stream) {
+                                const void* cu_q, void* lens, int window, int n_seqs, int rows_per, int page, int width,
+                                void* stream) {
   using namespace xllm;
   using namespace xllm::mla;
   if (n_seqs == 0 || rows_per == 0) return 0;
-  if (width % 8 || page <= 0 || (((uintptr_t)out | (uintptr_t)cache) & 15)) return (int)cudaErrorInvalidValue;
+  if (width % 8 || page <= 0 || window < 0 || (window > 0 && (cu_q == nullptr || lens == nullptr)) || (((uintptr_t)out | (uintptr_t)cache) & 15)) return (int)cudaErrorInvalidValue;
   launch_pdl(latent_gather_kernel, dim3((rows_per + 7) / 8, n_seqs), dim3(256), 0, (cudaStream_t)stream, (uint4*)out,
-             (const uint4*)cache, (const int32_t*)block_table, bt_stride, (const int32_t*)kv_lens, rows_per, page, width / 8);
+             (const uint4*)cache, (const int32_t*)block_table, bt_stride, (const int32_t*)kv_lens, (const int32_t*)cu_q,
+             (int32_t*)lens, window, rows_per, page, width / 8);
   return XLLM_LAUNCH_CHECK();
 }
 

@@ -10,6 +10,12 @@
 // row is reduced in the same order whatever batch it arrives in.  No counterpart in the reference, whose
 // residual stream is bf16 (xllm/core/kernels/cuda/norm.cu:43-174).
 //
+// Norm after the sum (a stream that is itself normed, in `groups` consecutive parts of its own mean square each):
+//
+//   x[t] = norm(alpha * x[t] + y[t]) * w;   out[t] = cast(x[t])   or   norm(x[t]) * w_out
+//
+// A part depends on nothing outside it, so the kernel takes every part as a row.
+//
 // Also here: the token-indexed gated activation of a per-token side input, and the fp32 form of the gated
 // activation of a dense MLP.
 #include "vec_io.cuh"
@@ -192,6 +198,104 @@ static int launch_residual(const ResidualParams& p, cudaStream_t s) {
   return XLLM_LAUNCH_CHECK();
 }
 
+struct PostNormParams {
+  float* x;               // [T, hidden] fp32, dense
+  const void* y;          // row stride y_ld
+  const void *w, *w_out;  // [hidden]; w_out null: cast
+  void* out;              // [T, hidden] dense
+  int64_t y_ld, rows;     // rows: tokens * groups
+  int hidden, groups, part;
+  float alpha, eps;
+};
+
+template <typename T, int V, int TPR>
+__global__ void __launch_bounds__(TPR > 256 ? TPR : 256) postnorm_kernel(PostNormParams p) {
+  __shared__ float red[32];
+  const int t = threadIdx.x % TPR;
+  const int64_t row = (int64_t)blockIdx.x * (blockDim.x / TPR) + threadIdx.x / TPR;
+  const bool live = row < p.rows;
+  const int64_t tok = live ? row / p.groups : 0;
+  const int col = live ? (int)(row - tok * p.groups) * p.part : 0;
+  const int nvec = p.part / V;
+  pdl_wait();
+  pdl_launch_dependents();
+  float* xr = p.x + tok * p.hidden + col;
+  const T* yr = reinterpret_cast<const T*>(p.y) + tok * p.y_ld + col;
+  float acc[kResVec][V], br[kResVec][V];
+#pragma unroll
+  for (int i = 0; i < kResVec; ++i) {
+    const int v = t + i * TPR;
+#pragma unroll
+    for (int j = 0; j < V; ++j) acc[i][j] = br[i][j] = 0.f;
+    if (live && v < nvec) {
+      load_f32<V>(xr + v * V, acc[i]);
+      load_f32<V>(yr + v * V, br[i]);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < kResVec; ++i)
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      acc[i][j] = fmaf(p.alpha, acc[i][j], br[i][j]);
+      ss += acc[i][j] * acc[i][j];
+    }
+  float inv = 1.f / sqrtf(row_sum<TPR>(ss, red) / (float)p.part + p.eps);
+  ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < kResVec; ++i) {
+    const int v = t + i * TPR;
+    if (!(live && v < nvec)) continue;
+    float w[V];
+    load_f32<V>(reinterpret_cast<const T*>(p.w) + col + v * V, w);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      acc[i][j] *= inv * w[j];
+      ss += acc[i][j] * acc[i][j];
+    }
+    store_f32<V>(xr + v * V, acc[i]);
+  }
+  if (p.w_out != nullptr) inv = 1.f / sqrtf(row_sum<TPR>(ss, red) / (float)p.part + p.eps);
+  T* orow = reinterpret_cast<T*>(p.out) + tok * p.hidden + col;
+#pragma unroll
+  for (int i = 0; i < kResVec; ++i) {
+    const int v = t + i * TPR;
+    if (!(live && v < nvec)) continue;
+    if (p.w_out != nullptr) {
+      float w[V];
+      load_f32<V>(reinterpret_cast<const T*>(p.w_out) + col + v * V, w);
+#pragma unroll
+      for (int j = 0; j < V; ++j) acc[i][j] *= inv * w[j];
+    }
+    store_f32<V>(orow + v * V, acc[i]);
+  }
+}
+
+template <typename T, int V>
+static int launch_postnorm(const PostNormParams& p, cudaStream_t s) {
+  const int nvec = p.part / V;
+  int tpr = 32;
+  while (tpr < 1024 && nvec > tpr * kResVec) tpr <<= 1;
+  if (nvec > tpr * kResVec) return (int)cudaErrorInvalidValue;
+  const int block = tpr > 256 ? tpr : 256;
+  const int rows = block / tpr;
+  const dim3 grid((unsigned)((p.rows + rows - 1) / rows));
+#define XLLM_POST_CASE(N)                                                  \
+  case N:                                                                  \
+    launch_pdl(postnorm_kernel<T, V, N>, grid, dim3(block), 0, s, p);      \
+    break;
+  switch (tpr) {
+    XLLM_POST_CASE(32)
+    XLLM_POST_CASE(64)
+    XLLM_POST_CASE(128)
+    XLLM_POST_CASE(256)
+    XLLM_POST_CASE(512)
+    XLLM_POST_CASE(1024)
+  }
+#undef XLLM_POST_CASE
+  return XLLM_LAUNCH_CHECK();
+}
+
 // out[t, i] = gelu_tanh(gate[t, i]) * table[ids[t], col0 + i] for i < dim, 0 for dim <= i < dim_pad; V columns a thread.
 template <typename T, int V>
 __global__ void __launch_bounds__(256) gelu_mul_rows_kernel(T* __restrict__ out, const T* __restrict__ gate, int64_t gate_ld,
@@ -223,9 +327,9 @@ __global__ void __launch_bounds__(256) gelu_mul_rows_kernel(T* __restrict__ out,
   }
 }
 
-// out[t, i] = silu(x[t, i]) * x[t, d + i], fp32; limit > 0: the clamped form of clamped_glu
-__global__ void __launch_bounds__(256) silu_mul_f32_kernel(float* __restrict__ out, const float* __restrict__ x, int64_t tokens,
-                                                           int d, int64_t x_ld, float limit, float alpha) {
+// out[t, i] = act(x[t, i]) * x[t, d + i], fp32; act: 0 silu, 2 gelu (tanh form), 3 clamped_glu
+__global__ void __launch_bounds__(256) act_mul_f32_kernel(float* __restrict__ out, const float* __restrict__ x, int64_t tokens,
+                                                          int d, int64_t x_ld, int act, float limit, float alpha) {
   pdl_wait();
   pdl_launch_dependents();
   const int64_t total = tokens * d;
@@ -233,7 +337,9 @@ __global__ void __launch_bounds__(256) silu_mul_f32_kernel(float* __restrict__ o
     const int64_t t = n / d;
     const int i = (int)(n - t * d);
     float z = x[t * x_ld + i], u = x[t * x_ld + d + i];
-    if (limit > 0.f) {
+    if (act == 2) {
+      out[n] = 0.5f * z * (1.f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z))) * u;
+    } else if (act == 3) {
       z = fminf(z, limit);
       out[n] = z / (1.f + expf(-alpha * z)) * (fminf(fmaxf(u, -limit), limit) + 1.f);
     } else {
@@ -303,12 +409,30 @@ XLLM_API int xllm_gelu_mul_rows(void* out, const void* gate, int64_t gate_ld, co
   return XLLM_LAUNCH_CHECK();
 }
 
-XLLM_API int xllm_silu_mul_f32(void* out, const void* x, int64_t tokens, int d, int64_t x_ld, float limit, float alpha,
-                               void* stream) {
+// act: 0 silu, 2 gelu (tanh form), 3 clamped_glu with `limit` and `alpha`.
+XLLM_API int xllm_act_mul_f32(void* out, const void* x, int64_t tokens, int d, int64_t x_ld, int act, float limit, float alpha,
+                              void* stream) {
   using namespace xllm;
   if (tokens == 0) return 0;
+  if (act != 0 && act != 2 && act != 3) return (int)cudaErrorInvalidValue;
   const int64_t want = (tokens * d + 255) / 256;
-  launch_pdl(silu_mul_f32_kernel, dim3((unsigned)(want < 148 * 8 ? want : 148 * 8)), dim3(256), 0, (cudaStream_t)stream,
-             (float*)out, (const float*)x, tokens, d, x_ld, limit, alpha);
+  launch_pdl(act_mul_f32_kernel, dim3((unsigned)(want < 148 * 8 ? want : 148 * 8)), dim3(256), 0, (cudaStream_t)stream,
+             (float*)out, (const float*)x, tokens, d, x_ld, act, limit, alpha);
   return XLLM_LAUNCH_CHECK();
+}
+
+// x [tokens, hidden] fp32 <- norm(alpha x + y) * w in `groups` parts; out [tokens, hidden] the stream cast or normed with w_out.
+// dtype: 0 bf16, 1 fp32 (y, w, w_out, out).
+XLLM_API int xllm_postnorm_update(void* x, const void* y, int64_t y_ld, const void* w, const void* w_out, void* out, int64_t tokens,
+                                  int hidden, int groups, float alpha, float eps, int dtype, void* stream) {
+  using namespace xllm;
+  if (tokens == 0) return 0;
+  if (hidden <= 0 || groups <= 0 || hidden % groups != 0 || x == nullptr || y == nullptr || w == nullptr || out == nullptr)
+    return (int)cudaErrorInvalidValue;
+  PostNormParams p{(float*)x, y, w, w_out, out, y_ld, tokens * groups, hidden, groups, hidden / groups, alpha, eps};
+  const auto a16 = [](const void* q) { return (((uintptr_t)q) & 15) == 0; };
+  const bool v8 = p.part % 8 == 0 && y_ld % 8 == 0 && a16(x) && a16(y) && a16(w) && a16(w_out) && a16(out);
+  cudaStream_t s = (cudaStream_t)stream;
+  if (dtype == 0) return v8 ? launch_postnorm<bf16, 8>(p, s) : launch_postnorm<bf16, 1>(p, s);
+  return v8 ? launch_postnorm<float, 8>(p, s) : launch_postnorm<float, 1>(p, s);
 }

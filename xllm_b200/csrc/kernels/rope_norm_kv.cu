@@ -3,7 +3,10 @@
 //   a short causal convolution over time per channel of q, k and v,
 //   a per-head RMS norm of q and k with a weight shared by the heads,
 //   rotary positions on the first `rot` elements of q and k,
-//   a per-head RMS norm of q and k without a weight.
+//   a per-head RMS norm of q and k without a weight;
+// or, behind the convolution and without rotation (xllm_conv_row_norm_kv):
+//   an RMS norm of all of q, and one of all of k, with a weight per element,
+//   a per-head RMS norm of the values without a weight.
 // k goes to the paged K cache and the values (any column block of the row: their own projection, or the keys as projected)
 // to the V cache.
 //
@@ -431,6 +434,204 @@ __global__ void __launch_bounds__(256) conv_keep_kernel(RopeNormParams<T> p) {
     p.ring[((int64_t)slot * p.taps + (p.kv_lens[b] - n + i) % p.taps) * C + c] = x[(int64_t)(first + i) * p.ld];
 }
 
+// Norms over whole rows.  One CTA takes RUN token rows one after another; a thread owns NV vectors of eight channels of q | k | v,
+// keeps their last inputs in registers, and the sums of squares meet once per row: those of q and k through the
+// warps, those of the values as one number per vector, so that every head adds its own in a fixed order.
+constexpr int kRowThreads = 512;
+
+template <int RUN, int NV>
+__global__ void __launch_bounds__(kRowThreads) conv_row_norm_kernel(RopeNormParams<bf16> p) {
+  __shared__ ConvPlace place[RUN];
+  __shared__ int64_t cache_row[RUN];
+  __shared__ float sums[2][2][kRowThreads / 32];
+  extern __shared__ float vsum[];                                    // [2][value vectors]
+  const int first = blockIdx.x * RUN, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int nq = p.nq * p.d / 8, nk = p.nkv * p.d / 8, nv = p.nkv * p.dv / 8, n = nq + nk + nv;
+  const int64_t C = (int64_t)n * 8;
+  pdl_wait();
+  pdl_launch_dependents();
+  const bf16* src[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int v = threadIdx.x + i * kRowThreads;
+    src[i] = v < nq ? p.q + v * 8 : (v < nq + nk ? p.k + (v - nq) * 8 : p.v + (v - nq - nk) * 8);
+  }
+  const auto fetch = [&](int i, int row) {
+    bf16x8 f{};
+    if ((int)threadIdx.x + i * kRowThreads < n && row >= 0 && row < p.tokens) f = *reinterpret_cast<const bf16x8*>(src[i] + row * p.ld);
+    return f;
+  };
+  constexpr bool HOLD = NV == 1;                                     // weights stay in registers, else in L1
+  const auto weight = [&](int i, int b) {
+    const int v = threadIdx.x + i * kRowThreads;
+    return v < n && b < p.taps ? *reinterpret_cast<const bf16x8*>(p.conv_w + (p.taps - 1 - b) * C + v * 8) : bf16x8{};
+  };
+  bf16x8 w[HOLD ? 1 : NV][HOLD ? kMaxTaps : 1], win[NV][kMaxTaps];   // win[b]: the input b tokens back
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    win[i][0] = fetch(i, first);
+#pragma unroll
+    for (int b = 0; b < kMaxTaps; ++b) {
+      if constexpr (HOLD) w[i][b] = weight(i, b);
+      if (b > 0) win[i][b] = RUN > 1 && b < p.taps ? fetch(i, first - b) : bf16x8{};
+    }
+  }
+  if (threadIdx.x < RUN) {
+    const int row = first + threadIdx.x;
+    ConvPlace c{-1, 0, 0, 0};
+    int64_t at = -1;
+    if (row < p.tokens) {
+      c = conv_place(p, row);
+      const int cs = p.slots[row];
+      if (cs >= 0) at = (int64_t)(cs / p.page) * p.nkv * p.page + cs % p.page;
+    }
+    place[threadIdx.x] = c;
+    cache_row[threadIdx.x] = at;
+  }
+  __syncthreads();
+#pragma unroll 1
+  for (int r = 0; r < RUN; ++r) {
+    const int row = first + r;
+    if (row >= p.tokens) break;
+    const ConvPlace c = place[r];
+    float y[NV][8], qs = 0.f, ks = 0.f;
+    bf16x8 next[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int v = threadIdx.x + i * kRowThreads;
+      next[i] = r + 1 < RUN ? fetch(i, row + 1) : bf16x8{};
+#pragma unroll
+      for (int j = 0; j < 8; ++j) y[i][j] = 0.f;
+      if (c.slot >= 0 && v < n) {
+        bf16* ring = p.ring + (int64_t)c.slot * p.taps * C + v * 8;
+        if (c.back < kMaxTaps - 1) {                                 // inputs of earlier steps, or of none
+#pragma unroll
+          for (int b = 1; b < kMaxTaps; ++b) {
+            if (b <= c.back) continue;
+            win[i][b] = bf16x8{};
+            if (b < p.taps && b <= c.pos) win[i][b] = *reinterpret_cast<const bf16x8*>(ring + (c.pos - b) % p.taps * C);
+          }
+          if (c.alone) *reinterpret_cast<bf16x8*>(ring + c.pos % p.taps * C) = win[i][0];
+        }
+        float ss = 0.f;
+#pragma unroll
+        for (int b = 0; b < kMaxTaps; ++b) {
+          float f[8], g[8];
+          unpack8(win[i][b], f);
+          if constexpr (HOLD) unpack8(w[i][b], g);
+          else unpack8(weight(i, b), g);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) y[i][j] = fmaf(f[j], g[j], y[i][j]);
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ss += y[i][j] * y[i][j];
+        if (v < nq) qs += ss;
+        else if (v < nq + nk) ks += ss;
+        else vsum[(r & 1) * nv + v - nq - nk] = ss;
+      } else if (v >= nq + nk && v < n) {
+        vsum[(r & 1) * nv + v - nq - nk] = 0.f;
+      }
+#pragma unroll
+      for (int b = kMaxTaps - 1; b > 0; --b) win[i][b] = win[i][b - 1];
+      win[i][0] = next[i];
+    }
+    qs = warp_sum(qs);
+    ks = warp_sum(ks);
+    if (lane == 0) {
+      sums[r & 1][0][warp] = qs;
+      sums[r & 1][1][warp] = ks;
+    }
+    __syncthreads();
+    qs = ks = 0.f;
+#pragma unroll
+    for (int i = 0; i < kRowThreads / 32; ++i) {
+      qs += sums[r & 1][0][i];
+      ks += sums[r & 1][1][i];
+    }
+    const float qi = 1.f / sqrtf(qs / (float)(p.nq * p.d) + p.eps), ki = 1.f / sqrtf(ks / (float)(p.nkv * p.d) + p.eps);
+    const int64_t at = cache_row[r];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int v = threadIdx.x + i * kRowThreads;
+      if (v >= n || (v >= nq && at < 0)) continue;
+      const bool is_q = v < nq, is_v = v >= nq + nk;
+      const int u = is_q ? v : (is_v ? v - nq - nk : v - nq), size = is_v ? p.dv : p.d;
+      const int h = u * 8 / size, e = u * 8 - h * size;
+      if (!is_v) {
+        float g[8];
+        load_f32<8>((is_q ? p.q_w : p.k_w) + u * 8, g);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) y[i][j] *= (is_q ? qi : ki) * g[j];
+      } else {
+        float ss = 0.f;
+        for (int k = 0; k < p.dv / 8; ++k) ss += vsum[(r & 1) * nv + h * (p.dv / 8) + k];
+        const float inv = 1.f / sqrtf(ss / (float)p.dv + p.eps);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) y[i][j] *= inv;
+      }
+      bf16* dst = is_q ? p.q_out + ((int64_t)row * p.nq + h) * p.d_pad : (is_v ? p.v_cache : p.k_cache) + (at + h * p.page) * p.d_pad;
+      store_f32<8>(dst + e, y[i]);
+      for (int z = size + e; z < p.d_pad; z += size) *reinterpret_cast<uint4*>(dst + z) = make_uint4(0, 0, 0, 0);
+    }
+  }
+}
+
+// any sizes and taps: one CTA per token row, the convolution is computed twice
+template <typename T>
+__global__ void __launch_bounds__(256) conv_row_norm_any_kernel(RopeNormParams<T> p) {
+  __shared__ float red[32];
+  const int row = blockIdx.x;
+  pdl_wait();
+  pdl_launch_dependents();
+  const ConvPlace c = conv_place(p, row);
+  ConvPlace look = c;
+  look.alone = 0;                                                    // the ring row is stored in the second pass
+  const int64_t nq = (int64_t)p.nq * p.d, nk = (int64_t)p.nkv * p.d;
+  const int slot = p.slots[row];
+  const int64_t at = slot >= 0 ? (int64_t)(slot / p.page) * p.nkv * p.page + slot % p.page : 0;
+  int64_t ch = 0;
+  for (int part = 0; part < 2; ++part) {
+    const int64_t size = part == 0 ? nq : nk;
+    const T* x = (part == 0 ? p.q : p.k) + row * p.ld;
+    const T* w = part == 0 ? p.q_w : p.k_w;
+    float ss = 0.f;
+    for (int64_t i = threadIdx.x; i < size; i += 256) {
+      const float y = conv_one(p, look, x + i, ch + i);
+      ss += y * y;
+    }
+    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)size + p.eps);
+    for (int64_t i = threadIdx.x; i < size; i += 256) {
+      const float y = conv_one(p, c, x + i, ch + i);
+      const int h = (int)(i / p.d), e = (int)(i - (int64_t)h * p.d);
+      if (part == 0) p.q_out[((int64_t)row * p.nq + h) * p.d_pad + e] = from_f32<T>(y * inv * to_f32(w[i]));
+      else if (slot >= 0) p.k_cache[(at + h * p.page) * p.d_pad + e] = from_f32<T>(y * inv * to_f32(w[i]));
+    }
+    const int heads = part == 0 ? p.nq : p.nkv, gap = p.d_pad - p.d;
+    for (int i = threadIdx.x; i < heads * gap; i += 256) {
+      const int h = i / gap, e = p.d + i - h * gap;
+      if (part == 0) p.q_out[((int64_t)row * p.nq + h) * p.d_pad + e] = from_f32<T>(0.f);
+      else if (slot >= 0) p.k_cache[(at + h * p.page) * p.d_pad + e] = from_f32<T>(0.f);
+    }
+    ch += size;
+  }
+  const int lane = threadIdx.x & 31;
+  for (int h = threadIdx.x >> 5; h < p.nkv; h += 8) {
+    const T* x = p.v + row * p.ld + (int64_t)h * p.dv;
+    const int64_t vch = ch + (int64_t)h * p.dv;
+    float ss = 0.f;
+    for (int i = lane; i < p.dv; i += 32) {
+      const float y = conv_one(p, look, x + i, vch + i);
+      ss += y * y;
+    }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)p.dv + p.eps);
+    T* dst = p.v_cache + (at + h * p.page) * p.d_pad;
+    for (int i = lane; i < p.d_pad; i += 32) {
+      const float y = i < p.dv ? conv_one(p, c, x + i, vch + i) : 0.f;
+      if (slot >= 0) dst[i] = from_f32<T>(y * inv);
+    }
+  }
+}
+
 }  // namespace xllm
 
 // dtype: 0 bf16, 1 fp32.  rot <= d, rot even.  dv: size of a value head (d where v is the key block).
@@ -493,6 +694,51 @@ XLLM_API int xllm_rope_norm_kv(const void* q, const void* k, const void* v, int6
     }
     launch_pdl(rope_norm_kv_kernel<T>, grid, block, 0, s, p);
     keep();
+  };
+  if (dtype == 0) run(bf16());
+  else run(float());
+  return XLLM_LAUNCH_CHECK();
+}
+
+// Convolution (taps >= 1), norms of whole q and k rows with weights [nq * d] and [nkv * d], unit norm of every value head, cache
+// write; arguments as above.
+XLLM_API int xllm_conv_row_norm_kv(const void* q, const void* k, const void* v, int64_t ld, void* q_out, void* k_cache, void* v_cache,
+                                   const void* slots, int tokens, int nq, int nkv, int d, int dv, int d_pad, int page, float eps,
+                                   const void* q_w, const void* k_w, const void* conv_w, void* ring, const void* state_slots,
+                                   const void* cu_q, const void* kv_lens, int n_seqs, int taps, int long_portions, int dtype,
+                                   void* stream) {
+  using namespace xllm;
+  if (tokens == 0) return 0;
+  if (d <= 0 || dv <= 0 || d_pad < d || d_pad < dv || page <= 0 || nq <= 0 || nkv <= 0 || q_w == nullptr || k_w == nullptr ||
+      taps < 1 || conv_w == nullptr || ring == nullptr || state_slots == nullptr || cu_q == nullptr || kv_lens == nullptr || n_seqs <= 0)
+    return (int)cudaErrorInvalidValue;
+  cudaStream_t s = (cudaStream_t)stream;
+  const auto run = [&](auto tag) {
+    using T = decltype(tag);
+    RopeNormParams<T> p{};
+    p.q = (const T*)q; p.k = (const T*)k; p.v = (const T*)v; p.ld = ld; p.q_out = (T*)q_out; p.k_cache = (T*)k_cache;
+    p.v_cache = (T*)v_cache; p.slots = (const int32_t*)slots; p.tokens = tokens; p.nq = nq; p.nkv = nkv; p.d = d; p.dv = dv;
+    p.d_pad = d_pad; p.page = page; p.eps = eps; p.q_w = (const T*)q_w; p.k_w = (const T*)k_w; p.conv_w = (const T*)conv_w;
+    p.ring = (T*)ring; p.state_slots = (const int32_t*)state_slots; p.cu_q = (const int32_t*)cu_q;
+    p.kv_lens = (const int32_t*)kv_lens; p.n_seqs = n_seqs; p.taps = taps;
+    bool done = false;
+    if constexpr (sizeof(T) == 2) {
+      const auto a16 = [](const void* x) { return (((uintptr_t)x) & 15) == 0; };
+      const int64_t vecs = p.channels() / 8;
+      const size_t smem = (size_t)nkv * (dv / 8) * 2 * 4;
+      if (d % 8 == 0 && dv % 8 == 0 && d_pad % 8 == 0 && ld % 8 == 0 && taps <= kMaxTaps && vecs <= 3 * kRowThreads && smem <= 32768 &&
+          a16(q) && a16(k) && a16(v) && a16(q_out) && a16(k_cache) && a16(v_cache) && a16(q_w) && a16(k_w) && a16(conv_w) && a16(ring)) {
+        const bool runs = long_portions && tokens > 4 * 148;
+        const dim3 grid(runs ? (tokens + kConvRun - 1) / kConvRun : tokens), block(kRowThreads);
+        const auto go = [&](auto many, auto one) { launch_pdl(runs ? many : one, grid, block, smem, s, p); };
+        if (vecs <= kRowThreads) go(conv_row_norm_kernel<kConvRun, 1>, conv_row_norm_kernel<1, 1>);
+        else if (vecs <= 2 * kRowThreads) go(conv_row_norm_kernel<kConvRun, 2>, conv_row_norm_kernel<1, 2>);
+        else go(conv_row_norm_kernel<kConvRun, 3>, conv_row_norm_kernel<1, 3>);
+        done = true;
+      }
+    }
+    if (!done) launch_pdl(conv_row_norm_any_kernel<T>, dim3(tokens), dim3(256), 0, s, p);
+    if (taps > 1 && long_portions) launch_pdl(conv_keep_kernel<T>, dim3((unsigned)((p.channels() + 255) / 256), n_seqs), dim3(256), 0, s, p);
   };
   if (dtype == 0) run(bf16());
   else run(float());

@@ -193,8 +193,31 @@ def _lukinex_args(cfg: Dict[str, Any], shapes: Dict[str, List[int]]) -> ModelArg
     return a
 
 
+def _vivazen_args(cfg: Dict[str, Any], shapes: Dict[str, List[int]]) -> ModelArgs:
+    """Vivazen configurations list every layer; nothing is left to a tensor's shape."""
+    import copy
+    layers = copy.deepcopy(cfg["layers"])
+    a = ModelArgs(model_type="vivazen", architectures=["Vivazen"], vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
+                  num_hidden_layers=len(layers), rms_norm_eps=float(cfg["norm"]["eps"]), qk_norm=False, tie_word_embeddings=False)
+    att = [l["mixer"] for l in layers if l["type"] == "attention"]
+    latent = [l["mixer"] for l in layers if l["type"] == "latent_attention"]
+    a.num_attention_heads = max([m["heads"] for m in att + latent] + [1])
+    a.num_key_value_heads = max([m["kv_heads"] for m in att] + [1])
+    a.head_dim = max([max(m["dim"], m["vdim"]) for m in att] + [1])
+    a.intermediate_size = max([l["mlp"]["ff"] for l in layers if l.get("mlp")] + [a.hidden_size])
+    a.max_position_embeddings = int(_g(cfg, "max_position_embeddings", default=32768))
+    a.extra = {"layers": layers, "norm_groups": int(cfg["norm"].get("groups", 1)), "postln_alpha": float(cfg["postln_alpha"]),
+               "unbounded_positions": "max_position_embeddings" not in cfg}
+    if not att:
+        # every layer has a window: what lies before the widest one can be given back
+        a.sliding_window = max([int(m["mask"]["size"]) for m in latent] + [0])
+    a.bos_token_id = _g(cfg, "bos_token_id", default=-1)
+    a.eos_token_id, a.stop_token_ids = _eos_list(_g(cfg, "eos_token_id"))
+    return a
+
+
 # `architecture` names whose configurations do not follow the HuggingFace layout: name -> fn(config, tensor shapes)
-_OWN_LAYOUTS = {"femirax": _femirax_args, "sodedra": _sodedra_args, "lukinex": _lukinex_args}
+_OWN_LAYOUTS = {"femirax": _femirax_args, "sodedra": _sodedra_args, "lukinex": _lukinex_args, "vivazen": _vivazen_args}
 
 
 def model_args_from_dict(cfg: Dict[str, Any], shapes: Optional[Dict[str, List[int]]] = None) -> ModelArgs:

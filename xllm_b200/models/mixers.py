@@ -1,7 +1,7 @@
 """Sublayers of hybrid decoders over an fp32 residual stream, with their constants as parameters: decayed linear
 attention (per-head or per-channel decay), the gated delta rule with channel decays, exponentially gated matrix memory,
 attention whose values are its keys, windowed attention with an output gate, windowed attention with kept first tokens,
-attention over cached latents, a gated per-token side input.
+attention over cached latents (with a rotated part, a window, sinks), attention with mixed heads, a gated per-token side input.
 
 Each mixer names its tensors as a checkpoint does (loader names relative to the mixer) and exposes
   width_parts()   the projections it needs of its input, which the owner fuses into one GEMM,
@@ -15,7 +15,7 @@ from typing import Dict, List, Tuple
 import torch
 
 from .. import ops
-from ..ops import mla
+from ..ops import mla, talking
 from ..ops.delta_rule import ChannelDelta
 from ..ops.head_norm import head_gate
 from ..ops.linear_attn import LinearAttention
@@ -29,8 +29,9 @@ def round_up(n, m):
 
 
 class FusedProjection(Module):
-    """Several projections of one input as one GEMM.  `parts`: (loader name, rows); every part starts at a multiple of
-    eight columns of the output (16-byte aligned rows for the kernels behind it; the gaps are zero weights).  `biased`:
+    """Several projections of one input as one GEMM.  `parts`: (loader name, rows) or, for heads stored zero-padded, (loader name,
+    heads, head, head_pad); every part starts at a multiple of eight columns of the output (16-byte aligned rows for the kernels
+    behind it; the gaps are zero weights).  `biased`:
     the parts with a bias (loader name + ".b").  `f32`: the result stays fp32 (few columns: router logits, gates)."""
 
     def __init__(self, in_f: int, parts: List[Tuple[str, int]], dtype, device, biased=(), f32=False):
@@ -38,13 +39,21 @@ class FusedProjection(Module):
         self.f32 = f32
         self.at: Dict[str, Tuple[int, int]] = {}
         off = 0
-        for name, n in parts:
+        heads = {}
+        for name, *size in parts:
+            n = size[0] if len(size) == 1 else size[0] * size[2]
+            if len(size) == 3:
+                heads[name] = size
             self.at[name] = (off, n)
             off += round_up(n, 8)
         self.weight = torch.zeros(off, in_f, dtype=dtype, device=device)
         self._params["weight"] = self.weight
         for name, (o, n) in self.at.items():
             self._loaders[name] = lambda w, o=o, n=n: self.weight[o:o + n].copy_(w.to(self.weight.dtype))
+            if name in heads:
+                h, d, pad = heads[name]
+                self._loaders[name] = lambda w, o=o, n=n, h=h, d=d, pad=pad: \
+                    self.weight[o:o + n].view(h, pad, in_f)[:, :d].copy_(w.view(h, d, in_f).to(self.weight.dtype))
         self.bias = None
         if biased:
             self.bias = self._params["bias"] = torch.zeros(off, dtype=dtype, device=device)
@@ -315,36 +324,70 @@ class KeptWindowAttention(Module):
 
 
 class LatentAttention(Module):
-    """Causal attention without positions over cached latents: queries behind a latent of their own (dq, its norm, uq), one
-    normed latent c per token (dkv, its norm) that all heads share, keys W_uk c and values W_uv c.  Only c is cached.
-    `own_latents` False: the cache is another layer's, which has written this step's rows already.
+    """Causal attention over cached latents: one normed latent c per token (dkv, its norm) that all heads share, keys W_uk c and
+    values W_uv c.  Queries come from a latent of their own (`q_rank` > 0: dq, its norm, uq) or straight from the input (q).
+    Optional: a rotated part beside them (`rope`: the last elements of every query head, one key part per token from the rows of dkv
+    behind the latent, not normed), a sliding window, a sink per head in the softmax denominators, a sigmoid gate per head (g).
+    Only c and the rotated key part are cached.  `own_latents` False: the cache is another layer's, which has written this step's
+    rows already.
 
     Two forms of one sum.  Absorbed: the query of a head is taken into the latent space (q W_uk), attends to the cached rows
     themselves, and W_uv is applied to what comes back; decoding reads one row per token for all heads.  Expanded, for prompts
-    of many tokens: the context's latents become keys and values once per step."""
+    of many tokens: the context's rows become keys and values once per step."""
 
-    def __init__(self, hidden, heads, d, dv, q_rank, rank, scale, eps, dtype, device, own_latents=True):
+    def __init__(self, hidden, heads, d, dv, q_rank, rank, scale, eps, dtype, device, own_latents=True, rope: RotaryEmbedding = None,
+                 window=0, sink=False, gate=False):
         super().__init__()
+        if rope is not None and (q_rank or not own_latents or not rope.interleaved):
+            raise ValueError("rotated latent attention takes its queries from the input, its own latents, and turns neighbours")
+        if int(window) < 0:
+            raise ValueError("the window must not be negative")
         self.heads, self.d, self.dv, self.q_rank, self.rank = heads, d, dv, q_rank, rank
-        self.scale, self.eps, self.own = float(scale), eps, own_latents
-        self.width, self.q_pad = mla.latent_width(rank, dtype, device), round_up(q_rank, 8)
-        self.q_norm = self.add_param("dq.norm", torch.ones(q_rank, dtype=dtype, device=device))
+        self.scale, self.eps, self.own, self.rope, self.window = float(scale), eps, own_latents, rope, int(window)
+        self.rot = rope.rot_dim if rope is not None else 0
+        self.width, self.rot_at, self.v_width = mla.row_layout(rank, self.rot, dtype, device)
+        fast = dtype == torch.bfloat16 and torch.device(device).type == "cuda" and self.v_width in mla.LATENT_WIDTHS
+        # prompt rows from which expanding pays: absorbed, a pair costs 2 width products a head, expanded 256
+        expand = fast and (d == dv == 128 if rope is None else d + self.rot <= 128 and dv <= 128 and self.width >= 256)
+        self.fast, self.expand_from, self.expand_bytes = fast, 256 if expand else None, 2 << 30
+        # head sizes of queries and keys, and of values, as they are stored for the expanded form
+        self.kp, self.vp = (128, 128) if expand else (d + self.rot, dv)
+        self.q_norm = self.sink = None
+        if q_rank:
+            self.q_pad = round_up(q_rank, 8)
+            self.q_norm = self.add_param("dq.norm", torch.ones(q_rank, dtype=dtype, device=device))
+            self.uq = self._params["uq"] = torch.zeros(heads * d, self.q_pad, dtype=dtype, device=device)
+            self._loaders["uq"] = lambda w: self.uq[:, :q_rank].copy_(w.to(dtype))
         self.c_norm = self.add_param("dkv.norm", torch.ones(rank, dtype=dtype, device=device)) if own_latents else None
-        self.uq = self._params["uq"] = torch.zeros(heads * d, self.q_pad, dtype=dtype, device=device)
-        self._loaders["uq"] = lambda w: self.uq[:, :q_rank].copy_(w.to(dtype))
-        # W_uk and W_uv behind one another, their columns padded as the cache's rows are
-        self.ukv = self._params["ukv"] = torch.zeros(heads * (d + dv), self.width, dtype=dtype, device=device)
-        self.uk, self.uv = self.ukv[:heads * d].view(heads, d, self.width), self.ukv[heads * d:].view(heads, dv, self.width)
-        self._loaders["uk"] = lambda w: self.ukv[:heads * d, :rank].copy_(w.to(dtype))
-        self._loaders["uv"] = lambda w: self.ukv[heads * d:, :rank].copy_(w.to(dtype))
+        if sink:
+            self.sink = self.add_param("sink", torch.zeros(heads, dtype=torch.float32, device=device))
+        self.gate = gate
+        # W_uk and W_uv behind one another, their columns padded as the cache's rows are; expanded keys copy the rotated part
+        k_rows, kp, vp = heads * self.kp, self.kp, self.vp
+        self.ukv = self._params["ukv"] = torch.zeros(k_rows + heads * vp, self.width, dtype=dtype, device=device)
+        self.uk = self.ukv[:k_rows].view(heads, kp, self.width)[:, :d, :self.rot_at if self.rot else self.width]
+        self.uv = self.ukv[k_rows:].view(heads, vp, self.width)[:, :dv, :self.v_width]
+        self._loaders["uk"] = lambda w: self.uk[:, :, :rank].copy_(w.view(heads, d, rank).to(dtype))
+        self._loaders["uv"] = lambda w: self.uv[:, :, :rank].copy_(w.view(heads, dv, rank).to(dtype))
+        self.fill_padding()
         self.o = self.add_module("o", Linear(heads * dv, hidden, False, dtype, device))
         self.biased = ()
-        # prompt rows from which expanding pays: absorbed, a pair costs 2 width products a head, expanded d + dv
-        self.expand_from = 256 if dtype == torch.bfloat16 and d == dv == 128 and self.width in mla.LATENT_WIDTHS else None
-        self.expand_bytes = 2 << 30
+
+    def fill_padding(self):
+        """What no checkpoint tensor holds: zeros, and ones that carry the rotated key part into expanded keys."""
+        if not self.rot:
+            return
+        uk, uv = self.uk[:, :, :self.rank].clone(), self.uv[:, :, :self.rank].clone()
+        self.ukv.zero_()
+        self.uk[:, :, :self.rank].copy_(uk)
+        self.uv[:, :, :self.rank].copy_(uv)
+        if self.expand_from is not None:
+            i = torch.arange(self.rot, device=self.ukv.device)
+            self.ukv[:self.heads * self.kp].view(self.heads, self.kp, self.width)[:, self.d + i, self.rot_at + i] = 1.0
 
     def width_parts(self):
-        return [("dq", self.q_rank)] + ([("dkv", self.rank)] if self.own else [])
+        q = ("dq", self.q_rank) if self.q_rank else ("q", self.heads, self.d + self.rot, self.kp)
+        return [q] + ([("dkv", self.rank + self.rot)] if self.own else []) + ([("g", self.heads)] if self.gate else [])
 
     def kv_geometry(self):
         return (1, 1, self.width) if self.own else None
@@ -354,55 +397,125 @@ class LatentAttention(Module):
 
     def _expandable(self, rows, cache, meta: AttentionMetadata):
         """Rows a sequence's context takes when the prompts of this step run expanded, or 0."""
-        if self.expand_from is None or not rows.is_cuda or meta.padded or meta.max_kv_len <= 0:
-            return 0
+        longest = meta.max_kv_len if not meta.padded and meta.max_kv_len > 0 else 0
         page = cache.shape[-2]
-        per = round_up(meta.max_kv_len, page)
+        if self.expand_from is None or not rows.is_cuda or page not in (16, 32, 64, 128):
+            return 0
+        if self.window:                               # a portion sees itself and what its first row's window holds
+            longest = min(longest or meta.block_table.shape[1] * page, meta.max_q_len + self.window - 1)
+        if longest <= 0:
+            return 0
+        per = round_up(longest, 128)
         small = rows.shape[0] - meta.n_decode < self.expand_from
         big = meta.n_prefill * per * self.ukv.shape[0] * 2 > self.expand_bytes
-        return 0 if small or big or page not in (16, 32, 64, 128) else per
+        return 0 if small or big else per
 
-    def _absorbed(self, q, cache, positions, meta: AttentionMetadata, prompts, out):
-        """out [T, heads, dv] from q [T, heads, d]: of the decode rows alone, or (`prompts`) of all rows."""
+    def _absorbed(self, q, qa, cache, positions, meta: AttentionMetadata, prompts, out):
+        """out [T, heads, >= dv] from q [T, heads, >= d]: of the decode rows alone, or (`prompts`) of all rows.  qa: where queries in
+        the latent space go, with their rotated parts in place."""
         nd = meta.n_decode
         T = q.shape[0] if prompts else nd
-        q, out, alloc = q[:T], out[:T], torch.zeros if meta.padded else torch.empty
-        qa = torch.empty((T, self.heads, self.width), dtype=q.dtype, device=q.device)
-        torch.bmm(q.transpose(0, 1), self.uk, out=qa.transpose(0, 1))
-        oa = alloc(qa.shape, dtype=q.dtype, device=q.device)
+        q, out, alloc = q[:T, :, :self.d], out[:T, :, :self.dv], torch.zeros if meta.padded else torch.empty
+        if qa is None:
+            qa = torch.empty((T, self.heads, self.width), dtype=q.dtype, device=q.device)
+        torch.bmm(q.transpose(0, 1), self.uk, out=qa[:T, :, :self.uk.shape[2]].transpose(0, 1))
+        oa = alloc((T, self.heads, self.v_width), dtype=q.dtype, device=q.device)
         n = meta.n_seqs if prompts else nd
         bt, lens, cu = meta.block_table[:n], meta.kv_lens[:n], meta.cu_q[:n + 1]
-        if not q.is_cuda or q.dtype != torch.bfloat16 or self.width not in mla.LATENT_WIDTHS:
-            ops.paged_attention_generic(qa, cache, cache, bt, cu, lens, self.scale, out=oa)
+        seen = dict(window=self.window, sink=self.sink)
+        if not q.is_cuda or not self.fast:
+            ops.paged_attention_generic(qa, cache, cache, bt, cu, lens, self.scale, out=oa, **seen)
         else:
             if nd > 0:
-                mla.latent_decode(qa[:nd], cache, bt, self.scale, seq_lens=lens[:nd], out=oa[:nd])
+                mla.latent_decode(qa[:nd], cache, bt, self.scale, seq_lens=lens[:nd], out=oa[:nd], **seen)
             if T > nd and self.width <= 256:
                 # the latents as keys and values of one head that all query heads share
-                ops.paged_prefill_attention(qa, cache, cache, bt[nd:], cu[nd:], lens[nd:], meta.max_q_len, self.scale, out=oa)
+                ops.paged_prefill_attention(qa, cache, cache, bt[nd:], cu[nd:], lens[nd:], meta.max_q_len, self.scale, out=oa, **seen)
             elif T > nd:
                 row = torch.arange(nd, T, device=q.device, dtype=torch.int32)
                 seq = torch.bucketize(row, cu[nd + 1:].contiguous(), right=True).clamp_(max=meta.n_prefill - 1)
                 mla.latent_decode(qa[nd:], cache, bt, self.scale, positions=positions[nd:], bt_rows=(seq + nd).to(torch.int32),
-                                  out=oa[nd:])
+                                  out=oa[nd:], **seen)
         torch.bmm(oa.transpose(0, 1), self.uv.transpose(1, 2), out=out.transpose(0, 1))
 
     def forward(self, fused: FusedProjection, rows, positions, meta: AttentionMetadata, kv, state):
         cache, nd, T = kv[0], meta.n_decode, rows.shape[0]
-        c = dict(c=fused.part(rows, "dkv"), c_w=self.c_norm, slots=meta.slots, cache=cache) if self.own else {}
-        cq = mla.latent_norm(fused.part(rows, "dq"), self.q_norm, self.q_pad, self.eps, **c)
-        q = ops.linear(cq, self.uq).view(T, self.heads, self.d)
-        out = torch.empty((T, self.heads, self.dv), dtype=rows.dtype, device=rows.device)
-        per = self._expandable(rows, cache, meta) if meta.n_prefill > 0 else 0
+        per, qa = self._expandable(rows, cache, meta) if meta.n_prefill > 0 else 0, None
+        if self.q_rank:
+            c = dict(c=fused.part(rows, "dkv"), c_w=self.c_norm, slots=meta.slots, cache=cache) if self.own else {}
+            cq = mla.latent_norm(fused.part(rows, "dq"), self.q_norm, self.q_pad, self.eps, **c)
+            q = ops.linear(cq, self.uq)
+        else:
+            q = fused.part(rows, "q")
+            absorbed = nd if per else T
+            if absorbed:
+                qa = torch.empty((absorbed, self.heads, self.width), dtype=rows.dtype, device=rows.device)
+            mla.rope_write(q, self.heads, self.d, fused.part(rows, "dkv"), self.c_norm, self.rank, self.rot, self.rot_at,
+                           self.rope.cos_sin, positions, meta.slots, cache, self.eps, qa=qa, qa_rows=absorbed)
+        q = q.unflatten(1, (self.heads, self.kp if not self.q_rank else self.d))
+        out = (torch.zeros if meta.padded and per else torch.empty)((T, self.heads, self.vp), dtype=rows.dtype, device=rows.device)
         if per:
-            n, page = meta.n_prefill, cache.shape[-2]
-            kv_rows = ops.linear(mla.latent_gather(cache, meta.block_table[nd:], meta.kv_lens[nd:], per), self.ukv)
+            n, page, kvp = meta.n_prefill, 128, self.heads * self.kp
+            lens = meta.kv_lens[nd:]
+            dense = mla.latent_gather(cache, meta.block_table[nd:], lens, per, meta.cu_q[nd:], self.window)
+            if self.window:
+                dense, lens = dense
+            kv_rows = ops.linear(dense, self.ukv)
             pages = torch.arange(n * per // page, dtype=torch.int32, device=rows.device).view(n, per // page)
-            ops.ragged_prefill_attention(q, kv_rows[:, :self.heads * self.d], kv_rows[:, self.heads * self.d:], pages, page,
-                                         meta.cu_q[nd:], meta.kv_lens[nd:], meta.max_q_len, self.scale, out)
+            ops.ragged_prefill_attention(q, kv_rows[:, :kvp], kv_rows[:, kvp:], pages, page, meta.cu_q[nd:], lens, meta.max_q_len,
+                                         self.scale, out, window=self.window, sink=self.sink)
         if nd > 0 or not per:
-            self._absorbed(q, cache, positions, meta, not per, out)
-        return self.o(out.view(T, self.heads * self.dv))
+            self._absorbed(q, qa, cache, positions, meta, not per, out)
+        if self.gate:
+            return self.o(head_gate(out, fused.part(rows, "g"), self.dv))
+        return self.o(out[..., :self.dv].reshape(T, self.heads * self.dv))
+
+    __call__ = forward
+
+
+class TalkingAttention(Module):
+    """Causal GQA behind short convolutions on q, k and v: all of q and all of k normed together with weights, every value head over
+    its own root mean square, no positions, a soft cap on the scores, and softmax weights mixed across heads (talk [heads, heads])
+    before they meet the values (ops/talking.py)."""
+
+    def __init__(self, hidden, heads, kv_heads, d, dv, scale, softcap, taps, eps, dtype, device):
+        super().__init__()
+        if heads % kv_heads:
+            raise ValueError("the query heads must be a multiple of the key/value heads")
+        if int(taps) < 1 or float(softcap) < 0:
+            raise ValueError("the convolution has a tap at least, and the soft cap must not be negative")
+        self.heads, self.kv_heads, self.d, self.dv, self.eps = heads, kv_heads, d, dv, eps
+        self.scale, self.softcap, self.taps = float(scale), float(softcap), int(taps)
+        self.d_pad = talking.head_size(d, dv, dtype, device)
+        self.q_norm = self.add_param("q.norm", torch.ones(heads * d, dtype=dtype, device=device))
+        self.k_norm = self.add_param("k.norm", torch.ones(kv_heads * d, dtype=dtype, device=device))
+        self.talk = self.add_param("talk", torch.zeros(heads, heads, dtype=dtype, device=device))
+        self.conv = self._params["conv"] = torch.zeros(self.taps, sum(w for _, w in self.width_parts()), dtype=dtype, device=device)
+        at = 0
+        for n, c in self.width_parts():
+            self._loaders[n + ".conv"] = lambda w, o=at, c=c: self.conv[:, o:o + c].copy_(w.reshape(c, self.taps).T.to(dtype))
+            at += c
+        self.o = self.add_module("o", Linear(heads * dv, hidden, False, dtype, device))
+        self.biased = ()
+
+    def width_parts(self):
+        return [("q", self.heads * self.d), ("k", self.kv_heads * self.d), ("v", self.kv_heads * self.dv)]
+
+    def kv_geometry(self):
+        return (2, self.kv_heads, self.d_pad)
+
+    def state_parts(self):
+        return {"conv": (tuple(self.conv.shape), self.conv.dtype)}
+
+    def forward(self, fused: FusedProjection, rows, positions, meta: AttentionMetadata, kv, state):
+        q, k, v = (fused.part(rows, n) for n in "qkv")
+        k_cache, v_cache = kv
+        q = talking.conv_row_norm_kv_write(q, k, v, self.heads, self.kv_heads, self.d, meta.slots, k_cache, v_cache, self.q_norm,
+                                           self.k_norm, (self.conv, state["conv"], meta.state_slots, meta.cu_q, meta.kv_lens),
+                                           eps=self.eps, long_portions=meta.n_prefill > 0)
+        out = (torch.zeros if meta.padded else torch.empty)((q.shape[0], self.heads, self.dv), dtype=q.dtype, device=q.device)
+        talking.attention(q, k_cache, v_cache, meta, self.scale, self.softcap, self.talk, self.dv, out)
+        return self.o(out.view(q.shape[0], self.heads * self.dv))
 
     __call__ = forward
 

@@ -79,13 +79,13 @@ def act_and_mul(x, act="silu", out=None):
     if not x.is_cuda:
         return reference.act_and_mul(x, act)
     code, limit, alpha = glu.code(act)
-    if x.dtype == torch.float32 and code in (0, 3):
+    if x.dtype == torch.float32 and code in (0, 2, 3):
         d = x.shape[-1] // 2
         x2 = x.reshape(-1, 2 * d)
         if out is None:
             out = torch.empty((x2.shape[0], d), dtype=x.dtype, device=x.device)
-        check(_lib_().xllm_silu_mul_f32(ptr(out), ptr(x2), x2.shape[0], d, x2.stride(0), limit, alpha, stream()),
-              "silu_mul_f32")
+        check(_lib_().xllm_act_mul_f32(ptr(out), ptr(x2), x2.shape[0], d, x2.stride(0), code, limit, alpha, stream()),
+              "act_mul_f32")
         _count()
         return out.reshape(*x.shape[:-1], d)
     _bf16(x, "act_and_mul")
@@ -187,15 +187,23 @@ def attention_head_size(d):
     return next((s for s in (64, 128, 256) if d <= s), d)
 
 
+def _sink(sink, nq, name):
+    """fp32 [nq] score per head that joins the softmax denominator, or None."""
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != nq or not sink.is_contiguous()):
+        raise TypeError(f"{name}: sinks are fp32, one per query head")
+    return sink
+
+
 def paged_attention_generic(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, out=None, row0=0, rows=None, window=0,
-                            keep=0, softcap=0.0):
+                            keep=0, softcap=0.0, sink=None):
     """Rows [row0, row0 + rows) of q [T, nq, d], decode rows and prompt chunks alike (row ranges by cu_q), fp32 or bf16
     caches, any head size up to 1024: the path of the fp32 execution type.  With a window the first `keep` positions of a
-    sequence stay visible; softcap > 0: scores become softcap * tanh(score / softcap)."""
+    sequence stay visible; softcap > 0: scores become softcap * tanh(score / softcap); sink [nq] fp32: exp(sink) joins every
+    denominator of its head."""
     T, nq, d = q.shape
     rows = T - row0 if rows is None else rows
     if not q.is_cuda:
-        y = reference.paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, True, window, keep, softcap)
+        y = reference.paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, True, window, keep, softcap, sink)
         if out is not None:
             out[row0:row0 + rows].copy_(y[row0:row0 + rows])
             return out
@@ -208,7 +216,8 @@ def paged_attention_generic(q, k_cache, v_cache, block_table, cu_q, kv_lens, sca
     check(_lib_().xllm_paged_attn_generic(ptr(out), out.stride(0), ptr(q), q.stride(0), ptr(k_cache), ptr(v_cache),
                                           ptr(block_table), block_table.stride(0), ptr(cu_q), ptr(kv_lens), kv_lens.shape[0],
                                           row0, rows, nq, k_cache.shape[1], d, k_cache.shape[2], scale, int(window or 0),
-                                          int(keep), float(softcap or 0.0), 0 if q.dtype == torch.bfloat16 else 1, stream()), "paged_attn_generic")
+                                          int(keep), float(softcap or 0.0), ptr(_sink(sink, nq, "paged_attention_generic")),
+                                          0 if q.dtype == torch.bfloat16 else 1, stream()), "paged_attn_generic")
     _count()
     return out
 
@@ -288,15 +297,15 @@ def paged_decode_attention(q, k_cache, v_cache, block_table, seq_lens, scale, sp
 
 
 def paged_prefill_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, max_q_len, scale,
-                            causal=True, window=0, out=None, keep=0, softcap=0.0):
-    """q: [T, nq, d] ragged by cu_q -> [T, nq, d]; attends to cache positions [0, kv_len); window, keep, softcap as in
-    paged_decode_attention."""
+                            causal=True, window=0, out=None, keep=0, softcap=0.0, sink=None):
+    """q: [T, nq, d] ragged by cu_q -> [T, nq, d]; attends to cache positions [0, kv_len); window, keep, softcap, sink as in
+    paged_attention_generic."""
     if _debug.enabled():
         _debug.check_block_table(block_table, kv_lens, k_cache.shape[0], k_cache.shape[2], "paged_prefill_attention")
         _debug.check_range(cu_q, 0, q.shape[0] + 1, "paged_prefill_attention cu_q")
     if not q.is_cuda:
         y = reference.paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale,
-                                      causal, window, keep, softcap)
+                                      causal, window, keep, softcap, sink)
         if out is not None:
             r0 = int(cu_q[0])
             out[r0:].copy_(y[r0:])
@@ -319,20 +328,21 @@ def paged_prefill_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, max
                                                       ptr(v_cache), k_cache.shape[0], 0, ptr(block_table),
                                                       block_table.stride(0), ptr(cu_q), ptr(kv_lens), B, int(max_q_len),
                                                       nq, nkv, page, scale, int(causal), int(window), int(keep),
-                                                      float(softcap or 0.0), stream()), "paged_prefill_attn_tc")
+                                                      float(softcap or 0.0), ptr(_sink(sink, nq, "paged_prefill_attention")),
+                                                      stream()), "paged_prefill_attn_tc")
         _count()
         return out
     check(_lib_().xllm_paged_prefill_attn_kept(ptr(out), out.stride(0), ptr(q), q.stride(0), ptr(k_cache),
                                                ptr(v_cache), ptr(block_table), block_table.stride(0),
                                                ptr(cu_q), ptr(kv_lens), B, int(max_q_len), nq, nkv, d,
                                                page, scale, int(causal), int(window), int(keep), float(softcap or 0.0),
-                                               stream()), "paged_prefill_attn")
+                                               ptr(_sink(sink, nq, "paged_prefill_attention")), stream()), "paged_prefill_attn")
     _count()
     return out
 
 
-def ragged_prefill_attention(q, k, v, block_table, page, cu_q, kv_lens, max_q_len, scale, out):
-    """Causal attention of q [T, nq, 128] over keys and values that are rows of all heads: k, v [pages * page, nkv * 128]
+def ragged_prefill_attention(q, k, v, block_table, page, cu_q, kv_lens, max_q_len, scale, out, window=0, sink=None):
+    """Causal (windowed) attention of q [T, nq, 128] over keys and values that are rows of all heads: k, v [pages * page, nkv * 128]
     column blocks of one matrix, a sequence's pages named by its block-table row.  CUDA, bf16."""
     T, nq, d = q.shape
     R, width = k.shape
@@ -344,7 +354,8 @@ def ragged_prefill_attention(q, k, v, block_table, page, cu_q, kv_lens, max_q_le
     check(_lib_().xllm_paged_prefill_attn_tc_kept(ptr(out), out.stride(0), ptr(q), q.stride(0), T, ptr(k), ptr(v), R // page,
                                                   k.stride(0), ptr(block_table), block_table.stride(0), ptr(cu_q),
                                                   ptr(kv_lens), kv_lens.shape[0], int(max_q_len), nq, width // 128, page, scale,
-                                                  1, 0, 0, 0.0, stream()), "ragged_prefill_attn_tc")
+                                                  1, int(window), 0, 0.0, ptr(_sink(sink, nq, "ragged_prefill_attention")), stream()),
+          "ragged_prefill_attn_tc")
     _count()
     return out
 

@@ -103,8 +103,8 @@ def _declare(lib):
         "xllm_paged_decode_attn": [P, P, L, P, P, P, I, P, I, I, I, I, I, F, I, P, P],
         "xllm_paged_decode_attn_window": [P, P, L, P, P, P, I, P, I, I, I, I, I, F, I, P, I, P],
         "xllm_paged_decode_attn_kept": [P, P, L, P, P, P, I, P, I, I, I, I, I, F, I, P, I, I, F, P],
-        "xllm_paged_prefill_attn_kept": [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, F, I, I, I, F, P],
-        "xllm_paged_prefill_attn_tc_kept": [P, L, P, L, L, P, P, L, L, P, I, P, P, I, I, I, I, I, F, I, I, I, F, P],
+        "xllm_paged_prefill_attn_kept": [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, F, I, I, I, F, P, P],
+        "xllm_paged_prefill_attn_tc_kept": [P, L, P, L, L, P, P, L, L, P, I, P, P, I, I, I, I, I, F, I, I, I, F, P, P],
         "xllm_attn_merge": [P, P, P, L, I, I, P],
         "xllm_paged_prefill_attn": [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, F, I, I, P],
         "xllm_paged_prefill_attn_tc": [P, L, P, L, L, P, P, L, P, I, P, P, I, I, I, I, I, F, I, I, P],
@@ -121,8 +121,8 @@ def _declare(lib):
         "xllm_resolve_placeholders": [P, P, L, L, P],
         "xllm_rope_norm_kv": [P, P, P, L, P, P, P, P, L, P, P, I, I, I, I, I, I, I, I, I, I, F] + [P] * 7 + [I] * 4 + [P],
         "xllm_proj_f32": [P, L, P, L, P, P, I, I, I, P],
-        "xllm_paged_attn_generic": [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, I, F, I, I, F, I, P],
-        "xllm_silu_mul_f32": [P, P, L, I, L, F, F, P],
+        "xllm_paged_attn_generic": [P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, I, F, I, I, F, P, I, P],
+        "xllm_act_mul_f32": [P, P, L, I, L, I, F, F, P],
     }
     for name, args in sig.items():
         lib.declare(name, args, I)

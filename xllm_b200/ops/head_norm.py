@@ -8,7 +8,7 @@ from . import _lib
 from ._lib import F, I, L, P, check, ptr, stream
 
 _lib.register_signature("xllm_head_norm_gate", [P, L, P, P, P, L, P, I, L, I, I, I, I, F, I, P])
-_lib.register_signature("xllm_head_gate", [P, P, P, L, L, I, I, I, I, P])
+_lib.register_signature("xllm_head_gate", [P, P, P, L, L, I, I, I, I, I, P])
 
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 _ACT = {"silu": 0, "sigmoid": 1}
@@ -41,13 +41,17 @@ def head_norm_gate(o, out, div=None, g=None, w=None, unit_norm=True, act="silu",
 
 
 def head_gate(a, g, dv):
-    """a [T, H, d_pad] (heads of dv, stored wider) -> [T, H * dv] times sigmoid(g [T, H * dv])."""
+    """a [T, H, d_pad] (heads of dv, stored wider) -> [T, H * dv] times sigmoid(g), g [T, H * dv] or one per head [T, H]."""
     T, H, dp = a.shape
+    per_head = g.shape[1] == H and dv > 1
     if not a.is_cuda:
+        if per_head:
+            return (a[..., :dv].float() * torch.sigmoid(g.float())[..., None]).to(a.dtype).reshape(T, H * dv)
         return (a[..., :dv].reshape(T, H * dv).float() * torch.sigmoid(g.float())).to(a.dtype)
     assert a.is_contiguous() and g.stride(1) == 1 and g.dtype == a.dtype
     out = torch.empty((T, H * dv), dtype=a.dtype, device=a.device)
-    check(_lib.load().xllm_head_gate(ptr(out), ptr(a), ptr(g), g.stride(0), T, H, dv, dp, _DT[a.dtype], stream()), "head_gate")
+    check(_lib.load().xllm_head_gate(ptr(out), ptr(a), ptr(g), g.stride(0), T, H, dv, dp, int(per_head), _DT[a.dtype], stream()),
+          "head_gate")
     from . import _count
     _count()
     return out

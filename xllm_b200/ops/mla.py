@@ -113,9 +113,10 @@ def decode(q_cat, cache, block_table, scale, seq_lens=None, positions=None, bt_r
 
 
 # ----------------------------------------------------------------------------- caches of latents alone
-_lib.register_signature("xllm_latent_decode", [P, P, L, P, I, P, I, P, P, P, I, I, I, F, I, P, P])
+_lib.register_signature("xllm_latent_decode", [P, P, L, P, I, P, I, P, P, P, I, I, I, F, I, P, I, P, P])
 _lib.register_signature("xllm_latent_norm", [P, P, P, I, I, P, P, P, I, I, P, L, I, F, I, P])
-_lib.register_signature("xllm_latent_gather", [P, P, P, I, P, I, I, I, I, P])
+_lib.register_signature("xllm_latent_gather", [P, P, P, I, P, P, P, I, I, I, I, I, P])
+_lib.register_signature("xllm_latent_rope_write", [P, I, I, I, P, P, I, I, I, L, P, L, P, P, P, I, P, I, I, F, I, P])
 
 LATENT_WIDTHS = (128, 256, 512)
 
@@ -123,9 +124,53 @@ LATENT_WIDTHS = (128, 256, 512)
 def latent_width(rank, dtype, device):
     """Row size a cache of latents of `rank` values should have: the widths of the tensor-core kernels in bf16 on the device
     (zero filled), the rank itself otherwise."""
+    return row_layout(rank, 0, dtype, device)[0]
+
+
+def row_layout(rank, rot, dtype, device):
+    """(row size, place of the rotated part, how many leading values of a row are value) of a cache of latents with `rot`
+    rotated key values beside each."""
     if dtype == torch.bfloat16 and torch.device(device).type == "cuda":
-        return next((w for w in LATENT_WIDTHS if rank <= w), (rank + 7) // 8 * 8)
-    return rank
+        for w in LATENT_WIDTHS:
+            if rank + rot <= w:
+                return w, rank, w
+        if rank <= LATENT and 0 < rot <= ROT:
+            return LATENT + ROT, LATENT, LATENT
+        w = (rank + rot + 7) // 8 * 8
+        return w, rank, w
+    return rank + rot, rank, rank + rot
+
+
+def rope_write(q, heads, d, c, c_w, rank, rot, rot_at, cos_sin, positions, slots, cache, eps, qa=None, qa_rows=0):
+    """Cache row of every token's slot = [rmsnorm(c[:, :rank]) * c_w | rotated c[:, rank:] at rot_at], zeros elsewhere; the part
+    [d, d + rot) of every head of q turns in place.  q [T, heads * head stride] and c [T, rank + rot]: column blocks of the same
+    rows; neighbouring elements are a pair.  qa [T, heads, width]: absorbed queries, whose first `qa_rows` rows get their columns
+    from `rank` on."""
+    T, hs, width = q.shape[0], q.shape[1] // heads, cache.shape[-1]
+    assert q.stride() == c.stride() and q.stride(1) == 1 and c.shape[1] == rank + rot and cache.is_contiguous()
+    if not q.is_cuda:
+        cs = cos_sin[positions.long()]
+        row = torch.zeros(T, width, dtype=cache.dtype)
+        x = c[:, :rank].float()
+        row[:, :rank] = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * c_w.float()
+        row[:, rot_at:rot_at + rot] = rope_pairs(c[:, rank:], cs)
+        ok = slots >= 0
+        cache.view(-1, width)[slots[ok].long()] = row[ok]
+        part = q.unflatten(1, (heads, hs))[:, :, d:d + rot]
+        part.copy_(rope_pairs(part, cs))
+        if qa is not None:
+            qa[:qa_rows, :, rank:] = 0
+            qa[:qa_rows, :, rot_at:rot_at + rot] = part[:qa_rows]
+        return
+    from . import _count, _index
+    assert q.dtype == c.dtype == cache.dtype == c_w.dtype and q.dtype in (torch.bfloat16, torch.float32) and cache.shape[1] == 1
+    assert cos_sin.dtype == torch.float32 and cos_sin.shape[1] == rot and cos_sin.is_contiguous()
+    assert qa is None or (qa.is_contiguous() and qa.dtype == q.dtype and qa.shape[1:] == (heads, width) and qa.shape[0] >= qa_rows)
+    check(_lib.load().xllm_latent_rope_write(
+        ptr(q), heads, hs, d, ptr(c), ptr(c_w), rank, rot, rot_at, q.stride(0), ptr(cos_sin), cos_sin.shape[0],
+        ptr(_index(positions, torch.int64, "rope_write positions")), ptr(_index(slots, torch.int32, "rope_write slots")), ptr(cache),
+        width, ptr(qa), int(qa_rows), T, float(eps), 0 if q.dtype == torch.bfloat16 else 1, stream()), "latent_rope_write")
+    _count()
 
 
 def latent_norm(q, q_w, q_pad, eps, c=None, c_w=None, slots=None, cache=None):
@@ -156,37 +201,47 @@ def latent_norm(q, q_w, q_pad, eps, c=None, c_w=None, slots=None, cache=None):
     return out
 
 
-def latent_decode(q, cache, block_table, scale, seq_lens=None, positions=None, bt_rows=None, splits=None, out=None):
-    """`decode` over a cache [n_blocks, 1, page, width] of latents alone: q, out [N, nh, width].  CUDA, bf16, width in
-    LATENT_WIDTHS."""
+def latent_decode(q, cache, block_table, scale, seq_lens=None, positions=None, bt_rows=None, splits=None, out=None, window=0,
+                  sink=None):
+    """`decode` over a cache [n_blocks, 1, page, width]: q [N, nh, width], out the same (512 wide over rows of 576).  CUDA, bf16,
+    width in LATENT_WIDTHS or 576.  window > 0: a row sees its last `window` tokens; sink [nh] fp32: exp(sink) joins the denominators."""
     N, nh, width = q.shape
+    dv = LATENT if width == LATENT + ROT else width
     assert q.dtype == cache.dtype == torch.bfloat16 and q.is_contiguous() and cache.is_contiguous() and cache.shape[-1] == width
     assert block_table.dtype == torch.int32 and block_table.stride(1) == 1
     if out is None:
-        out = torch.empty_like(q)
-    assert out.is_contiguous()
+        out = torch.empty((N, nh, dv), dtype=q.dtype, device=q.device)
+    assert out.is_contiguous() and out.shape == (N, nh, dv)
     if N == 0:
         return out
+    from . import _sink
     if splits is None:
         from . import decode_splits
         splits = decode_splits(N, 1, nh)
-    ws = torch.empty(N * nh * splits * (width + 1), dtype=torch.float32, device=q.device) if splits > 1 else None
+        if window:
+            splits = min(splits, max(1, window // 256))
+    ws = torch.empty(N * nh * splits * (dv + 1), dtype=torch.float32, device=q.device) if splits > 1 else None
     check(_lib.load().xllm_latent_decode(ptr(out), ptr(q), q.stride(0), ptr(cache), width, ptr(block_table),
                                          block_table.stride(0), ptr(seq_lens), ptr(positions), ptr(bt_rows), N, nh,
-                                         cache.shape[-2], float(scale), int(splits), ptr(ws), stream()), "latent_decode")
+                                         cache.shape[-2], float(scale), int(splits), ptr(ws), int(window), ptr(_sink(sink, nh, "latent_decode")),
+                                         stream()), "latent_decode")
     from . import _count
     _count(2 if splits > 1 else 1)
     return out
 
 
-def latent_gather(cache, block_table, kv_lens, rows_per):
-    """The cached latents of a few sequences as dense rows [n_seqs * rows_per, width], zeros behind each sequence."""
+def latent_gather(cache, block_table, kv_lens, rows_per, cu_q=None, window=0):
+    """The cached rows of a few sequences, dense [n_seqs * rows_per, width], zeros behind each sequence.  With a window (and cu_q
+    [n_seqs + 1], the rows of the batch) only what these rows see; returns (rows, their number per sequence)."""
     n, width = kv_lens.shape[0], cache.shape[-1]
     assert cache.dtype == torch.bfloat16 and cache.is_contiguous() and cache.shape[1] == 1
     assert block_table.dtype == kv_lens.dtype == torch.int32 and block_table.stride(1) == 1
+    assert not window or (cu_q.dtype == torch.int32 and cu_q.is_contiguous())
     out = torch.empty((n * rows_per, width), dtype=cache.dtype, device=cache.device)
-    check(_lib.load().xllm_latent_gather(ptr(out), ptr(cache), ptr(block_table), block_table.stride(0), ptr(kv_lens), n,
-                                         rows_per, cache.shape[-2], width, stream()), "latent_gather")
+    lens = torch.empty(n, dtype=torch.int32, device=cache.device) if window else None
+    check(_lib.load().xllm_latent_gather(ptr(out), ptr(cache), ptr(block_table), block_table.stride(0), ptr(kv_lens),
+                                         ptr(cu_q), ptr(lens), int(window), n, rows_per, cache.shape[-2], width, stream()),
+          "latent_gather")
     from . import _count
     _count()
-    return out
+    return (out, lens) if window else out

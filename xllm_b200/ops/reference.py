@@ -193,9 +193,10 @@ def _gather_kv(cache, block_table_row, kv_len):
     return x[:, :kv_len]  # [nkv, kv_len, d]
 
 
-def paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, causal=True, window=0, keep=0, softcap=0.0):
+def paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, causal=True, window=0, keep=0, softcap=0.0,
+                    sink=None):
     """q: [T, nq, d]; returns [T, nq, d]. Sequence b owns q rows cu_q[b]:cu_q[b+1].  With a window the first `keep`
-    positions stay visible; softcap > 0 bounds the scores."""
+    positions stay visible; softcap > 0 bounds the scores; exp(sink) [nq] joins the denominators."""
     out = torch.zeros_like(q)
     nq, nkv = q.shape[1], k_cache.shape[1]
     group = nq // nkv
@@ -219,7 +220,9 @@ def paged_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, caus
         if window and window > 0:
             mask |= (kpos <= qpos - window) & (kpos >= keep)
         s = s.masked_fill(mask[None], float("-inf"))
-        p = torch.softmax(s, dim=-1)
+        if sink is not None:
+            s = torch.cat([s, sink.float().view(nq, 1, 1).expand(nq, ql, 1)], dim=-1)
+        p = torch.softmax(s, dim=-1)[..., :kl]
         p = torch.nan_to_num(p, nan=0.0)
         o = torch.einsum("hqk,hkd->hqd", p, v)
         out[qs:qe] = o.transpose(0, 1).to(q.dtype)

@@ -10,6 +10,8 @@ from ._lib import F, I, L, P, check, ptr, stream
 _lib.register_signature("xllm_residual_update", [P, P, L, P, P, L, P, P, P, L, P, P, I, I, I, F, F, F, I, P])
 _lib.register_signature("xllm_gelu_mul_rows", [P, P, L, P, L, L, P, L, I, I, I, I, P])
 
+_lib.register_signature("xllm_postnorm_update", [P, P, L, P, P, P, L, I, I, F, F, I, P])
+
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 
 
@@ -50,6 +52,26 @@ def residual_update(x, y, w=None, y2=None, w2=None, coef=1.0, rows=None, w_out=N
     check(_lib.load().xllm_residual_update(
         ptr(x), ptr(y), y.stride(0), ptr(w), ptr(y2), y2.stride(0) if y2 is not None else 0, ptr(w2), ptr(w_sum), ptr(rows), y.shape[0],
         ptr(w_out), ptr(out), T, H, int(init), float(coef), float(eps), float(w_out_offset), _DT[y.dtype], stream()), "residual_update")
+    from . import _count
+    _count()
+    return x, out
+
+
+def postnorm_update(x, y, w, alpha=1.0, groups=1, w_out=None, eps=1e-6):
+    """x <- n(alpha * x + y) * w, n = RMS norm of `groups` equal consecutive parts on their own; returns (x, out) with
+    out = x cast to the branch type, or n(x) * w_out.  x is fp32 [T, H] and updated in place."""
+    T, H = y.shape
+    assert H % groups == 0
+    if not y.is_cuda:
+        def n(b, wt):
+            b = b.view(T, groups, H // groups)
+            return (b / torch.sqrt(b.pow(2).mean(-1, keepdim=True) + eps)).view(T, H) * wt.float()
+        x.copy_(n(alpha * x + y.float(), w))
+        return x, (x.clone() if w_out is None else n(x, w_out)).to(y.dtype)
+    assert x.dtype == torch.float32 and x.is_contiguous() and x.shape == (T, H) and y.stride(1) == 1
+    out = torch.empty((T, H), dtype=y.dtype, device=y.device)
+    check(_lib.load().xllm_postnorm_update(ptr(x), ptr(y), y.stride(0), ptr(w), ptr(w_out), ptr(out), T, H, int(groups), float(alpha),
+                                           float(eps), _DT[y.dtype], stream()), "postnorm_update")
     from . import _count
     _count()
     return x, out

@@ -1,0 +1,104 @@
+"""Attention whose heads' softmax weights are mixed before they meet the values ("talking heads" behind the softmax), and what lies
+between its projections and the cache: a short convolution, norms of whole rows, unit-norm values."""
+from __future__ import annotations
+
+import torch
+
+from . import _lib, reference
+from ._lib import F, I, L, P, check, ptr, stream
+
+_lib.register_signature("xllm_conv_row_norm_kv", [P, P, P, L, P, P, P, P] + [I] * 7 + [F] + [P] * 7 + [I] * 4 + [P])
+_lib.register_signature("xllm_talk_attn_generic", [P, P, P, P, P, P, L, P, I, P, P] + [I] * 9 + [F, F, I, P])
+
+_DT = {torch.bfloat16: 0, torch.float32: 1}
+
+WORKSPACE_BYTES = 256 << 20          # of a chunk of rows
+
+
+def conv_row_norm_kv_write(q, k, v, heads, kv_heads, d, slots, k_cache, v_cache, q_w, k_w, conv, eps=1e-6, long_portions=True):
+    """A causal convolution per channel, then an RMS norm of all of q and of all of k with weights [heads * d], [kv_heads * d], and
+    every value head over its own root mean square; k and v rows go to the paged caches, whose heads may be wider (zero filled).
+    q, k, v: column blocks of the same rows; conv as in ops.rope_norm_kv_write.  Returns q [T, heads, cache head size]."""
+    T, dp = q.shape[0], k_cache.shape[3]
+    dv = v.shape[1] // kv_heads
+    cw, ring, st, cu, kl = conv
+    if not q.is_cuda:
+        y = reference.conv_portions(torch.cat([q, k, v], dim=1), *conv)
+        q, k, v = y.split([q.shape[1], k.shape[1], v.shape[1]], dim=1)
+        norm = lambda x: x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+        pad = lambda x: torch.nn.functional.pad(x, (0, dp - x.shape[-1])).to(k_cache.dtype)
+        reference.write_kv_cache(pad((norm(k) * k_w.float()).view(T, kv_heads, d)), pad(norm(v.reshape(T, kv_heads, dv))), k_cache,
+                                 v_cache, slots)
+        return pad((norm(q) * q_w.float()).view(T, heads, d))
+    from . import _count, _index
+    assert q.stride(0) == k.stride(0) == v.stride(0) and q.stride(1) == k.stride(1) == v.stride(1) == 1
+    assert q.dtype == k_cache.dtype == cw.dtype == ring.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert cw.is_contiguous() and ring.is_contiguous() and ring.shape[1:] == cw.shape
+    assert cw.shape[1] == q.shape[1] + k.shape[1] + v.shape[1] and q_w.numel() == q.shape[1] and k_w.numel() == k.shape[1]
+    assert st.dtype == cu.dtype == kl.dtype == torch.int32 and cu.shape[0] > st.shape[0] and kl.shape[0] >= st.shape[0]
+    slots = _index(slots, torch.int32, "conv_row_norm_kv_write slots")
+    out = torch.empty((T, heads, dp), dtype=q.dtype, device=q.device)
+    check(_lib.load().xllm_conv_row_norm_kv(
+        ptr(q), ptr(k), ptr(v), q.stride(0), ptr(out), ptr(k_cache), ptr(v_cache), ptr(slots), T, heads, kv_heads, d, dv, dp,
+        k_cache.shape[2], float(eps), ptr(q_w), ptr(k_w), ptr(cw), ptr(ring), ptr(st), ptr(cu), ptr(kl), st.shape[0], cw.shape[0],
+        int(long_portions), _DT[q.dtype], stream()), "conv_row_norm_kv")
+    _count(2 if long_portions and cw.shape[0] > 1 else 1)
+    return out
+
+
+def reference_attention(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, softcap, talk, dv, out):
+    """Tensor operations of the same sums, sequence by sequence."""
+    nq, nkv, d = q.shape[1], k_cache.shape[1], q.shape[2]
+    for b in range(len(kv_lens)):
+        qs, qe, kl = int(cu_q[b]), int(cu_q[b + 1]), int(kv_lens[b])
+        if qe == qs or kl == 0:
+            continue
+        k = reference._gather_kv(k_cache, block_table[b], kl).float().repeat_interleave(nq // nkv, dim=0)
+        v = reference._gather_kv(v_cache, block_table[b], kl)[..., :dv].float().repeat_interleave(nq // nkv, dim=0)
+        s = torch.einsum("qhd,hkd->hqk", q[qs:qe].float(), k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
+        place = torch.arange(qe - qs)[:, None] + (kl - (qe - qs))
+        s = s.masked_fill(torch.arange(kl)[None] > place, float("-inf"))
+        w = torch.einsum("hg,gqk->hqk", talk.float(), torch.softmax(s, dim=-1))
+        out[qs:qe] = torch.einsum("hqk,hkd->qhd", w, v).to(out.dtype)
+    return out
+
+
+def head_size(d, dv, dtype, device):
+    """Head size of the paged cache for key heads of d and value heads of dv."""
+    n = max(d, dv)
+    return (n + 7) // 8 * 8 if dtype == torch.bfloat16 and torch.device(device).type == "cuda" else n
+
+
+def attention(q, k_cache, v_cache, meta, scale, softcap, talk, dv, out):
+    """Rows of q [T, heads, cache head size] of all sequences (meta: decode rows and prompt portions) -> out [T, heads, dv].  Every row
+    sees its whole past; softcap > 0: scores become softcap * tanh(score / softcap); the softmax weights are mixed by talk
+    [heads, heads], weight_h <- sum_g talk[h, g] weight_g, and head h applies its own to the values of its key/value head."""
+    n = meta.n_seqs
+    args = (meta.block_table[:n], meta.cu_q[:n + 1], meta.kv_lens[:n], scale, softcap, talk, dv, out)
+    if not q.is_cuda:
+        return reference_attention(q, k_cache, v_cache, *args)
+    longest = meta.max_kv_len if meta.max_kv_len > 0 and not meta.padded else meta.block_table.shape[1] * k_cache.shape[2]
+    return attention_generic(q, k_cache, v_cache, *args, longest)
+
+
+def attention_generic(q, k_cache, v_cache, block_table, cu_q, kv_lens, scale, softcap, talk, dv, out, max_kv_len, row0=0, rows=None):
+    """Any sizes, bf16 or fp32: three launches for a chunk of rows over a table of their weights."""
+    from . import _count, _index
+    T, nq, d = q.shape
+    rows = T - row0 if rows is None else rows
+    assert q.is_contiguous() and out.is_contiguous() and q.dtype == k_cache.dtype == out.dtype == talk.dtype and talk.is_contiguous()
+    assert block_table.dtype == torch.int32 and block_table.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous()
+    cu_q, kv_lens = _index(cu_q, torch.int32, "talking attention cu_q"), _index(kv_lens, torch.int32, "talking attention kv_lens")
+    ld = (max_kv_len + 63) // 64 * 64
+    per = max(1, min(rows, WORKSPACE_BYTES // (nq * ld * 4)))
+    w = torch.empty(per * nq * ld, dtype=torch.float32, device=q.device)
+    for r in range(row0, row0 + rows, per):
+        n = min(per, row0 + rows - r)
+        check(_lib.load().xllm_talk_attn_generic(
+            ptr(out), ptr(q), ptr(k_cache), ptr(v_cache), ptr(talk), ptr(w), ld, ptr(block_table), block_table.stride(0), ptr(cu_q),
+            ptr(kv_lens), kv_lens.shape[0], r, n, nq, k_cache.shape[1], d, dv, d, k_cache.shape[2], float(scale),
+            float(softcap or 0.0), _DT[q.dtype], stream()), "talk_attn_generic")
+        _count(3)
+    return out
