@@ -115,10 +115,9 @@ def talking_attention(q, k, v, scale, softcap, talk):
         s = (q[:, h] @ k[:, h // (H // G)].T) * scale
         p.append(softmax(softcap * torch.tanh(s / softcap), mask))
     out = q.new_zeros(T, H, v.shape[-1])
+    p = torch.stack(p)
     for h in range(H):
-        mixed = torch.zeros_like(p[0])
-        for g in range(H):
-            mixed = mixed + talk[h, g] * p[g]
+        mixed = (talk[h][:, None, None] * p).sum(0)
         out[:, h] = mixed @ v[:, h // (H // G)]
     return out
 

@@ -436,11 +436,12 @@ __global__ void __launch_bounds__(256) conv_keep_kernel(RopeNormParams<T> p) {
 
 // Norms over whole rows.  One CTA takes RUN token rows one after another; a thread owns NV vectors of eight channels of q | k | v,
 // keeps their last inputs in registers, and the sums of squares meet once per row: those of q and k through the
-// warps, those of the values as one number per vector, so that every head adds its own in a fixed order.
+// warps, those of the values as one number per vector, so that every head adds its own in a fixed order.  portions: a sequence may
+// have several rows.
 constexpr int kRowThreads = 512;
 
 template <int RUN, int NV>
-__global__ void __launch_bounds__(kRowThreads) conv_row_norm_kernel(RopeNormParams<bf16> p) {
+__global__ void __launch_bounds__(kRowThreads) conv_row_norm_kernel(RopeNormParams<bf16> p, int portions) {
   __shared__ ConvPlace place[RUN];
   __shared__ int64_t cache_row[RUN];
   __shared__ float sums[2][2][kRowThreads / 32];
@@ -473,7 +474,7 @@ __global__ void __launch_bounds__(kRowThreads) conv_row_norm_kernel(RopeNormPara
 #pragma unroll
     for (int b = 0; b < kMaxTaps; ++b) {
       if constexpr (HOLD) w[i][b] = weight(i, b);
-      if (b > 0) win[i][b] = RUN > 1 && b < p.taps ? fetch(i, first - b) : bf16x8{};
+      if (b > 0) win[i][b] = portions && b < p.taps ? fetch(i, first - b) : bf16x8{};
     }
   }
   if (threadIdx.x < RUN) {
@@ -730,7 +731,7 @@ XLLM_API int xllm_conv_row_norm_kv(const void* q, const void* k, const void* v, 
           a16(q) && a16(k) && a16(v) && a16(q_out) && a16(k_cache) && a16(v_cache) && a16(q_w) && a16(k_w) && a16(conv_w) && a16(ring)) {
         const bool runs = long_portions && tokens > 4 * 148;
         const dim3 grid(runs ? (tokens + kConvRun - 1) / kConvRun : tokens), block(kRowThreads);
-        const auto go = [&](auto many, auto one) { launch_pdl(runs ? many : one, grid, block, smem, s, p); };
+        const auto go = [&](auto many, auto one) { launch_pdl(runs ? many : one, grid, block, smem, s, p, long_portions); };
         if (vecs <= kRowThreads) go(conv_row_norm_kernel<kConvRun, 1>, conv_row_norm_kernel<1, 1>);
         else if (vecs <= 2 * kRowThreads) go(conv_row_norm_kernel<kConvRun, 2>, conv_row_norm_kernel<1, 2>);
         else go(conv_row_norm_kernel<kConvRun, 3>, conv_row_norm_kernel<1, 3>);
