@@ -6,7 +6,7 @@ BASELINE.json on N GPUs of one node.
     python bench.py --gpus 1 --steps 20 --warmup 5  # config 2, K steps of the steady state
     python bench.py --gpus 8 --config 3 --steps 20  # Qwen3-32B shape, chunked 2048-token prefill
     python bench.py --gpus 8 --config 4 --steps 20  # Qwen3-30B-A3B shape, EP + DP attention
-    python bench.py --design femirax                # a model design at a few sizes beside Qwen3-Next (benchmarks/design_bench.py; also sodedra, lukinex)
+    python bench.py --design femirax                # a model design at a few sizes beside Qwen3-Next (benchmarks/design_bench.py; also sodedra, lukinex, vivazen)
 
 Workload (config 2): Qwen3-8B-shaped bf16 decoder, random-init weights, 1024 requests of uniform
 random token ids, input 1024 / output 512 with ignore_eos, at most 256 requests in flight (a closed
@@ -497,7 +497,7 @@ def main():
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="xllm_b200", choices=["xllm_b200", "ours", "reference", "library"])
     ap.add_argument("--library-attention", default="", help="library arm: attention backend name handed to vLLM")
-    ap.add_argument("--design", default="", choices=["", "femirax", "sodedra", "lukinex"],
+    ap.add_argument("--design", default="", choices=["", "femirax", "sodedra", "lukinex", "vivazen"],
                     help="throughput of one model design at a few sizes, beside the closest model (benchmarks/design_bench.py)")
     ap.add_argument("--config", default="2", choices=sorted(CONFIGS), help="BASELINE.json config number")
     ap.add_argument("--model", default="")

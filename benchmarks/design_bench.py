@@ -6,6 +6,7 @@ weights, one GPU.
     python bench.py --design femirax [--steps K] [--warmup W]      # prints one JSON line
     python bench.py --design sodedra
     python bench.py --design lukinex
+    python bench.py --design vivazen
 
 Prefill: four prompts of 2048 tokens in one step.  Decode: 64 sequences of 512 prompt tokens, one token each per step.
 Both go through the engine (scheduler, state slots, cache, sampling) and are timed with CUDA events around K steps
@@ -76,6 +77,36 @@ def lukinex_args(W):
     return model_args_from_dict({"architecture": "Lukinex", "vocab": VOCAB, "width": W, "norm": {"eps": 1e-6}, "layers": layers})
 
 
+def vivazen_args(W):
+    """Mixed-head attention and rotated latent attention in turn; the second latent layer uses the first one's tensors."""
+    from xllm_b200.models import model_args_from_dict
+    H = W // 128
+    att = ("attention", {"heads": H, "kv_heads": max(1, H // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "conv": 4, "softcap": 30.0})
+    lat = ("latent_attention", {"heads": H, "dim": 64, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 128 ** -0.5,
+                                "mask": {"size": 1024}, "rot": {"base": 1e6, "dims": 64, "scaling": {
+                                    "factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}})
+    kinds = [att, lat]
+    layers = [{"type": kinds[i % 2][0], "mixer": dict(kinds[i % 2][1]), "mlp": {"kind": "dense", "ff": 3 * W}} for i in range(LAYERS)]
+    layers[3]["weights_of"] = 1
+    return model_args_from_dict({"architecture": "Vivazen", "vocab": VOCAB, "width": W, "norm": {"eps": 1e-6, "groups": 4},
+                                 "postln_alpha": 2.0, "layers": layers})
+
+
+def lukinex_dense_args(W):
+    """Convolved, capped attention and latent attention in turn, without the recurrent branches' share of the layers; one expert and a
+    shared one, together as wide as a dense feed-forward."""
+    a = lukinex_args(W)
+    H, layers = W // 128, []
+    moe = {"kind": "moe", "expert": {"ff": 3 * W // 2, "limit": 7.0}, "router": {"experts": 1, "top": 1},
+           "shared": {"ff": 3 * W // 2, "limit": 7.0}}
+    att = {**next(l["mixer"] for l in a.extra["layers"] if l["type"] == "attention")}
+    lat = {**next(l["mixer"] for l in a.extra["layers"] if l["type"] == "latent_attention"), "q_rank": W}
+    for i in range(LAYERS):
+        layers.append({"type": ("attention", "latent_attention")[i % 2], "mixer": dict((att, lat)[i % 2]), "mlp": moe})
+    from xllm_b200.models import model_args_from_dict
+    return model_args_from_dict({"architecture": "Lukinex", "vocab": VOCAB, "width": W, "norm": {"eps": 1e-6}, "layers": layers})
+
+
 def qwen3_next_args(W):
     from xllm_b200.models import ModelArgs
     H = W // 128
@@ -110,7 +141,8 @@ def qwen3_next_shared_args(W):
 # name -> (title, arguments of the design, {model beside it: its arguments})
 DESIGNS = {"femirax": ("Femirax", femirax_args, {"qwen3_next": qwen3_next_args}),
            "sodedra": ("Sodedra", sodedra_args, {"qwen3_next": qwen3_next_moe_args}),
-           "lukinex": ("Lukinex", lukinex_args, {"qwen3_next": qwen3_next_shared_args, "sodedra": sodedra_moe_args})}
+           "lukinex": ("Lukinex", lukinex_args, {"qwen3_next": qwen3_next_shared_args, "sodedra": sodedra_moe_args}),
+           "vivazen": ("Vivazen", vivazen_args, {"qwen3_next": qwen3_next_args, "lukinex": lukinex_dense_args})}
 
 
 def engine_of(args):

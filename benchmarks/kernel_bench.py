@@ -637,6 +637,126 @@ def latent_rows(results, hbm, tf, tag):
                 xb, lg, w1, w2, K, ws=ws, interleaved=True, act=act)), nb, 6.0 * T * K * W * I)
 
 
+def talking_rows(results, hbm, tf, tag):
+    """The kernels of Vivazen beside their likes: attention with mixed heads against soft-capped attention without the mixture,
+    windowed rotated latents with sinks against latents and MLA, convolution with row norms against convolution with rotation, the
+    norm behind the sum against the other residual updates.  32 heads of 128, 8 key/value heads, width 4096."""
+    from xllm_b200.models.layers import AttentionMetadata
+    from xllm_b200.ops import mla, talking
+    from xllm_b200.ops.head_norm import head_gate
+    from xllm_b200.ops.residual import postnorm_update, residual_update
+    dev, bf, d, W, nq, nkv, R, win = "cuda", torch.bfloat16, 128, 4096, 32, 8, 512, 1024
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    rows = lambda t, n: torch.randn(t, n, device=dev, dtype=bf)
+
+    def report(name, shape, t, nbytes, flops=0.0):
+        ideal = max(nbytes / (hbm * 1e9), flops / (tf * 1e12))
+        results.append(dict(kernel=name, shape=shape, ms=t * 1e3, gbs=nbytes / t / 1e9, tflops=flops / t / 1e12,
+                            frac_of_roofline=ideal / t, peaks=tag))
+        print(f"{name:<38} {shape:<26} {t*1e6:9.1f} us {nbytes/t/1e9:7.0f} GB/s {flops/t/1e12:7.1f} TF/s  {ideal/t:6.3f} of {tag}",
+              flush=True)
+
+    talk = torch.eye(nq, device=dev, dtype=bf) + rows(nq, nq) * 0.1
+    for S, L in ((4, 512), (4, 2048), (1, 8192)):
+        T = S * L
+        kc, vc = (rows(T // 16 * nkv * 16, d).view(T // 16, nkv, 16, d) for _ in range(2))
+        bt = torch.arange(T // 16, device=dev, dtype=torch.int32).view(S, L // 16)
+        cu, kl, q = i32([i * L for i in range(S + 1)]), i32([L] * S), rows(T, nq * d).view(T, nq, d)
+        out, pairs = torch.empty_like(q), S * L * (L + 1) / 2
+        nb = T * d * 2 * (2 * nq + 2 * nkv)
+        report("prompts, capped", f"{S} x {L}", bench_queued(lambda: ops.paged_prefill_attention(
+            q, kc, vc, bt, cu, kl, L, d ** -0.5, softcap=30.0, out=out), iters=5), nb, 4.0 * pairs * nq * d)
+        report("prompts, capped, heads mixed", f"{S} x {L}", bench_queued(lambda: talking.prefill(
+            q, kc, vc, bt, cu, kl, L, d ** -0.5, 30.0, talk, d, out, L, 0), iters=5), nb, pairs * nq * (4.0 * d + 2.0 * nq))
+        lib, s = ops._lib.load(), ops.stream()
+        lse = torch.empty(T, nq, device=dev)
+        report("  row sums", f"{S} x {L}", bench_queued(lambda: lib.xllm_prefill_lse_tc(
+            lse.data_ptr(), q.data_ptr(), q.stride(0), T, kc.data_ptr(), kc.shape[0], bt.data_ptr(), bt.stride(0), cu.data_ptr(),
+            kl.data_ptr(), S, L, nq, nkv, 16, d ** -0.5, 30.0, ops.stream()), iters=5), 0.0, 2.0 * pairs * nq * d)
+        n = min(T, max(128, talking.WORKSPACE_BYTES // (nq * L * 2) // 128 * 128))
+        w = torch.empty(nq * n * L, device=dev, dtype=bf)
+        r0 = T - n                                    # the last chunk of rows
+        seen = sum(r % L + 1 for r in range(r0, T))
+        for keys in (128, 512, 1024):
+            report(f"  mixed weights of {n} rows, {keys} keys", f"{S} x {L}", bench_queued(lambda: lib.xllm_talk_weights(
+                w.data_ptr(), n, L, q.data_ptr(), kc.data_ptr(), talk.data_ptr(), lse.data_ptr(), bt.data_ptr(), bt.stride(0), cu.data_ptr(),
+                kl.data_ptr(), S, L, r0, n, nq, nkv, 16, d ** -0.5, 30.0, keys, ops.stream()), iters=5), 2.0 * seen * nq,
+                seen * nq * (2.0 * d + 2.0 * nq))
+        report(f"  values of {n} rows", f"{S} x {L}", bench_queued(lambda: lib.xllm_talk_values_tc(
+            out.data_ptr(), d, w.data_ptr(), n, L, vc.data_ptr(), vc.shape[0], bt.data_ptr(), bt.stride(0), cu.data_ptr(), kl.data_ptr(), S, L,
+            r0, n, nq, nkv, 16, ops.stream()), iters=5), 2.0 * seen * nq, 2.0 * seen * nq * d)
+        del kc, vc, w
+    for B, ctx in ((16, 8192), (64, 2048), (64, 8192), (256, 2048)):
+        kc, vc = (rows(B * ctx // 16 * nkv * 16, d).view(B * ctx // 16, nkv, 16, d) for _ in range(2))
+        bt = torch.randperm(B * ctx // 16, device=dev).to(torch.int32).view(B, ctx // 16)
+        kl, q = i32([ctx] * B), rows(B, nq * d).view(B, nq, d)
+        out, nb = torch.empty_like(q), 4.0 * B * ctx * nkv * d
+        report("decode, capped", f"B={B} ctx {ctx}", bench_queued(lambda: ops.paged_decode_attention(
+            q, kc, vc, bt, kl, d ** -0.5, softcap=30.0, out=out)), nb)
+        report("decode, capped, heads mixed", f"B={B} ctx {ctx}", bench_queued(lambda: talking.decode(
+            q, kc, vc, bt, kl, d ** -0.5, 30.0, talk, d, out, ctx)), nb)
+        del kc, vc
+    sink = torch.zeros(nq, device=dev)
+    for B, ctx in ((16, 8192), (64, 4096), (256, 2048)):
+        bt = (torch.randperm(B * (ctx // 16), device=dev) + 1).view(B, -1).to(torch.int32)
+        sl, cache = i32([ctx] * B), rows((B * (ctx // 16) + 1) * 16, R + 64).view(-1, 1, 16, R + 64)
+        q, out = rows(B, nq * (R + 64)).view(B, nq, R + 64) * 0.3, torch.empty(B, nq, R, device=dev, dtype=bf)
+        for name, n, kw in (("latent decode, window, sinks", min(win, ctx), dict(window=win, sink=sink)), ("latent decode, sinks", ctx, dict(sink=sink)),
+                            ("mla decode", ctx, {})):
+            report(name, f"B={B} ctx {ctx}", bench_queued(lambda: mla.latent_decode(q, cache, bt, 0.09, seq_lens=sl, out=out, **kw)),
+                   2.0 * B * n * (R + 64), 2.0 * B * nq * n * (2 * R + 64))
+        del cache
+    for S, L in ((4, 512), (4, 2048), (1, 8192)):
+        T, bt = S * L, torch.arange(1, S * L // 16 + 1, device=dev, dtype=torch.int32).view(S, L // 16)
+        cu, kl, pages = i32([i * L for i in range(S + 1)]), i32([L] * S), torch.arange(T // 128, device=dev, dtype=torch.int32).view(S, -1)
+        cache, ukv, q = rows((T // 16 + 1) * 16, R + 64).view(-1, 1, 16, R + 64), rows(2 * nq * d, R + 64), rows(T, nq * d).view(T, nq, d)
+        out = torch.empty(T, nq, d, device=dev, dtype=bf)
+        for name, wn, kw in (("latent prompts, window, sinks", win, dict(window=win, sink=sink)), ("latent prompts", L, {})):
+            def expanded():
+                dense, n = mla.latent_gather(cache, bt, kl, L, cu, win) if kw else (mla.latent_gather(cache, bt, kl, L), kl)
+                kv = ops.linear(dense, ukv)
+                ops.ragged_prefill_attention(q, kv[:, :nq * d], kv[:, nq * d:], pages, 128, cu, n, L, 0.09, out, **kw)
+            pairs = S * sum(min(i + 1, wn) for i in range(L))
+            report(name, f"{S} x {L}", bench_queued(expanded, iters=5), 0.0, 4.0 * pairs * nq * d + 4.0 * T * (R + 64) * nq * d)
+        del cache
+    C = (nq + 2 * nkv) * d
+    for T in (64, 8192):
+        qkv, cs = rows(T, C), torch.randn(8192, d, device=dev)
+        kc = torch.zeros(T // 16 + 2, nkv, 16, d, device=dev, dtype=bf)
+        vc, sl = torch.zeros_like(kc), torch.arange(16, 16 + T, dtype=torch.int32, device=dev)
+        q, k, v = qkv[:, :nq * d], qkv[:, nq * d:(nq + nkv) * d], qkv[:, (nq + nkv) * d:]
+        n = T if T == 64 else 4                                       # decode rows, or four prompts
+        ring, cw, L = torch.zeros(n + 1, 4, C, device=dev, dtype=bf), rows(4, C), T // n
+        conv = (cw, ring, i32(list(range(n))), i32([i * L for i in range(n + 1)]), i32([L if n == 4 else 100] * n))
+        pos, nb, one = torch.arange(T, device=dev) % 2048, T * d * 4 * (nq + 2 * nkv), torch.ones(nq * d, device=dev, dtype=bf)
+        nb += T * C * 8 if T == 64 else 0
+        report("convolution + rotation + cache write", f"T={T}", bench_queued(lambda: ops.rope_norm_kv_write(
+            q, k, v, nq, nkv, d, pos, cs, d, sl, kc, vc, unit_norm=False, conv=conv, long_portions=n == 4)), nb)
+        report("convolution + row norms + cache write", f"T={T}", bench_queued(lambda: talking.conv_row_norm_kv_write(
+            q, k, v, nq, nkv, d, sl, kc, vc, one, one[:nkv * d], conv, long_portions=n == 4)), nb)
+        x, y, w = torch.randn(T, W, device=dev), rows(T, W), torch.ones(W, device=dev, dtype=bf)
+        report("residual, branch normed", f"T={T}", bench_queued(lambda: residual_update(x, y, w=w, w_out=w)), T * W * 12)
+        for g in (1, 4):
+            report(f"residual, sum normed, {g} parts", f"T={T}", bench_queued(lambda: postnorm_update(x, y, w, alpha=0.5, groups=g)), T * W * 12)
+        ld = nq * d + R + 64 + nq
+        lat, cache = rows(T, ld), torch.zeros(T // 16 + 2, 1, 16, R + 64, device=dev, dtype=bf)
+        cw2, qa = torch.ones(R, device=dev, dtype=bf), torch.empty(T, nq, R + 64, device=dev, dtype=bf)
+        ql, c, cos = lat[:, :nq * d], lat[:, nq * d:nq * d + R + 64], torch.randn(8192, 64, device=dev)
+        nqa = T if T == 64 else 0
+        report("latent rows + rotation", f"T={T}", bench_queued(lambda: mla.rope_write(
+            ql, nq, 64, c, cw2, R, 64, R, cos, pos, sl, cache, 1e-6, qa=qa if nqa else None, qa_rows=nqa)),
+            T * ((R + 64) * 4 + nq * 64 * 4) + nqa * nq * 64 * 2)
+        c8 = rows(T, 2048 + R)
+        report("latent norms + cache write", f"T={T}", bench_queued(lambda: mla.latent_norm(
+            c8[:, :2048], torch.ones(2048, device=dev, dtype=bf), 2048, 1e-6, c=c8[:, 2048:], c_w=cw2, slots=sl,
+            cache=cache.view(-1)[:(T // 16 + 2) * 16 * R].view(-1, 1, 16, R))), T * (2048 + R) * 4)
+        a = rows(T, nq * d).view(T, nq, d)
+        report("gate per head", f"T={T}", bench_queued(lambda: head_gate(a, lat[:, ld - nq:], d)), T * nq * d * 4)
+        gu = rows(T, 6 * W)
+        report("gelu gate", f"T={T}", bench_queued(lambda: gemm_tcgen05.act_and_mul_interleaved(gu, "gelu_tanh")), T * W * 18)
+        report("silu gate", f"T={T}", bench_queued(lambda: gemm_tcgen05.act_and_mul_interleaved(gu, "silu")), T * W * 18)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--what", default="gemm,decode,prefill,small")
@@ -647,7 +767,7 @@ def main():
     for w in a.what.split(","):
         {"gemm": gemm_rows, "decode": decode_rows, "prefill": prefill_rows, "small": small_rows, "gdn": gdn_rows, "mla": mla_rows,
          "fp8": fp8_rows, "moe": moe_rows, "hybrid": hybrid_rows, "recurrent": recurrent_rows,
-         "latent": latent_rows}[w](results, hbm, tf, tag)
+         "latent": latent_rows, "talking": talking_rows}[w](results, hbm, tf, tag)
     if a.json:
         with open(a.json, "w") as f:
             json.dump(results, f, indent=1)

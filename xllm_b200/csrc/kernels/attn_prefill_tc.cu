@@ -150,7 +150,8 @@ struct Params {
   float* lse;                  // optional [total_q, nq]: log2-domain log-sum-exp of every row's scaled scores
 };
 
-template <bool CAP>
+// LSE: nothing but the log-sum-exp of every row (no values, no output).
+template <bool CAP, bool LSE>
 __global__ void __launch_bounds__(320, 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                   const __grid_constant__ CUtensorMap tma_v, const Params p) {
@@ -242,6 +243,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
         tma_load_2d(kdst + off, &tma_k, x, y, k_full(st));
         tma_load_2d(kdst + kHalf + off, &tma_k, x + 64, y, k_full(st));
       }
+      if constexpr (LSE) continue;
       if (!mbar_wait_warp(v_empty(st), ((j >> 1) & 1) ^ 1, abort_flag)) { ok = false; break; }
       if (lane == 0) mbar_expect_tx(v_full(st), kTile);
       __syncwarp();
@@ -268,8 +270,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
           const uint32_t o = (ks >> 2) * kHalf + (ks & 3) * 32;
           umma(TS0 + (j & 1) * 128, smem_desc(sbase + Q_OFF + o, 16, 1024), smem_desc(kaddr + o, 16, 1024), ID_QK, ks != 0);
         }
+        if constexpr (LSE) umma_commit(k_empty(j & 1));   // the last commit of all is one that somebody waits for
         umma_commit(s_full(j & 1));
-        umma_commit(k_empty(j & 1));   // the K slot may be refilled once these MMAs have read it
+        if constexpr (!LSE) umma_commit(k_empty(j & 1));  // the K slot may be refilled once these MMAs have read it
       }
       __syncwarp();
     };
@@ -286,6 +289,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
         tc_fence_after();
         issue_qk(j + 1);
       }
+      if constexpr (LSE) continue;
       if (!mbar_wait_warp(v_full(j & 1), (j >> 1) & 1, abort_flag)) { ok = false; break; }
       if (!mbar_wait_warp(p_full, j & 1, abort_flag)) { ok = false; break; }   // also: O has been rescaled if need be
       tc_fence_after();
@@ -375,6 +379,13 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
         m = m_true;
       }
       const float m_use = m == -INFINITY ? 0.f : m;
+      if constexpr (LSE) {
+        float rs = 0.f;
+#pragma unroll
+        for (int i = 0; i < 64; ++i) rs += exp2f(__uint_as_float(sv[i]) * sc - m_use);
+        l = l * factor + rs;
+        continue;
+      }
       // P may be overwritten, and O touched, once the PV product of the previous tile has completed
       ok = ok && mbar_wait(p_free, (j & 1) ^ 1, abort_flag);
       if (j > 0 && __any_sync(0xffffffffu, factor != 1.f)) {
@@ -416,7 +427,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       l = l * factor + rs;
     }
     float o[64];
-    if (n_tiles > 0) {
+    if (!LSE && n_tiles > 0) {
       ok = ok && mbar_wait(o_full, 0, abort_flag);
       tc_fence_after();
 #pragma unroll
@@ -441,7 +452,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       p.lse[(int64_t)(q_begin + m0 + row) * p.nq + h] = l > 0.f ? m + log2f(l) : -INFINITY;
     uint8_t* stage = smem + Q_OFF;                    // [128 rows][256 bytes], 16-byte units XOR-swizzled by row
 #pragma unroll
-    for (int u = 0; u < 8; ++u) {
+    for (int u = 0; u < (LSE ? 0 : 8); ++u) {
       float f[8];
 #pragma unroll
       for (int e = 0; e < 8; ++e) f[e] = o[u * 8 + e] * inv;
@@ -449,7 +460,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       *reinterpret_cast<uint4*>(stage + row * 256 + (((half * 8 + u) ^ (row & 15)) << 4)) = *reinterpret_cast<const uint4*>(&v);
     }
     asm volatile("bar.sync 1, 256;" ::: "memory");
-    if (ok) {
+    if (!LSE && ok) {
       const int t = threadIdx.x - 64;                 // 0..255
       const int u = t & 15;
       for (int r0 = t >> 4; r0 < kBM; r0 += 16) {     // 16 rows per pass, 16 threads x 16 bytes per row
@@ -466,6 +477,144 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
   if (warp == 1) {
     tc_fence_after();
     asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512));
+  }
+}
+
+// Weights that another kernel left in memory times the values: one CTA = (sequence, query head, tile of 128 rows of a window of
+// batch rows), 192 threads: warp 0 loads tiles of weights and gathers the values' pages (TMA, three stages), warp 1 issues the
+// products into one TMEM accumulator, warps 2-5 store it.
+struct WvParams {
+  bf16* out;                   // [total_q, nq, dv]
+  const int32_t *block_table, *cu_q, *kv_lens;
+  int64_t w_rows;              // rows a head takes in the table of weights
+  int dv, bt_stride, nq, nkv, page, row0, rows;
+  int* err;
+};
+constexpr int kWvStages = 3;
+constexpr int WV_BAR = kWvStages * 2 * kTile;
+constexpr int WV_SMEM = WV_BAR + 64 + 16 + 1024;
+
+__global__ void __launch_bounds__(192, 1)
+weights_values_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_constant__ CUtensorMap tma_v, const WvParams p) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+  const uint32_t sbase = smem_u32(smem), bar0 = sbase + WV_BAR;
+  auto full = [&](int s) { return bar0 + 8u * s; };
+  auto empty = [&](int s) { return bar0 + 8u * (kWvStages + s); };
+  const uint32_t o_full = bar0 + 8u * 2 * kWvStages;
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(smem + WV_BAR + 64);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_holder + 1);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int b = blockIdx.z, h = blockIdx.y, hk = h / (p.nq / p.nkv);
+  const int q_end = p.cu_q[b + 1], q_lo = max(p.cu_q[b], p.row0), q_hi = min(q_end, p.row0 + p.rows);
+  const int n_q_tiles = q_hi > q_lo ? (q_hi - q_lo + kBM - 1) / kBM : 0;
+  if ((int)blockIdx.x >= n_q_tiles) return;          // uniform for the whole CTA: nothing allocated yet
+  const int r0 = q_lo + (n_q_tiles - 1 - (int)blockIdx.x) * kBM;   // heavy (late) tiles first
+  const int kv_len = p.kv_lens[b];
+  const int kv_hi = min(kv_len, kv_len - (q_end - r0) + kBM);
+  const int n_tiles = max(0, (kv_hi + kBN - 1) / kBN);
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < kWvStages; ++s) {
+      mbar_init(full(s), 1);
+      mbar_init(empty(s), 1);
+    }
+    mbar_init(o_full, 1);
+    *abort_flag = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (warp == 1) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_holder)), "r"(128));
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::);
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_holder;
+  if (warp == 0) {
+    const int pages = kBN / p.page, n_blk = (kv_len + p.page - 1) / p.page;
+    const int32_t* bt = p.block_table + (int64_t)b * p.bt_stride;
+    const int wy = (int)(h * p.w_rows) + r0 - p.row0;
+    bool ok = true;
+    for (int j = 0; j < n_tiles && ok; ++j) {
+      const int st = j % kWvStages, pg = j * pages + lane;
+      const int y = ((lane < pages && pg < n_blk ? bt[pg] : 0) * p.nkv + hk) * p.page;   // past the sequence: block 0, weights 0
+      const uint32_t wdst = sbase + st * 2 * kTile, vdst = wdst + kTile, off = (uint32_t)(lane * p.page * 128);
+      if (!mbar_wait_warp(empty(st), ((j / kWvStages) & 1) ^ 1, abort_flag)) { ok = false; break; }
+      if (lane == 0) {
+        mbar_expect_tx(full(st), 2 * kTile);
+        tma_load_2d(wdst, &tma_w, j * kBN, wy, full(st));
+        tma_load_2d(wdst + kHalf, &tma_w, j * kBN + 64, wy, full(st));
+      }
+      __syncwarp();
+      if (lane < pages) {
+        tma_load_2d(vdst + off, &tma_v, 0, y, full(st));
+        tma_load_2d(vdst + kHalf + off, &tma_v, 64, y, full(st));
+      }
+      __syncwarp();
+    }
+    if (!ok) {
+      const long long t0 = clock64();
+      while (clock64() - t0 < 20000000LL) {}          // bounded grace period for copies in flight
+    }
+  } else if (warp == 1) {
+    constexpr uint32_t ID_PV = idesc(true);
+    for (int j = 0; j < n_tiles; ++j) {
+      const int st = j % kWvStages;
+      if (!mbar_wait_warp(full(st), (j / kWvStages) & 1, abort_flag)) break;
+      tc_fence_after();
+      if (lane == 0) {
+        const uint32_t wa = sbase + st * 2 * kTile, va = wa + kTile;
+#pragma unroll
+        for (int ks = 0; ks < 8; ++ks)
+          umma(tmem, smem_desc(wa + (ks >> 2) * kHalf + (ks & 3) * 32, 16, 1024), smem_desc(va + ks * 16 * 128, kHalf, 1024), ID_PV,
+               (j | ks) != 0);
+        umma_commit(empty(st));
+        if (j == n_tiles - 1) umma_commit(o_full);
+      }
+      __syncwarp();
+    }
+  } else {
+    const int quarter = warp & 3, row = quarter * 32 + lane;
+    bool ok = true;
+    if (n_tiles > 0) {
+      ok = mbar_wait_warp(o_full, 0, abort_flag);
+      tc_fence_after();
+    }
+    bf16* dst = p.out + ((int64_t)(r0 + row) * p.nq + h) * p.dv;
+    const bool live = ok && r0 + row < q_hi, vec = p.dv % 8 == 0;
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      uint32_t r[32];
+      if (n_tiles > 0) {
+        tmem_ld32(tmem + ((uint32_t)(quarter * 32) << 16) + c * 32, r);
+        tmem_ld_wait();
+      } else {
+#pragma unroll
+        for (int i = 0; i < 32; ++i) r[i] = 0;
+      }
+      if (!live) continue;
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int e = c * 32 + u * 8;
+        float f[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(r[u * 8 + i]);
+        if (vec) {
+          if (e < p.dv) *reinterpret_cast<bf16x8*>(dst + e) = pack8(f);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+            if (e + i < p.dv) dst[e + i] = __float2bfloat16(f[i]);
+        }
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (threadIdx.x == 0 && *abort_flag && p.err != nullptr) atomicExch(p.err, 1);
+  if (warp == 1) {
+    tc_fence_after();
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(128));
   }
 }
 
@@ -519,9 +668,10 @@ static int prefill_tc(void* out, int64_t o_stride, const void* q, int64_t q_stri
   cudaGetDevice(&dev);
   static bool attr_done[64] = {};
   if (!attr_done[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
-    if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
+    cudaError_t e = cudaSuccess;
+    for (const auto kernel : {prefill_tc_kernel<false, false>, prefill_tc_kernel<true, false>, prefill_tc_kernel<false, true>,
+                              prefill_tc_kernel<true, true>})
+      if (e == cudaSuccess) e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
     if (e != cudaSuccess) return (int)e;
     attr_done[dev & 63] = true;
   }
@@ -541,8 +691,9 @@ static int prefill_tc(void* out, int64_t o_stride, const void* q, int64_t q_stri
   p.page = page_size; p.causal = causal; p.window = window; p.scale_log2 = scale * 1.4426950408889634f; p.err = g_err[dev & 63];
   p.lse = (float*)lse; p.sink = (const float*)sink; p.keep = window > 0 ? keep : 0; p.rows_kv = kv_ld > 0; p.cap = make_soft_cap(scale, softcap);
   dim3 grid((max_q_len + kBM - 1) / kBM, nq, batch);
-  if (softcap > 0.f) prefill_tc_kernel<true><<<grid, 320, SMEM_TOTAL, (cudaStream_t)stream>>>(tq, tk, tv, p);
-  else prefill_tc_kernel<false><<<grid, 320, SMEM_TOTAL, (cudaStream_t)stream>>>(tq, tk, tv, p);
+  const auto kernel = out == nullptr ? (softcap > 0.f ? prefill_tc_kernel<true, true> : prefill_tc_kernel<false, true>)
+                                     : (softcap > 0.f ? prefill_tc_kernel<true, false> : prefill_tc_kernel<false, false>);
+  kernel<<<grid, 320, SMEM_TOTAL, (cudaStream_t)stream>>>(tq, tk, tv, p);
   return XLLM_LAUNCH_CHECK();
 }
 
@@ -574,6 +725,49 @@ XLLM_API int xllm_paged_prefill_attn_tc(void* out, int64_t o_stride, const void*
   return xllm_paged_prefill_attn_tc_lse(out, o_stride, q, q_stride, total_q, k_cache, v_cache, n_blocks, block_table,
                                         bt_stride, cu_q, kv_lens, batch, max_q_len, nq, nkv, page_size, scale, causal,
                                         window, nullptr, stream);
+}
+
+// lse [total_q, nq] fp32: the log-sum-exp (log2 domain) of every row's scores over all it may see, and nothing else.
+XLLM_API int xllm_prefill_lse_tc(void* lse, const void* q, int64_t q_stride, int64_t total_q, const void* k_cache, int64_t n_blocks,
+                                 const void* block_table, int bt_stride, const void* cu_q, const void* kv_lens, int batch,
+                                 int max_q_len, int nq, int nkv, int page_size, float scale, float softcap, void* stream) {
+  if (lse == nullptr) return (int)cudaErrorInvalidValue;
+  return prefill_tc(nullptr, 0, q, q_stride, total_q, k_cache, k_cache, n_blocks, 0, block_table, bt_stride, cu_q, kv_lens, batch,
+                    max_q_len, nq, nkv, page_size, scale, 1, 0, 0, softcap, nullptr, lse, stream);
+}
+
+// Rows [row0, row0 + rows) of out [total_q, nq, dv] = tables of weights times the values of each head's key/value head:
+// w [nq, w_rows, ld] bf16, row r - row0 of head h; a row's weights are defined (zero beyond what it sees) up to the last key that
+// its tile of 128 rows sees, rounded up to 128.  v_cache [n_blocks, nkv, page, 128]; ld a multiple of 128.
+XLLM_API int xllm_talk_values_tc(void* out, int dv, const void* w, int64_t w_rows, int64_t ld, const void* v_cache, int64_t n_blocks,
+                                 const void* block_table, int bt_stride, const void* cu_q, const void* kv_lens, int batch,
+                                 int max_q_len, int row0, int rows, int nq, int nkv, int page_size, void* stream) {
+  using namespace xllm;
+  using namespace xllm::fmha;
+  if (batch == 0 || rows == 0 || max_q_len == 0) return 0;
+  if (nq % nkv != 0 || (page_size != 16 && page_size != 32 && page_size != 64 && page_size != 128) || ld <= 0 || ld % 128 || dv <= 0 ||
+      dv > kD || w_rows < rows || (((uintptr_t)w | (uintptr_t)v_cache) & 15))
+    return (int)cudaErrorInvalidValue;
+  int dev = 0;
+  cudaGetDevice(&dev);
+  static bool attr_done[64] = {};
+  if (!attr_done[dev & 63]) {
+    const cudaError_t e = cudaFuncSetAttribute(weights_values_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, WV_SMEM);
+    if (e != cudaSuccess) return (int)e;
+    attr_done[dev & 63] = true;
+  }
+  if (g_err[dev & 63] == nullptr) {
+    if (cudaMalloc(&g_err[dev & 63], sizeof(int)) != cudaSuccess) return (int)cudaErrorMemoryAllocation;
+    cudaMemset(g_err[dev & 63], 0, sizeof(int));
+  }
+  CUtensorMap tw, tv;
+  if (!make_map(&tw, w, (int64_t)nq * w_rows, ld, ld, kBM) || !make_map(&tv, v_cache, n_blocks * nkv * page_size, kD, kD, page_size))
+    return (int)cudaErrorInvalidValue;
+  WvParams p{(bf16*)out, (const int32_t*)block_table, (const int32_t*)cu_q, (const int32_t*)kv_lens, w_rows, dv, bt_stride, nq, nkv,
+             page_size, row0, rows, g_err[dev & 63]};
+  const dim3 grid((min(max_q_len, rows) + kBM - 1) / kBM, nq, batch);
+  weights_values_kernel<<<grid, 192, WV_SMEM, (cudaStream_t)stream>>>(tw, tv, p);
+  return XLLM_LAUNCH_CHECK();
 }
 
 // 0 = no bounded wait expired in the prefill kernel on this device since the last call.

@@ -83,8 +83,8 @@ class VivazenCausalLM(Module):
     supports_graph = True
     supports_prefill_graph = True
     # the kernel sources a process that runs nothing but this model needs
-    kernel_sources = ("gemm_tcgen05", "activation", "attn_decode", "attn_prefill", "attn_prefill_tc", "attn_generic", "head_norm", "mla",
-                      "residual", "rope_norm_kv", "misc", "sampling")
+    kernel_sources = ("gemm_tcgen05", "activation", "attn_decode", "attn_prefill", "attn_prefill_tc", "attn_generic", "attn_talk", "head_norm",
+                      "mla", "residual", "rope_norm_kv", "misc", "sampling")
     fused_tp = False
 
     def __init__(self, args, dtype=torch.bfloat16, device="cpu", ps=None):
