@@ -679,7 +679,7 @@ def talking_rows(results, hbm, tf, tag):
         seen = sum(r % L + 1 for r in range(r0, T))
         for keys in (128, 512, 1024):
             report(f"  mixed weights of {n} rows, {keys} keys", f"{S} x {L}", bench_queued(lambda: lib.xllm_talk_weights(
-                w.data_ptr(), n, L, q.data_ptr(), kc.data_ptr(), talk.data_ptr(), lse.data_ptr(), bt.data_ptr(), bt.stride(0), cu.data_ptr(),
+                w.data_ptr(), n, L, q.data_ptr(), T, kc.data_ptr(), kc.shape[0], talk.data_ptr(), lse.data_ptr(), bt.data_ptr(), bt.stride(0), cu.data_ptr(),
                 kl.data_ptr(), S, L, r0, n, nq, nkv, 16, d ** -0.5, 30.0, keys, ops.stream()), iters=5), 2.0 * seen * nq,
                 seen * nq * (2.0 * d + 2.0 * nq))
         report(f"  values of {n} rows", f"{S} x {L}", bench_queued(lambda: lib.xllm_talk_values_tc(

@@ -20,17 +20,18 @@
 // Every mbarrier wait is bounded; on expiry all roles leave, TMEM is released and an error word
 // is set (xllm_fmha_error_status).
 #include "attn_common.cuh"
-#include <cuda.h>
+#include "tc_common.cuh"
 
 namespace xllm {
 namespace fmha {
+
+using namespace tc;
 
 constexpr int kD = 128;
 constexpr int kBM = 128;  // query rows per CTA
 constexpr int kBN = 128;  // kv tokens per tile
 constexpr int kHalf = kBM * 128;          // bytes of one [128 rows x 64 elements] swizzled half tile
 constexpr int kTile = 2 * kHalf;          // 32 KB: a [128 x 128] bf16 operand tile
-constexpr long long kWaitBudget = 4000000000LL;
 
 constexpr int Q_OFF = 0;
 constexpr int KV_OFF = kTile;                       // 2 stages x (K, V)
@@ -38,100 +39,7 @@ constexpr int P_OFF = KV_OFF + 4 * kTile;
 constexpr int BAR_OFF = P_OFF + kTile;
 constexpr int XCH_OFF = BAR_OFF + 24 * 8 + 16;          // row-max / row-sum exchange between the two halves of a row
 constexpr int SMEM_TOTAL = XCH_OFF + (2 * 2 + 2) * kBM * 4 + 1024;
-
-__device__ __forceinline__ void mbar_init(uint32_t bar, uint32_t count) {
-  asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count));
-}
-__device__ __forceinline__ void mbar_expect_tx(uint32_t bar, uint32_t bytes) {
-  asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void mbar_arrive(uint32_t bar) {
-  asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
-}
-__device__ __forceinline__ bool mbar_try(uint32_t bar, uint32_t parity) {
-  uint32_t ok;
-  asm volatile(
-      "{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\tselp.u32 %0, 1, 0, p;\n\t}"
-      : "=r"(ok)
-      : "r"(bar), "r"(parity)
-      : "memory");
-  return ok != 0;
-}
-__device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, volatile int* abort_flag) {
-  if (mbar_try(bar, parity)) return true;
-  const long long t0 = clock64();
-  int spins = 0;
-  while (true) {
-    if (mbar_try(bar, parity)) return true;
-    if ((++spins & 63) == 0) {
-      if (*abort_flag) return false;
-      if (clock64() - t0 > kWaitBudget) {
-        *abort_flag = 1;
-        return false;
-      }
-    }
-  }
-}
-__device__ __forceinline__ bool mbar_wait_warp(uint32_t bar, uint32_t parity, volatile int* abort_flag) {
-  return __all_sync(0xffffffffu, mbar_wait(bar, parity, abort_flag));
-}
-__device__ __forceinline__ void tma_load_2d(uint32_t smem_dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
-  asm volatile(
-      "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"
-      ::"r"(smem_dst), "l"(map), "r"(bar), "r"(x), "r"(y)
-      : "memory");
-}
-// shared-memory operand descriptor, 128-byte swizzle; lbo / sbo in bytes
-__device__ __forceinline__ uint64_t smem_desc(uint32_t addr, uint32_t lbo, uint32_t sbo) {
-  uint64_t d = 0;
-  d |= (uint64_t)((addr & 0x3FFFFu) >> 4);
-  d |= (uint64_t)(lbo >> 4) << 16;
-  d |= (uint64_t)(sbo >> 4) << 32;
-  d |= (uint64_t)1 << 46;
-  d |= (uint64_t)2 << 61;
-  return d;
-}
-// D = f32, A = B = bf16, M = 128, N = 128; b_mn: B is MN-major (bit 16)
-__host__ __device__ constexpr uint32_t idesc(bool b_mn) {
-  return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn ? (1u << 16) : 0u) | ((uint32_t)(128 >> 3) << 17) |
-         ((uint32_t)(128 >> 4) << 24);
-}
-__device__ __forceinline__ void umma(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t id, uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-      ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(id), "r"(accumulate)
-      : "memory");
-}
-__device__ __forceinline__ void umma_commit(uint32_t bar) {
-  asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t* r) {
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-      "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
-      "%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),
-        "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]),
-        "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]),
-        "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-      : "r"(taddr));
-}
-__device__ __forceinline__ void tmem_ld_wait() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
-__device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t* r) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, "
-      "%17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31, %32};"
-      ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]),
-        "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]),
-        "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]), "r"(r[24]), "r"(r[25]), "r"(r[26]),
-        "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
-      : "memory");
-}
-__device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+constexpr int LSE_CUT = 3 * kTile;                  // what a CTA without values and weights does not need: two of them fit an SM
 
 struct Params {
   bf16* out;
@@ -152,13 +60,14 @@ struct Params {
 
 // LSE: nothing but the log-sum-exp of every row (no values, no output).
 template <bool CAP, bool LSE>
-__global__ void __launch_bounds__(320, 1)
+__global__ void __launch_bounds__(320, LSE ? 2 : 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                   const __grid_constant__ CUtensorMap tma_v, const Params p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   const uint32_t sbase = smem_u32(smem);
-  const uint32_t bar0 = sbase + BAR_OFF;
+  constexpr int CUT = LSE ? LSE_CUT : 0, KV_STAGE = LSE ? kTile : 2 * kTile, TMEM_COLS = LSE ? 256 : 512;
+  const uint32_t bar0 = sbase + BAR_OFF - CUT;
   // barrier slots
   // K and V have rings of their own: a K slot is free again as soon as the QK product that read it
   // has completed, a V slot after its PV product, so the load of K_{j+2} starts a whole tile earlier
@@ -172,7 +81,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
   auto s_free = [&](int b) { return bar0 + 8u * (11 + b); };
   const uint32_t p_full = bar0 + 8u * 13, p_free = bar0 + 8u * 14;
   const uint32_t o_full = bar0 + 8u * 15;             // the last PV product has completed
-  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(smem + BAR_OFF + 24 * 8);
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(smem + BAR_OFF - CUT + 24 * 8);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_holder + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -207,7 +116,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
   if (warp == 1) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_holder)), "r"(512));
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_holder)), "r"(TMEM_COLS));
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::);
   }
   tc_fence_before();
@@ -234,7 +143,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       const int y = p.rows_kv ? myblk * p.page : (myblk * p.nkv + hk) * p.page;
       const int x = p.rows_kv ? hk * kD : 0;
       const uint32_t off = (uint32_t)(lane * p.page * 128);
-      const uint32_t kdst = sbase + KV_OFF + st * 2 * kTile, vdst = kdst + kTile;
+      const uint32_t kdst = sbase + KV_OFF + st * KV_STAGE, vdst = kdst + kTile;
       // every lane gathers its own page: the copies of all pages issue together
       if (!mbar_wait_warp(k_empty(st), ((j >> 1) & 1) ^ 1, abort_flag)) { ok = false; break; }
       if (lane == 0) mbar_expect_tx(k_full(st), kTile);
@@ -259,11 +168,11 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issuer
-    constexpr uint32_t ID_QK = idesc(false), ID_PV = idesc(true);
+    constexpr uint32_t ID_QK = idesc(false, 128), ID_PV = idesc(true, 128);
     bool ok = mbar_wait_warp(q_full, 0, abort_flag);
     auto issue_qk = [&](int j) {
       // S[j & 1] = Q K_j^T : 8 steps of 16 along head_dim, two 64-element halves
-      const uint32_t kaddr = sbase + KV_OFF + (j & 1) * 2 * kTile;
+      const uint32_t kaddr = sbase + KV_OFF + (j & 1) * KV_STAGE;
       if (lane == 0) {
 #pragma unroll
         for (int ks = 0; ks < 8; ++ks) {
@@ -320,7 +229,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
     const int q_pos = ctx_off + m0 + row;             // absolute position of this query token
     const int limit = p.causal ? min(kv_len - 1, q_pos) : kv_len - 1;   // last kv index this row may see
     const int low = p.window > 0 ? q_pos - p.window + 1 : 0;            // the first one
-    float* smax = reinterpret_cast<float*>(smem + XCH_OFF);             // [2 tile parities][2 halves][128 rows]
+    float* smax = reinterpret_cast<float*>(smem + XCH_OFF - CUT);             // [2 tile parities][2 halves][128 rows]
     float* lsum = smax + 2 * 2 * kBM;                                   // [2 halves][128 rows]
     // O stays in TMEM and the MMAs accumulate into it over all kv tiles.  The exponent uses a row
     // maximum m that lags the true one: it moves (and O and l are rescaled) only when the true
@@ -352,8 +261,16 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       __syncwarp();
       if (lane == 0) mbar_arrive(s_free(sb));         // S has been read out: the next QK may overwrite it
       if constexpr (CAP) {
+        float top = 0.f;
 #pragma unroll
-        for (int i = 0; i < 64; ++i) sv[i] = __float_as_uint(soft_cap(__uint_as_float(sv[i]), p.cap));
+        for (int i = 0; i < 64; ++i) top = fmaxf(top, fabsf(__uint_as_float(sv[i])));
+        if (__all_sync(0xffffffffu, top <= p.cap.small)) {
+#pragma unroll
+          for (int i = 0; i < 64; ++i) sv[i] = __float_as_uint(soft_cap_small(__uint_as_float(sv[i]), p.cap));
+        } else {
+#pragma unroll
+          for (int i = 0; i < 64; ++i) sv[i] = __float_as_uint(soft_cap(__uint_as_float(sv[i]), p.cap));
+        }
       }
       if (!full_tile) {                               // bit i: column i is seen
         const auto below = [&](int t) {               // columns of positions before t
@@ -365,6 +282,16 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
 #pragma unroll
         for (int i = 0; i < 64; ++i)
           if (!((i < 32 ? s0 : s1) & (1u << (i & 31)))) sv[i] = 0xff800000u;      // -inf
+      }
+      if constexpr (LSE && CAP) {
+        if (p.cap.out <= 100.f) {                     // sums of 2^score stay within fp32 without a reference
+          m = 0.f;
+          float rs = 0.f;
+#pragma unroll
+          for (int i = 0; i < 64; ++i) rs += exp2f(__uint_as_float(sv[i]));
+          l += rs;
+          continue;
+        }
       }
       float mx = -INFINITY;
 #pragma unroll
@@ -476,13 +403,13 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
   if (threadIdx.x == 0 && *abort_flag && p.err != nullptr) atomicExch(p.err, 1);
   if (warp == 1) {
     tc_fence_after();
-    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512));
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(TMEM_COLS));
   }
 }
 
 // Weights that another kernel left in memory times the values: one CTA = (sequence, query head, tile of 128 rows of a window of
-// batch rows), 192 threads: warp 0 loads tiles of weights and gathers the values' pages (TMA, three stages), warp 1 issues the
-// products into one TMEM accumulator, warps 2-5 store it.
+// batch rows), 192 threads, two CTAs an SM: warp 0 loads 64 keys of weights and gathers the values' pages (TMA, three stages), warp
+// 1 issues the products into one TMEM accumulator, warps 2-5 store it.
 struct WvParams {
   bf16* out;                   // [total_q, nq, dv]
   const int32_t *block_table, *cu_q, *kv_lens;
@@ -490,11 +417,12 @@ struct WvParams {
   int dv, bt_stride, nq, nkv, page, row0, rows;
   int* err;
 };
-constexpr int kWvStages = 3;
-constexpr int WV_BAR = kWvStages * 2 * kTile;
+constexpr int kWvStages = 3, kWvKeys = 64;
+constexpr int kWvW = kBM * kWvKeys * 2, kWvV = kWvKeys * kD * 2;     // bytes of a stage's weights and values
+constexpr int WV_BAR = kWvStages * (kWvW + kWvV);
 constexpr int WV_SMEM = WV_BAR + 64 + 16 + 1024;
 
-__global__ void __launch_bounds__(192, 1)
+__global__ void __launch_bounds__(192, 2)
 weights_values_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_constant__ CUtensorMap tma_v, const WvParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -512,7 +440,7 @@ weights_values_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_co
   const int r0 = q_lo + (n_q_tiles - 1 - (int)blockIdx.x) * kBM;   // heavy (late) tiles first
   const int kv_len = p.kv_lens[b];
   const int kv_hi = min(kv_len, kv_len - (q_end - r0) + kBM);
-  const int n_tiles = max(0, (kv_hi + kBN - 1) / kBN);
+  const int n_tiles = max(0, (kv_hi + kWvKeys - 1) / kWvKeys);
   if (threadIdx.x == 0) {
     for (int s = 0; s < kWvStages; ++s) {
       mbar_init(full(s), 1);
@@ -531,24 +459,24 @@ weights_values_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_co
   tc_fence_after();
   const uint32_t tmem = *tmem_holder;
   if (warp == 0) {
-    const int pages = kBN / p.page, n_blk = (kv_len + p.page - 1) / p.page;
+    const int per = min(p.page, kWvKeys), copies = kWvKeys / per;      // tokens of a copy
     const int32_t* bt = p.block_table + (int64_t)b * p.bt_stride;
     const int wy = (int)(h * p.w_rows) + r0 - p.row0;
     bool ok = true;
     for (int j = 0; j < n_tiles && ok; ++j) {
-      const int st = j % kWvStages, pg = j * pages + lane;
-      const int y = ((lane < pages && pg < n_blk ? bt[pg] : 0) * p.nkv + hk) * p.page;   // past the sequence: block 0, weights 0
-      const uint32_t wdst = sbase + st * 2 * kTile, vdst = wdst + kTile, off = (uint32_t)(lane * p.page * 128);
+      const int st = j % kWvStages, tok = j * kWvKeys + lane * per;
+      const int blk = lane < copies && tok < kv_len ? bt[tok / p.page] : 0;            // past the sequence: block 0, weights 0
+      const int y = (blk * p.nkv + hk) * p.page + tok % p.page;
+      const uint32_t wdst = sbase + st * (kWvW + kWvV), vdst = wdst + kWvW, off = (uint32_t)(lane * per * 128);
       if (!mbar_wait_warp(empty(st), ((j / kWvStages) & 1) ^ 1, abort_flag)) { ok = false; break; }
       if (lane == 0) {
-        mbar_expect_tx(full(st), 2 * kTile);
-        tma_load_2d(wdst, &tma_w, j * kBN, wy, full(st));
-        tma_load_2d(wdst + kHalf, &tma_w, j * kBN + 64, wy, full(st));
+        mbar_expect_tx(full(st), kWvW + kWvV);
+        tma_load_2d(wdst, &tma_w, j * kWvKeys, wy, full(st));
       }
       __syncwarp();
-      if (lane < pages) {
+      if (lane < copies) {
         tma_load_2d(vdst + off, &tma_v, 0, y, full(st));
-        tma_load_2d(vdst + kHalf + off, &tma_v, 64, y, full(st));
+        tma_load_2d(vdst + kWvV / 2 + off, &tma_v, 64, y, full(st));
       }
       __syncwarp();
     }
@@ -557,17 +485,16 @@ weights_values_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_co
       while (clock64() - t0 < 20000000LL) {}          // bounded grace period for copies in flight
     }
   } else if (warp == 1) {
-    constexpr uint32_t ID_PV = idesc(true);
+    constexpr uint32_t ID_PV = idesc(true, 128);
     for (int j = 0; j < n_tiles; ++j) {
       const int st = j % kWvStages;
       if (!mbar_wait_warp(full(st), (j / kWvStages) & 1, abort_flag)) break;
       tc_fence_after();
       if (lane == 0) {
-        const uint32_t wa = sbase + st * 2 * kTile, va = wa + kTile;
+        const uint32_t wa = sbase + st * (kWvW + kWvV), va = wa + kWvW;
 #pragma unroll
-        for (int ks = 0; ks < 8; ++ks)
-          umma(tmem, smem_desc(wa + (ks >> 2) * kHalf + (ks & 3) * 32, 16, 1024), smem_desc(va + ks * 16 * 128, kHalf, 1024), ID_PV,
-               (j | ks) != 0);
+        for (int ks = 0; ks < kWvKeys / 16; ++ks)
+          umma(tmem, smem_desc(wa + ks * 32, 16, 1024), smem_desc(va + ks * 16 * 128, kWvV / 2, 1024), ID_PV, (j | ks) != 0);
         umma_commit(empty(st));
         if (j == n_tiles - 1) umma_commit(o_full);
       }
@@ -618,32 +545,6 @@ weights_values_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_co
   }
 }
 
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-static EncodeTiledFn encode_fn() {
-  static EncodeTiledFn fn = nullptr;
-  if (fn == nullptr) {
-    void* ptr = nullptr;
-    cudaDriverEntryPointQueryResult q;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &q) == cudaSuccess &&
-        q == cudaDriverEntryPointSuccess)
-      fn = reinterpret_cast<EncodeTiledFn>(ptr);
-  }
-  return fn;
-}
-// bf16 [rows, cols] with row stride ld elements; box = [box_rows, 64 cols], 128-byte swizzle
-static bool make_map(CUtensorMap* map, const void* ptr, int64_t rows, int64_t cols, int64_t ld, int box_rows) {
-  EncodeTiledFn fn = encode_fn();
-  if (fn == nullptr) return false;
-  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-  cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
-  cuuint32_t box[2] = {64, (cuuint32_t)box_rows};
-  cuuint32_t estr[2] = {1, 1};
-  return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims, strides, box, estr,
-            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
 static int* g_err[64] = {};
 
 }  // namespace fmha
@@ -693,7 +594,7 @@ static int prefill_tc(void* out, int64_t o_stride, const void* q, int64_t q_stri
   dim3 grid((max_q_len + kBM - 1) / kBM, nq, batch);
   const auto kernel = out == nullptr ? (softcap > 0.f ? prefill_tc_kernel<true, true> : prefill_tc_kernel<false, true>)
                                      : (softcap > 0.f ? prefill_tc_kernel<true, false> : prefill_tc_kernel<false, false>);
-  kernel<<<grid, 320, SMEM_TOTAL, (cudaStream_t)stream>>>(tq, tk, tv, p);
+  kernel<<<grid, 320, out == nullptr ? SMEM_TOTAL - LSE_CUT : SMEM_TOTAL, (cudaStream_t)stream>>>(tq, tk, tv, p);
   return XLLM_LAUNCH_CHECK();
 }
 
@@ -761,7 +662,7 @@ XLLM_API int xllm_talk_values_tc(void* out, int dv, const void* w, int64_t w_row
     cudaMemset(g_err[dev & 63], 0, sizeof(int));
   }
   CUtensorMap tw, tv;
-  if (!make_map(&tw, w, (int64_t)nq * w_rows, ld, ld, kBM) || !make_map(&tv, v_cache, n_blocks * nkv * page_size, kD, kD, page_size))
+  if (!make_map(&tw, w, (int64_t)nq * w_rows, ld, ld, kBM) || !make_map(&tv, v_cache, n_blocks * nkv * page_size, kD, kD, min(page_size, kWvKeys)))
     return (int)cudaErrorInvalidValue;
   WvParams p{(bf16*)out, (const int32_t*)block_table, (const int32_t*)cu_q, (const int32_t*)kv_lens, w_rows, dv, bt_stride, nq, nkv,
              page_size, row0, rows, g_err[dev & 63]};

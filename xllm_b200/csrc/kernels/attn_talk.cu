@@ -16,13 +16,15 @@
 //   talk_weights_kernel     mixed weights of 16 rows and a range of keys to the table
 // and its product with the values (xllm_talk_values_tc).
 //
-// The mixture of 16 rows: a warp owns up to four heads of one key/value head, whose queries stay in registers, and makes the
-// transposed scores [16 keys x 8 rows] of each (mma.sync m16n8k16, keys as M), so that it has the weights of four heads for its
-// pairs and stores them as one 16-byte chunk of a pair's line: four leading terms, four remainders.  The lines of all units are the
-// B operand of the mixture (pairs as N, chunks as K), T repeated for leading terms and remainders the A operand, and what comes
-// out is four neighbouring keys per thread.  A step's mixture is computed beside the next step's scores.
+// The mixture of 16 rows, 128 keys at a time.  tcgen05 products leave transposed scores in tensor memory: a lane per key, and per unit
+// (up to four heads of one key/value head) row by row its heads.  So a thread has the weights of a unit for a pair at once and stores
+// them as one 16-byte chunk of the pair's line: four leading terms, four remainders.  The lines of a row are the B operand of its
+// mixture (mma.sync m16n8k16, pairs as N, chunks as K), T repeated for leading terms and remainders the A operand, and what comes out
+// is four neighbouring keys per thread.  A row's mixture is computed beside the next row's exponentials.  Every mbarrier wait is
+// bounded; on expiry all roles leave, tensor memory is released and an error word is set (xllm_talk_error_status).
 #include "attn_common.cuh"
-#include <atomic>
+#include "tc_common.cuh"
+#include <type_traits>
 
 namespace xllm {
 namespace talk {
@@ -342,183 +344,335 @@ struct WeightsParams {
   bf16* w;                    // [nq, w_rows, ld]
   const int32_t *block_table, *cu_q, *kv_lens;
   int64_t w_rows, ld;
-  int bt_stride, nq, nkv, group, page, row0, rows, keys;   // keys: of a block, a multiple of 16
+  int bt_stride, nq, nkv, group, page_log2, row0, rows, keys;   // keys: of a block, a multiple of 16
   SoftCap cap;
   float scale_log2;
+  int* err;
 };
+static int* g_err[64] = {};
 
-constexpr int kUnits = 8, kBM = 16, kKStages = 3, kPairLine = 128;
-constexpr int kPairBytes = kBM * 16 * kPairLine;      // pairs of one step
+constexpr int kUnits = 8, kBM = 16, kBN = 128;        // rows of a CTA, keys of a tile
+constexpr int kUnitCols = 4 * kBM;                    // scores of a key: row by row four heads
+constexpr int kQUnit = kUnitCols * D * 2;             // bytes of a unit's queries
+constexpr int kKTile = kBN * D * 2, kHalf = kKTile / 2;
+constexpr int kLine = 128, kLines = kBN * kLine;      // weights of a pair, of a row's pairs in one tile
+constexpr int kWorkers = 16, kThreads = (kWorkers + 2) * 32;
+constexpr int kNlOff = kUnits * kQUnit + 2 * kKTile + 2 * kLines, kBarOff = kNlOff + kBM * kUnits * 4 * 4;
+constexpr int kWeightsSmem = kBarOff + (1 + 4 + 2 * kUnits) * 8 + 16;     // no slack: the block's limit is near
 
+// The line of a pair keeps chunk c at c ^ spread(key): eight neighbouring keys (stores) and the eight keys of half an operand (loads)
+// meet eight different places.
 __device__ __forceinline__ int spread(int key) { return (key & 1) | ((key >> 1) & 2) | (((key >> 1 ^ key >> 3) & 1) << 2); }
 
-// grid (tiles of 16 rows, ranges of keys, sequences), 8 warps.  HB: tiles of 16 heads; KS: tiles of 16 columns of T (two units each).
-template <int HB, int KS>
-__global__ void __launch_bounds__(256, 1) talk_weights_kernel(WeightsParams p) {
-  extern __shared__ __align__(128) uint8_t smem[];
+// Pairs of fp32 values in one instruction.
+__device__ __forceinline__ uint64_t pack2(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void unpack2f(uint64_t v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
+// Two weights from their scores; CAP: 0 none, 1 the polynomial, 2 any score.
+template <int CAP>
+__device__ __forceinline__ void weigh(const uint32_t* x, uint64_t nl, const uint64_t (&k)[4], const SoftCap& cap, float& f0, float& f1) {
+  const float x0 = __uint_as_float(x[0]), x1 = __uint_as_float(x[1]);
+  if constexpr (CAP == 2) {
+    unpack2f(add2(pack2(soft_cap(x0, cap), soft_cap(x1, cap)), nl), f0, f1);
+  } else {
+    const uint64_t v = pack2(x0, x1);
+    if constexpr (CAP == 1) {
+      const uint64_t v2 = mul2(v, v);
+      unpack2f(fma2(v, fma2(v2, fma2(v2, fma2(v2, k[3], k[2]), k[1]), k[0]), nl), f0, f1);
+    } else {
+      unpack2f(fma2(v, k[0], nl), f0, f1);
+    }
+  }
+  f0 = exp2f(f0);
+  f1 = exp2f(f1);
+}
+
+// The chunk of one unit's four heads: leading terms cut off, remainders rounded.
+template <int CAP>
+__device__ __forceinline__ void chunk_out(uint32_t at, const uint32_t* x, uint32_t nl_at, const uint64_t (&k)[4], const SoftCap& cap,
+                                          bool hidden) {
+  uint64_t nl[2];
+  asm volatile("ld.shared.v2.b64 {%0, %1}, [%2];" : "=l"(nl[0]), "=l"(nl[1]) : "r"(nl_at));
+  uint32_t hi[2], lo[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    float f0, f1, r0, r1;
+    weigh<CAP>(x + 2 * i, nl[i], k, cap, f0, f1);
+    if (hidden) f0 = f1 = 0.f;
+    const uint32_t u0 = __float_as_uint(f0), u1 = __float_as_uint(f1);
+    asm("prmt.b32 %0, %1, %2, 0x7632;" : "=r"(hi[i]) : "r"(u0), "r"(u1));
+    unpack2f(fma2(pack2(__uint_as_float(u0 & 0xffff0000u), __uint_as_float(u1 & 0xffff0000u)), pack2(-1.f, -1.f), pack2(f0, f1)), r0, r1);
+    lo[i] = pack_bf162(r0, r1);
+  }
+  asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(at), "r"(hi[0]), "r"(hi[1]), "r"(lo[0]), "r"(lo[1]) : "memory");
+}
+
+// grid (tiles of 16 rows, ranges of keys, sequences).  Warps 0-15: worker w has keys 32 (w % 4) .. + 31 of a tile for units 2 (w / 4)
+// and the next, and mixes keys 16 (w % 8) .. + 15 for heads 16 (w / 8) .. + 15; warp 16 loads, warp 17 issues the products.  KS: tiles
+// of 16 columns of T (two units each).
+template <int KS>
+__global__ void __launch_bounds__(kThreads, 1)
+talk_weights_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k, const __grid_constant__ WeightsParams p) {
+  using namespace tc;
+  extern __shared__ __align__(1024) uint8_t smem[];
+  const auto nl = reinterpret_cast<float(*)[kUnits * 4]>(smem + kNlOff);  // minus the log-sum-exps; -inf: no such pair
+  uint32_t* tmem_holder = reinterpret_cast<uint32_t*>(smem + kBarOff + (1 + 4 + 2 * kUnits) * 8);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int b = blockIdx.z;
-  pdl_wait();
-  pdl_launch_dependents();
   const int q_end = p.cu_q[b + 1], q_lo = max(p.cu_q[b], p.row0), q_hi = min(q_end, p.row0 + p.rows);
   const int tiles = q_hi > q_lo ? (q_hi - q_lo + kBM - 1) / kBM : 0;
-  if ((int)blockIdx.x >= tiles) return;
+  if ((int)blockIdx.x >= tiles) return;               // uniform for the whole CTA: nothing allocated yet
   const int tile = tiles - 1 - blockIdx.x, r0 = q_lo + tile * kBM;                 // late tiles first
   const int kv_len = p.kv_lens[b], pos0 = kv_len - (q_end - r0);                   // position of row r0
   const int k0 = blockIdx.y * p.keys;
-  // the product with the values takes tiles of 128 rows and of 128 keys: what their last row sees is defined for all of them
+  // the product with the values takes tiles of 128 rows: what their last row sees, rounded up, is defined for all of them
   const int big = q_lo + tile * kBM / 128 * 128;
   const int defined = (max(0, min(kv_len, kv_len - (q_end - big) + 128)) + 127) / 128 * 128;
   if (k0 >= defined) return;
   const int k_end = min(k0 + p.keys, defined);
   const int seen = min(kv_len, pos0 + min(kBM, q_hi - r0));                        // keys that some row of the tile sees
-  const int steps = max(0, (min(k_end, seen) - k0 + 15) >> 4);
+  const int n = max(0, (min(k_end, seen) - k0 + kBN - 1) / kBN);                   // key tiles
   const int subs = (p.group + 3) >> 2, units = p.nkv * subs;
-  const bool mine = warp < units;
-  const int kvh = mine ? warp / subs : 0, head0 = kvh * p.group + (mine ? (warp - kvh * subs) * 4 : 0);
-  const int heads = mine ? min(4, kvh * p.group + p.group - head0) : 0;
-  const uint32_t kring = smem_u32(smem);
-  const int kbytes = p.nkv * kTileBytes;
-  uint8_t* pair = smem + kKStages * kbytes;
-  const uint32_t pair_u32 = smem_u32(pair);
-  const int32_t* bt = p.block_table + (int64_t)b * p.bt_stride;
-
-  const auto load = [&](int s) {                      // keys of step s of all kv heads
-    if (s < steps) {
-      const int tok0 = k0 + s * 16, pg = tok0 / p.page;
-      const bf16* kb = p.k_cache + ((int64_t)bt[pg] * p.nkv * p.page + tok0 - pg * p.page) * D;
-      const uint32_t dst = kring + (s % kKStages) * kbytes;
-      for (int id = threadIdx.x; id < p.nkv * 16 * CH; id += 256) {
-        const int c = id % CH, r = id / CH % 16, g = id / (16 * CH);
-        const bool in = tok0 + r < kv_len;
-        cp_async16(dst + g * kTileBytes + swz<CH>(r, c), kb + (in ? ((int64_t)g * p.page + r) * D + c * 8 : 0), in);
-      }
-    }
-    cp_async_commit();
-  };
-#pragma unroll
-  for (int s = 0; s < kKStages - 1; ++s) load(s);
-  if (units < 2 * KS)                                 // a chunk without a unit meets zeros of T and must be finite
-    for (int i = threadIdx.x; i < 2 * kPairBytes / 16; i += 256) reinterpret_cast<uint4*>(pair)[i] = make_uint4(0, 0, 0, 0);
-
-  // queries: B operand, columns are rows 0..7 and 8..15 of the tile
-  uint32_t qf[4][2][16];
-  float nl[4][2][2];                                  // minus the log-sum-exp of (head, row); -inf: no such pair
-#pragma unroll
-  for (int u = 0; u < 4; ++u)
-#pragma unroll
-    for (int n = 0; n < 2; ++n) {
-      const int row = r0 + n * 8 + (lane >> 2);
-      const bool in = u < heads && row < q_hi;
-      const bf16* src = p.q + ((int64_t)row * p.nq + head0 + u) * D + (lane & 3) * 2;
-#pragma unroll
-      for (int ks = 0; ks < 16; ++ks) qf[u][n][ks] = in ? *reinterpret_cast<const uint32_t*>(src + ks * 8) : 0u;
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int r = r0 + n * 8 + (lane & 3) * 2 + e;
-        nl[u][n][e] = u < heads && r < q_hi ? -p.lse[(int64_t)r * p.nq + head0 + u] : -INFINITY;
-      }
-    }
-  // T: A operand, columns: unit by unit four leading terms, four remainders
-  uint32_t ta[HB][KS][4];
-#pragma unroll
-  for (int hb = 0; hb < HB; ++hb)
-#pragma unroll
-    for (int ks = 0; ks < KS; ++ks)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int h = hb * 16 + (lane >> 2) + (i & 1) * 8, u = (lane & 1) * 2, un = ks * 2 + (i >> 1);
-        const int c = un / subs, first = (un - c * subs) * 4;
-        const bf16 zero = __float2bfloat16(0.f);
-        const auto at = [&](int e) {
-          return h < p.nq && un < units && first + u + e < p.group ? p.talk[h * p.nq + c * p.group + first + u + e] : zero;
-        };
-        const bf162 v = __halves2bfloat162(at(0), at(1));
-        ta[hb][ks][i] = *reinterpret_cast<const uint32_t*>(&v);
-      }
-
-  const auto scores = [&](int s) {
-    const uint32_t ka = kring + (s % kKStages) * kbytes + kvh * kTileBytes;
-    float x[4][2][4];
-#pragma unroll
-    for (int u = 0; u < 4; ++u)
-#pragma unroll
-      for (int n = 0; n < 2; ++n) x[u][n][0] = x[u][n][1] = x[u][n][2] = x[u][n][3] = 0.f;
-#pragma unroll
-    for (int ks = 0; ks < 8; ++ks) {
-      uint32_t a[4];
-      ldmatrix_x4(a[0], a[1], a[2], a[3], ka + swz<CH>(lane & 15, ks * 2 + (lane >> 4)));
-#pragma unroll
-      for (int u = 0; u < 4; ++u)
-#pragma unroll
-        for (int n = 0; n < 2; ++n) mma_bf16_16816(x[u][n], a, qf[u][n][ks * 2], qf[u][n][ks * 2 + 1]);
-    }
-    const int key0 = k0 + s * 16;
-    const bool edge = key0 + 15 > pos0;               // some row does not see all of these keys
-    const uint32_t dst = pair_u32 + (s & 1) * kPairBytes;
-#pragma unroll
-    for (int n = 0; n < 2; ++n)
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int key = (lane >> 2) + (j >> 1) * 8, r = n * 8 + (lane & 3) * 2 + (j & 1);
-        float f[4];
-#pragma unroll
-        for (int u = 0; u < 4; ++u) f[u] = exp2f(score(x[u][n][j], p.cap, p.scale_log2) + nl[u][n][j & 1]);
-        if (edge && key0 + key > pos0 + r) f[0] = f[1] = f[2] = f[3] = 0.f;
-        uint32_t hi[2], lo[2];
-        split_pack(f[0], f[1], hi[0], lo[0]);
-        split_pack(f[2], f[3], hi[1], lo[1]);
-        const uint32_t at = dst + (r * 16 + key) * kPairLine + ((warp ^ spread(key)) << 4);
-        asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(at), "r"(hi[0]), "r"(hi[1]), "r"(lo[0]), "r"(lo[1]) : "memory");
-      }
-  };
-  const auto mix = [&](int s) {
-    const uint32_t src = pair_u32 + (s & 1) * kPairBytes;
-    const int n = lane & 7, mi = lane >> 3, key = 4 * (n >> 1) + (n & 1) + (mi >> 1) * 2;     // this lane's line
-#pragma unroll
-    for (int i = 0; i < kBM / 8; ++i) {
-      const int r = warp + 8 * i;
-      float d[HB][2][4];
-#pragma unroll
-      for (int hb = 0; hb < HB; ++hb)
-#pragma unroll
-        for (int t = 0; t < 2; ++t) d[hb][t][0] = d[hb][t][1] = d[hb][t][2] = d[hb][t][3] = 0.f;
-#pragma unroll
-      for (int ks = 0; ks < KS; ++ks) {
-        uint32_t b0, b1, b2, b3;
-        ldmatrix_x4(b0, b1, b2, b3, src + (r * 16 + key) * kPairLine + (((ks * 2 + (mi & 1)) ^ spread(key)) << 4));
-#pragma unroll
-        for (int hb = 0; hb < HB; ++hb) {
-          mma_bf16_16816(d[hb][0], ta[hb][ks], b0, b1);
-          mma_bf16_16816(d[hb][1], ta[hb][ks], b2, b3);
-        }
-      }
-      if (r0 + r >= q_hi) continue;
-      bf16* dst = p.w + (int64_t)(r0 + r - p.row0) * p.ld + k0 + s * 16 + 4 * (lane & 3);
-#pragma unroll
-      for (int hb = 0; hb < HB; ++hb)
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int h = hb * 16 + (lane >> 2) + half * 8;
-          if (h < p.nq)
-            *reinterpret_cast<uint2*>(dst + (int64_t)h * p.w_rows * p.ld) =
-                make_uint2(pack_bf162(d[hb][0][half * 2], d[hb][0][half * 2 + 1]), pack_bf162(d[hb][1][half * 2], d[hb][1][half * 2 + 1]));
-        }
-    }
-  };
-  for (int s = 0; s < steps; ++s) {
-    cp_async_wait<kKStages - 2>();
-    __syncthreads();                                  // keys of step s are here; step s - 1's weights are; step s - 2's mixture is done
-    load(s + kKStages - 1);
-    if (mine) scores(s);
-    if (s > 0) mix(s - 1);
+  const auto head_of = [&](int unit) { return unit / subs * p.group + unit % subs * 4; };
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_holder + 1);
+  const uint32_t sbase = smem_u32(smem);
+  if (sbase & 1023) {                                 // swizzled tiles need the alignment asked for above
+    if (threadIdx.x == 0 && p.err != nullptr) atomicExch(p.err, 2);
+    return;
   }
-  cp_async_wait<0>();
-  __syncthreads();
-  if (steps > 0) mix(steps - 1);
+  const uint32_t qsm = sbase, ksm = qsm + kUnits * kQUnit, lines = ksm + 2 * kKTile;
+  const uint32_t bar0 = sbase + kBarOff, q_full = bar0;
+  const auto k_full = [&](int s) { return bar0 + 8u * (1 + s); };
+  const auto k_empty = [&](int s) { return bar0 + 8u * (3 + s); };
+  const auto s_full = [&](int u) { return bar0 + 8u * (5 + u); };
+  const auto s_free = [&](int u) { return bar0 + 8u * (5 + kUnits + u); };
+
+  if (n > 0) {
+    if (threadIdx.x == 0) {
+      mbar_init(q_full, 1);
+      for (int s = 0; s < 2; ++s) {
+        mbar_init(k_full(s), 1);
+        mbar_init(k_empty(s), 1);
+      }
+      for (int u = 0; u < kUnits; ++u) {
+        mbar_init(s_full(u), 1);
+        mbar_init(s_free(u), 4);
+      }
+      *abort_flag = 0;
+      asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == kWorkers + 1) {
+      asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_holder)), "r"(512));
+      asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::);
+    }
+    for (int i = threadIdx.x; i < kBM * kUnits * 4; i += kThreads) {
+      const int r = i / (kUnits * 4), c = i % (kUnits * 4), unit = c >> 2, u = c & 3;
+      const bool in = unit < units && unit % subs * 4 + u < p.group && r0 + r < q_hi;
+      nl[r][c] = in ? -p.lse[(int64_t)(r0 + r) * p.nq + head_of(unit) + u] : -INFINITY;
+    }
+    for (int i = threadIdx.x; i < 2 * kLines / 16; i += kThreads)      // chunks without a unit meet zeros of T and must be finite
+      asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(lines + i * 16), "r"(0) : "memory");
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = *tmem_holder;
+
+    if (warp == kWorkers) {
+      // ---------------------------------------------------------------- loads
+      if (lane == 0) {
+        mbar_expect_tx(q_full, units * kQUnit);
+        for (int u = 0; u < units; ++u)
+          for (int h = 0; h < 2; ++h) tma_load_3d(qsm + u * kQUnit + h * (kQUnit / 2), &tma_q, h * 64, head_of(u), r0, q_full);
+      }
+      __syncwarp();
+      const int page = 1 << p.page_log2, pages = kBN >> p.page_log2, n_blk = (kv_len + page - 1) >> p.page_log2;
+      const int32_t* bt = p.block_table + (int64_t)b * p.bt_stride;
+      bool ok = true;
+      for (int t = 0, i = 0; t < n && ok; ++t) {
+        const int pg = ((k0 + t * kBN) >> p.page_log2) + lane;
+        const int blk = lane < pages && pg < n_blk ? bt[pg] : 0;       // pages past the sequence read block 0 (hidden)
+        for (int c = 0; c < p.nkv; ++c, ++i) {
+          const int st = i & 1;
+          if (!mbar_wait_warp(k_empty(st), ((i >> 1) & 1) ^ 1, abort_flag)) { ok = false; break; }
+          if (lane == 0) mbar_expect_tx(k_full(st), kKTile);
+          __syncwarp();
+          if (lane < pages) {
+            const uint32_t dst = ksm + st * kKTile + lane * page * 128;
+            const int y = (blk * p.nkv + c) << p.page_log2;
+            tma_load_2d(dst, &tma_k, 0, y, k_full(st));
+            tma_load_2d(dst + kHalf, &tma_k, 64, y, k_full(st));
+          }
+          __syncwarp();
+        }
+      }
+      if (!ok) {
+        const long long t0 = clock64();
+        while (clock64() - t0 < 20000000LL) {}        // bounded grace period for copies in flight
+      }
+    } else if (warp == kWorkers + 1) {
+      // ---------------------------------------------------------------- products: [128 keys] x [16 rows x 4 heads] per unit
+      constexpr uint32_t ID = idesc(false, kUnitCols);
+      bool ok = mbar_wait_warp(q_full, 0, abort_flag);
+      for (int t = 0, i = 0; t < n && ok; ++t)
+        for (int c = 0; c < p.nkv && ok; ++c, ++i) {
+          const int st = i & 1;
+          ok = mbar_wait_warp(k_full(st), (i >> 1) & 1, abort_flag);
+          for (int j = 0; j < subs && ok; ++j) {
+            const int u = c * subs + j;
+            ok = mbar_wait_warp(s_free(u), (t & 1) ^ 1, abort_flag);
+            if (!ok) break;
+            tc_fence_after();
+            if (lane == 0) {
+              const uint32_t ka = ksm + st * kKTile, qa = qsm + u * kQUnit;
+#pragma unroll
+              for (int ks = 0; ks < 8; ++ks)
+                umma(tmem + u * kUnitCols, smem_desc(ka + (ks >> 2) * kHalf + (ks & 3) * 32, 16, 1024),
+                     smem_desc(qa + (ks >> 2) * (kQUnit / 2) + (ks & 3) * 32, 16, 1024), ID, ks != 0);
+              if (j == subs - 1 && i + 2 < n * p.nkv) umma_commit(k_empty(st));
+              umma_commit(s_full(u));
+            }
+            __syncwarp();
+          }
+        }
+    } else {
+      // ---------------------------------------------------------------- weights and their mixture
+      const int quarter = warp & 3, u0 = (warp >> 2) * 2, key = quarter * 32 + lane;
+      const int hb = warp >> 3, kb = (warp & 7) * 16;
+      const bool mixes = hb * 16 < p.nq;
+      uint64_t k[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) k[i] = pack2(p.cap.k[i], p.cap.k[i]);
+      if (!(p.cap.out > 0.f)) k[0] = pack2(p.scale_log2, p.scale_log2);
+      // T: A operand, columns: unit by unit four leading terms, four remainders
+      uint32_t ta[KS][4];
+#pragma unroll
+      for (int ks = 0; ks < KS; ++ks)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int h = hb * 16 + (lane >> 2) + (i & 1) * 8, u = (lane & 1) * 2, un = ks * 2 + (i >> 1), first = un % subs * 4 + u;
+          const bf16 zero = __float2bfloat16(0.f);
+          const auto at = [&](int e) { return h < p.nq && un < units && first + e < p.group ? p.talk[h * p.nq + head_of(un) + u + e] : zero; };
+          const bf162 v = __halves2bfloat162(at(0), at(1));
+          ta[ks][i] = *reinterpret_cast<const uint32_t*>(&v);
+        }
+      uint32_t chunk[2];
+#pragma unroll
+      for (int j = 0; j < 2; ++j) chunk[j] = lines + key * kLine + (((u0 + j) ^ spread(key & 15)) << 4);
+      const int mi = lane >> 3, mkey = 4 * ((lane & 7) >> 1) + (lane & 1) + (mi >> 1) * 2;
+      const uint32_t line = lines + (kb + mkey) * kLine + (((mi & 1) ^ spread(mkey)) << 4);
+      const uint32_t nl_at = sbase + kNlOff + u0 * 16;
+      const uint32_t taddr = tmem + ((uint32_t)(quarter * 32) << 16) + u0 * kUnitCols;
+      // place of (head hb 16 + lane / 4, row 0, key kb + 4 (lane % 4)) in the table
+      const uint32_t place = (uint32_t)(((int64_t)(hb * 16 + (lane >> 2)) * p.w_rows + r0 - p.row0) * p.ld + k0 + kb + 4 * (lane & 3));
+      const uint32_t heads8 = (uint32_t)(8 * p.w_rows * p.ld), ld = (uint32_t)p.ld;
+      const bool h0 = hb * 16 + (lane >> 2) < p.nq, h1 = hb * 16 + 8 + (lane >> 2) < p.nq;
+      const int rows = min(kBM, q_hi - r0);
+      bool ok = true;
+
+      const auto mix = [&](int t, int r) {            // row r of tile t
+        if (!mixes) return;
+        float d[2][4];
+#pragma unroll
+        for (int ks = 0; ks < KS; ++ks) {
+          uint32_t b0, b1, b2, b3;
+          ldmatrix_x4(b0, b1, b2, b3, (line + (r & 1) * kLines) ^ (ks << 5));
+          if (ks == 0) {
+            mma_bf16_16816_first(d[0], ta[0], b0, b1);
+            mma_bf16_16816_first(d[1], ta[0], b2, b3);
+          } else {
+            mma_bf16_16816(d[0], ta[ks], b0, b1);
+            mma_bf16_16816(d[1], ta[ks], b2, b3);
+          }
+        }
+        if (r >= rows) return;
+        const uint32_t at = place + r * ld + t * kBN;
+        if (h0) *reinterpret_cast<uint2*>(p.w + at) = make_uint2(pack_bf162(d[0][0], d[0][1]), pack_bf162(d[1][0], d[1][1]));
+        if (h1) *reinterpret_cast<uint2*>(p.w + at + heads8) = make_uint2(pack_bf162(d[0][2], d[0][3]), pack_bf162(d[1][2], d[1][3]));
+      };
+      for (int t = 0; t < n; ++t) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+          if (u0 + j < units) ok = ok && mbar_wait_warp(s_full(u0 + j), t & 1, abort_flag);
+        tc_fence_after();
+        const int late = k0 + t * kBN + key - pos0;   // rows before it do not see the key
+        const bool edge = k0 + t * kBN + kBN - 1 > pos0;
+#pragma unroll 1
+        for (int q = 0; q < kBM / 4; ++q) {           // four rows from tensor memory at a time
+          uint32_t x[2][16];
+          float top = 0.f;
+#pragma unroll
+          for (int j = 0; j < 2; ++j)
+            if (u0 + j < units) tmem_ld16(taddr + j * kUnitCols + q * 16, x[j]);
+          tmem_ld_wait();
+          if (q == kBM / 4 - 1) {                     // the next tile's products may overwrite the scores
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) {
+#pragma unroll
+              for (int j = 0; j < 2; ++j)
+                if (u0 + j < units) mbar_arrive(s_free(u0 + j));
+            }
+          }
+          if (p.cap.out > 0.f) {
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+              if (u0 + j < units) {
+#pragma unroll
+                for (int i = 0; i < 16; ++i) top = fmaxf(top, fabsf(__uint_as_float(x[j][i])));
+              }
+          }
+          const int kind = p.cap.out > 0.f ? (__all_sync(0xffffffffu, top <= p.cap.small) ? 1 : 2) : 0;
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int r = q * 4 + e;
+            const bool hidden = edge && late > r;
+            // the row before: its lines are complete since the last barrier
+            if (r > 0) mix(t, r - 1);
+            else if (t > 0) mix(t - 1, kBM - 1);
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+              if (u0 + j >= units) continue;
+              const uint32_t at = chunk[j] + (e & 1) * kLines, from = nl_at + (r * kUnits + j) * 16;
+              if (kind == 1) chunk_out<1>(at, x[j] + e * 4, from, k, p.cap, hidden);
+              else if (kind == 2) chunk_out<2>(at, x[j] + e * 4, from, k, p.cap, hidden);
+              else chunk_out<0>(at, x[j] + e * 4, from, k, p.cap, hidden);
+            }
+            asm volatile("bar.sync 1, 512;" ::: "memory");
+          }
+        }
+      }
+      mix(n - 1, kBM - 1);
+    }
+    tc_fence_before();
+    __syncthreads();
+    if (threadIdx.x == 0 && *abort_flag && p.err != nullptr) atomicExch(p.err, 1);
+    if (warp == kWorkers + 1) {
+      tc_fence_after();
+      asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512));
+    }
+  }
   // keys that no row of the tile sees
-  const int z0 = k0 + steps * 16, per = (k_end - z0) / 8;
-  for (int i = threadIdx.x; per > 0 && i < p.nq * kBM * per; i += 256) {
+  const int z0 = k0 + n * kBN, per = (k_end - z0) / 8;
+  for (int i = threadIdx.x; per > 0 && i < p.nq * kBM * per; i += kThreads) {
     const int c = i % per, r = i / per % kBM, h = i / (per * kBM);
     if (r0 + r < q_hi)
       *reinterpret_cast<uint4*>(p.w + ((int64_t)h * p.w_rows + r0 + r - p.row0) * p.ld + z0 + c * 8) = make_uint4(0, 0, 0, 0);
@@ -580,35 +734,54 @@ XLLM_API int xllm_talk_decode(void* out, const void* q, const void* k_cache, con
 
 // Mixed weights of the rows [row0, row0 + rows) of all sequences to w [nq, w_rows, ld] bf16 (see xllm_talk_values_tc), from q
 // [total_q, nq, 128], the K cache and lse [total_q, nq] (xllm_prefill_lse_tc).  ld a multiple of 128 no less than the longest sequence;
-// page % 16 == 0; no more than eight units of four heads of one key/value head.
-XLLM_API int xllm_talk_weights(void* w, int64_t w_rows, int64_t ld, const void* q, const void* k_cache, const void* talk_w, const void* lse,
+// page 16, 32, 64 or 128; no more than eight units of four heads of one key/value head, nor 32 heads.
+XLLM_API int xllm_talk_weights(void* w, int64_t w_rows, int64_t ld, const void* q, int64_t total_q, const void* k_cache, int64_t n_blocks,
+                               const void* talk_w, const void* lse,
                                const void* block_table, int bt_stride, const void* cu_q, const void* kv_lens, int batch, int max_q_len,
                                int row0, int rows, int nq, int nkv, int page, float scale, float softcap, int keys, void* stream) {
   using namespace xllm;
   using namespace xllm::talk;
   if (batch == 0 || rows == 0 || max_q_len == 0) return 0;
-  if (nq <= 0 || nkv <= 0 || nq % nkv || page <= 0 || page % 16 || ld <= 0 || ld % 128 || w_rows < rows || keys <= 0 || keys % 128 ||
+  if (nq <= 0 || nkv <= 0 || nq % nkv || nq > 32 || page < 16 || page > 128 || (page & (page - 1)) || ld <= 0 || ld % 128 || w_rows < rows || keys <= 0 || keys % 128 ||
+      (int64_t)nq * w_rows * ld >= (1LL << 32) ||
       (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)w) & 15))
     return (int)cudaErrorInvalidValue;
   const int units = nkv * ((nq / nkv + 3) / 4);
   if (units > kUnits) return (int)cudaErrorInvalidValue;
-  WeightsParams p;
+  WeightsParams p{};
   p.q = (const bf16*)q; p.k_cache = (const bf16*)k_cache; p.talk = (const bf16*)talk_w; p.lse = (const float*)lse; p.w = (bf16*)w;
   p.block_table = (const int32_t*)block_table; p.cu_q = (const int32_t*)cu_q; p.kv_lens = (const int32_t*)kv_lens; p.w_rows = w_rows;
-  p.ld = ld; p.bt_stride = bt_stride; p.nq = nq; p.nkv = nkv; p.group = nq / nkv; p.page = page; p.row0 = row0; p.rows = rows;
+  p.ld = ld; p.bt_stride = bt_stride; p.nq = nq; p.nkv = nkv; p.group = nq / nkv; p.row0 = row0; p.rows = rows;
+  while ((16 << p.page_log2) < page) ++p.page_log2;
+  p.page_log2 += 4;
   p.keys = keys; p.cap = make_soft_cap(scale, softcap); p.scale_log2 = scale * kLog2e;
   const dim3 grid((unsigned)((min(max_q_len, rows) + kBM - 1) / kBM), (unsigned)((ld + keys - 1) / keys), batch);
-  const size_t smem = (size_t)kKStages * nkv * kTileBytes + 2 * kPairBytes;
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (g_err[dev & 63] == nullptr) {
+    if (cudaMalloc(&g_err[dev & 63], sizeof(int)) != cudaSuccess) return (int)cudaErrorMemoryAllocation;
+    cudaMemset(g_err[dev & 63], 0, sizeof(int));
+  }
+  p.err = g_err[dev & 63];
+  CUtensorMap tq, tk;
+  if (!tc::make_map_heads(&tq, q, total_q, nq, kBM, 4) || !tc::make_map(&tk, k_cache, n_blocks * nkv * page, D, D, page))
+    return (int)cudaErrorInvalidValue;
   const auto run = [&](auto kernel) {
-    const int e = prepare(kernel, smem);
+    const int e = prepare(kernel, kWeightsSmem);
     if (e != 0) return e;
-    launch_pdl(kernel, grid, dim3(256), smem, (cudaStream_t)stream, p);
+    kernel<<<grid, kThreads, kWeightsSmem, (cudaStream_t)stream>>>(tq, tk, p);
     return XLLM_LAUNCH_CHECK();
   };
-  if (nq <= 16) {
-    if (units <= 2) return run(talk_weights_kernel<1, 1>);
-    if (units <= 4) return run(talk_weights_kernel<1, 2>);
-    return run(talk_weights_kernel<1, 4>);
-  }
-  return run(talk_weights_kernel<2, 4>);
+  return units <= 2 ? run(talk_weights_kernel<1>) : (units <= 4 ? run(talk_weights_kernel<2>) : run(talk_weights_kernel<4>));
+}
+
+// 0 = no bounded wait expired in the prompt kernel on this device since the last call.
+XLLM_API int xllm_talk_error_status() {
+  int dev = 0, v = 0;
+  cudaGetDevice(&dev);
+  int* e = xllm::talk::g_err[dev & 63];
+  if (e == nullptr) return 0;
+  cudaMemcpy(&v, e, sizeof(int), cudaMemcpyDeviceToHost);
+  if (v != 0) cudaMemset(e, 0, sizeof(int));
+  return v;
 }

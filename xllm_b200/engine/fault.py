@@ -101,7 +101,10 @@ class DeviceWatchdog:
         if engine.device.type == "cuda":
             from ..ops import _lib, gemm_tcgen05
             src["gemm"] = gemm_tcgen05.error_status
+            from ..ops import talking  # noqa: F401  (declares its kernels)
             src["attention"] = lambda: int(_lib.load().xllm_fmha_error_status())
+            if hasattr(_lib.load(), "xllm_talk_error_status"):          # a library of one model's kernels may be without it
+                src["mixed-head attention"] = lambda: int(_lib.load().xllm_talk_error_status())
         comm = getattr(engine.ps, "comm", None)
         if comm is not None:
             src["tp_comm"] = comm.error_status

@@ -11,13 +11,14 @@ _lib.register_signature("xllm_conv_row_norm_kv", [P, P, P, L, P, P, P, P] + [I] 
 _lib.register_signature("xllm_talk_decode", [P, P, P, P, P, P, I, P, I, I, I, I, I, F, F, L, I, I, P, P])
 _lib.register_signature("xllm_talk_decode_workspace", [L, I, L, I, I], L)
 _lib.register_signature("xllm_prefill_lse_tc", [P, P, L, L, P, L, P, I, P, P, I, I, I, I, I, F, F, P])
-_lib.register_signature("xllm_talk_weights", [P, L, L, P, P, P, P, P, I, P, P, I, I, I, I, I, I, I, F, F, I, P])
+_lib.register_signature("xllm_talk_weights", [P, L, L, P, L, P, L, P, P, P, I, P, P, I, I, I, I, I, I, I, F, F, I, P])
+_lib.register_signature("xllm_talk_error_status", [])
 _lib.register_signature("xllm_talk_values_tc", [P, I, P, L, L, P, L, P, I, P, P, I, I, I, I, I, I, I, P])
 _lib.register_signature("xllm_talk_attn_generic", [P, P, P, P, P, P, L, P, I, P, P] + [I] * 9 + [F, F, I, P])
 
 _DT = {torch.bfloat16: 0, torch.float32: 1}
 
-WORKSPACE_BYTES = 256 << 20          # of a chunk of rows
+WORKSPACE_BYTES = 1 << 30              # of a chunk of rows
 TC_HEAD = 128                        # head size of the tensor-core kernels' caches
 
 
@@ -141,11 +142,13 @@ def prefill(q, k_cache, v_cache, block_table, cu_q, kv_lens, max_q_len, scale, s
     check(lib.xllm_prefill_lse_tc(ptr(lse), ptr(q), q.stride(0), T, ptr(k_cache), blocks, ptr(block_table), block_table.stride(0), ptr(cu_q),
                                   ptr(kv_lens), B, int(max_q_len), nq, nkv, page, float(scale), float(softcap or 0.0), s), "prefill_lse_tc")
     per = max(128, min(T - row0, WORKSPACE_BYTES // (nq * ld * 2) // 128 * 128))
-    keys = min(ld, 512 if per * ld >= 1 << 21 else 128)
+    # a block takes 16 rows and a range of keys: a few blocks per SM, the long rows first
+    tiles = -(-min(per, T - row0) // 16)
+    keys = max(128, -(-ld // max(1, 600 // tiles)) // 128 * 128)
     w = torch.empty(nq * per * ld, dtype=torch.bfloat16, device=q.device)
     for r in range(row0, T, per):
         n = min(per, T - r)
-        check(lib.xllm_talk_weights(ptr(w), per, ld, ptr(q), ptr(k_cache), ptr(talk), ptr(lse), ptr(block_table), block_table.stride(0),
+        check(lib.xllm_talk_weights(ptr(w), per, ld, ptr(q), T, ptr(k_cache), blocks, ptr(talk), ptr(lse), ptr(block_table), block_table.stride(0),
                                     ptr(cu_q), ptr(kv_lens), B, int(max_q_len), r, n, nq, nkv, page, float(scale), float(softcap or 0.0),
                                     keys, s), "talk_weights")
         check(lib.xllm_talk_values_tc(ptr(out), dv, ptr(w), per, ld, ptr(v_cache), blocks, ptr(block_table), block_table.stride(0), ptr(cu_q),
