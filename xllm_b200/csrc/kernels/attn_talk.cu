@@ -406,8 +406,8 @@ __device__ __forceinline__ void weigh(const uint32_t* x, uint64_t nl, const uint
   f1 = exp2f(f1);
 }
 
-// The chunk of one unit's four heads: leading terms cut off, remainders rounded.
-template <int CAP>
+// The chunk of one unit's four heads: the weights rounded to bf16, and what that left.
+template <int CAP, bool EDGE>
 __device__ __forceinline__ void chunk_out(uint32_t at, const uint32_t* x, uint32_t nl_at, const uint64_t (&k)[4], const SoftCap& cap,
                                           bool hidden) {
   uint64_t nl[2];
@@ -417,11 +417,12 @@ __device__ __forceinline__ void chunk_out(uint32_t at, const uint32_t* x, uint32
   for (int i = 0; i < 2; ++i) {
     float f0, f1, r0, r1;
     weigh<CAP>(x + 2 * i, nl[i], k, cap, f0, f1);
-    if (hidden) f0 = f1 = 0.f;
-    const uint32_t u0 = __float_as_uint(f0), u1 = __float_as_uint(f1);
-    asm("prmt.b32 %0, %1, %2, 0x7632;" : "=r"(hi[i]) : "r"(u0), "r"(u1));
-    unpack2f(fma2(pack2(__uint_as_float(u0 & 0xffff0000u), __uint_as_float(u1 & 0xffff0000u)), pack2(-1.f, -1.f), pack2(f0, f1)), r0, r1);
-    lo[i] = pack_bf162(r0, r1);
+    if (EDGE && hidden) f0 = f1 = 0.f;
+    hi[i] = pack_bf162(f0, f1);
+    asm("{.reg .b16 a, b; mov.b32 {a, b}, %2; sub.rn.f32.bf16 %0, a, %3; sub.rn.f32.bf16 %1, b, %4;}"
+        : "=f"(r0), "=f"(r1)
+        : "r"(hi[i]), "f"(f0), "f"(f1));
+    lo[i] = pack_bf162(-r0, -r1);
   }
   asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(at), "r"(hi[0]), "r"(hi[1]), "r"(lo[0]), "r"(lo[1]) : "memory");
 }
@@ -578,7 +579,9 @@ talk_weights_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_cons
 #pragma unroll
       for (int j = 0; j < 2; ++j) chunk[j] = lines + key * kLine + (((u0 + j) ^ spread(key & 15)) << 4);
       const int mi = lane >> 3, mkey = 4 * ((lane & 7) >> 1) + (lane & 1) + (mi >> 1) * 2;
-      const uint32_t line = lines + (kb + mkey) * kLine + (((mi & 1) ^ spread(mkey)) << 4);
+      uint32_t line[KS];                              // of row 0, by tile of T's columns
+#pragma unroll
+      for (int ks = 0; ks < KS; ++ks) line[ks] = lines + (kb + mkey) * kLine + (((ks * 2 + (mi & 1)) ^ spread(mkey)) << 4);
       const uint32_t nl_at = sbase + kNlOff + u0 * 16;
       const uint32_t taddr = tmem + ((uint32_t)(quarter * 32) << 16) + u0 * kUnitCols;
       // place of (head hb 16 + lane / 4, row 0, key kb + 4 (lane % 4)) in the table
@@ -594,7 +597,7 @@ talk_weights_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_cons
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks) {
           uint32_t b0, b1, b2, b3;
-          ldmatrix_x4(b0, b1, b2, b3, (line + (r & 1) * kLines) ^ (ks << 5));
+          ldmatrix_x4(b0, b1, b2, b3, line[ks] + (r & 1) * kLines);
           if (ks == 0) {
             mma_bf16_16816_first(d[0], ta[0], b0, b1);
             mma_bf16_16816_first(d[1], ta[0], b2, b3);
@@ -637,27 +640,32 @@ talk_weights_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_cons
             for (int j = 0; j < 2; ++j)
               if (u0 + j < units) {
 #pragma unroll
-                for (int i = 0; i < 16; ++i) top = fmaxf(top, fabsf(__uint_as_float(x[j][i])));
+                for (int i = 0; i < 16; i += 2)
+                  asm("{.reg .f32 a, b; abs.f32 a, %1; abs.f32 b, %2; max.f32 %0, %0, a, b;}"
+                      : "+f"(top)
+                      : "f"(__uint_as_float(x[j][i])), "f"(__uint_as_float(x[j][i + 1])));
               }
           }
-          const int kind = p.cap.out > 0.f ? (__all_sync(0xffffffffu, top <= p.cap.small) ? 1 : 2) : 0;
+          const auto four_rows = [&](auto cap, auto edge) {
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int r = q * 4 + e;
-            const bool hidden = edge && late > r;
-            // the row before: its lines are complete since the last barrier
-            if (r > 0) mix(t, r - 1);
-            else if (t > 0) mix(t - 1, kBM - 1);
+            for (int e = 0; e < 4; ++e) {
+              const int r = q * 4 + e;
+              // the row before: its lines are complete since the last barrier
+              if (r > 0) mix(t, r - 1);
+              else if (t > 0) mix(t - 1, kBM - 1);
 #pragma unroll
-            for (int j = 0; j < 2; ++j) {
-              if (u0 + j >= units) continue;
-              const uint32_t at = chunk[j] + (e & 1) * kLines, from = nl_at + (r * kUnits + j) * 16;
-              if (kind == 1) chunk_out<1>(at, x[j] + e * 4, from, k, p.cap, hidden);
-              else if (kind == 2) chunk_out<2>(at, x[j] + e * 4, from, k, p.cap, hidden);
-              else chunk_out<0>(at, x[j] + e * 4, from, k, p.cap, hidden);
+              for (int j = 0; j < 2; ++j)
+                if (u0 + j < units)
+                  chunk_out<decltype(cap)::value, decltype(edge)::value>(chunk[j] + (e & 1) * kLines, x[j] + e * 4,
+                                                                         nl_at + (r * kUnits + j) * 16, k, p.cap, late > r);
+              asm volatile("bar.sync 1, 512;" ::: "memory");
             }
-            asm volatile("bar.sync 1, 512;" ::: "memory");
-          }
+          };
+          using std::integral_constant;
+          if (!(p.cap.out > 0.f)) four_rows(integral_constant<int, 0>(), std::true_type());
+          else if (!__all_sync(0xffffffffu, top <= p.cap.small)) four_rows(integral_constant<int, 2>(), std::true_type());
+          else if (edge) four_rows(integral_constant<int, 1>(), std::true_type());
+          else four_rows(integral_constant<int, 1>(), std::false_type());
         }
       }
       mix(n - 1, kBM - 1);
