@@ -93,17 +93,15 @@ def vivazen_args(W):
 
 
 def lukinex_dense_args(W):
-    """Convolved, capped attention and latent attention in turn, without the recurrent branches' share of the layers; one expert and a
-    shared one, together as wide as a dense feed-forward."""
-    a = lukinex_args(W)
-    H, layers = W // 128, []
+    """Windowed attention and latent attention in turn; one expert and a shared one, together as wide as a dense feed-forward."""
+    from xllm_b200.models import model_args_from_dict
+    a, layers = lukinex_args(W), []
     moe = {"kind": "moe", "expert": {"ff": 3 * W // 2, "limit": 7.0}, "router": {"experts": 1, "top": 1},
            "shared": {"ff": 3 * W // 2, "limit": 7.0}}
     att = {**next(l["mixer"] for l in a.extra["layers"] if l["type"] == "attention")}
     lat = {**next(l["mixer"] for l in a.extra["layers"] if l["type"] == "latent_attention"), "q_rank": W}
     for i in range(LAYERS):
         layers.append({"type": ("attention", "latent_attention")[i % 2], "mixer": dict((att, lat)[i % 2]), "mlp": moe})
-    from xllm_b200.models import model_args_from_dict
     return model_args_from_dict({"architecture": "Lukinex", "vocab": VOCAB, "width": W, "norm": {"eps": 1e-6}, "layers": layers})
 
 

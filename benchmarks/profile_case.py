@@ -231,6 +231,17 @@ def main():
             mst = {"S": st, "n": torch.zeros(S + 1, H, d, device=dev), "m": torch.zeros(S + 1, H, device=dev)}
             run = op.decode if L == 1 else op.prefill
             fn = lambda: run(mst, sl, cu, kl, *c[:3], z[:, :H], z[:, H:], c[3], out)
+    elif a.kernel == "talking":                     # prompts of attention with mixed heads: row sums, mixed weights, values
+        from xllm_b200.ops import talking
+        S, L, H, G, d = 4, 1024, 32, 8, 128
+        T = S * L
+        rnd = lambda *s: torch.randn(*s, device=dev, dtype=torch.bfloat16)
+        i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+        kc, vc = rnd(T // 16, G, 16, d), rnd(T // 16, G, 16, d)
+        bt = torch.arange(T // 16, device=dev, dtype=torch.int32).view(S, L // 16)
+        cu, kl, q = i32([i * L for i in range(S + 1)]), i32([L] * S), rnd(T, H, d)
+        talk, out = torch.eye(H, device=dev, dtype=torch.bfloat16) + rnd(H, H) * 0.1, torch.empty_like(q)
+        fn = lambda: talking.prefill(q, kc, vc, bt, cu, kl, L, d ** -0.5, 30.0, talk, d, out, L, 0)
     else:
         raise SystemExit(f"unknown kernel {a.kernel}")
     for _ in range(a.iters):

@@ -27,7 +27,9 @@ from .state import RecurrentStatePool
 
 def _yarn(rot, args, device):
     """Neighbouring elements turn together; low frequencies are divided by the factor, and cos and sin grow with its logarithm."""
-    s = rot["scaling"]
+    s = rot.get("scaling")
+    if s is None:
+        return RotaryEmbedding(int(rot["dims"]), args.max_position_embeddings, float(rot["base"]), None, device, interleaved=True)
     return RotaryEmbedding(int(rot["dims"]), args.max_position_embeddings, float(rot["base"]),
                            {"rope_type": "yarn", "factor": float(s["factor"]), "original_max_position_embeddings": s["original"],
                             "beta_fast": s["fast"], "beta_slow": s["slow"],
