@@ -219,7 +219,7 @@ def latent_decode(q, cache, block_table, scale, seq_lens=None, positions=None, b
         from . import decode_splits
         splits = decode_splits(N, 1, nh)
         if window:
-            splits = min(splits, max(1, window // 128))
+            splits = min(splits, max(1, window // 256))
     ws = torch.empty(N * nh * splits * (dv + 1), dtype=torch.float32, device=q.device) if splits > 1 else None
     check(_lib.load().xllm_latent_decode(ptr(out), ptr(q), q.stride(0), ptr(cache), width, ptr(block_table),
                                          block_table.stride(0), ptr(seq_lens), ptr(positions), ptr(bt_rows), N, nh,
