@@ -229,6 +229,33 @@ def test_talking_attention_in_chunks_of_rows(monkeypatch):
         near(out, want, GPU16)
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("heads,kv,d,dv", [(32, 8, 128, 128), (20, 1, 128, 72), (12, 4, 64, 40), (7, 7, 128, 96), (2, 1, 32, 128)])
+def test_talking_decode_in_splits(heads, kv, d, dv):
+    """Any cut of the context for the scores and for the values, empty shares included."""
+    lens = [1290, 1, 64, 65, 700, 128]
+    b, q, kc, vc, t, scale, want = talk_case(lens, [1] * 6, heads, kv, d, dv, GPU16, 20.0)
+    for splits, vsplits in ((None, None), (1, 1), (3, 1), (1, 5), (9, 16), (16, 30)):
+        out = torch.zeros(6, heads, dv, dtype=torch.bfloat16, device="cuda")
+        talking.decode(q, kc, vc, b.block_table, b.kv_lens, scale, 20.0, t, dv, out, max(lens), splits=splits, vsplits=vsplits)
+        near(out, want, GPU16)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("heads,kv,d,dv", [(32, 8, 128, 128), (12, 4, 64, 40), (5, 5, 128, 96), (3, 1, 32, 128)])
+@pytest.mark.parametrize("cap,spread", [(30.0, 1.0), (6.0, 4.0), (300.0, 2.0), (0.0, 1.0)])
+def test_talking_prompts_of_many_key_tiles(heads, kv, d, dv, cap, spread):
+    """Blocks that walk over several tiles of keys; scores within the polynomial's reach, beyond it, under a cap too high for sums
+    without a reference, and without a cap; portions behind long contexts."""
+    lens, new = [700, 1290, 513], [700, 90, 17]
+    b, q, kc, vc, t, scale, want = talk_case(lens, new, heads, kv, d, dv, GPU16, cap or 1e6, spread=spread)
+    for keys in (128, 384, 1408):
+        out = torch.zeros(b.cu[-1], heads, dv, dtype=torch.bfloat16, device="cuda")
+        talking.prefill(q, kc, vc, b.block_table, b.cu_q, b.kv_lens, max(new), scale, cap, t, dv, out, max(lens), 0, keys=keys)
+        near(out, want, GPU16)
+    assert ops._lib.load().xllm_talk_error_status() == 0 and ops._lib.load().xllm_fmha_error_status() == 0
+
+
 # ------------------------------------------------------------------------------------------- latent attention
 ROTS = [dict(base=10000.0, dims=16, scaling=dict(factor=3.0, original=64, fast=8.0, slow=0.5)),
         dict(base=500.0, dims=32, scaling=dict(factor=1.0, original=2048, fast=32.0, slow=1.0)),

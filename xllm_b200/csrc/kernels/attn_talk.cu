@@ -337,8 +337,6 @@ __global__ void __launch_bounds__(128) talk_merge_kernel(bf16* __restrict__ out,
 
 // ------------------------------------------------------------------------------------------------ prompts
 struct WeightsParams {
-  const bf16* q;              // [total_q, nq, 128]
-  const bf16* k_cache;
   const bf16* talk;
   const float* lse;           // [total_q, nq], log2 domain
   bf16* w;                    // [nq, w_rows, ld]
@@ -757,7 +755,7 @@ XLLM_API int xllm_talk_weights(void* w, int64_t w_rows, int64_t ld, const void* 
   const int units = nkv * ((nq / nkv + 3) / 4);
   if (units > kUnits) return (int)cudaErrorInvalidValue;
   WeightsParams p{};
-  p.q = (const bf16*)q; p.k_cache = (const bf16*)k_cache; p.talk = (const bf16*)talk_w; p.lse = (const float*)lse; p.w = (bf16*)w;
+  p.talk = (const bf16*)talk_w; p.lse = (const float*)lse; p.w = (bf16*)w;
   p.block_table = (const int32_t*)block_table; p.cu_q = (const int32_t*)cu_q; p.kv_lens = (const int32_t*)kv_lens; p.w_rows = w_rows;
   p.ld = ld; p.bt_stride = bt_stride; p.nq = nq; p.nkv = nkv; p.group = nq / nkv; p.row0 = row0; p.rows = rows;
   while ((16 << p.page_log2) < page) ++p.page_log2;

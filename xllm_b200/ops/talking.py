@@ -127,9 +127,10 @@ def decode(q, k_cache, v_cache, block_table, seq_lens, scale, softcap, talk, dv,
     return out
 
 
-def prefill(q, k_cache, v_cache, block_table, cu_q, kv_lens, max_q_len, scale, softcap, talk, dv, out, longest, row0):
+def prefill(q, k_cache, v_cache, block_table, cu_q, kv_lens, max_q_len, scale, softcap, talk, dv, out, longest, row0,
+            keys=None):
     """Prompt rows [row0, T) of q [T, heads, 128] -> the same rows of out [T, heads, dv]; cu_q holds row numbers of q.  The softmax's
-    sums of all rows first, then for a chunk of rows the table of mixed weights and its product with the values."""
+    sums of all rows first, then for a chunk of rows the table of mixed weights and its product with the values.  keys: how many a block of the table takes (a multiple of 128)."""
     from . import _count, _index
     T, nq, _ = q.shape
     B, nkv, page, blocks = kv_lens.shape[0], k_cache.shape[1], k_cache.shape[2], k_cache.shape[0]
@@ -144,7 +145,7 @@ def prefill(q, k_cache, v_cache, block_table, cu_q, kv_lens, max_q_len, scale, s
     per = max(128, min(T - row0, WORKSPACE_BYTES // (nq * ld * 2) // 128 * 128))
     # a block takes 16 rows and a range of keys: a few blocks per SM, the long rows first
     tiles = -(-min(per, T - row0) // 16)
-    keys = max(128, -(-ld // max(1, 600 // tiles)) // 128 * 128)
+    keys = keys or max(128, -(-ld // max(1, 600 // tiles)) // 128 * 128)
     w = torch.empty(nq * per * ld, dtype=torch.bfloat16, device=q.device)
     for r in range(row0, T, per):
         n = min(per, T - r)
